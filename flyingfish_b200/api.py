@@ -7,6 +7,7 @@ calls (``generate_batch``) expose continuous batching.
 """
 from __future__ import annotations
 
+import dataclasses
 import os
 import time
 from dataclasses import dataclass, field
@@ -14,12 +15,19 @@ from pathlib import Path
 
 import torch
 
-from .config import ModelSpec, Settings, named_shape, read_model_spec
+from .config import GPU_FP32_ARCHS, ModelSpec, Settings, named_shape, read_model_spec
 from .engine.engine import Engine, Sequence
 from .models.decoder import DecoderModel
 from .models.weights import TPInfo, random_decoder_weights
 from .planner.plan import plan_engine
 from .utils.log import log_json
+
+
+def with_dtype(spec: ModelSpec, settings: Settings) -> ModelSpec:
+    """The spec with the compute type the settings ask for."""
+    if settings.dtype is None or settings.dtype == spec.dtype:
+        return spec
+    return dataclasses.replace(spec, dtype=settings.dtype)
 
 
 @dataclass
@@ -68,8 +76,16 @@ class Model:
         if preset is None and path.is_dir() and not random_init:
             from .loaders.checkpoint import load_decoder_weights
             from .loaders.tokenizer import load_tokenizer
-            spec = read_model_spec(path)
-            if spec.extra.get("hrm"):
+            spec = with_dtype(read_model_spec(path), settings)
+            if spec.arch == "duponex":
+                from .loaders.checkpoint import audited_source
+                from .models.duponex import build_duponex_weights
+                source, close = audited_source(path, spec, device)
+                try:
+                    weights = build_duponex_weights(spec, source)
+                finally:
+                    close()
+            elif spec.extra.get("hrm"):
                 # looped two-stack decoder: its own weight assembly over the published tensor names (text side only)
                 from .loaders.checkpoint import checkpoint_source
                 from .models.hrm import build_hrm_weights
@@ -84,7 +100,11 @@ class Model:
             name = path.name
         else:
             spec = preset if preset is not None else (read_model_spec(path) if path.is_dir() else named_shape(model))
-            if spec.extra.get("v41"):
+            spec = with_dtype(spec, settings)
+            if spec.arch == "duponex":
+                from .models.duponex import random_duponex_weights
+                weights = random_duponex_weights(spec, seed, device)
+            elif spec.extra.get("v41"):
                 from .models.deepseek_v41 import build_v41_weights
                 from .models.weights import DTYPES, synthetic_source
                 weights = build_v41_weights(spec, seed, device, synthetic_source(spec, seed, device, DTYPES[spec.dtype]),
@@ -114,6 +134,9 @@ class Model:
         elif spec.extra.get("hrm"):
             from .models.hrm import HrmModel
             net = HrmModel(weights, comm=comm)
+        elif spec.arch == "duponex":
+            from .models.duponex import DuponexModel
+            net = DuponexModel(weights, comm=comm)
         elif spec.extra.get("flint"):
             from .models.flint import FlintModel
             net = FlintModel(weights, comm=comm, seed=seed, state=weights.extra.get("state"))
@@ -125,6 +148,8 @@ class Model:
             net = HybridModel(weights, comm=comm, max_sequences=settings.max_batch, seed=seed)
         else:
             net = DecoderModel(weights, comm=comm)
+        if device.type == "cuda" and spec.dtype == "fp32" and spec.arch not in GPU_FP32_ARCHS:
+            raise ValueError(f"{spec.arch} has no 32-bit kernels (BF16 only on a GPU)")
         if ep is not None:
             net.ep = ep
         if device.type == "cuda":

@@ -48,6 +48,9 @@ def _global_parser() -> argparse.ArgumentParser:
     p.add_argument("--dram-gb-s", type=float, default=6550.0)
     p.add_argument("--gemm-tflops", type=float, default=1385.0)
     p.add_argument("--max-batch", type=int, default=64)
+    p.add_argument("--kv-tokens", type=int, default=None, help="tokens the whole KV pool holds (default: what the planner finds room for)")
+    p.add_argument("--dtype", choices=["bf16", "fp32"], default=None,
+                   help="compute type (default: the checkpoint's; fp32 on a GPU only for architectures with 32-bit kernels)")
     p.add_argument("--tp", type=int, default=1, help="tensor-parallel ranks (the command re-launches itself, one process per GPU)")
     p.add_argument("--cpu", action="store_true", help="run on the host (tiny shapes / debugging)")
     p.add_argument("--seed", type=int, default=0)
@@ -191,7 +194,7 @@ def settings_from(args) -> Settings:
                     spec_budget=args.spec_budget if args.draft_model else "chain",
                     spec_graph=args.spec_graph, prefix_cache=args.prefix_cache, kv_format=args.kv_format, kv_recent=args.kv_recent,
                     runtime_dir=args.runtime_dir, dram_gb_s=args.dram_gb_s, gemm_tflops=args.gemm_tflops,
-                    verbose=args.verbose, max_batch=args.max_batch, tp=args.tp)
+                    verbose=args.verbose, max_batch=args.max_batch, tp=args.tp, kv_tokens=args.kv_tokens, dtype=args.dtype)
 
 
 def resolve_mtp_depth(requested: int | None, has_mtp: bool, arch: str) -> int:
@@ -398,10 +401,15 @@ def cmd_bench(args) -> dict:
             eng.free_sequence(s.seq_id)
     med = statistics.median(r["median_ms"] for r in runs)
     ctx = args.prompt_tokens + args.warmup + args.steps // 2
-    kv_bytes = args.batch * ctx * spec.layers * 2 * spec.kv_heads * spec.head_dim * 2
-    moved = spec.decode_weight_bytes() + kv_bytes
     t_, L, h, f = args.prompt_tokens, spec.layers, spec.hidden, spec.ffn
-    flops = 2 * t_ * L * (h * spec.qkv_dim + h * h + 3 * h * f) + 2 * h * spec.vocab + 2 * h * t_ * (t_ + 1) * L
+    if spec.layer_specs is not None:
+        kv_bytes = args.batch * spec.elem_bytes * sum(l.keys_seen(ctx) * l.kv_heads * (l.dim + l.vdim) for l in spec.layer_specs)
+        flops = 2 * t_ * (spec.dense_param_count() - 2 * spec.vocab * h) + 2 * h * spec.vocab + \
+            sum(2 * l.heads * (l.dim + l.vdim) * l.pairs_seen(t_) for l in spec.layer_specs)
+    else:
+        kv_bytes = args.batch * ctx * spec.layers * 2 * spec.kv_heads * spec.head_dim * 2
+        flops = 2 * t_ * L * (h * spec.qkv_dim + h * h + 3 * h * f) + 2 * h * spec.vocab + 2 * h * t_ * (t_ + 1) * L
+    moved = spec.decode_weight_bytes() + kv_bytes
     ptok = statistics.median(prefill_tok_s)
     return {"model": model.name, "batch": args.batch, "steps": args.steps, "warmup": args.warmup, "runs": runs,
             "median_ms": med, "decode_tok_s": args.batch * 1000.0 / med, "graph": eng.use_graph,

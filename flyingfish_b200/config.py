@@ -43,9 +43,51 @@ class MlaSpec:
 
 
 @dataclass
+class LayerSpec:
+    """One layer of a design whose layers need not look alike (``ModelSpec.layer_specs``)."""
+    heads: int
+    kv_heads: int
+    dim: int                          # width of a query / key head
+    vdim: int                         # width of a value head
+    scale: float                      # factor of the attention scores
+    mixer: str = "attention"
+    chunk: int = 0                    # > 0: position i sees only keys of its own block of ``chunk`` positions
+    v_mix: bool = False               # values are mixed with those of the first layer that has the flag
+    ffn: int = 0                      # width of the feed-forward (0: the layer has none)
+    ffn_act: str = "relu2"
+
+    @property
+    def dim_pad(self) -> int:
+        return pad_to(self.dim, 16)
+
+    @property
+    def vdim_pad(self) -> int:
+        return pad_to(self.vdim, 16)
+
+    def keys_seen(self, ctx: int) -> int:
+        """Keys the last of ``ctx`` positions sees."""
+        return (ctx - 1) % self.chunk + 1 if self.chunk else ctx
+
+    def pairs_seen(self, n: int) -> int:
+        """(query, key) pairs of a prompt of ``n`` positions."""
+        if not self.chunk:
+            return n * (n + 1) // 2
+        full, rest = divmod(n, self.chunk)
+        return full * self.chunk * (self.chunk + 1) // 2 + rest * (rest + 1) // 2
+
+
+# architectures whose every operator has a 32-bit kernel on the GPU
+GPU_FP32_ARCHS = ("duponex",)
+
+
+def pad_to(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+@dataclass
 class ModelSpec:
     name: str
-    arch: str                         # llama | qwen3 | qwen3_moe | deepseek_v3 | deepseek_v41 | glm5_next | flint | loop_vl | tiny_moe | qwen3_vl | embedding | diffusion_lm | qwen35_text | gemma
+    arch: str                         # llama | qwen3 | qwen3_moe | deepseek_v3 | deepseek_v41 | glm5_next | flint | loop_vl | tiny_moe | qwen3_vl | embedding | diffusion_lm | qwen35_text | gemma | duponex
     layers: int
     hidden: int
     heads: int
@@ -65,6 +107,7 @@ class ModelSpec:
     moe: MoeSpec | None = None
     mla: MlaSpec | None = None
     mtp_layers: int = 0               # multi-token-prediction heads shipped with the checkpoint
+    layer_specs: list[LayerSpec] | None = None    # per-layer sizes, for designs whose layers differ
     extra: dict[str, Any] = field(default_factory=dict)
 
     @property
@@ -79,13 +122,34 @@ class ModelSpec:
     def qkv_dim(self) -> int:
         return self.q_dim + 2 * self.kv_dim
 
+    @property
+    def elem_bytes(self) -> int:
+        return 4 if self.dtype == "fp32" else 2
+
+    def kv_geometry(self) -> list[tuple[int, int, int]] | None:
+        """(kv heads, key width, value width) of every cache layer where the layers differ, None where one size serves
+        all. Widths are padded to 16 elements, the alignment of the attention kernels' tiles."""
+        if self.layer_specs is None:
+            return None
+        return [(l.kv_heads, l.dim_pad, l.vdim_pad) for l in self.layer_specs]
+
+    def _layer_spec_params(self) -> int:
+        n = 0
+        for l in self.layer_specs:
+            n += self.hidden * (l.heads * (l.dim + 2 * l.vdim) + l.kv_heads * (l.dim + l.vdim)) + 2 * self.hidden * l.ffn
+        return n
+
     def dense_param_count(self) -> int:
+        if self.layer_specs is not None:
+            return self._layer_spec_params() + (1 if self.tie_embeddings else 2) * self.vocab * self.hidden
         per_layer = self.hidden * self.qkv_dim + self.q_dim * self.hidden + 3 * self.hidden * self.ffn + 2 * self.hidden
         return self.layers * per_layer + (1 if self.tie_embeddings else 2) * self.vocab * self.hidden + self.hidden
 
     def decode_weight_bytes(self) -> int:
         """Bytes of weights read by one decode step (embedding row gathers excluded, lm_head
         included) -- the numerator of the reference's decode roofline (src/bench.rs:137-160)."""
+        if self.layer_specs is not None:
+            return self.elem_bytes * (self._layer_spec_params() + self.vocab * self.hidden)
         per_layer = self.hidden * self.qkv_dim + self.q_dim * self.hidden + 3 * self.hidden * self.ffn + 2 * self.hidden
         return 2 * (self.layers * per_layer + self.vocab * self.hidden + self.hidden)
 
@@ -286,6 +350,50 @@ def loopvl_text() -> ModelSpec:
     return _loop_spec("loopvl-text-shape", 1536, 12, 4096, 65536, per_stack=16, h_cycles=2, l_cycles=3, original_max=4096)
 
 
+def _duponex_spec_of(name: str, hidden: int, vocab: int, layers: list[LayerSpec], streams: int, residual_mult: float,
+                     embed_scale: float, eps: float) -> ModelSpec:
+    if not layers:
+        raise ConfigError("a Duponex model needs at least one layer")
+    mixing = [l for l in layers if l.v_mix]
+    if any((l.kv_heads, l.vdim) != (mixing[0].kv_heads, mixing[0].vdim) for l in mixing):
+        raise ConfigError("layers that mix values need the same number and width of value heads")
+    for l in layers:
+        if l.heads % l.kv_heads:
+            raise ConfigError("heads must be a multiple of kv_heads")
+        if min(l.heads, l.kv_heads, l.dim, l.vdim) < 1 or l.chunk < 0 or not l.scale > 0:
+            raise ConfigError(f"unusable mixer sizes {l}")
+    if not 1 <= streams <= 16:
+        raise ConfigError(f"{streams} residual streams (1 to 16 are supported)")
+    wide = max(layers, key=lambda l: l.heads * l.dim)
+    return ModelSpec(
+        name=name, arch="duponex", layers=len(layers), hidden=hidden, heads=wide.heads, kv_heads=wide.kv_heads, head_dim=wide.dim,
+        ffn=max(l.ffn for l in layers), vocab=vocab, rms_eps=eps, layer_specs=layers,
+        extra={"duponex": {"streams": streams, "residual_mult": residual_mult, "embed_scale": embed_scale}})
+
+
+def duponex_tiny() -> ModelSpec:
+    """Small Duponex shape whose layers differ: three residual streams, attention inside blocks of 72 or 40 positions,
+    unequal key and value widths, one layer without value mixing and one without a feed-forward."""
+    layer = dict(heads=4, kv_heads=2, dim=32, vdim=40, scale=0.2, v_mix=True, chunk=72, ffn=192)
+    return _duponex_spec_of("duponex-tiny", 160, 512, [LayerSpec(**layer), LayerSpec(**dict(layer, heads=6, dim=48, chunk=40)),
+                                                       LayerSpec(**dict(layer, v_mix=False, vdim=16, kv_heads=1)),
+                                                       LayerSpec(**dict(layer, ffn=0))],
+                            streams=3, residual_mult=0.5, embed_scale=4.0, eps=1e-5)
+
+
+def duponex_8b() -> ModelSpec:
+    """Duponex layers at the size of an 8-billion-parameter decoder (random weights, for measurements): 4096 wide, 32 / 8
+    heads of 128, blocks of 1024 positions, four residual streams."""
+    layers = [LayerSpec(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, v_mix=True, chunk=1024, ffn=14336) for _ in range(8)]
+    return _duponex_spec_of("duponex-8b-shape", 4096, 128256, layers, streams=4, residual_mult=0.5, embed_scale=8.0, eps=1e-5)
+
+
+def duponex_2b() -> ModelSpec:
+    """As :func:`duponex_8b` at 2048 wide: 16 / 4 heads of 128, blocks of 512 positions."""
+    layers = [LayerSpec(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, v_mix=True, chunk=512, ffn=8192) for _ in range(16)]
+    return _duponex_spec_of("duponex-2b-shape", 2048, 65536, layers, streams=4, residual_mult=0.5, embed_scale=8.0, eps=1e-5)
+
+
 def glm5_next_tiny() -> ModelSpec:
     """Small GLM-5-style shape: the hyper-connection program with every stage collapsing on its own pre-mix, top-k sparse
     attention with the pooled indexer in every layer, sigmoid routing with selection bias."""
@@ -300,6 +408,7 @@ NAMED_SHAPES = {
     "tiny-gemma": tiny_gemma, "qwen3-moe-fp4-tiny": qwen3_moe_fp4_tiny, "tiny-hybrid": tiny_hybrid, "tiny-embed": tiny_embed, "tiny-diffusion": tiny_diffusion, "tiny-vl": tiny_vl, "tiny-minicpm": tiny_minicpm, "tiny-moe": tiny_moe, "tiny-llama": tiny_llama, "llama3-8b-shape": llama3_8b, "llama3-70b-shape": llama3_70b,
     "deepseek-v3-shape": deepseek_v3, "deepseek-v3-tiny": deepseek_v3_tiny, "deepseek-v3-mini": deepseek_v3_mini,
     "deepseek-v3-fp8-mini": deepseek_v3_fp8_mini, "deepseek-v41-tiny": deepseek_v41_tiny, "glm5-next-tiny": glm5_next_tiny, "flint-tiny": flint_tiny,
+    "duponex-tiny": duponex_tiny, "duponex-8b-shape": duponex_8b, "duponex-2b-shape": duponex_2b,
     "loop-tiny": loop_tiny, "loopvl-text-shape": loopvl_text,
     "qwen3-moe-235b-shape": qwen3_moe_235b, "qwen3-moe-tiny": qwen3_moe_tiny,
 }
@@ -408,9 +517,28 @@ def _flint_spec(cfg: dict[str, Any], name: str) -> ModelSpec:
         extra=extra)
 
 
+def _duponex_spec(cfg: dict[str, Any], name: str) -> ModelSpec:
+    """``"architecture": "Duponex"``: a list of layers, each with its own mixer sizes and feed-forward."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+        if entry.get("type") != "attention":
+            raise ConfigError(f"layer {i}: unsupported mixer {entry.get('type')!r}")
+        m, mlp = entry["mixer"], entry.get("mlp")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ConfigError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r}")
+        layers.append(LayerSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                                scale=float(m["scale"]), chunk=int((m.get("mask") or {}).get("size", 0)),
+                                v_mix=bool(m.get("v_mix", False)), ffn=int(mlp["ff"]) if mlp is not None else 0))
+    return _duponex_spec_of(name, int(cfg["width"]), int(cfg["vocab"]), layers, streams=int(cfg["streams"]),
+                            residual_mult=float(cfg["residual_mult"]), embed_scale=float(cfg["embedding"]["scale"]),
+                            eps=float(cfg["norm"]["eps"]))
+
+
 def spec_from_hf_config(cfg: dict[str, Any], name: str = "model") -> ModelSpec:
     """Normalise a Hugging Face ``config.json``. Hard checks mirror the reference's: SiLU
     activation only, 16-bit or 32-bit floats, no unsupported rope scaling for plain Llama."""
+    if cfg.get("architecture") == "Duponex":
+        return _duponex_spec(cfg, name)
     archs = cfg.get("architectures") or []
     arch = next((_ARCH_MAP[a] for a in archs if a in _ARCH_MAP), None)
     if arch is None:
@@ -511,6 +639,8 @@ class Settings:
     ep: int = 1
     max_batch: int = 64
     kv_block: int = 64
+    kv_tokens: int | None = None          # tokens the whole KV pool holds (planner-derived when None)
+    dtype: str | None = None              # compute dtype override: bf16 | fp32 (the checkpoint's when None)
     graph: bool = True
 
     def resolved_runtime_dir(self) -> Path:

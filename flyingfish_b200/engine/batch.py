@@ -2,7 +2,8 @@
 
 A forward pass processes ``rows`` token rows that belong to ``batch`` sequences. Prefill chunks
 contribute ``q_len`` consecutive rows per sequence, decode contributes ``nq`` rows per sequence
-(1 for plain decode, k+1 for speculative verification). All per-step metadata lives in ONE int32
+(1 for plain decode, k+1 for speculative verification). A mixed batch holds prompt portions and,
+behind them, ``singles`` sequences with one row each. All per-step metadata lives in ONE int32
 buffer so a step needs a single host-to-device copy from pinned memory; the layout is fixed per
 (batch capacity, row capacity, block-table width), which also makes it a stable input of a CUDA
 graph. The reference's equivalent is the 32-byte ``SequenceMeta`` record and row work layout for
@@ -56,6 +57,7 @@ class ForwardBatch:
         self.rows = 0
         self.nq = 1
         self.is_decode = True
+        self.singles = 0                  # trailing one-row sequences of a batch that is not a decode batch
         self.max_q_len = 1
         self.max_ctx = 0
         self.n_logit_rows = 0
@@ -107,14 +109,14 @@ class ForwardBatch:
 
     # -- host fill -----------------------------------------------------------------------------
     def fill(self, *, ids, positions, slots, q_lens, ctx_lens, block_rows, logit_rows, is_decode: bool, nq: int = 1,
-             tree_mask=None, kv_start=None, group_rows=None, state_slots=None) -> None:
+             tree_mask=None, kv_start=None, group_rows=None, state_slots=None, singles: int = 0) -> None:
         """Write one step's metadata into the pinned host buffer (lists of ints)."""
         L = self.layout
         h = self.host
         rows, batch = len(ids), len(q_lens)
         assert rows <= L.max_rows and batch <= L.max_batch, "batch exceeds the layout capacity"
         assert len(logit_rows) <= L.n_logit
-        self.rows, self.batch, self.nq, self.is_decode = rows, batch, nq, is_decode
+        self.rows, self.batch, self.nq, self.is_decode, self.singles = rows, batch, nq, is_decode, singles
         h[L.ids: L.ids + rows] = torch.as_tensor(ids, dtype=torch.int32)
         h[L.positions: L.positions + rows] = torch.as_tensor(positions, dtype=torch.int32)
         h[L.slots: L.slots + rows] = torch.as_tensor(slots, dtype=torch.int32)

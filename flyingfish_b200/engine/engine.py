@@ -60,6 +60,15 @@ class _Graph:
         self.graph: torch.cuda.CUDAGraph | None = None
         self.batch: ForwardBatch | None = None
         self.out: torch.Tensor | None = None
+        self.logits: torch.Tensor | None = None
+
+
+@dataclass
+class Span:
+    """New tokens of one sequence in a step, and the rows among them whose logits are computed."""
+    seq: Sequence
+    tokens: list[int]
+    want: list[int] = field(default_factory=list)
 
 
 class Engine:
@@ -78,13 +87,14 @@ class Engine:
             # for positions and capacity
             self.kv = PagedKVCache(spec.layers, 1, 8, num_blocks, settings.kv_block, dtype, self.device, v_head_dim=0)
         else:
-            self.kv = PagedKVCache(spec.layers, hkv, spec.head_dim, num_blocks, settings.kv_block, dtype, self.device)
+            self.kv = PagedKVCache(spec.layers, hkv, spec.head_dim, num_blocks, settings.kv_block, dtype, self.device,
+                                   geometry=spec.kv_geometry())
         # 8-bit store behind the block cache: groups that leave the recent window are sealed after every step
         self.max_groups = 0
         if settings.kv_format == "affine8":
             from .kv_compact import CompactKV
             if spec.mla is not None or getattr(model, "state_slot_count", 0) or getattr(model, "owns_token_state", False) \
-                    or spec.head_dim != 128 or settings.kv_block != 64 or spec.extra.get("gemma"):
+                    or spec.layer_specs is not None or spec.head_dim != 128 or settings.kv_block != 64 or spec.extra.get("gemma"):
                 raise ValueError("--kv-format affine8 needs a GQA decoder with 128-wide heads and 64-token blocks")
             self.kv.compact = CompactKV(spec.layers, hkv, spec.head_dim, max(num_blocks // 2, 1), self.device,
                                         recent=settings.kv_recent)
@@ -96,6 +106,8 @@ class Engine:
         # models that encode a prompt bidirectionally need all of it in one chunk: a prompt is never split, it waits
         # for a chunk with room (and is refused when it is longer than a chunk)
         self.whole_prompt = bool(getattr(model, "whole_prompt_prefill", False))
+        # models whose forward takes prompt portions and single decoded tokens in one batch
+        self.mixed_batches = bool(getattr(model, "mixed_batches", False))
         self.prefill_batch = ForwardBatch(BatchLayout(self.max_batch, max(max_prefill_rows, self.max_batch),
                                                       self.max_blocks), self.device)
         self.graphs: dict[tuple[int, int], _Graph] = {}
@@ -209,10 +221,24 @@ class Engine:
         their first generated token is in ``pending`` / ``output``. This is the unit the scheduler interleaves with
         decode steps, so that a long prompt does not stall the sequences that are already generating."""
         self._check()
+        part = self._take(seqs, max_rows, self.max_batch)
+        if not part:
+            return []
+        try:
+            toks = self._prefill_chunk(part)
+        except OutOfBlocks:
+            raise
+        except Exception:
+            self.poisoned = True
+            raise
+        return self._first_tokens(part, toks)
+
+    def _take(self, seqs: list[Sequence], max_rows: int, max_seqs: int) -> list[tuple[Sequence, int]]:
+        """(sequence, prompt rows) of one chunk: in order, as many remaining prompt tokens as fit ``max_rows``."""
         rows_left = min(max_rows, self.max_prefill_rows)
         part: list[tuple[Sequence, int]] = []
         for s in seqs:
-            if rows_left <= 0 or len(part) >= self.max_batch:
+            if rows_left <= 0 or len(part) >= max_seqs:
                 break
             rem = len(s.prompt) - s.prefilled
             if rem <= 0:
@@ -224,15 +250,11 @@ class Engine:
                 break
             part.append((s, take))
             rows_left -= take
-        if not part:
-            return []
-        try:
-            toks = self._prefill_chunk(part)
-        except OutOfBlocks:
-            raise
-        except Exception:
-            self.poisoned = True
-            raise
+        return part
+
+    @staticmethod
+    def _first_tokens(part: list[tuple[Sequence, int]], toks: list[int]) -> list[Sequence]:
+        """Publish the first generated token of the sequences whose prompt a chunk completed."""
         done = []
         for (s, _), t in zip(part, toks):
             if s.prefilled == len(s.prompt):
@@ -248,21 +270,23 @@ class Engine:
         if need > self.kv.alloc.free_blocks:
             raise OutOfBlocks(f"step needs {need} KV blocks, {self.kv.alloc.free_blocks} free")
 
-    def _prefill_chunk(self, part: list[tuple[Sequence, int]]) -> list[int]:
-        self._need_blocks([(s.seq_id, take) for s, take in part])
+    def _fill_spans(self, spans: list[Span], singles: int = 0) -> ForwardBatch:
+        """Pack the spans row-wise into the prefill batch and upload it (reserves their KV rows; commits nothing). With
+        ``singles``, that many spans at the end are one row each and take the decode attention."""
+        self._need_blocks([(sp.seq.seq_id, len(sp.tokens)) for sp in spans])
         fb = self.prefill_batch
         ids, positions, slots, q_lens, ctx_lens, block_rows, logit_rows = [], [], [], [], [], [], []
         row = 0
-        for s, take in part:
-            kvs = self.kv.seqs[s.seq_id]
-            sl = self.kv.reserve(s.seq_id, take)
-            ids += s.prompt[s.prefilled: s.prefilled + take]
+        for sp in spans:
+            kvs, take = self.kv.seqs[sp.seq.seq_id], len(sp.tokens)
+            sl = self.kv.reserve(sp.seq.seq_id, take)
+            ids += sp.tokens
             positions += list(range(kvs.length, kvs.length + take))
             slots += sl
             q_lens.append(take)
             ctx_lens.append(kvs.length + take)
             block_rows.append(list(kvs.blocks))
-            logit_rows.append(row + take - 1)
+            logit_rows += [row + k for k in sp.want]
             row += take
         mult = getattr(self.model.comm, "size", 1) * 128 if getattr(self.model.comm, "fused", False) else 1
         if mult > 1 and row >= mult and (row + mult - 1) // mult * mult <= fb.layout.max_rows:
@@ -270,19 +294,157 @@ class Engine:
             # that belong to no sequence (no KV write, no logits)
             pad = (row + mult - 1) // mult * mult - row
             ids += [0] * pad; positions += [0] * pad; slots += [-1] * pad
+        state_slots = [sp.seq.state_slot for sp in spans]
         fb.fill(ids=ids, positions=positions, slots=slots, q_lens=q_lens, ctx_lens=ctx_lens, block_rows=block_rows,
-                logit_rows=logit_rows, is_decode=False,
-                state_slots=[s.state_slot for s, _ in part] if self.state_slots is not None else None)
+                logit_rows=logit_rows, is_decode=False, state_slots=state_slots if self.state_slots is not None else None,
+                singles=singles)
         fb.upload()
-        fb.state_slots = [s.state_slot for s, _ in part]
-        out = self.model.forward(fb, self.kv, inputs_embeds=self._mm_embeds(part, fb, len(ids)))
+        fb.state_slots = state_slots
+        return fb
+
+    def _prefill_chunk(self, part: list[tuple[Sequence, int]]) -> list[int]:
+        fb = self._fill_spans([Span(s, s.prompt[s.prefilled: s.prefilled + take], [take - 1]) for s, take in part])
+        out = self.model.forward(fb, self.kv, inputs_embeds=self._mm_embeds(part, fb, fb.rows))
         toks = [int(t) for t in out.cpu().tolist()]
         self._after_sync()
         for s, take in part:
             self.kv.commit(s.seq_id, take)
             s.prefilled += take
-        self.stats["prefill_tokens"] += row
+            self.stats["prefill_tokens"] += take
         return toks
+
+    # -- mixed steps ---------------------------------------------------------------------------
+    def _run_mixed(self, spans: list[Span], greedy: bool) -> torch.Tensor | None:
+        """One forward over prompt portions and single tokens together; returns the greedy ids (``greedy``) or the logits
+        of the wanted rows in the order of the spans, or None when no row is wanted. Commits every span."""
+        order = sorted(range(len(spans)), key=lambda i: len(spans[i].tokens) == 1)         # portions first, stable
+        packed = [spans[i] for i in order]
+        fb = self._fill_spans(packed, singles=sum(len(sp.tokens) == 1 for sp in packed))
+        if fb.n_logit_rows:
+            out = self.model.forward(fb, self.kv, return_logits=not greedy)
+            # wanted rows came out in packed order: put them back into the order of the spans
+            first = {}
+            at = 0
+            for i in order:
+                first[i] = at
+                at += len(spans[i].want)
+            back = [first[i] + k for i in range(len(spans)) for k in range(len(spans[i].want))]
+            if back != list(range(at)):
+                out = out[torch.tensor(back, device=out.device)]
+        else:
+            self.model.hidden_states(fb, self.kv)
+            out = None
+        for sp in packed:
+            self.kv.commit(sp.seq.seq_id, len(sp.tokens))
+        return out
+
+    def mixed_step(self, decoding: list[Sequence], prefilling: list[Sequence], max_rows: int) -> tuple[list[int], list[Sequence]]:
+        """One forward that decodes a token of every sequence of ``decoding`` and prefills up to ``max_rows`` prompt rows of
+        ``prefilling``. Returns (decoded tokens, sequences whose prompt was completed), as :meth:`decode` and
+        :meth:`prefill_some` do one after the other."""
+        self._check()
+        if not self.mixed_batches:
+            raise ValueError("this model's forward does not take mixed batches")
+        part = self._take(prefilling, min(max_rows, self.max_prefill_rows - len(decoding)), self.max_batch - len(decoding))
+        if not part:
+            return self.decode(decoding), []
+        if self.fail_next_step:
+            self.fail_next_step = False
+            self.poisoned = True
+            raise RuntimeError("injected step failure")
+        try:
+            self._check_capacity(decoding)
+            spans = [Span(s, [s.pending], [0]) for s in decoding]
+            spans += [Span(s, s.prompt[s.prefilled: s.prefilled + take], [take - 1]) for s, take in part]
+            toks = [int(t) for t in self._run_mixed(spans, greedy=True).cpu().tolist()]
+            self._after_sync()
+        except OutOfBlocks:
+            raise
+        except Exception:
+            self.poisoned = True
+            raise
+        n = len(decoding)
+        for s, t in zip(decoding, toks):
+            s.pending = t
+            s.output.append(t)
+        for s, take in part:
+            s.prefilled += take
+            self.stats["prefill_tokens"] += take
+        self.stats["decode_steps"] += 1
+        self.stats["decode_tokens"] += n
+        self.stats["mixed_steps"] = self.stats.get("mixed_steps", 0) + 1
+        return toks[:n], self._first_tokens(part, toks[n:])
+
+    def feed(self, spans: list[Span]) -> torch.Tensor | None:
+        """Feed given tokens instead of sampled ones: one batch of spans (portions of several sequences beside single
+        tokens), committed; returns the logits of the wanted rows in order, or None. Batches of single tokens replay the
+        captured decode step. Nothing is sampled."""
+        self._check()
+        if not self.mixed_batches:
+            raise ValueError("this model's forward does not take mixed batches")
+        try:
+            for sp in spans:
+                if self.kv.seqs[sp.seq.seq_id].length + len(sp.tokens) > self.settings.capacity:
+                    raise OutOfBlocks(f"sequence {sp.seq.seq_id} exceeds the KV capacity {self.settings.capacity}")
+            self._need_blocks([(sp.seq.seq_id, len(sp.tokens)) for sp in spans])
+            if all(len(sp.tokens) == 1 for sp in spans):
+                for sp in spans:
+                    sp.seq.pending = sp.tokens[0]
+                _, logits, _ = self._launch_decode([sp.seq for sp in spans])
+                for sp in spans:
+                    self.kv.commit(sp.seq.seq_id, 1)
+                rows = [i for i, sp in enumerate(spans) for _ in sp.want]
+                out = logits[torch.tensor(rows, device=logits.device)] if rows else None
+            else:
+                parts, got = self._split_spans(spans), []
+                for group in parts:
+                    r = self._run_mixed(group, greedy=False)
+                    if r is not None:
+                        got.append(r)
+                out = None if not got else (got[0] if len(got) == 1 else torch.cat(got))
+                if len(parts) > 1 and out is not None:
+                    out = out[torch.tensor(self._span_order(spans, parts), device=out.device)]
+            if self.device.type == "cuda":
+                torch.cuda.synchronize(self.device)
+            self._after_sync()
+            for sp in spans:
+                sp.seq.prefilled = max(sp.seq.prefilled, min(self.kv.seqs[sp.seq.seq_id].length, len(sp.seq.prompt)))
+            return out
+        except OutOfBlocks:
+            raise
+        except Exception:
+            self.poisoned = True
+            raise
+
+    def _split_spans(self, spans: list[Span]) -> list[list[Span]]:
+        """The spans cut into groups of at most ``max_prefill_rows`` rows (a batch larger than a forward)."""
+        groups: list[list[Span]] = [[]]
+        left = self.max_prefill_rows
+        for sp in spans:
+            at = 0
+            while at < len(sp.tokens):
+                if left == 0 or len(groups[-1]) >= self.max_batch:
+                    groups.append([])
+                    left = self.max_prefill_rows
+                n = min(left, len(sp.tokens) - at)
+                groups[-1].append(Span(sp.seq, sp.tokens[at: at + n], [k - at for k in sp.want if at <= k < at + n]))
+                at, left = at + n, left - n
+        return groups
+
+    @staticmethod
+    def _span_order(spans: list[Span], groups: list[list[Span]]) -> list[int]:
+        """Index of every wanted row, in the order the spans ask for them, among the rows the groups produced."""
+        made: dict[tuple[int, int], int] = {}
+        at: dict[int, int] = {}
+        n = 0
+        for g in groups:
+            for sp in g:
+                base = at.get(sp.seq.seq_id, 0)
+                for k in sp.want:
+                    made.setdefault((sp.seq.seq_id, base + k), n)
+                    n += 1
+                at[sp.seq.seq_id] = base + len(sp.tokens)
+        return [made[(sp.seq.seq_id, k)] for sp in spans for k in sp.want]
 
     def _mm_embeds(self, part: list[tuple[Sequence, int]], fb: ForwardBatch, rows: int) -> torch.Tensor | None:
         """Embedding rows of a prefill chunk with the multimodal rows replaced, or None for text-only chunks."""
@@ -364,11 +526,34 @@ class Engine:
         graph = torch.cuda.CUDAGraph()
         with torch.cuda.graph(graph):
             out = self.model.forward(fb, self.kv)
-        g.graph, g.batch, g.out = graph, fb, out
+        g.graph, g.batch, g.out, g.logits = graph, fb, out, getattr(self.model, "last_logits", None)
         self.graphs[key] = g
         self.stats["captures"] += 1
         log_json("graph_capture", bucket=bucket, ms=(time.perf_counter() - t0) * 1e3, verbose_only=True)
         return g
+
+    def _check_capacity(self, seqs: list[Sequence]) -> None:
+        for s in seqs:
+            if self.kv.seqs[s.seq_id].length + 1 > self.settings.capacity:
+                raise OutOfBlocks(f"sequence {s.seq_id} reached the KV capacity {self.settings.capacity}")
+
+    def _launch_decode(self, seqs: list[Sequence]) -> tuple[torch.Tensor, torch.Tensor | None, ForwardBatch]:
+        """Upload and launch the decode step of every sequence's pending token (a graph replay where graphs are on);
+        returns (greedy ids, logits, batch), all of the padded bucket. Commits nothing."""
+        bucket = bucket_for(len(seqs))
+        if self.use_graph and getattr(self.model, "expert_provider", None) is None:
+            g = self.capture(bucket)
+            fb = g.batch
+            self._fill_decode(fb, seqs, bucket)
+            fb.upload()
+            g.graph.replay()
+            self.stats["graph_replays"] += 1
+            return g.out, g.logits, fb
+        fb = self._decode_batch(bucket)
+        self._fill_decode(fb, seqs, bucket)
+        fb.upload()
+        out = self.model.forward(fb, self.kv)
+        return out, getattr(self.model, "last_logits", None), fb
 
     def decode(self, seqs: list[Sequence]) -> list[int]:
         """One decode step for the given sequences (each must have a pending token)."""
@@ -379,31 +564,16 @@ class Engine:
             raise RuntimeError("injected step failure")
         try:
             n = len(seqs)
-            bucket = bucket_for(n)
             provider = getattr(self.model, "expert_provider", None)
             if provider is not None:
                 provider.begin_token()
-            for s in seqs:
-                if self.kv.seqs[s.seq_id].length + 1 > self.settings.capacity:
-                    raise OutOfBlocks(f"sequence {s.seq_id} reached the KV capacity {self.settings.capacity}")
-            if self.use_graph and provider is None:
-                g = self.capture(bucket)
-                fb = g.batch
-                self._fill_decode(fb, seqs, bucket)
-                fb.upload()
-                g.graph.replay()
-                out = g.out
-                self.stats["graph_replays"] += 1
-            else:
-                fb = self._decode_batch(bucket)
-                self._fill_decode(fb, seqs, bucket)
-                fb.upload()
-                out = self.model.forward(fb, self.kv)
+            self._check_capacity(seqs)
+            out, _, fb = self._launch_decode(seqs)
             toks = [int(t) for t in out[:n].cpu().tolist()]
             if provider is not None:
                 provider.finish_token()
             self.stats["h2d_bytes"] += fb.h2d_bytes()
-            self.stats["d2h_bytes"] += 4 * bucket
+            self.stats["d2h_bytes"] += 4 * fb.batch
             self._after_sync()
             for s, t in zip(seqs, toks):
                 self.kv.commit(s.seq_id, 1)

@@ -68,15 +68,19 @@ class PagedKVCache:
 
     def __init__(self, layers: int, kv_heads: int, head_dim: int, num_blocks: int, block_size: int = 64,
                  dtype: torch.dtype = torch.bfloat16, device: torch.device | str = "cpu",
-                 v_head_dim: int | None = None):
+                 v_head_dim: int | None = None, geometry: list[tuple[int, int, int]] | None = None):
+        """``geometry``: (kv heads, key width, value width) per layer, for models whose layers differ; otherwise every
+        layer has ``kv_heads`` heads of ``head_dim`` (values: ``v_head_dim``)."""
         self.layers, self.kv_heads, self.head_dim = layers, kv_heads, head_dim
         self.block_size, self.num_blocks = block_size, num_blocks
         self.device = torch.device(device)
         vd = v_head_dim if v_head_dim is not None else head_dim
-        self.k = [torch.zeros(num_blocks, kv_heads, block_size, head_dim, dtype=dtype, device=self.device)
-                  for _ in range(layers)]
-        self.v = [torch.zeros(num_blocks, kv_heads, block_size, vd, dtype=dtype, device=self.device)
-                  for _ in range(layers)] if vd > 0 else [None] * layers
+        self.geometry = list(geometry) if geometry is not None else [(kv_heads, head_dim, vd)] * layers
+        assert len(self.geometry) == layers, "one cache geometry per layer"
+        self.uniform = all(g == self.geometry[0] for g in self.geometry)
+        zeros = lambda h, d: torch.zeros(num_blocks, h, block_size, d, dtype=dtype, device=self.device) if d > 0 else None
+        self.k = [zeros(h, dk) for h, dk, _ in self.geometry]
+        self.v = [zeros(h, dv) for h, _, dv in self.geometry]
         self.alloc = BlockAllocator(num_blocks)
         self.seqs: dict[int, SequenceKV] = {}
         self.compact = None                 # engine.kv_compact.CompactKV when the cache format is affine8
@@ -161,7 +165,7 @@ class PagedKVCache:
         s = self.seqs[seq_id]
         bs = self.block_size
         dev = self.device
-        if dev.type == "cuda" and self.k[0].dtype == torch.bfloat16 and self.head_dim % 8 == 0 and \
+        if dev.type == "cuda" and self.uniform and self.k[0].dtype == torch.bfloat16 and self.geometry[0][1] % 8 == 0 and \
                 (self.v[0] is None or self.v[0].shape == self.k[0].shape):
             # two launches for all layers and both tensors (csrc/kv_util.cu)
             from ..ops.lib import check, kernels, ptr, status_tensor, stream_ptr

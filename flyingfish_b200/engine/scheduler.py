@@ -7,6 +7,8 @@ batch and ONE packed prefill chunk: waiting requests are admitted while KV block
 are free, every sequence that is already generating decodes one token, and the rest of the budget
 goes to prompt rows of the sequences still prefilling (oldest first). A long prompt is therefore
 spread over several iterations and never stalls the running streams for more than one chunk.
+Where the model's forward takes prompt portions and single tokens together (``engine.mixed_batches``)
+an iteration with both is one batch, otherwise a decode step followed by a prefill chunk.
 Requests can be aborted at any iteration (client disconnect), which frees their blocks at once.
 
 The scheduler is synchronous and engine-agnostic (it only needs ``add_sequence / prefill /
@@ -98,11 +100,18 @@ class Scheduler:
         bs = self.engine.kv.block_size
         return (tokens + bs - 1) // bs
 
+    def _promised_blocks(self) -> int:
+        kv = self.engine.kv
+        if not hasattr(kv, "blocks_needed"):
+            return 0
+        return sum(kv.blocks_needed(r.seq.seq_id, max(len(r.seq.prompt) - r.seq.prefilled, 0) + 1) for r in self.running)
+
     def _admit(self) -> list[Request]:
         admitted = []
-        free = self.engine.kv.alloc.free_blocks
-        # blocks already promised to running sequences for their remaining growth are not
-        # reserved: a sequence that cannot grow is preempted (see _decode)
+        # the blocks the running sequences take next (the rest of a prompt, the next decoded token) are theirs: admitting
+        # a request into them would preempt it again in the same iteration. Growth beyond that is not reserved: a
+        # sequence that cannot grow is preempted (see step)
+        free = self.engine.kv.alloc.free_blocks - self._promised_blocks()
         while self.waiting and len(self.running) + len(admitted) < self.max_running:
             req = self.waiting[0]
             need = self._blocks_for(len(req.prompt) + len(req.output) + 1)
@@ -159,6 +168,8 @@ class Scheduler:
         self.running.extend(self._admit())
         decoding = [r for r in self.running if r.seq.prefilled >= len(r.seq.prompt)][: self.engine.max_batch]
         prefilling = [r for r in self.running if r.seq.prefilled < len(r.seq.prompt)]
+        if decoding and prefilling and getattr(self.engine, "mixed_batches", False) and self._mixed_room(decoding):
+            return self._step_mixed(decoding, prefilling)
         # ---- decode step of every generating sequence ----
         if decoding:
             try:
@@ -184,6 +195,27 @@ class Scheduler:
                     produced += 1
         self.running = [r for r in self.running if r.state == "running" and not (r.output and self._maybe_finish(r))]
         return produced
+
+    def _mixed_room(self, decoding: list[Request]) -> bool:
+        return self.token_budget > len(decoding) and self.engine.max_batch > len(decoding)
+
+    def _step_mixed(self, decoding: list[Request], prefilling: list[Request]) -> int:
+        """An iteration of a model whose forward takes both kinds of rows: the decoded tokens and the prefill chunk are
+        one batch, so the weights are read once for both."""
+        try:
+            toks, done = self.engine.mixed_step([r.seq for r in decoding], [r.seq for r in prefilling],
+                                                self.token_budget - len(decoding))
+        except OutOfBlocks:
+            self._preempt_youngest()
+            return 0
+        for r, t in zip(decoding, toks):
+            self._emit(r, [t])
+        finished_ids = {s.seq_id for s in done}
+        for r in prefilling:
+            if r.seq.seq_id in finished_ids:
+                self._emit(r, [r.seq.output[-1]])
+        self.running = [r for r in self.running if r.state == "running" and not (r.output and self._maybe_finish(r))]
+        return len(toks) + len(done)
 
     def run_until_idle(self, max_iters: int = 1_000_000) -> None:
         it = 0

@@ -38,6 +38,9 @@ def _linear_entries(name: str, out_f: int, in_f: int, fmt: str) -> dict[str, tup
 
 def manifest(spec: ModelSpec, policy: LoadPolicy = LoadPolicy.TEXT_ONLY) -> dict[str, tuple[tuple[int, ...], str]]:
     """name -> (shape, dtype class in {float, f32, fp8, u8})."""
+    if spec.arch == "duponex":
+        from ..models.duponex import expected_tensors
+        return {n: (shape, "float") for n, shape in expected_tensors(spec).items()}
     m: dict[str, tuple[tuple[int, ...], str]] = {}
     h, d = spec.hidden, spec.head_dim
     m["model.embed_tokens.weight"] = ((spec.vocab, h), "float")
@@ -244,6 +247,16 @@ def checkpoint_source(model_dir: str | Path, spec: ModelSpec, device: torch.devi
             raise CheckpointError(f"{name}: dtype {ck.info(name).dtype} is not a float tensor")
         return t.to(device=device, dtype=dtype)
     return source, ck.close
+
+
+def audited_source(model_dir: str | Path, spec: ModelSpec, device: torch.device | str):
+    """:func:`checkpoint_source` of a directory that holds exactly the manifest of ``spec``."""
+    ck = MappedCheckpoint(Path(model_dir))
+    try:
+        audit(ck, spec)
+    finally:
+        ck.close()
+    return checkpoint_source(model_dir, spec, device)
 
 
 def save_decoder_checkpoint(model_dir: str | Path, spec: ModelSpec, tensors: dict[str, torch.Tensor],

@@ -54,6 +54,7 @@ class DecoderModel:
         self.capture_taps: dict[int, int] = {}    # layer index -> tap slot for draft-model hidden taps
         self.capture_slab: torch.Tensor | None = None
         self.normed_sink: list | None = None      # when a list: every forward appends its final-normed rows
+        self.last_logits: torch.Tensor | None = None   # logits of the latest forward (a captured step keeps its own)
         self._rope_cs: torch.Tensor | None = None  # per-forward cos/sin table of the fused QKV kernels
         # encoders and diffusion language models attend in both directions inside a sequence; they run whole
         # sequences in one prefill chunk and never decode
@@ -242,6 +243,7 @@ class DecoderModel:
                 inputs_embeds: torch.Tensor | None = None) -> torch.Tensor:
         n = self.hidden_states(b, kv, inputs_embeds)
         lg = self.logits(n, b)
+        self.last_logits = lg
         if self.trace is not None:
             self.trace.record("logits", lg)
         if return_logits:

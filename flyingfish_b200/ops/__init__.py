@@ -110,15 +110,21 @@ FUSE_ATTN_MERGE = os.environ.get("FLYINGFISH_FUSE_ATTN_MERGE", "0") == "1"
 ATTN_PREFILL_TC = os.environ.get("FF_ATTN_PREFILL", "tc") != "mma"
 
 
+ACTIVATIONS = {None: 0, "relu2": 1}
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
-           out_dtype: torch.dtype | None = None) -> torch.Tensor:
-    """``y[M,N] = x[M,K] @ w[N,K].T`` (BF16 operands, FP32 accumulation).
+           out_dtype: torch.dtype | None = None, bias: torch.Tensor | None = None, act: str | None = None) -> torch.Tensor:
+    """``y[M,N] = act(x[M,K] @ w[N,K].T + bias[N])`` (BF16 operands, FP32 accumulation, bias and activation in the GEMM's
+    epilogue; ``act``: "relu2", the square of the positive part). FP32 operands take the SIMT kernel of
+    ``csrc/gemm_f32.cu`` (true 32-bit products).
 
     CUDA path: tcgen05 kernels -- the weight-streaming decode kernel of ``csrc/gemm_skinny.cu`` (tokens on
     the UMMA M side, cluster split-K or stream-K) for M <= 128, the persistent 128x256x64 kernel of
     ``csrc/gemm_bf16.cu`` otherwise. ``w`` may be an FP8-resident weight (``quant_ops.Fp8Weight``): the block-scaled
     W8A8 GEMM of ``csrc/gemm_fp8.cu`` (CPU: its oracle) runs instead."""
     if not isinstance(w, torch.Tensor):
+        _require(bias is None and act is None, "linear: FP8-resident weights take no bias or activation")
         from . import quant_ops
         tok = min(128, (x.shape[0] + 15) // 16 * 16)
         if x.shape[0] > FP8_DENSE_ROWS or w.shape[1] > FP8_MAX_K or (w.shape[1] // 128) * tok * 4 > 64 * 1024:
@@ -134,11 +140,16 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
             return out
         return y
     if not _is_cuda(x):
-        y = ref.linear(x, w, out_dtype)
+        y = ref.linear(x, w, out_dtype, bias, act)
         if out is not None:
             out.copy_(y)
             return out
         return y
+    if bias is not None:
+        _require(bias.dtype == x.dtype and bias.numel() == w.shape[0] and bias.is_contiguous() and bias.data_ptr() % 16 == 0,
+                 "linear: bias must be one aligned vector of the operands' type")
+    if x.dtype == torch.float32:
+        return _linear_f32(x, w, out, out_dtype, bias, act)
     _require(x.dtype == BF16 and w.dtype == BF16, "linear: BF16 operands required on CUDA")
     m, ldx = _rows2d(x)
     n, ldw = _rows2d(w)
@@ -150,20 +161,45 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
     _require(out.shape == (m, n) and out.stride(1) == 1 and out.dtype == odt, "linear: bad output tensor")
     lib = kernels()
     st = status_tensor(x.device)
+    plain = bias is None and act is None
+    _require(plain or odt == BF16, "linear: bias and activation come with a bf16 output")
     if m <= SKINNY_MAX_M and odt == BF16:
         scratch_b, counter_b = c_longlong(0), c_longlong(0)
         splits = lib.ff_gemm_skinny_plan(m, n, k, ctypes.byref(scratch_b), ctypes.byref(counter_b))
         ws = workspace(x.device)
         scratch = ws.ensure("gemm_scratch", scratch_b.value // 4) if scratch_b.value > 0 else None
         _require(counter_b.value // 4 <= ws.gemm_counters.numel(), "linear: too many column tiles for counters")
-        rc = lib.ff_gemm_skinny(ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), splits, ptr(scratch),
-                                ptr(ws.gemm_counters), ptr(st), stream_ptr())
+        args = (ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), splits, ptr(scratch), ptr(ws.gemm_counters))
+        if plain:
+            rc = lib.ff_gemm_skinny(*args, ptr(st), stream_ptr())
+        else:
+            rc = lib.ff_gemm_skinny_act(*args, ptr(bias), ACTIVATIONS[act], ptr(st), stream_ptr())
         check(rc, "ff_gemm_skinny")
     else:
         epi = 0 if odt == BF16 else 2
         _require(odt in (BF16, torch.float32), "linear: output dtype must be bf16 or fp32")
-        rc = lib.ff_gemm_bf16(ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), epi, ptr(st), stream_ptr())
+        if plain:
+            rc = lib.ff_gemm_bf16(ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), epi, ptr(st), stream_ptr())
+        else:
+            rc = lib.ff_gemm_bf16_act(ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), ptr(bias), ACTIVATIONS[act], ptr(st),
+                                      stream_ptr())
         check(rc, "ff_gemm_bf16")
+    _count()
+    return out
+
+
+def _linear_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None, out_dtype: torch.dtype | None,
+                bias: torch.Tensor | None, act: str | None) -> torch.Tensor:
+    _require(w.dtype == torch.float32 and out_dtype in (None, torch.float32), "linear: FP32 operands give an FP32 result")
+    m, ldx = _rows2d(x)
+    n, ldw = _rows2d(w)
+    _require(w.shape[1] == x.shape[1], "linear: inner dimensions differ")
+    if out is None:
+        out = torch.empty(m, n, dtype=torch.float32, device=x.device)
+    _require(out.shape == (m, n) and out.stride(1) == 1 and out.dtype == torch.float32, "linear: bad output tensor")
+    rc = kernels().ff_gemm_f32(ptr(x), ptr(w), ptr(out), m, n, x.shape[1], ldx, ldw, out.stride(0), ptr(bias), ACTIVATIONS[act],
+                               stream_ptr())
+    check(rc, "ff_gemm_f32")
     _count()
     return out
 
@@ -377,6 +413,33 @@ def linear_rope_kv(x: torch.Tensor, wqkv: torch.Tensor, positions: torch.Tensor,
     return out
 
 
+def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, hq: int, hkv: int,
+                 dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0) -> None:
+    """Packed rows ``[q heads | k heads | v heads | ...]``: q and k are divided by their root mean square per head (no
+    weight; ``dim`` elements count, the row's heads may carry padding up to the cache's width), v is blended with
+    ``first_v`` (``(1 - mix) v + mix first_v``; a column slice of an earlier layer's packed rows), k and v are written to
+    ``slots`` of the paged cache and q back into the row. No positions enter. BF16 or FP32."""
+    if not _is_cuda(qkv):
+        ref.head_norm_kv(qkv, slots, kcache, vcache, hq, hkv, dim, vdim, eps, first_v, mix)
+        return
+    rows, ld = _rows2d(qkv)
+    nb, ch, bs, dk = kcache.shape
+    dv = vcache.shape[3]
+    _require(slots.dtype == torch.int32 and kcache.is_contiguous() and vcache.is_contiguous(), "head_norm_kv: metadata / cache layout")
+    _require(ch == hkv == vcache.shape[1] and vcache.shape[0] == nb and vcache.shape[2] == bs and dk >= dim and dv >= vdim,
+             "head_norm_kv: cache geometry differs from the heads")
+    _require(qkv.shape[1] >= (hq + hkv) * dk + hkv * dv and qkv.dtype == kcache.dtype == vcache.dtype, "head_norm_kv: packed row")
+    ldf = 0
+    if first_v is not None:
+        _require(first_v.shape == (rows, hkv * dv) and first_v.stride(1) == 1 and first_v.dtype == qkv.dtype, "head_norm_kv: first values")
+        ldf = first_v.stride(0)
+    rc = kernels().ff_head_norm_kv(ptr(qkv), ptr(slots), ptr(kcache), ptr(vcache), ptr(first_v), rows, hq, hkv, dim, dk, dv, bs, nb, ld,
+                                   ldf, c_float(eps), c_float(mix), int(qkv.dtype == torch.float32), ptr(status_tensor(qkv.device)),
+                                   stream_ptr())
+    check(rc, "ff_head_norm_kv")
+    _count()
+
+
 def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0, out: torch.Tensor | None = None,
              interleaved: bool = False) -> torch.Tensor:
     if not _is_cuda(gu):
@@ -410,27 +473,42 @@ def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
 def attn_decode(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_table: torch.Tensor,
                 ctx_lens: torch.Tensor, hq: int, hkv: int, dim: int, scale: float, nq: int = 1,
                 tree_mask: torch.Tensor | None = None, max_ctx: int | None = None,
-                out: torch.Tensor | None = None, window: int = 0, sinks: torch.Tensor | None = None) -> torch.Tensor:
+                out: torch.Tensor | None = None, window: int = 0, sinks: torch.Tensor | None = None, chunk: int = 0,
+                vdim: int | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
     """Decode / multi-row verify attention. ``q`` holds ``batch * nq`` rows (heads at columns
     ``h*dim``; it may be the packed QKV buffer). ``ctx_lens[b]`` counts the keys visible to the last
     of the ``nq`` rows. ``window > 0``: every row sees only its last ``window`` keys (local-attention
     layers; not together with a tree mask). ``sinks`` (float32 [hq]): learnable soft-max, one sink logit per head in the
-    denominator. Returns ``[batch*nq, hq*dim]``."""
+    denominator. ``chunk > 0``: a row sees only keys of its own block of ``chunk`` positions. ``vdim``: width of the value
+    heads (default ``dim``). ``gate`` ([rows, hq*vdim], a column slice of the packed rows): the result is multiplied by its
+    sigmoid before it is rounded. Heads up to 128 wide (multiples of 16) take the tensor-core kernel, other widths and
+    FP32 the SIMT kernel. Returns ``[batch*nq, hq*vdim]``."""
     batch = block_table.shape[0]
+    vdim = vdim or dim
+    _require(not (chunk > 0 and (window > 0 or tree_mask is not None)), "attn_decode: one kind of mask at a time")
     _require(not (window > 0 and tree_mask is not None), "attn_decode: window and tree mask are exclusive")
     _require(not (sinks is not None and tree_mask is not None), "attn_decode: sinks and tree mask are exclusive")
     if not _is_cuda(q):
         q_start = torch.arange(batch, dtype=torch.int32) * nq
         q_lens = torch.full((batch,), nq, dtype=torch.int32)
         tm = None if tree_mask is None else tree_mask.view(batch, nq)
-        return ref.attention_paged(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, scale, tm,
-                                   window, sinks)
+        y = ref.attention_paged(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, scale, tm, window, sinks,
+                                chunk, vdim, gate)
+        if out is not None:
+            out.copy_(y)
+            return out
+        return y
     rows, ldq = _rows2d(q)
     _require(rows == batch * nq, "attn_decode: q rows must equal batch * nq")
     _require(block_table.dtype == torch.int32 and block_table.is_contiguous(), "attn_decode: block table int32")
     _require(ctx_lens.dtype == torch.int32, "attn_decode: ctx_lens int32")
     nb = kcache.shape[0]
-    _require(kcache.shape[2] == 64 and kcache.shape[3] == dim == 128, "attn_decode: block 64 / head_dim 128 only")
+    if q.dtype == torch.float32 or max(dim, vdim) > 128:
+        _require(sinks is None and tree_mask is None, "attn_decode: the SIMT kernel has no sinks or tree masks")
+        return _attn_simt(q, kcache, vcache, block_table, None, None, ctx_lens, nq, hq, hkv, dim, vdim, scale, window, chunk, gate, out)
+    _require(kcache.shape[2] == 64 and kcache.shape[3] == dim and vcache.shape[3] == vdim, "attn_decode: 64-token blocks of these heads")
+    _require(dim % 16 == 0 and vdim % 16 == 0, "attn_decode: head widths must be multiples of 16")
+    general = chunk > 0 or gate is not None or dim != 128 or vdim != 128
     if max_ctx is None:
         max_ctx = block_table.shape[1] * 64
     lib = kernels()
@@ -440,14 +518,23 @@ def attn_decode(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, blo
     part_o = ws.ensure("attn_o", po.value // 4) if nsplit > 1 else None
     part_ml = ws.ensure("attn_ml", pml.value // 4) if nsplit > 1 else None
     if out is None:
-        out = torch.empty(rows, hq * dim, dtype=BF16, device=q.device)
+        out = torch.empty(rows, hq * vdim, dtype=BF16, device=q.device)
     if tree_mask is not None:
         _require(tree_mask.dtype == torch.int64 and tree_mask.numel() == batch * nq, "attn_decode: tree mask int64")
     # optionally the last split of a (sequence, kv head, row tile) merges in place of a second kernel; measured
     # slower on B200 (81.8 vs 75.6 us at batch 64 / context 1100: every CTA pays a fence and an atomic), so off
     items = batch * hkv * ((nq * (hq // hkv) + 15) // 16)
     counters = ws.attn_counters if (FUSE_ATTN_MERGE and nsplit > 1 and items <= ws.attn_counters.numel()) else None
-    if sinks is not None:
+    if general:
+        _require(tree_mask is None and out.is_contiguous() and out.shape == (rows, hq * vdim), "attn_decode: masks / output of general heads")
+        _require(sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == hq and sinks.is_contiguous()),
+                 "attn_decode: sinks float32 [hq]")
+        rc = lib.ff_attn_decode_general(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(ctx_lens), ptr(out), ptr(part_o),
+                                        ptr(part_ml), batch, hq, hkv, dim, vdim, nq, ldq, block_table.shape[1], nb, nsplit,
+                                        c_float(scale), max(window, 0), chunk, ptr(sinks), ptr(gate), _gate_ld(gate, rows, hq * vdim),
+                                        ptr(status_tensor(q.device)), stream_ptr())
+        counters = None
+    elif sinks is not None:
         _require(sinks.dtype == torch.float32 and sinks.numel() == hq and sinks.is_contiguous(), "attn_decode: sinks float32 [hq]")
         counters = None
         rc = lib.ff_attn_decode_sink(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(ctx_lens), ptr(out),
@@ -465,6 +552,32 @@ def attn_decode(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, blo
                                 nb, nsplit, c_float(scale), ptr(counters), ptr(status_tensor(q.device)), stream_ptr())
     check(rc, "ff_attn_decode")
     _count(1 if (nsplit == 1 or counters is not None) else 2)
+    return out
+
+
+def _gate_ld(gate: torch.Tensor | None, rows: int, width: int) -> int:
+    if gate is None:
+        return 0
+    _require(gate.shape == (rows, width) and gate.stride(1) == 1 and gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0,
+             "attention: the gate must be aligned rows as wide as the output")
+    return gate.stride(0)
+
+
+def _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, nq: int, hq: int, hkv: int, dim: int, vdim: int,
+               scale: float, window: int, chunk: int, gate: torch.Tensor | None, out: torch.Tensor | None) -> torch.Tensor:
+    """Paged attention of any head width, BF16 or FP32 (``csrc/attention_simt.cu``): one warp per query row and head.
+    Rows come as ranges (``q_start`` / ``q_lens``) or, without them, ``nq`` per sequence."""
+    rows, ldq = _rows2d(q)
+    if out is None:
+        out = torch.empty(rows, hq * vdim, dtype=q.dtype, device=q.device)
+    _require(q.dtype == kcache.dtype == vcache.dtype == out.dtype and q.dtype in (BF16, torch.float32), "attention: one type throughout")
+    _require(kcache.shape[1] == hkv and kcache.shape[3] == dim and vcache.shape[3] == vdim and out.stride(1) == 1, "attention: geometry")
+    rc = kernels().ff_attn_simt(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(out),
+                                block_table.shape[0], rows, nq, hq, hkv, dim, vdim, ldq, out.stride(0), kcache.shape[2],
+                                block_table.shape[1], kcache.shape[0], c_float(scale), window, chunk, ptr(gate),
+                                _gate_ld(gate, rows, hq * vdim), int(q.dtype == torch.float32), ptr(status_tensor(q.device)), stream_ptr())
+    check(rc, "ff_attn_simt")
+    _count()
     return out
 
 
@@ -538,28 +651,43 @@ def attn_decode_mixed(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tenso
 def attn_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_table: torch.Tensor,
                  q_start: torch.Tensor, q_lens: torch.Tensor, ctx_lens: torch.Tensor, max_q_len: int, hq: int,
                  hkv: int, dim: int, scale: float, window: int = 0, out: torch.Tensor | None = None,
-                 sinks: torch.Tensor | None = None) -> torch.Tensor:
+                 sinks: torch.Tensor | None = None, chunk: int = 0, vdim: int | None = None,
+                 gate: torch.Tensor | None = None) -> torch.Tensor:
     """Causal chunked-prefill attention of packed query rows against the paged cache. ``window < 0`` makes it
     bidirectional: every query row sees all ``ctx_lens`` keys of its sequence (encoders, vision towers). ``sinks``
-    (float32 [hq]): learnable soft-max, one sink logit per head in the denominator (tcgen05 kernel only)."""
+    (float32 [hq]): learnable soft-max, one sink logit per head in the denominator (tcgen05 kernel only). ``chunk``,
+    ``vdim`` and ``gate`` as in :func:`attn_decode`."""
+    vdim = vdim or dim
+    _require(not (chunk > 0 and window != 0), "attn_prefill: one kind of mask at a time")
     if not _is_cuda(q):
-        return ref.attention_paged(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, scale,
-                                   None, window, sinks)
+        y = ref.attention_paged(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, scale, None, window, sinks,
+                                chunk, vdim, gate)
+        if out is not None:
+            out.copy_(y)
+            return out
+        return y
     rows, ldq = _rows2d(q)
     batch = block_table.shape[0]
     if out is None:
-        out = torch.empty(rows, hq * dim, dtype=BF16, device=q.device)
+        out = torch.empty(rows, hq * vdim, dtype=q.dtype, device=q.device)
     nb = kcache.shape[0]
-    _require(kcache.shape[2] == 64 and dim == 128, "attn_prefill: block 64 / head_dim 128 only")
+    if q.dtype == torch.float32 or max(dim, vdim) > 128:
+        _require(sinks is None, "attn_prefill: the SIMT kernel has no sinks")
+        return _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, 1, hq, hkv, dim, vdim, scale, window, chunk, gate, out)
+    general = chunk > 0 or gate is not None or dim != 128 or vdim != 128
+    _require(kcache.shape[2] == 64 and kcache.shape[3] == dim and vcache.shape[3] == vdim and dim % 16 == 0 and vdim % 16 == 0,
+             "attn_prefill: 64-token blocks, head widths in multiples of 16")
+    if general:
+        _require(out.stride(0) % 8 == 0 and ldq % 8 == 0, "attn_prefill: 16-byte aligned rows")
     if sinks is not None:
         _require(sinks.dtype == torch.float32 and sinks.numel() == hq and sinks.is_contiguous(), "attn_prefill: sinks float32 [hq]")
         _require(out.stride(0) % 8 == 0 and ldq % 8 == 0, "attn_prefill: sinks need the tcgen05 kernel (16-byte aligned rows)")
-    if (ATTN_PREFILL_TC or sinks is not None) and out.stride(0) % 8 == 0 and ldq % 8 == 0:
+    if (ATTN_PREFILL_TC or sinks is not None or general) and out.stride(0) % 8 == 0 and ldq % 8 == 0:
         # tcgen05 kernel: Q Kᵀ and P V on the tensor cores with S and O in tensor memory
         rc = kernels().ff_attn_prefill_tc(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens),
-                                          ptr(ctx_lens), ptr(out), batch, rows, max_q_len, hq, hkv, dim, ldq, out.stride(0),
-                                          block_table.shape[1], nb, c_float(scale), window, ptr(sinks),
-                                          ptr(status_tensor(q.device)), stream_ptr())
+                                          ptr(ctx_lens), ptr(out), batch, rows, max_q_len, hq, hkv, dim, vdim, ldq, out.stride(0),
+                                          block_table.shape[1], nb, c_float(scale), window, chunk, ptr(sinks), ptr(gate),
+                                          _gate_ld(gate, rows, hq * vdim), ptr(status_tensor(q.device)), stream_ptr())
         check(rc, "ff_attn_prefill_tc")
         _count()
         return out

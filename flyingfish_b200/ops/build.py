@@ -48,8 +48,24 @@ def _hash(files: list[Path], extra: str = "") -> str:
     return h.hexdigest()
 
 
-def kernel_sources() -> list[Path]:
-    return sorted(CSRC.glob("*.cu"))
+# sources a process needs that serves nothing but the architecture (see lib.restrict_to)
+ARCH_SOURCES = {
+    "duponex": ("attention_paged", "attention_simt", "attention_tc", "gemm_bf16", "gemm_f32", "gemm_skinny", "head_norm",
+                "kv_util", "rope_act_sample", "streams"),
+}
+
+
+def kernel_sources(only: tuple[str, ...] | None = None) -> list[Path]:
+    return sorted(p for p in CSRC.glob("*.cu") if only is None or p.stem in only)
+
+
+def _stamp_of(srcs: list[Path], flags: list[str]) -> str:
+    return _hash(srcs + sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h")), " ".join(flags))
+
+
+def kernels_up_to_date() -> bool:
+    """Whether the library of all kernels is built from the present sources."""
+    return _up_to_date(HERE / "_ff_kernels.so", _stamp_of(kernel_sources(), NVCC_FLAGS))
 
 
 def host_sources() -> list[Path]:
@@ -65,7 +81,7 @@ SHORT_WAIT_NS = 5_000_000      # bound of every device-side wait in the short-wa
 
 
 def build_kernels(verbose: bool = False, force: bool = False, ptxas_info: bool = False, timeline: bool = False,
-                  short_wait: bool = False, debug_checks: bool = False) -> Path:
+                  short_wait: bool = False, debug_checks: bool = False, only: tuple[str, ...] | None = None) -> Path:
     """Compile all ``csrc/*.cu`` into ``_ff_kernels.so`` (no-op when up to date).
 
     ``timeline=True`` builds the tracing variant ``_ff_kernels_tl.so`` (``-DFF_TIMELINE``): kernels
@@ -74,14 +90,16 @@ def build_kernels(verbose: bool = False, force: bool = False, ptxas_info: bool =
     tests of the time-out paths load it, so that a wait nobody answers runs out at once.
     ``debug_checks=True`` builds ``_ff_kernels_dbg.so`` (``-DFF_DEBUG_CHECKS``): scratch with a single-writer
     contract claims its elements in a ledger and a second claim inside one launch raises a status error; extra
-    in-kernel bounds words are compiled in."""
+    in-kernel bounds words are compiled in.
+    ``only`` (source stems) builds a partial library ``_ff_kernels_part.so``; its objects are the full library's."""
     tag = "tl" if timeline else "sw" if short_wait else "dbg" if debug_checks else ""
     lib = HERE / (f"_ff_kernels_{tag}.so" if tag else "_ff_kernels.so")
-    srcs = kernel_sources()
-    deps = srcs + sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+    srcs = kernel_sources(only)
+    if only is not None:
+        lib = HERE / f"{lib.stem}_part.so"
     base_flags = list(NVCC_FLAGS) + (["-DFF_TIMELINE"] if timeline else []) + \
         ([f"-DFF_WAIT_NS={SHORT_WAIT_NS}ull"] if short_wait else []) + (["-DFF_DEBUG_CHECKS"] if debug_checks else [])
-    stamp = _hash(deps, " ".join(base_flags))
+    stamp = _stamp_of(srcs, base_flags)
     if not force and _up_to_date(lib, stamp):
         return lib
     build_dir = BUILD / tag if tag else BUILD

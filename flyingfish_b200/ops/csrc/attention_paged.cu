@@ -1,4 +1,6 @@
-// Paged GQA attention (head_dim 128) over the block cache written by rope_kv_paged:
+// Paged GQA attention over the block cache written by rope_kv_paged / head_norm_kv. Prefill: head_dim 128. Decode: key and
+// value heads of up to 128 elements (multiples of 16, not necessarily equal) in 128-wide tiles -- TMA fills the columns
+// past a head with zeros, which neither product sees.
 //   attn_decode : split-KV flash-decode. One CTA = (split, kv head, sequence); the G query heads of
 //                 the group (times up to 16/G query rows for multi-row verification) are packed
 //                 into one 16-row MMA tile so each K/V byte is read once per group. Partials
@@ -78,10 +80,12 @@ struct RowState {
 //   key0      : global key index of smem row key_off
 //   lim0/lim1 : last visible key index for rows g and g+8 (inclusive); mask0/mask1: optional
 //               64-bit ancestor sets over keys >= tail_start (bit i = key tail_start+i visible)
+//   kd, vd    : 16-element steps of the key heads and pairs of 8-element columns of the value heads to run (8: 128 wide)
 template <int NT8>
 __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[8][4], RowState& st, uint32_t sK, uint32_t sV,
                                           int key_off, int key0, int lim0, int lim1, bool use_mask, int tail_start,
-                                          unsigned long long mask0, unsigned long long mask1, float scale_log2) {
+                                          unsigned long long mask0, unsigned long long mask1, float scale_log2, int kd = 8,
+                                          int vd = 8) {
   const int lane = threadIdx.x & 31, t = lane & 3;
   float s[NT8][4];
 #pragma unroll
@@ -92,6 +96,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[8][4], RowState& 
   const uint32_t khx = ((lane >> 3) & 1) ^ (lane & 7);
 #pragma unroll
   for (int kk = 0; kk < 8; ++kk) {
+    if (kk >= kd) break;
 #pragma unroll
     for (int np = 0; np < NT8 / 2; ++np) {
       uint32_t b0, b1, b2, b3;
@@ -153,6 +158,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[8][4], RowState& 
     const uint32_t vhx = (lane >> 4) ^ (lane & 7);
 #pragma unroll
     for (int dp = 0; dp < 8; ++dp) {
+      if (dp >= vd) break;
       uint32_t b0, b1, b2, b3;
       ldmatrix_x4_trans(vbase + (uint32_t)((dp >> 2) * (PAGE * 128)) + (((uint32_t)(2 * (dp & 3)) ^ vhx) << 4), b0, b1, b2, b3);
       mma_bf16(st.o[2 * dp], pa, b0, b1);
@@ -168,16 +174,31 @@ __device__ __forceinline__ void init_state(RowState& st) {
 }
 
 // Q fragments for rows (r0, r0+8) given per-row pointers (null -> zero row)
-__device__ __forceinline__ void load_q_frags(uint32_t (&qf)[8][4], const __nv_bfloat16* q0, const __nv_bfloat16* q1) {
+__device__ __forceinline__ void load_q_frags(uint32_t (&qf)[8][4], const __nv_bfloat16* q0, const __nv_bfloat16* q1, int kd = 8) {
   const int t = threadIdx.x & 3;
 #pragma unroll
   for (int kk = 0; kk < 8; ++kk) {
     const int d = kk * 16 + 2 * t;
+    if (kk >= kd) { qf[kk][0] = qf[kk][1] = qf[kk][2] = qf[kk][3] = 0u; continue; }
     qf[kk][0] = q0 ? *reinterpret_cast<const uint32_t*>(q0 + d) : 0u;
     qf[kk][1] = q1 ? *reinterpret_cast<const uint32_t*>(q1 + d) : 0u;
     qf[kk][2] = q0 ? *reinterpret_cast<const uint32_t*>(q0 + d + 8) : 0u;
     qf[kk][3] = q1 ? *reinterpret_cast<const uint32_t*>(q1 + d + 8) : 0u;
   }
+}
+
+// What a decode launch adds to plain causal 128-wide attention. A row at position p sees keys
+//   window > 0: p - window + 1 .. p          chunk > 0: the keys <= p of p's own block of `chunk` positions
+// dk / dv: widths of the key / value heads; gate: [rows, hq * dv] (row pitch ldg), the result is multiplied by its sigmoid.
+struct DecodeForm {
+  int window, chunk, dk, dv, ldg;
+  const __nv_bfloat16* gate;
+};
+__device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
+  return window > 0 ? max(0, pos - window + 1) : (chunk > 0 ? max(0, pos) / chunk * chunk : 0);
+}
+__device__ __forceinline__ float gate_factor(const __nv_bfloat16* gate, int ldg, size_t row, int col) {
+  return gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-__bfloat162float(gate[row * ldg + col])));
 }
 
 // ---------------------------------------------------------------------------------------
@@ -198,7 +219,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
                    const int* __restrict__ ctx_lens, const unsigned long long* __restrict__ tree_mask,
                    __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int hq,
                    int hkv, int nq, int ldq, int max_blocks, int num_blocks, int nsplit, float scale_log2,
-                   int* status, int* __restrict__ split_counters, int window, const int* __restrict__ kv_start,
+                   int* status, int* __restrict__ split_counters, const DecodeForm f, const int* __restrict__ kv_start,
                    int pstride, const float* __restrict__ sinks) {
   pdl_trigger();
   if (threadIdx.x == 0) FF_TL(status, KID_ATTN_DECODE, 0);
@@ -217,7 +238,9 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   // sees keys pos - window + 1 .. pos, so the pages before the earliest bound of the nq queries are not visited
   // kv_start (mixed cache formats): keys below kv_start[b] (a multiple of the page size) are not in BF16 pages any
   // more; another kernel covers them and writes its partials behind this kernel's splits (stride pstride)
-  int pfirst = window > 0 ? max(0, ctx - nq - window + 1) / PAGE : 0;
+  const int window = f.window, chunk = f.chunk, kd = f.dk >> 4, vd = f.dv >> 4;
+  const bool k_hi = f.dk > 64, v_hi = f.dv > 64;           // heads up to 64 wide: the upper half of a tile is not loaded
+  int pfirst = first_visible(ctx - nq, window, chunk) / PAGE;
   if (kv_start != nullptr) pfirst = max(pfirst, min(kv_start[b], ctx) / PAGE);
   const int per = (pages - pfirst + nsplit - 1) / nsplit;
   const int p0 = pfirst + split * per, p1 = min(pages, p0 + per);
@@ -231,13 +254,13 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     const int r = rt * 16 + g + e * 8;
     if (r < rows_total) {
       const int qi = r / G, hh = kvh * G + r % G;
-      qp[e] = q + (size_t)(b * nq + qi) * ldq + (size_t)hh * HD;
+      qp[e] = q + (size_t)(b * nq + qi) * ldq + (size_t)hh * f.dk;
       lim[e] = ctx - nq + qi;
       mk[e] = tree_mask ? tree_mask[(size_t)b * nq + qi] : ~0ull;
     } else { qp[e] = nullptr; lim[e] = -1; mk[e] = 0ull; }
   }
   uint32_t qf[8][4];
-  load_q_frags(qf, qp[0], qp[1]);
+  load_q_frags(qf, qp[0], qp[1], kd);
   RowState st; init_state(st);
 
   // DEC_STAGES stages of (K page, V page); thread 0 keeps DEC_STAGES-1 pages requested by TMA (four 8-KiB
@@ -262,11 +285,11 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     const int row = (blk * hkv + kvh) * PAGE;
     uint8_t* sk = smem + buf * STAGE_BYTES;
     uint8_t* sv = sk + PAGE * HD * 2;
-    mbar_expect_tx(&full_bar[buf], STAGE_BYTES);
+    mbar_expect_tx(&full_bar[buf], (2 + (k_hi ? 1 : 0) + (v_hi ? 1 : 0)) * PAGE * 128);
     tma_load_2d(sk, &tmK, &full_bar[buf], 0, row);
-    tma_load_2d(sk + PAGE * 128, &tmK, &full_bar[buf], 64, row);
+    if (k_hi) tma_load_2d(sk + PAGE * 128, &tmK, &full_bar[buf], 64, row);
     tma_load_2d(sv, &tmV, &full_bar[buf], 0, row);
-    tma_load_2d(sv + PAGE * 128, &tmV, &full_bar[buf], 64, row);
+    if (v_hi) tma_load_2d(sv + PAGE * 128, &tmV, &full_bar[buf], 64, row);
   };
   if (threadIdx.x == 0)
     for (int i = 0; i < DEC_STAGES - 1 && p0 + i < p1; ++i) issue(p0 + i, i);
@@ -284,13 +307,14 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
       bool um = tree_mask != nullptr;
       int ts = ctx - nq;
       unsigned long long a0 = mk[0], a1 = mk[1];
-      if (window > 0 && !um) {                         // lower bound of each row as a visibility set over this warp's keys
-        const int lo0 = lim[0] - window + 1 - key0, lo1 = lim[1] - window + 1 - key0;
+      if ((window > 0 || chunk > 0) && !um) {          // lower bound of each row as a visibility set over this warp's keys
+        const int lo0 = first_visible(lim[0], window, chunk) - key0, lo1 = first_visible(lim[1], window, chunk) - key0;
         um = true; ts = key0;
         a0 = lo0 <= 0 ? ~0ull : (lo0 >= 64 ? 0ull : (~0ull << lo0));
         a1 = lo1 <= 0 ? ~0ull : (lo1 >= 64 ? 0ull : (~0ull << lo1));
       }
-      warp_tile<KPW / 8>(qf, st, sk, sk + PAGE * HD * 2, warp * KPW, key0, lim[0], lim[1], um, ts, a0, a1, scale_log2);
+      warp_tile<KPW / 8>(qf, st, sk, sk + PAGE * HD * 2, warp * KPW, key0, lim[0], lim[1], um, ts, a0, a1, scale_log2,
+                         kd, vd);
     }
     __syncthreads();
   }
@@ -322,14 +346,15 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 #pragma unroll
     for (int w = 0; w < NW; ++w) { sc[w] = exp2f(sml[(w * 16 + r) * 2] - M); L += sml[(w * 16 + r) * 2 + 1] * sc[w]; }
     const int qi = rg / G, hh = kvh * G + rg % G;
-    for (int d = threadIdx.x; d < HD; d += 32 * NW) {
+    for (int d = threadIdx.x; d < f.dv; d += 32 * NW) {
       float acc = 0.f;
 #pragma unroll
       for (int w = 0; w < NW; ++w) acc += so[(w * 16 + r) * HD + d] * sc[w];
       if (nsplit == 1 && pstride == 0) {
         // learnable soft-max: the head's sink logit enters the denominator only
         const float Ls = sinks ? L + exp2f(sinks[hh] * 1.4426950408889634f - M) : L;
-        out[((size_t)(b * nq + qi) * hq + hh) * HD + d] = __float2bfloat16(Ls > 0.f ? acc / Ls : 0.f);
+        const float gf = gate_factor(f.gate, f.ldg, (size_t)(b * nq + qi), hh * f.dv + d);
+        out[((size_t)(b * nq + qi) * hq + hh) * f.dv + d] = __float2bfloat16(Ls > 0.f ? acc / Ls * gf : 0.f);
       } else {
         const size_t pr = ((size_t)b * (pstride ? pstride : nsplit) + split) * (nq * hq) + (size_t)qi * hq + hh;
         part_o[pr * HD + d] = acc;
@@ -359,7 +384,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
         const size_t row = (size_t)qi * hq + hh;
         float M = NEG_BIG;
         for (int sp = 0; sp < nsplit; ++sp) M = fmaxf(M, __ldcg(&part_ml[(((size_t)b * nsplit + sp) * (nq * hq) + row) * 2]));
-        for (int d = threadIdx.x; d < HD; d += 32 * NW) {
+        for (int d = threadIdx.x; d < f.dv; d += 32 * NW) {
           float L = 0.f, acc = 0.f;
           for (int sp = 0; sp < nsplit; ++sp) {
             const size_t pr = ((size_t)b * nsplit + sp) * (nq * hq) + row;
@@ -368,7 +393,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
             acc += __ldcg(&part_o[pr * HD + d]) * sc;
           }
           if (sinks) L += exp2f(sinks[hh] * 1.4426950408889634f - M);
-          out[((size_t)(b * nq + qi) * hq + hh) * HD + d] = __float2bfloat16(L > 0.f ? acc / L : 0.f);
+          const float gf = gate_factor(f.gate, f.ldg, (size_t)(b * nq + qi), hh * f.dv + d);
+          out[((size_t)(b * nq + qi) * hq + hh) * f.dv + d] = __float2bfloat16(L > 0.f ? acc / L * gf : 0.f);
         }
       }
     }
@@ -378,10 +404,12 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 // grid (B * nq * hq), 128 threads
 __global__ void __launch_bounds__(128)
 attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out,
-                  int rows_per_seq, int nsplit, const float* __restrict__ sinks, int hq) {
+                  int rows_per_seq, int nsplit, const float* __restrict__ sinks, int hq, int dv, const __nv_bfloat16* __restrict__ gate,
+                  int ldg) {
   pdl_trigger();
   pdl_wait();
   const int row = blockIdx.x, b = row / rows_per_seq, r = row % rows_per_seq, d = threadIdx.x;
+  if (d >= dv) return;
   float M = NEG_BIG;
   for (int s = 0; s < nsplit; ++s) M = fmaxf(M, part_ml[(((size_t)b * nsplit + s) * rows_per_seq + r) * 2]);
   float L = 0.f, acc = 0.f;
@@ -392,7 +420,8 @@ attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ pa
     acc += part_o[pr * HD + d] * sc;
   }
   if (sinks) L += exp2f(sinks[r % hq] * 1.4426950408889634f - M);
-  out[(size_t)row * HD + d] = __float2bfloat16(L > 0.f ? acc / L : 0.f);
+  const float gf = gate_factor(gate, ldg, (size_t)(row / hq), (row % hq) * dv + d);
+  out[(size_t)row * dv + d] = __float2bfloat16(L > 0.f ? acc / L * gf : 0.f);
 }
 
 // ---------------------------------------------------------------------------------------
@@ -518,8 +547,10 @@ static int attn_decode_launch(const void* q, const void* kcache, const void* vca
                               const int* ctx_lens, const unsigned long long* tree_mask, void* out, float* part_o,
                               float* part_ml, int batch, int hq, int hkv, int head_dim, int nq, int ldq, int max_blocks,
                               int num_blocks, int nsplit, float scale, int* split_counters, int* status, cudaStream_t s,
-                              int window, const int* kv_start = nullptr, int pstride = 0, const float* sinks = nullptr) {
-  if (window > 0 && tree_mask) return FF_HOST_UNSUPPORTED;
+                              const DecodeForm& f, const int* kv_start = nullptr, int pstride = 0, const float* sinks = nullptr) {
+  if ((f.window > 0 || f.chunk > 0) && tree_mask) return FF_HOST_UNSUPPORTED;
+  if (f.window > 0 && f.chunk > 0) return FF_HOST_UNSUPPORTED;
+  if (f.dk < 16 || f.dk > HD || f.dk % 16 || f.dv < 16 || f.dv > HD || f.dv % 16) return FF_HOST_BAD_SHAPE;
   if (pstride != 0 && (pstride < nsplit || !part_o || !part_ml)) return FF_HOST_BAD_SHAPE;
   if (head_dim != HD || batch <= 0 || hq <= 0 || hkv <= 0 || hq % hkv) return FF_HOST_BAD_SHAPE;
   if (nq < 1 || nq > 64) return FF_HOST_BAD_SHAPE;
@@ -533,15 +564,15 @@ static int attn_decode_launch(const void* q, const void* kcache, const void* vca
   // the caches as [blocks * hkv * 64 rows][128]; a box is one half (64 dims) of one page of one head
   CUtensorMap tmK, tmV;
   const uint64_t cache_rows = (uint64_t)num_blocks * hkv * PAGE;
-  if (int r = make_tmap_2d(&tmK, kcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, HD, cache_rows, HD * 2, 64, PAGE)) return r;
-  if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, HD, cache_rows, HD * 2, 64, PAGE)) return r;
+  if (int r = make_tmap_2d(&tmK, kcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, f.dk, cache_rows, f.dk * 2, 64, PAGE)) return r;
+  if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, f.dv, cache_rows, f.dv * 2, 64, PAGE)) return r;
   if (int lr_ = launch_pdl(attn_decode_kernel<NW>, dim3(grid), dim3(32 * NW), DEC_SMEM, s, 0, tmK, tmV, (const __nv_bfloat16*)q,
       block_table, ctx_lens, tree_mask, (__nv_bfloat16*)out, part_o, part_ml, hq, hkv, nq,
-      ldq, max_blocks, num_blocks, nsplit, scale_log2, status, split_counters, window, kv_start, pstride, sinks)) return lr_;
+      ldq, max_blocks, num_blocks, nsplit, scale_log2, status, split_counters, f, kv_start, pstride, sinks)) return lr_;
   if (int r = launch_result()) return r;
   if (pstride != 0) return 0;                      // partials only: the caller merges after the other kernel has added its own
   if (nsplit > 1 && split_counters == nullptr) {
-    if (int lr_ = launch_pdl(attn_merge_kernel, dim3(batch * nq * hq), dim3(128), 0, s, 0, part_o, part_ml, (__nv_bfloat16*)out, nq * hq, nsplit, sinks, hq)) return lr_;
+    if (int lr_ = launch_pdl(attn_merge_kernel, dim3(batch * nq * hq), dim3(128), 0, s, 0, part_o, part_ml, (__nv_bfloat16*)out, nq * hq, nsplit, sinks, hq, f.dv, f.gate, f.ldg)) return lr_;
     return launch_result();
   }
   return 0;
@@ -552,7 +583,8 @@ FF_EXPORT int ff_attn_decode(const void* q, const void* kcache, const void* vcac
                              float* part_ml, int batch, int hq, int hkv, int head_dim, int nq, int ldq, int max_blocks,
                              int num_blocks, int nsplit, float scale, int* split_counters, int* status, cudaStream_t s) {
   return attn_decode_launch(q, kcache, vcache, block_table, ctx_lens, tree_mask, out, part_o, part_ml, batch, hq, hkv,
-                            head_dim, nq, ldq, max_blocks, num_blocks, nsplit, scale, split_counters, status, s, 0);
+                            head_dim, nq, ldq, max_blocks, num_blocks, nsplit, scale, split_counters, status, s,
+                            DecodeForm{0, 0, HD, HD, 0, nullptr});
 }
 
 // BF16 part of a decode step over a cache whose older keys are sealed in the 8-bit store: visits the pages from
@@ -564,7 +596,8 @@ FF_EXPORT int ff_attn_decode_partial(const void* q, const void* kcache, const vo
                                      int pstride, float scale, int* status, cudaStream_t s) {
   if (!kv_start || pstride < 1) return FF_HOST_BAD_SHAPE;
   return attn_decode_launch(q, kcache, vcache, block_table, ctx_lens, nullptr, nullptr, part_o, part_ml, batch, hq, hkv,
-                            head_dim, 1, ldq, max_blocks, num_blocks, nsplit, scale, nullptr, status, s, 0, kv_start, pstride);
+                            head_dim, 1, ldq, max_blocks, num_blocks, nsplit, scale, nullptr, status, s,
+                            DecodeForm{0, 0, HD, HD, 0, nullptr}, kv_start, pstride);
 }
 
 // Merge `nsplit` partials per (sequence row, head) into out [rows * hq, 128] bf16.
@@ -572,7 +605,8 @@ FF_EXPORT int ff_attn_merge(const float* part_o, const float* part_ml, void* out
                             cudaStream_t s) {
   if (batch <= 0 || rows_per_seq <= 0 || nsplit < 1) return FF_HOST_BAD_SHAPE;
   if (int lr_ = launch_pdl(attn_merge_kernel, dim3(batch * rows_per_seq), dim3(128), 0, s, 0, part_o, part_ml,
-                           (__nv_bfloat16*)out, rows_per_seq, nsplit, (const float*)nullptr, rows_per_seq)) return lr_;
+                           (__nv_bfloat16*)out, rows_per_seq, nsplit, (const float*)nullptr, rows_per_seq, HD,
+                           (const __nv_bfloat16*)nullptr, 0)) return lr_;
   return launch_result();
 }
 
@@ -584,8 +618,21 @@ FF_EXPORT int ff_attn_decode_sink(const void* q, const void* kcache, const void*
                                   float scale, int window, const float* sinks, int* status, cudaStream_t s) {
   if (window < 0 || sinks == nullptr) return FF_HOST_BAD_SHAPE;
   return attn_decode_launch(q, kcache, vcache, block_table, ctx_lens, nullptr, out, part_o, part_ml, batch, hq, hkv,
-                            head_dim, nq, ldq, max_blocks, num_blocks, nsplit, scale, nullptr, status, s, window, nullptr, 0,
-                            sinks);
+                            head_dim, nq, ldq, max_blocks, num_blocks, nsplit, scale, nullptr, status, s,
+                            DecodeForm{window, 0, HD, HD, 0, nullptr}, nullptr, 0, sinks);
+}
+
+// Decode attention in its general form: key heads of dk and value heads of dv elements (multiples of 16, at most 128; the
+// cache rows and the head pitch of q are dk wide, output heads dv wide), optional window or block-local mask (chunk), sinks
+// and output gate. The partials of a split launch keep 128 floats per row.
+FF_EXPORT int ff_attn_decode_general(const void* q, const void* kcache, const void* vcache, const int* block_table,
+                                     const int* ctx_lens, void* out, float* part_o, float* part_ml, int batch, int hq, int hkv, int dk,
+                                     int dv, int nq, int ldq, int max_blocks, int num_blocks, int nsplit, float scale, int window,
+                                     int chunk, const float* sinks, const void* gate, int ldg, int* status, cudaStream_t s) {
+  if (window < 0 || chunk < 0) return FF_HOST_BAD_SHAPE;
+  return attn_decode_launch(q, kcache, vcache, block_table, ctx_lens, nullptr, out, part_o, part_ml, batch, hq, hkv, HD, nq, ldq, max_blocks,
+                            num_blocks, nsplit, scale, nullptr, status, s,
+                            DecodeForm{window, chunk, dk, dv, ldg, (const __nv_bfloat16*)gate}, nullptr, 0, sinks);
 }
 
 // Decode attention of a local-attention layer: every query sees its last `window` keys.
@@ -595,7 +642,8 @@ FF_EXPORT int ff_attn_decode_window(const void* q, const void* kcache, const voi
                                     float scale, int window, int* split_counters, int* status, cudaStream_t s) {
   if (window <= 0) return FF_HOST_BAD_SHAPE;
   return attn_decode_launch(q, kcache, vcache, block_table, ctx_lens, nullptr, out, part_o, part_ml, batch, hq, hkv,
-                            head_dim, nq, ldq, max_blocks, num_blocks, nsplit, scale, split_counters, status, s, window);
+                            head_dim, nq, ldq, max_blocks, num_blocks, nsplit, scale, split_counters, status, s,
+                            DecodeForm{window, 0, HD, HD, 0, nullptr});
 }
 
 // window > 0: sliding window (exact); 0: causal; < 0: bidirectional (every query sees all ctx keys:

@@ -1,5 +1,5 @@
-// Prefill attention on 5th-generation tensor cores: paged KV, 128-dim heads, GQA, causal / sliding-window /
-// bidirectional masks, chunked prefill (query rows are the last q_len positions of a context of ctx_len).
+// Prefill attention on 5th-generation tensor cores: paged KV, heads of up to 128 elements, GQA, causal / sliding-window /
+// block-local / bidirectional masks, optional output gate, chunked prefill (query rows are the last q_len positions of a context of ctx_len).
 //
 // One CTA per (sequence, query head, tile of 128 query rows). Both contractions run as tcgen05.mma with
 // FP32 accumulators in tensor memory:
@@ -356,10 +356,40 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 // warp per lane quadrant, a thread owning a row). Q K(j+1)ᵀ is issued as soon as its K page is there, i.e. while the
 // softmax warps are still on tile j; P V(j) runs while they are on tile j + 1; only the rare rescale of O waits for the
 // previous P V. FF_ATTN_PREFILL_SPLIT=2 puts two softmax warps on every lane quadrant (32 columns each).
+// Key heads of dk and value heads of dv elements (multiples of 16): Q Kᵀ runs dk / 16 steps, P V covers 64 or 128 columns;
+// TMA fills the columns of a box that lie past the head with zeros.
 // ------------------------------------------------------------------------------------------------
 constexpr int T2_BN = 64;                                          // keys per tile = one cache page
 constexpr int T2_KV_BYTES = T2_BN * TC_HD * 2;                     // 16 KiB
 constexpr int TC2_SMEM = TC_Q_BYTES + 4 * T2_KV_BYTES + 1024;      // 97 KiB
+
+// what a launch adds to plain causal attention over 128-wide heads
+struct PrefillForm {
+  int window, chunk, causal, dk, dv, ldg;
+  const __nv_bfloat16* gate;       // [rows, hq * dv]: the result is multiplied by its sigmoid
+};
+
+// o * inv, times the sigmoid of the gate where there is one; 16 columns, two 16-byte stores
+__device__ __forceinline__ void store_o16(__nv_bfloat16* dst, const uint32_t* r, float inv, const __nv_bfloat16* gate) {
+  float v[16];
+#pragma unroll
+  for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]) * inv;
+  if (gate != nullptr) {
+    const uint4 g0 = reinterpret_cast<const uint4*>(gate)[0], g1 = reinterpret_cast<const uint4*>(gate)[1];
+    const uint32_t gw[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float2 g = unpack_bf16x2(gw[i]);
+      v[2 * i] *= 1.0f / (1.0f + __expf(-g.x));
+      v[2 * i + 1] *= 1.0f / (1.0f + __expf(-g.y));
+    }
+  }
+  uint32_t o[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) o[i] = pack_bf16x2(v[2 * i], v[2 * i + 1]);
+  reinterpret_cast<uint4*>(dst)[0] = make_uint4(o[0], o[1], o[2], o[3]);
+  reinterpret_cast<uint4*>(dst)[1] = make_uint4(o[4], o[5], o[6], o[7]);
+}
 
 struct alignas(8) Tc2Bars {
   uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], pv_done[2];
@@ -374,7 +404,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
                         const __grid_constant__ CUtensorMap tmV, const int* __restrict__ block_table,
                         const int* __restrict__ q_start, const int* __restrict__ q_lens,
                         const int* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out, int hq, int hkv, int ldo,
-                        int max_blocks, int num_blocks, float scale_log2, int window, int causal, int* status,
+                        int max_blocks, int num_blocks, float scale_log2, const PrefillForm f, int* status,
                         const float* __restrict__ sinks) {
   const int b = blockIdx.z, h = blockIdx.y;
   const int qlen = q_lens[b];
@@ -390,8 +420,11 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   const int kvh = h / (hq / hkv);
   const int past = ctx - qlen;
   const int real = min(TC_BM, qlen - r0);
+  const int causal = f.causal, window = f.window, chunk = f.chunk, dk = f.dk, dv = f.dv;
+  const bool k_hi = dk > 64, v_hi = dv > 64;                       // heads up to 64 wide: the upper 64 columns are not loaded
+  auto first_visible = [&](int pos) { return window > 0 ? max(0, pos - window + 1) : (chunk > 0 ? pos / chunk * chunk : 0); };
   const int last_key = causal ? past + r0 + real - 1 : ctx - 1;
-  const int first_key = window > 0 ? max(0, past + r0 - window + 1) : 0;
+  const int first_key = first_visible(past + r0);
   const int t0 = first_key / T2_BN, t1 = last_key / T2_BN + 1;
   const int ntiles = t1 - t0;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -416,9 +449,9 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 
   if (warp == 0) {
     if (lane == 0) {
-      mbar_expect_tx(&bars.q_full, TC_Q_BYTES);
-      tma_load_2d(sQ, &tmQ, &bars.q_full, h * TC_HD, qs + r0);
-      tma_load_2d(sQ + TC_BM * 128, &tmQ, &bars.q_full, h * TC_HD + 64, qs + r0);
+      mbar_expect_tx(&bars.q_full, k_hi ? TC_Q_BYTES : TC_Q_BYTES / 2);
+      tma_load_2d(sQ, &tmQ, &bars.q_full, h * dk, qs + r0);
+      if (k_hi) tma_load_2d(sQ + TC_BM * 128, &tmQ, &bars.q_full, h * dk + 64, qs + r0);
       bool ok = true, bad = false;
       const int nblk = (ctx + TC_PAGE - 1) / TC_PAGE;
       auto tile_row = [&](int j) -> int {
@@ -434,9 +467,9 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
         const int row = tile_row(j);
         if (!mbar_wait(&bars.k_empty[st], ph ^ 1, abort_flag, status, KID_ATTN_PREFILL, 21)) return false;
-        mbar_expect_tx(&bars.k_full[st], T2_KV_BYTES);
+        mbar_expect_tx(&bars.k_full[st], k_hi ? T2_KV_BYTES : T2_KV_BYTES / 2);
         tma_load_2d(sK + st * T2_KV_BYTES, &tmK, &bars.k_full[st], 0, row);
-        tma_load_2d(sK + st * T2_KV_BYTES + 8192, &tmK, &bars.k_full[st], 64, row);
+        if (k_hi) tma_load_2d(sK + st * T2_KV_BYTES + 8192, &tmK, &bars.k_full[st], 64, row);
         return true;
       };
       ok = load_k(0);
@@ -445,16 +478,17 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
         const int row = tile_row(j);
         if (!mbar_wait(&bars.v_empty[st], ph ^ 1, abort_flag, status, KID_ATTN_PREFILL, 22)) { ok = false; break; }
-        mbar_expect_tx(&bars.v_full[st], T2_KV_BYTES);
+        mbar_expect_tx(&bars.v_full[st], v_hi ? T2_KV_BYTES : T2_KV_BYTES / 2);
         tma_load_2d(sV + st * T2_KV_BYTES, &tmV, &bars.v_full[st], 0, row);
-        tma_load_2d(sV + st * T2_KV_BYTES + 8192, &tmV, &bars.v_full[st], 64, row);
+        if (v_hi) tma_load_2d(sV + st * T2_KV_BYTES + 8192, &tmV, &bars.v_full[st], 64, row);
       }
       if (bad) set_status(status, KID_ATTN_PREFILL, FF_ERR_BOUNDS, b, r0 / TC_BM);
     }
   } else if (warp == 1) {
     if (lane == 0) {
       const uint32_t idesc_s = umma_idesc(1, 1, 0, 0, TC_BM, T2_BN);
-      const uint32_t idesc_o = umma_idesc(1, 1, 0, 1, TC_BM, TC_HD);
+      const uint32_t idesc_o = umma_idesc(1, 1, 0, 1, TC_BM, v_hi ? TC_HD : TC_HD / 2);
+      const int ksteps = dk >> 4;
       const uint32_t q_addr = smem_u32(sQ);
       bool ok = mbar_wait(&bars.q_full, 0, abort_flag, status, KID_ATTN_PREFILL, 23);
       auto issue_s = [&](int j) -> bool {
@@ -466,6 +500,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         const uint32_t k_addr = smem_u32(sK + st * T2_KV_BYTES);
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
+          if (k >= ksteps) break;
           // Q: 64-column block k / 4 of a 128-row tile (16 KiB), 32 bytes per k-step; K: the same with 64 rows (8 KiB)
           umma_f16(tmem_s + st * T2_BN, umma_desc_sw128(q_addr + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024),
                    umma_desc_sw128(k_addr + (k >> 2) * 8192 + (k & 3) * 32, 16, 1024), idesc_s, k != 0);
@@ -501,12 +536,12 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     const bool live = row < real;
     const int pos = past + r0 + row;
     const int hi = live ? (causal ? pos : ctx - 1) : -1;
-    const int lo = (live && window > 0) ? max(0, pos - window + 1) : 0;
+    const int lo = live ? first_visible(pos) : 0;
     float m_ref = -INFINITY, l_sum = 0.f;
     bool ok = true;
     const uint32_t lane_base = (uint32_t(q * 32) << 16);
     const int tile_hi_min = causal ? past + r0 : ctx - 1;
-    const int tile_lo_max = window > 0 ? max(0, past + r0 + real - window) : 0;
+    const int tile_lo_max = first_visible(past + r0 + real - 1);
     for (int j = 0; j < ntiles; ++j) {
       const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
       if (ok && !mbar_wait(&bars.s_full[st], ph, abort_flag, status, KID_ATTN_PREFILL, 28)) ok = false;
@@ -561,6 +596,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
           tc_fence_after();
 #pragma unroll
           for (int c = 0; c < TC_HD / SPLIT; c += 16) {
+            if (hf * (TC_HD / SPLIT) + c >= dv) break;
             uint32_t r[16];
             tmem_ld_x16(tmem_o + lane_base + hf * (TC_HD / SPLIT) + c, r);
             tmem_ld_wait();
@@ -609,25 +645,15 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       tc_fence_after();
       if (sinks != nullptr) l_sum += (m_ref == -INFINITY) ? 1.f : exp2f(sinks[h] * 1.4426950408889634f - m_ref);
       const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
-      __nv_bfloat16* orow = out + (size_t)(qs + r0 + row) * ldo + (size_t)h * TC_HD + hf * (TC_HD / SPLIT);
+      __nv_bfloat16* orow = out + (size_t)(qs + r0 + row) * ldo + (size_t)h * dv + hf * (TC_HD / SPLIT);
+      const __nv_bfloat16* grow = f.gate == nullptr ? nullptr : f.gate + (size_t)(qs + r0 + row) * f.ldg + (size_t)h * dv + hf * (TC_HD / SPLIT);
 #pragma unroll
       for (int c = 0; c < TC_HD / SPLIT; c += 16) {
+        if (hf * (TC_HD / SPLIT) + c >= dv) break;
         uint32_t r[16];
         tmem_ld_x16(tmem_o + lane_base + hf * (TC_HD / SPLIT) + c, r);
         tmem_ld_wait();
-        if (live) {
-          uint4 o0, o1;
-          o0.x = pack_bf16x2(__uint_as_float(r[0]) * inv, __uint_as_float(r[1]) * inv);
-          o0.y = pack_bf16x2(__uint_as_float(r[2]) * inv, __uint_as_float(r[3]) * inv);
-          o0.z = pack_bf16x2(__uint_as_float(r[4]) * inv, __uint_as_float(r[5]) * inv);
-          o0.w = pack_bf16x2(__uint_as_float(r[6]) * inv, __uint_as_float(r[7]) * inv);
-          o1.x = pack_bf16x2(__uint_as_float(r[8]) * inv, __uint_as_float(r[9]) * inv);
-          o1.y = pack_bf16x2(__uint_as_float(r[10]) * inv, __uint_as_float(r[11]) * inv);
-          o1.z = pack_bf16x2(__uint_as_float(r[12]) * inv, __uint_as_float(r[13]) * inv);
-          o1.w = pack_bf16x2(__uint_as_float(r[14]) * inv, __uint_as_float(r[15]) * inv);
-          *reinterpret_cast<uint4*>(orow + c) = o0;
-          *reinterpret_cast<uint4*>(orow + c + 8) = o1;
-        }
+        if (live) store_o16(orow + c, r, inv, grow == nullptr ? nullptr : grow + c);
       }
     }
   }
@@ -643,47 +669,51 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 }  // namespace ff
 using namespace ff;
 
-// Same contract as ff_attn_prefill (attention_paged.cu). q: packed rows [rows, ldq] with head h at columns h*128;
-// out rows 16-byte aligned (ldo % 8 == 0). window > 0 sliding, 0 causal, < 0 bidirectional.
+// Same contract as ff_attn_prefill (attention_paged.cu). q: packed rows [rows, ldq] with head h at columns h*dk;
+// out rows 16-byte aligned (ldo % 8 == 0). window > 0 sliding, 0 causal, < 0 bidirectional; chunk > 0: a query sees the keys
+// of its own block of `chunk` positions that are not after it. dk / dv: widths of the key and value heads (multiples of 16,
+// at most 128). gate: optional [rows, hq * dv] with row pitch ldg, 16-byte aligned.
 FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* vcache, const int* block_table,
                                  const int* q_start, const int* q_lens, const int* ctx_lens, void* out, int batch,
-                                 int total_rows, int max_q_len, int hq, int hkv, int head_dim, int ldq, int ldo,
-                                 int max_blocks, int num_blocks, float scale, int window, const float* sinks, int* status,
-                                 cudaStream_t s) {
-  if (head_dim != TC_HD || batch <= 0 || max_q_len <= 0 || hq <= 0 || hkv <= 0 || hq % hkv || total_rows <= 0) return FF_HOST_BAD_SHAPE;
+                                 int total_rows, int max_q_len, int hq, int hkv, int dk, int dv, int ldq, int ldo,
+                                 int max_blocks, int num_blocks, float scale, int window, int chunk, const float* sinks,
+                                 const void* gate, int ldg, int* status, cudaStream_t s) {
+  if (batch <= 0 || max_q_len <= 0 || hq <= 0 || hkv <= 0 || hq % hkv || total_rows <= 0) return FF_HOST_BAD_SHAPE;
+  if (dk < 16 || dk > TC_HD || dk % 16 || dv < 16 || dv > TC_HD || dv % 16 || chunk < 0 || !(scale > 0.f)) return FF_HOST_BAD_SHAPE;
+  if (chunk > 0 && window != 0) return FF_HOST_UNSUPPORTED;
   if (ldq % 8 || ldo % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return FF_HOST_BAD_ALIGN;
+  if (gate != nullptr && (ldg % 8 || (reinterpret_cast<uintptr_t>(gate) & 15))) return FF_HOST_BAD_ALIGN;
   CUtensorMap tmQ, tmK, tmV;
   if (int r = make_tmap_2d(&tmQ, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)ldq, (uint64_t)total_rows,
                            (uint64_t)ldq * 2, 64, TC_BM)) return r;
   const uint64_t cache_rows = (uint64_t)num_blocks * hkv * TC_PAGE;
-  if (int r = make_tmap_2d(&tmK, kcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, TC_HD, cache_rows, TC_HD * 2, 64, TC_PAGE)) return r;
-  if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, TC_HD, cache_rows, TC_HD * 2, 64, TC_PAGE)) return r;
+  if (int r = make_tmap_2d(&tmK, kcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dk, cache_rows, dk * 2, 64, TC_PAGE)) return r;
+  if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dv, cache_rows, dv * 2, 64, TC_PAGE)) return r;
   const float scale_log2 = scale * 1.4426950408889634f;
   dim3 grid((max_q_len + TC_BM - 1) / TC_BM, hq, batch);
-  // FF_ATTN_PREFILL_CTAS = 1 selects the one-CTA-per-SM kernel (deep K / V rings, eight softmax warps); the default is the
-  // two-CTAs-per-SM kernel
+  const PrefillForm f = {window < 0 ? 0 : window, chunk, window < 0 ? 0 : 1, dk, dv, ldg, (const __nv_bfloat16*)gate};
+  // FF_ATTN_PREFILL_CTAS = 1 selects the one-CTA-per-SM kernel (deep K / V rings, eight softmax warps; plain 128-wide heads
+  // only); the default is the two-CTAs-per-SM kernel
   static int two = -1;
   if (two < 0) { const char* e = getenv("FF_ATTN_PREFILL_CTAS"); two = (e != nullptr && e[0] == '1') ? 0 : TC_TWO_CTAS_DEFAULT; }
-  if (two) {
+  if (two || chunk > 0 || gate != nullptr || dk != TC_HD || dv != TC_HD) {
     // FF_ATTN_PREFILL_SPLIT = 2: two softmax warps per lane quadrant (64 columns each) instead of one
     static int split = -1;
     if (split < 0) { const char* e = getenv("FF_ATTN_PREFILL_SPLIT"); split = (e != nullptr && (e[0] == '1' || e[0] == '2')) ? e[0] - '0' : TC2_SPLIT_DEFAULT; }
     if (split == 2) {
       if (int r = opt_in_smem(attn_prefill_tc2_kernel<2>, TC2_SMEM)) return r;
-      attn_prefill_tc2_kernel<2><<<grid, 320, TC2_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens,
-                                                             (__nv_bfloat16*)out, hq, hkv, ldo, max_blocks, num_blocks, scale_log2,
-                                                             window < 0 ? 0 : window, window < 0 ? 0 : 1, status, sinks);
+      attn_prefill_tc2_kernel<2><<<grid, 320, TC2_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out,
+                                                             hq, hkv, ldo, max_blocks, num_blocks, scale_log2, f, status, sinks);
       return launch_result();
     }
     if (int r = opt_in_smem(attn_prefill_tc2_kernel<1>, TC2_SMEM)) return r;
-    attn_prefill_tc2_kernel<1><<<grid, 192, TC2_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens,
-                                                           (__nv_bfloat16*)out, hq, hkv, ldo, max_blocks, num_blocks, scale_log2,
-                                                           window < 0 ? 0 : window, window < 0 ? 0 : 1, status, sinks);
+    attn_prefill_tc2_kernel<1><<<grid, 192, TC2_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out,
+                                                           hq, hkv, ldo, max_blocks, num_blocks, scale_log2, f, status, sinks);
     return launch_result();
   }
   if (int r = opt_in_smem(attn_prefill_tc_kernel, TC_SMEM)) return r;
   attn_prefill_tc_kernel<<<grid, 320, TC_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens,
                                                     (__nv_bfloat16*)out, hq, hkv, ldo, max_blocks, num_blocks, scale_log2,
-                                                    window < 0 ? 0 : window, window < 0 ? 0 : 1, status, sinks);
+                                                    f.window, f.causal, status, sinks);
   return launch_result();
 }

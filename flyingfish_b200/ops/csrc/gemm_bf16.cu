@@ -118,6 +118,10 @@ __device__ __forceinline__ int comm_tm(int tm, int tiles_per_rank, int rank, int
   return ((rank + j) % world) * tiles_per_rank + r;
 }
 
+// Optional tail of the plain BF16 store (epi 0): bias per output column, then act 1 = square of the positive part. Both work
+// on the FP32 accumulator; the result is rounded once.
+struct LinTail { const __nv_bfloat16* bias; int act; };
+
 constexpr int RS_STG_PITCH = 144, RS_STG_BYTES = 32 * RS_STG_PITCH;   // COMM 2 epilogue staging, per warp
 constexpr int COMM_PARTS = 4;       // a 128-row block is pushed (COMM 1) / reduced (COMM 2) in this many pieces
 
@@ -125,7 +129,7 @@ template <int BN, int STAGES, int COMM>
 __global__ void __launch_bounds__(COMM == 1 ? 320 : 192, 1)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmA1,
                  const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmB, void* __restrict__ Cout, int M, int N, int K, int ldc, int epi,
-                 int* status, CommArgs ca, GroupArgs ga) {
+                 int* status, CommArgs ca, GroupArgs ga, LinTail tail) {
   extern __shared__ uint8_t smem_raw[];
   __shared__ PipeBars bars;
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -332,6 +336,30 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           uint32_t r[32];
           tmem_ld_x32(taddr + c, r);
           tmem_ld_wait();
+          if (COMM == 0 && tail.bias != nullptr) {
+            const int col = tn * BN + c;
+            if (col + 32 <= N) {
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                const uint4 bv = __ldg(reinterpret_cast<const uint4*>(tail.bias + col) + j);
+                const uint32_t bw[4] = {bv.x, bv.y, bv.z, bv.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                  const float2 f = unpack_bf16x2(bw[i]);
+                  r[8 * j + 2 * i] = __float_as_uint(__uint_as_float(r[8 * j + 2 * i]) + f.x);
+                  r[8 * j + 2 * i + 1] = __float_as_uint(__uint_as_float(r[8 * j + 2 * i + 1]) + f.y);
+                }
+              }
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (col + j < N) r[j] = __float_as_uint(__uint_as_float(r[j]) + __bfloat162float(tail.bias[col + j]));
+            }
+          }
+          if (COMM == 0 && tail.act == 1) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) { const float v = fmaxf(__uint_as_float(r[j]), 0.f); r[j] = __float_as_uint(v * v); }
+          }
           if (row < row_end) {
             if (tn * BN + c + 32 <= N) {
               uint4* dst = reinterpret_cast<uint4*>(crow + c);
@@ -488,8 +516,8 @@ using namespace ff;
 
 // Y[M,N] = X[M,K] · W[N,K]ᵀ. epi: 0 bf16 out, 1 fused SwiGLU (out has N/2 columns), 2 fp32 out.
 // ldx / ldw / ldy in elements. Returns 0 or an error code (see host_util.h).
-FF_EXPORT int ff_gemm_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
-                           int epi, int* status, cudaStream_t stream) {
+static int gemm_bf16_launch(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
+                            int epi, LinTail tail, int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return FF_HOST_BAD_SHAPE;
   if ((K % 8) || (ldx % 8) || (ldw % 8)) return FF_HOST_BAD_ALIGN;
   if (epi == 1 && (N % 256)) return FF_HOST_BAD_SHAPE;
@@ -509,8 +537,21 @@ FF_EXPORT int ff_gemm_bf16(const void* X, const void* W, void* Y, int M, int N, 
   const int tiles = ((M + BM - 1) / BM) * ((N + BN - 1) / BN);
   const int grid = tiles < sm_count() ? tiles : sm_count();
   CommArgs none = {};
-  kern<<<grid, 192, smem, stream>>>(tmA, tmA, tmA, tmB, Y, M, N, K, ldy, epi, status, none, GroupArgs{});
+  kern<<<grid, 192, smem, stream>>>(tmA, tmA, tmA, tmB, Y, M, N, K, ldy, epi, status, none, GroupArgs{}, tail);
   return launch_result();
+}
+
+FF_EXPORT int ff_gemm_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
+                           int epi, int* status, cudaStream_t stream) {
+  return gemm_bf16_launch(X, W, Y, M, N, K, ldx, ldw, ldy, epi, LinTail{nullptr, 0}, status, stream);
+}
+
+// Y = act(X Wᵀ + bias) in BF16. bias: [N] or null; act 0 none, 1 square of the positive part.
+FF_EXPORT int ff_gemm_bf16_act(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
+                               const void* bias, int act, int* status, cudaStream_t stream) {
+  if ((unsigned)act > 1u) return FF_HOST_UNSUPPORTED;
+  if (reinterpret_cast<uintptr_t>(bias) & 15) return FF_HOST_BAD_ALIGN;
+  return gemm_bf16_launch(X, W, Y, M, N, K, ldx, ldw, ldy, 0, LinTail{static_cast<const __nv_bfloat16*>(bias), act}, status, stream);
 }
 
 // Grouped GEMM over expert segments with 128-row token tiles (prefill sizes; the swap-AB kernel of moe.cu serves
@@ -534,7 +575,7 @@ FF_EXPORT int ff_moe_grouped_gemm_tiled(const void* Xs, const void* W, void* Y, 
   r = opt_in_smem(kern, smem); if (r) return r;
   CommArgs none = {};
   GroupArgs ga = {seg_off, counts, E_local};
-  kern<<<sm_count(), 192, smem, stream>>>(tmA, tmA, tmA, tmB, Y, capacity, Nw, K, ldy, epi, status, none, ga);
+  kern<<<sm_count(), 192, smem, stream>>>(tmA, tmA, tmA, tmB, Y, capacity, Nw, K, ldy, epi, status, none, ga, LinTail{nullptr, 0});
   return launch_result();
 }
 
@@ -584,7 +625,7 @@ FF_EXPORT int ff_ag_gemm(const unsigned long long* ptrs, int rank, int world, lo
   r = opt_in_smem(kern, smem); if (r) return r;
   const int tiles = (M / BM) * ((N + BN - 1) / BN);
   const int grid = tiles < sm_count() ? tiles : sm_count();
-  kern<<<grid, 320, smem, stream>>>(tmA0, tmA1, tmX, tmB, Y, M, N, K, ldy, epi, status, ca, GroupArgs{});
+  kern<<<grid, 320, smem, stream>>>(tmA0, tmA1, tmX, tmB, Y, M, N, K, ldy, epi, status, ca, GroupArgs{}, LinTail{nullptr, 0});
   return launch_result();
 }
 
@@ -610,7 +651,7 @@ FF_EXPORT int ff_gemm_rs(const unsigned long long* ptrs, int rank, int world, lo
   r = opt_in_smem(kern, smem); if (r) return r;
   const int tiles = (M / BM) * ((N + BN - 1) / BN);
   const int grid = tiles < sm_count() ? tiles : sm_count();
-  kern<<<grid, 192, smem, stream>>>(tmA, tmA, tmA, tmB, nullptr, M, N, K, N, 0, status, ca, GroupArgs{});
+  kern<<<grid, 192, smem, stream>>>(tmA, tmA, tmA, tmB, nullptr, M, N, K, N, 0, status, ca, GroupArgs{}, LinTail{nullptr, 0});
   return launch_result();
 }
 

@@ -52,12 +52,26 @@ struct alignas(8) SkinnyBars {
 template <bool FUSE_AR>
 struct TileSink {
   __nv_bfloat16* Y; int N, ldy; bool vec8;      // vec8: 16-byte stores of eight values are aligned
+  const __nv_bfloat16* bias; int act;           // added to the finished sums; act 1: square of the positive part
   PeerArena ar; int parity;
 
   // eight consecutive columns col..col+7 of token row t (col is a multiple of 8)
-  __device__ __forceinline__ void put8(int t, int col, const float* a) const {
+  __device__ __forceinline__ void put8(int t, int col, const float* sums) const {
     if (col >= N) return;
     uint4 o;
+    float a[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) a[j] = sums[j];
+    if (!FUSE_AR) {
+      if (bias != nullptr) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) if (col + j < N) a[j] += __bfloat162float(bias[col + j]);
+      }
+      if (act == 1) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { const float v = fmaxf(a[j], 0.f); a[j] = v * v; }
+      }
+    }
     o.x = pack_bf16x2(a[0], a[1]); o.y = pack_bf16x2(a[2], a[3]);
     o.z = pack_bf16x2(a[4], a[5]); o.w = pack_bf16x2(a[6], a[7]);
     if (!FUSE_AR) {
@@ -196,7 +210,7 @@ __global__ void __launch_bounds__(192, 2)
 gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW,
                    __nv_bfloat16* __restrict__ Y, int M, int N, int K, int ldy, int ntok, int tile_rows, int stages,
                    int cl_size, int pipe_off, float* __restrict__ scratch, int* __restrict__ counters, int* status,
-                   PeerArena ar, SkinnyEpi ep) {
+                   PeerArena ar, SkinnyEpi ep, const __nv_bfloat16* __restrict__ bias, int act) {
   pdl_trigger();
   if (cl_size > 1) cluster_arrive_relaxed();         // phase A: "this CTA runs" (waited on before the first remote store)
   if (threadIdx.x == 0) FF_TL(status, KID_GEMM_SKINNY, 0);
@@ -317,6 +331,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
     if (FUSE_AR) ar_epoch = ld_volatile(arena_epoch(ar)) + 1;
     TileSink<FUSE_AR> sink;
     sink.Y = Y; sink.N = N; sink.ldy = ldy; sink.ar = ar; sink.parity = ar_epoch & 1;
+    sink.bias = bias; sink.act = act;
     sink.vec8 = FUSE_AR || ((ldy % 8 == 0) && ((reinterpret_cast<uintptr_t>(Y) & 15) == 0));
     uint32_t seg_it = 0; bool ok = true;
     long long u = u0; Segment sg;
@@ -792,7 +807,8 @@ FF_EXPORT int ff_gemm_skinny_plan_epi(int M, int N, int K, int epi, long long* s
 
 static int gemm_skinny_launch(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
                               int grid, float* scratch, int* counters, int* status, cudaStream_t stream,
-                              const PeerArena* arena, const SkinnyEpi* epi = nullptr) {
+                              const PeerArena* arena, const SkinnyEpi* epi = nullptr, const __nv_bfloat16* bias = nullptr,
+                              int act = 0) {
   if (M <= 0 || N <= 0 || K <= 0) return FF_HOST_BAD_SHAPE;
   SkinnyEpi ep = {};
   if (epi != nullptr) {
@@ -826,18 +842,26 @@ static int gemm_skinny_launch(const void* X, const void* W, void* Y, int M, int 
     r = opt_in_smem(kern, SK_SMEM_FULL + 1024); if (r) return r;
     PeerArena none = {};
     return launch_pdl(kern, dim3(grid), dim3(192), smem, stream, cl, tmX, tmW, y, M, N, K, ldy, ntok, cfg.tile_rows,
-                      cfg.stages, cl, cfg.pipe_off, scratch, counters, status, none, ep);
+                      cfg.stages, cl, cfg.pipe_off, scratch, counters, status, none, ep, bias, act);
   }
   auto kern = gemm_skinny_kernel<true>;
   r = opt_in_smem(kern, SK_SMEM_FULL + 1024); if (r) return r;
   return launch_pdl(kern, dim3(grid), dim3(192), smem, stream, cl, tmX, tmW, y, M, N, K, ldy, ntok, cfg.tile_rows,
-                    cfg.stages, cl, cfg.pipe_off, scratch, counters, status, *arena, ep);
+                    cfg.stages, cl, cfg.pipe_off, scratch, counters, status, *arena, ep, bias, act);
 }
 
 // `grid` is the value returned by ff_gemm_skinny_plan for the same problem.
 FF_EXPORT int ff_gemm_skinny(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
                              int grid, float* scratch, int* counters, int* status, cudaStream_t stream) {
   return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr);
+}
+
+// Y = act(X Wᵀ + bias): bias [N] or null, act 0 none, 1 square of the positive part (both on the FP32 sums). `grid` as above.
+FF_EXPORT int ff_gemm_skinny_act(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
+                                 int grid, float* scratch, int* counters, const void* bias, int act, int* status, cudaStream_t stream) {
+  if ((unsigned)act > 1u) return FF_HOST_UNSUPPORTED;
+  return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr, nullptr,
+                            static_cast<const __nv_bfloat16*>(bias), act);
 }
 
 // Gate/up projection with the SwiGLU applied in the epilogue: W is [N, K] with gate/up rows interleaved per

@@ -1,0 +1,110 @@
+// Per-head RMS norm of packed projection rows, value blending, and the paged-cache write (layers without positions; the
+// rotary counterpart is rope_kv_paged in rope_act_sample.cu).
+//   row = [hq query heads | hkv key heads | hkv value heads | ...], heads `dk` / `dv` elements apart of which the first
+//   `dim` count for the norm (the rest is zero padding)
+//   q <- q / rms(q)                      in the row
+//   k <- k / rms(k)                      to its slot of the K cache [block][kv head][block_size][dk]
+//   v <- (1 - mix) v + mix first_v       to its slot of the V cache (first_v: the same token's values of an earlier layer)
+// FP32 arithmetic, BF16 or FP32 storage. A group of G lanes owns one head of one row and keeps it in registers.
+#include "dtype_io.cuh"
+#include "host_util.h"
+
+namespace ff {
+
+constexpr int HN_THREADS = 256;
+constexpr int HN_VECS = 4;              // vectors of 8 elements a lane may hold
+
+template <typename T, int G>
+__global__ void __launch_bounds__(HN_THREADS)
+head_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __restrict__ kcache, T* __restrict__ vcache,
+                    const T* __restrict__ first_v, int rows, int hq, int hkv, int dim, int dk, int dv, int block_size, int num_blocks,
+                    int ld, int ldf, float eps, float mix, int* status) {
+  pdl_trigger();
+  pdl_wait();
+  const int heads = hq + 2 * hkv;
+  const long long item = ((long long)blockIdx.x * HN_THREADS + threadIdx.x) / G;
+  const int gl = threadIdx.x & (G - 1);
+  const bool live = item < (long long)rows * heads;
+  const int row = live ? (int)(item / heads) : 0, head = live ? (int)(item % heads) : 0;
+  const bool is_q = head < hq, is_v = head >= hq + hkv;
+  const int d = is_v ? dv : dk;
+  T* base = qkv + (size_t)row * ld + (is_v ? (size_t)(hq + hkv) * dk + (size_t)(head - hq - hkv) * dv : (size_t)head * dk);
+  float v[HN_VECS][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < HN_VECS; ++i) {
+    const int c = (gl + i * G) * 8;
+    if (live && c < d) {
+      load8(base + c, v[i]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(v[i][j], v[i][j], ss);
+    }
+  }
+#pragma unroll
+  for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o, G);
+  if (!live) return;
+  if (!is_v) {
+    const float r = 1.0f / sqrtf(ss / (float)dim + eps);
+#pragma unroll
+    for (int i = 0; i < HN_VECS; ++i)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] *= r;
+  } else if (first_v != nullptr) {
+    const T* fv = first_v + (size_t)row * ldf + (size_t)(head - hq - hkv) * dv;
+#pragma unroll
+    for (int i = 0; i < HN_VECS; ++i) {
+      const int c = (gl + i * G) * 8;
+      if (c < d) {
+        float f[8];
+        load8(fv + c, f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[i][j] = (1.0f - mix) * v[i][j] + mix * f[j];
+      }
+    }
+  }
+  T* dst = base;
+  if (!is_q) {
+    const int slot = slots[row];
+    if (slot < 0) return;                                  // padding row: nothing cached
+    const int blk = slot / block_size, off = slot - blk * block_size;
+    const int kvh = is_v ? head - hq - hkv : head - hq;
+    if (blk >= num_blocks) { if (gl == 0) set_status(status, KID_ROPE_KV, FF_ERR_BOUNDS, row, slot); return; }
+    if (gl == 0) dbg_write_once(status, KID_ROPE_KV, is_v ? DBG_KV_V : DBG_KV_K, (long long)slot * hkv + kvh);
+    dst = (is_v ? vcache : kcache) + (((size_t)blk * hkv + kvh) * block_size + off) * d;
+  }
+#pragma unroll
+  for (int i = 0; i < HN_VECS; ++i) {
+    const int c = (gl + i * G) * 8;
+    if (c < d) store8(dst + c, v[i]);
+  }
+}
+
+template <typename T>
+static int head_norm_launch(void* qkv, const int* slots, void* kcache, void* vcache, const void* first_v, int rows, int hq, int hkv, int dim,
+                            int dk, int dv, int block_size, int num_blocks, int ld, int ldf, float eps, float mix, int* status,
+                            cudaStream_t s) {
+  const int vecs = (dk > dv ? dk : dv) / 8;
+  const long long items = (long long)rows * (hq + 2 * hkv);
+  auto go = [&](auto kern, int g) -> int {
+    if (vecs > g * HN_VECS) return FF_HOST_TOO_LARGE;
+    const long long blocks = (items * g + HN_THREADS - 1) / HN_THREADS;
+    if (int r = launch_pdl(kern, dim3((unsigned)blocks), dim3(HN_THREADS), 0, s, 0, (T*)qkv, slots, (T*)kcache, (T*)vcache, (const T*)first_v,
+                           rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, status)) return r;
+    return launch_result();
+  };
+  if (vecs <= 8) return go(head_norm_kv_kernel<T, 8>, 8);
+  if (vecs <= 16) return go(head_norm_kv_kernel<T, 16>, 16);
+  return go(head_norm_kv_kernel<T, 32>, 32);
+}
+
+}  // namespace ff
+using namespace ff;
+
+FF_EXPORT int ff_head_norm_kv(void* qkv, const int* slots, void* kcache, void* vcache, const void* first_v, int rows, int hq, int hkv,
+                              int dim, int dk, int dv, int block_size, int num_blocks, int ld, int ldf, float eps, float mix, int f32,
+                              int* status, cudaStream_t s) {
+  if (rows <= 0 || hq <= 0 || hkv <= 0 || dim <= 0 || dk < dim || dk % 8 || dv <= 0 || dv % 8 || block_size <= 0) return FF_HOST_BAD_SHAPE;
+  if (ld % 8 || (first_v != nullptr && ldf % 8)) return FF_HOST_BAD_ALIGN;
+  if (f32) return head_norm_launch<float>(qkv, slots, kcache, vcache, first_v, rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, status, s);
+  return head_norm_launch<__nv_bfloat16>(qkv, slots, kcache, vcache, first_v, rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, status, s);
+}

@@ -39,13 +39,27 @@ _HOST_ERR = {
 }
 
 
+_only: tuple[str, ...] | None = None
+
+
+def restrict_to(arch: str) -> None:
+    """For a process that serves one architecture: where the library of all kernels is not built yet, compile only the
+    sources that architecture uses (``build.ARCH_SOURCES``). Call before the first kernel."""
+    global _only
+    from . import build
+    _only = build.ARCH_SOURCES.get(arch)
+
+
 def kernels() -> ctypes.CDLL:
     global _kernels
     if _kernels is None:
         with _lock:
             if _kernels is None:
                 from . import build
-                path = build.build_kernels(timeline=TIMELINE, debug_checks=DEBUG_CHECKS and not TIMELINE)
+                if _only is not None and not TIMELINE and not DEBUG_CHECKS and not build.kernels_up_to_date():
+                    path = build.build_kernels(only=_only)
+                else:
+                    path = build.build_kernels(timeline=TIMELINE, debug_checks=DEBUG_CHECKS and not TIMELINE)
                 lib = ctypes.CDLL(str(path), mode=ctypes.RTLD_GLOBAL)
                 _kernels = _EpochProxy(lib) if DEBUG_CHECKS and not TIMELINE else lib
     return _kernels

@@ -30,12 +30,15 @@ def _r(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
 # ------------------------------------------------------------------------------------------
 # linear
 # ------------------------------------------------------------------------------------------
-def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None) -> torch.Tensor:
+def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None, bias: torch.Tensor | None = None,
+           act: str | None = None) -> torch.Tensor:
     """``y = x @ w.T``, one rounding to the output dtype. The products are accumulated in FP64 so
     the oracle does not depend on how a BLAS blocks the sum for a given batch size (results are
     batch-invariant, as the device kernels' are)."""
     y = x.to(torch.float64) @ w.to(torch.float64).t()
-    return y.to(out_dtype or x.dtype)
+    if bias is not None:
+        y = y + bias.to(torch.float64)
+    return activate(y, act).to(out_dtype or x.dtype)
 
 
 def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, mode: int = 0) -> torch.Tensor:
@@ -182,16 +185,20 @@ def gather_kv(cache: torch.Tensor, block_table_row: torch.Tensor, ctx: int) -> t
 def attention_paged(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_table: torch.Tensor,
                     q_start: torch.Tensor, q_lens: torch.Tensor, ctx_lens: torch.Tensor, hq: int, hkv: int,
                     dim: int, scale: float, tree_mask: torch.Tensor | None = None, window: int = 0,
-                    sinks: torch.Tensor | None = None) -> torch.Tensor:
-    """Causal attention of packed query rows against the paged cache. ``sinks`` (float [hq]): learnable soft-max, one
+                    sinks: torch.Tensor | None = None, chunk: int = 0, vdim: int | None = None,
+                    gate: torch.Tensor | None = None) -> torch.Tensor:
+    """Causal attention of packed query rows against the paged cache. ``chunk > 0``: a query sees only keys of its own
+    block of ``chunk`` positions. ``vdim``: width of a value head (default ``dim``). ``gate`` ([rows, hq*vdim]): the
+    result is multiplied by its sigmoid. ``sinks`` (float [hq]): learnable soft-max, one
     extra logit per head that takes probability mass but contributes no value.
 
     q: [rows, >= hq*dim] (head h at columns h*dim). Sequence b owns rows
     ``q_start[b] : q_start[b]+q_lens[b]`` and ``ctx_lens[b]`` cached keys; its query i sits at
     position ``ctx - q_len + i``. ``tree_mask`` (int64 [B, q_len]) replaces causality inside the
-    last q_len positions by an ancestor bit set. Returns [rows, hq*dim]."""
+    last q_len positions by an ancestor bit set. Returns [rows, hq*vdim]."""
     rows = q.shape[0]
-    out = torch.zeros(rows, hq * dim, dtype=q.dtype, device=q.device)
+    vdim = vdim or dim
+    out = torch.zeros(rows, hq * vdim, dtype=q.dtype, device=q.device)
     g = hq // hkv
     for b in range(block_table.shape[0]):
         ql, ctx, qs = int(q_lens[b]), int(ctx_lens[b]), int(q_start[b])
@@ -208,6 +215,8 @@ def attention_paged(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
         vis = pos_k <= pos_q if window >= 0 else torch.ones(ql, ctx, dtype=torch.bool)   # window < 0: bidirectional
         if window > 0:
             vis &= pos_k > pos_q - window
+        if chunk > 0:
+            vis &= pos_k >= torch.div(pos_q, chunk, rounding_mode="floor") * chunk
         if tree_mask is not None:
             tail = ctx - ql
             bits = tree_mask[b, :ql].to(torch.int64)
@@ -222,8 +231,41 @@ def attention_paged(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
         if sinks is not None:
             p = p[..., :-1]
         o = torch.einsum("hqk,khd->qhd", p, v)
-        out[qs: qs + ql] = o.reshape(ql, hq * dim).to(q.dtype)
+        o = o.reshape(ql, hq * vdim)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[qs: qs + ql].to(F32))
+        out[qs: qs + ql] = o.to(q.dtype)
     return out
+
+
+# ------------------------------------------------------------------------------------------
+# per-head norm + cache write
+# ------------------------------------------------------------------------------------------
+def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, hq: int, hkv: int,
+                 dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0) -> None:
+    """In place on the q heads of ``qkv``: q and k divided by their root mean square over ``dim`` (heads may be padded in
+    the row: the caches' widths are the row's head widths), v blended with ``first_v``; k and v go to ``slots``."""
+    rows, bs = qkv.shape[0], kcache.shape[2]
+    dk, dv = kcache.shape[3], vcache.shape[3]
+    nq, nk = hq * dk, hkv * dk
+    qk = qkv[:, : nq + nk].to(F32).view(rows, hq + hkv, dk)
+    qk = qk * torch.rsqrt((qk * qk).sum(-1, keepdim=True) / dim + eps)
+    qkv[:, : nq] = qk[:, :hq].reshape(rows, nq).to(qkv.dtype)
+    v = qkv[:, nq + nk: nq + nk + hkv * dv].to(F32)
+    if first_v is not None:
+        v = (1.0 - mix) * v + mix * first_v.to(F32)
+    for r in range(rows):
+        s = int(slots[r])
+        if s >= 0:
+            kcache[s // bs, :, s % bs] = qk[r, hq:].to(kcache.dtype)
+            vcache[s // bs, :, s % bs] = v[r].view(hkv, dv).to(vcache.dtype)
+
+
+def activate(x: torch.Tensor, act: str | None) -> torch.Tensor:
+    if act is None:
+        return x
+    assert act == "relu2", act
+    return torch.relu(x) ** 2
 
 
 # ------------------------------------------------------------------------------------------

@@ -202,6 +202,14 @@ def measure_disk_rate(runtime_dir: Path, nbytes: int = 64 << 20) -> float:
 # ------------------------------------------------------------------------------------------------
 def decode_linear_shapes(spec, tp: int = 1) -> list[tuple[str, int, int, int]]:
     """(name, N, K, epilogue id) of the decode projections of a dense / GQA layer on one rank of ``tp``."""
+    if spec.layer_specs is not None:          # designs whose layers differ: every distinct projection once
+        seen: dict[tuple[int, int], str] = {}
+        for l in spec.layer_specs:
+            q, kv, o = l.heads * l.dim_pad, l.kv_heads * (l.dim_pad + l.vdim_pad), l.heads * l.vdim_pad
+            for name, n, k in (("qkv", q + kv + o, spec.hidden), ("o", spec.hidden, o)) + \
+                    ((("up", l.ffn, spec.hidden), ("down", spec.hidden, l.ffn)) if l.ffn else ()):
+                seen.setdefault((n, k), name)
+        return [(name, n, k, 0) for (n, k), name in seen.items()]
     d, h = spec.head_dim, spec.hidden
     hq, hkv = spec.heads // tp, max(1, spec.kv_heads // tp)
     f = spec.ffn // tp

@@ -59,6 +59,11 @@ def workspace_row_bytes(spec: ModelSpec, tp: int = 1) -> int:
     """Bytes of activation workspace per prefill row: residual, normed, attention out, projection
     out (4 x hidden), packed QKV, gate/up + activated (3 x ffn), ids/positions/slots
     (the reference's formula, src/prefill.rs:302-307, with the parallel shards applied)."""
+    if spec.layer_specs is not None:
+        # FP32 residual streams; per layer the packed projection, attention output and FFN rows
+        streams = int(spec.extra.get("duponex", {}).get("streams", 1))
+        wide = max(l.heads * (l.dim_pad + 3 * l.vdim_pad) + l.kv_heads * (l.dim_pad + l.vdim_pad) + l.ffn for l in spec.layer_specs)
+        return 4 * spec.hidden * streams + (4 * spec.hidden + 2 * wide) * spec.elem_bytes + 12
     ffn = spec.moe.expert_ffn * spec.moe.top_k if spec.moe is not None else spec.ffn
     return (4 * spec.hidden + spec.qkv_dim // tp + 3 * ffn // tp) * 2 + 12 + spec.heads * 4
 
@@ -107,6 +112,8 @@ def plan_memory(spec: ModelSpec, settings: Settings, info: DeviceInfo, weights_b
     hkv = max(1, spec.kv_heads // tp)
     if spec.mla is not None:
         block_bytes = spec.layers * settings.kv_block * (spec.mla.kv_lora_rank + spec.mla.qk_rope_dim) * 2
+    elif spec.kv_geometry() is not None:
+        block_bytes = settings.kv_block * spec.elem_bytes * sum(h * (dk + dv) for h, dk, dv in spec.kv_geometry())
     else:
         block_bytes = spec.layers * hkv * settings.kv_block * spec.head_dim * 2 * 2
     blocks_per_seq = (settings.capacity + settings.kv_block - 1) // settings.kv_block
@@ -125,6 +132,8 @@ def plan_memory(spec: ModelSpec, settings: Settings, info: DeviceInfo, weights_b
     workspace = chunk * row_bytes
     kv_budget = free_after_weights - workspace
     want = blocks_per_seq * settings.max_batch + 1
+    if settings.kv_tokens is not None:
+        want = (settings.kv_tokens + settings.kv_block - 1) // settings.kv_block
     kv_blocks = int(min(kv_budget // block_bytes, want))
     if kv_blocks < blocks_per_seq:
         raise PlanError("no room for the KV cache of one full sequence")
@@ -144,7 +153,10 @@ def plan_engine(spec: ModelSpec, settings: Settings, device: torch.device | str,
         # small, fixed arena
         blocks_per_seq = (settings.capacity + settings.kv_block - 1) // settings.kv_block
         chunk = settings.chunk or 512
-        return EnginePlan(prefill_chunk=chunk, kv_blocks=blocks_per_seq * min(settings.max_batch, 8) + 1, kv_bytes=0,
+        blocks = blocks_per_seq * min(settings.max_batch, 8) + 1
+        if settings.kv_tokens is not None:
+            blocks = (settings.kv_tokens + settings.kv_block - 1) // settings.kv_block
+        return EnginePlan(prefill_chunk=chunk, kv_blocks=blocks, kv_bytes=0,
                           workspace_bytes=0, reserve_bytes=0, weights_bytes=weights_bytes, budget_bytes=0,
                           graph_buckets=())
     # weights are already resident when the planner runs, so `free` excludes them

@@ -41,8 +41,10 @@ def identity_for(model) -> PrefixIdentity:
     spec = model.spec
     tk = model.tokenizer
     tk_id = f"{type(tk).__name__}:{getattr(tk, 'vocab_size', spec.vocab)}"
-    rope = hashlib.sha256(json.dumps([spec.rope_theta, spec.head_dim, spec.extra.get("rope_scaling")],
-                                     sort_keys=True).encode()).hexdigest()[:16]
+    fields = [spec.rope_theta, spec.head_dim, spec.extra.get("rope_scaling")]
+    if spec.layer_specs is not None:          # designs whose layers differ: every layer's cache geometry and masks, and the type
+        fields.append([spec.dtype, [l.__dict__ for l in spec.layer_specs], spec.extra])
+    rope = hashlib.sha256(json.dumps(fields, sort_keys=True).encode()).hexdigest()[:16]
     return PrefixIdentity(model.name, tk_id, rope, model.settings.kv_format)
 
 
