@@ -7,6 +7,8 @@ head_dim 128, SwiGLU 14336, vocab 128256, BF16, random-init N(0, 0.02) weights, 
 parallel over the N GPUs of one node. ``--config 3`` selects the Llama-3-70B shape (batch 32,
 prompt 4096). A step is one decode step of the whole batch.
 
+``--design duponex`` measures another model design beside its closest relative instead (``utils/designbench.py``).
+
 Three arms (``--impl``):
   * ``ours``      -- this framework's engine and kernels. Reports
       ``value``  device-timed: K decode steps queued without host synchronisation (per-step
@@ -74,6 +76,8 @@ def parse() -> argparse.Namespace:
     p.add_argument("--skip-e2e", action="store_true")
     p.add_argument("--skip-baseline", action="store_true")
     p.add_argument("--skip-extras", action="store_true", help="no TTFT run and no other batch sizes")
+    p.add_argument("--design", default=None, choices=["duponex"],
+                   help="instead of the headline benchmark: throughput and kernels of this design beside the closest model at equal size")
     p.add_argument("--device", default="cuda", choices=["cuda", "cpu"], help="cpu is for debugging the harness only")
     a = p.parse_args()
     c = CONFIGS[a.config]
@@ -550,7 +554,12 @@ def main() -> None:
     cx = Ctx(args)
     cx.sampler.wait_first()
     try:
-        if args.impl == "baseline":
+        if args.design is not None:
+            from flyingfish_b200.utils import designbench
+            t0 = time.perf_counter()
+            out = designbench.run(cx.device, args.steps, args.warmup, layers=args.layers)
+            out["clocks"] = cx.sampler.window(t0, time.perf_counter())
+        elif args.impl == "baseline":
             out = run_baseline(cx)
         else:
             out = run_ours(cx)

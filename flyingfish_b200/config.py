@@ -383,14 +383,14 @@ def duponex_tiny() -> ModelSpec:
 
 def duponex_8b() -> ModelSpec:
     """Duponex layers at the size of an 8-billion-parameter decoder (random weights, for measurements): 4096 wide, 32 / 8
-    heads of 128, blocks of 1024 positions, four residual streams."""
-    layers = [LayerSpec(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, v_mix=True, chunk=1024, ffn=14336) for _ in range(8)]
+    heads of 128, blocks of 2048 positions, four residual streams."""
+    layers = [LayerSpec(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, v_mix=True, chunk=2048, ffn=14336) for _ in range(8)]
     return _duponex_spec_of("duponex-8b-shape", 4096, 128256, layers, streams=4, residual_mult=0.5, embed_scale=8.0, eps=1e-5)
 
 
 def duponex_2b() -> ModelSpec:
-    """As :func:`duponex_8b` at 2048 wide: 16 / 4 heads of 128, blocks of 512 positions."""
-    layers = [LayerSpec(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, v_mix=True, chunk=512, ffn=8192) for _ in range(16)]
+    """As :func:`duponex_8b` at 2048 wide: 16 / 4 heads of 128, 16 layers."""
+    layers = [LayerSpec(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, v_mix=True, chunk=2048, ffn=8192) for _ in range(16)]
     return _duponex_spec_of("duponex-2b-shape", 2048, 65536, layers, streams=4, residual_mult=0.5, embed_scale=8.0, eps=1e-5)
 
 

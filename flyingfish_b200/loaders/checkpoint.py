@@ -250,10 +250,15 @@ def checkpoint_source(model_dir: str | Path, spec: ModelSpec, device: torch.devi
 
 
 def audited_source(model_dir: str | Path, spec: ModelSpec, device: torch.device | str):
-    """:func:`checkpoint_source` of a directory that holds exactly the manifest of ``spec``."""
+    """:func:`checkpoint_source` of a directory that holds the manifest of ``spec`` (and nothing the architecture does not
+    know)."""
     ck = MappedCheckpoint(Path(model_dir))
+    extra: tuple[str, ...] = ()
+    if spec.arch == "duponex":
+        from ..models.duponex import unused_tensors
+        extra = unused_tensors(spec)
     try:
-        audit(ck, spec)
+        audit(ck, spec, allow_extra=extra)
     finally:
         ck.close()
     return checkpoint_source(model_dir, spec, device)

@@ -54,6 +54,17 @@ def expected_tensors(spec: ModelSpec) -> dict[str, tuple[int, ...]]:
     return m
 
 
+def unused_tensors(spec: ModelSpec) -> tuple[str, ...]:
+    """Tensors of parts a layer's configuration switches off: a checkpoint may carry them, nothing reads them."""
+    names = []
+    for i, l in enumerate(spec.layer_specs):
+        if not l.v_mix:
+            names.append(f"l{i}.mix.vmix")
+        if not l.ffn:
+            names += [f"l{i}." + n for n in ("norm2", "ls2", "hc2.in", "hc2.out", "hc2.mix", "mlp.up", "mlp.down")]
+    return tuple(names)
+
+
 def _pad_cols(t: torch.Tensor, cols: int) -> torch.Tensor:
     if t.shape[-1] == cols:
         return t.contiguous()

@@ -485,12 +485,14 @@ def test_configuration_is_read_and_checked(base):
 
 def test_checkpoint_is_audited(tmp_path):
     w = O.tensors(CFG)
-    for i, (drop, put) in enumerate((("l1.mix.vmix", None), (None, ("l3.mlp.up", torch.zeros(2, 2))), ("l0.hc1.in", ("l0.hc1.in", torch.zeros(4))))):
+    for i, (drop, put) in enumerate((("l1.mix.vmix", None), (None, ("l3.mlp.gate", torch.zeros(2, 2))), ("l0.hc1.in", ("l0.hc1.in", torch.zeros(4))))):
         t = {n: x for n, x in w.items() if n != drop}
         if put:
             t[put[0]] = put[1].to(torch.bfloat16)
         with pytest.raises(CheckpointError):
             load(write(tmp_path, CFG, t, f"m{i}"), "cpu", "bf16")
+    # tensors of a part the configuration switches off may be there
+    load(write(tmp_path, CFG, dict(w, **{"l0.mix.vmix": torch.tensor(0.5).to(torch.bfloat16), "l3.norm2": w["l3.norm1"].clone()}), "more"), "cpu", "bf16")
 
 
 def test_planner_counts_unequal_layers():
