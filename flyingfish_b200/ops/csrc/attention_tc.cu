@@ -365,23 +365,24 @@ constexpr int TC2_SMEM = TC_Q_BYTES + 4 * T2_KV_BYTES + 1024;      // 97 KiB
 
 // what a launch adds to plain causal attention over 128-wide heads
 struct PrefillForm {
-  int window, chunk, causal, dk, dv, ldg;
-  const __nv_bfloat16* gate;       // [rows, hq * dv]: the result is multiplied by its sigmoid
+  int window, chunk, causal, dk, dv;
+  int gated;                       // the result is multiplied by the sigmoid of a [rows, hq * dv] gate (tensor map tmG)
 };
 
-// o * inv, times the sigmoid of the gate where there is one; 16 columns, two 16-byte stores
-__device__ __forceinline__ void store_o16(__nv_bfloat16* dst, const uint32_t* r, float inv, const __nv_bfloat16* gate) {
+// o * inv, times the sigmoid of the gate where there is one (`gate`: the row of a swizzled gate tile in shared memory, `sw` =
+// row % 8, `chunk` its first 16-byte chunk); 16 columns, two 16-byte stores
+__device__ __forceinline__ void store_o16(__nv_bfloat16* dst, const uint32_t* r, float inv, const uint8_t* gate, int chunk, int sw) {
   float v[16];
 #pragma unroll
   for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]) * inv;
   if (gate != nullptr) {
-    const uint4 g0 = reinterpret_cast<const uint4*>(gate)[0], g1 = reinterpret_cast<const uint4*>(gate)[1];
+    const uint4 g0 = *reinterpret_cast<const uint4*>(gate + ((chunk ^ sw) << 4)), g1 = *reinterpret_cast<const uint4*>(gate + (((chunk + 1) ^ sw) << 4));
     const uint32_t gw[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       const float2 g = unpack_bf16x2(gw[i]);
-      v[2 * i] *= 1.0f / (1.0f + __expf(-g.x));
-      v[2 * i + 1] *= 1.0f / (1.0f + __expf(-g.y));
+      v[2 * i] = __fdividef(v[2 * i], 1.0f + __expf(-g.x));
+      v[2 * i + 1] = __fdividef(v[2 * i + 1], 1.0f + __expf(-g.y));
     }
   }
   uint32_t o[8];
@@ -392,7 +393,7 @@ __device__ __forceinline__ void store_o16(__nv_bfloat16* dst, const uint32_t* r,
 }
 
 struct alignas(8) Tc2Bars {
-  uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], pv_done[2];
+  uint64_t q_full, g_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], pv_done[2];
   uint32_t tmem_base;
   int abort_flag;
   float xmax[2][TC_BM];
@@ -401,7 +402,7 @@ struct alignas(8) Tc2Bars {
 template <int SPLIT>
 __global__ void __launch_bounds__(64 + 128 * SPLIT, 2)
 attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                        const __grid_constant__ CUtensorMap tmV, const int* __restrict__ block_table,
+                        const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmG, const int* __restrict__ block_table,
                         const int* __restrict__ q_start, const int* __restrict__ q_lens,
                         const int* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out, int hq, int hkv, int ldo,
                         int max_blocks, int num_blocks, float scale_log2, const PrefillForm f, int* status,
@@ -431,7 +432,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 
   if (threadIdx.x == 0) {
     tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
-    mbar_init(&bars.q_full, 1);
+    mbar_init(&bars.q_full, 1); mbar_init(&bars.g_full, 1);
     for (int i = 0; i < 2; ++i) {
       mbar_init(&bars.k_full[i], 1); mbar_init(&bars.k_empty[i], 1); mbar_init(&bars.v_full[i], 1); mbar_init(&bars.v_empty[i], 1);
       mbar_init(&bars.s_full[i], 1); mbar_init(&bars.p_full[i], 1); mbar_init(&bars.pv_done[i], 1);
@@ -481,6 +482,15 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         mbar_expect_tx(&bars.v_full[st], v_hi ? T2_KV_BYTES : T2_KV_BYTES / 2);
         tma_load_2d(sV + st * T2_KV_BYTES, &tmV, &bars.v_full[st], 0, row);
         if (v_hi) tma_load_2d(sV + st * T2_KV_BYTES + 8192, &tmV, &bars.v_full[st], 64, row);
+      }
+      if (ok && f.gated) {
+        // the gate tile takes the place of Q once the last Q Kᵀ has read it; it arrives under the last soft-max and P V
+        const int st = (ntiles - 1) & 1;
+        if (mbar_wait(&bars.k_empty[st], ((ntiles - 1) >> 1) & 1, abort_flag, status, KID_ATTN_PREFILL, 31)) {
+          mbar_expect_tx(&bars.g_full, v_hi ? TC_Q_BYTES : TC_Q_BYTES / 2);
+          tma_load_2d(sQ, &tmG, &bars.g_full, h * dv, qs + r0);
+          if (v_hi) tma_load_2d(sQ + TC_BM * 128, &tmG, &bars.g_full, h * dv + 64, qs + r0);
+        }
       }
       if (bad) set_status(status, KID_ATTN_PREFILL, FF_ERR_BOUNDS, b, r0 / TC_BM);
     }
@@ -635,6 +645,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     }
     // the last P V
     if (ok && !mbar_wait(&bars.pv_done[(ntiles - 1) & 1], ((ntiles - 1) >> 1) & 1, abort_flag, status, KID_ATTN_PREFILL, 29)) ok = false;
+    if (ok && f.gated && !mbar_wait(&bars.g_full, 0, abort_flag, status, KID_ATTN_PREFILL, 32)) ok = false;
     ok = __all_sync(0xffffffffu, ok);
     if (SPLIT == 2) {
       bars.xmax[hf][row] = l_sum;
@@ -646,14 +657,14 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       if (sinks != nullptr) l_sum += (m_ref == -INFINITY) ? 1.f : exp2f(sinks[h] * 1.4426950408889634f - m_ref);
       const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
       __nv_bfloat16* orow = out + (size_t)(qs + r0 + row) * ldo + (size_t)h * dv + hf * (TC_HD / SPLIT);
-      const __nv_bfloat16* grow = f.gate == nullptr ? nullptr : f.gate + (size_t)(qs + r0 + row) * f.ldg + (size_t)h * dv + hf * (TC_HD / SPLIT);
 #pragma unroll
       for (int c = 0; c < TC_HD / SPLIT; c += 16) {
         if (hf * (TC_HD / SPLIT) + c >= dv) break;
         uint32_t r[16];
         tmem_ld_x16(tmem_o + lane_base + hf * (TC_HD / SPLIT) + c, r);
         tmem_ld_wait();
-        if (live) store_o16(orow + c, r, inv, grow == nullptr ? nullptr : grow + c);
+        const int col = hf * (TC_HD / SPLIT) + c;                       // gate tile: 64-column halves of [128 rows][128 bytes]
+        if (live) store_o16(orow + c, r, inv, f.gated ? sQ + (col >> 6) * (TC_BM * 128) + row * 128 : nullptr, (col & 63) >> 3, row & 7);
       }
     }
   }
@@ -691,7 +702,10 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
   if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dv, cache_rows, dv * 2, 64, TC_PAGE)) return r;
   const float scale_log2 = scale * 1.4426950408889634f;
   dim3 grid((max_q_len + TC_BM - 1) / TC_BM, hq, batch);
-  const PrefillForm f = {window < 0 ? 0 : window, chunk, window < 0 ? 0 : 1, dk, dv, ldg, (const __nv_bfloat16*)gate};
+  const PrefillForm f = {window < 0 ? 0 : window, chunk, window < 0 ? 0 : 1, dk, dv, gate != nullptr ? 1 : 0};
+  CUtensorMap tmG = tmQ;
+  if (gate != nullptr)
+    if (int r = make_tmap_2d(&tmG, gate, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)hq * dv, (uint64_t)total_rows, (uint64_t)ldg * 2, 64, TC_BM)) return r;
   // FF_ATTN_PREFILL_CTAS = 1 selects the one-CTA-per-SM kernel (deep K / V rings, eight softmax warps; plain 128-wide heads
   // only); the default is the two-CTAs-per-SM kernel
   static int two = -1;
@@ -702,12 +716,12 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
     if (split < 0) { const char* e = getenv("FF_ATTN_PREFILL_SPLIT"); split = (e != nullptr && (e[0] == '1' || e[0] == '2')) ? e[0] - '0' : TC2_SPLIT_DEFAULT; }
     if (split == 2) {
       if (int r = opt_in_smem(attn_prefill_tc2_kernel<2>, TC2_SMEM)) return r;
-      attn_prefill_tc2_kernel<2><<<grid, 320, TC2_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out,
+      attn_prefill_tc2_kernel<2><<<grid, 320, TC2_SMEM, s>>>(tmQ, tmK, tmV, tmG, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out,
                                                              hq, hkv, ldo, max_blocks, num_blocks, scale_log2, f, status, sinks);
       return launch_result();
     }
     if (int r = opt_in_smem(attn_prefill_tc2_kernel<1>, TC2_SMEM)) return r;
-    attn_prefill_tc2_kernel<1><<<grid, 192, TC2_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out,
+    attn_prefill_tc2_kernel<1><<<grid, 192, TC2_SMEM, s>>>(tmQ, tmK, tmV, tmG, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out,
                                                            hq, hkv, ldo, max_blocks, num_blocks, scale_log2, f, status, sinks);
     return launch_result();
   }
