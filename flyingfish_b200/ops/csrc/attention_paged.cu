@@ -212,7 +212,9 @@ __device__ __forceinline__ float gate_factor(const __nv_bfloat16* gate, int ldg,
 // Measured on B200 (batch 64, context 1100, 32/8 heads): four 16-key warps 75.6 us, two 32-key warps
 // 80.3 us -- the wider warps issue fewer instructions per key but leave too few warps per SM.
 // ---------------------------------------------------------------------------------------
-template <int NW>
+// WIDE: heads are exactly 128 wide (widths known at compile time); EXTRA: the launch may have a block-local mask or a gate.
+// Plain causal / windowed attention keeps its own instance: the run-time widths cost it a tenth of its time.
+template <int NW, bool WIDE, bool EXTRA>
 __global__ void __launch_bounds__(32 * NW)
 attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                    const __nv_bfloat16* __restrict__ q, const int* __restrict__ block_table,
@@ -238,8 +240,9 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   // sees keys pos - window + 1 .. pos, so the pages before the earliest bound of the nq queries are not visited
   // kv_start (mixed cache formats): keys below kv_start[b] (a multiple of the page size) are not in BF16 pages any
   // more; another kernel covers them and writes its partials behind this kernel's splits (stride pstride)
-  const int window = f.window, chunk = f.chunk, kd = f.dk >> 4, vd = f.dv >> 4;
-  const bool k_hi = f.dk > 64, v_hi = f.dv > 64;           // heads up to 64 wide: the upper half of a tile is not loaded
+  const int window = f.window, chunk = EXTRA ? f.chunk : 0, dk = WIDE ? HD : f.dk, dv = WIDE ? HD : f.dv, kd = dk >> 4, vd = dv >> 4;
+  const __nv_bfloat16* const gate = EXTRA ? f.gate : nullptr;
+  const bool k_hi = dk > 64, v_hi = dv > 64;           // heads up to 64 wide: the upper half of a tile is not loaded
   int pfirst = first_visible(ctx - nq, window, chunk) / PAGE;
   if (kv_start != nullptr) pfirst = max(pfirst, min(kv_start[b], ctx) / PAGE);
   const int per = (pages - pfirst + nsplit - 1) / nsplit;
@@ -254,7 +257,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     const int r = rt * 16 + g + e * 8;
     if (r < rows_total) {
       const int qi = r / G, hh = kvh * G + r % G;
-      qp[e] = q + (size_t)(b * nq + qi) * ldq + (size_t)hh * f.dk;
+      qp[e] = q + (size_t)(b * nq + qi) * ldq + (size_t)hh * dk;
       lim[e] = ctx - nq + qi;
       mk[e] = tree_mask ? tree_mask[(size_t)b * nq + qi] : ~0ull;
     } else { qp[e] = nullptr; lim[e] = -1; mk[e] = 0ull; }
@@ -346,15 +349,15 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 #pragma unroll
     for (int w = 0; w < NW; ++w) { sc[w] = exp2f(sml[(w * 16 + r) * 2] - M); L += sml[(w * 16 + r) * 2 + 1] * sc[w]; }
     const int qi = rg / G, hh = kvh * G + rg % G;
-    for (int d = threadIdx.x; d < f.dv; d += 32 * NW) {
+    for (int d = threadIdx.x; d < dv; d += 32 * NW) {
       float acc = 0.f;
 #pragma unroll
       for (int w = 0; w < NW; ++w) acc += so[(w * 16 + r) * HD + d] * sc[w];
       if (nsplit == 1 && pstride == 0) {
         // learnable soft-max: the head's sink logit enters the denominator only
         const float Ls = sinks ? L + exp2f(sinks[hh] * 1.4426950408889634f - M) : L;
-        const float gf = gate_factor(f.gate, f.ldg, (size_t)(b * nq + qi), hh * f.dv + d);
-        out[((size_t)(b * nq + qi) * hq + hh) * f.dv + d] = __float2bfloat16(Ls > 0.f ? acc / Ls * gf : 0.f);
+        const float gf = gate_factor(gate, f.ldg, (size_t)(b * nq + qi), hh * dv + d);
+        out[((size_t)(b * nq + qi) * hq + hh) * dv + d] = __float2bfloat16(Ls > 0.f ? acc / Ls * gf : 0.f);
       } else {
         const size_t pr = ((size_t)b * (pstride ? pstride : nsplit) + split) * (nq * hq) + (size_t)qi * hq + hh;
         part_o[pr * HD + d] = acc;
@@ -384,7 +387,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
         const size_t row = (size_t)qi * hq + hh;
         float M = NEG_BIG;
         for (int sp = 0; sp < nsplit; ++sp) M = fmaxf(M, __ldcg(&part_ml[(((size_t)b * nsplit + sp) * (nq * hq) + row) * 2]));
-        for (int d = threadIdx.x; d < f.dv; d += 32 * NW) {
+        for (int d = threadIdx.x; d < dv; d += 32 * NW) {
           float L = 0.f, acc = 0.f;
           for (int sp = 0; sp < nsplit; ++sp) {
             const size_t pr = ((size_t)b * nsplit + sp) * (nq * hq) + row;
@@ -393,8 +396,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
             acc += __ldcg(&part_o[pr * HD + d]) * sc;
           }
           if (sinks) L += exp2f(sinks[hh] * 1.4426950408889634f - M);
-          const float gf = gate_factor(f.gate, f.ldg, (size_t)(b * nq + qi), hh * f.dv + d);
-          out[((size_t)(b * nq + qi) * hq + hh) * f.dv + d] = __float2bfloat16(L > 0.f ? acc / L * gf : 0.f);
+          const float gf = gate_factor(gate, f.ldg, (size_t)(b * nq + qi), hh * dv + d);
+          out[((size_t)(b * nq + qi) * hq + hh) * dv + d] = __float2bfloat16(L > 0.f ? acc / L * gf : 0.f);
         }
       }
     }
@@ -557,7 +560,9 @@ static int attn_decode_launch(const void* q, const void* kcache, const void* vca
   if (ldq % 8 || nsplit < 1) return FF_HOST_BAD_ALIGN;
   if (nsplit > 1 && (!part_o || !part_ml)) return FF_HOST_BAD_SHAPE;
   constexpr int NW = DEC_WARPS;
-  if (int r = opt_in_smem(attn_decode_kernel<NW>, DEC_SMEM)) return r;
+  const bool wide = f.dk == HD && f.dv == HD, extra = f.chunk > 0 || f.gate != nullptr;
+  auto kern = !wide ? attn_decode_kernel<NW, false, true> : extra ? attn_decode_kernel<NW, true, true> : attn_decode_kernel<NW, true, false>;
+  if (int r = opt_in_smem(kern, DEC_SMEM)) return r;
   const float scale_log2 = scale * 1.4426950408889634f;
   const int row_tiles = (nq * (hq / hkv) + 15) / 16;
   dim3 grid(nsplit, hkv * row_tiles, batch);
@@ -566,7 +571,7 @@ static int attn_decode_launch(const void* q, const void* kcache, const void* vca
   const uint64_t cache_rows = (uint64_t)num_blocks * hkv * PAGE;
   if (int r = make_tmap_2d(&tmK, kcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, f.dk, cache_rows, f.dk * 2, 64, PAGE)) return r;
   if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, f.dv, cache_rows, f.dv * 2, 64, PAGE)) return r;
-  if (int lr_ = launch_pdl(attn_decode_kernel<NW>, dim3(grid), dim3(32 * NW), DEC_SMEM, s, 0, tmK, tmV, (const __nv_bfloat16*)q,
+  if (int lr_ = launch_pdl(kern, dim3(grid), dim3(32 * NW), DEC_SMEM, s, 0, tmK, tmV, (const __nv_bfloat16*)q,
       block_table, ctx_lens, tree_mask, (__nv_bfloat16*)out, part_o, part_ml, hq, hkv, nq,
       ldq, max_blocks, num_blocks, nsplit, scale_log2, status, split_counters, f, kv_start, pstride, sinks)) return lr_;
   if (int r = launch_result()) return r;

@@ -399,7 +399,9 @@ struct alignas(8) Tc2Bars {
   float xmax[2][TC_BM];
 };
 
-template <int SPLIT>
+// WIDE: heads are exactly 128 wide; EXTRA: the launch may have a block-local mask or a gate (plain launches keep an instance
+// with neither).
+template <int SPLIT, bool WIDE, bool EXTRA>
 __global__ void __launch_bounds__(64 + 128 * SPLIT, 2)
 attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                         const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmG, const int* __restrict__ block_table,
@@ -421,7 +423,8 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   const int kvh = h / (hq / hkv);
   const int past = ctx - qlen;
   const int real = min(TC_BM, qlen - r0);
-  const int causal = f.causal, window = f.window, chunk = f.chunk, dk = f.dk, dv = f.dv;
+  const int causal = f.causal, window = f.window, chunk = EXTRA ? f.chunk : 0, dk = WIDE ? TC_HD : f.dk, dv = WIDE ? TC_HD : f.dv;
+  const bool gated = EXTRA && f.gated != 0;
   const bool k_hi = dk > 64, v_hi = dv > 64;                       // heads up to 64 wide: the upper 64 columns are not loaded
   auto first_visible = [&](int pos) { return window > 0 ? max(0, pos - window + 1) : (chunk > 0 ? pos / chunk * chunk : 0); };
   const int last_key = causal ? past + r0 + real - 1 : ctx - 1;
@@ -483,7 +486,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         tma_load_2d(sV + st * T2_KV_BYTES, &tmV, &bars.v_full[st], 0, row);
         if (v_hi) tma_load_2d(sV + st * T2_KV_BYTES + 8192, &tmV, &bars.v_full[st], 64, row);
       }
-      if (ok && f.gated) {
+      if (ok && gated) {
         // the gate tile takes the place of Q once the last Q Kᵀ has read it; it arrives under the last soft-max and P V
         const int st = (ntiles - 1) & 1;
         if (mbar_wait(&bars.k_empty[st], ((ntiles - 1) >> 1) & 1, abort_flag, status, KID_ATTN_PREFILL, 31)) {
@@ -645,7 +648,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     }
     // the last P V
     if (ok && !mbar_wait(&bars.pv_done[(ntiles - 1) & 1], ((ntiles - 1) >> 1) & 1, abort_flag, status, KID_ATTN_PREFILL, 29)) ok = false;
-    if (ok && f.gated && !mbar_wait(&bars.g_full, 0, abort_flag, status, KID_ATTN_PREFILL, 32)) ok = false;
+    if (ok && gated && !mbar_wait(&bars.g_full, 0, abort_flag, status, KID_ATTN_PREFILL, 32)) ok = false;
     ok = __all_sync(0xffffffffu, ok);
     if (SPLIT == 2) {
       bars.xmax[hf][row] = l_sum;
@@ -664,7 +667,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         tmem_ld_x16(tmem_o + lane_base + hf * (TC_HD / SPLIT) + c, r);
         tmem_ld_wait();
         const int col = hf * (TC_HD / SPLIT) + c;                       // gate tile: 64-column halves of [128 rows][128 bytes]
-        if (live) store_o16(orow + c, r, inv, f.gated ? sQ + (col >> 6) * (TC_BM * 128) + row * 128 : nullptr, (col & 63) >> 3, row & 7);
+        if (live) store_o16(orow + c, r, inv, gated ? sQ + (col >> 6) * (TC_BM * 128) + row * 128 : nullptr, (col & 63) >> 3, row & 7);
       }
     }
   }
@@ -714,16 +717,16 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
     // FF_ATTN_PREFILL_SPLIT = 2: two softmax warps per lane quadrant (64 columns each) instead of one
     static int split = -1;
     if (split < 0) { const char* e = getenv("FF_ATTN_PREFILL_SPLIT"); split = (e != nullptr && (e[0] == '1' || e[0] == '2')) ? e[0] - '0' : TC2_SPLIT_DEFAULT; }
-    if (split == 2) {
-      if (int r = opt_in_smem(attn_prefill_tc2_kernel<2>, TC2_SMEM)) return r;
-      attn_prefill_tc2_kernel<2><<<grid, 320, TC2_SMEM, s>>>(tmQ, tmK, tmV, tmG, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out,
-                                                             hq, hkv, ldo, max_blocks, num_blocks, scale_log2, f, status, sinks);
+    auto go = [&](auto kern, int threads) -> int {
+      if (int r = opt_in_smem(kern, TC2_SMEM)) return r;
+      kern<<<grid, threads, TC2_SMEM, s>>>(tmQ, tmK, tmV, tmG, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out, hq, hkv, ldo,
+                                           max_blocks, num_blocks, scale_log2, f, status, sinks);
       return launch_result();
-    }
-    if (int r = opt_in_smem(attn_prefill_tc2_kernel<1>, TC2_SMEM)) return r;
-    attn_prefill_tc2_kernel<1><<<grid, 192, TC2_SMEM, s>>>(tmQ, tmK, tmV, tmG, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out,
-                                                           hq, hkv, ldo, max_blocks, num_blocks, scale_log2, f, status, sinks);
-    return launch_result();
+    };
+    const bool wide = dk == TC_HD && dv == TC_HD, extra = chunk > 0 || gate != nullptr;
+    if (!wide) return go(attn_prefill_tc2_kernel<1, false, true>, 192);
+    if (split == 2) return extra ? go(attn_prefill_tc2_kernel<2, true, true>, 320) : go(attn_prefill_tc2_kernel<2, true, false>, 320);
+    return extra ? go(attn_prefill_tc2_kernel<1, true, true>, 192) : go(attn_prefill_tc2_kernel<1, true, false>, 192);
   }
   if (int r = opt_in_smem(attn_prefill_tc_kernel, TC_SMEM)) return r;
   attn_prefill_tc_kernel<<<grid, 320, TC_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens,

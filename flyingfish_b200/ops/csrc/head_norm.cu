@@ -12,9 +12,9 @@
 namespace ff {
 
 constexpr int HN_THREADS = 256;
-constexpr int HN_VECS = 4;              // vectors of 8 elements a lane may hold
 
-template <typename T, int G>
+// NV: vectors of 8 elements a lane holds
+template <typename T, int G, int NV>
 __global__ void __launch_bounds__(HN_THREADS)
 head_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __restrict__ kcache, T* __restrict__ vcache,
                     const T* __restrict__ first_v, int rows, int hq, int hkv, int dim, int dk, int dv, int block_size, int num_blocks,
@@ -29,10 +29,10 @@ head_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __res
   const bool is_q = head < hq, is_v = head >= hq + hkv;
   const int d = is_v ? dv : dk;
   T* base = qkv + (size_t)row * ld + (is_v ? (size_t)(hq + hkv) * dk + (size_t)(head - hq - hkv) * dv : (size_t)head * dk);
-  float v[HN_VECS][8];
+  float v[NV][8];
   float ss = 0.f;
 #pragma unroll
-  for (int i = 0; i < HN_VECS; ++i) {
+  for (int i = 0; i < NV; ++i) {
     const int c = (gl + i * G) * 8;
     if (live && c < d) {
       load8(base + c, v[i]);
@@ -46,13 +46,13 @@ head_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __res
   if (!is_v) {
     const float r = 1.0f / sqrtf(ss / (float)dim + eps);
 #pragma unroll
-    for (int i = 0; i < HN_VECS; ++i)
+    for (int i = 0; i < NV; ++i)
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[i][j] *= r;
   } else if (first_v != nullptr) {
     const T* fv = first_v + (size_t)row * ldf + (size_t)(head - hq - hkv) * dv;
 #pragma unroll
-    for (int i = 0; i < HN_VECS; ++i) {
+    for (int i = 0; i < NV; ++i) {
       const int c = (gl + i * G) * 8;
       if (c < d) {
         float f[8];
@@ -73,7 +73,7 @@ head_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __res
     dst = (is_v ? vcache : kcache) + (((size_t)blk * hkv + kvh) * block_size + off) * d;
   }
 #pragma unroll
-  for (int i = 0; i < HN_VECS; ++i) {
+  for (int i = 0; i < NV; ++i) {
     const int c = (gl + i * G) * 8;
     if (c < d) store8(dst + c, v[i]);
   }
@@ -86,15 +86,16 @@ static int head_norm_launch(void* qkv, const int* slots, void* kcache, void* vca
   const int vecs = (dk > dv ? dk : dv) / 8;
   const long long items = (long long)rows * (hq + 2 * hkv);
   auto go = [&](auto kern, int g) -> int {
-    if (vecs > g * HN_VECS) return FF_HOST_TOO_LARGE;
     const long long blocks = (items * g + HN_THREADS - 1) / HN_THREADS;
     if (int r = launch_pdl(kern, dim3((unsigned)blocks), dim3(HN_THREADS), 0, s, 0, (T*)qkv, slots, (T*)kcache, (T*)vcache, (const T*)first_v,
                            rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, status)) return r;
     return launch_result();
   };
-  if (vecs <= 8) return go(head_norm_kv_kernel<T, 8>, 8);
-  if (vecs <= 16) return go(head_norm_kv_kernel<T, 16>, 16);
-  return go(head_norm_kv_kernel<T, 32>, 32);
+  if (vecs <= 8) return go(head_norm_kv_kernel<T, 8, 1>, 8);
+  if (vecs <= 16) return go(head_norm_kv_kernel<T, 16, 1>, 16);
+  if (vecs <= 32) return go(head_norm_kv_kernel<T, 32, 1>, 32);
+  if (vecs <= 128) return go(head_norm_kv_kernel<T, 32, 4>, 32);
+  return FF_HOST_TOO_LARGE;
 }
 
 }  // namespace ff

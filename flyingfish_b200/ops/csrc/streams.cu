@@ -108,7 +108,9 @@ static int stream_launch(const int* ids, const T* table, float scale, int vocab,
   const int smem = width * 4;
   if (smem > 200 * 1024) return FF_HOST_TOO_LARGE;
   int threads = (width / 4 + 31) / 32 * 32;
-  if (threads > ST_THREADS) threads = ST_THREADS;
+  // a few rows (a decode step): wide blocks, for latency; many: more, smaller blocks per SM keep more loads in flight
+  const int cap = rows >= 2 * sm_count() ? ST_THREADS / 2 : ST_THREADS;
+  if (threads > cap) threads = cap;
   auto go = [&](auto kern) -> int {
     if (int r = opt_in_smem(kern, smem)) return r;
     if (int r = launch_pdl(kern, dim3(rows), dim3(threads), smem, s, 0, ids, table, scale, vocab, x, y, chan, coef, norm_w, n, streams,

@@ -462,6 +462,26 @@ def test_prefix_cache_restores_unequal_layers(base, tmp_path):
     assert m.prefill(p) == int(O.forward(CFG, w, p)[0][-1].argmax()) and m.prefix_store().hits == 1
 
 
+@each_form
+def test_verification_rows_and_draft_chain(base, device, dtype):
+    """Several rows per sequence in one decode-style step, across page and block edges; drafts of another model accepted or
+    refused give the tokens of plain decoding."""
+    from flyingfish_b200.spec.chain import ChainSpeculator
+    path, w = base
+    m = load(path, device, dtype)
+    for n in (48, 62, 99, 73):
+        toks = ids(n + 4, seed=100 + n)
+        s = m.engine.add_sequence(toks[:n])
+        m.engine.prefill([s])
+        s.pending = toks[n]
+        got = m.engine.verify([s], [toks[n + 1:]])[0]
+        lg = O.forward(CFG, w, toks)[0][n:]
+        assert all(row.max() - row[t] <= (1e-4 if dtype == "fp32" else 0.12) * row.std() for row, t in zip(lg, got)), n
+        m.engine.free_sequence(s.seq_id)
+    out = ChainSpeculator(m, load(path, device, dtype), k=3).generate(ids(40, seed=7), 30, ignore_eos=True)
+    greedy_agrees(w, ids(40, seed=7), out.ids[:30], dtype)
+
+
 # ------------------------------------------------------------------------------------------
 # configuration, checkpoint, command line, runner
 # ------------------------------------------------------------------------------------------
