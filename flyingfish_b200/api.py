@@ -18,6 +18,7 @@ import torch
 from .config import GPU_FP32_ARCHS, ModelSpec, Settings, named_shape, read_model_spec
 from .engine.engine import Engine, Sequence
 from .models.decoder import DecoderModel
+from .models.designs import design
 from .models.weights import TPInfo, random_decoder_weights
 from .planner.plan import plan_engine
 from .utils.log import log_json
@@ -77,12 +78,11 @@ class Model:
             from .loaders.checkpoint import load_decoder_weights
             from .loaders.tokenizer import load_tokenizer
             spec = with_dtype(read_model_spec(path), settings)
-            if spec.arch == "duponex":
+            if design(spec.arch) is not None:
                 from .loaders.checkpoint import audited_source
-                from .models.duponex import build_duponex_weights
                 source, close = audited_source(path, spec, device)
                 try:
-                    weights = build_duponex_weights(spec, source)
+                    weights = design(spec.arch).build_weights(spec, source)
                 finally:
                     close()
             elif spec.extra.get("hrm"):
@@ -101,9 +101,8 @@ class Model:
         else:
             spec = preset if preset is not None else (read_model_spec(path) if path.is_dir() else named_shape(model))
             spec = with_dtype(spec, settings)
-            if spec.arch == "duponex":
-                from .models.duponex import random_duponex_weights
-                weights = random_duponex_weights(spec, seed, device)
+            if design(spec.arch) is not None:
+                weights = design(spec.arch).random_weights(spec, seed, device)
             elif spec.extra.get("v41"):
                 from .models.deepseek_v41 import build_v41_weights
                 from .models.weights import DTYPES, synthetic_source
@@ -134,9 +133,8 @@ class Model:
         elif spec.extra.get("hrm"):
             from .models.hrm import HrmModel
             net = HrmModel(weights, comm=comm)
-        elif spec.arch == "duponex":
-            from .models.duponex import DuponexModel
-            net = DuponexModel(weights, comm=comm)
+        elif design(spec.arch) is not None:
+            net = design(spec.arch).build_model(weights, settings, comm)
         elif spec.extra.get("flint"):
             from .models.flint import FlintModel
             net = FlintModel(weights, comm=comm, seed=seed, state=weights.extra.get("state"))

@@ -403,9 +403,9 @@ def cmd_bench(args) -> dict:
     ctx = args.prompt_tokens + args.warmup + args.steps // 2
     t_, L, h, f = args.prompt_tokens, spec.layers, spec.hidden, spec.ffn
     if spec.layer_specs is not None:
-        kv_bytes = args.batch * spec.elem_bytes * sum(l.keys_seen(ctx) * l.kv_heads * (l.dim + l.vdim) for l in spec.layer_specs)
-        flops = 2 * t_ * (spec.dense_param_count() - 2 * spec.vocab * h) + 2 * h * spec.vocab + \
-            sum(2 * l.heads * (l.dim + l.vdim) * l.pairs_seen(t_) for l in spec.layer_specs)
+        runs = [spec.layer_specs[i] for i in spec.runs]
+        kv_bytes = args.batch * sum(l.cache_bytes_read(ctx, spec.elem_bytes) for l in runs)
+        flops = 2 * t_ * spec.run_params() + 2 * h * spec.vocab + sum(l.mixer_flops(t_) for l in runs)
     else:
         kv_bytes = args.batch * ctx * spec.layers * 2 * spec.kv_heads * spec.head_dim * 2
         flops = 2 * t_ * L * (h * spec.qkv_dim + h * h + 3 * h * f) + 2 * h * spec.vocab + 2 * h * t_ * (t_ + 1) * L

@@ -10,6 +10,7 @@ from __future__ import annotations
 
 import dataclasses
 import json
+import math
 from dataclasses import dataclass, field
 from pathlib import Path
 from typing import Any
@@ -29,6 +30,7 @@ class MoeSpec:
     renormalize: bool = True
     first_dense_layers: int = 0       # leading layers with a dense FFN
     dense_ffn: int = 0
+    identity: int = 0                 # router outputs behind the experts whose output is the input itself
     shared_gate: bool = False         # sigmoid gate on the shared expert (Qwen-style)
     expert_format: str = "bf16"       # bf16 | fp8_block | nvfp4
 
@@ -43,18 +45,45 @@ class MlaSpec:
 
 
 @dataclass
+class RopeSpec:
+    """Rotary positions on the first ``dims`` elements of a head, pairs being neighbours (2i, 2i + 1)."""
+    base: float
+    dims: int
+    factor: float = 1.0               # > 0 with ``original``: YaRN-scaled frequencies and amplitude
+    original: int = 0
+    fast: float = 32.0
+    slow: float = 1.0
+
+    def frequencies(self) -> tuple[list[float], float]:
+        """(angle per position of every pair, factor of cosine and sine), in double precision."""
+        plain = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if not self.original:
+            return plain, 1.0
+        turn = lambda t: self.dims * math.log(self.original / (2.0 * math.pi * t)) / (2.0 * math.log(self.base))
+        lo, hi = max(math.floor(turn(self.fast)), 0), min(math.ceil(turn(self.slow)), self.dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(self.dims // 2)]
+        return [f / self.factor * r + f * (1.0 - r) for f, r in zip(plain, ramp)], 0.1 * math.log(self.factor) + 1.0
+
+
+@dataclass
 class LayerSpec:
     """One layer of a design whose layers need not look alike (``ModelSpec.layer_specs``)."""
     heads: int
     kv_heads: int
     dim: int                          # width of a query / key head
     vdim: int                         # width of a value head
-    scale: float                      # factor of the attention scores
-    mixer: str = "attention"
+    scale: float                      # factor of the attention scores (of the queries, for a matrix memory)
+    mixer: str = "attention"          # attention | mlstm (matrix memory: per-sequence state instead of a cache)
     chunk: int = 0                    # > 0: position i sees only keys of its own block of ``chunk`` positions
+    window: int = 0                   # > 0: position i sees itself and the ``window - 1`` positions before it
+    sink: bool = False                # learnable soft-max: one extra logit per head in the denominator
+    rope: RopeSpec | None = None
+    gate_cap: float = 0.0             # matrix memory: soft cap of the gates' logits
+    out_gate: bool = True             # the heads' outputs are multiplied by the sigmoid of a projection
     v_mix: bool = False               # values are mixed with those of the first layer that has the flag
-    ffn: int = 0                      # width of the feed-forward (0: the layer has none)
+    ffn: int = 0                      # width of the feed-forward (0: the layer has none, or experts)
     ffn_act: str = "relu2"
+    moe: MoeSpec | None = None        # experts in place of a dense feed-forward
 
     @property
     def dim_pad(self) -> int:
@@ -66,18 +95,50 @@ class LayerSpec:
 
     def keys_seen(self, ctx: int) -> int:
         """Keys the last of ``ctx`` positions sees."""
+        if self.window:
+            return min(ctx, self.window)
         return (ctx - 1) % self.chunk + 1 if self.chunk else ctx
 
     def pairs_seen(self, n: int) -> int:
         """(query, key) pairs of a prompt of ``n`` positions."""
+        if self.window:
+            w = min(n, self.window)
+            return w * (w + 1) // 2 + (n - w) * w
         if not self.chunk:
             return n * (n + 1) // 2
         full, rest = divmod(n, self.chunk)
         return full * self.chunk * (self.chunk + 1) // 2 + rest * (rest + 1) // 2
 
+    def cache_bytes_read(self, ctx: int, elem_bytes: int) -> int:
+        """Bytes of cache or state one decoded token moves at a context of ``ctx``."""
+        if self.mixer == "mlstm":
+            return 2 * 4 * self.heads * self.dim * (self.vdim + 1)
+        return elem_bytes * self.keys_seen(ctx) * self.kv_heads * (self.dim + self.vdim)
+
+    def mixer_flops(self, n: int) -> int:
+        """FLOPs of a prompt of ``n`` positions outside the projections."""
+        if self.mixer == "mlstm":         # the recurrence: state update and read of every position
+            return 4 * n * self.heads * self.dim * self.vdim
+        return 2 * self.heads * (self.dim + self.vdim) * self.pairs_seen(n)
+
+    @property
+    def projection_cols(self) -> int:
+        """Columns of the fused input projection, heads padded."""
+        g = self.heads * self.vdim_pad if self.out_gate else 0
+        return self.heads * self.dim_pad + self.kv_heads * (self.dim_pad + self.vdim_pad) + g
+
+    def params(self, hidden: int, active: bool = False) -> int:
+        """Matrix weights of the layer; ``active``: those one token uses."""
+        n = hidden * (self.heads * (self.dim + self.vdim * (2 if self.out_gate else 1)) + self.kv_heads * (self.dim + self.vdim))
+        n += 2 * hidden * self.ffn + (2 * hidden * self.heads if self.mixer == "mlstm" else 0)
+        if self.moe is not None:
+            m = self.moe
+            n += hidden * (m.num_experts + m.identity) + 3 * hidden * (m.expert_ffn * (m.top_k if active else m.num_experts) + m.shared_ffn * m.n_shared)
+        return n
+
 
 # architectures whose every operator has a 32-bit kernel on the GPU
-GPU_FP32_ARCHS = ("duponex",)
+GPU_FP32_ARCHS = ("duponex", "rudorax")
 
 
 def pad_to(n: int, m: int) -> int:
@@ -87,7 +148,7 @@ def pad_to(n: int, m: int) -> int:
 @dataclass
 class ModelSpec:
     name: str
-    arch: str                         # llama | qwen3 | qwen3_moe | deepseek_v3 | deepseek_v41 | glm5_next | flint | loop_vl | tiny_moe | qwen3_vl | embedding | diffusion_lm | qwen35_text | gemma | duponex
+    arch: str                         # llama | qwen3 | qwen3_moe | deepseek_v3 | deepseek_v41 | glm5_next | flint | loop_vl | tiny_moe | qwen3_vl | embedding | diffusion_lm | qwen35_text | gemma | duponex | rudorax
     layers: int
     hidden: int
     heads: int
@@ -108,6 +169,7 @@ class ModelSpec:
     mla: MlaSpec | None = None
     mtp_layers: int = 0               # multi-token-prediction heads shipped with the checkpoint
     layer_specs: list[LayerSpec] | None = None    # per-layer sizes, for designs whose layers differ
+    loop: tuple[int, int, int] | None = None      # (start, stop, times): these layers run ``times`` times in a row; ``layers`` counts every run
     extra: dict[str, Any] = field(default_factory=dict)
 
     @property
@@ -126,30 +188,39 @@ class ModelSpec:
     def elem_bytes(self) -> int:
         return 4 if self.dtype == "fp32" else 2
 
+    @property
+    def runs(self) -> list[int]:
+        """Layer (index into ``layer_specs``) of every layer run, in order. A run has a cache or state of its own."""
+        n = len(self.layer_specs)
+        if self.loop is None:
+            return list(range(n))
+        a, b, times = self.loop
+        return list(range(a)) + list(range(a, b)) * times + list(range(b, n))
+
     def kv_geometry(self) -> list[tuple[int, int, int]] | None:
         """(kv heads, key width, value width) of every cache layer where the layers differ, None where one size serves
-        all. Widths are padded to 16 elements, the alignment of the attention kernels' tiles."""
+        all. Widths are padded to 16 elements, the alignment of the attention kernels' tiles; a run that keeps its past in a
+        per-sequence state has none."""
         if self.layer_specs is None:
             return None
-        return [(l.kv_heads, l.dim_pad, l.vdim_pad) for l in self.layer_specs]
+        size = lambda l: (l.kv_heads, l.dim_pad, l.vdim_pad) if l.mixer == "attention" else (0, 0, 0)
+        return [size(self.layer_specs[i]) for i in self.runs]
 
-    def _layer_spec_params(self) -> int:
-        n = 0
-        for l in self.layer_specs:
-            n += self.hidden * (l.heads * (l.dim + 2 * l.vdim) + l.kv_heads * (l.dim + l.vdim)) + 2 * self.hidden * l.ffn
-        return n
+    def run_params(self) -> int:
+        """Matrix weights one token passes through in all layer runs (a looped layer counts every time)."""
+        return sum(self.layer_specs[i].params(self.hidden, active=True) for i in self.runs)
 
     def dense_param_count(self) -> int:
         if self.layer_specs is not None:
-            return self._layer_spec_params() + (1 if self.tie_embeddings else 2) * self.vocab * self.hidden
+            return sum(l.params(self.hidden) for l in self.layer_specs) + (1 if self.tie_embeddings else 2) * self.vocab * self.hidden
         per_layer = self.hidden * self.qkv_dim + self.q_dim * self.hidden + 3 * self.hidden * self.ffn + 2 * self.hidden
         return self.layers * per_layer + (1 if self.tie_embeddings else 2) * self.vocab * self.hidden + self.hidden
 
     def decode_weight_bytes(self) -> int:
         """Bytes of weights read by one decode step (embedding row gathers excluded, lm_head
         included) -- the numerator of the reference's decode roofline (src/bench.rs:137-160)."""
-        if self.layer_specs is not None:
-            return self.elem_bytes * (self._layer_spec_params() + self.vocab * self.hidden)
+        if self.layer_specs is not None:      # experts: those one token uses
+            return self.elem_bytes * (self.run_params() + self.vocab * self.hidden)
         per_layer = self.hidden * self.qkv_dim + self.q_dim * self.hidden + 3 * self.hidden * self.ffn + 2 * self.hidden
         return 2 * (self.layers * per_layer + self.vocab * self.hidden + self.hidden)
 
@@ -394,6 +465,62 @@ def duponex_2b() -> ModelSpec:
     return _duponex_spec_of("duponex-2b-shape", 2048, 65536, layers, streams=4, residual_mult=0.5, embed_scale=8.0, eps=1e-5)
 
 
+def _rudorax_spec_of(name: str, hidden: int, vocab: int, layers: list[LayerSpec], embed_scale: float, eps: float,
+                     loop: tuple[int, int, int] | None = None, softcap: float = 0.0) -> ModelSpec:
+    if not layers:
+        raise ConfigError("a Rudorax model needs at least one layer")
+    for l in layers:
+        if min(l.heads, l.kv_heads, l.dim, l.vdim) < 1 or l.heads % l.kv_heads or l.window < 0 or not l.scale > 0:
+            raise ConfigError(f"unusable mixer sizes {l}")
+        if l.rope is not None and (l.rope.dims % 2 or not 0 < l.rope.dims <= l.dim or not l.rope.base > 1):
+            raise ConfigError(f"unusable rotation {l.rope} of heads of {l.dim}")
+        if l.mixer == "mlstm" and (not l.gate_cap > 0 or l.kv_heads != l.heads):
+            raise ConfigError("a matrix memory needs a positive gate cap and one key head per query head")
+        m = l.moe
+        if m is not None and (m.num_experts < 1 or m.identity < 0 or not 1 <= m.top_k <= min(m.num_experts + m.identity, 32) or m.expert_ffn < 1):
+            raise ConfigError(f"unusable experts {m}")
+    if loop is not None and not (0 <= loop[0] < loop[1] <= len(layers) and loop[2] >= 1):
+        raise ConfigError(f"loop {loop} outside the layers")
+    wide = max(layers, key=lambda l: l.heads * l.dim)
+    spec = ModelSpec(
+        name=name, arch="rudorax", layers=len(layers), hidden=hidden, heads=wide.heads, kv_heads=wide.kv_heads, head_dim=wide.dim,
+        ffn=0, vocab=vocab, rms_eps=eps, qk_norm=True, layer_specs=layers, loop=loop,
+        extra={"rudorax": {"embed_scale": embed_scale, "softcap": softcap}})
+    spec.layers = len(spec.runs)
+    return spec
+
+
+def rudorax_tiny() -> ModelSpec:
+    """Small Rudorax shape: windowed attention with sinks and scaled rotary positions, a matrix-memory layer, layers run
+    twice, experts with identity outputs and a shared expert."""
+    moe = MoeSpec(num_experts=6, top_k=3, expert_ffn=72, identity=2, n_shared=1, shared_ffn=104)
+    attn = dict(heads=4, kv_heads=2, dim=32, vdim=40, scale=0.2, window=72, sink=True, out_gate=False, moe=moe,
+                rope=RopeSpec(base=1e4, dims=24, factor=2.0, original=256))
+    mem = dict(heads=3, kv_heads=3, dim=24, vdim=48, scale=24 ** -0.5, mixer="mlstm", gate_cap=10.0, moe=moe)
+    return _rudorax_spec_of("rudorax-tiny", 160, 512, [LayerSpec(**attn), LayerSpec(**mem), LayerSpec(**dict(attn, kv_heads=1, window=40)),
+                                                       LayerSpec(**dict(attn, moe=None))],
+                            embed_scale=4.0, eps=1e-5, loop=(1, 3, 2), softcap=20.0)
+
+
+def _rudorax_bench(name: str, hidden: int, heads: int, kv_heads: int, experts: int, ff: int, vocab: int) -> ModelSpec:
+    moe = MoeSpec(num_experts=experts, top_k=8, expert_ffn=ff, identity=experts // 8, n_shared=1, shared_ffn=ff)
+    attn = LayerSpec(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, window=2048, sink=True, out_gate=False, moe=moe,
+                     rope=RopeSpec(base=1e6, dims=128, factor=4.0, original=8192))
+    mem = LayerSpec(heads=hidden // 256, kv_heads=hidden // 256, dim=128, vdim=256, scale=128 ** -0.5, mixer="mlstm", gate_cap=15.0, moe=moe)
+    return _rudorax_spec_of(name, hidden, vocab, [attn, mem, attn, mem], embed_scale=8.0, eps=1e-5, loop=(1, 3, 2), softcap=30.0)
+
+
+def rudorax_2k() -> ModelSpec:
+    """Rudorax layers 2048 wide (random weights, for measurements): 16 / 4 attention heads of 128, 8 memories of 128 x 256,
+    64 experts of 768 and 8 identity outputs, top 8, six layer runs."""
+    return _rudorax_bench("rudorax-2k-shape", 2048, 16, 4, 64, 768, 65536)
+
+
+def rudorax_4k() -> ModelSpec:
+    """As :func:`rudorax_2k` at 4096: 32 / 8 heads, 16 memories, 64 experts of 1536."""
+    return _rudorax_bench("rudorax-4k-shape", 4096, 32, 8, 64, 1536, 128256)
+
+
 def glm5_next_tiny() -> ModelSpec:
     """Small GLM-5-style shape: the hyper-connection program with every stage collapsing on its own pre-mix, top-k sparse
     attention with the pooled indexer in every layer, sigmoid routing with selection bias."""
@@ -409,6 +536,7 @@ NAMED_SHAPES = {
     "deepseek-v3-shape": deepseek_v3, "deepseek-v3-tiny": deepseek_v3_tiny, "deepseek-v3-mini": deepseek_v3_mini,
     "deepseek-v3-fp8-mini": deepseek_v3_fp8_mini, "deepseek-v41-tiny": deepseek_v41_tiny, "glm5-next-tiny": glm5_next_tiny, "flint-tiny": flint_tiny,
     "duponex-tiny": duponex_tiny, "duponex-8b-shape": duponex_8b, "duponex-2b-shape": duponex_2b,
+    "rudorax-tiny": rudorax_tiny, "rudorax-2k-shape": rudorax_2k, "rudorax-4k-shape": rudorax_4k,
     "loop-tiny": loop_tiny, "loopvl-text-shape": loopvl_text,
     "qwen3-moe-235b-shape": qwen3_moe_235b, "qwen3-moe-tiny": qwen3_moe_tiny,
 }
@@ -534,11 +662,47 @@ def _duponex_spec(cfg: dict[str, Any], name: str) -> ModelSpec:
                             eps=float(cfg["norm"]["eps"]))
 
 
+def _rudorax_spec(cfg: dict[str, Any], name: str) -> ModelSpec:
+    """``"architecture": "Rudorax"``: a list of layers with attention or matrix-memory mixers and expert feed-forwards, a range of
+    which may run several times."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+        m, mlp, moe = entry["mixer"], entry.get("mlp"), None
+        if mlp is not None:
+            if mlp.get("kind", "moe") != "moe":
+                raise ConfigError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r}")
+            r, sh = mlp["router"], mlp.get("shared")
+            moe = MoeSpec(num_experts=int(r["experts"]), top_k=int(r["top"]), expert_ffn=int(mlp["expert"]["ff"]), score="softmax",
+                          identity=int(r.get("identity") or 0), n_shared=1 if sh else 0, shared_ffn=int(sh["ff"]) if sh else 0)
+        sizes = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), moe=moe)
+        if entry.get("type") == "attention":
+            rot = m.get("rot")
+            rope = None
+            if rot is not None:
+                sc = rot.get("scaling")
+                rope = RopeSpec(base=float(rot["base"]), dims=int(rot["dims"]))
+                if sc is not None:
+                    rope = dataclasses.replace(rope, factor=float(sc["factor"]), original=int(sc["original"]), fast=float(sc["fast"]),
+                                               slow=float(sc["slow"]))
+            layers.append(LayerSpec(kv_heads=int(m["kv_heads"]), scale=float(m["scale"]), window=int((m.get("mask") or {}).get("size", 0)),
+                                    sink=True, rope=rope, out_gate=False, **sizes))
+        elif entry.get("type") == "mlstm":
+            layers.append(LayerSpec(kv_heads=sizes["heads"], scale=sizes["dim"] ** -0.5, mixer="mlstm", gate_cap=float(m["gate_cap"]), **sizes))
+        else:
+            raise ConfigError(f"layer {i}: unsupported mixer {entry.get('type')!r}")
+    loop = cfg.get("loop")
+    return _rudorax_spec_of(name, int(cfg["width"]), int(cfg["vocab"]), layers, embed_scale=float(cfg["embedding"]["scale"]),
+                            eps=float(cfg["norm"]["eps"]), softcap=float(cfg.get("logit_softcap") or 0.0),
+                            loop=(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None)
+
+
 def spec_from_hf_config(cfg: dict[str, Any], name: str = "model") -> ModelSpec:
     """Normalise a Hugging Face ``config.json``. Hard checks mirror the reference's: SiLU
     activation only, 16-bit or 32-bit floats, no unsupported rope scaling for plain Llama."""
     if cfg.get("architecture") == "Duponex":
         return _duponex_spec(cfg, name)
+    if cfg.get("architecture") == "Rudorax":
+        return _rudorax_spec(cfg, name)
     archs = cfg.get("architectures") or []
     arch = next((_ARCH_MAP[a] for a in archs if a in _ARCH_MAP), None)
     if arch is None:

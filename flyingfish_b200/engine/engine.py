@@ -125,6 +125,8 @@ class Engine:
             # a model whose state kernels take their slots from the packed step metadata can be captured
             if not getattr(model, "graph_safe_state", False):
                 self.use_graph = False
+            if settings.prefix_cache:
+                raise ValueError("--prefix-cache keeps K and V only: not available for a model with recurrent state")
         self.stats = {"prefill_tokens": 0, "decode_steps": 0, "decode_tokens": 0, "graph_replays": 0,
                       "captures": 0, "h2d_bytes": 0, "d2h_bytes": 0}
         self.fail_next_step = False      # host-side fault injection hook for tests
@@ -600,8 +602,11 @@ class Engine:
                 c.seal(self.kv, s.seq_id)
 
     def _no_compact(self, what: str) -> None:
+        """Refuse what only works on the BF16 block cache: rows that may be taken back."""
         if self.kv.compact is not None:
             raise ValueError(f"{what} reads BF16 pages only and is not available with --kv-format affine8")
+        if self.state_slots is not None:
+            raise ValueError(f"{what} is not available for a model with recurrent state (a state cannot be taken back)")
 
     def capture_verify(self, bucket: int, nq: int) -> _Graph:
         """Capture the verification step of ``nq`` rows per sequence for a batch bucket (decode-style attention over

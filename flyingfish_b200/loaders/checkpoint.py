@@ -17,6 +17,7 @@ from pathlib import Path
 import torch
 
 from ..config import ModelSpec, read_model_spec
+from ..models.designs import design
 from ..models.weights import DTYPES, ModelWeights, TPInfo, build_decoder_weights
 from .safetensors_io import CheckpointError, MappedCheckpoint
 
@@ -38,9 +39,8 @@ def _linear_entries(name: str, out_f: int, in_f: int, fmt: str) -> dict[str, tup
 
 def manifest(spec: ModelSpec, policy: LoadPolicy = LoadPolicy.TEXT_ONLY) -> dict[str, tuple[tuple[int, ...], str]]:
     """name -> (shape, dtype class in {float, f32, fp8, u8})."""
-    if spec.arch == "duponex":
-        from ..models.duponex import expected_tensors
-        return {n: (shape, "float") for n, shape in expected_tensors(spec).items()}
+    if design(spec.arch) is not None:
+        return {n: (shape, "float") for n, shape in design(spec.arch).expected_tensors(spec).items()}
     m: dict[str, tuple[tuple[int, ...], str]] = {}
     h, d = spec.hidden, spec.head_dim
     m["model.embed_tokens.weight"] = ((spec.vocab, h), "float")
@@ -254,9 +254,8 @@ def audited_source(model_dir: str | Path, spec: ModelSpec, device: torch.device 
     know)."""
     ck = MappedCheckpoint(Path(model_dir))
     extra: tuple[str, ...] = ()
-    if spec.arch == "duponex":
-        from ..models.duponex import unused_tensors
-        extra = unused_tensors(spec)
+    if design(spec.arch) is not None:
+        extra = design(spec.arch).unused_tensors(spec)
     try:
         audit(ck, spec, allow_extra=extra)
     finally:

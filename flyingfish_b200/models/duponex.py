@@ -29,7 +29,7 @@ from .. import ops
 from ..config import LayerSpec, ModelSpec, pad_to
 from ..ops import stream_ops
 from .decoder import DecoderModel
-from .weights import DTYPES, LayerWeights, ModelWeights, TensorSource, TPInfo, random_tensor
+from .weights import DTYPES, LayerWeights, ModelWeights, TensorSource, TPInfo, pad_cols, pad_heads, random_tensor
 
 
 # ------------------------------------------------------------------------------------------
@@ -65,30 +65,13 @@ def unused_tensors(spec: ModelSpec) -> tuple[str, ...]:
     return tuple(names)
 
 
-def _pad_cols(t: torch.Tensor, cols: int) -> torch.Tensor:
-    if t.shape[-1] == cols:
-        return t.contiguous()
-    out = t.new_zeros(*t.shape[:-1], cols)
-    out[..., : t.shape[-1]] = t
-    return out
-
-
-def _pad_heads(t: torch.Tensor, heads: int, width: int, padded: int) -> torch.Tensor:
-    """Rows of ``heads`` heads of ``width`` -> heads of ``padded`` rows (zeros behind each head's own)."""
-    if width == padded:
-        return t
-    out = t.new_zeros(heads, padded, *t.shape[1:])
-    out[:, :width] = t.view(heads, width, *t.shape[1:])
-    return out.reshape(heads * padded, *t.shape[1:])
-
-
-def build_duponex_weights(spec: ModelSpec, source: TensorSource) -> ModelWeights:
+def build_weights(spec: ModelSpec, source: TensorSource) -> ModelWeights:
     """Fused and padded weights: ``wqkv`` = [q | k | v | gate] with one bias vector, heads padded to 16 elements, the
     residual width and the feed-forward width to 8."""
     shapes = expected_tensors(spec)
     get = lambda n: source(n, shapes[n])
     wp = pad_to(spec.hidden, 8)
-    vec = lambda n: _pad_cols(get(n), wp)
+    vec = lambda n: pad_cols(get(n), wp)
     layers = []
     for i, l in enumerate(spec.layer_specs):
         p = f"l{i}."
@@ -99,32 +82,32 @@ def build_duponex_weights(spec: ModelSpec, source: TensorSource) -> ModelWeights
         w, b = [], []
         for name, heads, width, padded in parts:
             t = get(p + "mix." + name)
-            w.append(_pad_heads(_pad_cols(t, wp), heads, width, padded))
+            w.append(pad_heads(pad_cols(t, wp), heads, width, padded))
             bias = get(p + f"mix.{name}.b") if name != "g" else t.new_zeros(heads * width)
-            b.append(_pad_heads(bias, heads, width, padded))
+            b.append(pad_heads(bias, heads, width, padded))
         lw.wqkv, lw.extra["bqkv"] = torch.cat(w).contiguous(), torch.cat(b).contiguous()
-        o = _pad_heads(get(p + "mix.o").t().contiguous(), l.heads, l.vdim, dv).t()
-        lw.wo = _pad_cols(o.t().contiguous(), wp).t().contiguous()
+        o = pad_heads(get(p + "mix.o").t().contiguous(), l.heads, l.vdim, dv).t()
+        lw.wo = pad_cols(o.t().contiguous(), wp).t().contiguous()
         lw.extra["bo"] = vec(p + "mix.o.b")
         lw.extra["vmix"] = float(get(p + "mix.vmix")) if l.v_mix else 0.0
         if l.ffn:
             lw.post_ln = vec(p + "norm2")
             fp = pad_to(l.ffn, 8)
-            up, down = _pad_cols(get(p + "mlp.up"), wp), _pad_cols(get(p + "mlp.down"), fp)
-            lw.wgu = _pad_cols(up.t().contiguous(), fp).t().contiguous()
-            lw.wdown = _pad_cols(down.t().contiguous(), wp).t().contiguous()
+            up, down = pad_cols(get(p + "mlp.up"), wp), pad_cols(get(p + "mlp.down"), fp)
+            lw.wgu = pad_cols(up.t().contiguous(), fp).t().contiguous()
+            lw.wdown = pad_cols(down.t().contiguous(), wp).t().contiguous()
             lw.wgu_interleaved = False
         for n in (1, 2) if l.ffn else (1,):
             lw.extra[f"ls{n}"] = vec(p + f"ls{n}")
             lw.extra[f"hc{n}"] = {k: get(p + f"hc{n}.{k}").float().cpu() for k in ("in", "out", "mix")}
         layers.append(lw)
-    head = _pad_cols(get("head"), wp)
-    head = _pad_cols(head.t().contiguous(), pad_to(spec.vocab, 8)).t().contiguous()
-    return ModelWeights(spec=spec, embed=_pad_cols(get("embed"), wp), final_norm=vec("final.norm"), lm_head=head, layers=layers,
+    head = pad_cols(get("head"), wp)
+    head = pad_cols(head.t().contiguous(), pad_to(spec.vocab, 8)).t().contiguous()
+    return ModelWeights(spec=spec, embed=pad_cols(get("embed"), wp), final_norm=vec("final.norm"), lm_head=head, layers=layers,
                         tp=TPInfo(), vocab_shard=(0, spec.vocab))
 
 
-def random_duponex_weights(spec: ModelSpec, seed: int, device: torch.device | str) -> ModelWeights:
+def random_weights(spec: ModelSpec, seed: int, device: torch.device | str) -> ModelWeights:
     """Seeded weights in which every mechanism counts: norms, layer scales and stream matrices near one, none equal."""
     device = torch.device(device)
     dtype = DTYPES[spec.dtype]
@@ -147,7 +130,7 @@ def random_duponex_weights(spec: ModelSpec, seed: int, device: torch.device | st
         elif leaf.endswith(".b"):
             t = 0.3 * t
         return t.to(dtype)
-    return build_duponex_weights(spec, source)
+    return build_weights(spec, source)
 
 
 # ------------------------------------------------------------------------------------------
@@ -242,3 +225,7 @@ class DuponexModel(DecoderModel):
 
     def logits(self, n, b):
         return super().logits(n, b)[:, : self.spec.vocab]
+
+
+def build_model(weights: ModelWeights, settings, comm=None) -> DuponexModel:
+    return DuponexModel(weights, comm=comm)

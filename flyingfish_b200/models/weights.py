@@ -130,6 +130,24 @@ def shard_range(n: int, rank: int, size: int) -> tuple[int, int]:
     return rank * per, (rank + 1) * per
 
 
+def pad_cols(t: torch.Tensor, cols: int) -> torch.Tensor:
+    """The last dimension widened to ``cols`` with zeros."""
+    if t.shape[-1] == cols:
+        return t.contiguous()
+    out = t.new_zeros(*t.shape[:-1], cols)
+    out[..., : t.shape[-1]] = t
+    return out
+
+
+def pad_heads(t: torch.Tensor, heads: int, width: int, padded: int) -> torch.Tensor:
+    """Rows of ``heads`` heads of ``width`` -> heads of ``padded`` rows (zeros behind each head's own)."""
+    if width == padded:
+        return t.contiguous()
+    out = t.new_zeros(heads, padded, *t.shape[1:])
+    out[:, :width] = t.view(heads, width, *t.shape[1:])
+    return out.reshape(heads * padded, *t.shape[1:])
+
+
 def pack_ffn_fp8(lw: "LayerWeights") -> None:
     """Re-encode a layer's feed-forward matrices as FP8-resident weights (E4M3 codes + 128x128 block scales): the
     dense gate/up and down projections, the shared expert, and the routed experts (gate/up interleaved per 64 rows,

@@ -67,6 +67,7 @@ def _rows2d(t: torch.Tensor) -> tuple[int, int]:
 class _Workspace:
     def __init__(self, device: torch.device):
         self.device = device
+        self.retired: list[torch.Tensor] = []
         self.gemm_scratch = torch.empty(8 << 20, dtype=torch.float32, device=device)      # 32 MiB
         self.gemm_counters = torch.zeros(4096, dtype=torch.int32, device=device)
         self.attn_o = torch.empty(4 << 20, dtype=torch.float32, device=device)             # 16 MiB
@@ -79,6 +80,7 @@ class _Workspace:
             t = torch.empty(0, dtype=torch.float32, device=self.device)
         if t.numel() < numel:
             _require(not torch.cuda.is_current_stream_capturing(), f"workspace {name} too small during graph capture")
+            self.retired.append(t)         # captured graphs keep writing to the buffer they were captured with
             t = torch.empty(int(numel * 1.25), dtype=t.dtype, device=self.device)
             setattr(self, name, t)
         return t
@@ -163,21 +165,23 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
     st = status_tensor(x.device)
     plain = bias is None and act is None
     _require(plain or odt == BF16, "linear: bias and activation come with a bf16 output")
-    if m <= SKINNY_MAX_M and odt == BF16:
+    _require(odt in (BF16, torch.float32), "linear: output dtype must be bf16 or fp32")
+    if m <= SKINNY_MAX_M:
         scratch_b, counter_b = c_longlong(0), c_longlong(0)
         splits = lib.ff_gemm_skinny_plan(m, n, k, ctypes.byref(scratch_b), ctypes.byref(counter_b))
         ws = workspace(x.device)
         scratch = ws.ensure("gemm_scratch", scratch_b.value // 4) if scratch_b.value > 0 else None
         _require(counter_b.value // 4 <= ws.gemm_counters.numel(), "linear: too many column tiles for counters")
         args = (ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), splits, ptr(scratch), ptr(ws.gemm_counters))
-        if plain:
+        if odt == torch.float32:
+            rc = lib.ff_gemm_skinny_f32out(*args, ptr(st), stream_ptr())
+        elif plain:
             rc = lib.ff_gemm_skinny(*args, ptr(st), stream_ptr())
         else:
             rc = lib.ff_gemm_skinny_act(*args, ptr(bias), ACTIVATIONS[act], ptr(st), stream_ptr())
         check(rc, "ff_gemm_skinny")
     else:
         epi = 0 if odt == BF16 else 2
-        _require(odt in (BF16, torch.float32), "linear: output dtype must be bf16 or fp32")
         if plain:
             rc = lib.ff_gemm_bf16(ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), epi, ptr(st), stream_ptr())
         else:
@@ -210,6 +214,8 @@ def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tenso
     the per-64 interleaved ``[2f, h]`` matrix built by :func:`ref.interleave_gate_up`."""
     if not _is_cuda(x):
         return ref.linear_swiglu(x, w_interleaved, mode)
+    if x.dtype == torch.float32:
+        return silu_mul_interleaved(linear(x, w_interleaved), out)
     m, ldx = _rows2d(x)
     n, ldw = _rows2d(w_interleaved)
     k = x.shape[1]
@@ -414,13 +420,16 @@ def linear_rope_kv(x: torch.Tensor, wqkv: torch.Tensor, positions: torch.Tensor,
 
 
 def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, hq: int, hkv: int,
-                 dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0) -> None:
-    """Packed rows ``[q heads | k heads | v heads | ...]``: q and k are divided by their root mean square per head (no
-    weight; ``dim`` elements count, the row's heads may carry padding up to the cache's width), v is blended with
+                 dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0,
+                 q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None,
+                 cos_sin: torch.Tensor | None = None) -> None:
+    """Packed rows ``[q heads | k heads | v heads | ...]``: q and k are divided by their root mean square per head
+    (``dim`` elements count, the row's heads may carry padding up to the cache's width), v is blended with
     ``first_v`` (``(1 - mix) v + mix first_v``; a column slice of an earlier layer's packed rows), k and v are written to
-    ``slots`` of the paged cache and q back into the row. No positions enter. BF16 or FP32."""
+    ``slots`` of the paged cache and q back into the row. ``q_weight`` / ``k_weight``: FP32 norm weights as wide
+    as the row's heads; ``cos_sin`` (:func:`rope_angles`): neighbours (2i, 2i + 1) of the normed q and k turn. BF16 or FP32."""
     if not _is_cuda(qkv):
-        ref.head_norm_kv(qkv, slots, kcache, vcache, hq, hkv, dim, vdim, eps, first_v, mix)
+        ref.head_norm_kv(qkv, slots, kcache, vcache, hq, hkv, dim, vdim, eps, first_v, mix, q_weight, k_weight, cos_sin)
         return
     rows, ld = _rows2d(qkv)
     nb, ch, bs, dk = kcache.shape
@@ -433,11 +442,39 @@ def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, v
     if first_v is not None:
         _require(first_v.shape == (rows, hkv * dv) and first_v.stride(1) == 1 and first_v.dtype == qkv.dtype, "head_norm_kv: first values")
         ldf = first_v.stride(0)
+    for w in (q_weight, k_weight):
+        _require(w is None or (w.dtype == torch.float32 and w.numel() == dk and w.is_contiguous()), "head_norm_kv: norm weights")
+    half = 0
+    if cos_sin is not None:
+        half = cos_sin.shape[1]
+        _require(cos_sin.shape == (rows, half, 2) and cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and 2 * half <= dim,
+                 "head_norm_kv: rotation table")
     rc = kernels().ff_head_norm_kv(ptr(qkv), ptr(slots), ptr(kcache), ptr(vcache), ptr(first_v), rows, hq, hkv, dim, dk, dv, bs, nb, ld,
-                                   ldf, c_float(eps), c_float(mix), int(qkv.dtype == torch.float32), ptr(status_tensor(qkv.device)),
-                                   stream_ptr())
+                                   ldf, c_float(eps), c_float(mix), ptr(q_weight), ptr(k_weight), ptr(cos_sin), half,
+                                   int(qkv.dtype == torch.float32), ptr(status_tensor(qkv.device)), stream_ptr())
     check(rc, "ff_head_norm_kv")
     _count()
+
+
+def rope_frequencies(freqs: list[float], device) -> torch.Tensor:
+    """Frequencies given in double precision as FP32 (value, remainder) pairs [n, 2], the form :func:`rope_angles` takes."""
+    f = torch.tensor(freqs, dtype=torch.float64)
+    hi = f.float()
+    return torch.stack([hi, (f - hi.double()).float()], dim=-1).contiguous().to(device)
+
+
+def rope_angles(positions: torch.Tensor, freqs: torch.Tensor, amp: float = 1.0) -> torch.Tensor:
+    """``[rows, n, 2]`` FP32 (cos, sin) of ``position * frequency``, times ``amp``; nothing is rounded to 16 bits. Computed once
+    per step for every layer with the same rotation."""
+    if not _is_cuda(positions):
+        a = positions.double()[:, None] * freqs.double().sum(-1)[None, :]
+        return torch.stack([torch.cos(a) * amp, torch.sin(a) * amp], dim=-1).float()
+    rows, half = positions.shape[0], freqs.shape[0]
+    _require(positions.dtype == torch.int32 and freqs.dtype == torch.float32 and freqs.is_contiguous(), "rope_angles: operand types")
+    out = torch.empty(rows, half, 2, dtype=torch.float32, device=positions.device)
+    check(kernels().ff_rope_angles(ptr(positions), ptr(freqs), c_float(amp), ptr(out), rows, half, stream_ptr()), "ff_rope_angles")
+    _count()
+    return out
 
 
 def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0, out: torch.Tensor | None = None,
@@ -450,6 +487,13 @@ def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0, out: torch.Ten
         return ref.silu_mul(gu, mode, limit)
     rows, ld = _rows2d(gu)
     f = gu.shape[1] // 2
+    if gu.dtype == torch.float32:          # 32-bit form: nothing in between is rounded
+        _require(mode in (0, 1), "silu_mul: the FP32 form is plain SwiGLU")
+        if out is None:
+            out = torch.empty(rows, f, dtype=torch.float32, device=gu.device)
+        check(kernels().ff_silu_mul_f32(ptr(gu), ptr(out), rows, f, ld, out.stride(0), int(interleaved), stream_ptr()), "ff_silu_mul_f32")
+        _count()
+        return out
     if out is None:
         out = torch.empty(rows, f, dtype=BF16, device=gu.device)
     rc = kernels().ff_silu_mul(ptr(gu), ptr(out), rows, f, ld, out.stride(0), mode, c_float(limit), int(interleaved), stream_ptr())
@@ -461,8 +505,8 @@ def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0, out: torch.Ten
 def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
     if not _is_cuda(x):
         return ref.softcap(x, cap)
-    _require(x.is_contiguous() and x.dtype == BF16, "softcap: contiguous bf16")
-    check(kernels().ff_softcap(ptr(x), c_longlong(x.numel()), c_float(cap), stream_ptr()), "ff_softcap")
+    _require(x.is_contiguous() and x.dtype in (BF16, torch.float32), "softcap: contiguous bf16 or fp32")
+    check(kernels().ff_softcap(ptr(x), c_longlong(x.numel()), c_float(cap), int(x.dtype == torch.float32), stream_ptr()), "ff_softcap")
     _count()
     return x
 
@@ -504,8 +548,8 @@ def attn_decode(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, blo
     _require(ctx_lens.dtype == torch.int32, "attn_decode: ctx_lens int32")
     nb = kcache.shape[0]
     if q.dtype == torch.float32 or max(dim, vdim) > 128:
-        _require(sinks is None and tree_mask is None, "attn_decode: the SIMT kernel has no sinks or tree masks")
-        return _attn_simt(q, kcache, vcache, block_table, None, None, ctx_lens, nq, hq, hkv, dim, vdim, scale, window, chunk, gate, out)
+        _require(tree_mask is None, "attn_decode: the SIMT kernel has no tree masks")
+        return _attn_simt(q, kcache, vcache, block_table, None, None, ctx_lens, nq, hq, hkv, dim, vdim, scale, window, chunk, gate, out, sinks)
     _require(kcache.shape[2] == 64 and kcache.shape[3] == dim and vcache.shape[3] == vdim, "attn_decode: 64-token blocks of these heads")
     _require(dim % 16 == 0 and vdim % 16 == 0, "attn_decode: head widths must be multiples of 16")
     general = chunk > 0 or gate is not None or dim != 128 or vdim != 128
@@ -564,7 +608,8 @@ def _gate_ld(gate: torch.Tensor | None, rows: int, width: int) -> int:
 
 
 def _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, nq: int, hq: int, hkv: int, dim: int, vdim: int,
-               scale: float, window: int, chunk: int, gate: torch.Tensor | None, out: torch.Tensor | None) -> torch.Tensor:
+               scale: float, window: int, chunk: int, gate: torch.Tensor | None, out: torch.Tensor | None,
+               sinks: torch.Tensor | None = None) -> torch.Tensor:
     """Paged attention of any head width, BF16 or FP32 (``csrc/attention_simt.cu``): one warp per query row and head.
     Rows come as ranges (``q_start`` / ``q_lens``) or, without them, ``nq`` per sequence."""
     rows, ldq = _rows2d(q)
@@ -572,10 +617,11 @@ def _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, nq: in
         out = torch.empty(rows, hq * vdim, dtype=q.dtype, device=q.device)
     _require(q.dtype == kcache.dtype == vcache.dtype == out.dtype and q.dtype in (BF16, torch.float32), "attention: one type throughout")
     _require(kcache.shape[1] == hkv and kcache.shape[3] == dim and vcache.shape[3] == vdim and out.stride(1) == 1, "attention: geometry")
+    _require(sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == hq and sinks.is_contiguous()), "attention: sinks float32 [hq]")
     rc = kernels().ff_attn_simt(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(out),
                                 block_table.shape[0], rows, nq, hq, hkv, dim, vdim, ldq, out.stride(0), kcache.shape[2],
                                 block_table.shape[1], kcache.shape[0], c_float(scale), window, chunk, ptr(gate),
-                                _gate_ld(gate, rows, hq * vdim), int(q.dtype == torch.float32), ptr(status_tensor(q.device)), stream_ptr())
+                                _gate_ld(gate, rows, hq * vdim), ptr(sinks), int(q.dtype == torch.float32), ptr(status_tensor(q.device)), stream_ptr())
     check(rc, "ff_attn_simt")
     _count()
     return out
@@ -672,8 +718,8 @@ def attn_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
         out = torch.empty(rows, hq * vdim, dtype=q.dtype, device=q.device)
     nb = kcache.shape[0]
     if q.dtype == torch.float32 or max(dim, vdim) > 128:
-        _require(sinks is None, "attn_prefill: the SIMT kernel has no sinks")
-        return _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, 1, hq, hkv, dim, vdim, scale, window, chunk, gate, out)
+        return _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, 1, hq, hkv, dim, vdim, scale, window, chunk, gate, out,
+                          sinks)
     general = chunk > 0 or gate is not None or dim != 128 or vdim != 128
     _require(kcache.shape[2] == 64 and kcache.shape[3] == dim and vcache.shape[3] == vdim and dim % 16 == 0 and vdim % 16 == 0,
              "attn_prefill: 64-token blocks, head widths in multiples of 16")

@@ -52,6 +52,8 @@ def _hash(files: list[Path], extra: str = "") -> str:
 ARCH_SOURCES = {
     "duponex": ("attention_paged", "attention_simt", "attention_tc", "gemm_bf16", "gemm_f32", "gemm_skinny", "head_norm",
                 "kv_util", "rope_act_sample", "streams"),
+    "rudorax": ("attention_paged", "attention_simt", "attention_tc", "gemm_bf16", "gemm_f32", "gemm_skinny", "head_norm",
+                "kv_util", "mlstm", "moe", "residual", "rope_act_sample"),
 }
 
 

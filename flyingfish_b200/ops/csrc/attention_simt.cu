@@ -1,7 +1,7 @@
 // Paged attention on the CUDA cores, for what the tensor-core kernels do not take: FP32 caches and head widths above 128.
 // One warp per (query row, head): 32 keys at a time, a key per lane for the scores, a channel per lane for the values,
 // soft-max and accumulation in FP32 (online). Causal, sliding window, block-local (`chunk`) or bidirectional; an optional
-// output gate. Rows come as ranges (q_start / q_lens; chunked prefill) or nq per sequence (decode).
+// output gate and sinks. Rows come as ranges (q_start / q_lens; chunked prefill) or nq per sequence (decode).
 #include "dtype_io.cuh"
 #include "host_util.h"
 
@@ -14,7 +14,7 @@ __global__ void __launch_bounds__(32 * AS_WARPS)
 attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kcache, const T* __restrict__ vcache, const int* __restrict__ block_table,
                  const int* __restrict__ q_start, const int* __restrict__ q_lens, const int* __restrict__ ctx_lens, T* __restrict__ out,
                  int batch, int rows, int nq, int hq, int hkv, int dk, int dv, int ldq, int ldo, int page, int max_blocks,
-                 int num_blocks, float scale, int window, int chunk, const T* __restrict__ gate, int ldg, int* status) {
+                 int num_blocks, float scale, int window, int chunk, const T* __restrict__ gate, int ldg, const float* __restrict__ sinks, int* status) {
   pdl_trigger();
   pdl_wait();
   extern __shared__ __align__(16) float as_q[];            // [AS_WARPS][dk]
@@ -85,6 +85,13 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kcache, const T*
       }
     }
   }
+  // learnable soft-max: the head's sink logit enters the denominator only
+  if (sinks != nullptr && m > -INFINITY) {
+    const float sk = sinks[h], mn = fmaxf(m, sk), a = expf(m - mn);
+    l = l * a + expf(sk - mn);
+#pragma unroll
+    for (int j = 0; j < NV; ++j) acc[j] *= a;
+  }
   const float inv = l > 0.f ? 1.0f / l : 0.f;
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
@@ -101,14 +108,14 @@ template <typename T>
 static int attn_simt_launch(const void* q, const void* kc, const void* vc, const int* bt, const int* q_start, const int* q_lens,
                             const int* ctx_lens, void* out, int batch, int rows, int nq, int hq, int hkv, int dk, int dv, int ldq, int ldo,
                             int page, int max_blocks, int num_blocks, float scale, int window, int chunk, const void* gate, int ldg,
-                            int* status, cudaStream_t s) {
+                            const float* sinks, int* status, cudaStream_t s) {
   const long long blocks = ((long long)rows * hq + AS_WARPS - 1) / AS_WARPS;
   const int smem = AS_WARPS * dk * 4;
   auto go = [&](auto kern) -> int {
     if (int r = opt_in_smem(kern, smem)) return r;
     if (int r = launch_pdl(kern, dim3((unsigned)blocks), dim3(32 * AS_WARPS), smem, s, 0, (const T*)q, (const T*)kc, (const T*)vc, bt, q_start, q_lens,
                            ctx_lens, (T*)out, batch, rows, nq, hq, hkv, dk, dv, ldq, ldo, page, max_blocks, num_blocks, scale, window, chunk,
-                           (const T*)gate, ldg, status)) return r;
+                           (const T*)gate, ldg, sinks, status)) return r;
     return launch_result();
   };
   if (dv <= 128) return go(attn_simt_kernel<T, 4>);
@@ -123,11 +130,11 @@ using namespace ff;
 FF_EXPORT int ff_attn_simt(const void* q, const void* kcache, const void* vcache, const int* block_table, const int* q_start,
                            const int* q_lens, const int* ctx_lens, void* out, int batch, int rows, int nq, int hq, int hkv, int dk, int dv,
                            int ldq, int ldo, int page, int max_blocks, int num_blocks, float scale, int window, int chunk, const void* gate,
-                           int ldg, int f32, int* status, cudaStream_t s) {
+                           int ldg, const float* sinks, int f32, int* status, cudaStream_t s) {
   if (batch <= 0 || rows <= 0 || nq < 1 || hq <= 0 || hkv <= 0 || hq % hkv || dk <= 0 || dk % 4 || dv <= 0 || page <= 0 || chunk < 0)
     return FF_HOST_BAD_SHAPE;
   if ((q_start == nullptr) != (q_lens == nullptr) || (q_start == nullptr && rows != batch * nq)) return FF_HOST_BAD_SHAPE;
   if (window != 0 && chunk > 0) return FF_HOST_UNSUPPORTED;
-  if (f32) return attn_simt_launch<float>(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, out, batch, rows, nq, hq, hkv, dk, dv, ldq, ldo, page, max_blocks, num_blocks, scale, window, chunk, gate, ldg, status, s);
-  return attn_simt_launch<__nv_bfloat16>(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, out, batch, rows, nq, hq, hkv, dk, dv, ldq, ldo, page, max_blocks, num_blocks, scale, window, chunk, gate, ldg, status, s);
+  if (f32) return attn_simt_launch<float>(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, out, batch, rows, nq, hq, hkv, dk, dv, ldq, ldo, page, max_blocks, num_blocks, scale, window, chunk, gate, ldg, sinks, status, s);
+  return attn_simt_launch<__nv_bfloat16>(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, out, batch, rows, nq, hq, hkv, dk, dv, ldq, ldo, page, max_blocks, num_blocks, scale, window, chunk, gate, ldg, sinks, status, s);
 }

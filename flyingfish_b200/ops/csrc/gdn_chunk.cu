@@ -36,36 +36,6 @@ struct GdnSmem {
   float beta[GC], c[GC], ec[GC], bec[GC], edec[GC];   // beta, c_t, e^{c_t}, beta e^{c_t}, e^{c_C - c_t}
 };
 
-// store a pair of accumulator values as BF16 at (row, col .. col+1) of a swizzled tile with `chunks` 16-byte chunks per row
-__device__ __forceinline__ void gdn_store2(uint8_t* tile, int row, int col, int chunks, float x, float y) {
-  *reinterpret_cast<uint32_t*>(tile + ms_off(row, col >> 3, chunks) + (col & 7) * 2) = pack_bf16x2(x, y);
-}
-
-// acc[NT][4] (+)= A[m0 .. m0+15][0 .. 16 KS) . B, A row-major tile (a_chunks per row);
-// B_TRANS = false: B given as [n][k] rows (b_chunks per row), n-tiles n0 .. n0 + 8 NT
-// B_TRANS = true : B given as [k][n] rows, same n range
-template <int NT, int KS, bool B_TRANS>
-__device__ __forceinline__ void gdn_mma(float (&acc)[NT][4], uint32_t a_base, int a_chunks, int m0, uint32_t b_base, int b_chunks,
-                                        int n0, int lane) {
-#pragma unroll
-  for (int ks = 0; ks < KS; ++ks) {
-    uint32_t a[4];
-    ms_ldsm4(a_base + ms_off(m0 + (lane & 7) + (((lane >> 3) & 1) << 3), 2 * ks + (lane >> 4), a_chunks), a[0], a[1], a[2], a[3]);
-#pragma unroll
-    for (int np = 0; np < NT / 2; ++np) {
-      uint32_t b0, b1, b2, b3;
-      if (B_TRANS) {
-        const int krow = ks * 16 + (((lane >> 3) & 1) << 3) + (lane & 7);
-        ms_ldsm4t(b_base + ms_off(krow, (n0 >> 3) + 2 * np + (lane >> 4), b_chunks), b0, b1, b2, b3);
-      } else {
-        ms_ldsm4(b_base + ms_off(n0 + 16 * np + ((lane >> 4) << 3) + (lane & 7), 2 * ks + ((lane >> 3) & 1), b_chunks), b0, b1, b2, b3);
-      }
-      ms_mma(acc[2 * np], a, b0, b1);
-      ms_mma(acc[2 * np + 1], a, b2, b3);
-    }
-  }
-}
-
 // grid (heads, sequences), 256 threads. q, k, v [rows, heads, 128] f32; beta, g [rows, heads] f32;
 // S [slots, heads, 128, 128] f32 (read at the start, written at the end); out [rows, heads, 128] bf16.
 __global__ void __launch_bounds__(256, 1)
@@ -137,8 +107,8 @@ gdn_chunked_kernel(const float* __restrict__ q, const float* __restrict__ k, con
     // state mirror in BF16 [k dim][v dim]
 #pragma unroll
     for (int nt = 0; nt < 16; ++nt) {
-      gdn_store2(sm.s16, warp * 16 + gq, nt * 8 + 2 * tq, GCH, st[nt][0], st[nt][1]);
-      gdn_store2(sm.s16, warp * 16 + gq + 8, nt * 8 + 2 * tq, GCH, st[nt][2], st[nt][3]);
+      ms_store2(sm.s16, warp * 16 + gq, nt * 8 + 2 * tq, GCH, st[nt][0], st[nt][1]);
+      ms_store2(sm.s16, warp * 16 + gq + 8, nt * 8 + 2 * tq, GCH, st[nt][2], st[nt][3]);
     }
     __syncthreads();
 
@@ -148,8 +118,8 @@ gdn_chunked_kernel(const float* __restrict__ q, const float* __restrict__ k, con
       float kk[4][4], qk[4][4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) { kk[i][0] = kk[i][1] = kk[i][2] = kk[i][3] = 0.f; qk[i][0] = qk[i][1] = qk[i][2] = qk[i][3] = 0.f; }
-      gdn_mma<4, GD / 16, false>(kk, aK, GCH, m0, aK, GCH, n0, lane);
-      gdn_mma<4, GD / 16, false>(qk, aQ, GCH, m0, aK, GCH, n0, lane);
+      ms_product<4, GD / 16, false>(kk, aK, GCH, m0, aK, GCH, n0, lane);
+      ms_product<4, GD / 16, false>(qk, aQ, GCH, m0, aK, GCH, n0, lane);
 #pragma unroll
       for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
@@ -164,7 +134,7 @@ gdn_chunked_kernel(const float* __restrict__ q, const float* __restrict__ k, con
             sm.a[t * GC + i] = (i < t) ? bt * dec * kk[nt][2 * e + j] : 0.f;
             pa[j] = dec * qk[nt][2 * e + j];
           }
-          gdn_store2(sm.p, t, n0 + nt * 8 + 2 * tq, GC / 8, pa[0], pa[1]);
+          ms_store2(sm.p, t, n0 + nt * 8 + 2 * tq, GC / 8, pa[0], pa[1]);
         }
     }
     __syncthreads();
@@ -207,23 +177,23 @@ gdn_chunked_kernel(const float* __restrict__ q, const float* __restrict__ k, con
       float wacc[8][4];
 #pragma unroll
       for (int i = 0; i < 8; ++i) wacc[i][0] = wacc[i][1] = wacc[i][2] = wacc[i][3] = 0.f;
-      gdn_mma<8, GC / 16, true>(wacc, aT1, GC / 8, m0, aK, GCH, n0, lane);           // W = T1 K
+      ms_product<8, GC / 16, true>(wacc, aT1, GC / 8, m0, aK, GCH, n0, lane);           // W = T1 K
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
-        gdn_store2(sm.w, m0 + gq, n0 + nt * 8 + 2 * tq, GCH, -wacc[nt][0], -wacc[nt][1]);
-        gdn_store2(sm.w, m0 + gq + 8, n0 + nt * 8 + 2 * tq, GCH, -wacc[nt][2], -wacc[nt][3]);
+        ms_store2(sm.w, m0 + gq, n0 + nt * 8 + 2 * tq, GCH, -wacc[nt][0], -wacc[nt][1]);
+        ms_store2(sm.w, m0 + gq + 8, n0 + nt * 8 + 2 * tq, GCH, -wacc[nt][2], -wacc[nt][3]);
       }
     }
     float dacc[8][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i) dacc[i][0] = dacc[i][1] = dacc[i][2] = dacc[i][3] = 0.f;
-    gdn_mma<8, GC / 16, true>(dacc, aT2, GC / 8, m0, aV, GCH, n0, lane);             // U = T2 V
+    ms_product<8, GC / 16, true>(dacc, aT2, GC / 8, m0, aV, GCH, n0, lane);             // U = T2 V
     __syncthreads();                                                                  // -W complete; K no longer read raw
-    gdn_mma<8, GD / 16, true>(dacc, aW, GCH, m0, aS, GCH, n0, lane);                 // D = U - W S0
+    ms_product<8, GD / 16, true>(dacc, aW, GCH, m0, aS, GCH, n0, lane);                 // D = U - W S0
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt) {
-      gdn_store2(sm.d, m0 + gq, n0 + nt * 8 + 2 * tq, GCH, dacc[nt][0], dacc[nt][1]);
-      gdn_store2(sm.d, m0 + gq + 8, n0 + nt * 8 + 2 * tq, GCH, dacc[nt][2], dacc[nt][3]);
+      ms_store2(sm.d, m0 + gq, n0 + nt * 8 + 2 * tq, GCH, dacc[nt][0], dacc[nt][1]);
+      ms_store2(sm.d, m0 + gq + 8, n0 + nt * 8 + 2 * tq, GCH, dacc[nt][2], dacc[nt][3]);
     }
     // scale Q rows by e^{c_t} and K rows by e^{c_C - c_t} in place (each thread its own elements; both tiles were last
     // read before the barrier above)
@@ -250,8 +220,8 @@ gdn_chunked_kernel(const float* __restrict__ q, const float* __restrict__ k, con
       float oacc[8][4];
 #pragma unroll
       for (int i = 0; i < 8; ++i) oacc[i][0] = oacc[i][1] = oacc[i][2] = oacc[i][3] = 0.f;
-      gdn_mma<8, GD / 16, true>(oacc, aQ, GCH, m0, aS, GCH, n0, lane);
-      gdn_mma<8, GC / 16, true>(oacc, aP, GC / 8, m0, aD, GCH, n0, lane);
+      ms_product<8, GD / 16, true>(oacc, aQ, GCH, m0, aS, GCH, n0, lane);
+      ms_product<8, GC / 16, true>(oacc, aP, GC / 8, m0, aD, GCH, n0, lane);
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int t = m0 + gq + 8 * e;

@@ -9,14 +9,11 @@ namespace ff {
 
 constexpr int F32_T = 64, F32_K = 16;
 
-__global__ void __launch_bounds__(256)
-gemm_f32_kernel(const float* __restrict__ X, const float* __restrict__ W, float* __restrict__ Y, int M, int N, int K, int ldx, int ldw,
-                int ldy, const float* __restrict__ bias, int act) {
-  pdl_trigger();
-  pdl_wait();
+// one 64 x 64 tile at (m0, n0)
+__device__ __forceinline__ void gemm_f32_tile(const float* __restrict__ X, const float* __restrict__ W, float* __restrict__ Y, int m0, int n0,
+                                              int M, int N, int K, int ldx, int ldw, int ldy, const float* __restrict__ bias, int act) {
   __shared__ __align__(16) float sx[F32_K][F32_T + 4];
   __shared__ __align__(16) float sw[F32_K][F32_T + 4];
-  const int m0 = blockIdx.y * F32_T, n0 = blockIdx.x * F32_T;
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += F32_K) {
@@ -53,6 +50,26 @@ gemm_f32_kernel(const float* __restrict__ X, const float* __restrict__ W, float*
   }
 }
 
+__global__ void __launch_bounds__(256)
+gemm_f32_kernel(const float* __restrict__ X, const float* __restrict__ W, float* __restrict__ Y, int M, int N, int K, int ldx, int ldw,
+                int ldy, const float* __restrict__ bias, int act) {
+  pdl_trigger();
+  pdl_wait();
+  gemm_f32_tile(X, W, Y, blockIdx.y * F32_T, blockIdx.x * F32_T, M, N, K, ldx, ldw, ldy, bias, act);
+}
+
+// expert segments (seg_off / counts on the device): Y[segment rows, N] = X[segment rows, K] · W[e][N, K]ᵀ
+__global__ void __launch_bounds__(256)
+gemm_f32_grouped_kernel(const float* __restrict__ X, const float* __restrict__ W, float* __restrict__ Y, const int* __restrict__ seg_off,
+                        const int* __restrict__ counts, int N, int K, int ldy, int capacity) {
+  pdl_trigger();
+  pdl_wait();
+  const int e = blockIdx.y, r0 = seg_off[e];
+  const int cnt = min(counts[e], capacity - r0);           // an overflowed dispatch is cut at the end of the buffers
+  for (int m0 = blockIdx.z * F32_T; m0 < cnt; m0 += gridDim.z * F32_T)
+    gemm_f32_tile(X + (size_t)r0 * K, W + (size_t)e * N * K, Y + (size_t)r0 * ldy, m0, blockIdx.x * F32_T, cnt, N, K, K, K, ldy, nullptr, 0);
+}
+
 }  // namespace ff
 using namespace ff;
 
@@ -62,5 +79,16 @@ FF_EXPORT int ff_gemm_f32(const float* X, const float* W, float* Y, int M, int N
   const long long my = (M + F32_T - 1) / F32_T;
   if (my > 65535) return FF_HOST_TOO_LARGE;
   if (int r = launch_pdl(gemm_f32_kernel, dim3((N + F32_T - 1) / F32_T, (unsigned)my), dim3(256), 0, s, 0, X, W, Y, M, N, K, ldx, ldw, ldy, bias, act)) return r;
+  return launch_result();
+}
+
+// Xs [capacity, K] contiguous rows, W [E * N, K], Y rows of ldy; segments as in ff_moe_grouped_gemm
+FF_EXPORT int ff_gemm_f32_grouped(const float* Xs, const float* W, float* Y, const int* seg_off, const int* counts, int E, int N, int K,
+                                  int capacity, int ldy, cudaStream_t s) {
+  if (E <= 0 || E > 65535 || N <= 0 || K <= 0 || capacity <= 0 || ldy < N) return FF_HOST_BAD_SHAPE;
+  int z = (capacity / E + F32_T - 1) / F32_T;
+  if (z < 1) z = 1;
+  if (z > 64) z = 64;
+  if (int r = launch_pdl(gemm_f32_grouped_kernel, dim3((N + F32_T - 1) / F32_T, E, z), dim3(256), 0, s, 0, Xs, W, Y, seg_off, counts, N, K, ldy, capacity)) return r;
   return launch_result();
 }

@@ -52,7 +52,7 @@ struct alignas(8) SkinnyBars {
 template <bool FUSE_AR>
 struct TileSink {
   __nv_bfloat16* Y; int N, ldy; bool vec8;      // vec8: 16-byte stores of eight values are aligned
-  const __nv_bfloat16* bias; int act;           // added to the finished sums; act 1: square of the positive part
+  const __nv_bfloat16* bias; int act;           // added to the finished sums; act 1: square of the positive part, 2: Y is FP32
   PeerArena ar; int parity;
 
   // eight consecutive columns col..col+7 of token row t (col is a multiple of 8)
@@ -70,6 +70,17 @@ struct TileSink {
       if (act == 1) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) { const float v = fmaxf(a[j], 0.f); a[j] = v * v; }
+      }
+      if (act == 2) {
+        float* dst = reinterpret_cast<float*>(Y) + (size_t)t * ldy + col;
+        if (vec8 && col + 8 <= N) {
+          reinterpret_cast<float4*>(dst)[0] = make_float4(a[0], a[1], a[2], a[3]);
+          reinterpret_cast<float4*>(dst)[1] = make_float4(a[4], a[5], a[6], a[7]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) if (col + j < N) dst[j] = a[j];
+        }
+        return;
       }
     }
     o.x = pack_bf16x2(a[0], a[1]); o.y = pack_bf16x2(a[2], a[3]);
@@ -862,6 +873,12 @@ FF_EXPORT int ff_gemm_skinny_act(const void* X, const void* W, void* Y, int M, i
   if ((unsigned)act > 1u) return FF_HOST_UNSUPPORTED;
   return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr, nullptr,
                             static_cast<const __nv_bfloat16*>(bias), act);
+}
+
+// Y = X Wᵀ with the FP32 sums stored as they are (router and gate logits, vocabulary logits). `grid` as above.
+FF_EXPORT int ff_gemm_skinny_f32out(const void* X, const void* W, float* Y, int M, int N, int K, int ldx, int ldw, int ldy,
+                                    int grid, float* scratch, int* counters, int* status, cudaStream_t stream) {
+  return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr, nullptr, nullptr, 2);
 }
 
 // Gate/up projection with the SwiGLU applied in the epilogue: W is [N, K] with gate/up rows interleaved per

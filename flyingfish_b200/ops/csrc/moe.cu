@@ -12,14 +12,14 @@
 //   moe_combine   : FP32 sum of a row's k contributions in ascending expert id, one BF16 rounding
 // Semantics follow kernels/moe_route.cu:1-30,155-390, kernels/moe_prefill.cu and
 // kernels/moe_combine.cu:1-96 of the reference.
-#include "ptx.cuh"
+#include "dtype_io.cuh"
 #include "host_util.h"
 
 namespace ff {
 
 // ---------------------------------------------------------------------------------------
 // routing: one warp per row, scores in shared memory
-// score_mode: 0 softmax, 1 sigmoid, 2 noaux (sigmoid + bias for selection, groups), 3 as 2 with sqrt(softplus(x)) scores
+// score_mode: 0 softmax (bias: for the selection only), 1 sigmoid, 2 noaux (sigmoid + bias for selection, groups), 3 as 2 with sqrt(softplus(x)) scores
 // ---------------------------------------------------------------------------------------
 constexpr int ROUTE_WARPS = 4;
 constexpr int ROUTE_MAX_E = 512;
@@ -33,8 +33,9 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
   }
 }
 
+template <typename T>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_topk_kernel(const __nv_bfloat16* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ out_w,
+moe_topk_kernel(const T* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ out_w,
                 int* __restrict__ out_ids, int rows, int E, int top_k, int score_mode, int n_groups, int topk_groups,
                 float routed_scaling, int renormalize, int ld, int* status) {
   __shared__ float s_score[ROUTE_WARPS][ROUTE_MAX_E];   // unbiased score
@@ -44,19 +45,19 @@ moe_topk_kernel(const __nv_bfloat16* __restrict__ logits, const float* __restric
   if (row >= rows) return;
   float* sc = s_score[warp];
   float* sel = s_sel[warp];
-  const __nv_bfloat16* lg = logits + (size_t)row * ld;
+  const T* lg = logits + (size_t)row * ld;
   if (score_mode == 0) {
     float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, __bfloat162float(lg[e]));
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, to_float(lg[e]));
     mx = warp_max(mx);
     float sum = 0.f;
-    for (int e = lane; e < E; e += 32) { const float v = expf(__bfloat162float(lg[e]) - mx); sc[e] = v; sum += v; }
+    for (int e = lane; e < E; e += 32) { const float v = expf(to_float(lg[e]) - mx); sc[e] = v; sum += v; }
     sum = warp_sum(sum);
     const float inv = 1.0f / sum;
-    for (int e = lane; e < E; e += 32) { sc[e] *= inv; sel[e] = sc[e]; }
+    for (int e = lane; e < E; e += 32) { sc[e] *= inv; sel[e] = bias ? sc[e] + bias[e] : sc[e]; }
   } else {
     for (int e = lane; e < E; e += 32) {
-      const float x = __bfloat162float(lg[e]);
+      const float x = to_float(lg[e]);
       const float v = (score_mode == 3) ? sqrtf(x > 20.f ? x : log1pf(expf(x))) : 1.0f / (1.0f + expf(-x));
       sc[e] = v;
       sel[e] = (score_mode >= 2 && bias) ? v + bias[e] : v;
@@ -148,9 +149,9 @@ moe_scan_kernel(const int* __restrict__ counts, int* __restrict__ seg_off, int* 
 
 // one block per assignment (row, j): claim a slot in the expert's segment, copy the token row
 __global__ void __launch_bounds__(128)
-moe_permute_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ ids, const int* __restrict__ seg_off,
-                   int* __restrict__ cursors, __nv_bfloat16* __restrict__ sorted, int* __restrict__ pos, int hidden,
-                   int top_k, int e_lo, int e_hi, int capacity, int ldx) {
+moe_permute_kernel(const uint4* __restrict__ x, const int* __restrict__ ids, const int* __restrict__ seg_off,
+                   int* __restrict__ cursors, uint4* __restrict__ sorted, int* __restrict__ pos, int vecs,
+                   int top_k, int e_lo, int e_hi, int capacity, int ldx_vecs) {
   const int a = blockIdx.x;
   const int e = ids[a];
   __shared__ int slot_s;
@@ -161,9 +162,9 @@ moe_permute_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ 
   if (threadIdx.x == 0) pos[a] = slot < capacity ? slot : -1;
   if (slot >= capacity) return;
   const int row = a / top_k;
-  const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)row * ldx);
-  uint4* dst = reinterpret_cast<uint4*>(sorted + (size_t)slot * hidden);
-  for (int v = threadIdx.x; v < hidden / 8; v += blockDim.x) dst[v] = src[v];
+  const uint4* src = x + (size_t)row * ldx_vecs;
+  uint4* dst = sorted + (size_t)slot * vecs;
+  for (int v = threadIdx.x; v < vecs; v += blockDim.x) dst[v] = src[v];
 }
 
 // ---------------------------------------------------------------------------------------
@@ -387,36 +388,43 @@ using namespace ff;
 
 FF_EXPORT int ff_moe_topk(const void* logits, const float* bias, float* out_w, int* out_ids, int rows, int E,
                           int top_k, int score_mode, int n_groups, int topk_groups, float routed_scaling,
-                          int renormalize, int ld, int* status, cudaStream_t s) {
+                          int renormalize, int ld, int f32, int* status, cudaStream_t s) {
   if (rows <= 0 || E <= 0 || E > ROUTE_MAX_E || top_k < 1 || top_k > 32 || top_k > E) return FF_HOST_BAD_SHAPE;
   if (n_groups < 1 || n_groups > 32 || E % n_groups || topk_groups < 1 || topk_groups > n_groups) return FF_HOST_BAD_SHAPE;
-  moe_topk_kernel<<<(rows + ROUTE_WARPS - 1) / ROUTE_WARPS, ROUTE_WARPS * 32, 0, s>>>(
-      (const __nv_bfloat16*)logits, bias, out_w, out_ids, rows, E, top_k, score_mode, n_groups, topk_groups,
-      routed_scaling, renormalize, ld, status);
+  const dim3 grid((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), block(ROUTE_WARPS * 32);
+  if (f32)
+    moe_topk_kernel<<<grid, block, 0, s>>>((const float*)logits, bias, out_w, out_ids, rows, E, top_k, score_mode, n_groups, topk_groups,
+                                           routed_scaling, renormalize, ld, status);
+  else
+    moe_topk_kernel<<<grid, block, 0, s>>>((const __nv_bfloat16*)logits, bias, out_w, out_ids, rows, E, top_k, score_mode, n_groups,
+                                           topk_groups, routed_scaling, renormalize, ld, status);
   return launch_result();
 }
 
 // counts/cursors: int32[E_local]; seg_off: int32[E_local + 1]; pos: int32[rows * top_k];
-// sorted: bf16 [capacity, hidden]. Experts [e_lo, e_hi) are local.
+// sorted: [capacity, hidden] rows of elem_bytes elements. Experts [e_lo, e_hi) are local.
 FF_EXPORT int ff_moe_dispatch_local(const void* x, const int* ids, int rows, int top_k, int hidden, int ldx, int E,
                                     int e_lo, int e_hi, int* counts, int* seg_off, int* cursors, void* sorted,
-                                    int* pos, int capacity, int* status, cudaStream_t s) {
+                                    int* pos, int capacity, int elem_bytes, int* status, cudaStream_t s) {
   const int el = e_hi - e_lo;
   if (rows <= 0 || top_k < 1 || hidden % 8 || el < 1 || el > 1024 || ldx % 8) return FF_HOST_BAD_SHAPE;
+  if (elem_bytes != 2 && elem_bytes != 4) return FF_HOST_UNSUPPORTED;
+  const int per_vec = 16 / elem_bytes;
   cudaError_t e = cudaMemsetAsync(counts, 0, (size_t)el * 4, s);
   if (e != cudaSuccess) return (int)e;
   const int n = rows * top_k;
   moe_count_kernel<<<(n + 255) / 256, 256, 0, s>>>(ids, n, E, e_lo, e_hi, counts, status);
   moe_scan_kernel<<<1, 1024, 0, s>>>(counts, seg_off, cursors, el, capacity, status);
-  moe_permute_kernel<<<n, 128, 0, s>>>((const __nv_bfloat16*)x, ids, seg_off, cursors, (__nv_bfloat16*)sorted, pos,
-                                       hidden, top_k, e_lo, e_hi, capacity, ldx);
+  moe_permute_kernel<<<n, 128, 0, s>>>((const uint4*)x, ids, seg_off, cursors, (uint4*)sorted, pos, hidden / per_vec, top_k, e_lo, e_hi,
+                                       capacity, ldx / per_vec);
   return launch_result();
 }
 
 FF_EXPORT int ff_moe_grouped_gemm(const void* xs, const void* w, void* y, const int* seg_off, const int* counts,
                                   int E_local, int Nw, int K, int capacity, int ldy, int epi, int* status,
                                   cudaStream_t s) {
-  if (E_local < 1 || Nw % 128 || K % 8 || capacity % 16) return FF_HOST_BAD_SHAPE;
+  // a plain store cuts its last tile at Nw (multiples of 8); the SwiGLU epilogue takes whole 128-row tiles
+  if (E_local < 1 || Nw % (epi == 1 ? 128 : 8) || K % 8 || capacity % 16) return FF_HOST_BAD_SHAPE;
   if (epi == 1 && ldy < Nw / 2) return FF_HOST_BAD_SHAPE;
   if (ldy % 8) return FF_HOST_BAD_ALIGN;
   CUtensorMap tmW, tmX;
@@ -432,7 +440,7 @@ FF_EXPORT int ff_moe_grouped_gemm(const void* xs, const void* w, void* y, const 
   const int pipe_bytes = small ? 76 * 1024 : 3 * (GBM * GBK * 2 + G_TOK * GBK * 2);   // 3 full-width stages = 144 KiB
   const int smem = staging + pipe_bytes + 1024;
   r = opt_in_smem(moe_grouped_gemm_kernel, 200 * 1024); if (r) return r;
-  dim3 grid(Nw / GBM, E_local);
+  dim3 grid((Nw + GBM - 1) / GBM, E_local);
   moe_grouped_gemm_kernel<<<grid, 192, smem, s>>>(tmW, tmX, (__nv_bfloat16*)y, seg_off, counts, Nw, K, ldy, epi,
                                                   pipe_bytes, staging, status, capacity);
   return launch_result();

@@ -1,0 +1,145 @@
+// FP32 residual stream of layers whose mixer and feed-forward read the same rows through two norms (parallel layers):
+//   embed : x = table[id] * scale
+//   step  : x += a + b + sum_j w_j y_j          a, b: rows of the mixer and of a dense or shared feed-forward
+//   n1 = x / rms(x) * w1     n2 = x / rms(x) * w2      the operands of the next layer (n2 optional)
+// The sum over a row's chosen experts is taken here, straight from the rows the grouped GEMM wrote (y_j = y[pos_j]; a choice
+// beyond the last expert is an identity output: y_j is the row h the experts were given), so a layer ends in one kernel: the
+// residual is read and written once in FP32 and nothing is rounded on the way. One block per row; a thread owns the same
+// columns in both passes. Norm weights are FP32 (offsets already added).
+#include "dtype_io.cuh"
+#include "host_util.h"
+
+namespace ff {
+
+constexpr int RN_THREADS = 512;
+constexpr int RN_TOP_MAX = 32;
+
+// the chosen experts' contributions of a row; top == 0: none
+template <typename T>
+struct ExpertRows {
+  const T* y; const int* pos; const int* ids; const float* w; const T* h;
+  int top, experts, ldy;
+};
+
+template <typename T, bool EMBED>
+__global__ void __launch_bounds__(RN_THREADS)
+residual_norms_kernel(float* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ table, float scale, int vocab,
+                      const T* __restrict__ a, const T* __restrict__ b, const ExpertRows<T> ex, const float* __restrict__ w1,
+                      const float* __restrict__ w2, T* __restrict__ n1, T* __restrict__ n2, int width, int true_width, float eps,
+                      int* status) {
+  pdl_trigger();
+  extern __shared__ __align__(16) float rn_x[];            // [width] the row between the two passes
+  __shared__ const T* s_src[RN_TOP_MAX];
+  __shared__ float s_w[RN_TOP_MAX];
+  __shared__ float s_red[RN_THREADS / 32];
+  const int row = blockIdx.x, tid = threadIdx.x;
+  pdl_wait();
+  const T* src = nullptr;
+  if (EMBED) {
+    int id = ids[row];
+    if (id < 0 || id >= vocab) { if (tid == 0) set_status(status, KID_EMBED, FF_ERR_BOUNDS, row, id); id = 0; }
+    src = table + (size_t)id * width;
+  } else if (ex.top > 0) {
+    if (tid < ex.top) {
+      const int i = row * ex.top + tid, e = ex.ids[i], p = ex.pos[i];
+      s_src[tid] = e >= ex.experts ? ex.h + (size_t)row * width : (p >= 0 ? ex.y + (size_t)p * ex.ldy : nullptr);
+      s_w[tid] = ex.w[i];
+    }
+    __syncthreads();
+  }
+  float* xr = x + (size_t)row * width;
+  float ss = 0.f;
+  for (int c = tid * 4; c < width; c += blockDim.x * 4) {
+    float v[4];
+    if (EMBED) {
+      load4(src + c, v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] *= scale;
+    } else {
+      float t[4];
+      load4(xr + c, v);
+      load4(a + (size_t)row * width + c, t);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] += t[j];
+      if (b != nullptr) {
+        load4(b + (size_t)row * width + c, t);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[j] += t[j];
+      }
+      for (int k = 0; k < ex.top; ++k) {
+        const T* p = s_src[k];
+        if (p == nullptr) continue;                        // not served (overflow, reported by the dispatch)
+        load4(p + c, t);
+        const float w = s_w[k];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[j] = fmaf(w, t[j], v[j]);
+      }
+    }
+    store4(xr + c, v);
+    store4(rn_x + c, v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) ss = fmaf(v[j], v[j], ss);
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) s_red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = (tid & 31) < (int)(blockDim.x >> 5) ? s_red[tid & 31] : 0.f;
+  tot = warp_sum(tot);
+  const float r = 1.0f / sqrtf(tot / (float)true_width + eps);
+  for (int c = tid * 4; c < width; c += blockDim.x * 4) {      // the thread's own columns again
+    float v[4], w[4], o[4];
+    load4(rn_x + c, v);
+    load4(w1 + c, w);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { v[j] *= r; o[j] = v[j] * w[j]; }
+    store4(n1 + (size_t)row * width + c, o);
+    if (w2 != nullptr) {
+      load4(w2 + c, w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[j] = v[j] * w[j];
+      store4(n2 + (size_t)row * width + c, o);
+    }
+  }
+}
+
+template <typename T, bool EMBED>
+static int residual_launch(float* x, const int* ids, const void* table, float scale, int vocab, const void* a, const void* b,
+                           const ExpertRows<T>& ex, const float* w1, const float* w2, void* n1, void* n2, int rows, int width, int true_width,
+                           float eps, int* status, cudaStream_t s) {
+  if (rows <= 0 || width <= 0 || width % 8 || true_width <= 0 || true_width > width || (w2 == nullptr) != (n2 == nullptr)) return FF_HOST_BAD_SHAPE;
+  if (ex.top < 0 || ex.top > RN_TOP_MAX || (ex.top > 0 && (ex.ldy % 8 || ex.pos == nullptr || ex.ids == nullptr || ex.w == nullptr))) return FF_HOST_BAD_SHAPE;
+  const int smem = width * 4;
+  if (smem > 200 * 1024) return FF_HOST_TOO_LARGE;
+  auto kern = residual_norms_kernel<T, EMBED>;
+  if (int r = opt_in_smem(kern, smem)) return r;
+  int threads = (width / 4 + 31) / 32 * 32;
+  // a few rows (a decode step): wide blocks, for latency; many: more, smaller blocks per SM keep more loads in flight
+  const int cap = rows >= 2 * sm_count() ? RN_THREADS / 2 : RN_THREADS;
+  if (threads > cap) threads = cap;
+  if (int r = launch_pdl(kern, dim3(rows), dim3(threads), smem, s, 0, x, ids, (const T*)table, scale, vocab, (const T*)a, (const T*)b, ex, w1,
+                         w2, (T*)n1, (T*)n2, width, true_width, eps, status)) return r;
+  return launch_result();
+}
+
+}  // namespace ff
+using namespace ff;
+
+// x FP32 [rows, width]; table, n1, n2 in BF16 (f32 = 0) or FP32; w1, w2 FP32 [width] (w2, n2: both or neither)
+FF_EXPORT int ff_residual_embed(const int* ids, const void* table, float scale, float* x, const float* w1, const float* w2, void* n1, void* n2,
+                                int rows, int width, int true_width, int vocab, float eps, int f32, int* status, cudaStream_t s) {
+  if (f32) return residual_launch<float, true>(x, ids, table, scale, vocab, nullptr, nullptr, ExpertRows<float>{}, w1, w2, n1, n2, rows, width, true_width, eps, status, s);
+  return residual_launch<__nv_bfloat16, true>(x, ids, table, scale, vocab, nullptr, nullptr, ExpertRows<__nv_bfloat16>{}, w1, w2, n1, n2, rows, width, true_width, eps, status, s);
+}
+
+// a: [rows, width]; b: the same or null; y, pos, eids, ew, h: the experts' rows, the row of every choice (negative: none), the
+// choices [rows, top] and weights, and the experts' input (top = 0: no experts)
+FF_EXPORT int ff_residual_step(float* x, const void* a, const void* b, const void* y, const int* pos, const int* eids, const float* ew,
+                               const void* h, int top, int experts, int ldy, const float* w1, const float* w2, void* n1, void* n2, int rows,
+                               int width, int true_width, float eps, int f32, cudaStream_t s) {
+  if (f32) {
+    const ExpertRows<float> ex = {(const float*)y, pos, eids, ew, (const float*)h, top, experts, ldy};
+    return residual_launch<float, false>(x, nullptr, nullptr, 1.f, 0, a, b, ex, w1, w2, n1, n2, rows, width, true_width, eps, nullptr, s);
+  }
+  const ExpertRows<__nv_bfloat16> ex = {(const __nv_bfloat16*)y, pos, eids, ew, (const __nv_bfloat16*)h, top, experts, ldy};
+  return residual_launch<__nv_bfloat16, false>(x, nullptr, nullptr, 1.f, 0, a, b, ex, w1, w2, n1, n2, rows, width, true_width, eps, nullptr, s);
+}

@@ -7,7 +7,7 @@
 //   sample_rows    : temperature / top-k / top-p / repetition penalty + Philox4x32-10 categorical
 // Contracts follow kernels/rope_kv.cu:34-53, kernels/act.cu:220-262, kernels/sample.cu:3-6,276-279
 // and src/sampling.rs:4-130 of the reference.
-#include "ptx.cuh"
+#include "dtype_io.cuh"
 #include "host_util.h"
 
 namespace ff {
@@ -141,12 +141,48 @@ __global__ void silu_mul_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloa
   reinterpret_cast<uint4*>(out + (size_t)row * ldo)[c] = o;
 }
 
+// the same in FP32 (no intermediate rounding), four elements per thread
+__global__ void silu_mul_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int f, int ldgu, int ldo,
+                                    int interleaved) {
+  pdl_trigger();
+  pdl_wait();
+  const int vec_per_row = f >> 2;
+  const long long gid = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (gid >= (long long)rows * vec_per_row) return;
+  const int row = (int)(gid / vec_per_row), c = (int)(gid % vec_per_row) * 4;
+  const int gc = interleaved ? (c >> 6) * 128 + (c & 63) : c, uc = interleaved ? gc + 64 : c + f;
+  float g[4], u[4];
+  load4(gu + (size_t)row * ldgu + gc, g);
+  load4(gu + (size_t)row * ldgu + uc, u);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) g[j] = g[j] * sigmoid_f(g[j]) * u[j];
+  store4(out + (size_t)row * ldo + c, g);
+}
+
 // logits softcap: x = cap * tanh(x / cap) (Gemma), in place
-__global__ void softcap_kernel(__nv_bfloat16* __restrict__ x, long long n, float cap) {
+template <typename T>
+__global__ void softcap_kernel(T* __restrict__ x, long long n, float cap) {
   pdl_trigger();
   pdl_wait();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < n) x[i] = __float2bfloat16(cap * tanhf(__bfloat162float(x[i]) / cap));
+  if (i < n) from_float(x + i, cap * tanhf(to_float(x[i]) / cap));
+}
+
+// (cos, sin) * amp of position * frequency in FP32. A frequency comes as a pair (hi, lo) with hi + lo its value to twice the
+// precision: the angle's rounding error does not grow with the position.
+__global__ void rope_angles_kernel(const int* __restrict__ positions, const float2* __restrict__ freq, float amp, float2* __restrict__ out,
+                                   int rows, int half) {
+  pdl_trigger();
+  pdl_wait();
+  const int gid = blockIdx.x * blockDim.x + threadIdx.x;
+  if (gid >= rows * half) return;
+  const int row = gid / half, i = gid - row * half;
+  const float p = (float)positions[row];
+  const float2 f = freq[i];
+  const float a = p * f.x, rest = fmaf(p, f.x, -a) + p * f.y;
+  float sn, cs;
+  sincosf(a, &sn, &cs);
+  out[gid] = make_float2(amp * fmaf(-sn, rest, cs), amp * fmaf(cs, rest, sn));
 }
 
 // ---------------------------------------------------------------------------------------
@@ -418,9 +454,27 @@ FF_EXPORT int ff_silu_mul(const void* gu, void* out, int rows, int f, int ldgu, 
   return launch_result();
 }
 
-FF_EXPORT int ff_softcap(void* x, long long n, float cap, cudaStream_t s) {
+// gate/up rows in FP32: out = silu(gate) * up
+FF_EXPORT int ff_silu_mul_f32(const float* gu, float* out, int rows, int f, int ldgu, int ldo, int interleaved, cudaStream_t s) {
+  if (rows <= 0 || f <= 0 || f % 4 || ldgu % 4 || ldo % 4 || (interleaved && f % 64)) return FF_HOST_BAD_SHAPE;
+  const long long total = (long long)rows * (f / 4);
+  if (int r = launch_pdl(silu_mul_f32_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, 0, gu, out, rows, f, ldgu, ldo, interleaved)) return r;
+  return launch_result();
+}
+
+FF_EXPORT int ff_softcap(void* x, long long n, float cap, int f32, cudaStream_t s) {
   if (n <= 0) return FF_HOST_BAD_SHAPE;
-  if (int lr_ = launch_pdl(softcap_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, 0, (__nv_bfloat16*)x, n, cap)) return lr_;
+  const dim3 grid((unsigned)((n + 255) / 256));
+  const int r = f32 ? launch_pdl(softcap_kernel<float>, grid, dim3(256), 0, s, 0, (float*)x, n, cap)
+                    : launch_pdl(softcap_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, 0, (__nv_bfloat16*)x, n, cap);
+  return r ? r : launch_result();
+}
+
+// freq: float2 [half] (hi, lo) pairs; out: float2 [rows, half]
+FF_EXPORT int ff_rope_angles(const int* positions, const float* freq, float amp, float* out, int rows, int half, cudaStream_t s) {
+  if (rows <= 0 || half <= 0) return FF_HOST_BAD_SHAPE;
+  if (int r = launch_pdl(rope_angles_kernel, dim3((unsigned)(((long long)rows * half + 127) / 128)), dim3(128), 0, s, 0, positions,
+                         reinterpret_cast<const float2*>(freq), amp, reinterpret_cast<float2*>(out), rows, half)) return r;
   return launch_result();
 }
 

@@ -16,15 +16,15 @@ from .lib import check, kernels, ptr, status_tensor, stream_ptr
 SCORE_MODES = {"softmax": 0, "sigmoid": 1, "noaux": 2, "sqrt_softplus": 3}
 
 
-def route(x, w_router, top_k, score, bias, n_groups, topk_groups, routed_scaling, renormalize):
+def route(x, w_router, top_k, score, bias, n_groups, topk_groups, routed_scaling, renormalize, exact=False, experts=None):
     rows = x.shape[0]
-    e = w_router.shape[0]
-    logits = linear(x, w_router)                       # FP32 accumulate, rounded to BF16
+    e = experts or w_router.shape[0]
+    logits = linear(x, w_router, out_dtype=torch.float32 if exact else None)       # FP32 accumulate, kept or rounded to BF16
     out_w = torch.empty(rows, top_k, dtype=torch.float32, device=x.device)
     out_ids = torch.empty(rows, top_k, dtype=torch.int32, device=x.device)
     rc = kernels().ff_moe_topk(ptr(logits), ptr(bias), ptr(out_w), ptr(out_ids), rows, e, top_k, SCORE_MODES[score],
                                n_groups, topk_groups, c_float(routed_scaling), int(renormalize), logits.stride(0),
-                               ptr(status_tensor(x.device)), stream_ptr())
+                               int(logits.dtype == torch.float32), ptr(status_tensor(x.device)), stream_ptr())
     check(rc, "ff_moe_topk")
     _count()
     return out_w, out_ids
@@ -58,23 +58,6 @@ def _gu_interleaved(w_gate_up: torch.Tensor) -> torch.Tensor:
     return t
 
 
-class _MoeWorkspace:
-    def __init__(self):
-        self.sorted: torch.Tensor | None = None
-
-
-_moe_ws: dict[int, _MoeWorkspace] = {}
-
-
-def _sorted_buffer(device, capacity: int, hidden: int) -> torch.Tensor:
-    ws = _moe_ws.setdefault(device.index or 0, _MoeWorkspace())
-    need = capacity * hidden
-    if ws.sorted is None or ws.sorted.numel() < need:
-        _require(not torch.cuda.is_current_stream_capturing(), "MoE workspace too small during graph capture")
-        ws.sorted = torch.zeros(int(need * 1.2) + 16 * hidden, dtype=torch.bfloat16, device=device)
-    return ws.sorted[:need].view(capacity, hidden)
-
-
 def dispatch_local(x, ids, n_experts_total: int, e_lo: int, e_hi: int):
     """Device-side count / scan / permute for the experts [e_lo, e_hi) owned locally.
     Returns (sorted rows, pos, seg_off, counts, capacity)."""
@@ -86,10 +69,12 @@ def dispatch_local(x, ids, n_experts_total: int, e_lo: int, e_hi: int):
     meta = torch.empty(3 * el + 1, dtype=torch.int32, device=dev)
     counts, seg_off, cursors = meta[:el], meta[el: 2 * el + 1], meta[2 * el + 1:]
     pos = torch.empty(rows * top_k, dtype=torch.int32, device=dev)
-    sorted_x = _sorted_buffer(dev, capacity, hidden)
+    # rows between the segments are never written; a GEMM computes them and stores nothing of them. The buffer comes from the
+    # allocator per call: a captured step has its own
+    sorted_x = torch.empty(capacity, hidden, dtype=x.dtype, device=dev)
     rc = kernels().ff_moe_dispatch_local(ptr(x), ptr(ids), rows, top_k, hidden, x.stride(0), n_experts_total, e_lo, e_hi,
                                          ptr(counts), ptr(seg_off), ptr(cursors), ptr(sorted_x), ptr(pos), capacity,
-                                         ptr(status_tensor(dev)), stream_ptr())
+                                         x.element_size(), ptr(status_tensor(dev)), stream_ptr())
     check(rc, "ff_moe_dispatch_local")
     _count(3)
     return sorted_x, pos, seg_off, counts, capacity
@@ -113,6 +98,31 @@ def grouped_gemm(xs, w, seg_off, counts, capacity: int, epi: int, rows_per_exper
     check(rc, "ff_moe_grouped_gemm")
     _count()
     return y
+
+
+def _grouped_gemm_f32(xs, w, seg_off, counts, capacity: int) -> torch.Tensor:
+    el, nw, k = w.shape
+    y = torch.empty(capacity, nw, dtype=torch.float32, device=xs.device)
+    check(kernels().ff_gemm_f32_grouped(ptr(xs), ptr(w), ptr(y), ptr(seg_off), ptr(counts), el, nw, k, capacity, nw, stream_ptr()),
+          "ff_gemm_f32_grouped")
+    _count()
+    return y
+
+
+def expert_rows(x, weights, ids, gu, down):
+    """See :func:`moe_ops.expert_rows`."""
+    from . import silu_mul
+    from .moe_ops import ExpertRows
+    el = gu.shape[0]
+    _require(gu.shape[1] == 2 * down.shape[2] and gu.shape[1] % 128 == 0 and gu.is_contiguous() and down.is_contiguous(), "expert stacks")
+    xs, pos, seg_off, counts, cap = dispatch_local(x, ids, 1 << 30, 0, el)
+    if x.dtype == torch.float32:
+        y = _grouped_gemm_f32(silu_mul(_grouped_gemm_f32(xs, gu, seg_off, counts, cap), interleaved=True), down, seg_off, counts, cap)
+    else:
+        rpe = x.shape[0] * ids.shape[1] / el
+        h = grouped_gemm(xs, gu, seg_off, counts, cap, epi=1, rows_per_expert=rpe)
+        y = grouped_gemm(h, down, seg_off, counts, cap, epi=0, rows_per_expert=rpe)
+    return ExpertRows(y, pos, ids, weights, x, el)
 
 
 def combine(y, pos, ids, weights, rows: int, hidden: int, out: torch.Tensor | None = None,

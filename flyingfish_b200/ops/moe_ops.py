@@ -20,12 +20,48 @@ from .lib import check, kernels, ptr, status_tensor, stream_ptr
 
 def route(x: torch.Tensor, w_router: torch.Tensor, top_k: int, score: str = "softmax",
           bias: torch.Tensor | None = None, n_groups: int = 1, topk_groups: int = 1, routed_scaling: float = 1.0,
-          renormalize: bool = True) -> tuple[torch.Tensor, torch.Tensor]:
-    """Returns (weights fp32 [rows, k], expert ids int32 [rows, k])."""
+          renormalize: bool = True, exact: bool = False, experts: int | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+    """Returns (weights fp32 [rows, k], expert ids int32 [rows, k]). ``exact``: the logits stay in FP32 (otherwise they are
+    rounded to the activations' type). ``experts``: rows of ``w_router`` that count, where it carries padding."""
     if not x.is_cuda:
-        return ref.moe_route(x, w_router, top_k, score, bias, n_groups, topk_groups, routed_scaling, renormalize)
+        w = w_router[:experts] if experts is not None else w_router
+        return ref.moe_route(x, w, top_k, score, bias, n_groups, topk_groups, routed_scaling, renormalize, torch.float32 if exact else None)
     from . import moe_cuda
-    return moe_cuda.route(x, w_router, top_k, score, bias, n_groups, topk_groups, routed_scaling, renormalize)
+    return moe_cuda.route(x, w_router, top_k, score, bias, n_groups, topk_groups, routed_scaling, renormalize, exact, experts)
+
+
+class ExpertRows:
+    """What the routed experts of a batch leave behind for the kernel that sums them (``residual_ops.step``): their output rows,
+    the row of every choice (negative: none), the choices and weights, and the experts' input (the output of an identity
+    choice: an id from ``experts`` on)."""
+
+    def __init__(self, y, pos, ids, weights, h, experts: int):
+        self.y, self.pos, self.ids, self.weights, self.h, self.experts = y, pos, ids, weights, h, experts
+
+    def total(self) -> torch.Tensor:
+        """The weighted sum in FP32 (CPU)."""
+        out = torch.zeros(self.h.shape, dtype=torch.float32)
+        for j in range(self.ids.shape[1]):
+            ident = self.ids[:, j] >= self.experts
+            row = torch.where(ident[:, None], self.h.float(), self.y[self.pos.view(self.ids.shape)[:, j].clamp(min=0).long()].float())
+            out += self.weights[:, j, None] * row
+        return out
+
+
+def expert_rows(x: torch.Tensor, weights: torch.Tensor, ids: torch.Tensor, gu: torch.Tensor, down: torch.Tensor) -> ExpertRows:
+    """SwiGLU experts on the rows that chose them, without the final sum. ``gu`` [E, 2f, h] with gate / up rows interleaved per
+    64, ``down`` [E, h, f]; ids from ``E`` on are not served here (identity outputs). BF16 or FP32."""
+    if x.is_cuda:
+        from . import moe_cuda
+        return moe_cuda.expert_rows(x, weights, ids, gu, down)
+    e = gu.shape[0]
+    y = torch.zeros(ids.numel(), x.shape[1], dtype=x.dtype)
+    pos = torch.where(ids < e, torch.arange(ids.numel()).view(ids.shape), -1).reshape(-1)
+    for k in range(e):
+        r, c = torch.nonzero(ids == k, as_tuple=True)
+        if r.numel():
+            y[r * ids.shape[1] + c] = ref.linear(ref.linear_swiglu(x[r], gu[k]), down[k])
+    return ExpertRows(y, pos, ids, weights, x, e)
 
 
 def experts_forward(x: torch.Tensor, weights: torch.Tensor, ids: torch.Tensor, w_gate_up: torch.Tensor,

@@ -242,14 +242,26 @@ def attention_paged(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
 # per-head norm + cache write
 # ------------------------------------------------------------------------------------------
 def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, hq: int, hkv: int,
-                 dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0) -> None:
+                 dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0,
+                 q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None,
+                 cos_sin: torch.Tensor | None = None) -> None:
     """In place on the q heads of ``qkv``: q and k divided by their root mean square over ``dim`` (heads may be padded in
-    the row: the caches' widths are the row's head widths), v blended with ``first_v``; k and v go to ``slots``."""
+    the row: the caches' widths are the row's head widths), weighted and rotated where that is given, v blended with ``first_v``; k and v go to ``slots``."""
     rows, bs = qkv.shape[0], kcache.shape[2]
     dk, dv = kcache.shape[3], vcache.shape[3]
     nq, nk = hq * dk, hkv * dk
     qk = qkv[:, : nq + nk].to(F32).view(rows, hq + hkv, dk)
     qk = qk * torch.rsqrt((qk * qk).sum(-1, keepdim=True) / dim + eps)
+    if q_weight is not None:
+        qk[:, :hq] *= q_weight
+    if k_weight is not None:
+        qk[:, hq:] *= k_weight
+    if cos_sin is not None:
+        r = 2 * cos_sin.shape[1]
+        c, s = cos_sin[:, None, :, 0], cos_sin[:, None, :, 1]
+        u, w = qk[..., 0:r:2].clone(), qk[..., 1:r:2].clone()
+        qk[..., 0:r:2] = u * c - w * s
+        qk[..., 1:r:2] = w * c + u * s
     qkv[:, : nq] = qk[:, :hq].reshape(rows, nq).to(qkv.dtype)
     v = qkv[:, nq + nk: nq + nk + hkv * dv].to(F32)
     if first_v is not None:
@@ -361,7 +373,7 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top_k: int, score: str = 
     """Router (kernels/moe_route.cu:1-30, 155-390 of the reference).
 
     * logits = x @ w_router.T accumulated in FP32, rounded to the activation dtype;
-    * ``softmax``: softmax over all experts, top-k, renormalise;
+    * ``softmax``: softmax over all experts, top-k (on ``score + bias`` where a bias is given), renormalise;
     * ``sigmoid``: sigmoid scores, top-k, renormalise;
     * ``noaux``: selection on ``sigmoid(logit) + bias`` restricted to the ``topk_groups`` best of
       ``n_groups`` groups (group score = sum of its two best biased scores), weights are the
@@ -372,7 +384,8 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top_k: int, score: str = 
     logits = _r((x.to(torch.float64) @ w_router.to(torch.float64).t()).to(F32), dt)
     if score == "softmax":
         s = torch.softmax(logits, dim=-1)
-        w, ids = topk_lower_tie(s, top_k)
+        _, ids = topk_lower_tie(s if bias is None else s + bias.to(F32), top_k)
+        w = torch.gather(s, -1, ids)
     elif score == "sigmoid":
         s = torch.sigmoid(logits)
         w, ids = topk_lower_tie(s, top_k)

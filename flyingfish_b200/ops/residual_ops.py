@@ -1,0 +1,72 @@
+"""FP32 residual stream of parallel layers: the sums a layer ends with, and the one or two norms the next one starts with, in one
+kernel. CUDA: ``csrc/residual.cu``; CPU: FP32 arithmetic on the same layouts.
+
+The stream is FP32 ``[rows, width]``; norm weights are FP32 vectors with any offset already added; ``true_width`` is the width the
+norms divide by where ``width`` carries padding."""
+from __future__ import annotations
+
+from ctypes import c_float
+
+import torch
+
+from . import _count, _require
+from .lib import check, kernels, ptr, status_tensor, stream_ptr
+from .moe_ops import ExpertRows
+
+
+def _norms(x: torch.Tensor, w1: torch.Tensor, w2: torch.Tensor | None, eps: float, true_width: int, dtype) -> tuple:
+    n = x * torch.rsqrt((x * x).sum(-1, keepdim=True) / true_width + eps)
+    return (n * w1).to(dtype), None if w2 is None else (n * w2).to(dtype)
+
+
+def _outputs(x: torch.Tensor, w1: torch.Tensor, w2: torch.Tensor | None, dtype) -> tuple:
+    for w in (w1, w2):
+        _require(w is None or (w.dtype == torch.float32 and w.numel() == x.shape[1] and w.is_contiguous()), "residual norms: FP32 weights")
+    new = lambda: torch.empty(x.shape, dtype=dtype, device=x.device)
+    return new(), None if w2 is None else new()
+
+
+def embed(ids: torch.Tensor, table: torch.Tensor, scale: float, w1: torch.Tensor, w2: torch.Tensor | None, eps: float,
+          true_width: int) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor | None]:
+    """(stream ``table[ids] * scale``, its norm times ``w1``, its norm times ``w2``)."""
+    if not table.is_cuda:
+        x = table[ids.long()].float() * scale
+        return (x,) + _norms(x, w1, w2, eps, true_width, table.dtype)
+    rows, (vocab, width) = ids.numel(), table.shape
+    _require(ids.dtype == torch.int32 and table.is_contiguous() and width % 8 == 0, "residual embed: int32 ids, rows of 8 elements")
+    x = torch.empty(rows, width, dtype=torch.float32, device=table.device)
+    n1, n2 = _outputs(x, w1, w2, table.dtype)
+    rc = kernels().ff_residual_embed(ptr(ids), ptr(table), c_float(scale), ptr(x), ptr(w1), ptr(w2), ptr(n1), ptr(n2), rows, width, true_width,
+                                     vocab, c_float(eps), int(table.dtype == torch.float32), ptr(status_tensor(table.device)), stream_ptr())
+    check(rc, "ff_residual_embed")
+    _count()
+    return x, n1, n2
+
+
+def step(x: torch.Tensor, a: torch.Tensor, b: torch.Tensor | None, experts: ExpertRows | None, w1: torch.Tensor, w2: torch.Tensor | None,
+         eps: float, true_width: int) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """``x += a + b + (weighted sum of the experts' rows)`` in place; returns the norms as :func:`embed` does."""
+    if not x.is_cuda:
+        x += a.float()
+        if b is not None:
+            x += b.float()
+        if experts is not None:
+            x += experts.total()
+        return _norms(x, w1, w2, eps, true_width, a.dtype)
+    rows, width = x.shape
+    _require(x.dtype == torch.float32 and x.is_contiguous() and width % 8 == 0, "residual step: FP32 rows of 8 elements")
+    ok = lambda t: t is None or (t.shape == x.shape and t.is_contiguous() and t.dtype == a.dtype)
+    _require(ok(a) and ok(b) and (experts is None or ok(experts.h)), "residual step: rows of one type")
+    n1, n2 = _outputs(x, w1, w2, a.dtype)
+    e, top, ldy, first = experts, 0, 0, 0
+    if e is not None:
+        top, ldy, first = e.ids.shape[1], e.y.stride(0), e.experts
+        _require(e.y.dtype == a.dtype and e.ids.is_contiguous() and e.weights.is_contiguous() and e.weights.dtype == torch.float32 and
+                 e.ids.dtype == e.pos.dtype == torch.int32, "residual step: expert rows")
+    g = lambda name: None if e is None else getattr(e, name)
+    rc = kernels().ff_residual_step(ptr(x), ptr(a), ptr(b), ptr(g("y")), ptr(g("pos")), ptr(g("ids")), ptr(g("weights")), ptr(g("h")), top,
+                                    first, ldy, ptr(w1), ptr(w2), ptr(n1), ptr(n2), rows, width, true_width, c_float(eps),
+                                    int(a.dtype == torch.float32), stream_ptr())
+    check(rc, "ff_residual_step")
+    _count()
+    return n1, n2

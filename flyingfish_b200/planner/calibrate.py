@@ -205,8 +205,7 @@ def decode_linear_shapes(spec, tp: int = 1) -> list[tuple[str, int, int, int]]:
     if spec.layer_specs is not None:          # designs whose layers differ: every distinct projection once
         seen: dict[tuple[int, int], str] = {}
         for l in spec.layer_specs:
-            q, kv, o = l.heads * l.dim_pad, l.kv_heads * (l.dim_pad + l.vdim_pad), l.heads * l.vdim_pad
-            for name, n, k in (("qkv", q + kv + o, spec.hidden), ("o", spec.hidden, o)) + \
+            for name, n, k in (("qkv", l.projection_cols, spec.hidden), ("o", spec.hidden, l.heads * l.vdim_pad)) + \
                     ((("up", l.ffn, spec.hidden), ("down", spec.hidden, l.ffn)) if l.ffn else ()):
                 seen.setdefault((n, k), name)
         return [(name, n, k, 0) for (n, k), name in seen.items()]

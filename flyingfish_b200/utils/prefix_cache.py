@@ -10,6 +10,7 @@ the length, after which generation continues as if the prefix had just been pref
 """
 from __future__ import annotations
 
+import dataclasses
 import hashlib
 import json
 from dataclasses import dataclass
@@ -43,7 +44,7 @@ def identity_for(model) -> PrefixIdentity:
     tk_id = f"{type(tk).__name__}:{getattr(tk, 'vocab_size', spec.vocab)}"
     fields = [spec.rope_theta, spec.head_dim, spec.extra.get("rope_scaling")]
     if spec.layer_specs is not None:          # designs whose layers differ: every layer's cache geometry and masks, and the type
-        fields.append([spec.dtype, [l.__dict__ for l in spec.layer_specs], spec.extra])
+        fields.append([spec.dtype, [dataclasses.asdict(l) for l in spec.layer_specs], spec.loop, spec.extra])
     rope = hashlib.sha256(json.dumps(fields, sort_keys=True).encode()).hexdigest()[:16]
     return PrefixIdentity(model.name, tk_id, rope, model.settings.kv_format)
 
