@@ -76,7 +76,7 @@ def parse() -> argparse.Namespace:
     p.add_argument("--skip-e2e", action="store_true")
     p.add_argument("--skip-baseline", action="store_true")
     p.add_argument("--skip-extras", action="store_true", help="no TTFT run and no other batch sizes")
-    p.add_argument("--design", default=None, choices=["duponex"],
+    p.add_argument("--design", default=None, choices=["duponex", "rudorax"],
                    help="instead of the headline benchmark: throughput and kernels of this design beside the closest model at equal size")
     p.add_argument("--device", default="cuda", choices=["cuda", "cpu"], help="cpu is for debugging the harness only")
     a = p.parse_args()
@@ -557,7 +557,7 @@ def main() -> None:
         if args.design is not None:
             from flyingfish_b200.utils import designbench
             t0 = time.perf_counter()
-            out = designbench.run(cx.device, args.steps, args.warmup, layers=args.layers)
+            out = designbench.run(cx.device, args.steps, args.warmup, args.design, layers=args.layers)
             out["clocks"] = cx.sampler.window(t0, time.perf_counter())
         elif args.impl == "baseline":
             out = run_baseline(cx)

@@ -479,7 +479,7 @@ def _rudorax_spec_of(name: str, hidden: int, vocab: int, layers: list[LayerSpec]
         m = l.moe
         if m is not None and (m.num_experts < 1 or m.identity < 0 or not 1 <= m.top_k <= min(m.num_experts + m.identity, 32) or m.expert_ffn < 1):
             raise ConfigError(f"unusable experts {m}")
-    if loop is not None and not (0 <= loop[0] < loop[1] <= len(layers) and loop[2] >= 1):
+    if loop is not None and not (0 <= loop[0] <= loop[1] <= len(layers) and loop[2] >= 1):
         raise ConfigError(f"loop {loop} outside the layers")
     wide = max(layers, key=lambda l: l.heads * l.dim)
     spec = ModelSpec(

@@ -115,7 +115,7 @@ def plan_memory(spec: ModelSpec, settings: Settings, info: DeviceInfo, weights_b
     if spec.mla is not None:
         block_bytes = spec.layers * settings.kv_block * (spec.mla.kv_lora_rank + spec.mla.qk_rope_dim) * 2
     elif spec.kv_geometry() is not None:
-        block_bytes = settings.kv_block * spec.elem_bytes * sum(h * (dk + dv) for h, dk, dv in spec.kv_geometry())
+        block_bytes = max(settings.kv_block * spec.elem_bytes * sum(h * (dk + dv) for h, dk, dv in spec.kv_geometry()), 1)
     else:
         block_bytes = spec.layers * hkv * settings.kv_block * spec.head_dim * 2 * 2
     blocks_per_seq = (settings.capacity + settings.kv_block - 1) // settings.kv_block

@@ -1,6 +1,8 @@
-"""A design's throughput and kernels beside the closest other model at equal size (``bench.py --design duponex``).
+"""A design's throughput and kernels beside the closest other model at equal size (``bench.py --design duponex|rudorax``).
 
-The closest model of a Duponex shape is the Gemma layout (QK-norm, local attention in every layer, extra norms per
+The closest model of a Rudorax shape is the Flint layout (QK-norm, windowed attention with sinks, routed and shared experts): same
+width, heads, window, experts and number of layers (Rudorax: layer runs); a memory layer's kernels are timed beside those of the
+gated delta net. The closest model of a Duponex shape is the Gemma layout (QK-norm, local attention in every layer, extra norms per
 sub-layer, operator-by-operator decode step): same width, heads and layers, a sliding window as long as the block, and a
 gated feed-forward of the width that makes the layers' weights equal. Prompts end inside a block, so both attentions see
 the same keys. Weights are random. Every kernel of the design is timed beside its like kernel on the same rows; a
@@ -14,16 +16,24 @@ import dataclasses
 import torch
 
 from .. import ops
-from ..config import ModelSpec, Settings, named_shape
-from ..ops import stream_ops
+from ..config import ModelSpec, MoeSpec, Settings, named_shape
+from ..ops import gdn_ops, mlstm_ops, moe_cuda, moe_ops, residual_ops, stream_ops
 from .kbench import Flusher, peaks, time_op
 
-SIZES = ("duponex-2b-shape", "duponex-8b-shape")
+SIZES = {"duponex": ("duponex-2b-shape", "duponex-8b-shape"), "rudorax": ("rudorax-2k-shape", "rudorax-4k-shape")}
 
 
 def closest_spec(spec: ModelSpec) -> ModelSpec:
-    """Gemma-layout shape with the layer weights of a Duponex shape of equal layers."""
+    """Gemma-layout shape with the layer weights of a Duponex shape of equal layers; Flint-layout shape with the attention and
+    experts of a Rudorax shape."""
     l = spec.layer_specs[0]
+    if spec.arch == "rudorax":
+        m = l.moe
+        return ModelSpec(name=spec.name.replace("rudorax", "flint-layout"), arch="flint", layers=spec.layers, hidden=spec.hidden, heads=l.heads,
+                         kv_heads=l.kv_heads, head_dim=l.dim, ffn=m.expert_ffn, vocab=spec.vocab, qk_norm=True, rms_eps=spec.rms_eps,
+                         moe=MoeSpec(num_experts=m.num_experts, top_k=m.top_k, expert_ffn=m.expert_ffn, score="sigmoid", n_shared=1,
+                                     shared_ffn=m.shared_ffn),
+                         extra={"flint": {"window": l.window, "no_rope_layers": []}})
     f = (l.heads * l.vdim + 2 * l.ffn) // 3 // 128 * 128
     return ModelSpec(name=spec.name.replace("duponex", "gemma-layout"), arch="gemma", layers=spec.layers, hidden=spec.hidden,
                      heads=l.heads, kv_heads=l.kv_heads, head_dim=l.dim, ffn=f, vocab=spec.vocab, qk_norm=True, swiglu_mode=2,
@@ -78,8 +88,9 @@ def model_throughput(spec: ModelSpec, prompt: int, batches, steps: int, warmup: 
         out["decode_tokens_per_s"][str(b)] = b / out["decode_ms"][str(b)] * 1e3
         drop(seqs)
     ops.check_status()
-    out["layer_weights"] = spec.dense_param_count() - 2 * spec.vocab * spec.hidden if spec.layer_specs is not None else \
-        spec.layers * (spec.hidden * spec.qkv_dim + spec.q_dim * spec.hidden + 3 * spec.hidden * spec.ffn)
+    out["run_weights"] = spec.run_params() if spec.layer_specs is not None else \
+        spec.layers * (spec.hidden * spec.qkv_dim + spec.q_dim * spec.hidden + 3 * spec.hidden *
+                       (spec.ffn if spec.moe is None else spec.moe.top_k * spec.moe.expert_ffn + spec.moe.shared_ffn))
     del m, eng
     torch.cuda.empty_cache()
     return out
@@ -98,28 +109,39 @@ class _Paged:
         self.ctx = torch.full((batch,), ctx, dtype=torch.int32, device=dev)
 
 
+class _Pairs:
+    """Times pairs of kernels on ``rows`` rows; a cost is (bytes, FLOPs)."""
+
+    def __init__(self, rows: int, iters: int, dev):
+        self.rows, self.iters, self.flush, self.pk, self.lines = rows, iters, Flusher(dev), peaks(), []
+
+    def bound(self, byts, flops):
+        return max(byts / (self.pk["hbm_gbs"] * 1e9), flops / (self.pk["bf16_tflops"] * 1e12)) * 1e6
+
+    def __call__(self, name, mine, mine_cost, like_name, like, like_cost):
+        a, b = (time_op(fn, self.iters, 3, self.flush, graph=True)["us_median"] for fn in (mine, like))
+        fa, fb = self.bound(*mine_cost) / a, self.bound(*like_cost) / b
+        self.lines.append({"kernel": name, "us": round(a, 2), "frac": round(fa, 3), "like": like_name, "like_us": round(b, 2),
+                           "like_frac": round(fb, 3), "distance": round(fb / fa, 2)})
+
+    def gemm(self, n, k, out_cols=None, out_bytes=2):
+        return (2 * (self.rows * k + n * k) + out_bytes * self.rows * (out_cols or n), 2 * self.rows * n * k)
+
+
 def kernel_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> list[dict]:
     """One line per pair: the design's kernel and its like on ``rows`` rows (``rows`` <= 128: a decode step of that batch at
     context ``ctx``; more: prefill of rows / ctx prompts)."""
+    return {"duponex": _duponex_table, "rudorax": _rudorax_table}[spec.arch](spec, rows, ctx, iters, device)
+
+
+def _duponex_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> list[dict]:
     l, other = spec.layer_specs[0], closest_spec(spec)
     dev, bf = torch.device(device), torch.bfloat16
     W, S, H, G, d, f = spec.hidden, int(spec.extra["duponex"]["streams"]), l.heads, l.kv_heads, l.dim, l.ffn
     rn = lambda *s: torch.randn(*s, device=dev).to(bf)
-    pk, flush = peaks(), Flusher(dev)
     decode = rows <= 128
-    res: list[dict] = []
-
-    def bound(byts, flops):
-        return max(byts / (pk["hbm_gbs"] * 1e9), flops / (pk["bf16_tflops"] * 1e12)) * 1e6
-
-    def pair(name, mine, mine_cost, like_name, like, like_cost):
-        a, b = (time_op(fn, iters, 3, flush, graph=True)["us_median"] for fn in (mine, like))
-        fa, fb = bound(*mine_cost) / a, bound(*like_cost) / b
-        res.append({"kernel": name, "us": round(a, 2), "frac": round(fa, 3), "like": like_name, "like_us": round(b, 2),
-                    "like_frac": round(fb, 3), "distance": round(fb / fa, 2)})
-
-    def gemm_cost(n, k, out_cols=None):
-        return (2 * (rows * k + n * k + rows * (out_cols or n)), 2 * rows * n * k)
+    pair = _Pairs(rows, iters, dev)
+    gemm_cost = pair.gemm
     x, n1, a1 = rn(rows, W), rn(W), rn(rows, H * d)
     # projections
     nq, no = H * d + 2 * G * d + H * d, H * d + 2 * G * d
@@ -175,19 +197,142 @@ def kernel_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> li
              out=out, chunk=l.chunk, gate=gate), cost(pairs), "prefill attention, window",
              lambda: ops.attn_prefill(qk, pg.k, pg.v, pg.table, qs, ql, pg.ctx, ctx, H, G, d, l.scale, window=l.chunk), cost(wpairs))
     ops.check_status()
-    return res
+    return pair.lines
 
 
-def run(device, steps: int, warmup: int, sizes=SIZES, batches=(1, 8, 64), prompt: int = 1024, layers: int | None = None) -> dict:
-    out: dict = {"design": "duponex", "prompt": prompt, "peaks": peaks(), "sizes": {}}
-    for name in sizes:
+def _rudorax_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> list[dict]:
+    l, mem = (next(x for x in spec.layer_specs if x.mixer == k) for k in ("attention", "mlstm"))
+    dev, bf, f32 = torch.device(device), torch.bfloat16, torch.float32
+    W, H, G, d, e = spec.hidden, l.heads, l.kv_heads, l.dim, l.moe
+    rn = lambda *s: torch.randn(*s, device=dev).to(bf)
+    fl = lambda *s: torch.randn(*s, device=dev)
+    i32 = lambda t: t.to(torch.int32)
+    decode = rows <= 128
+    pair = _Pairs(rows, iters, dev)
+    x = rn(rows, W)
+    nq, outs, f = H * d + 2 * G * d, e.num_experts + e.identity, e.expert_ffn
+    # projections
+    for name, n, k in (("qkv projection", nq, W), ("output projection", W, H * d)):
+        w, r = rn(n, k), x if k == W else rn(rows, k)
+        pair(name, lambda: ops.linear(r, w), pair.gemm(n, k), name, lambda: ops.linear(r, w), pair.gemm(n, k))
+    # head norm + rotation + cache write against the two norms, the rotation and the cache write of the like layer
+    batch = rows if decode else rows // ctx
+    pg = _Paged(batch, ctx, G, d, dev)
+    slots, pos = i32(torch.randperm(pg.k.shape[0] * 64, device=dev)[:rows]), i32(torch.arange(rows, device=dev)) % ctx
+    qkv, qn, kn = rn(rows, nq), rn(d), rn(d)
+    freqs, amp = l.rope.frequencies()
+    fr = ops.rope_frequencies(freqs, dev)
+    table = ops.rope_angles(pos, fr, amp)
+
+    def like_norm_rope():
+        q, k = qkv[:, : H * d].reshape(rows * H, d), qkv[:, H * d: (H + G) * d].reshape(rows * G, d)
+        qkv[:, : H * d] = ops.rmsnorm(q.contiguous(), qn, 1e-5).view(rows, -1)
+        qkv[:, H * d: (H + G) * d] = ops.rmsnorm(k.contiguous(), kn, 1e-5).view(rows, -1)
+        ops.rope_kv_paged(qkv, pos, slots, pg.k, pg.v, H, G, d, 1e4)
+    byts = 2 * rows * d * (2 * H + 2 * G + 2 * G)
+    qnf, knf = qn.float(), kn.float()
+    pair("head norm + rotation + cache write", lambda: ops.head_norm_kv(qkv, slots, pg.k, pg.v, H, G, d, d, 1e-5, q_weight=qnf, k_weight=knf, cos_sin=table),
+         (byts, 0), "head norms, rotation + cache write", like_norm_rope, (byts, 0))
+    pair("angles of a step", lambda: ops.rope_angles(pos, fr, amp), (rows * d * 4, 0), "angles of a step", lambda: ops.rope_table(pos, d, 1e4), (rows * d * 4, 0))
+    # attention
+    sinks = fl(H)
+    if decode:
+        cost = (2 * rows * (2 * l.keys_seen(ctx) * G * d + 2 * H * d), 4 * rows * l.keys_seen(ctx) * H * d)
+        at = lambda: ops.attn_decode(qkv, pg.k, pg.v, pg.table, pg.ctx, H, G, d, l.scale, max_ctx=ctx, window=l.window, sinks=sinks)
+    else:
+        qs, ql = i32(torch.arange(batch, device=dev) * ctx), torch.full((batch,), ctx, dtype=torch.int32, device=dev)
+        cost = (2 * rows * (2 * H * d + 2 * G * d), 4 * batch * l.pairs_seen(ctx) * H * d)
+        at = lambda: ops.attn_prefill(qkv, pg.k, pg.v, pg.table, qs, ql, pg.ctx, ctx, H, G, d, l.scale, window=l.window, sinks=sinks)
+    pair("attention, window + sinks", at, cost, "attention, window + sinks", at, cost)
+    del pg, qkv
+    # router, experts
+    wr, corr = rn((outs + 15) // 16 * 16, W) * 0.02, fl(outs) * 0.01
+    pair("router, 32-bit logits", lambda: moe_ops.route(x, wr, e.top_k, "softmax", corr, exact=True, experts=outs), pair.gemm(outs, W, out_bytes=8),
+         "router", lambda: moe_ops.route(x, wr[: e.num_experts], e.top_k, "sigmoid"), pair.gemm(e.num_experts, W, out_bytes=4))
+    weights, ids = moe_ops.route(x, wr, e.top_k, "softmax", corr, exact=True, experts=outs)
+    lw, lids = moe_ops.route(x, wr[: e.num_experts], e.top_k, "sigmoid")
+    gu, down = rn(e.num_experts, 2 * f, W), rn(e.num_experts, W, f)
+
+    def expert_cost(ids):
+        served = int((ids < e.num_experts).sum())
+        touched = int(torch.unique(ids[ids < e.num_experts]).numel())
+        return (2 * (touched * 3 * f * W + served * (2 * W + 3 * f)), 2 * served * 3 * f * W)
+    holder = {}
+
+    def like_experts():
+        xs, p, so, ct, cap = moe_cuda.dispatch_local(x, lids, e.num_experts, 0, e.num_experts)
+        rpe = rows * e.top_k / e.num_experts
+        h = moe_cuda.grouped_gemm(xs, gu, so, ct, cap, epi=1, rows_per_expert=rpe)
+        holder["y"], holder["pos"] = moe_cuda.grouped_gemm(h, down, so, ct, cap, epi=0, rows_per_expert=rpe), p
+    pair("experts (dispatch, two grouped GEMMs)", lambda: moe_ops.expert_rows(x, weights, ids, gu, down), expert_cost(ids),
+         "experts (dispatch, two grouped GEMMs)", like_experts, expert_cost(lids))
+    er = moe_ops.expert_rows(x, weights, ids, gu, down)
+    like_experts()
+    sg, sd = rn(2 * e.shared_ffn, W), rn(W, e.shared_ffn)
+    cost = (2 * (3 * e.shared_ffn * W + rows * (2 * W + 2 * e.shared_ffn)), 6 * rows * e.shared_ffn * W)
+    pair("shared expert", lambda: ops.linear(ops.linear_swiglu(x, sg), sd), cost, "shared expert",
+         lambda: ops.linear(ops.silu_mul(ops.linear(x, sg)), sd), cost)
+    # the layer's end: sums and the next norms
+    xs, a, b, w1, w2, w16, r16 = fl(rows, W), rn(rows, W), rn(rows, W), fl(W), fl(W), rn(W), rn(rows, W)
+
+    def like_end():
+        y = moe_cuda.combine(holder["y"], holder["pos"], lids, lw, rows, W)
+        ops.add_rmsnorm(a, r16, w16, 1e-5)
+        ops.add_rmsnorm(moe_ops.add_shared(y, b), r16, w16, 1e-5)
+    pair("residual step (all sums, two norms)", lambda: residual_ops.step(xs, a, b, er, w1, w2, 1e-5, W), (rows * W * (8 + 4 + 4 + 2 * e.top_k), 0),
+         "expert sum, shared sum, two add + norm", like_end, (rows * W * (2 * e.top_k + 2 * 6), 0))
+    tok, tab = i32(torch.randint(0, 1024, (rows,), device=dev)), rn(1024, W)
+    pair("embed + two norms", lambda: residual_ops.embed(tok, tab, 2.0, w1, w2, 1e-5, W), (rows * W * 10, 0), "embed + norm",
+         lambda: ops.embed_rmsnorm(tok, tab, w16, 1e-5), (rows * W * 6, 0))
+    del gu, down, er, holder, xs
+    # matrix memory against the gated delta net (128 x 128 heads, as many state elements)
+    M, dk, dv = mem.heads, mem.dim_pad, mem.vdim_pad
+    pn = mem.projection_cols
+    wp = rn(pn, W)
+    pair("memory projection", lambda: ops.linear(x, wp), pair.gemm(pn, W), "qkv projection, same size", lambda: ops.linear(x, wp), pair.gemm(pn, W))
+    wg = rn(max(2 * M, 16), W) * 0.02
+    pair("gate logits, 32-bit", lambda: ops.linear(x, wg, out_dtype=f32), pair.gemm(wg.shape[0], W, out_bytes=4), "projection of that size",
+         lambda: ops.linear(x, wg), pair.gemm(wg.shape[0], W))
+    del wp
+    st = mlstm_ops.MemoryState(batch, M, dk, dv, dev)
+    packed, gates, gb, o = rn(rows, pn), fl(rows, wg.shape[0]), fl(2 * M), torch.empty(rows, M, dv, device=dev)
+    starts = i32(torch.arange(batch + 1, device=dev) * (rows // batch))
+    sl = i32(torch.randperm(batch, device=dev))
+    V = M * dv // 128
+    q, k, v = (fl(rows, V, 128) for _ in range(3))
+    beta, dec = torch.rand(rows, V, device=dev), -torch.rand(rows, V, device=dev)
+    gst = torch.zeros(batch, V, 128, 128, device=dev)
+    state = 8 * batch * M * dk * dv
+    flops = 4 * rows * M * dk * dv + (0 if decode else 2 * rows * 64 * M * (dk + dv))       # prompts: and the triangle inside a chunk
+    gflops = 4 * rows * V * 128 * 128 + (0 if decode else 2 * rows * 64 * V * 128 * 4)
+    pair("memory recurrence" if decode else "memory, chunked", lambda: mlstm_ops.memory(packed, gates, gb, mem.gate_cap, st, starts, sl, mem.scale, o, rows // batch),
+         (state + rows * M * (4 * dk + 2 * dv + 4 * dv + 8), flops), "gated delta net recurrence" if decode else "gated delta net, chunked",
+         (lambda: gdn_ops.recurrent_slots(q, k, v, beta, dec, gst, starts, sl)) if decode else (lambda: gdn_ops.chunked_slots(q, k, v, beta, dec, gst, starts, sl)),
+         (8 * batch * V * 128 * 128 + rows * V * 128 * (12 + 2), gflops))
+    gate, wn, z = packed[:, M * (2 * dk + dv):], fl(M * dv), rn(rows, V * 128)
+    on = rn(rows * V, 128)
+    pair("head norm + output gate", lambda: mlstm_ops.head_out(o, gate, wn, dv, 1e-5), (rows * M * dv * 8, 0), "head norm, output gate",
+         lambda: (ops.rmsnorm(on, qn, 1e-5).view(rows, -1).float() * torch.nn.functional.silu(z.float())).to(bf), (rows * M * dv * 8, 0))
+    # vocabulary logits of a step
+    if decode:
+        wv = rn(spec.vocab, W)
+        pair("logits, 32-bit, soft cap", lambda: ops.softcap(ops.linear(x, wv, out_dtype=f32), 30.0), pair.gemm(spec.vocab, W, out_bytes=4), "logits",
+             lambda: ops.linear(x, wv), pair.gemm(spec.vocab, W))
+    ops.check_status()
+    return pair.lines
+
+
+def run(device, steps: int, warmup: int, design: str = "duponex", batches=(1, 8, 64), prompt: int = 1024, layers: int | None = None) -> dict:
+    out: dict = {"design": design, "prompt": prompt, "peaks": peaks(), "sizes": {}}
+    for name in SIZES[design]:
         spec = named_shape(name)
         if layers:
-            spec = dataclasses.replace(spec, layers=layers, layer_specs=spec.layer_specs[:layers])
+            spec = dataclasses.replace(spec, layer_specs=spec.layer_specs[:layers], loop=None)
+            spec.layers = len(spec.runs)
         other = closest_spec(spec)
         out["sizes"][name] = {
             "closest": {"name": other.name, "ffn": other.ffn},
-            "duponex": model_throughput(spec, prompt, batches, steps, warmup, device),
+            design: model_throughput(spec, prompt, batches, steps, warmup, device),
             "closest_model": model_throughput(other, prompt, batches, steps, warmup, device),
             "kernels": {"decode rows 64, context 1024": kernel_table(spec, 64, 1024, 30, device),
                         "prefill 8 x 1024": kernel_table(spec, 8192, 1024, 15, device),
