@@ -131,6 +131,7 @@ mlstm_recurrent_kernel(const MlstmArgs<T> p) {
 // chunked: grid (tiles, heads, sequences x segments), 256 threads. KP: key width padded to 64, 128 or 256.
 // ---------------------------------------------------------------------------------------
 constexpr int MC = 64;               // tokens per chunk
+constexpr int MGB = 4;               // chunks whose gates are worked out together, a warp each
 constexpr int MTC = ML_TILE / 8;     // 16-byte chunks per row of a 64-column tile
 
 template <int KP>
@@ -139,10 +140,11 @@ struct MlstmSmem {
   uint8_t s[2][KP * ML_TILE * 2];    // operand copy of the state: value, remainder
   uint8_t vw[2][MC * ML_TILE * 2];   // e^{a_j - M_C} v_j: value, remainder
   uint8_t p[2][MC * MC * 2];         // P: value, remainder
-  float n[KP];
-  float a[MC], top[MC], carry[MC], floor[MC], kw[MC];      // a_j, M_t, e^{m_0 - M_t}, e^{-m_t}, e^{a_j - M_C}
+  float n[KP], np[4][KP];            // n as the chunk finds it; its next value in four parts (16 tokens each)
+  float ga[MGB][MC], gf[MGB][MC], gm[MGB][MC];             // a_j, F_j and max_{i<=j} a_i of the next chunks
+  float top[MC], carry[MC], floor[MC];                     // M_t, e^{m_0 - M_t}, e^{-m_t}
+  alignas(16) float kw[MC];                                // e^{a_j - M_C}
   float qn[MC], rs[2][MC];
-  float keep, m_next, f_sum;         // e^{m_0 - M_C}, F_C + M_C, F_C
 };
 
 // Segments of a long prompt. count == 1: a sequence is one segment, the state comes from and goes to its slot.
@@ -161,7 +163,7 @@ __device__ __forceinline__ void store_split(uint8_t (*tile)[MC * ML_TILE * 2], i
 }
 
 template <int KP>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, KP == 256 ? 1 : 2)
 mlstm_chunk_kernel(const MlstmArgs<__nv_bfloat16> p, const MlstmSegments sg) {
   pdl_trigger();
   pdl_wait();
@@ -197,14 +199,48 @@ mlstm_chunk_kernel(const MlstmArgs<__nv_bfloat16> p, const MlstmSegments sg) {
         if (!own && k < dk && col < dv) f = *reinterpret_cast<const float2*>(Sin + (size_t)k * dv + col);
         st[i][nt][2 * e] = f.x; st[i][nt][2 * e + 1] = f.y;
       }
-  for (int k = tid; k < KP; k += 256) sm.n[k] = !own && k < dk ? nin[k] : 0.f;
+  for (int k = tid; k < KP; k += 256) {
+    sm.np[0][k] = !own && k < dk ? nin[k] : 0.f;
+    sm.np[1][k] = sm.np[2][k] = sm.np[3][k] = 0.f;
+  }
   float m = own ? -INFINITY : (sg.count == 1 ? p.m[hs * p.tiles + tile] : sg.m_start[hseg * p.tiles + tile]);
   float f_all = 0.f;
   const float bi = p.gate_bias[h], bf = p.gate_bias[H + h];
 
-  for (int t0 = r0; t0 < r1; t0 += MC) {
+  for (int t0 = r0, ci = 0; t0 < r1; t0 += MC, ci = (ci + 1) % MGB) {
     const int n = min(MC, r1 - t0);
     __syncthreads();                                       // the previous chunk's tiles are no longer read
+    if (ci == 0) {
+      // gates, prefix sums of f and prefix maxima of a of the next chunks, two tokens per lane; past the end: f = 0, a = -inf
+      const int ta = 2 * lane, tb = ta + 1, tw = t0 + warp * MC;
+      if (warp < MGB && tw < r1) {
+        LogGates g0 = {-INFINITY, 0.f}, g1 = g0;
+        if (tw + ta < r1) { const float* z = p.gates + (size_t)(tw + ta) * p.ldg; g0 = log_gates(z[h] + bi, z[H + h] + bf, p.cap); }
+        if (tw + tb < r1) { const float* z = p.gates + (size_t)(tw + tb) * p.ldg; g1 = log_gates(z[h] + bi, z[H + h] + bf, p.cap); }
+        float run = g0.f + g1.f;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) { const float up = __shfl_up_sync(0xffffffffu, run, o); if (lane >= o) run += up; }
+        const float f1 = run, f0 = run - g1.f, a0 = g0.i - f0, a1 = g1.i - f1;
+        float mx = fmaxf(a0, a1);
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) { const float up = __shfl_up_sync(0xffffffffu, mx, o); if (lane >= o) mx = fmaxf(mx, up); }
+        float before = __shfl_up_sync(0xffffffffu, mx, 1);
+        if (lane == 0) before = -INFINITY;
+        sm.ga[warp][ta] = a0; sm.ga[warp][tb] = a1;
+        sm.gf[warp][ta] = f0; sm.gf[warp][tb] = f1;
+        sm.gm[warp][ta] = fmaxf(before, a0); sm.gm[warp][tb] = mx;
+      }
+      __syncthreads();
+    }
+    const float Mc = fmaxf(m, sm.gm[ci][MC - 1]), Fc = sm.gf[ci][MC - 1], keep = expf(m - Mc);
+    if (tid < MC) {
+      const float M = fmaxf(m, sm.gm[ci][tid]);
+      sm.top[tid] = M;
+      sm.carry[tid] = expf(m - M);
+      sm.floor[tid] = expf(-(sm.gf[ci][tid] + M));
+      sm.kw[tid] = expf(sm.ga[ci][tid] - Mc);
+    }
+    for (int k = tid; k < KP; k += 256) sm.n[k] = (sm.np[0][k] + sm.np[1][k]) + (sm.np[2][k] + sm.np[3][k]);
     // ---- tiles of the chunk; rows past n and columns past the heads are zero
     for (int i = tid; i < MC * KCH; i += 256) {
       const int t = i / KCH, cch = i - t * KCH;
@@ -224,30 +260,14 @@ mlstm_chunk_kernel(const MlstmArgs<__nv_bfloat16> p, const MlstmSegments sg) {
         vv = *reinterpret_cast<const uint4*>(p.x + (size_t)(t0 + t) * p.ldx + (size_t)2 * H * dk + (size_t)h * dv + c0 + cch * 8);
       *reinterpret_cast<uint4*>(sm.v + ms_off(t, cch, MTC)) = vv;
     }
-    if (warp == 0) {
-      // gates, prefix sums of f and prefix maxima of a: two tokens per lane; past n: f = 0, a = -inf
-      const int ta = 2 * lane, tb = ta + 1;
-      LogGates ga = {-INFINITY, 0.f}, gb = ga;
-      if (ta < n) { const float* z = p.gates + (size_t)(t0 + ta) * p.ldg; ga = log_gates(z[h] + bi, z[H + h] + bf, p.cap); }
-      if (tb < n) { const float* z = p.gates + (size_t)(t0 + tb) * p.ldg; gb = log_gates(z[h] + bi, z[H + h] + bf, p.cap); }
-      float run = ga.f + gb.f;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) { const float up = __shfl_up_sync(0xffffffffu, run, o); if (lane >= o) run += up; }
-      const float Fb = run, Fa = run - gb.f;
-      const float aa = ga.i - Fa, ab = gb.i - Fb;
-      float mx = fmaxf(aa, ab);
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) { const float up = __shfl_up_sync(0xffffffffu, mx, o); if (lane >= o) mx = fmaxf(mx, up); }
-      float before = __shfl_up_sync(0xffffffffu, mx, 1);
-      if (lane == 0) before = -INFINITY;
-      const float Ma = fmaxf(m, fmaxf(before, aa)), Mb = fmaxf(m, mx);
-      const float Mc = __shfl_sync(0xffffffffu, Mb, 31), Fc = __shfl_sync(0xffffffffu, Fb, 31);
-      sm.a[ta] = aa; sm.a[tb] = ab;
-      sm.top[ta] = Ma; sm.top[tb] = Mb;
-      sm.carry[ta] = expf(m - Ma); sm.carry[tb] = expf(m - Mb);
-      sm.floor[ta] = expf(-(Fa + Ma)); sm.floor[tb] = expf(-(Fb + Mb));
-      sm.kw[ta] = expf(aa - Mc); sm.kw[tb] = expf(ab - Mc);
-      if (lane == 0) { sm.keep = expf(m - Mc); sm.m_next = Fc + Mc; sm.f_sum = Fc; }
+    // the next chunk's rows on their way into the L2 cache
+    for (int i = tid; i < MC * (2 * KP / 64 + 1); i += 256) {
+      const int t = t0 + MC + i % MC, part = i / MC;
+      if (t >= r1) continue;
+      const __nv_bfloat16* xr = p.x + (size_t)t * p.ldx;
+      const int col = part * 64 - (part >= KP / 64 ? KP : 0);
+      const __nv_bfloat16* at = part == 2 * KP / 64 ? xr + (size_t)2 * H * dk + (size_t)h * dv + c0 : xr + (size_t)(part >= KP / 64 ? H + h : h) * dk + col;
+      if (part == 2 * KP / 64 || col < dk) asm volatile("prefetch.global.L2 [%0];" ::"l"(at));
     }
     if (!own) {
 #pragma unroll
@@ -290,7 +310,7 @@ mlstm_chunk_kernel(const MlstmArgs<__nv_bfloat16> p, const MlstmSegments sg) {
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
             const int i = half * 32 + nt * 8 + 2 * tq + j;
-            v[j] = i <= t ? expf(sm.a[i] - top) * p.qscale * qk[nt][2 * e + j] : 0.f;
+            v[j] = i <= t ? __expf(sm.ga[ci][i] - top) * p.qscale * qk[nt][2 * e + j] : 0.f;
             sum += v[j];
           }
           store_split(sm.p, t, half * 32 + nt * 8 + 2 * tq, v[0], v[1]);
@@ -349,7 +369,6 @@ mlstm_chunk_kernel(const MlstmArgs<__nv_bfloat16> p, const MlstmSegments sg) {
       }
     }
     // ---- S <- keep S + K^T (weighted V); A read transposed from the K tile
-    const float keep = sm.keep;
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
@@ -371,16 +390,23 @@ mlstm_chunk_kernel(const MlstmArgs<__nv_bfloat16> p, const MlstmSegments sg) {
           for (int i = 0; i < MT; ++i) { ms_mma(st[i][2 * np], a[i], b0, b1); ms_mma(st[i][2 * np + 1], a[i], b2, b3); }
         }
     }
-    // ---- n <- keep n + sum_j e^{a_j - M_C} k_j (read above as the incoming n, before the last barrier)
-    for (int k = tid; k < KP; k += 256) {
-      float s = keep * sm.n[k];
-      for (int t = 0; t < n; ++t)
-        s = fmaf(sm.kw[t], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(sm.k + ms_off(t, k >> 3, KCH) + (k & 7) * 2)), s);
-      sm.n[k] = s;
+    // ---- n <- keep n + sum_j e^{a_j - M_C} k_j: a thread takes two key elements and 16 tokens
+    for (int i = tid; i < 2 * KP; i += 256) {
+      const int k = (i % (KP / 2)) * 2, part = i / (KP / 2);
+      float x = part == 0 ? keep * sm.n[k] : 0.f, y = part == 0 ? keep * sm.n[k + 1] : 0.f;
+#pragma unroll
+      for (int t = 0; t < 16; ++t) {
+        const float w = sm.kw[part * 16 + t];
+        const float2 f = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(sm.k + ms_off(part * 16 + t, k >> 3, KCH) + (k & 7) * 2));
+        x = fmaf(w, f.x, x);
+        y = fmaf(w, f.y, y);
+      }
+      sm.np[part][k] = x; sm.np[part][k + 1] = y;
     }
-    m = sm.m_next;
-    f_all += sm.f_sum;
+    m = Fc + Mc;
+    f_all += Fc;
   }
+  __syncthreads();
   // ---- state out
   if (!own && !last) return;
   float* So = own ? sg.S + hseg * dk * dv : p.S + hs * dk * dv;
@@ -394,7 +420,7 @@ mlstm_chunk_kernel(const MlstmArgs<__nv_bfloat16> p, const MlstmSegments sg) {
         const int k = (mt0 + i) * 16 + gq + 8 * e, col = c0 + n0 + nt * 8 + 2 * tq;
         if (k < dk && col < dv) *reinterpret_cast<float2*>(So + (size_t)k * dv + col) = make_float2(st[i][nt][2 * e], st[i][nt][2 * e + 1]);
       }
-  for (int k = tid; k < dk; k += 256) no[k] = sm.n[k];     // the thread's own elements
+  for (int k = tid; k < dk; k += 256) no[k] = (sm.np[0][k] + sm.np[1][k]) + (sm.np[2][k] + sm.np[3][k]);
   if (tid == 0) {
     if (own) { sg.m_own[hseg * p.tiles + tile] = m; sg.f_own[hseg * p.tiles + tile] = f_all; }
     else p.m[hs * p.tiles + tile] = m;
