@@ -113,9 +113,15 @@ def gated_silu(h, t, p):
     return (g * torch.sigmoid(g) * (h @ t(p + "up").T)) @ t(p + "down").T
 
 
+MARGINS: list[float] = []        # distance between the last choice and the first refused one, of every choice made
+
+
 def choose_experts(h, t, p, top):
     """(ids [n, top], weights [n, top]): the bias moves the choice, not the weights."""
     s = torch.softmax(h @ t(p + "router").T, -1)
+    ordered = torch.sort(s + t(p + "correction"), dim=-1, descending=True).values
+    if top < ordered.shape[1]:
+        MARGINS.append(float((ordered[:, top - 1] - ordered[:, top]).min()))
     ids = torch.sort(s + t(p + "correction"), dim=-1, descending=True, stable=True).indices[:, :top]
     w = s.gather(1, ids)
     return ids, w / (w.sum(-1, keepdim=True) + 1e-20)
@@ -189,19 +195,31 @@ def config(layers, width=104, vocab=198, scale=3.0, eps=1e-5, softcap=9.0, loop=
             "loop": loop and {"start": loop[0], "stop": loop[1], "times": loop[2]}, "logit_softcap": softcap, "vocab": vocab, "width": width}
 
 
+CLASSES = 5
+
+
 def tensors(cfg, seed=0):
-    """Random weights (BF16 values) in which every mechanism counts."""
+    """Random weights (BF16 values) in which every mechanism counts. The experts a token gets hang on its class alone (its number
+    modulo ``CLASSES``): the last channels carry the class and no layer writes to them, so that no choice is a close call which
+    16-bit rounding could turn."""
     g = torch.Generator().manual_seed(seed)
     w = cfg["width"]
     rn = lambda *shape: torch.randn(*shape, generator=g)
     lin = lambda o, i, gain=1.0: gain * rn(o, i) / i ** 0.5
+
+    def writes(i):
+        m = lin(w, i)
+        m[-CLASSES:] = 0.0
+        return m
     out = {"embed": rn(cfg["vocab"], w) / cfg["embedding"]["scale"], "head": lin(cfg["vocab"], w, 3.0), "final.norm": 0.2 * rn(w)}
+    out["embed"][:, -CLASSES:] = 0.0
+    out["embed"][torch.arange(cfg["vocab"]), w - CLASSES + torch.arange(cfg["vocab"]) % CLASSES] = 4.0 / cfg["embedding"]["scale"]
     for i, l in enumerate(cfg["layers"]):
         p, m = f"l{i}.mix.", l["mixer"]
         out[f"l{i}.norm1"] = 0.2 * rn(w)
         H, dk, dv = m["heads"], m["dim"], m["vdim"]
         G = m.get("kv_heads", H)
-        out.update({p + "q": lin(H * dk, w), p + "k": lin(G * dk, w), p + "v": lin(G * dv, w), p + "o": lin(w, H * dv)})
+        out.update({p + "q": lin(H * dk, w), p + "k": lin(G * dk, w), p + "v": lin(G * dv, w), p + "o": writes(H * dv)})
         if l["type"] == "attention":
             out.update({p + "q.norm": 1 + 0.3 * rn(dk), p + "k.norm": 1 + 0.3 * rn(dk), p + "sink": 1.0 + 0.7 * rn(H)})
         else:
@@ -212,8 +230,16 @@ def tensors(cfg, seed=0):
             p, r = f"l{i}.mlp.", f["router"]
             out[f"l{i}.norm2"] = 0.2 * rn(w)
             n = r["experts"] + r["identity"]
-            out[p + "router"], out[p + "correction"] = lin(n, w, 1.5), 0.05 * rn(n)
+            out[p + "router"] = torch.zeros(n, w)
+            always = int(torch.randint(0, n, (1,), generator=g))                # the output that the bias puts into every choice
+            others = torch.tensor([j for j in range(n) if j != always], dtype=torch.long)
+            for c in range(CLASSES):                      # a class's own outputs, the rest well below, the biased one anywhere
+                level = torch.where(torch.arange(n - 1) < r["top"] - 1, 1.6 + 0.1 * rn(n - 1), -0.4 + 0.1 * rn(n - 1))
+                out[p + "router"][others[torch.randperm(n - 1, generator=g)], w - CLASSES + c] = level
+                out[p + "router"][always, w - CLASSES + c] = 2.0 * torch.rand((), generator=g) - 0.4
+            out[p + "correction"] = 0.004 * rn(n)
+            out[p + "correction"][always] = 2.0
             names = [(f"e{e}.", f["expert"]["ff"]) for e in range(r["experts"])] + ([("shared.", f["shared"]["ff"])] if f.get("shared") else [])
             for name, ff in names:
-                out.update({p + name + "gate": lin(ff, w), p + name + "up": lin(ff, w), p + name + "down": lin(w, ff)})
+                out.update({p + name + "gate": lin(ff, w), p + name + "up": lin(ff, w), p + name + "down": writes(ff)})
     return {n: t.to(torch.bfloat16) for n, t in out.items()}
