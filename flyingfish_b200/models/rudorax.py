@@ -10,6 +10,8 @@ run several times.
   ``ops.mlstm_ops`` runs the recurrence from the sequence's state slot; the heads are normed and gated on the way out.
 * Experts: FP32 router logits, soft-max over all outputs, the choice moved by a bias the weights do not see. Outputs behind the
   experts are identities. A shared expert runs for every token.
+* The mixer and the feed-forward do not depend on each other: a decode step runs the routed experts on a second stream beside the
+  mixer and the shared expert.
 * The residual is FP32. Its sums (mixer, shared expert, the chosen experts' rows with their weights, identity outputs) and the two
   norms of the next layer are one kernel (``ops.residual_ops``).
 
@@ -18,6 +20,8 @@ hold portions of prompts and single decoded tokens together (``mixed_batches``):
 take the decode kernels. Sizes that are not multiples of the kernels' vectors are padded here, once, with zeros.
 """
 from __future__ import annotations
+
+import os
 
 import torch
 
@@ -129,6 +133,10 @@ def random_weights(spec: ModelSpec, seed: int, device: torch.device | str) -> Mo
 # ------------------------------------------------------------------------------------------
 # model
 # ------------------------------------------------------------------------------------------
+# decode steps of up to this many rows run a layer's mixer and its experts side by side on two streams (0: never)
+OVERLAP_ROWS = int(os.environ.get("FLYINGFISH_OVERLAP_ROWS", "64"))
+
+
 class RudoraxModel(DecoderModel):
     mixed_batches = True               # prompt portions and single decoded tokens in one forward
     graph_safe_state = True            # slots and row ranges come from the packed step metadata
@@ -144,6 +152,7 @@ class RudoraxModel(DecoderModel):
         memories = [(r, spec.layer_specs[i]) for r, i in enumerate(self.runs) if spec.layer_specs[i].mixer == "mlstm"]
         self.state_slot_count = max_sequences + 1 if memories else 0          # the last slot is scratch of padding rows
         self.states = {r: mlstm_ops.MemoryState(self.state_slot_count, l.heads, l.dim_pad, l.vdim_pad, dev) for r, l in memories}
+        self.lane = ops.SideLane(dev) if dev.type == "cuda" else None
         # rotations, one table per step for all layers that share one
         self.rotations: list[tuple[torch.Tensor, float]] = []
         self.rotation_of: list[int] = []
@@ -204,26 +213,37 @@ class RudoraxModel(DecoderModel):
         return mlstm_ops.head_out(o, x[:, l.heads * (2 * l.dim_pad + dv):], lw.extra["norm"], l.vdim, self.spec.rms_eps)
 
     # -- feed-forward --------------------------------------------------------------------------
-    def _experts(self, i: int, l: LayerSpec, lw: LayerWeights, n: torch.Tensor):
-        """(the shared expert's rows or None, the routed experts' rows)."""
+    def _experts(self, i: int, l: LayerSpec, lw: LayerWeights, n: torch.Tensor) -> moe_ops.ExpertRows:
+        """The routed experts' rows."""
         m = l.moe
-        weights, ids = moe_ops.route(n, lw.router, m.top_k, m.score, lw.router_bias, exact=True, experts=m.num_experts + m.identity)
+        rows = moe_ops.routed_rows(n, lw.router, m.top_k, m.score, lw.router_bias, m.num_experts + m.identity, lw.experts_gu, lw.experts_down)
         if getattr(self, "route_hook", None) is not None:
-            self.route_hook(i, ids, weights)
-        rows = moe_ops.expert_rows(n, weights, ids, lw.experts_gu, lw.experts_down)
-        shared = ops.linear(ops.linear_swiglu(n, lw.shared_gu), lw.shared_down) if m.n_shared else None
-        return shared, rows
+            self.route_hook(i, rows.ids, rows.weights)
+        return rows
+
+    @staticmethod
+    def _shared(l: LayerSpec, lw: LayerWeights, n: torch.Tensor) -> torch.Tensor | None:
+        """The shared expert's rows."""
+        return ops.linear(ops.linear_swiglu(n, lw.shared_gu), lw.shared_down) if l.moe is not None and l.moe.n_shared else None
 
     # -- forward -----------------------------------------------------------------------------
     def hidden_states(self, b, kv, inputs_embeds=None):
         assert inputs_embeds is None, "the Rudorax model takes token ids"
         assert b.tree_mask is None, "tree verification is not available with a learnable soft-max or recurrent state"
         w, spec, eps = self.w, self.spec, self.spec.rms_eps
+        side = self.lane is not None and b.is_decode and b.rows <= OVERLAP_ROWS
         tables = [ops.rope_angles(b.positions, f, amp) for f, amp in self.rotations]
         norms = [(w.layers[i].input_ln, w.layers[i].post_ln) for i in self.runs] + [(w.final_norm, None)]
         x, n1, n2 = residual_ops.embed(b.ids, w.embed, self.embed_scale, *norms[0], eps, self.width)
         for r, i in enumerate(self.runs):
             l, lw = spec.layer_specs[i], w.layers[i]
+            rows = None
+            if l.moe is not None and side:
+                self.lane.fork()
+                with self.lane:
+                    rows = self._experts(i, l, lw, n2)
+            elif l.moe is not None:
+                rows = self._experts(i, l, lw, n2)
             if l.mixer == "attention":
                 a = self._attention_run(r, l, lw, n1, b, kv, tables[self.rotation_of[i]] if l.rope is not None else None)
             else:
@@ -231,7 +251,9 @@ class RudoraxModel(DecoderModel):
             if self.trace is not None:
                 self.trace.record(f"run.{r}.mixer", a)
             y = ops.linear(a, lw.wo)
-            shared, rows = self._experts(i, l, lw, n2) if l.moe is not None else (None, None)
+            shared = self._shared(l, lw, n2)
+            if side and rows is not None:
+                self.lane.join()
             n1, n2 = residual_ops.step(x, y, shared, rows, *norms[r + 1], eps, self.width)
             if self.trace is not None:
                 self.trace.record(f"run.{r}", x[:, : self.width].clone())

@@ -86,16 +86,50 @@ class _Workspace:
         return t
 
 
-_workspaces: dict[int, _Workspace] = {}
+_workspaces: dict[tuple[int, int], _Workspace] = {}
+_lane = 0
 
 
 def workspace(device: torch.device) -> _Workspace:
     idx = device.index if device.index is not None else torch.cuda.current_device()
-    ws = _workspaces.get(idx)
+    ws = _workspaces.get((idx, _lane))
     if ws is None:
         ws = _Workspace(torch.device("cuda", idx))
-        _workspaces[idx] = ws
+        _workspaces[(idx, _lane)] = ws
     return ws
+
+
+class SideLane:
+    """A second stream with a workspace of its own, for a branch of a layer that does not depend on the other:
+
+        lane.fork()
+        with lane: ...          (this branch)
+        ...                     (the other branch, on the current stream)
+        lane.join()
+
+    Tensors may cross both ways: a branch starts after everything the current stream has been given and is joined before its
+    results are used, so neither stream's freed memory is handed out while the other still reads it."""
+
+    def __init__(self, device: torch.device):
+        self.stream = torch.cuda.Stream(device)
+
+    def fork(self) -> None:
+        self.stream.wait_stream(torch.cuda.current_stream())
+
+    def join(self) -> None:
+        torch.cuda.current_stream().wait_stream(self.stream)
+
+    def __enter__(self):
+        global _lane
+        self._ctx = torch.cuda.stream(self.stream)
+        self._ctx.__enter__()
+        _lane = 1
+        return self
+
+    def __exit__(self, *exc):
+        global _lane
+        _lane = 0
+        return self._ctx.__exit__(*exc)
 
 
 # ------------------------------------------------------------------------------------------

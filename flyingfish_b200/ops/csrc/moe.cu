@@ -5,6 +5,7 @@
 //                   of token rows into expert order -- all on the device, no host read-back
 //                   (the reference syncs the counts to the host before its grouped GEMM,
 //                   src/backend/cuda/moe/prefill.rs:1137)
+//   moe_plan      : for decode-sized batches choices, counts and offsets in one block (moe_gather: the rows)
 //   moe_grouped_gemm : Y[seg rows, N] = Xsorted[seg rows, K] · W[e][N, K]ᵀ for every expert segment,
 //                   swap-AB on tcgen05 (a 128-row slice of the expert weight is the UMMA A operand,
 //                   up to 256 tokens of the segment are the UMMA N dimension), optional SwiGLU
@@ -33,19 +34,12 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
   }
 }
 
+// One row of E logits by one warp; lane j returns the j-th choice (my_w not yet renormalised, wsum the sum of the chosen
+// scores). sc, sel: E floats each of shared memory.
 template <typename T>
-__global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_topk_kernel(const T* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ out_w,
-                int* __restrict__ out_ids, int rows, int E, int top_k, int score_mode, int n_groups, int topk_groups,
-                float routed_scaling, int renormalize, int ld, int* status) {
-  __shared__ float s_score[ROUTE_WARPS][ROUTE_MAX_E];   // unbiased score
-  __shared__ float s_sel[ROUTE_WARPS][ROUTE_MAX_E];     // selection score
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int row = blockIdx.x * ROUTE_WARPS + warp;
-  if (row >= rows) return;
-  float* sc = s_score[warp];
-  float* sel = s_sel[warp];
-  const T* lg = logits + (size_t)row * ld;
+__device__ __forceinline__ void route_row(const T* __restrict__ lg, const float* __restrict__ bias, float* sc, float* sel, int row, int E,
+                                          int top_k, int score_mode, int n_groups, int topk_groups, int lane, float& my_w, int& my_id,
+                                          float& wsum, int* status) {
   if (score_mode == 0) {
     float mx = -INFINITY;
     for (int e = lane; e < E; e += 32) mx = fmaxf(mx, to_float(lg[e]));
@@ -86,8 +80,7 @@ moe_topk_kernel(const T* __restrict__ logits, const float* __restrict__ bias, fl
     for (int e = lane; e < E; e += 32) if (!((keep >> (e / gsz)) & 1u)) sel[e] = -INFINITY;
     __syncwarp();
   }
-  float wsum = 0.f;
-  float my_w = 0.f; int my_id = 0;     // lane j keeps the j-th selection
+  wsum = 0.f; my_w = 0.f; my_id = 0;
   for (int it = 0; it < top_k; ++it) {
     float v = -INFINITY; int i = 0x7fffffff;
     for (int e = lane; e < E; e += 32) {
@@ -103,12 +96,104 @@ moe_topk_kernel(const T* __restrict__ logits, const float* __restrict__ bias, fl
     if (lane == 0) sel[i] = -INFINITY;
     __syncwarp();
   }
+}
+
+__device__ __forceinline__ float route_weight(float w, float wsum, float routed_scaling, int renormalize) {
+  return (renormalize ? w / fmaxf(wsum, 1e-20f) : w) * routed_scaling;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(ROUTE_WARPS * 32)
+moe_topk_kernel(const T* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ out_w,
+                int* __restrict__ out_ids, int rows, int E, int top_k, int score_mode, int n_groups, int topk_groups,
+                float routed_scaling, int renormalize, int ld, int* status) {
+  __shared__ float s_score[ROUTE_WARPS][ROUTE_MAX_E];   // unbiased score
+  __shared__ float s_sel[ROUTE_WARPS][ROUTE_MAX_E];     // selection score
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int row = blockIdx.x * ROUTE_WARPS + warp;
+  if (row >= rows) return;
+  float my_w, wsum; int my_id;                          // lane j keeps the j-th selection
+  route_row(logits + (size_t)row * ld, bias, s_score[warp], s_sel[warp], row, E, top_k, score_mode, n_groups, topk_groups, lane, my_w, my_id, wsum, status);
   if (lane < top_k) {
-    float w = my_w;
-    if (renormalize) w = w / fmaxf(wsum, 1e-20f);
-    out_w[(size_t)row * top_k + lane] = w * routed_scaling;
+    out_w[(size_t)row * top_k + lane] = route_weight(my_w, wsum, routed_scaling, renormalize);
     out_ids[(size_t)row * top_k + lane] = my_id;
   }
+}
+
+// A decode-sized batch: choices, per-expert counts, segment offsets and the row of every choice in one block (32 warps, a row
+// per warp at a time), in place of top-k, count and scan. Outputs from `experts` on are not served (identity outputs).
+constexpr int PLAN_WARPS = 32, PLAN_MAX_ROWS = 64, PLAN_MAX_E = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(PLAN_WARPS * 32)
+moe_plan_kernel(const T* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ out_w, int* __restrict__ out_ids,
+                int* __restrict__ counts, int* __restrict__ seg_off, int* __restrict__ pos, int rows, int E, int experts, int top_k, int score_mode,
+                int ld, int capacity, int* status) {
+  pdl_trigger();
+  extern __shared__ float plan_s[];                     // [PLAN_WARPS][2][E]
+  __shared__ int s_cnt[PLAN_MAX_E], s_off[PLAN_MAX_E], s_warp[PLAN_WARPS];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  for (int e = tid; e < experts; e += blockDim.x) s_cnt[e] = 0;
+  __syncthreads();
+  pdl_wait();
+  constexpr int PER = PLAN_MAX_ROWS / PLAN_WARPS;
+  int id[PER], at[PER];
+#pragma unroll
+  for (int k = 0; k < PER; ++k) {
+    const int row = warp + k * PLAN_WARPS;
+    id[k] = -1; at[k] = 0;
+    if (row >= rows) continue;
+    float my_w, wsum; int my_id;
+    float* sc = plan_s + (size_t)warp * 2 * E;
+    __syncwarp();
+    route_row(logits + (size_t)row * ld, bias, sc, sc + E, row, E, top_k, score_mode, 1, 1, lane, my_w, my_id, wsum, status);
+    if (lane < top_k) {
+      out_w[row * top_k + lane] = route_weight(my_w, wsum, 1.0f, 1);
+      out_ids[row * top_k + lane] = my_id;
+      id[k] = my_id;
+      if (my_id < experts) at[k] = atomicAdd(&s_cnt[my_id], 1);
+    }
+  }
+  __syncthreads();
+  // offsets: segments of multiples of 16 rows, one expert per thread (experts <= 256: eight warps)
+  const int c = tid < experts ? (s_cnt[tid] + 15) / 16 * 16 : 0;
+  int run = c;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) { const int up = __shfl_up_sync(0xffffffffu, run, o); if (lane >= o) run += up; }
+  if (lane == 31) s_warp[warp] = run;
+  __syncthreads();
+  int before = 0;
+  for (int w = 0; w < warp; ++w) before += s_warp[w];
+  run += before;
+  if (tid < experts) {
+    s_off[tid] = run - c;
+    counts[tid] = s_cnt[tid];
+    seg_off[tid] = run - c;
+    if (tid == experts - 1) {
+      seg_off[experts] = run;
+      if (run > capacity) set_status(status, KID_MOE_DISPATCH, FF_ERR_CAPACITY, run, capacity);
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < PER; ++k) {
+    const int row = warp + k * PLAN_WARPS;
+    if (row >= rows || lane >= top_k) continue;
+    const int p = id[k] < experts ? s_off[id[k]] + at[k] : -1;
+    pos[row * top_k + lane] = p < capacity ? p : -1;
+  }
+}
+
+// copies the row of every served choice to its place; one block per choice
+__global__ void __launch_bounds__(128)
+moe_gather_kernel(const uint4* __restrict__ x, const int* __restrict__ pos, uint4* __restrict__ sorted, int vecs, int top_k, int ldx_vecs) {
+  pdl_trigger();
+  pdl_wait();
+  const int p = pos[blockIdx.x];
+  if (p < 0) return;
+  const uint4* src = x + (size_t)(blockIdx.x / top_k) * ldx_vecs;
+  uint4* dst = sorted + (size_t)p * vecs;
+  for (int v = threadIdx.x; v < vecs; v += blockDim.x) dst[v] = src[v];
 }
 
 // ---------------------------------------------------------------------------------------
@@ -192,6 +277,8 @@ __global__ void __launch_bounds__(192, 1)
 moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
                         __nv_bfloat16* __restrict__ Y, const int* __restrict__ seg_off, const int* __restrict__ counts,
                         int Nw, int K, int ldy, int epi, int pipe_bytes, int stage_off, int* status, int capacity) {
+  pdl_trigger();
+  pdl_wait();
   int stages;
   extern __shared__ uint8_t smem_raw[];
   __shared__ GroupBars bars;
@@ -401,6 +488,25 @@ FF_EXPORT int ff_moe_topk(const void* logits, const float* bias, float* out_w, i
   return launch_result();
 }
 
+// Decode-sized batches (rows <= 64, E <= 256, top_k <= 32): renormalised choices over E outputs of which the first `experts` are
+// served, counts int[experts], seg_off int[experts + 1], pos int[rows * top_k], and the served rows of x in `sorted`.
+FF_EXPORT int ff_moe_plan(const void* logits, const float* bias, float* out_w, int* out_ids, int* counts, int* seg_off, int* pos, int rows, int E,
+                          int experts, int top_k, int score_mode, int ld, int f32, const void* x, void* sorted, int hidden, int ldx, int elem_bytes,
+                          int capacity, int* status, cudaStream_t s) {
+  if (rows <= 0 || rows > PLAN_MAX_ROWS || E <= 0 || E > PLAN_MAX_E || experts < 1 || experts > E || top_k < 1 || top_k > 32 || top_k > E) return FF_HOST_BAD_SHAPE;
+  if (hidden % 8 || ldx % 8 || (elem_bytes != 2 && elem_bytes != 4)) return FF_HOST_BAD_ALIGN;
+  const int smem = PLAN_WARPS * 2 * E * 4, per_vec = 16 / elem_bytes;
+  auto go = [&](auto kern, auto lg) -> int {
+    if (int r = opt_in_smem(kern, smem)) return r;
+    return launch_pdl(kern, dim3(1), dim3(PLAN_WARPS * 32), smem, s, 0, lg, bias, out_w, out_ids, counts, seg_off, pos, rows, E, experts, top_k,
+                      score_mode, ld, capacity, status);
+  };
+  if (int r = f32 ? go(moe_plan_kernel<float>, (const float*)logits) : go(moe_plan_kernel<__nv_bfloat16>, (const __nv_bfloat16*)logits)) return r;
+  if (int r = launch_pdl(moe_gather_kernel, dim3(rows * top_k), dim3(128), 0, s, 0, (const uint4*)x, (const int*)pos, (uint4*)sorted, hidden / per_vec,
+                         top_k, ldx / per_vec)) return r;
+  return launch_result();
+}
+
 // counts/cursors: int32[E_local]; seg_off: int32[E_local + 1]; pos: int32[rows * top_k];
 // sorted: [capacity, hidden] rows of elem_bytes elements. Experts [e_lo, e_hi) are local.
 FF_EXPORT int ff_moe_dispatch_local(const void* x, const int* ids, int rows, int top_k, int hidden, int ldx, int E,
@@ -441,8 +547,8 @@ FF_EXPORT int ff_moe_grouped_gemm(const void* xs, const void* w, void* y, const 
   const int smem = staging + pipe_bytes + 1024;
   r = opt_in_smem(moe_grouped_gemm_kernel, 200 * 1024); if (r) return r;
   dim3 grid((Nw + GBM - 1) / GBM, E_local);
-  moe_grouped_gemm_kernel<<<grid, 192, smem, s>>>(tmW, tmX, (__nv_bfloat16*)y, seg_off, counts, Nw, K, ldy, epi,
-                                                  pipe_bytes, staging, status, capacity);
+  if (int lr = launch_pdl(moe_grouped_gemm_kernel, grid, dim3(192), smem, s, 0, tmW, tmX, (__nv_bfloat16*)y, seg_off, counts, Nw, K, ldy, epi,
+                          pipe_bytes, staging, status, capacity)) return lr;
   return launch_result();
 }
 

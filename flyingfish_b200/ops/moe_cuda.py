@@ -109,13 +109,41 @@ def _grouped_gemm_f32(xs, w, seg_off, counts, capacity: int) -> torch.Tensor:
     return y
 
 
+PLAN_MAX_ROWS, PLAN_MAX_OUTPUTS = 64, 256
+
+
 def expert_rows(x, weights, ids, gu, down):
     """See :func:`moe_ops.expert_rows`."""
+    return _served(x, weights, ids, gu, down, dispatch_local(x, ids, 1 << 30, 0, gu.shape[0]))
+
+
+def routed_rows(x, w_router, top_k, score, bias, outputs: int, gu, down):
+    """See :func:`moe_ops.routed_rows`; batches of up to ``PLAN_MAX_ROWS`` rows are routed and dispatched by one block."""
+    rows, el = x.shape[0], gu.shape[0]
+    if rows > PLAN_MAX_ROWS or outputs > PLAN_MAX_OUTPUTS:
+        return expert_rows(x, *route(x, w_router, top_k, score, bias, 1, 1, 1.0, True, True, outputs), gu, down)
+    logits = linear(x, w_router, out_dtype=torch.float32)
+    dev, cap = x.device, ((rows * top_k + 16 * el + 15) // 16) * 16
+    weights = torch.empty(rows, top_k, dtype=torch.float32, device=dev)
+    meta = torch.empty(2 * el + 1 + 2 * rows * top_k, dtype=torch.int32, device=dev)
+    counts, seg_off = meta[:el], meta[el: 2 * el + 1]
+    pos, ids = meta[2 * el + 1:].view(2, rows * top_k)
+    xs = torch.empty(cap, x.shape[1], dtype=x.dtype, device=dev)
+    rc = kernels().ff_moe_plan(ptr(logits), ptr(bias), ptr(weights), ptr(ids), ptr(counts), ptr(seg_off), ptr(pos), rows, outputs, el, top_k,
+                               SCORE_MODES[score], logits.stride(0), 1, ptr(x), ptr(xs), x.shape[1], x.stride(0), x.element_size(), cap,
+                               ptr(status_tensor(dev)), stream_ptr())
+    check(rc, "ff_moe_plan")
+    _count(2)
+    return _served(x, weights, ids.view(rows, top_k), gu, down, (xs, pos, seg_off, counts, cap))
+
+
+def _served(x, weights, ids, gu, down, plan):
+    """The experts' two products over dispatched rows."""
     from . import silu_mul
     from .moe_ops import ExpertRows
     el = gu.shape[0]
     _require(gu.shape[1] == 2 * down.shape[2] and gu.shape[1] % 128 == 0 and gu.is_contiguous() and down.is_contiguous(), "expert stacks")
-    xs, pos, seg_off, counts, cap = dispatch_local(x, ids, 1 << 30, 0, el)
+    xs, pos, seg_off, counts, cap = plan
     if x.dtype == torch.float32:
         y = _grouped_gemm_f32(silu_mul(_grouped_gemm_f32(xs, gu, seg_off, counts, cap), interleaved=True), down, seg_off, counts, cap)
     else:

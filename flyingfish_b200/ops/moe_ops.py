@@ -79,3 +79,14 @@ def add_shared(routed: torch.Tensor, shared: torch.Tensor) -> torch.Tensor:
         return (routed.to(torch.float32) + shared.to(torch.float32)).to(routed.dtype)
     from . import residual_add
     return residual_add(routed, shared)
+
+
+def routed_rows(x: torch.Tensor, w_router: torch.Tensor, top_k: int, score: str, bias: torch.Tensor | None, outputs: int, gu: torch.Tensor,
+                down: torch.Tensor) -> ExpertRows:
+    """:func:`route` with FP32 logits over the first ``outputs`` rows of ``w_router`` and renormalised weights, then
+    :func:`expert_rows`."""
+    if x.is_cuda:
+        from . import moe_cuda
+        return moe_cuda.routed_rows(x, w_router, top_k, score, bias, outputs, gu, down)
+    weights, ids = route(x, w_router, top_k, score, bias, exact=True, experts=outputs)
+    return expert_rows(x, weights, ids, gu, down)

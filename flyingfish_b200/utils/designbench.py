@@ -264,8 +264,14 @@ def _rudorax_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> 
         rpe = rows * e.top_k / e.num_experts
         h = moe_cuda.grouped_gemm(xs, gu, so, ct, cap, epi=1, rows_per_expert=rpe)
         holder["y"], holder["pos"] = moe_cuda.grouped_gemm(h, down, so, ct, cap, epi=0, rows_per_expert=rpe), p
-    pair("experts (dispatch, two grouped GEMMs)", lambda: moe_ops.expert_rows(x, weights, ids, gu, down), expert_cost(ids),
-         "experts (dispatch, two grouped GEMMs)", like_experts, expert_cost(lids))
+    add = lambda p, q: (p[0] + q[0], p[1] + q[1])
+
+    def like_routed():
+        moe_ops.route(x, wr[: e.num_experts], e.top_k, "sigmoid")
+        like_experts()
+    pair("router, dispatch, two grouped GEMMs", lambda: moe_ops.routed_rows(x, wr, e.top_k, "softmax", corr, outs, gu, down),
+         add(expert_cost(ids), pair.gemm(outs, W, out_bytes=8)), "router, dispatch, two grouped GEMMs", like_routed,
+         add(expert_cost(lids), pair.gemm(e.num_experts, W, out_bytes=4)))
     er = moe_ops.expert_rows(x, weights, ids, gu, down)
     like_experts()
     sg, sd = rn(2 * e.shared_ffn, W), rn(W, e.shared_ffn)

@@ -289,11 +289,14 @@ def test_experts(device, dtype, experts, identity, top, ff, width, rows):
     assert torch.equal(chosen.cpu().long(), want_ids)
     close(w, want_w, dtype, "weights", 1e-5)
     assert (want_ids != O.choose_experts(x.double(), lambda k: get(k) * (k != "correction"), "", top)[0]).any() or top == n
-    er = moe_ops.expert_rows(dev(x), w, chosen, dev(gu), dev(down))
-    s = torch.zeros(rows, width, device=device)
-    residual_ops.step(s, dev(torch.zeros_like(x)), None, er, torch.ones(width, device=device), None, 1e-5, width)
     cfg = {"router": {"experts": experts, "identity": identity, "top": top}}
-    close(s, O.mixture(x.double(), get, "", cfg), dtype, "sum", 1e-5 if dtype == "fp32" else 2e-2)
+    want = O.mixture(x.double(), get, "", cfg)
+    for er in (moe_ops.expert_rows(dev(x), w, chosen, dev(gu), dev(down)),
+               moe_ops.routed_rows(dev(x), dev(pad), top, "softmax", dev(t["correction"]), n, dev(gu), dev(down))):
+        assert torch.equal(er.ids.cpu().long(), want_ids)
+        s = torch.zeros(rows, width, device=device)
+        residual_ops.step(s, dev(torch.zeros_like(x)), None, er, torch.ones(width, device=device), None, 1e-5, width)
+        close(s, want, dtype, "sum", 1e-5 if dtype == "fp32" else 2e-2)
 
 
 # ------------------------------------------------------------------------------------------
