@@ -207,7 +207,7 @@ def decode_linear_shapes(spec, tp: int = 1) -> list[tuple[str, int, int, int]]:
         for l in spec.layer_specs:
             for name, n, k in (("qkv", l.projection_cols, spec.hidden), ("o", spec.hidden, l.heads * l.vdim_pad)) + \
                     ((("up", l.ffn, spec.hidden), ("down", spec.hidden, l.ffn)) if l.ffn else ()):
-                seen.setdefault((n, k), name)
+                seen.setdefault((n, k), name if name not in seen.values() else f"{name} {n} x {k}")
         return [(name, n, k, 0) for (n, k), name in seen.items()]
     d, h = spec.head_dim, spec.hidden
     hq, hkv = spec.heads // tp, max(1, spec.kv_heads // tp)
