@@ -46,19 +46,21 @@ class MlaSpec:
 
 @dataclass
 class RopeSpec:
-    """Rotary positions on the first ``dims`` elements of a head, pairs being neighbours (2i, 2i + 1)."""
+    """Rotary positions on the first ``dims`` elements of a head. Pairs are neighbours (2i, 2i + 1) or, with ``halves``, elements
+    (i, i + dims / 2)."""
     base: float
     dims: int
-    factor: float = 1.0               # > 0 with ``original``: YaRN-scaled frequencies and amplitude
+    factor: float = 1.0               # with ``original``: YaRN-scaled frequencies and amplitude; without: frequencies / factor
     original: int = 0
     fast: float = 32.0
     slow: float = 1.0
+    halves: bool = False
 
     def frequencies(self) -> tuple[list[float], float]:
         """(angle per position of every pair, factor of cosine and sine), in double precision."""
         plain = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
         if not self.original:
-            return plain, 1.0
+            return [f / self.factor for f in plain], 1.0
         turn = lambda t: self.dims * math.log(self.original / (2.0 * math.pi * t)) / (2.0 * math.log(self.base))
         lo, hi = max(math.floor(turn(self.fast)), 0), min(math.ceil(turn(self.slow)), self.dims - 1)
         ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(self.dims // 2)]
@@ -73,16 +75,24 @@ class LayerSpec:
     dim: int                          # width of a query / key head
     vdim: int                         # width of a value head
     scale: float                      # factor of the attention scores (of the queries, for a matrix memory)
-    mixer: str = "attention"          # attention | mlstm (matrix memory: per-sequence state instead of a cache)
+    mixer: str = "attention"          # attention | mlstm (matrix memory: per-sequence state instead of a cache) | latent (latent attention)
     chunk: int = 0                    # > 0: position i sees only keys of its own block of ``chunk`` positions
     window: int = 0                   # > 0: position i sees itself and the ``window - 1`` positions before it
+    keep_first: int = 0               # with a window: the sequence's first ``keep_first`` positions stay visible
     sink: bool = False                # learnable soft-max: one extra logit per head in the denominator
     rope: RopeSpec | None = None
+    qk_norm: str = "head"             # RMS norm of q and k: over every head, or over the whole projection ("row")
+    bias: bool = False                # the projections have biases
+    softcap: float = 0.0              # > 0: scores become softcap * tanh(score / softcap)
+    q_temp: tuple[float, int] | None = None       # (coef, every): the query at p is multiplied by 1 + coef ln((p + 1) // every + 1)
+    kv_from: int = -1                 # >= 0: keys and values are those of that layer's cache
+    kv_rank: int = 0                  # latent attention: width of the latent a token caches
+    rot_dim: int = 0                  # latent attention: width of the rotated key part all heads share (and of the queries')
     gate_cap: float = 0.0             # matrix memory: soft cap of the gates' logits
     out_gate: bool = True             # the heads' outputs are multiplied by the sigmoid of a projection
     v_mix: bool = False               # values are mixed with those of the first layer that has the flag
     ffn: int = 0                      # width of the feed-forward (0: the layer has none, or experts)
-    ffn_act: str = "relu2"
+    ffn_act: str = "relu2"            # relu2 (two matrices) | geglu (gate, up and down matrices, tanh-GELU)
     moe: MoeSpec | None = None        # experts in place of a dense feed-forward
 
     @property
@@ -93,17 +103,26 @@ class LayerSpec:
     def vdim_pad(self) -> int:
         return pad_to(self.vdim, 16)
 
+    @property
+    def rot_pad(self) -> int:
+        return pad_to(self.rot_dim, 16)
+
+    @property
+    def rank_pad(self) -> int:
+        return pad_to(self.kv_rank, 16)
+
     def keys_seen(self, ctx: int) -> int:
         """Keys the last of ``ctx`` positions sees."""
         if self.window:
-            return min(ctx, self.window)
+            return min(ctx, self.window) + min(max(ctx - self.window, 0), self.keep_first)
         return (ctx - 1) % self.chunk + 1 if self.chunk else ctx
 
     def pairs_seen(self, n: int) -> int:
         """(query, key) pairs of a prompt of ``n`` positions."""
         if self.window:
             w = min(n, self.window)
-            return w * (w + 1) // 2 + (n - w) * w
+            k = min(n - w, self.keep_first)        # row w + j sees j + 1 kept positions outside its window, up to keep_first
+            return w * (w + 1) // 2 + (n - w) * w + k * (k + 1) // 2 + (n - w - k) * self.keep_first
         if not self.chunk:
             return n * (n + 1) // 2
         full, rest = divmod(n, self.chunk)
@@ -113,24 +132,37 @@ class LayerSpec:
         """Bytes of cache or state one decoded token moves at a context of ``ctx``."""
         if self.mixer == "mlstm":
             return 2 * 4 * self.heads * self.dim * (self.vdim + 1)
+        if self.mixer == "latent":
+            return elem_bytes * self.keys_seen(ctx) * (self.kv_rank + self.rot_dim)
         return elem_bytes * self.keys_seen(ctx) * self.kv_heads * (self.dim + self.vdim)
 
     def mixer_flops(self, n: int) -> int:
         """FLOPs of a prompt of ``n`` positions outside the projections."""
         if self.mixer == "mlstm":         # the recurrence: state update and read of every position
             return 4 * n * self.heads * self.dim * self.vdim
+        if self.mixer == "latent":        # scores and values in the latent space
+            return 2 * self.heads * (2 * self.kv_rank + self.rot_dim) * self.pairs_seen(n)
         return 2 * self.heads * (self.dim + self.vdim) * self.pairs_seen(n)
 
     @property
     def projection_cols(self) -> int:
         """Columns of the fused input projection, heads padded."""
+        if self.mixer == "latent":        # [unrotated queries | rotated queries | latent | rotated key | head gates]
+            return self.heads * (self.dim_pad + self.rot_pad) + self.rank_pad + self.rot_pad + pad_to(self.heads, 8)
+        if self.kv_from >= 0:
+            return self.heads * self.dim_pad
         g = self.heads * self.vdim_pad if self.out_gate else 0
         return self.heads * self.dim_pad + self.kv_heads * (self.dim_pad + self.vdim_pad) + g
 
     def params(self, hidden: int, active: bool = False) -> int:
         """Matrix weights of the layer; ``active``: those one token uses."""
-        n = hidden * (self.heads * (self.dim + self.vdim * (2 if self.out_gate else 1)) + self.kv_heads * (self.dim + self.vdim))
-        n += 2 * hidden * self.ffn + (2 * hidden * self.heads if self.mixer == "mlstm" else 0)
+        if self.mixer == "latent":
+            n = hidden * (self.heads * (self.dim + self.rot_dim + self.vdim + 1) + self.kv_rank + self.rot_dim) + \
+                self.heads * self.kv_rank * (self.dim + self.vdim)
+        else:
+            own = self.kv_heads if self.kv_from < 0 else 0
+            n = hidden * (self.heads * (self.dim + self.vdim * (2 if self.out_gate else 1)) + own * (self.dim + self.vdim))
+        n += (3 if self.ffn_act == "geglu" else 2) * hidden * self.ffn + (2 * hidden * self.heads if self.mixer == "mlstm" else 0)
         if self.moe is not None:
             m = self.moe
             n += hidden * (m.num_experts + m.identity) + 3 * hidden * (m.expert_ffn * (m.top_k if active else m.num_experts) + m.shared_ffn * m.n_shared)
@@ -138,7 +170,7 @@ class LayerSpec:
 
 
 # architectures whose every operator has a 32-bit kernel on the GPU
-GPU_FP32_ARCHS = ("duponex", "rudorax")
+GPU_FP32_ARCHS = ("duponex", "rudorax", "kabavik")
 
 
 def pad_to(n: int, m: int) -> int:
@@ -148,7 +180,7 @@ def pad_to(n: int, m: int) -> int:
 @dataclass
 class ModelSpec:
     name: str
-    arch: str                         # llama | qwen3 | qwen3_moe | deepseek_v3 | deepseek_v41 | glm5_next | flint | loop_vl | tiny_moe | qwen3_vl | embedding | diffusion_lm | qwen35_text | gemma | duponex | rudorax
+    arch: str                         # llama | qwen3 | qwen3_moe | deepseek_v3 | deepseek_v41 | glm5_next | flint | loop_vl | tiny_moe | qwen3_vl | embedding | diffusion_lm | qwen35_text | gemma | duponex | rudorax | kabavik
     layers: int
     hidden: int
     heads: int
@@ -200,19 +232,29 @@ class ModelSpec:
     def kv_geometry(self) -> list[tuple[int, int, int]] | None:
         """(kv heads, key width, value width) of every cache layer where the layers differ, None where one size serves
         all. Widths are padded to 16 elements, the alignment of the attention kernels' tiles; a run that keeps its past in a
-        per-sequence state has none."""
+        per-sequence state or reads another layer's cache has none. A latent layer caches one row per token, the latent and
+        the rotated key part behind it; its values are the row's first columns."""
         if self.layer_specs is None:
             return None
-        size = lambda l: (l.kv_heads, l.dim_pad, l.vdim_pad) if l.mixer == "attention" else (0, 0, 0)
+
+        def size(l: LayerSpec) -> tuple[int, int, int]:
+            if l.mixer == "latent":
+                return 1, l.rank_pad + l.rot_pad, 0
+            return (l.kv_heads, l.dim_pad, l.vdim_pad) if l.mixer == "attention" and l.kv_from < 0 else (0, 0, 0)
         return [size(self.layer_specs[i]) for i in self.runs]
+
+    @property
+    def side_dim(self) -> int:
+        """Width of a layer's part of the per-layer token embeddings (0: the design has none)."""
+        return int(self.extra.get(self.arch, {}).get("side_dim", 0))
 
     def run_params(self) -> int:
         """Matrix weights one token passes through in all layer runs (a looped layer counts every time)."""
-        return sum(self.layer_specs[i].params(self.hidden, active=True) for i in self.runs)
+        return sum(self.layer_specs[i].params(self.hidden, active=True) + 2 * self.hidden * self.side_dim for i in self.runs)
 
     def dense_param_count(self) -> int:
         if self.layer_specs is not None:
-            return sum(l.params(self.hidden) for l in self.layer_specs) + (1 if self.tie_embeddings else 2) * self.vocab * self.hidden
+            return sum(l.params(self.hidden) + (2 * self.hidden + self.vocab) * self.side_dim for l in self.layer_specs) + (1 if self.tie_embeddings else 2) * self.vocab * self.hidden
         per_layer = self.hidden * self.qkv_dim + self.q_dim * self.hidden + 3 * self.hidden * self.ffn + 2 * self.hidden
         return self.layers * per_layer + (1 if self.tie_embeddings else 2) * self.vocab * self.hidden + self.hidden
 
@@ -521,6 +563,65 @@ def rudorax_4k() -> ModelSpec:
     return _rudorax_bench("rudorax-4k-shape", 4096, 32, 8, 64, 1536, 128256)
 
 
+def _kabavik_spec_of(name: str, hidden: int, vocab: int, layers: list[LayerSpec], embed_scale: float, residual_mult: float,
+                     logit_scale: float, side_dim: int, eps: float) -> ModelSpec:
+    if not layers:
+        raise ConfigError("a Kabavik model needs at least one layer")
+    for i, l in enumerate(layers):
+        if min(l.heads, l.kv_heads, l.dim, l.vdim) < 1 or l.heads % l.kv_heads or min(l.window, l.keep_first, l.ffn) < 0 or not l.scale > 0:
+            raise ConfigError(f"layer {i}: unusable mixer sizes {l}")
+        turned = l.rot_dim if l.mixer == "latent" else l.dim
+        if l.rope is not None and (l.rope.dims % 2 or not 0 < l.rope.dims <= turned or not l.rope.base > 1 or not l.rope.factor > 0):
+            raise ConfigError(f"layer {i}: unusable rotation {l.rope} of {turned} elements")
+        if l.mixer == "latent" and (min(l.kv_rank, l.rot_dim) < 1 or l.rope is None or l.rope.halves):
+            raise ConfigError(f"layer {i}: latent attention needs a latent and a part whose neighbours rotate")
+        if l.q_temp is not None and l.q_temp[1] < 1:
+            raise ConfigError(f"layer {i}: unusable query temperature {l.q_temp}")
+        if l.kv_from >= 0:
+            src = layers[l.kv_from] if l.kv_from < i else None
+            if src is None or src.kv_from >= 0 or (src.mixer, src.kv_heads, src.dim, src.vdim) != (l.mixer, l.kv_heads, l.dim, l.vdim):
+                raise ConfigError(f"layer {i}: cannot take keys and values from layer {l.kv_from}")
+    wide = max(layers, key=lambda l: l.heads * l.dim)
+    return ModelSpec(
+        name=name, arch="kabavik", layers=len(layers), hidden=hidden, heads=wide.heads, kv_heads=wide.kv_heads, head_dim=wide.dim,
+        ffn=max(l.ffn for l in layers), vocab=vocab, rms_eps=eps, qk_norm=True, layer_specs=layers,
+        extra={"kabavik": {"embed_scale": embed_scale, "residual_mult": residual_mult, "logit_scale": logit_scale, "side_dim": side_dim}})
+
+
+def kabavik_tiny() -> ModelSpec:
+    """Small Kabavik shape: windowed attention that keeps the first positions, a layer that shares its keys and values,
+    latent attention, and full attention with capped scores and a query temperature."""
+    win = dict(heads=4, kv_heads=2, dim=32, vdim=40, scale=0.2, window=72, keep_first=5, qk_norm="row", bias=True, out_gate=False, ffn=192,
+               ffn_act="geglu", rope=RopeSpec(base=1e4, dims=24, factor=2.0, halves=True))
+    lat = dict(heads=3, kv_heads=1, dim=24, vdim=40, scale=0.2, mixer="latent", window=56, kv_rank=40, rot_dim=16, out_gate=False, ffn=192,
+               ffn_act="geglu", rope=RopeSpec(base=1e4, dims=16, factor=4.0, original=128))
+    cap = dict(heads=4, kv_heads=1, dim=48, vdim=16, scale=0.2, softcap=20.0, q_temp=(0.2, 64), bias=True, out_gate=False, ffn=192, ffn_act="geglu")
+    return _kabavik_spec_of("kabavik-tiny", 160, 512, [LayerSpec(**win), LayerSpec(**lat), LayerSpec(**cap), LayerSpec(**dict(win, kv_from=0)),
+                                                       LayerSpec(**dict(cap, ffn=0))],
+                            embed_scale=1.0, residual_mult=0.8, logit_scale=0.5, side_dim=24, eps=1e-5)
+
+
+def _kabavik_bench(name: str, hidden: int, heads: int, kv_heads: int, ff: int, vocab: int) -> ModelSpec:
+    own = dict(out_gate=False, ffn=ff, ffn_act="geglu", scale=128 ** -0.5)
+    win = LayerSpec(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, window=2048, keep_first=64, qk_norm="row", bias=True,
+                    rope=RopeSpec(base=1e6, dims=128, factor=2.0, halves=True), **own)
+    lat = LayerSpec(heads=heads, kv_heads=1, dim=128, vdim=128, mixer="latent", window=2048, kv_rank=512, rot_dim=64,
+                    rope=RopeSpec(base=1e6, dims=64, factor=4.0, original=8192), **own)
+    cap = LayerSpec(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, softcap=30.0, q_temp=(0.1, 4096), bias=True, **own)
+    return _kabavik_spec_of(name, hidden, vocab, [win, lat, cap, dataclasses.replace(win, kv_from=0)] * 2, embed_scale=1.0, residual_mult=0.7,
+                            logit_scale=0.5, side_dim=256, eps=1e-5)
+
+
+def kabavik_2k() -> ModelSpec:
+    """Kabavik layers 2048 wide (random weights, for measurements): 16 / 4 heads of 128, latents of 512 + 64, feed-forward 8192."""
+    return _kabavik_bench("kabavik-2k-shape", 2048, 16, 4, 8192, 65536)
+
+
+def kabavik_4k() -> ModelSpec:
+    """As :func:`kabavik_2k` at 4096: 32 / 8 heads, feed-forward 14336."""
+    return _kabavik_bench("kabavik-4k-shape", 4096, 32, 8, 14336, 128256)
+
+
 def glm5_next_tiny() -> ModelSpec:
     """Small GLM-5-style shape: the hyper-connection program with every stage collapsing on its own pre-mix, top-k sparse
     attention with the pooled indexer in every layer, sigmoid routing with selection bias."""
@@ -537,6 +638,7 @@ NAMED_SHAPES = {
     "deepseek-v3-fp8-mini": deepseek_v3_fp8_mini, "deepseek-v41-tiny": deepseek_v41_tiny, "glm5-next-tiny": glm5_next_tiny, "flint-tiny": flint_tiny,
     "duponex-tiny": duponex_tiny, "duponex-8b-shape": duponex_8b, "duponex-2b-shape": duponex_2b,
     "rudorax-tiny": rudorax_tiny, "rudorax-2k-shape": rudorax_2k, "rudorax-4k-shape": rudorax_4k,
+    "kabavik-tiny": kabavik_tiny, "kabavik-2k-shape": kabavik_2k, "kabavik-4k-shape": kabavik_4k,
     "loop-tiny": loop_tiny, "loopvl-text-shape": loopvl_text,
     "qwen3-moe-235b-shape": qwen3_moe_235b, "qwen3-moe-tiny": qwen3_moe_tiny,
 }
@@ -696,6 +798,40 @@ def _rudorax_spec(cfg: dict[str, Any], name: str) -> ModelSpec:
                             loop=(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None)
 
 
+def _kabavik_spec(cfg: dict[str, Any], name: str) -> ModelSpec:
+    """``"architecture": "Kabavik"``: a list of layers with windowed, latent or capped full attention, gated feed-forwards and a
+    per-layer token input."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+        m, mlp, kind = entry["mixer"], entry.get("mlp"), entry.get("type")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ConfigError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r}")
+        mask, rot = m.get("mask") or {}, m.get("rot")
+        sizes = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]), window=int(mask.get("size", 0)),
+                     keep_first=int(mask.get("keep_first", 0)), kv_from=int(m["kv_from"]) if m.get("kv_from") is not None else -1,
+                     out_gate=False, ffn=int(mlp["ff"]) if mlp is not None else 0, ffn_act="geglu")
+        rope = None
+        if rot is not None:
+            sc = rot.get("scaling") or {}
+            rope = RopeSpec(base=float(rot["base"]), dims=int(rot["dims"]), factor=float(sc.get("factor", 1.0)), halves=kind == "attention")
+            if kind == "latent_attention" and sc:
+                rope = dataclasses.replace(rope, original=int(sc["original"]), fast=float(sc["fast"]), slow=float(sc["slow"]))
+        if kind == "attention":
+            layers.append(LayerSpec(kv_heads=int(m["kv_heads"]), qk_norm="row", bias=True, rope=rope, **sizes))
+        elif kind == "attention_2":
+            temp = m.get("q_temp")
+            layers.append(LayerSpec(kv_heads=int(m["kv_heads"]), bias=True, softcap=float(m.get("softcap") or 0.0),
+                                    q_temp=(float(temp["coef"]), int(temp["every"])) if temp else None, **sizes))
+        elif kind == "latent_attention":
+            layers.append(LayerSpec(kv_heads=1, mixer="latent", kv_rank=int(m["kv_rank"]), rot_dim=int(m["rot_dim"]), rope=rope, **sizes))
+        else:
+            raise ConfigError(f"layer {i}: unsupported mixer {kind!r}")
+    side = cfg.get("token_side")
+    return _kabavik_spec_of(name, int(cfg["width"]), int(cfg["vocab"]), layers, embed_scale=float(cfg["embedding"]["scale"]),
+                            residual_mult=float(cfg["residual_mult"]), logit_scale=float(cfg["logit_scale"]),
+                            side_dim=int(side["dim"]) if side else 0, eps=float(cfg["norm"]["eps"]))
+
+
 def spec_from_hf_config(cfg: dict[str, Any], name: str = "model") -> ModelSpec:
     """Normalise a Hugging Face ``config.json``. Hard checks mirror the reference's: SiLU
     activation only, 16-bit or 32-bit floats, no unsupported rope scaling for plain Llama."""
@@ -703,6 +839,8 @@ def spec_from_hf_config(cfg: dict[str, Any], name: str = "model") -> ModelSpec:
         return _duponex_spec(cfg, name)
     if cfg.get("architecture") == "Rudorax":
         return _rudorax_spec(cfg, name)
+    if cfg.get("architecture") == "Kabavik":
+        return _kabavik_spec(cfg, name)
     archs = cfg.get("architectures") or []
     arch = next((_ARCH_MAP[a] for a in archs if a in _ARCH_MAP), None)
     if arch is None:

@@ -6,7 +6,7 @@ from __future__ import annotations
 
 import importlib
 
-MODULES = {"duponex": "duponex", "rudorax": "rudorax"}
+MODULES = {"duponex": "duponex", "rudorax": "rudorax", "kabavik": "kabavik"}
 
 
 def design(arch: str):

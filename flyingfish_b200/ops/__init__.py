@@ -146,13 +146,15 @@ FUSE_ATTN_MERGE = os.environ.get("FLYINGFISH_FUSE_ATTN_MERGE", "0") == "1"
 ATTN_PREFILL_TC = os.environ.get("FF_ATTN_PREFILL", "tc") != "mma"
 
 
-ACTIVATIONS = {None: 0, "relu2": 1}
+ACTIVATIONS = {None: 0, "relu2": 1, "gelu_tanh": 3}
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
-           out_dtype: torch.dtype | None = None, bias: torch.Tensor | None = None, act: str | None = None) -> torch.Tensor:
+           out_dtype: torch.dtype | None = None, bias: torch.Tensor | None = None, act: str | None = None,
+           mul: tuple[torch.Tensor, torch.Tensor] | None = None) -> torch.Tensor:
     """``y[M,N] = act(x[M,K] @ w[N,K].T + bias[N])`` (BF16 operands, FP32 accumulation, bias and activation in the GEMM's
-    epilogue; ``act``: "relu2", the square of the positive part). FP32 operands take the SIMT kernel of
+    epilogue; ``act``: "relu2", the square of the positive part, or "gelu_tanh"). ``mul`` = (table [T, N] of the operands' type, int32
+    ids [M]): the result is multiplied by the table's row of every id, in the epilogue too. FP32 operands take the SIMT kernel of
     ``csrc/gemm_f32.cu`` (true 32-bit products).
 
     CUDA path: tcgen05 kernels -- the weight-streaming decode kernel of ``csrc/gemm_skinny.cu`` (tokens on
@@ -160,7 +162,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
     ``csrc/gemm_bf16.cu`` otherwise. ``w`` may be an FP8-resident weight (``quant_ops.Fp8Weight``): the block-scaled
     W8A8 GEMM of ``csrc/gemm_fp8.cu`` (CPU: its oracle) runs instead."""
     if not isinstance(w, torch.Tensor):
-        _require(bias is None and act is None, "linear: FP8-resident weights take no bias or activation")
+        _require(bias is None and act is None and mul is None, "linear: FP8-resident weights take no bias or activation")
         from . import quant_ops
         tok = min(128, (x.shape[0] + 15) // 16 * 16)
         if x.shape[0] > FP8_DENSE_ROWS or w.shape[1] > FP8_MAX_K or (w.shape[1] // 128) * tok * 4 > 64 * 1024:
@@ -176,7 +178,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
             return out
         return y
     if not _is_cuda(x):
-        y = ref.linear(x, w, out_dtype, bias, act)
+        y = ref.linear(x, w, out_dtype, bias, act, mul)
         if out is not None:
             out.copy_(y)
             return out
@@ -184,8 +186,12 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
     if bias is not None:
         _require(bias.dtype == x.dtype and bias.numel() == w.shape[0] and bias.is_contiguous() and bias.data_ptr() % 16 == 0,
                  "linear: bias must be one aligned vector of the operands' type")
+    if mul is not None:
+        table, rows_of = mul
+        _require(table.dtype == x.dtype and table.shape[1] == w.shape[0] and table.stride(1) == 1 and table.data_ptr() % 16 == 0 and
+                 table.stride(0) % 8 == 0 and rows_of.dtype == torch.int32 and rows_of.numel() == x.shape[0], "linear: table of factors")
     if x.dtype == torch.float32:
-        return _linear_f32(x, w, out, out_dtype, bias, act)
+        return _linear_f32(x, w, out, out_dtype, bias, act, mul)
     _require(x.dtype == BF16 and w.dtype == BF16, "linear: BF16 operands required on CUDA")
     m, ldx = _rows2d(x)
     n, ldw = _rows2d(w)
@@ -197,8 +203,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
     _require(out.shape == (m, n) and out.stride(1) == 1 and out.dtype == odt, "linear: bad output tensor")
     lib = kernels()
     st = status_tensor(x.device)
-    plain = bias is None and act is None
-    _require(plain or odt == BF16, "linear: bias and activation come with a bf16 output")
+    plain = bias is None and act is None and mul is None
+    _require(plain or odt == BF16, "linear: bias, activation and factors come with a bf16 output")
     _require(odt in (BF16, torch.float32), "linear: output dtype must be bf16 or fp32")
     if m <= SKINNY_MAX_M:
         scratch_b, counter_b = c_longlong(0), c_longlong(0)
@@ -212,22 +218,26 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None,
         elif plain:
             rc = lib.ff_gemm_skinny(*args, ptr(st), stream_ptr())
         else:
-            rc = lib.ff_gemm_skinny_act(*args, ptr(bias), ACTIVATIONS[act], ptr(st), stream_ptr())
+            rc = lib.ff_gemm_skinny_act(*args, ptr(bias), ACTIVATIONS[act], *_factors(mul), ptr(st), stream_ptr())
         check(rc, "ff_gemm_skinny")
     else:
         epi = 0 if odt == BF16 else 2
         if plain:
             rc = lib.ff_gemm_bf16(ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), epi, ptr(st), stream_ptr())
         else:
-            rc = lib.ff_gemm_bf16_act(ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), ptr(bias), ACTIVATIONS[act], ptr(st),
-                                      stream_ptr())
+            rc = lib.ff_gemm_bf16_act(ptr(x), ptr(w), ptr(out), m, n, k, ldx, ldw, out.stride(0), ptr(bias), ACTIVATIONS[act], *_factors(mul),
+                                      ptr(st), stream_ptr())
         check(rc, "ff_gemm_bf16")
     _count()
     return out
 
 
+def _factors(mul: tuple[torch.Tensor, torch.Tensor] | None) -> tuple:
+    return (None, None, 0, 0) if mul is None else (ptr(mul[0]), ptr(mul[1]), mul[0].stride(0), mul[0].shape[0])
+
+
 def _linear_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None, out_dtype: torch.dtype | None,
-                bias: torch.Tensor | None, act: str | None) -> torch.Tensor:
+                bias: torch.Tensor | None, act: str | None, mul: tuple[torch.Tensor, torch.Tensor] | None = None) -> torch.Tensor:
     _require(w.dtype == torch.float32 and out_dtype in (None, torch.float32), "linear: FP32 operands give an FP32 result")
     m, ldx = _rows2d(x)
     n, ldw = _rows2d(w)
@@ -236,8 +246,33 @@ def _linear_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None, out_
         out = torch.empty(m, n, dtype=torch.float32, device=x.device)
     _require(out.shape == (m, n) and out.stride(1) == 1 and out.dtype == torch.float32, "linear: bad output tensor")
     rc = kernels().ff_gemm_f32(ptr(x), ptr(w), ptr(out), m, n, x.shape[1], ldx, ldw, out.stride(0), ptr(bias), ACTIVATIONS[act],
-                               stream_ptr())
+                               *_factors(mul), stream_ptr())
     check(rc, "ff_gemm_f32")
+    _count()
+    return out
+
+
+def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, x_cols: int | None = None,
+                out_cols: int | None = None) -> torch.Tensor:
+    """Block-diagonal product: head h of ``x`` (``K`` columns from ``h * x_cols``) times ``w[h]`` ([heads, N, K]) goes to columns
+    ``h * out_cols .. + N`` of ``out``. ``x_cols`` / ``out_cols`` default to K / N. BF16 (tcgen05) or FP32."""
+    heads, n, k = w.shape
+    x_cols, out_cols = x_cols or k, out_cols or n
+    rows, ldx = _rows2d(x)
+    if out is None:
+        out = torch.empty(rows, heads * out_cols, dtype=x.dtype, device=x.device)
+    _require(x.dtype == w.dtype == out.dtype and w.is_contiguous() and out.shape[0] == rows and out.stride(1) == 1, "head_linear: operands of one type")
+    _require(x.shape[1] >= (heads - 1) * x_cols + k and out.shape[1] >= (heads - 1) * out_cols + n, "head_linear: rows too short")
+    if not _is_cuda(x):
+        for h in range(heads):
+            out[:, h * out_cols: h * out_cols + n] = ref.linear(x[:, h * x_cols: h * x_cols + k], w[h])
+        return out
+    args = (ptr(x), ptr(w), ptr(out), rows, heads, n, k, ldx, out.stride(0), x_cols, out_cols)
+    if x.dtype == torch.float32:
+        rc = kernels().ff_gemm_f32_heads(*args, stream_ptr())
+    else:
+        rc = kernels().ff_gemm_bf16_heads(*args, ptr(status_tensor(x.device)), stream_ptr())
+    check(rc, "ff_gemm_heads")
     _count()
     return out
 
@@ -249,15 +284,15 @@ def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tenso
     if not _is_cuda(x):
         return ref.linear_swiglu(x, w_interleaved, mode)
     if x.dtype == torch.float32:
-        return silu_mul_interleaved(linear(x, w_interleaved), out)
+        return silu_mul_interleaved(linear(x, w_interleaved), out, mode)
     m, ldx = _rows2d(x)
     n, ldw = _rows2d(w_interleaved)
     k = x.shape[1]
     _require(n % 256 == 0, "linear_swiglu: N must be a multiple of 256")
     if out is None:
         out = torch.empty(m, n // 2, dtype=BF16, device=x.device)
-    if mode != 0:
-        # the GEMM epilogues implement rounding mode 0; other gates (tanh-GELU, clamped) run as the activation kernel
+    if mode not in (0, 3):
+        # the GEMM epilogues implement modes 0 and 3 (tanh-GELU rounded once); other gates run as the activation kernel
         return silu_mul_interleaved(linear(x, w_interleaved), out, mode)
     if m <= SKINNY_MAX_M and not FUSE_SWIGLU:
         return silu_mul_interleaved(linear(x, w_interleaved), out)
@@ -271,12 +306,13 @@ def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tenso
         scratch = ws.ensure("gemm_scratch", scratch_b.value // 4) if scratch_b.value > 0 else None
         _require(counter_b.value // 4 <= ws.gemm_counters.numel(), "linear_swiglu: too many column tiles for counters")
         rc = lib.ff_gemm_skinny_swiglu(ptr(x), ptr(w_interleaved), ptr(out), m, n, k, ldx, ldw, out.stride(0), grid,
-                                       ptr(scratch), ptr(ws.gemm_counters), ptr(status_tensor(x.device)), stream_ptr())
+                                       ptr(scratch), ptr(ws.gemm_counters), mode, ptr(status_tensor(x.device)), stream_ptr())
         check(rc, "ff_gemm_skinny_swiglu")
         _count()
         return out
-    rc = kernels().ff_gemm_bf16(ptr(x), ptr(w_interleaved), ptr(out), m, n, k, ldx, ldw, out.stride(0), 1,
-                                ptr(status_tensor(x.device)), stream_ptr())
+    args = (ptr(x), ptr(w_interleaved), ptr(out), m, n, k, ldx, ldw, out.stride(0))
+    st = ptr(status_tensor(x.device))
+    rc = kernels().ff_gemm_bf16_geglu(*args, st, stream_ptr()) if mode == 3 else kernels().ff_gemm_bf16(*args, 1, st, stream_ptr())
     check(rc, "ff_gemm_bf16(swiglu)")
     _count()
     return out
@@ -456,36 +492,57 @@ def linear_rope_kv(x: torch.Tensor, wqkv: torch.Tensor, positions: torch.Tensor,
 def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, hq: int, hkv: int,
                  dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0,
                  q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None,
-                 cos_sin: torch.Tensor | None = None) -> None:
+                 cos_sin: torch.Tensor | None = None, whole: bool = False, halves: bool = False,
+                 temp: tuple[torch.Tensor, float, int] | None = None) -> None:
     """Packed rows ``[q heads | k heads | v heads | ...]``: q and k are divided by their root mean square per head
     (``dim`` elements count, the row's heads may carry padding up to the cache's width), v is blended with
     ``first_v`` (``(1 - mix) v + mix first_v``; a column slice of an earlier layer's packed rows), k and v are written to
     ``slots`` of the paged cache and q back into the row. ``q_weight`` / ``k_weight``: FP32 norm weights as wide
-    as the row's heads; ``cos_sin`` (:func:`rope_angles`): neighbours (2i, 2i + 1) of the normed q and k turn. BF16 or FP32."""
+    as the row's heads; ``cos_sin`` (:func:`rope_angles`): neighbours (2i, 2i + 1) of the normed q and k turn. BF16 or FP32.
+
+    ``whole``: q and k are normed over all their heads together (weights then cover every head). ``halves``: elements (i, i + half)
+    turn instead of neighbours. ``temp`` = (int32 positions, coef, every): the query at p is multiplied by
+    ``1 + coef ln((p + 1) // every + 1)``. ``hkv`` 0 (no caches): a row of queries alone."""
     if not _is_cuda(qkv):
-        ref.head_norm_kv(qkv, slots, kcache, vcache, hq, hkv, dim, vdim, eps, first_v, mix, q_weight, k_weight, cos_sin)
+        ref.head_norm_kv(qkv, slots, kcache, vcache, hq, hkv, dim, vdim, eps, first_v, mix, q_weight, k_weight, cos_sin, whole, halves, temp)
         return
     rows, ld = _rows2d(qkv)
-    nb, ch, bs, dk = kcache.shape
-    dv = vcache.shape[3]
-    _require(slots.dtype == torch.int32 and kcache.is_contiguous() and vcache.is_contiguous(), "head_norm_kv: metadata / cache layout")
-    _require(ch == hkv == vcache.shape[1] and vcache.shape[0] == nb and vcache.shape[2] == bs and dk >= dim and dv >= vdim,
-             "head_norm_kv: cache geometry differs from the heads")
-    _require(qkv.shape[1] >= (hq + hkv) * dk + hkv * dv and qkv.dtype == kcache.dtype == vcache.dtype, "head_norm_kv: packed row")
+    if hkv:
+        nb, ch, bs, dk = kcache.shape
+        dv = vcache.shape[3]
+        _require(slots.dtype == torch.int32 and kcache.is_contiguous() and vcache.is_contiguous(), "head_norm_kv: metadata / cache layout")
+        _require(ch == hkv == vcache.shape[1] and vcache.shape[0] == nb and vcache.shape[2] == bs and dk >= dim and dv >= vdim,
+                 "head_norm_kv: cache geometry differs from the heads")
+        _require(qkv.shape[1] >= (hq + hkv) * dk + hkv * dv and qkv.dtype == kcache.dtype == vcache.dtype, "head_norm_kv: packed row")
+    else:
+        _require(kcache is None and vcache is None and first_v is None and qkv.shape[1] % hq == 0, "head_norm_kv: a row of queries")
+        nb, bs, dk = 0, 64, qkv.shape[1] // hq
+        dv = dk
+        _require(dk >= dim, "head_norm_kv: heads narrower than their width")
     ldf = 0
     if first_v is not None:
         _require(first_v.shape == (rows, hkv * dv) and first_v.stride(1) == 1 and first_v.dtype == qkv.dtype, "head_norm_kv: first values")
         ldf = first_v.stride(0)
-    for w in (q_weight, k_weight):
-        _require(w is None or (w.dtype == torch.float32 and w.numel() == dk and w.is_contiguous()), "head_norm_kv: norm weights")
+    for w, n in ((q_weight, hq), (k_weight, hkv)):
+        _require(w is None or (w.dtype == torch.float32 and w.numel() == dk * (n if whole else 1) and w.is_contiguous()), "head_norm_kv: norm weights")
     half = 0
     if cos_sin is not None:
         half = cos_sin.shape[1]
         _require(cos_sin.shape == (rows, half, 2) and cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and 2 * half <= dim,
                  "head_norm_kv: rotation table")
+    pos, coef, every = temp if temp is not None else (None, 0.0, 1)
+    _require(pos is None or (pos.dtype == torch.int32 and pos.numel() == rows), "head_norm_kv: int32 positions")
+    if whole or halves:
+        _require(first_v is None, "head_norm_kv: values are blended by the per-head form only")
+        rc = kernels().ff_row_norm_kv(ptr(qkv), ptr(slots), ptr(kcache), ptr(vcache), rows, hq, hkv, dim, dk, dv, bs, nb, ld, c_float(eps),
+                                      ptr(q_weight), ptr(k_weight), ptr(cos_sin), half, int(whole), int(halves), ptr(pos), c_float(coef), every,
+                                      int(qkv.dtype == torch.float32), ptr(status_tensor(qkv.device)), stream_ptr())
+        check(rc, "ff_row_norm_kv")
+        _count()
+        return
     rc = kernels().ff_head_norm_kv(ptr(qkv), ptr(slots), ptr(kcache), ptr(vcache), ptr(first_v), rows, hq, hkv, dim, dk, dv, bs, nb, ld,
-                                   ldf, c_float(eps), c_float(mix), ptr(q_weight), ptr(k_weight), ptr(cos_sin), half,
-                                   int(qkv.dtype == torch.float32), ptr(status_tensor(qkv.device)), stream_ptr())
+                                   ldf, c_float(eps), c_float(mix), ptr(q_weight), ptr(k_weight), ptr(cos_sin), half, ptr(pos),
+                                   c_float(coef), every, int(qkv.dtype == torch.float32), ptr(status_tensor(qkv.device)), stream_ptr())
     check(rc, "ff_head_norm_kv")
     _count()
 
@@ -522,10 +579,10 @@ def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0, out: torch.Ten
     rows, ld = _rows2d(gu)
     f = gu.shape[1] // 2
     if gu.dtype == torch.float32:          # 32-bit form: nothing in between is rounded
-        _require(mode in (0, 1), "silu_mul: the FP32 form is plain SwiGLU")
+        _require(mode in (0, 1, 2, 3), "silu_mul: the FP32 form has no clamped gate")
         if out is None:
             out = torch.empty(rows, f, dtype=torch.float32, device=gu.device)
-        check(kernels().ff_silu_mul_f32(ptr(gu), ptr(out), rows, f, ld, out.stride(0), int(interleaved), stream_ptr()), "ff_silu_mul_f32")
+        check(kernels().ff_silu_mul_f32(ptr(gu), ptr(out), rows, f, ld, out.stride(0), mode, int(interleaved), stream_ptr()), "ff_silu_mul_f32")
         _count()
         return out
     if out is None:
@@ -552,26 +609,32 @@ def attn_decode(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, blo
                 ctx_lens: torch.Tensor, hq: int, hkv: int, dim: int, scale: float, nq: int = 1,
                 tree_mask: torch.Tensor | None = None, max_ctx: int | None = None,
                 out: torch.Tensor | None = None, window: int = 0, sinks: torch.Tensor | None = None, chunk: int = 0,
-                vdim: int | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
+                vdim: int | None = None, gate: torch.Tensor | None = None, keep: int = 0, softcap: float = 0.0,
+                head_gate: torch.Tensor | None = None) -> torch.Tensor:
     """Decode / multi-row verify attention. ``q`` holds ``batch * nq`` rows (heads at columns
     ``h*dim``; it may be the packed QKV buffer). ``ctx_lens[b]`` counts the keys visible to the last
     of the ``nq`` rows. ``window > 0``: every row sees only its last ``window`` keys (local-attention
     layers; not together with a tree mask). ``sinks`` (float32 [hq]): learnable soft-max, one sink logit per head in the
     denominator. ``chunk > 0``: a row sees only keys of its own block of ``chunk`` positions. ``vdim``: width of the value
     heads (default ``dim``). ``gate`` ([rows, hq*vdim], a column slice of the packed rows): the result is multiplied by its
-    sigmoid before it is rounded. Heads up to 128 wide (multiples of 16) take the tensor-core kernel, other widths and
+    sigmoid before it is rounded. ``keep``: with a window, the sequence's first ``keep`` positions stay visible. ``softcap > 0``:
+    scores become ``softcap * tanh(score / softcap)``. ``head_gate`` ([rows, hq], a column slice): a head's result is multiplied by
+    its sigmoid. ``vcache`` may be the first ``vdim`` columns of the key rows (latent attention). Heads up to 128 wide (multiples of 16) take the tensor-core kernel, other widths and
     FP32 the SIMT kernel. Returns ``[batch*nq, hq*vdim]``."""
     batch = block_table.shape[0]
     vdim = vdim or dim
     _require(not (chunk > 0 and (window > 0 or tree_mask is not None)), "attn_decode: one kind of mask at a time")
     _require(not (window > 0 and tree_mask is not None), "attn_decode: window and tree mask are exclusive")
     _require(not (sinks is not None and tree_mask is not None), "attn_decode: sinks and tree mask are exclusive")
+    _require(not (softcap and (sinks is not None or tree_mask is not None)), "attn_decode: capped scores come without sinks and tree masks")
+    _require(gate is None or head_gate is None, "attn_decode: one gate")
+    keep = keep if window > 0 else 0
     if not _is_cuda(q):
         q_start = torch.arange(batch, dtype=torch.int32) * nq
         q_lens = torch.full((batch,), nq, dtype=torch.int32)
         tm = None if tree_mask is None else tree_mask.view(batch, nq)
         y = ref.attention_paged(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, scale, tm, window, sinks,
-                                chunk, vdim, gate)
+                                chunk, vdim, gate, keep, softcap, head_gate)
         if out is not None:
             out.copy_(y)
             return out
@@ -583,10 +646,11 @@ def attn_decode(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, blo
     nb = kcache.shape[0]
     if q.dtype == torch.float32 or max(dim, vdim) > 128:
         _require(tree_mask is None, "attn_decode: the SIMT kernel has no tree masks")
-        return _attn_simt(q, kcache, vcache, block_table, None, None, ctx_lens, nq, hq, hkv, dim, vdim, scale, window, chunk, gate, out, sinks)
+        return _attn_simt(q, kcache, vcache, block_table, None, None, ctx_lens, nq, hq, hkv, dim, vdim, scale, window, chunk, gate, out, sinks, keep,
+                          softcap, head_gate)
     _require(kcache.shape[2] == 64 and kcache.shape[3] == dim and vcache.shape[3] == vdim, "attn_decode: 64-token blocks of these heads")
     _require(dim % 16 == 0 and vdim % 16 == 0, "attn_decode: head widths must be multiples of 16")
-    general = chunk > 0 or gate is not None or dim != 128 or vdim != 128
+    general = chunk > 0 or gate is not None or dim != 128 or vdim != 128 or keep > 0 or softcap > 0 or head_gate is not None
     if max_ctx is None:
         max_ctx = block_table.shape[1] * 64
     lib = kernels()
@@ -609,8 +673,9 @@ def attn_decode(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, blo
                  "attn_decode: sinks float32 [hq]")
         rc = lib.ff_attn_decode_general(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(ctx_lens), ptr(out), ptr(part_o),
                                         ptr(part_ml), batch, hq, hkv, dim, vdim, nq, ldq, block_table.shape[1], nb, nsplit,
-                                        c_float(scale), max(window, 0), chunk, ptr(sinks), ptr(gate), _gate_ld(gate, rows, hq * vdim),
-                                        ptr(status_tensor(q.device)), stream_ptr())
+                                        c_float(scale), max(window, 0), chunk, ptr(sinks), ptr(gate if head_gate is None else head_gate),
+                                        _gate_ld(gate, rows, hq * vdim) or _head_gate_ld(head_gate, rows, hq), int(head_gate is not None), keep,
+                                        c_float(softcap), vcache.stride(2), ptr(status_tensor(q.device)), stream_ptr())
         counters = None
     elif sinks is not None:
         _require(sinks.dtype == torch.float32 and sinks.numel() == hq and sinks.is_contiguous(), "attn_decode: sinks float32 [hq]")
@@ -641,9 +706,17 @@ def _gate_ld(gate: torch.Tensor | None, rows: int, width: int) -> int:
     return gate.stride(0)
 
 
+def _head_gate_ld(gate: torch.Tensor | None, rows: int, heads: int) -> int:
+    if gate is None:
+        return 0
+    _require(gate.shape == (rows, heads) and gate.stride(1) == 1, "attention: the head gate has one column per head")
+    return gate.stride(0)
+
+
 def _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, nq: int, hq: int, hkv: int, dim: int, vdim: int,
                scale: float, window: int, chunk: int, gate: torch.Tensor | None, out: torch.Tensor | None,
-               sinks: torch.Tensor | None = None) -> torch.Tensor:
+               sinks: torch.Tensor | None = None, keep: int = 0, softcap: float = 0.0,
+               head_gate: torch.Tensor | None = None) -> torch.Tensor:
     """Paged attention of any head width, BF16 or FP32 (``csrc/attention_simt.cu``): one warp per query row and head.
     Rows come as ranges (``q_start`` / ``q_lens``) or, without them, ``nq`` per sequence."""
     rows, ldq = _rows2d(q)
@@ -654,8 +727,10 @@ def _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, nq: in
     _require(sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == hq and sinks.is_contiguous()), "attention: sinks float32 [hq]")
     rc = kernels().ff_attn_simt(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(out),
                                 block_table.shape[0], rows, nq, hq, hkv, dim, vdim, ldq, out.stride(0), kcache.shape[2],
-                                block_table.shape[1], kcache.shape[0], c_float(scale), window, chunk, ptr(gate),
-                                _gate_ld(gate, rows, hq * vdim), ptr(sinks), int(q.dtype == torch.float32), ptr(status_tensor(q.device)), stream_ptr())
+                                block_table.shape[1], kcache.shape[0], c_float(scale), window, chunk,
+                                ptr(gate if head_gate is None else head_gate), _gate_ld(gate, rows, hq * vdim) or _head_gate_ld(head_gate, rows, hq),
+                                ptr(sinks), int(q.dtype == torch.float32), ptr(status_tensor(q.device)), vcache.stride(2), keep, c_float(softcap),
+                                int(head_gate is not None), stream_ptr())
     check(rc, "ff_attn_simt")
     _count()
     return out
@@ -732,16 +807,20 @@ def attn_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
                  q_start: torch.Tensor, q_lens: torch.Tensor, ctx_lens: torch.Tensor, max_q_len: int, hq: int,
                  hkv: int, dim: int, scale: float, window: int = 0, out: torch.Tensor | None = None,
                  sinks: torch.Tensor | None = None, chunk: int = 0, vdim: int | None = None,
-                 gate: torch.Tensor | None = None) -> torch.Tensor:
+                 gate: torch.Tensor | None = None, keep: int = 0, softcap: float = 0.0,
+                 head_gate: torch.Tensor | None = None) -> torch.Tensor:
     """Causal chunked-prefill attention of packed query rows against the paged cache. ``window < 0`` makes it
     bidirectional: every query row sees all ``ctx_lens`` keys of its sequence (encoders, vision towers). ``sinks``
     (float32 [hq]): learnable soft-max, one sink logit per head in the denominator (tcgen05 kernel only). ``chunk``,
-    ``vdim`` and ``gate`` as in :func:`attn_decode`."""
+    ``vdim``, ``gate``, ``keep``, ``softcap`` and ``head_gate`` as in :func:`attn_decode`."""
     vdim = vdim or dim
+    keep = keep if window > 0 else 0
+    _require(not (softcap and sinks is not None), "attn_prefill: capped scores come without sinks")
+    _require(gate is None or head_gate is None, "attn_prefill: one gate")
     _require(not (chunk > 0 and window != 0), "attn_prefill: one kind of mask at a time")
     if not _is_cuda(q):
         y = ref.attention_paged(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, scale, None, window, sinks,
-                                chunk, vdim, gate)
+                                chunk, vdim, gate, keep, softcap, head_gate)
         if out is not None:
             out.copy_(y)
             return out
@@ -753,8 +832,8 @@ def attn_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
     nb = kcache.shape[0]
     if q.dtype == torch.float32 or max(dim, vdim) > 128:
         return _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, 1, hq, hkv, dim, vdim, scale, window, chunk, gate, out,
-                          sinks)
-    general = chunk > 0 or gate is not None or dim != 128 or vdim != 128
+                          sinks, keep, softcap, head_gate)
+    general = chunk > 0 or gate is not None or dim != 128 or vdim != 128 or keep > 0 or softcap > 0 or head_gate is not None
     _require(kcache.shape[2] == 64 and kcache.shape[3] == dim and vcache.shape[3] == vdim and dim % 16 == 0 and vdim % 16 == 0,
              "attn_prefill: 64-token blocks, head widths in multiples of 16")
     if general:
@@ -767,7 +846,8 @@ def attn_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
         rc = kernels().ff_attn_prefill_tc(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens),
                                           ptr(ctx_lens), ptr(out), batch, rows, max_q_len, hq, hkv, dim, vdim, ldq, out.stride(0),
                                           block_table.shape[1], nb, c_float(scale), window, chunk, ptr(sinks), ptr(gate),
-                                          _gate_ld(gate, rows, hq * vdim), ptr(status_tensor(q.device)), stream_ptr())
+                                          _gate_ld(gate, rows, hq * vdim), vcache.stride(2), keep, c_float(softcap), ptr(head_gate),
+                                          _head_gate_ld(head_gate, rows, hq), ptr(status_tensor(q.device)), stream_ptr())
         check(rc, "ff_attn_prefill_tc")
         _count()
         return out

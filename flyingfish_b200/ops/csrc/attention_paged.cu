@@ -81,11 +81,12 @@ struct RowState {
 //   lim0/lim1 : last visible key index for rows g and g+8 (inclusive); mask0/mask1: optional
 //               64-bit ancestor sets over keys >= tail_start (bit i = key tail_start+i visible)
 //   kd, vd    : 16-element steps of the key heads and pairs of 8-element columns of the value heads to run (8: 128 wide)
-template <int NT8>
+//   CAP       : scores become cap tanh(score / cap), in log2 units and up to a constant: cap_out / (1 + 2^(s cap_in))
+template <int NT8, bool CAP = false>
 __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[8][4], RowState& st, uint32_t sK, uint32_t sV,
                                           int key_off, int key0, int lim0, int lim1, bool use_mask, int tail_start,
                                           unsigned long long mask0, unsigned long long mask1, float scale_log2, int kd = 8,
-                                          int vd = 8) {
+                                          int vd = 8, float cap_in = 0.f, float cap_out = 0.f) {
   const int lane = threadIdx.x & 31, t = lane & 3;
   float s[NT8][4];
 #pragma unroll
@@ -118,7 +119,8 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[8][4], RowState& 
         const unsigned long long mk = (j < 2) ? mask0 : mask1;
         vis = vis && ((mk >> (key - tail_start)) & 1ull);
       }
-      const float v = vis ? s[i][j] * scale_log2 : NEG_BIG;
+      const float z = CAP ? __fdividef(cap_out, 1.0f + exp2f(fminf(s[i][j] * cap_in, 100.0f))) : s[i][j] * scale_log2;
+      const float v = vis ? z : NEG_BIG;
       s[i][j] = v;
       if (j < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
     }
@@ -188,17 +190,20 @@ __device__ __forceinline__ void load_q_frags(uint32_t (&qf)[8][4], const __nv_bf
 }
 
 // What a decode launch adds to plain causal 128-wide attention. A row at position p sees keys
-//   window > 0: p - window + 1 .. p          chunk > 0: the keys <= p of p's own block of `chunk` positions
-// dk / dv: widths of the key / value heads; gate: [rows, hq * dv] (row pitch ldg), the result is multiplied by its sigmoid.
+//   window > 0: p - window + 1 .. p and 0 .. keep - 1          chunk > 0: the keys <= p of p's own block of `chunk` positions
+// dk / dv: widths of the key / value heads; gate: [rows, hq * dv] (row pitch ldg), the result is multiplied by its sigmoid;
+// head_gate: [rows, hq] in its place, a factor per head. cap_in / cap_out: see warp_tile. ldv: pitch of the value cache's rows.
 struct DecodeForm {
   int window, chunk, dk, dv, ldg;
   const __nv_bfloat16* gate;
+  int keep = 0, ldv = 0, head_gate = 0;
+  float cap_in = 0.f, cap_out = 0.f;
 };
 __device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
   return window > 0 ? max(0, pos - window + 1) : (chunk > 0 ? max(0, pos) / chunk * chunk : 0);
 }
-__device__ __forceinline__ float gate_factor(const __nv_bfloat16* gate, int ldg, size_t row, int col) {
-  return gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-__bfloat162float(gate[row * ldg + col])));
+__device__ __forceinline__ float gate_factor(const __nv_bfloat16* gate, int ldg, size_t row, int head, int dv, int d, int head_gate) {
+  return gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-__bfloat162float(gate[row * ldg + (head_gate ? head : head * dv + d)])));
 }
 
 // ---------------------------------------------------------------------------------------
@@ -212,9 +217,10 @@ __device__ __forceinline__ float gate_factor(const __nv_bfloat16* gate, int ldg,
 // Measured on B200 (batch 64, context 1100, 32/8 heads): four 16-key warps 75.6 us, two 32-key warps
 // 80.3 us -- the wider warps issue fewer instructions per key but leave too few warps per SM.
 // ---------------------------------------------------------------------------------------
-// WIDE: heads are exactly 128 wide (widths known at compile time); EXTRA: the launch may have a block-local mask or a gate.
-// Plain causal / windowed attention keeps its own instance: the run-time widths cost it a tenth of its time.
-template <int NW, bool WIDE, bool EXTRA>
+// WIDE: heads are exactly 128 wide (widths known at compile time); EXTRA: the launch may have a block-local mask, kept first positions
+// or a gate; CAP: scores are capped. Plain causal / windowed attention keeps its own instance: the run-time widths cost it a tenth of
+// its time.
+template <int NW, bool WIDE, bool EXTRA, bool CAP>
 __global__ void __launch_bounds__(32 * NW)
 attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                    const __nv_bfloat16* __restrict__ q, const int* __restrict__ block_table,
@@ -245,8 +251,14 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   const bool k_hi = dk > 64, v_hi = dv > 64;           // heads up to 64 wide: the upper half of a tile is not loaded
   int pfirst = first_visible(ctx - nq, window, chunk) / PAGE;
   if (kv_start != nullptr) pfirst = max(pfirst, min(kv_start[b], ctx) / PAGE);
-  const int per = (pages - pfirst + nsplit - 1) / nsplit;
-  const int p0 = pfirst + split * per, p1 = min(pages, p0 + per);
+  // kept first positions in pages before the window's first: pages are counted through, the kept ones in front
+  const int keep = EXTRA ? f.keep : 0;
+  const int nkeep = EXTRA ? min(pfirst, (keep + PAGE - 1) / PAGE) : 0;
+  const int skip = pfirst - nkeep;                     // pages between the kept ones and the window's first
+  auto page_of = [&](int p) { return EXTRA && p >= nkeep ? p + skip : p; };
+  const int first = EXTRA ? 0 : pfirst, last = EXTRA ? pages - skip : pages;
+  const int per = (last - first + nsplit - 1) / nsplit;
+  const int p0 = first + split * per, p1 = min(last, p0 + per);
   const int rows_total = nq * G;
   const int rows_used = min(16, rows_total - rt * 16);
 
@@ -275,7 +287,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   // the block ids of this CTA's pages, fetched once by all threads: the page loop then issues its
   // TMA loads without a dependent global load in front of each
   __shared__ int sblk[128];
-  for (int i = threadIdx.x; i < 128 && p0 + i < p1; i += 32 * NW) sblk[i] = block_table[(size_t)b * max_blocks + p0 + i];
+  for (int i = threadIdx.x; i < 128 && p0 + i < p1; i += 32 * NW) sblk[i] = block_table[(size_t)b * max_blocks + page_of(p0 + i)];
   if (threadIdx.x == 0) {
     for (int i = 0; i < DEC_STAGES; ++i) mbar_init(&full_bar[i], 1);
     abort_flag = 0;
@@ -283,7 +295,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   }
   __syncthreads();
   auto issue = [&](int page_idx, int buf) {
-    int blk = (page_idx - p0 < 128) ? sblk[page_idx - p0] : block_table[(size_t)b * max_blocks + page_idx];
+    int blk = (page_idx - p0 < 128) ? sblk[page_idx - p0] : block_table[(size_t)b * max_blocks + page_of(page_idx)];
     if (blk < 0 || blk >= num_blocks) { bad = true; blk = 0; }
     const int row = (blk * hkv + kvh) * PAGE;
     uint8_t* sk = smem + buf * STAGE_BYTES;
@@ -304,7 +316,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     if (threadIdx.x == 0 && p + DEC_STAGES - 1 < p1) issue(p + DEC_STAGES - 1, (it + DEC_STAGES - 1) % DEC_STAGES);
     if (ok && !mbar_wait(&full_bar[buf], ph, &abort_flag, status, KID_ATTN_DECODE, 1)) ok = false;
     constexpr int KPW = PAGE / NW;                     // keys per warp
-    const int key0 = p * PAGE + warp * KPW;
+    const int key0 = page_of(p) * PAGE + warp * KPW;
     const uint32_t sk = smem_u32(smem + buf * STAGE_BYTES);
     if (ok && key0 < ctx) {
       bool um = tree_mask != nullptr;
@@ -315,9 +327,13 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
         um = true; ts = key0;
         a0 = lo0 <= 0 ? ~0ull : (lo0 >= 64 ? 0ull : (~0ull << lo0));
         a1 = lo1 <= 0 ? ~0ull : (lo1 >= 64 ? 0ull : (~0ull << lo1));
+        if (EXTRA && keep > key0) {                    // this warp's keys below `keep` stay visible
+          const unsigned long long kept = keep - key0 >= 64 ? ~0ull : ~(~0ull << (keep - key0));
+          a0 |= kept; a1 |= kept;
+        }
       }
-      warp_tile<KPW / 8>(qf, st, sk, sk + PAGE * HD * 2, warp * KPW, key0, lim[0], lim[1], um, ts, a0, a1, scale_log2,
-                         kd, vd);
+      warp_tile<KPW / 8, CAP>(qf, st, sk, sk + PAGE * HD * 2, warp * KPW, key0, lim[0], lim[1], um, ts, a0, a1, scale_log2,
+                              kd, vd, f.cap_in, f.cap_out);
     }
     __syncthreads();
   }
@@ -356,7 +372,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
       if (nsplit == 1 && pstride == 0) {
         // learnable soft-max: the head's sink logit enters the denominator only
         const float Ls = sinks ? L + exp2f(sinks[hh] * 1.4426950408889634f - M) : L;
-        const float gf = gate_factor(gate, f.ldg, (size_t)(b * nq + qi), hh * dv + d);
+        const float gf = gate_factor(gate, f.ldg, (size_t)(b * nq + qi), hh, dv, d, f.head_gate);
         out[((size_t)(b * nq + qi) * hq + hh) * dv + d] = __float2bfloat16(Ls > 0.f ? acc / Ls * gf : 0.f);
       } else {
         const size_t pr = ((size_t)b * (pstride ? pstride : nsplit) + split) * (nq * hq) + (size_t)qi * hq + hh;
@@ -396,7 +412,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
             acc += __ldcg(&part_o[pr * HD + d]) * sc;
           }
           if (sinks) L += exp2f(sinks[hh] * 1.4426950408889634f - M);
-          const float gf = gate_factor(gate, f.ldg, (size_t)(b * nq + qi), hh * dv + d);
+          const float gf = gate_factor(gate, f.ldg, (size_t)(b * nq + qi), hh, dv, d, f.head_gate);
           out[((size_t)(b * nq + qi) * hq + hh) * dv + d] = __float2bfloat16(L > 0.f ? acc / L * gf : 0.f);
         }
       }
@@ -408,7 +424,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 __global__ void __launch_bounds__(128)
 attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out,
                   int rows_per_seq, int nsplit, const float* __restrict__ sinks, int hq, int dv, const __nv_bfloat16* __restrict__ gate,
-                  int ldg) {
+                  int ldg, int head_gate) {
   pdl_trigger();
   pdl_wait();
   const int row = blockIdx.x, b = row / rows_per_seq, r = row % rows_per_seq, d = threadIdx.x;
@@ -423,7 +439,7 @@ attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ pa
     acc += part_o[pr * HD + d] * sc;
   }
   if (sinks) L += exp2f(sinks[r % hq] * 1.4426950408889634f - M);
-  const float gf = gate_factor(gate, ldg, (size_t)(row / hq), (row % hq) * dv + d);
+  const float gf = gate_factor(gate, ldg, (size_t)(row / hq), row % hq, dv, d, head_gate);
   out[(size_t)row * dv + d] = __float2bfloat16(L > 0.f ? acc / L * gf : 0.f);
 }
 
@@ -560,8 +576,12 @@ static int attn_decode_launch(const void* q, const void* kcache, const void* vca
   if (ldq % 8 || nsplit < 1) return FF_HOST_BAD_ALIGN;
   if (nsplit > 1 && (!part_o || !part_ml)) return FF_HOST_BAD_SHAPE;
   constexpr int NW = DEC_WARPS;
-  const bool wide = f.dk == HD && f.dv == HD, extra = f.chunk > 0 || f.gate != nullptr;
-  auto kern = !wide ? attn_decode_kernel<NW, false, true> : extra ? attn_decode_kernel<NW, true, true> : attn_decode_kernel<NW, true, false>;
+  const int ldv = f.ldv > 0 ? f.ldv : f.dv;
+  if (ldv < f.dv || ldv % 8 || f.keep < 0 || (f.cap_in != 0.f && (sinks != nullptr || tree_mask != nullptr))) return FF_HOST_BAD_SHAPE;
+  const bool wide = f.dk == HD && f.dv == HD, extra = f.chunk > 0 || f.gate != nullptr || f.keep > 0, cap = f.cap_in != 0.f;
+  if (extra && kv_start != nullptr) return FF_HOST_UNSUPPORTED;
+  auto kern = cap ? (wide ? (extra ? attn_decode_kernel<NW, true, true, true> : attn_decode_kernel<NW, true, false, true>) : attn_decode_kernel<NW, false, true, true>)
+                  : (wide ? (extra ? attn_decode_kernel<NW, true, true, false> : attn_decode_kernel<NW, true, false, false>) : attn_decode_kernel<NW, false, true, false>);
   if (int r = opt_in_smem(kern, DEC_SMEM)) return r;
   const float scale_log2 = scale * 1.4426950408889634f;
   const int row_tiles = (nq * (hq / hkv) + 15) / 16;
@@ -570,14 +590,14 @@ static int attn_decode_launch(const void* q, const void* kcache, const void* vca
   CUtensorMap tmK, tmV;
   const uint64_t cache_rows = (uint64_t)num_blocks * hkv * PAGE;
   if (int r = make_tmap_2d(&tmK, kcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, f.dk, cache_rows, f.dk * 2, 64, PAGE)) return r;
-  if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, f.dv, cache_rows, f.dv * 2, 64, PAGE)) return r;
+  if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, f.dv, cache_rows, (uint64_t)ldv * 2, 64, PAGE)) return r;
   if (int lr_ = launch_pdl(kern, dim3(grid), dim3(32 * NW), DEC_SMEM, s, 0, tmK, tmV, (const __nv_bfloat16*)q,
       block_table, ctx_lens, tree_mask, (__nv_bfloat16*)out, part_o, part_ml, hq, hkv, nq,
       ldq, max_blocks, num_blocks, nsplit, scale_log2, status, split_counters, f, kv_start, pstride, sinks)) return lr_;
   if (int r = launch_result()) return r;
   if (pstride != 0) return 0;                      // partials only: the caller merges after the other kernel has added its own
   if (nsplit > 1 && split_counters == nullptr) {
-    if (int lr_ = launch_pdl(attn_merge_kernel, dim3(batch * nq * hq), dim3(128), 0, s, 0, part_o, part_ml, (__nv_bfloat16*)out, nq * hq, nsplit, sinks, hq, f.dv, f.gate, f.ldg)) return lr_;
+    if (int lr_ = launch_pdl(attn_merge_kernel, dim3(batch * nq * hq), dim3(128), 0, s, 0, part_o, part_ml, (__nv_bfloat16*)out, nq * hq, nsplit, sinks, hq, f.dv, f.gate, f.ldg, f.head_gate)) return lr_;
     return launch_result();
   }
   return 0;
@@ -611,7 +631,7 @@ FF_EXPORT int ff_attn_merge(const float* part_o, const float* part_ml, void* out
   if (batch <= 0 || rows_per_seq <= 0 || nsplit < 1) return FF_HOST_BAD_SHAPE;
   if (int lr_ = launch_pdl(attn_merge_kernel, dim3(batch * rows_per_seq), dim3(128), 0, s, 0, part_o, part_ml,
                            (__nv_bfloat16*)out, rows_per_seq, nsplit, (const float*)nullptr, rows_per_seq, HD,
-                           (const __nv_bfloat16*)nullptr, 0)) return lr_;
+                           (const __nv_bfloat16*)nullptr, 0, 0)) return lr_;
   return launch_result();
 }
 
@@ -629,15 +649,19 @@ FF_EXPORT int ff_attn_decode_sink(const void* q, const void* kcache, const void*
 
 // Decode attention in its general form: key heads of dk and value heads of dv elements (multiples of 16, at most 128; the
 // cache rows and the head pitch of q are dk wide, output heads dv wide), optional window or block-local mask (chunk), sinks
-// and output gate. The partials of a split launch keep 128 floats per row.
+// and output gate (head_gate: one factor per head). keep: with a window, the first `keep` positions stay visible; softcap > 0: scores
+// become softcap tanh(score / softcap); ldv: pitch of the value cache's rows. The partials of a split launch keep 128 floats per row.
 FF_EXPORT int ff_attn_decode_general(const void* q, const void* kcache, const void* vcache, const int* block_table,
                                      const int* ctx_lens, void* out, float* part_o, float* part_ml, int batch, int hq, int hkv, int dk,
                                      int dv, int nq, int ldq, int max_blocks, int num_blocks, int nsplit, float scale, int window,
-                                     int chunk, const float* sinks, const void* gate, int ldg, int* status, cudaStream_t s) {
-  if (window < 0 || chunk < 0) return FF_HOST_BAD_SHAPE;
+                                     int chunk, const float* sinks, const void* gate, int ldg, int head_gate, int keep, float softcap,
+                                     int ldv, int* status, cudaStream_t s) {
+  if (window < 0 || chunk < 0 || !(softcap >= 0.f)) return FF_HOST_BAD_SHAPE;
+  DecodeForm f{window, chunk, dk, dv, ldg, (const __nv_bfloat16*)gate};
+  f.keep = window > 0 ? keep : 0; f.ldv = ldv; f.head_gate = head_gate;
+  if (softcap > 0.f) { f.cap_in = 2.0f * 1.4426950408889634f * scale / softcap; f.cap_out = -2.0f * 1.4426950408889634f * softcap; }
   return attn_decode_launch(q, kcache, vcache, block_table, ctx_lens, nullptr, out, part_o, part_ml, batch, hq, hkv, HD, nq, ldq, max_blocks,
-                            num_blocks, nsplit, scale, nullptr, status, s,
-                            DecodeForm{window, chunk, dk, dv, ldg, (const __nv_bfloat16*)gate}, nullptr, 0, sinks);
+                            num_blocks, nsplit, scale, nullptr, status, s, f, nullptr, 0, sinks);
 }
 
 // Decode attention of a local-attention layer: every query sees its last `window` keys.

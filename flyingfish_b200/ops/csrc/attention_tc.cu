@@ -1,5 +1,6 @@
 // Prefill attention on 5th-generation tensor cores: paged KV, heads of up to 128 elements, GQA, causal / sliding-window /
-// block-local / bidirectional masks, optional output gate, chunked prefill (query rows are the last q_len positions of a context of ctx_len).
+// block-local / bidirectional masks, a sliding window that keeps the first positions, soft-capped scores, optional output gate (per
+// element or per head), chunked prefill (query rows are the last q_len positions of a context of ctx_len).
 //
 // One CTA per (sequence, query head, tile of 128 query rows). Both contractions run as tcgen05.mma with
 // FP32 accumulators in tensor memory:
@@ -367,7 +368,16 @@ constexpr int TC2_SMEM = TC_Q_BYTES + 4 * T2_KV_BYTES + 1024;      // 97 KiB
 struct PrefillForm {
   int window, chunk, causal, dk, dv;
   int gated;                       // the result is multiplied by the sigmoid of a [rows, hq * dv] gate (tensor map tmG)
+  int keep;                        // with a window: the first `keep` positions stay visible
+  float cap_in, cap_out;           // CAP: score s becomes cap tanh(s / cap); cap_in = 2 log2(e) scale / cap, cap_out = -2 log2(e) cap
+  const __nv_bfloat16* head_gate;  // the result of head h is multiplied by the sigmoid of head_gate[row * ldhg + h]
+  int ldhg;
 };
+
+// cap tanh(s / cap) up to the constant cap, which soft-max does not see, in log2 units: -2 cap / (1 + e^(2 s / cap))
+__device__ __forceinline__ float capped_log2(float s, float cap_in, float cap_out) {
+  return __fdividef(cap_out, 1.0f + ex2_approx(fminf(s * cap_in, 100.0f)));
+}
 
 // o * inv, times the sigmoid of the gate where there is one (`gate`: the row of a swizzled gate tile in shared memory, `sw` =
 // row % 8, `chunk` its first 16-byte chunk); 16 columns, two 16-byte stores
@@ -399,9 +409,9 @@ struct alignas(8) Tc2Bars {
   float xmax[2][TC_BM];
 };
 
-// WIDE: heads are exactly 128 wide; EXTRA: the launch may have a block-local mask or a gate (plain launches keep an instance
-// with neither).
-template <int SPLIT, bool WIDE, bool EXTRA>
+// WIDE: heads are exactly 128 wide; EXTRA: the launch may have a block-local mask, kept first positions or a gate (plain launches keep
+// an instance with none of them); CAP: scores are capped.
+template <int SPLIT, bool WIDE, bool EXTRA, bool CAP>
 __global__ void __launch_bounds__(64 + 128 * SPLIT, 2)
 attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                         const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmG, const int* __restrict__ block_table,
@@ -430,7 +440,11 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   const int last_key = causal ? past + r0 + real - 1 : ctx - 1;
   const int first_key = first_visible(past + r0);
   const int t0 = first_key / T2_BN, t1 = last_key / T2_BN + 1;
-  const int ntiles = t1 - t0;
+  // kept first positions in pages before the window's first: those pages come as the first tiles
+  const int keep = EXTRA ? f.keep : 0;
+  const int tkeep = EXTRA ? min(t0, (keep + T2_BN - 1) / T2_BN) : 0;
+  const int ntiles = t1 - t0 + tkeep;
+  auto tile_page = [&](int j) { return EXTRA && j < tkeep ? j : t0 + j - tkeep; };
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
   if (threadIdx.x == 0) {
@@ -459,7 +473,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       bool ok = true, bad = false;
       const int nblk = (ctx + TC_PAGE - 1) / TC_PAGE;
       auto tile_row = [&](int j) -> int {
-        int page = t0 + j;
+        int page = tile_page(j);
         if (page >= nblk) page = nblk - 1;                   // past the context: any valid page, its keys are masked
         int blk = block_table[(size_t)b * max_blocks + page];
         if (blk < 0 || blk >= num_blocks) { bad = true; blk = 0; }
@@ -572,21 +586,26 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 #pragma unroll
           for (int i = 0; i < HB; ++i) sv[i] = __uint_as_float(r[i]);
         }
-        const int k0 = (t0 + j) * T2_BN + hf * HB;
+        const int tile0 = tile_page(j) * T2_BN, k0 = tile0 + hf * HB;
+        if (CAP) {
+#pragma unroll
+          for (int i = 0; i < HB; ++i) sv[i] = capped_log2(sv[i], f.cap_in, f.cap_out);
+        }
         float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-        if ((t0 + j) * T2_BN >= tile_lo_max && (t0 + j) * T2_BN + T2_BN - 1 <= tile_hi_min) {
+        if ((tile0 >= tile_lo_max || (EXTRA && tile0 + T2_BN <= keep)) && tile0 + T2_BN - 1 <= tile_hi_min) {
 #pragma unroll
           for (int i = 0; i < HB; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
         } else {
 #pragma unroll
           for (int i = 0; i < HB; ++i) {
             const int key = k0 + i;
-            const float t = (key >= lo && key <= hi) ? sv[i] : -INFINITY;
+            const float t = ((key >= lo || (EXTRA && key < keep)) && key <= hi) ? sv[i] : -INFINITY;
             sv[i] = t;
             mx4[i & 3] = fmaxf(mx4[i & 3], t);
           }
         }
-        mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
+        mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+        if (!CAP) mx *= scale_log2;
       }
       if (SPLIT == 2) {
         // after this barrier both warps of the pair hold their S columns in registers: P may overwrite S
@@ -629,8 +648,8 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
           uint32_t pk[16];
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
-            const float p0 = ex2_approx(fmaf(sv[2 * (c + i)], scale_log2, -mr));
-            const float p1 = ex2_approx(fmaf(sv[2 * (c + i) + 1], scale_log2, -mr));
+            const float p0 = ex2_approx(CAP ? sv[2 * (c + i)] - mr : fmaf(sv[2 * (c + i)], scale_log2, -mr));
+            const float p1 = ex2_approx(CAP ? sv[2 * (c + i) + 1] - mr : fmaf(sv[2 * (c + i) + 1], scale_log2, -mr));
             pk[i] = pack_bf16x2(p0, p1);
             ls4[i & 3] += p0 + p1;
           }
@@ -658,7 +677,9 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     if (ok) {
       tc_fence_after();
       if (sinks != nullptr) l_sum += (m_ref == -INFINITY) ? 1.f : exp2f(sinks[h] * 1.4426950408889634f - m_ref);
-      const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+      float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+      if (EXTRA && f.head_gate != nullptr && live)
+        inv = __fdividef(inv, 1.0f + __expf(-__bfloat162float(f.head_gate[(size_t)(qs + r0 + row) * f.ldhg + h])));
       __nv_bfloat16* orow = out + (size_t)(qs + r0 + row) * ldo + (size_t)h * dv + hf * (TC_HD / SPLIT);
 #pragma unroll
       for (int c = 0; c < TC_HD / SPLIT; c += 16) {
@@ -686,12 +707,16 @@ using namespace ff;
 // Same contract as ff_attn_prefill (attention_paged.cu). q: packed rows [rows, ldq] with head h at columns h*dk;
 // out rows 16-byte aligned (ldo % 8 == 0). window > 0 sliding, 0 causal, < 0 bidirectional; chunk > 0: a query sees the keys
 // of its own block of `chunk` positions that are not after it. dk / dv: widths of the key and value heads (multiples of 16,
-// at most 128). gate: optional [rows, hq * dv] with row pitch ldg, 16-byte aligned.
+// at most 128); ldv: pitch of the value cache's rows (dv, or the key rows' width where the values are their first columns). gate:
+// optional [rows, hq * dv] with row pitch ldg, 16-byte aligned. keep: with a window, the first `keep` positions stay visible.
+// softcap > 0: scores become softcap tanh(score / softcap). head_gate: optional [rows, hq] with row pitch ldhg.
 FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* vcache, const int* block_table,
                                  const int* q_start, const int* q_lens, const int* ctx_lens, void* out, int batch,
                                  int total_rows, int max_q_len, int hq, int hkv, int dk, int dv, int ldq, int ldo,
                                  int max_blocks, int num_blocks, float scale, int window, int chunk, const float* sinks,
-                                 const void* gate, int ldg, int* status, cudaStream_t s) {
+                                 const void* gate, int ldg, int ldv, int keep, float softcap, const void* head_gate, int ldhg, int* status,
+                                 cudaStream_t s) {
+  if (ldv < dv || ldv % 8 || keep < 0 || !(softcap >= 0.f) || (softcap > 0.f && sinks != nullptr)) return FF_HOST_BAD_SHAPE;
   if (batch <= 0 || max_q_len <= 0 || hq <= 0 || hkv <= 0 || hq % hkv || total_rows <= 0) return FF_HOST_BAD_SHAPE;
   if (dk < 16 || dk > TC_HD || dk % 16 || dv < 16 || dv > TC_HD || dv % 16 || chunk < 0 || !(scale > 0.f)) return FF_HOST_BAD_SHAPE;
   if (chunk > 0 && window != 0) return FF_HOST_UNSUPPORTED;
@@ -702,10 +727,11 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
                            (uint64_t)ldq * 2, 64, TC_BM)) return r;
   const uint64_t cache_rows = (uint64_t)num_blocks * hkv * TC_PAGE;
   if (int r = make_tmap_2d(&tmK, kcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dk, cache_rows, dk * 2, 64, TC_PAGE)) return r;
-  if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dv, cache_rows, dv * 2, 64, TC_PAGE)) return r;
+  if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dv, cache_rows, (uint64_t)ldv * 2, 64, TC_PAGE)) return r;
   const float scale_log2 = scale * 1.4426950408889634f;
   dim3 grid((max_q_len + TC_BM - 1) / TC_BM, hq, batch);
-  const PrefillForm f = {window < 0 ? 0 : window, chunk, window < 0 ? 0 : 1, dk, dv, gate != nullptr ? 1 : 0};
+  const PrefillForm f = {window < 0 ? 0 : window, chunk, window < 0 ? 0 : 1, dk, dv, gate != nullptr ? 1 : 0, window > 0 ? keep : 0,
+                         softcap > 0.f ? 2.0f * scale_log2 / softcap : 0.f, -2.0f * 1.4426950408889634f * softcap, (const __nv_bfloat16*)head_gate, ldhg};
   CUtensorMap tmG = tmQ;
   if (gate != nullptr)
     if (int r = make_tmap_2d(&tmG, gate, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)hq * dv, (uint64_t)total_rows, (uint64_t)ldg * 2, 64, TC_BM)) return r;
@@ -713,7 +739,8 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
   // only); the default is the two-CTAs-per-SM kernel
   static int two = -1;
   if (two < 0) { const char* e = getenv("FF_ATTN_PREFILL_CTAS"); two = (e != nullptr && e[0] == '1') ? 0 : TC_TWO_CTAS_DEFAULT; }
-  if (two || chunk > 0 || gate != nullptr || dk != TC_HD || dv != TC_HD) {
+  const bool wide = dk == TC_HD && dv == TC_HD, extra = chunk > 0 || gate != nullptr || f.keep > 0 || head_gate != nullptr, cap = softcap > 0.f;
+  if (two || extra || cap || !wide) {
     // FF_ATTN_PREFILL_SPLIT = 2: two softmax warps per lane quadrant (64 columns each) instead of one
     static int split = -1;
     if (split < 0) { const char* e = getenv("FF_ATTN_PREFILL_SPLIT"); split = (e != nullptr && (e[0] == '1' || e[0] == '2')) ? e[0] - '0' : TC2_SPLIT_DEFAULT; }
@@ -723,10 +750,10 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
                                            max_blocks, num_blocks, scale_log2, f, status, sinks);
       return launch_result();
     };
-    const bool wide = dk == TC_HD && dv == TC_HD, extra = chunk > 0 || gate != nullptr;
-    if (!wide) return go(attn_prefill_tc2_kernel<1, false, true>, 192);
-    if (split == 2) return extra ? go(attn_prefill_tc2_kernel<2, true, true>, 320) : go(attn_prefill_tc2_kernel<2, true, false>, 320);
-    return extra ? go(attn_prefill_tc2_kernel<1, true, true>, 192) : go(attn_prefill_tc2_kernel<1, true, false>, 192);
+    if (!wide) return cap ? go(attn_prefill_tc2_kernel<1, false, true, true>, 192) : go(attn_prefill_tc2_kernel<1, false, true, false>, 192);
+    if (cap) return extra ? go(attn_prefill_tc2_kernel<1, true, true, true>, 192) : go(attn_prefill_tc2_kernel<1, true, false, true>, 192);
+    if (split == 2) return extra ? go(attn_prefill_tc2_kernel<2, true, true, false>, 320) : go(attn_prefill_tc2_kernel<2, true, false, false>, 320);
+    return extra ? go(attn_prefill_tc2_kernel<1, true, true, false>, 192) : go(attn_prefill_tc2_kernel<1, true, false, false>, 192);
   }
   if (int r = opt_in_smem(attn_prefill_tc_kernel, TC_SMEM)) return r;
   attn_prefill_tc_kernel<<<grid, 320, TC_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens,

@@ -52,6 +52,9 @@ struct GroupArgs {
   const int* seg_off;                 // nullptr: dense problem
   const int* counts;
   int E;
+  // dense problem with heads > 1: block-diagonal, head h multiplies columns h * a_cols.. of A with rows h * N.. of B and writes columns
+  // h * c_cols.. of the result
+  int heads, a_cols, c_cols;
 };
 
 struct TileWalk { int e = 0, base = 0; };
@@ -59,11 +62,14 @@ struct TileWalk { int e = 0, base = 0; };
 // Operand rows of linear tile t of this CTA's loop (t grows monotonically); false when the problem is done.
 __device__ __forceinline__ bool next_tile(const GroupArgs& g, TileWalk& w, int t, int tiles_m, int tiles_n,
                                           int M, int N, int BN, int& tm, int& tn, int& a_row0, int& b_row0,
-                                          int& row_end) {
+                                          int& row_end, int& head) {
+  head = 0;
   if (g.seg_off == nullptr) {
-    if (t >= tiles_m * tiles_n) return false;
-    tile_coords(t, tiles_m, tiles_n, tm, tn);
-    a_row0 = tm * BM; b_row0 = tn * BN; row_end = M;
+    const int all_n = g.heads > 1 ? tiles_n * g.heads : tiles_n;
+    if (t >= tiles_m * all_n) return false;
+    tile_coords(t, tiles_m, all_n, tm, tn);
+    if (g.heads > 1) { head = tn / tiles_n; tn -= head * tiles_n; }
+    a_row0 = tm * BM; b_row0 = head * N + tn * BN; row_end = M;
     return true;
   }
   while (w.e < g.E) {
@@ -118,9 +124,14 @@ __device__ __forceinline__ int comm_tm(int tm, int tiles_per_rank, int rank, int
   return ((rank + j) % world) * tiles_per_rank + r;
 }
 
-// Optional tail of the plain BF16 store (epi 0): bias per output column, then act 1 = square of the positive part. Both work
-// on the FP32 accumulator; the result is rounded once.
-struct LinTail { const __nv_bfloat16* bias; int act; };
+// Optional tail of the plain BF16 store (epi 0): bias per output column, then act 1 = square of the positive part or
+// 3 = tanh-GELU, then a factor per element (row mul_rows[row] of a table). All on the FP32 accumulator; the result is rounded once.
+// gate: activation of the gated epilogue (epi 1), 0 SiLU with the reference's roundings, 3 tanh-GELU with one rounding.
+struct LinTail {
+  const __nv_bfloat16* bias; int act;
+  const __nv_bfloat16* mul; const int* mul_rows; int ldm, mul_table;
+  int gate;
+};
 
 constexpr int RS_STG_PITCH = 144, RS_STG_BYTES = 32 * RS_STG_PITCH;   // COMM 2 epilogue staging, per warp
 constexpr int COMM_PARTS = 4;       // a 128-row block is pushed (COMM 1) / reduced (COMM 2) in this many pieces
@@ -165,8 +176,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       bool ok = true;
       TileWalk walk;
       for (int t = blockIdx.x; ok; t += gridDim.x) {
-        int tm, tn, a_row0, b_row0, row_end;
-        if (!next_tile(ga, walk, t, tiles_m, tiles_n, M, N, BN, tm, tn, a_row0, b_row0, row_end)) break;
+        int tm, tn, a_row0, b_row0, row_end, head;
+        if (!next_tile(ga, walk, t, tiles_m, tiles_n, M, N, BN, tm, tn, a_row0, b_row0, row_end, head)) break;
         if (COMM) { tm = comm_tm<COMM>(tm, tiles_per_rank, ca.ar.rank, ca.ar.world); a_row0 = tm * BM; }
         const int src = tm / tiles_per_rank, rb = tm - src * tiles_per_rank;
         if (COMM == 1 && src != ca.ar.rank) {
@@ -183,7 +194,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           uint8_t* sa = smem + s * STAGE_BYTES;
           if (COMM == 1 && src == ca.ar.rank) tma_load_2d(sa, &tmX, &bars.full[s], kb * BK, rb * BM);
           else if (COMM == 1) tma_load_3d(sa, parity ? &tmA1 : &tmA, &bars.full[s], kb * BK, rb * BM, src);
-          else tma_load_2d(sa, &tmA, &bars.full[s], kb * BK, a_row0);
+          else tma_load_2d(sa, &tmA, &bars.full[s], head * ga.a_cols + kb * BK, a_row0);
           tma_load_2d(sa + A_BYTES, &tmB, &bars.full[s], kb * BK, b_row0);
         }
       }
@@ -195,8 +206,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       bool ok = true;
       TileWalk walk;
       for (int t = blockIdx.x; ok; t += gridDim.x, ++tile_it) {
-        int tm_, tn_, a_, b_, re_;
-        if (!next_tile(ga, walk, t, tiles_m, tiles_n, M, N, BN, tm_, tn_, a_, b_, re_)) break;
+        int tm_, tn_, a_, b_, re_, hd_;
+        if (!next_tile(ga, walk, t, tiles_m, tiles_n, M, N, BN, tm_, tn_, a_, b_, re_, hd_)) break;
         const int acc = tile_it & 1; const uint32_t aph = (tile_it >> 1) & 1;
         if (!mbar_wait(&bars.tmem_empty[acc], aph ^ 1, abort_flag, status, KID_GEMM_BF16, 2)) { ok = false; break; }
         tc_fence_after();
@@ -226,8 +237,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     bool ok = true;
     TileWalk walk;
     for (int t = blockIdx.x; ok; t += gridDim.x, ++tile_it) {
-      int tm, tn, a_row0, b_row0, row_end;
-      if (!next_tile(ga, walk, t, tiles_m, tiles_n, M, N, BN, tm, tn, a_row0, b_row0, row_end)) break;
+      int tm, tn, a_row0, b_row0, row_end, head;
+      if (!next_tile(ga, walk, t, tiles_m, tiles_n, M, N, BN, tm, tn, a_row0, b_row0, row_end, head)) break;
       if (COMM) { tm = comm_tm<COMM>(tm, tiles_per_rank, ca.ar.rank, ca.ar.world); a_row0 = tm * BM; }
       const int acc = tile_it & 1; const uint32_t aph = (tile_it >> 1) & 1;
       if (!mbar_wait(&bars.tmem_full[acc], aph, abort_flag, status, KID_GEMM_BF16, 4)) { ok = false; break; }
@@ -251,6 +262,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             for (int j = 0; j < 8; ++j) {
               const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
               const float u0 = __uint_as_float(u[2 * j]), u1 = __uint_as_float(u[2 * j + 1]);
+              if (COMM == 0 && tail.gate == 3) { o[j] = pack_bf16x2(gelu_tanh_f(g0) * u0, gelu_tanh_f(g1) * u1); continue; }
               // rounding policy "mode 0" of the reference's silu_mul (kernels/act.cu:220-262):
               // gate and up are BF16 values, silu rounded to BF16, product rounded again.
               const float a0 = __bfloat162float(__float2bfloat16(silu_f(__bfloat162float(__float2bfloat16(g0)))));
@@ -289,7 +301,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           }
         }
       } else {
-        __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(Cout) + (size_t)row * ldc + (size_t)tn * BN;
+        __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(Cout) + (size_t)row * ldc + (size_t)head * ga.c_cols + (size_t)tn * BN;
         if (COMM == 2) {
           // the rows of this tile belong to rank `owner`: they go into its arena slot for source = me,
           // 64 columns at a time through a warp-private staging tile
@@ -359,6 +371,33 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           if (COMM == 0 && tail.act == 1) {
 #pragma unroll
             for (int j = 0; j < 32; ++j) { const float v = fmaxf(__uint_as_float(r[j]), 0.f); r[j] = __float_as_uint(v * v); }
+          }
+          if (COMM == 0 && tail.act == 3) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(gelu_tanh_f(__uint_as_float(r[j])));
+          }
+          if (COMM == 0 && tail.mul != nullptr && row < row_end) {
+            int mr = tail.mul_rows[row];
+            if (mr < 0 || mr >= tail.mul_table) mr = 0;          // reported where the id is first read (embedding)
+            const int col = tn * BN + c;
+            const __nv_bfloat16* f = tail.mul + (size_t)mr * tail.ldm + col;
+            if (col + 32 <= N) {
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                const uint4 fv = __ldg(reinterpret_cast<const uint4*>(f) + j);
+                const uint32_t fw[4] = {fv.x, fv.y, fv.z, fv.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                  const float2 m = unpack_bf16x2(fw[i]);
+                  r[8 * j + 2 * i] = __float_as_uint(__uint_as_float(r[8 * j + 2 * i]) * m.x);
+                  r[8 * j + 2 * i + 1] = __float_as_uint(__uint_as_float(r[8 * j + 2 * i + 1]) * m.y);
+                }
+              }
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (col + j < N) r[j] = __float_as_uint(__uint_as_float(r[j]) * __bfloat162float(f[j]));
+            }
           }
           if (row < row_end) {
             if (tn * BN + c + 32 <= N) {
@@ -543,15 +582,55 @@ static int gemm_bf16_launch(const void* X, const void* W, void* Y, int M, int N,
 
 FF_EXPORT int ff_gemm_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
                            int epi, int* status, cudaStream_t stream) {
-  return gemm_bf16_launch(X, W, Y, M, N, K, ldx, ldw, ldy, epi, LinTail{nullptr, 0}, status, stream);
+  return gemm_bf16_launch(X, W, Y, M, N, K, ldx, ldw, ldy, epi, LinTail{}, status, stream);
 }
 
-// Y = act(X Wᵀ + bias) in BF16. bias: [N] or null; act 0 none, 1 square of the positive part.
+// Y = act(X Wᵀ + bias) * mul[mul_rows[row], column] in BF16. bias: [N] or null; act 0 none, 1 square of the positive part, 3 tanh-GELU;
+// mul: table of mul_table rows (pitch ldm), or null.
 FF_EXPORT int ff_gemm_bf16_act(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
-                               const void* bias, int act, int* status, cudaStream_t stream) {
-  if ((unsigned)act > 1u) return FF_HOST_UNSUPPORTED;
+                               const void* bias, int act, const void* mul, const int* mul_rows, int ldm, int mul_table, int* status,
+                               cudaStream_t stream) {
+  if (act != 0 && act != 1 && act != 3) return FF_HOST_UNSUPPORTED;
   if (reinterpret_cast<uintptr_t>(bias) & 15) return FF_HOST_BAD_ALIGN;
-  return gemm_bf16_launch(X, W, Y, M, N, K, ldx, ldw, ldy, 0, LinTail{static_cast<const __nv_bfloat16*>(bias), act}, status, stream);
+  if (mul != nullptr && (mul_rows == nullptr || mul_table < 1 || ldm < N)) return FF_HOST_BAD_SHAPE;
+  if (mul != nullptr && (ldm % 8 || (reinterpret_cast<uintptr_t>(mul) & 15))) return FF_HOST_BAD_ALIGN;
+  return gemm_bf16_launch(X, W, Y, M, N, K, ldx, ldw, ldy, 0,
+                          LinTail{static_cast<const __nv_bfloat16*>(bias), act, static_cast<const __nv_bfloat16*>(mul), mul_rows, ldm, mul_table, 0},
+                          status, stream);
+}
+
+// Gate/up projection (rows interleaved per 64) with tanh-GELU(gate) * up in the epilogue, rounded once. Y has N / 2 columns.
+FF_EXPORT int ff_gemm_bf16_geglu(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy, int* status,
+                                 cudaStream_t stream) {
+  LinTail tail = {};
+  tail.gate = 3;
+  return gemm_bf16_launch(X, W, Y, M, N, K, ldx, ldw, ldy, 1, tail, status, stream);
+}
+
+// Block-diagonal product: for every head h, Y[:, h * c_cols + (0..N)] = X[:, h * a_cols + (0..K)] · W[h]ᵀ with W [heads * N, K]. Columns of
+// X past K that a tile reads meet zeros of W. a_cols, c_cols multiples of 8.
+FF_EXPORT int ff_gemm_bf16_heads(const void* X, const void* W, void* Y, int M, int heads, int N, int K, int ldx, int ldy, int a_cols, int c_cols,
+                                 int* status, cudaStream_t stream) {
+  if (M <= 0 || heads <= 0 || N <= 0 || K <= 0 || a_cols < K || c_cols < N) return FF_HOST_BAD_SHAPE;
+  if ((K % 8) || (ldx % 8) || (ldy % 8) || (a_cols % 8) || (c_cols % 8) || (reinterpret_cast<uintptr_t>(Y) & 15)) return FF_HOST_BAD_ALIGN;
+  if (ldx < (heads - 1) * a_cols + K || ldy < (heads - 1) * c_cols + N) return FF_HOST_BAD_SHAPE;
+  CUtensorMap tmA, tmB;
+  constexpr int BN = 256, STAGES = 4;
+  // the map ends with the last head's columns: what a row holds behind them is never read
+  int r = make_tmap_2d(&tmA, X, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)(heads - 1) * a_cols + K, M, (uint64_t)ldx * 2, BK, BM);
+  if (r) return r;
+  r = make_tmap_2d(&tmB, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, K, (uint64_t)heads * N, (uint64_t)K * 2, BK, BN);
+  if (r) return r;
+  const int smem = STAGES * (BM * BK * 2 + BN * BK * 2) + 1024;
+  auto kern = gemm_bf16_kernel<BN, STAGES, 0>;
+  r = opt_in_smem(kern, smem); if (r) return r;
+  const int tiles = ((M + BM - 1) / BM) * ((N + BN - 1) / BN) * heads;
+  const int grid = tiles < sm_count() ? tiles : sm_count();
+  CommArgs none = {};
+  GroupArgs ga = {};
+  ga.heads = heads; ga.a_cols = a_cols; ga.c_cols = c_cols;
+  kern<<<grid, 192, smem, stream>>>(tmA, tmA, tmA, tmB, Y, M, N, K, ldy, 0, status, none, ga, LinTail{});
+  return launch_result();
 }
 
 // Grouped GEMM over expert segments with 128-row token tiles (prefill sizes; the swap-AB kernel of moe.cu serves
@@ -575,7 +654,7 @@ FF_EXPORT int ff_moe_grouped_gemm_tiled(const void* Xs, const void* W, void* Y, 
   r = opt_in_smem(kern, smem); if (r) return r;
   CommArgs none = {};
   GroupArgs ga = {seg_off, counts, E_local};
-  kern<<<sm_count(), 192, smem, stream>>>(tmA, tmA, tmA, tmB, Y, capacity, Nw, K, ldy, epi, status, none, ga, LinTail{nullptr, 0});
+  kern<<<sm_count(), 192, smem, stream>>>(tmA, tmA, tmA, tmB, Y, capacity, Nw, K, ldy, epi, status, none, ga, LinTail{});
   return launch_result();
 }
 
@@ -625,7 +704,7 @@ FF_EXPORT int ff_ag_gemm(const unsigned long long* ptrs, int rank, int world, lo
   r = opt_in_smem(kern, smem); if (r) return r;
   const int tiles = (M / BM) * ((N + BN - 1) / BN);
   const int grid = tiles < sm_count() ? tiles : sm_count();
-  kern<<<grid, 320, smem, stream>>>(tmA0, tmA1, tmX, tmB, Y, M, N, K, ldy, epi, status, ca, GroupArgs{}, LinTail{nullptr, 0});
+  kern<<<grid, 320, smem, stream>>>(tmA0, tmA1, tmX, tmB, Y, M, N, K, ldy, epi, status, ca, GroupArgs{}, LinTail{});
   return launch_result();
 }
 
@@ -651,7 +730,7 @@ FF_EXPORT int ff_gemm_rs(const unsigned long long* ptrs, int rank, int world, lo
   r = opt_in_smem(kern, smem); if (r) return r;
   const int tiles = (M / BM) * ((N + BN - 1) / BN);
   const int grid = tiles < sm_count() ? tiles : sm_count();
-  kern<<<grid, 192, smem, stream>>>(tmA, tmA, tmA, tmB, nullptr, M, N, K, N, 0, status, ca, GroupArgs{}, LinTail{nullptr, 0});
+  kern<<<grid, 192, smem, stream>>>(tmA, tmA, tmA, tmB, nullptr, M, N, K, N, 0, status, ca, GroupArgs{}, LinTail{});
   return launch_result();
 }
 

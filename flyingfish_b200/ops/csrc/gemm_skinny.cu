@@ -48,11 +48,18 @@ struct alignas(8) SkinnyBars {
   int flag_b;
 };
 
+// What is done to the finished sums of a plain tile: bias per column, act 1 square of the positive part, 2 nothing (Y is FP32), 3
+// tanh-GELU, then a factor per element (row mul_rows[token] of a table).
+struct SkinnyTail {
+  const __nv_bfloat16* bias; int act;
+  const __nv_bfloat16* mul; const int* mul_rows; int ldm, mul_table;
+};
+
 // Where the final values of a tile go: Y, or (FUSE_AR) the arena slot of this rank on every rank.
 template <bool FUSE_AR>
 struct TileSink {
   __nv_bfloat16* Y; int N, ldy; bool vec8;      // vec8: 16-byte stores of eight values are aligned
-  const __nv_bfloat16* bias; int act;           // added to the finished sums; act 1: square of the positive part, 2: Y is FP32
+  SkinnyTail tail;
   PeerArena ar; int parity;
 
   // eight consecutive columns col..col+7 of token row t (col is a multiple of 8)
@@ -63,9 +70,21 @@ struct TileSink {
 #pragma unroll
     for (int j = 0; j < 8; ++j) a[j] = sums[j];
     if (!FUSE_AR) {
-      if (bias != nullptr) {
+      const int act = tail.act;
+      if (tail.bias != nullptr) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) if (col + j < N) a[j] += __bfloat162float(bias[col + j]);
+        for (int j = 0; j < 8; ++j) if (col + j < N) a[j] += __bfloat162float(tail.bias[col + j]);
+      }
+      if (act == 3) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) a[j] = gelu_tanh_f(a[j]);
+      }
+      if (tail.mul != nullptr) {
+        int mr = tail.mul_rows[t];
+        if (mr < 0 || mr >= tail.mul_table) mr = 0;          // reported where the id is first read (embedding)
+        const __nv_bfloat16* f = tail.mul + (size_t)mr * tail.ldm + col;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) if (col + j < N) a[j] *= __bfloat162float(f[j]);
       }
       if (act == 1) {
 #pragma unroll
@@ -221,7 +240,7 @@ __global__ void __launch_bounds__(192, 2)
 gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW,
                    __nv_bfloat16* __restrict__ Y, int M, int N, int K, int ldy, int ntok, int tile_rows, int stages,
                    int cl_size, int pipe_off, float* __restrict__ scratch, int* __restrict__ counters, int* status,
-                   PeerArena ar, SkinnyEpi ep, const __nv_bfloat16* __restrict__ bias, int act) {
+                   PeerArena ar, SkinnyEpi ep, const SkinnyTail tail) {
   pdl_trigger();
   if (cl_size > 1) cluster_arrive_relaxed();         // phase A: "this CTA runs" (waited on before the first remote store)
   if (threadIdx.x == 0) FF_TL(status, KID_GEMM_SKINNY, 0);
@@ -342,7 +361,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
     if (FUSE_AR) ar_epoch = ld_volatile(arena_epoch(ar)) + 1;
     TileSink<FUSE_AR> sink;
     sink.Y = Y; sink.N = N; sink.ldy = ldy; sink.ar = ar; sink.parity = ar_epoch & 1;
-    sink.bias = bias; sink.act = act;
+    sink.tail = tail;
     sink.vec8 = FUSE_AR || ((ldy % 8 == 0) && ((reinterpret_cast<uintptr_t>(Y) & 15) == 0));
     uint32_t seg_it = 0; bool ok = true;
     long long u = u0; Segment sg;
@@ -818,8 +837,7 @@ FF_EXPORT int ff_gemm_skinny_plan_epi(int M, int N, int K, int epi, long long* s
 
 static int gemm_skinny_launch(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
                               int grid, float* scratch, int* counters, int* status, cudaStream_t stream,
-                              const PeerArena* arena, const SkinnyEpi* epi = nullptr, const __nv_bfloat16* bias = nullptr,
-                              int act = 0) {
+                              const PeerArena* arena, const SkinnyEpi* epi = nullptr, const SkinnyTail& tail = SkinnyTail{}) {
   if (M <= 0 || N <= 0 || K <= 0) return FF_HOST_BAD_SHAPE;
   SkinnyEpi ep = {};
   if (epi != nullptr) {
@@ -853,12 +871,12 @@ static int gemm_skinny_launch(const void* X, const void* W, void* Y, int M, int 
     r = opt_in_smem(kern, SK_SMEM_FULL + 1024); if (r) return r;
     PeerArena none = {};
     return launch_pdl(kern, dim3(grid), dim3(192), smem, stream, cl, tmX, tmW, y, M, N, K, ldy, ntok, cfg.tile_rows,
-                      cfg.stages, cl, cfg.pipe_off, scratch, counters, status, none, ep, bias, act);
+                      cfg.stages, cl, cfg.pipe_off, scratch, counters, status, none, ep, tail);
   }
   auto kern = gemm_skinny_kernel<true>;
   r = opt_in_smem(kern, SK_SMEM_FULL + 1024); if (r) return r;
   return launch_pdl(kern, dim3(grid), dim3(192), smem, stream, cl, tmX, tmW, y, M, N, K, ldy, ntok, cfg.tile_rows,
-                    cfg.stages, cl, cfg.pipe_off, scratch, counters, status, *arena, ep, bias, act);
+                    cfg.stages, cl, cfg.pipe_off, scratch, counters, status, *arena, ep, tail);
 }
 
 // `grid` is the value returned by ff_gemm_skinny_plan for the same problem.
@@ -867,26 +885,31 @@ FF_EXPORT int ff_gemm_skinny(const void* X, const void* W, void* Y, int M, int N
   return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr);
 }
 
-// Y = act(X Wᵀ + bias): bias [N] or null, act 0 none, 1 square of the positive part (both on the FP32 sums). `grid` as above.
+// Y = act(X Wᵀ + bias) * mul[mul_rows[row], column]: bias [N] or null, act 0 none, 1 square of the positive part, 3 tanh-GELU; mul: table of
+// mul_table rows (pitch ldm), or null (all on the FP32 sums). `grid` as above.
 FF_EXPORT int ff_gemm_skinny_act(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
-                                 int grid, float* scratch, int* counters, const void* bias, int act, int* status, cudaStream_t stream) {
-  if ((unsigned)act > 1u) return FF_HOST_UNSUPPORTED;
+                                 int grid, float* scratch, int* counters, const void* bias, int act, const void* mul, const int* mul_rows,
+                                 int ldm, int mul_table, int* status, cudaStream_t stream) {
+  if (act != 0 && act != 1 && act != 3) return FF_HOST_UNSUPPORTED;
+  if (mul != nullptr && (mul_rows == nullptr || mul_table < 1 || ldm < N)) return FF_HOST_BAD_SHAPE;
   return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr, nullptr,
-                            static_cast<const __nv_bfloat16*>(bias), act);
+                            SkinnyTail{static_cast<const __nv_bfloat16*>(bias), act, static_cast<const __nv_bfloat16*>(mul), mul_rows, ldm, mul_table});
 }
 
 // Y = X Wᵀ with the FP32 sums stored as they are (router and gate logits, vocabulary logits). `grid` as above.
 FF_EXPORT int ff_gemm_skinny_f32out(const void* X, const void* W, float* Y, int M, int N, int K, int ldx, int ldw, int ldy,
                                     int grid, float* scratch, int* counters, int* status, cudaStream_t stream) {
-  return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr, nullptr, nullptr, 2);
+  return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr, nullptr,
+                            SkinnyTail{nullptr, 2, nullptr, nullptr, 0, 0});
 }
 
 // Gate/up projection with the SwiGLU applied in the epilogue: W is [N, K] with gate/up rows interleaved per
-// 64, Y is [M, N/2]. `grid` from ff_gemm_skinny_plan_epi(M, N, K, 1).
+// 64, Y is [M, N/2]. gate 0: SiLU, 3: tanh-GELU rounded once. `grid` from ff_gemm_skinny_plan_epi(M, N, K, 1).
 FF_EXPORT int ff_gemm_skinny_swiglu(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
-                                    int grid, float* scratch, int* counters, int* status, cudaStream_t stream) {
+                                    int grid, float* scratch, int* counters, int gate, int* status, cudaStream_t stream) {
+  if (gate != 0 && gate != 3) return FF_HOST_UNSUPPORTED;
   SkinnyEpi ep = {};
-  ep.mode = 1;
+  ep.mode = 1; ep.gate = gate;
   return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr, &ep);
 }
 

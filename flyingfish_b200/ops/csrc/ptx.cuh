@@ -353,6 +353,10 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
 }
+// 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), written as z times a logistic function; error of a few 1e-7 of |z|
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  return __fdividef(z, 1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
 __device__ __forceinline__ float2 unpack_bf16x2(uint32_t u) {
   __nv_bfloat162 v = *reinterpret_cast<__nv_bfloat162*>(&u);
   return __bfloat1622float2(v);

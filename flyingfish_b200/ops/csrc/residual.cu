@@ -6,6 +6,11 @@
 // beyond the last expert is an identity output: y_j is the row h the experts were given), so a layer ends in one kernel: the
 // residual is read and written once in FP32 and nothing is rounded on the way. One block per row; a thread owns the same
 // columns in both passes. Norm weights are FP32 (offsets already added).
+//
+// Layers whose sub-layers are normed on both sides (sequential layers) have a kernel of their own below:
+//   x += inner(y)        n = outer(x)
+// inner is the norm behind a sub-layer, outer the one in front of the next: an RMS norm, or tanh(alpha x) w + b (which needs no
+// statistics of the row); outer may also be a plain copy in the GEMM operand's type.
 #include "dtype_io.cuh"
 #include "host_util.h"
 
@@ -121,8 +126,152 @@ static int residual_launch(float* x, const int* ids, const void* table, float sc
   return launch_result();
 }
 
+// ------------------------------------------------------------------------------------------
+// norms on both sides of a sub-layer
+// ------------------------------------------------------------------------------------------
+enum { NORM_COPY = 0, NORM_RMS = 1, NORM_TANH = 2 };
+
+struct NormArgs { const float* w; const float* b; float alpha; int kind; };
+
+// BF16 results: 1 - 2 / (1 + e^2x), whose error (1e-7 of 1) vanishes in the rounding; FP32 results take tanhf
+__device__ __forceinline__ float norm_tanh(float x, __nv_bfloat16) { return 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * fminf(x, 20.0f))); }
+__device__ __forceinline__ float norm_tanh(float x, float) { return tanhf(x); }
+
+// four columns at c: v <- norm(v); r: one over the row's root mean square (RMS norm)
+template <typename T>
+__device__ __forceinline__ void apply_norm(const NormArgs& a, int c, float r, float (&v)[4]) {
+  if (a.kind == NORM_COPY) return;
+  float w[4];
+  load4(a.w + c, w);
+  if (a.kind == NORM_RMS) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] = v[j] * r * w[j];
+    return;
+  }
+  float b[4];
+  load4(a.b + c, b);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) v[j] = fmaf(norm_tanh(a.alpha * v[j], T()), w[j], b[j]);
+}
+
+// all threads of the block: one over the root mean square from the threads' sums of squares
+__device__ __forceinline__ float block_rms(float ss, float* s_red, int true_width, float eps) {
+  ss = warp_sum(ss);
+  __syncthreads();                                         // the previous reduction has been read
+  if ((threadIdx.x & 31) == 0) s_red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  const float tot = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? s_red[threadIdx.x & 31] : 0.f);
+  return 1.0f / sqrtf(tot / (float)true_width + eps);
+}
+
+template <typename T, bool EMBED>
+__global__ void __launch_bounds__(RN_THREADS)
+residual_sandwich_kernel(float* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ table, float scale, int vocab,
+                         const T* __restrict__ y, NormArgs inner, NormArgs outer, T* __restrict__ n, int width, int true_width, float eps,
+                         int* status) {
+  pdl_trigger();
+  extern __shared__ __align__(16) float rn_x[];            // [width] the row between passes (only with an RMS norm)
+  __shared__ float s_red[RN_THREADS / 32];
+  const int row = blockIdx.x, tid = threadIdx.x, step = blockDim.x * 4;
+  pdl_wait();
+  const T* src;
+  if (EMBED) {
+    int id = ids[row];
+    if (id < 0 || id >= vocab) { if (tid == 0) set_status(status, KID_EMBED, FF_ERR_BOUNDS, row, id); id = 0; }
+    src = table + (size_t)id * width;
+  } else {
+    src = y + (size_t)row * width;
+  }
+  float* xr = x + (size_t)row * width;
+  T* nr = n + (size_t)row * width;
+  float r_in = 1.f;
+  const bool stage = !EMBED && inner.kind == NORM_RMS;
+  if (stage) {
+    float ss = 0.f;
+    for (int c = tid * 4; c < width; c += step) {
+      float t[4];
+      load4(src + c, t);
+      store4(rn_x + c, t);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss = fmaf(t[j], t[j], ss);
+    }
+    r_in = block_rms(ss, s_red, true_width, eps);
+  }
+  float ss = 0.f;
+  for (int c = tid * 4; c < width; c += step) {
+    float v[4];
+    if (EMBED) {
+      load4(src + c, v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] *= scale;
+    } else {
+      float t[4];
+      load4(xr + c, v);
+      if (stage) load4(rn_x + c, t); else load4(src + c, t);
+      apply_norm<T>(inner, c, r_in, t);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] += t[j];
+    }
+    store4(xr + c, v);
+    if (outer.kind == NORM_RMS) {
+      store4(rn_x + c, v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss = fmaf(v[j], v[j], ss);
+    } else {
+      apply_norm<T>(outer, c, 1.f, v);
+      store4(nr + c, v);
+    }
+  }
+  if (outer.kind != NORM_RMS) return;
+  const float r = block_rms(ss, s_red, true_width, eps);
+  for (int c = tid * 4; c < width; c += step) {            // the thread's own columns again
+    float v[4];
+    load4(rn_x + c, v);
+    apply_norm<T>(outer, c, r, v);
+    store4(nr + c, v);
+  }
+}
+
+template <typename T, bool EMBED>
+static int sandwich_launch(float* x, const int* ids, const void* table, float scale, int vocab, const void* y, NormArgs inner, NormArgs outer,
+                           void* n, int rows, int width, int true_width, float eps, int* status, cudaStream_t s) {
+  if (rows <= 0 || width <= 0 || width % 8 || true_width <= 0 || true_width > width) return FF_HOST_BAD_SHAPE;
+  for (const NormArgs* a : {&inner, &outer}) {
+    if ((unsigned)a->kind > NORM_TANH || (a->kind != NORM_COPY && a->w == nullptr) || (a->kind == NORM_TANH && a->b == nullptr)) return FF_HOST_BAD_SHAPE;
+    if ((reinterpret_cast<uintptr_t>(a->w) & 15) || (reinterpret_cast<uintptr_t>(a->b) & 15)) return FF_HOST_BAD_ALIGN;
+  }
+  const int smem = inner.kind == NORM_RMS || outer.kind == NORM_RMS ? width * 4 : 0;
+  if (smem > 200 * 1024) return FF_HOST_TOO_LARGE;
+  auto kern = residual_sandwich_kernel<T, EMBED>;
+  if (int r = opt_in_smem(kern, smem)) return r;
+  int threads = (width / 4 + 31) / 32 * 32;
+  const int cap = rows >= 2 * sm_count() ? RN_THREADS / 2 : RN_THREADS;
+  if (threads > cap) threads = cap;
+  if (int r = launch_pdl(kern, dim3(rows), dim3(threads), smem, s, 0, x, ids, (const T*)table, scale, vocab, (const T*)y, inner, outer, (T*)n,
+                         width, true_width, eps, status)) return r;
+  return launch_result();
+}
+
 }  // namespace ff
 using namespace ff;
+
+// x FP32 [rows, width] = table[id] * scale; n = outer(x). kinds: 0 copy, 1 RMS norm times w, 2 tanh(alpha x) w + b; w, b FP32 [width]
+FF_EXPORT int ff_residual_embed_normed(const int* ids, const void* table, float scale, float* x, int kind, const float* w, const float* b,
+                                       float alpha, void* n, int rows, int width, int true_width, int vocab, float eps, int f32, int* status,
+                                       cudaStream_t s) {
+  const NormArgs none = {nullptr, nullptr, 0.f, NORM_COPY}, outer = {w, b, alpha, kind};
+  if (f32) return sandwich_launch<float, true>(x, ids, table, scale, vocab, nullptr, none, outer, n, rows, width, true_width, eps, status, s);
+  return sandwich_launch<__nv_bfloat16, true>(x, ids, table, scale, vocab, nullptr, none, outer, n, rows, width, true_width, eps, status, s);
+}
+
+// x += inner(y); n = outer(x)
+FF_EXPORT int ff_residual_add_normed(float* x, const void* y, int ikind, const float* iw, const float* ib, float ialpha, int okind, const float* ow,
+                                     const float* ob, float oalpha, void* n, int rows, int width, int true_width, float eps, int f32,
+                                     cudaStream_t s) {
+  const NormArgs inner = {iw, ib, ialpha, ikind}, outer = {ow, ob, oalpha, okind};
+  if (f32) return sandwich_launch<float, false>(x, nullptr, nullptr, 1.f, 0, y, inner, outer, n, rows, width, true_width, eps, nullptr, s);
+  return sandwich_launch<__nv_bfloat16, false>(x, nullptr, nullptr, 1.f, 0, y, inner, outer, n, rows, width, true_width, eps, nullptr, s);
+}
 
 // x FP32 [rows, width]; table, n1, n2 in BF16 (f32 = 0) or FP32; w1, w2 FP32 [width] (w2, n2: both or neither)
 FF_EXPORT int ff_residual_embed(const int* ids, const void* table, float scale, float* x, const float* w1, const float* w2, void* n1, void* n2,

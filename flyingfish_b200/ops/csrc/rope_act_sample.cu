@@ -96,6 +96,7 @@ __device__ __forceinline__ float act_combine(float g, float u, int mode, float l
     const float t = tanhf(k0 * (g + k1 * g * g * g));
     return bf16r(0.5f * g * (1.f + t)) * u;
   }
+  if (mode == 3) return gelu_tanh_f(g) * u;
   // clamped: gate <= limit, up in [-limit, limit]
   g = fminf(g, limit); u = fmaxf(fminf(u, limit), -limit);
   return (g / (1.f + __expf(-g))) * u;
@@ -141,9 +142,9 @@ __global__ void silu_mul_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloa
   reinterpret_cast<uint4*>(out + (size_t)row * ldo)[c] = o;
 }
 
-// the same in FP32 (no intermediate rounding), four elements per thread
+// the same in FP32 (no intermediate rounding; mode 2 and 3: tanh-GELU, otherwise SiLU), four elements per thread
 __global__ void silu_mul_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int f, int ldgu, int ldo,
-                                    int interleaved) {
+                                    int mode, int interleaved) {
   pdl_trigger();
   pdl_wait();
   const int vec_per_row = f >> 2;
@@ -155,7 +156,10 @@ __global__ void silu_mul_f32_kernel(const float* __restrict__ gu, float* __restr
   load4(gu + (size_t)row * ldgu + gc, g);
   load4(gu + (size_t)row * ldgu + uc, u);
 #pragma unroll
-  for (int j = 0; j < 4; ++j) g[j] = g[j] * sigmoid_f(g[j]) * u[j];
+  for (int j = 0; j < 4; ++j) {
+    const float z = g[j];
+    g[j] = (mode >= 2 ? 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))) : z * sigmoid_f(z)) * u[j];
+  }
   store4(out + (size_t)row * ldo + c, g);
 }
 
@@ -454,11 +458,12 @@ FF_EXPORT int ff_silu_mul(const void* gu, void* out, int rows, int f, int ldgu, 
   return launch_result();
 }
 
-// gate/up rows in FP32: out = silu(gate) * up
-FF_EXPORT int ff_silu_mul_f32(const float* gu, float* out, int rows, int f, int ldgu, int ldo, int interleaved, cudaStream_t s) {
+// gate/up rows in FP32: out = act(gate) * up; mode 0 and 1: SiLU, 2 and 3: tanh-GELU
+FF_EXPORT int ff_silu_mul_f32(const float* gu, float* out, int rows, int f, int ldgu, int ldo, int mode, int interleaved, cudaStream_t s) {
+  if (mode < 0 || mode > 3) return FF_HOST_UNSUPPORTED;
   if (rows <= 0 || f <= 0 || f % 4 || ldgu % 4 || ldo % 4 || (interleaved && f % 64)) return FF_HOST_BAD_SHAPE;
   const long long total = (long long)rows * (f / 4);
-  if (int r = launch_pdl(silu_mul_f32_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, 0, gu, out, rows, f, ldgu, ldo, interleaved)) return r;
+  if (int r = launch_pdl(silu_mul_f32_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, 0, gu, out, rows, f, ldgu, ldo, mode, interleaved)) return r;
   return launch_result();
 }
 

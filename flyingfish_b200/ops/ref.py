@@ -31,14 +31,17 @@ def _r(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
 # linear
 # ------------------------------------------------------------------------------------------
 def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None, bias: torch.Tensor | None = None,
-           act: str | None = None) -> torch.Tensor:
+           act: str | None = None, mul: tuple[torch.Tensor, torch.Tensor] | None = None) -> torch.Tensor:
     """``y = x @ w.T``, one rounding to the output dtype. The products are accumulated in FP64 so
     the oracle does not depend on how a BLAS blocks the sum for a given batch size (results are
     batch-invariant, as the device kernels' are)."""
     y = x.to(torch.float64) @ w.to(torch.float64).t()
     if bias is not None:
         y = y + bias.to(torch.float64)
-    return activate(y, act).to(out_dtype or x.dtype)
+    y = activate(y, act)
+    if mul is not None:
+        y = y * mul[0][mul[1].long()].to(torch.float64)
+    return y.to(out_dtype or x.dtype)
 
 
 def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, mode: int = 0) -> torch.Tensor:
@@ -49,8 +52,10 @@ def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, mode: int = 0) -
     n = y.shape[-1]
     y = y.view(*y.shape[:-1], n // 128, 2, 64)
     gate, up = y[..., 0, :], y[..., 1, :]
-    gu = torch.cat([gate.reshape(*y.shape[:-3], -1), up.reshape(*y.shape[:-3], -1)], dim=-1).to(x.dtype)
-    return silu_mul(gu, mode=mode)
+    gu = torch.cat([gate.reshape(*y.shape[:-3], -1), up.reshape(*y.shape[:-3], -1)], dim=-1)
+    if mode == 3:                                   # rounded once
+        return silu_mul(gu, mode=mode).to(x.dtype)
+    return silu_mul(gu.to(x.dtype), mode=mode)
 
 
 def interleave_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor:
@@ -147,7 +152,7 @@ def rope_kv_paged(qkv: torch.Tensor, positions: torch.Tensor, slots: torch.Tenso
 # ------------------------------------------------------------------------------------------
 def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0) -> torch.Tensor:
     """gu: [..., 2f] = gate | up. Modes: 0 = silu rounded then product rounded, 1 = single rounding,
-    2 = tanh-GELU twice rounded, 4 = clamped SwiGLU in FP32 (gate <= limit, |up| <= limit)."""
+    2 = tanh-GELU twice rounded, 3 = tanh-GELU with a single rounding, 4 = clamped SwiGLU in FP32 (gate <= limit, |up| <= limit)."""
     f = gu.shape[-1] // 2
     dt = gu.dtype
     g, u = gu[..., :f].to(F32), gu[..., f:].to(F32)
@@ -158,6 +163,8 @@ def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0) -> torch.Tenso
     elif mode == 2:
         t = torch.tanh(0.7978845608028654 * (g + 0.044715 * g ** 3))
         y = _r(0.5 * g * (1 + t), dt) * u
+    elif mode == 3:
+        y = activate(g, "gelu_tanh") * u
     elif mode == 4:
         g = torch.clamp(g, max=limit)
         u = torch.clamp(u, min=-limit, max=limit)
@@ -186,11 +193,14 @@ def attention_paged(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
                     q_start: torch.Tensor, q_lens: torch.Tensor, ctx_lens: torch.Tensor, hq: int, hkv: int,
                     dim: int, scale: float, tree_mask: torch.Tensor | None = None, window: int = 0,
                     sinks: torch.Tensor | None = None, chunk: int = 0, vdim: int | None = None,
-                    gate: torch.Tensor | None = None) -> torch.Tensor:
+                    gate: torch.Tensor | None = None, keep: int = 0, softcap: float = 0.0,
+                    head_gate: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of packed query rows against the paged cache. ``chunk > 0``: a query sees only keys of its own
     block of ``chunk`` positions. ``vdim``: width of a value head (default ``dim``). ``gate`` ([rows, hq*vdim]): the
     result is multiplied by its sigmoid. ``sinks`` (float [hq]): learnable soft-max, one
-    extra logit per head that takes probability mass but contributes no value.
+    extra logit per head that takes probability mass but contributes no value. ``keep``: with a window, the first ``keep``
+    positions stay visible. ``softcap``: scores become ``softcap * tanh(score / softcap)``. ``head_gate`` ([rows, hq]): a head's
+    result is multiplied by its sigmoid.
 
     q: [rows, >= hq*dim] (head h at columns h*dim). Sequence b owns rows
     ``q_start[b] : q_start[b]+q_lens[b]`` and ``ctx_lens[b]`` cached keys; its query i sits at
@@ -210,11 +220,13 @@ def attention_paged(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
         k = k.repeat_interleave(g, dim=1)
         v = v.repeat_interleave(g, dim=1)
         s = torch.einsum("qhd,khd->hqk", qb, k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         pos_q = torch.arange(ql)[:, None] + (ctx - ql)
         pos_k = torch.arange(ctx)[None, :]
         vis = pos_k <= pos_q if window >= 0 else torch.ones(ql, ctx, dtype=torch.bool)   # window < 0: bidirectional
         if window > 0:
-            vis &= pos_k > pos_q - window
+            vis &= (pos_k > pos_q - window) | (pos_k < keep)
         if chunk > 0:
             vis &= pos_k >= torch.div(pos_q, chunk, rounding_mode="floor") * chunk
         if tree_mask is not None:
@@ -234,6 +246,8 @@ def attention_paged(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
         o = o.reshape(ql, hq * vdim)
         if gate is not None:
             o = o * torch.sigmoid(gate[qs: qs + ql].to(F32))
+        if head_gate is not None:
+            o = o * torch.sigmoid(head_gate[qs: qs + ql].to(F32)).repeat_interleave(vdim, 1)
         out[qs: qs + ql] = o.to(q.dtype)
     return out
 
@@ -244,25 +258,40 @@ def attention_paged(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
 def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, hq: int, hkv: int,
                  dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0,
                  q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None,
-                 cos_sin: torch.Tensor | None = None) -> None:
+                 cos_sin: torch.Tensor | None = None, whole: bool = False, halves: bool = False,
+                 temp: tuple[torch.Tensor, float, int] | None = None) -> None:
     """In place on the q heads of ``qkv``: q and k divided by their root mean square over ``dim`` (heads may be padded in
-    the row: the caches' widths are the row's head widths), weighted and rotated where that is given, v blended with ``first_v``; k and v go to ``slots``."""
-    rows, bs = qkv.shape[0], kcache.shape[2]
-    dk, dv = kcache.shape[3], vcache.shape[3]
+    the row: the caches' widths are the row's head widths), or over all heads (``whole``), weighted and rotated where that is
+    given, v blended with ``first_v``; k and v go to ``slots``."""
+    rows = qkv.shape[0]
+    dk = kcache.shape[3] if hkv else qkv.shape[1] // hq
     nq, nk = hq * dk, hkv * dk
     qk = qkv[:, : nq + nk].to(F32).view(rows, hq + hkv, dk)
-    qk = qk * torch.rsqrt((qk * qk).sum(-1, keepdim=True) / dim + eps)
+    if whole:
+        ss = qk.square().sum(-1)
+        mean = torch.cat([ss[:, :hq].sum(-1, keepdim=True).expand(rows, hq) / hq, ss[:, hq:].sum(-1, keepdim=True).expand(rows, hkv) / max(hkv, 1)], 1)
+        qk = qk * torch.rsqrt(mean[..., None] / dim + eps)
+    else:
+        qk = qk * torch.rsqrt((qk * qk).sum(-1, keepdim=True) / dim + eps)
     if q_weight is not None:
-        qk[:, :hq] *= q_weight
-    if k_weight is not None:
-        qk[:, hq:] *= k_weight
+        qk[:, :hq] *= q_weight.view(-1, dk)
+    if k_weight is not None and hkv:
+        qk[:, hq:] *= k_weight.view(-1, dk)
     if cos_sin is not None:
         r = 2 * cos_sin.shape[1]
         c, s = cos_sin[:, None, :, 0], cos_sin[:, None, :, 1]
-        u, w = qk[..., 0:r:2].clone(), qk[..., 1:r:2].clone()
-        qk[..., 0:r:2] = u * c - w * s
-        qk[..., 1:r:2] = w * c + u * s
+        pu, pw = (slice(0, r // 2), slice(r // 2, r)) if halves else (slice(0, r, 2), slice(1, r, 2))
+        u, w = qk[..., pu].clone(), qk[..., pw].clone()
+        qk[..., pu] = u * c - w * s
+        qk[..., pw] = w * c + u * s
+    if temp is not None:
+        positions, coef, every = temp
+        f = 1.0 + coef * torch.log(torch.div(positions + 1, every, rounding_mode="floor").to(F32) + 1.0)
+        qk[:, :hq] *= f[:, None, None]
     qkv[:, : nq] = qk[:, :hq].reshape(rows, nq).to(qkv.dtype)
+    if not hkv:
+        return
+    bs, dv = kcache.shape[2], vcache.shape[3]
     v = qkv[:, nq + nk: nq + nk + hkv * dv].to(F32)
     if first_v is not None:
         v = (1.0 - mix) * v + mix * first_v.to(F32)
@@ -276,6 +305,8 @@ def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, v
 def activate(x: torch.Tensor, act: str | None) -> torch.Tensor:
     if act is None:
         return x
+    if act == "gelu_tanh":
+        return 0.5 * x * (1 + torch.tanh(0.7978845608028654 * (x + 0.044715 * x ** 3)))
     assert act == "relu2", act
     return torch.relu(x) ** 2
 

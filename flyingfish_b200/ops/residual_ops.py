@@ -1,11 +1,14 @@
-"""FP32 residual stream of parallel layers: the sums a layer ends with, and the one or two norms the next one starts with, in one
-kernel. CUDA: ``csrc/residual.cu``; CPU: FP32 arithmetic on the same layouts.
+"""FP32 residual stream. Parallel layers (:func:`embed`, :func:`step`): the sums a layer ends with, and the one or two norms the next
+one starts with, in one kernel. Sequential layers with norms on both sides of a sub-layer (:func:`embed_normed`, :func:`add_normed`):
+the norm behind one sub-layer, the sum and the norm in front of the next. CUDA: ``csrc/residual.cu``; CPU: FP32 arithmetic on the same
+layouts.
 
 The stream is FP32 ``[rows, width]``; norm weights are FP32 vectors with any offset already added; ``true_width`` is the width the
 norms divide by where ``width`` carries padding."""
 from __future__ import annotations
 
 from ctypes import c_float
+from dataclasses import dataclass
 
 import torch
 
@@ -70,3 +73,61 @@ def step(x: torch.Tensor, a: torch.Tensor, b: torch.Tensor | None, experts: Expe
     check(rc, "ff_residual_step")
     _count()
     return n1, n2
+
+
+# ------------------------------------------------------------------------------------------
+# norms on both sides of a sub-layer
+# ------------------------------------------------------------------------------------------
+@dataclass
+class Norm:
+    """``kind`` "rms": ``x / rms(x) * w``; "tanh": ``tanh(alpha x) * w + b``; "copy": the row in the operand type. FP32 vectors."""
+    kind: str = "copy"
+    w: torch.Tensor | None = None
+    b: torch.Tensor | None = None
+    alpha: float = 0.0
+
+    KINDS = {"copy": 0, "rms": 1, "tanh": 2}
+
+    def __call__(self, x: torch.Tensor, eps: float, true_width: int) -> torch.Tensor:
+        """FP32 rows normed (the oracle)."""
+        if self.kind == "rms":
+            return x * torch.rsqrt((x * x).sum(-1, keepdim=True) / true_width + eps) * self.w
+        return torch.tanh(self.alpha * x) * self.w + self.b if self.kind == "tanh" else x
+
+    def args(self, width: int) -> tuple:
+        for v in (self.w, self.b):
+            _require(v is None or (v.dtype == torch.float32 and v.numel() == width and v.is_contiguous()), "norm: FP32 vectors of the width")
+        return self.KINDS[self.kind], ptr(self.w), ptr(self.b), c_float(self.alpha)
+
+
+def embed_normed(ids: torch.Tensor, table: torch.Tensor, scale: float, outer: Norm, eps: float, true_width: int
+                 ) -> tuple[torch.Tensor, torch.Tensor]:
+    """(FP32 stream ``table[ids] * scale``, its norm)."""
+    if not table.is_cuda:
+        x = table[ids.long()].float() * scale
+        return x, outer(x, eps, true_width).to(table.dtype)
+    rows, (vocab, width) = ids.numel(), table.shape
+    _require(ids.dtype == torch.int32 and table.is_contiguous() and width % 8 == 0, "residual embed: int32 ids, rows of 8 elements")
+    x = torch.empty(rows, width, dtype=torch.float32, device=table.device)
+    n = torch.empty(rows, width, dtype=table.dtype, device=table.device)
+    rc = kernels().ff_residual_embed_normed(ptr(ids), ptr(table), c_float(scale), ptr(x), *outer.args(width), ptr(n), rows, width, true_width,
+                                            vocab, c_float(eps), int(table.dtype == torch.float32), ptr(status_tensor(table.device)), stream_ptr())
+    check(rc, "ff_residual_embed_normed")
+    _count()
+    return x, n
+
+
+def add_normed(x: torch.Tensor, y: torch.Tensor, inner: Norm, outer: Norm, eps: float, true_width: int) -> torch.Tensor:
+    """``x += inner(y)`` in place (FP32); returns ``outer(x)`` in the type of ``y``."""
+    if not x.is_cuda:
+        x += inner(y.float(), eps, true_width)
+        return outer(x, eps, true_width).to(y.dtype)
+    rows, width = x.shape
+    _require(x.dtype == torch.float32 and x.is_contiguous() and width % 8 == 0, "residual step: FP32 rows of 8 elements")
+    _require(y.shape == x.shape and y.is_contiguous(), "residual step: rows of the stream's shape")
+    n = torch.empty(rows, width, dtype=y.dtype, device=x.device)
+    rc = kernels().ff_residual_add_normed(ptr(x), ptr(y), *inner.args(width), *outer.args(width), ptr(n), rows, width, true_width, c_float(eps),
+                                          int(y.dtype == torch.float32), stream_ptr())
+    check(rc, "ff_residual_add_normed")
+    _count()
+    return n

@@ -26,7 +26,7 @@ from pathlib import Path
 
 import torch
 
-from ..config import Settings, named_shape, read_model_spec
+from ..config import Settings, named_shape, pad_to, read_model_spec
 from ..utils.log import log_json
 
 CAPACITY_BUCKETS = (2048, 16384, 49152, 98304, 131072)       # decode-attention plan buckets
@@ -203,12 +203,14 @@ def measure_disk_rate(runtime_dir: Path, nbytes: int = 64 << 20) -> float:
 def decode_linear_shapes(spec, tp: int = 1) -> list[tuple[str, int, int, int]]:
     """(name, N, K, epilogue id) of the decode projections of a dense / GQA layer on one rank of ``tp``."""
     if spec.layer_specs is not None:          # designs whose layers differ: every distinct projection once
-        seen: dict[tuple[int, int], str] = {}
+        seen: dict[tuple[int, int, int], str] = {}
         for l in spec.layer_specs:
-            for name, n, k in (("qkv", l.projection_cols, spec.hidden), ("o", spec.hidden, l.heads * l.vdim_pad)) + \
-                    ((("up", l.ffn, spec.hidden), ("down", spec.hidden, l.ffn)) if l.ffn else ()):
-                seen.setdefault((n, k), name if name not in seen.values() else f"{name} {n} x {k}")
-        return [(name, n, k, 0) for (n, k), name in seen.items()]
+            fp = pad_to(l.ffn, 128)
+            ffn = (("gate_up", 2 * fp, spec.hidden, 1), ("down", spec.hidden, fp, 0)) if l.ffn_act == "geglu" else \
+                (("up", l.ffn, spec.hidden, 0), ("down", spec.hidden, l.ffn, 0))
+            for name, *shape in (("qkv", l.projection_cols, spec.hidden, 0), ("o", spec.hidden, l.heads * l.vdim_pad, 0)) + (ffn if l.ffn else ()):
+                seen.setdefault(tuple(shape), name if name not in seen.values() else f"{name} {shape[0]} x {shape[1]}")
+        return [(name, *shape) for shape, name in seen.items()]
     d, h = spec.head_dim, spec.hidden
     hq, hkv = spec.heads // tp, max(1, spec.kv_heads // tp)
     f = spec.ffn // tp

@@ -64,7 +64,9 @@ def workspace_row_bytes(spec: ModelSpec, tp: int = 1) -> int:
         streams = int(spec.extra.get("duponex", {}).get("streams", 1))
         # experts: sorted rows, their two intermediates, and the shared expert's rows
         moe = lambda m: 0 if m is None else m.top_k * (2 * spec.hidden + 2 * m.expert_ffn) + 2 * m.shared_ffn
-        wide = max(l.projection_cols + 2 * l.heads * l.vdim_pad + l.ffn + moe(l.moe) for l in spec.layer_specs)
+        # latent attention: queries and results of every head in the latent space
+        lat = lambda l: l.heads * (2 * l.rank_pad + l.rot_pad)
+        wide = max(l.projection_cols + 2 * l.heads * l.vdim_pad + lat(l) + l.ffn + moe(l.moe) for l in spec.layer_specs)
         return 4 * spec.hidden * streams + (4 * spec.hidden + 2 * wide) * spec.elem_bytes + 12
     ffn = spec.moe.expert_ffn * spec.moe.top_k if spec.moe is not None else spec.ffn
     return (4 * spec.hidden + spec.qkv_dim // tp + 3 * ffn // tp) * 2 + 12 + spec.heads * 4
