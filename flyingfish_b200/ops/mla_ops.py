@@ -117,11 +117,11 @@ def latent_norm_kv(p: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, q_
             u, v = x[..., 0: 2 * half: 2].clone(), x[..., 1: 2 * half: 2].clone()
             x[..., 0: 2 * half: 2], x[..., 1: 2 * half: 2] = u * c - v * s, v * c + u * s
             return x
-        q = p[:, q_rot_col: q_rot_col + heads * rot].to(F32).view(rows, heads, rot)
+        q = p[:, q_rot_col: q_rot_col + heads * rot].to(F32, copy=True).view(rows, heads, rot)
         q_full[..., rank_pad:] = turn(q, c[:, None], s[:, None]).to(p.dtype)
         lat = p[:, latent_col: latent_col + rank_pad].to(F32)
         lat = lat * torch.rsqrt((lat * lat).sum(-1, keepdim=True) / rank + eps) * weight
-        k = turn(p[:, latent_col + rank_pad: latent_col + width].to(F32), c, s)
+        k = turn(p[:, latent_col + rank_pad: latent_col + width].to(F32, copy=True), c, s)
         ok = slots >= 0
         at = slots[ok].long()
         cache[at // bs, 0, at % bs] = torch.cat([lat, k], 1)[ok].to(cache.dtype)
