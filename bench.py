@@ -76,7 +76,7 @@ def parse() -> argparse.Namespace:
     p.add_argument("--skip-e2e", action="store_true")
     p.add_argument("--skip-baseline", action="store_true")
     p.add_argument("--skip-extras", action="store_true", help="no TTFT run and no other batch sizes")
-    p.add_argument("--design", default=None, choices=["duponex", "rudorax"],
+    p.add_argument("--design", default=None, choices=["duponex", "rudorax", "kabavik"],
                    help="instead of the headline benchmark: throughput and kernels of this design beside the closest model at equal size")
     p.add_argument("--device", default="cuda", choices=["cuda", "cpu"], help="cpu is for debugging the harness only")
     a = p.parse_args()

@@ -1,10 +1,12 @@
-"""A design's throughput and kernels beside the closest other model at equal size (``bench.py --design duponex|rudorax``).
+"""A design's throughput and kernels beside the closest other model at equal size (``bench.py --design duponex|rudorax|kabavik``).
 
 The closest model of a Rudorax shape is the Flint layout (QK-norm, windowed attention with sinks, routed and shared experts): same
 width, heads, window, experts and number of layers (Rudorax: layer runs); a memory layer's kernels are timed beside those of the
 gated delta net. The closest model of a Duponex shape is the Gemma layout (QK-norm, local attention in every layer, extra norms per
 sub-layer, operator-by-operator decode step): same width, heads and layers, a sliding window as long as the block, and a
-gated feed-forward of the width that makes the layers' weights equal. Prompts end inside a block, so both attentions see
+gated feed-forward of the width that makes the layers' weights equal. A Kabavik shape is measured beside the Gemma layout too, with a
+feed-forward that makes the mean weights of a layer equal; the kernels of its latent layers beside those of the DeepSeek layout.
+Prompts end inside a block, so both attentions see
 the same keys. Weights are random. Every kernel of the design is timed beside its like kernel on the same rows; a
 fraction of the roofline is algorithmic bytes (or FLOPs) over time over the measured peak, and ``distance`` is the ratio
 of the two fractions (above 1: the design's kernel is further from its roofline).
@@ -17,15 +19,16 @@ import torch
 
 from .. import ops
 from ..config import ModelSpec, MoeSpec, Settings, named_shape
-from ..ops import gdn_ops, mlstm_ops, moe_cuda, moe_ops, residual_ops, stream_ops
+from ..ops import gdn_ops, mla_ops, mlstm_ops, moe_cuda, moe_ops, residual_ops, stream_ops
 from .kbench import Flusher, peaks, time_op
 
-SIZES = {"duponex": ("duponex-2b-shape", "duponex-8b-shape"), "rudorax": ("rudorax-2k-shape", "rudorax-4k-shape")}
+SIZES = {"duponex": ("duponex-2b-shape", "duponex-8b-shape"), "rudorax": ("rudorax-2k-shape", "rudorax-4k-shape"),
+         "kabavik": ("kabavik-2k-shape", "kabavik-4k-shape")}
 
 
 def closest_spec(spec: ModelSpec) -> ModelSpec:
-    """Gemma-layout shape with the layer weights of a Duponex shape of equal layers; Flint-layout shape with the attention and
-    experts of a Rudorax shape."""
+    """Gemma-layout shape with the layer weights of a Duponex shape of equal layers or the mean layer weights of a Kabavik shape;
+    Flint-layout shape with the attention and experts of a Rudorax shape."""
     l = spec.layer_specs[0]
     if spec.arch == "rudorax":
         m = l.moe
@@ -34,10 +37,13 @@ def closest_spec(spec: ModelSpec) -> ModelSpec:
                          moe=MoeSpec(num_experts=m.num_experts, top_k=m.top_k, expert_ffn=m.expert_ffn, score="sigmoid", n_shared=1,
                                      shared_ffn=m.shared_ffn),
                          extra={"flint": {"window": l.window, "no_rope_layers": []}})
-    f = (l.heads * l.vdim + 2 * l.ffn) // 3 // 128 * 128
-    return ModelSpec(name=spec.name.replace("duponex", "gemma-layout"), arch="gemma", layers=spec.layers, hidden=spec.hidden,
+    f, window = (l.heads * l.vdim + 2 * l.ffn) // 3 // 128 * 128, l.chunk
+    if spec.arch == "kabavik":
+        f = (spec.run_params() // (spec.layers * spec.hidden) - 2 * (l.heads + l.kv_heads) * l.dim) // 3 // 128 * 128
+        window = l.window
+    return ModelSpec(name=spec.name.replace(spec.arch, "gemma-layout"), arch="gemma", layers=spec.layers, hidden=spec.hidden,
                      heads=l.heads, kv_heads=l.kv_heads, head_dim=l.dim, ffn=f, vocab=spec.vocab, qk_norm=True, swiglu_mode=2,
-                     rms_eps=spec.rms_eps, extra={"gemma": {"window": l.chunk, "global_every": spec.layers + 1}})
+                     rms_eps=spec.rms_eps, extra={"gemma": {"window": window, "global_every": spec.layers + 1}})
 
 
 def _device_ms(fn, n: int) -> float:
@@ -131,7 +137,7 @@ class _Pairs:
 def kernel_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> list[dict]:
     """One line per pair: the design's kernel and its like on ``rows`` rows (``rows`` <= 128: a decode step of that batch at
     context ``ctx``; more: prefill of rows / ctx prompts)."""
-    return {"duponex": _duponex_table, "rudorax": _rudorax_table}[spec.arch](spec, rows, ctx, iters, device)
+    return {"duponex": _duponex_table, "rudorax": _rudorax_table, "kabavik": _kabavik_table}[spec.arch](spec, rows, ctx, iters, device)
 
 
 def _duponex_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> list[dict]:
@@ -324,6 +330,125 @@ def _rudorax_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> 
         wv = rn(spec.vocab, W)
         pair("logits, 32-bit, soft cap", lambda: ops.softcap(ops.linear(x, wv, out_dtype=f32), 30.0), pair.gemm(spec.vocab, W, out_bytes=4), "logits",
              lambda: ops.linear(x, wv), pair.gemm(spec.vocab, W))
+    ops.check_status()
+    return pair.lines
+
+
+def _kabavik_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> list[dict]:
+    win, lat, cap = (next(l for l in spec.layer_specs if pick(l)) for pick in (lambda l: l.qk_norm == "row", lambda l: l.mixer == "latent", lambda l: l.softcap))
+    other = closest_spec(spec)
+    dev, bf, f32 = torch.device(device), torch.bfloat16, torch.float32
+    W, H, G, d, f, fo, side = spec.hidden, win.heads, win.kv_heads, win.dim, win.ffn, other.ffn, spec.side_dim
+    rn = lambda *s: torch.randn(*s, device=dev).to(bf)
+    fl = lambda *s: torch.randn(*s, device=dev)
+    i32 = lambda t: t.to(torch.int32)
+    decode = rows <= 128
+    pair = _Pairs(rows, iters, dev)
+    x = rn(rows, W)
+    nq = (H + 2 * G) * d
+    # projections
+    for name, n, k, like in (("qkv projection, bias", nq, W, "qkv projection"), ("output projection, bias", W, H * d, "output projection")):
+        w, b, r = rn(n, k), rn(n), x if k == W else rn(rows, k)
+        pair(name, lambda: ops.linear(r, w, bias=b), pair.gemm(n, k), like, lambda: ops.linear(r, w), pair.gemm(n, k))
+    wgu, wgo, h1, h2, wd, wdo = rn(2 * f, W), rn(2 * fo, W), rn(rows, f), rn(rows, fo), rn(W, f), rn(W, fo)
+    pair("gate/up projection, tanh-GELU", lambda: ops.linear_swiglu(x, wgu, mode=3), pair.gemm(2 * f, W, f), "gate/up projection, tanh-GELU",
+         lambda: ops.linear_swiglu(x, wgo, mode=2), pair.gemm(2 * fo, W, fo))
+    pair("down projection", lambda: ops.linear(h1, wd), pair.gemm(W, f), "down projection", lambda: ops.linear(h2, wdo), pair.gemm(W, fo))
+    del wgu, wgo, h1, h2, wd, wdo
+    # the residual between two sub-layers
+    xs, y, r16, w16, vec = fl(rows, W), rn(rows, W), rn(rows, W), rn(W), lambda: fl(W)
+    tanh = lambda: residual_ops.Norm("tanh", vec(), vec(), 0.7)
+    n1, n2, n3, copy = tanh(), tanh(), residual_ops.Norm("rms", vec()), residual_ops.Norm()
+
+    def like_step():
+        ops.add_rmsnorm(ops.rmsnorm(y, w16, 1e-5), r16, w16, 1e-5)
+    for name, a, b in (("residual step, two tanh norms", n1, n2), ("residual step, tanh norm and copy", n1, copy), ("residual step, RMS and tanh norm", n3, n2)):
+        pair(name, lambda: residual_ops.add_normed(xs, y, a, b, 1e-5, W), (rows * W * 12, 0), "norm, add + norm", like_step, (rows * W * 12, 0))
+    tok, tab = i32(torch.randint(0, 1024, (rows,), device=dev)), rn(1024, W)
+    pair("embed + norm", lambda: residual_ops.embed_normed(tok, tab, 2.0, n1, 1e-5, W), (rows * W * 8, 0), "embed + norm",
+         lambda: ops.embed_rmsnorm(tok, tab, w16, 1e-5), (rows * W * 6, 0))
+    # token input
+    wg, wp, es, g1 = rn(side, W), rn(W, side), rn(1024, 4 * side), rn(rows, side)
+    cost = pair.gemm(side, W)
+    pair("token gate, tanh-GELU, factors", lambda: ops.linear(x, wg, act="gelu_tanh", mul=(es[:, side: 2 * side], tok)), (cost[0] + 2 * rows * side, cost[1]),
+         "projection of that size", lambda: ops.linear(x, wg), cost)
+    pair("token projection", lambda: ops.linear(g1, wp), pair.gemm(W, side), "projection of that size", lambda: ops.linear(g1, wp), pair.gemm(W, side))
+    del xs, tab, es
+    # norms, rotation and cache write
+    batch = rows if decode else rows // ctx
+    pg = _Paged(batch, ctx, G, d, dev)
+    slots, pos = i32(torch.randperm(pg.k.shape[0] * 64, device=dev)[:rows]), i32(torch.arange(rows, device=dev)) % ctx
+    qkv, qn, kn, wq, wk = rn(rows, nq), rn(d), rn(d), fl(H * d), fl(G * d)
+    freqs, amp = win.rope.frequencies()
+    table = ops.rope_angles(pos, ops.rope_frequencies(freqs, dev), amp)
+
+    def like_norm_rope():
+        q, k = qkv[:, : H * d].reshape(rows * H, d), qkv[:, H * d: (H + G) * d].reshape(rows * G, d)
+        qkv[:, : H * d] = ops.rmsnorm(q.contiguous(), qn, 1e-5).view(rows, -1)
+        qkv[:, H * d: (H + G) * d] = ops.rmsnorm(k.contiguous(), kn, 1e-5).view(rows, -1)
+        ops.rope_kv_paged(qkv, pos, slots, pg.k, pg.v, H, G, d, 1e4)
+    byts = (2 * rows * d * (2 * H + 4 * G), 0)
+    pair("row norms, rotation + cache write", lambda: ops.head_norm_kv(qkv, slots, pg.k, pg.v, H, G, d, d, 1e-5, q_weight=wq, k_weight=wk, cos_sin=table,
+         whole=True, halves=True), byts, "head norms, rotation + cache write", like_norm_rope, byts)
+    pair("head norms, temperature + cache write", lambda: ops.head_norm_kv(qkv, slots, pg.k, pg.v, H, G, d, d, 1e-5, q_weight=wq[:d], k_weight=wk[:d],
+         temp=(pos, *cap.q_temp)), byts, "head norms, rotation + cache write", like_norm_rope, byts)
+    # attention
+    qs, ql = (i32(torch.arange(batch, device=dev) * (rows // batch)), torch.full((batch,), rows // batch, dtype=torch.int32, device=dev))
+    seen = lambda l: batch * (l.keys_seen(ctx) if decode else l.pairs_seen(ctx))       # (query, key) pairs
+
+    def cost(l, kv_width, pairs, q_width, flop_width):
+        keys = rows * l.keys_seen(ctx) if decode else rows
+        return 2 * (keys * kv_width + rows * H * q_width), 2 * pairs * H * flop_width
+    plain = dataclasses.replace(win, keep_first=0)
+    full = dataclasses.replace(win, window=0)
+    for name, l, like_name, like in (("attention, window + kept positions", win, "attention, window", plain),
+                                     ("attention, capped scores", cap, "attention, full", full)):
+        def at(z):
+            kw = dict(window=z.window, keep=z.keep_first if z.window else 0, softcap=z.softcap)
+            if decode:
+                return ops.attn_decode(qkv, pg.k, pg.v, pg.table, pg.ctx, H, G, d, l.scale, max_ctx=ctx, **kw)
+            return ops.attn_prefill(qkv, pg.k, pg.v, pg.table, qs, ql, pg.ctx, ctx, H, G, d, l.scale, **kw)
+        pair(name, lambda: at(l), cost(l, 2 * G * d, seen(l), 2 * d, 2 * d), like_name, lambda: at(like), cost(like, 2 * G * d, seen(like), 2 * d, 2 * d))
+    del pg, qkv
+    # latent attention
+    R, T = lat.rank_pad, lat.rot_pad
+    n = lat.projection_cols
+    w = rn(n, W)
+    pair("latent projection", lambda: ops.linear(x, w), pair.gemm(n, W), "projection of that size", lambda: ops.linear(x, w), pair.gemm(n, W))
+    p, wn = rn(rows, n), fl(R)
+    lg = _Paged(batch, ctx, 1, R + T, dev)
+    lfreqs, lamp = lat.rope.frequencies()
+    ltab = ops.rope_angles(pos, ops.rope_frequencies(lfreqs, dev), lamp)
+    q = torch.empty(rows, H, R + T, dtype=bf, device=dev)
+    rot, at0 = H * d, H * (d + T)
+    byts = (2 * rows * (2 * H * T + 2 * (R + T)), 0)
+
+    def like_latent():
+        c = ops.rmsnorm(p[:, at0: at0 + R].contiguous(), w16[:R].contiguous(), 1e-5)
+        kr, qr = p[:, at0 + R: at0 + R + T].contiguous(), p[:, rot: at0].contiguous()
+        ops.rope_inplace(qr, pos, H, T, 1e4)
+        ops.rope_inplace(kr, pos, 1, T, 1e4)
+        mla_ops.cache_write(c, kr, slots, lg.k)
+    pair("latent norm, rotations + cache write", lambda: mla_ops.latent_norm_kv(p, slots, lg.k, q, rot, at0, R, R, wn, ltab, 1e-5), byts,
+         "norm, rotations, cache write", like_latent, byts)
+    uk, uv, out = rn(H, R, d), rn(H, d, R), rn(rows, H * R)
+    per_head = lambda a, b: (2 * (rows * H * (a + b) + H * a * b), 2 * rows * H * a * b)
+    xq = p[:, :rot]
+    pair("queries into the latent space", lambda: ops.head_linear(xq, uk, out=q.view(rows, -1), out_cols=R + T), per_head(d, R), "per-head projection",
+         lambda: mla_ops.per_head_linear(xq.reshape(rows, H, d), uk), per_head(d, R))
+    pair("results out of the latent space", lambda: ops.head_linear(out, uv), per_head(R, d), "per-head projection",
+         lambda: mla_ops.per_head_linear(out.view(rows, H, R), uv), per_head(R, d))
+    q.normal_()
+    gate = p[:, at0 + R + T: at0 + R + T + H]
+    unbound = dataclasses.replace(lat, window=0)
+    lc = lambda l: cost(l, R + T, seen(l), 2 * R + T, 2 * R + T)
+    pair("latent attention, window, gated", lambda: mla_ops.latent_attention(q, lg.k, lg.table, qs, ql, lg.ctx, rows // batch, ctx, lat.scale, R, lat.window, gate,
+         out, decode=decode), lc(lat), "latent attention, full", lambda: mla_ops.attention(q, lg.k, lg.table, qs, ql, lg.ctx, rows // batch, ctx, lat.scale, R),
+         lc(unbound))
+    if decode:
+        wv = rn(spec.vocab, W)
+        pair("logits, 32-bit", lambda: ops.linear(x, wv, out_dtype=f32), pair.gemm(spec.vocab, W, out_bytes=4), "logits", lambda: ops.linear(x, wv),
+             pair.gemm(spec.vocab, W))
     ops.check_status()
     return pair.lines
 
