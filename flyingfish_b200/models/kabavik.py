@@ -9,9 +9,10 @@ token input per layer, all on an FP32 residual.
   i + half); a query sees its last ``window`` positions and the first ``keep_first`` of the sequence. A layer may read the keys and
   values another layer cached; it then projects queries alone.
 * Full attention: q and k are normed per head, nothing rotates, the query grows with the logarithm of its position, scores are capped.
-* Latent attention, in the absorbed form: a token caches its normed latent and one rotated key part; a head's query goes through its
-  key matrix into the latent space (``ops.head_linear``), all heads attend to the one cached row, and the result leaves through the
-  head's value matrix. A head's result is multiplied by a gate that the attention kernel applies.
+* Latent attention: a token caches its normed latent and one rotated key part. Decoded tokens and narrow latents take the absorbed form:
+  a head's query goes through its key matrix into the latent space (``ops.head_linear``), all heads attend to the one cached row, and
+  the result leaves through the head's value matrix. Portions over wide latents expand the visible rows to keys and values first
+  (``mla_ops.expanded_attention``). A head's result is multiplied by a gate that the attention kernels apply.
 * The norm behind a sub-layer, the sum and the norm in front of the next one are one kernel (``ops.residual_ops.add_normed``); the residual
   factor is part of the weights of the norms behind, the logits' factor of the final norm. The feed-forward's activation and the
   token input's activation and product are GEMM epilogues.
@@ -116,10 +117,11 @@ def build_weights(spec: ModelSpec, source: TensorSource) -> ModelWeights:
                                  _pad_rows(down[: l.kv_rank], rp), _pad_rows(down[l.kv_rank:], tp),
                                  _pad_rows(pad_cols(get(p + "g"), wp), pad_to(l.heads, 8))]).contiguous()
             lw.extra["latent_norm"] = pad_cols(get(p + "dkv.norm").float(), rp).contiguous()
-            # [heads, rank_pad, dim_pad]: a head's unrotated query into the latent space; [heads, vdim_pad, rank_pad]: its result out of it
-            up = pad_heads(pad_cols(get(p + "uk"), rp), l.heads, l.dim, dk).view(l.heads, dk, rp)
-            lw.extra["w_uk"] = up.transpose(1, 2).contiguous()
-            lw.extra["w_uv"] = pad_heads(pad_cols(get(p + "uv"), rp), l.heads, l.vdim, dv).view(l.heads, dv, rp).contiguous()
+            # all key matrices, then all value matrices; a head's unrotated query goes into the latent space through [rank_pad, dim_pad]
+            # and its result out of it through [vdim_pad, rank_pad]
+            up = pad_heads(pad_cols(get(p + "uk"), rp), l.heads, l.dim, dk)
+            lw.extra["w_kv"] = torch.cat([up, pad_heads(pad_cols(get(p + "uv"), rp), l.heads, l.vdim, dv)]).contiguous()
+            lw.extra["w_uk"] = up.view(l.heads, dk, rp).transpose(1, 2).contiguous()
         else:
             parts = [("q", l.heads, l.dim, dk)] + ([("k", l.kv_heads, l.dim, dk), ("v", l.kv_heads, l.vdim, dv)] if l.kv_from < 0 else [])
             lw.wqkv = torch.cat([rows_in(p + n, *s) for n, *s in parts]).contiguous()
@@ -219,23 +221,42 @@ class KabavikModel(DecoderModel):
         return out
 
     def _latent_layer(self, i: int, l: LayerSpec, lw: LayerWeights, n: torch.Tensor, b, kv, table) -> torch.Tensor:
-        dk, rp, tp = l.dim_pad, l.rank_pad, l.rot_pad
+        dk, dv, rp, tp = l.dim_pad, l.vdim_pad, l.rank_pad, l.rot_pad
         p = ops.linear(n, lw.wqkv)
         rot, lat = l.heads * dk, l.heads * (dk + tp)
         q = torch.empty(b.rows, l.heads, rp + tp, dtype=p.dtype, device=p.device)
         mla_ops.latent_norm_kv(p, b.slots, kv.k[i], q, rot, lat, l.kv_rank, rp, lw.extra["latent_norm"], table, self.spec.rms_eps)
-        ops.head_linear(p[:, :rot], lw.extra["w_uk"], out=q.view(b.rows, -1), out_cols=rp + tp)
         gate = p[:, lat + rp + tp: lat + rp + tp + l.heads]
-        out = torch.empty(b.rows, l.heads * rp, dtype=p.dtype, device=p.device)
+        out = torch.empty(b.rows, l.heads * dv, dtype=p.dtype, device=p.device)
         s, rows = self._split(b)
-        if s:
+        pages = self._key_pages(b, s, l.window, kv) if s and mla_ops.expands(p, rp + tp, dk, tp, dv, b.max_q_len) else None
+        first = 0                                                     # first row of the absorbed form
+        if pages is not None:
+            mla_ops.expanded_attention(p[:rows, :rot], q[:rows], kv.k[i], lw.extra["w_kv"], pages, b.block_table[:s], b.q_start[:s], b.q_lens[:s],
+                                       b.ctx_lens[:s], b.max_q_len, dk, dv, rp, l.scale, l.window, gate[:rows], out[:rows])
+            first = rows
+        if first == b.rows:
+            return out
+        ops.head_linear(p[first:, :rot], lw.extra["w_uk"], out=q[first:].view(b.rows - first, -1), out_cols=rp + tp)
+        a = torch.empty(b.rows - first, l.heads * rp, dtype=p.dtype, device=p.device)
+        if s and pages is None:
             mla_ops.latent_attention(q[:rows], kv.k[i], b.block_table[:s], b.q_start[:s], b.q_lens[:s], b.ctx_lens[:s], b.max_q_len, b.max_ctx, l.scale,
-                                     rp, l.window, gate[:rows], out[:rows])
+                                     rp, l.window, gate[:rows], a[:rows])
         if s < b.batch:
             starts = b.q_start if b.is_decode else b.q_start[s:] - rows
             mla_ops.latent_attention(q[rows:], kv.k[i], b.block_table[s:], starts, b.q_lens[s:], b.ctx_lens[s:], b.nq if b.is_decode else 1,
-                                     b.max_ctx, l.scale, rp, l.window, gate[rows:], out[rows:], decode=True)
-        return ops.head_linear(out, lw.extra["w_uv"])
+                                     b.max_ctx, l.scale, rp, l.window, gate[rows:], a[rows - first:], decode=True)
+        ops.head_linear(a, lw.extra["w_kv"][l.heads * dk:].view(l.heads, dv, rp), out=out[first:])
+        return out
+
+    def _key_pages(self, b, s: int, window: int, kv):
+        """Pages the portions of this step see through ``window`` (one list for all layers with that window)."""
+        if window not in self._pages:
+            L, h = b.layout, b.host
+            table = h[L.block_table: L.block_table + L.max_batch * L.max_blocks].view(L.max_batch, L.max_blocks)[:s]
+            self._pages[window] = mla_ops.KeyPages.of(h[L.q_lens: L.q_lens + s].tolist(), h[L.ctx_lens: L.ctx_lens + s].tolist(), table, window,
+                                                      kv.block_size, b.device)
+        return self._pages[window]
 
     # -- forward -----------------------------------------------------------------------------
     def hidden_states(self, b, kv, inputs_embeds=None):
@@ -243,6 +264,7 @@ class KabavikModel(DecoderModel):
         assert b.tree_mask is None, "tree verification is not available with capped scores or latent attention"
         w, spec, eps = self.w, self.spec, self.spec.rms_eps
         side, sp = w.extra.get("side_embed"), pad_to(spec.side_dim, 8)
+        self._pages = {}                                              # expanded pages of this step, per window
         tables = [ops.rope_angles(b.positions, f, amp) for f, amp in self.rotations]
         norms = [lw.extra["norms"] for lw in w.layers]
         add = lambda y, behind, front: residual_ops.add_normed(x, y, behind, front, eps, self.width)

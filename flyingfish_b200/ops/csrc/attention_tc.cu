@@ -363,20 +363,61 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 constexpr int T2_BN = 64;                                          // keys per tile = one cache page
 constexpr int T2_KV_BYTES = T2_BN * TC_HD * 2;                     // 16 KiB
 constexpr int TC2_SMEM = TC_Q_BYTES + 4 * T2_KV_BYTES + 1024;      // 97 KiB
+constexpr int LAT_SMEM = 3 * (16384 + 2 * 8192) + 2 * T2_KV_BYTES + 1024;      // latent form: three 64-column blocks of Q and K, 129 KiB
 
 // what a launch adds to plain causal attention over 128-wide heads
 struct PrefillForm {
   int window, chunk, causal, dk, dv;
   int gated;                       // the result is multiplied by the sigmoid of a [rows, hq * dv] gate (tensor map tmG)
   int keep;                        // with a window: the first `keep` positions stay visible
-  float cap_in, cap_out;           // CAP: score s becomes cap tanh(s / cap); cap_in = 2 log2(e) scale / cap, cap_out = -2 log2(e) cap
+  float cap_in;                    // CAP: score s becomes cap tanh(s / cap); cap_in = scale / cap
   const __nv_bfloat16* head_gate;  // the result of head h is multiplied by the sigmoid of head_gate[row * ldhg + h]
   int ldhg;
+  // LAT: keys and values expanded from latents. The maps of K and V are over expanded rows [key rows, heads * dk | heads * dv]; page t of
+  // sequence b is at key row (exp_off[b] + t) * 64. The last dr elements of queries and keys come from maps of their own: tmG, rows with
+  // head h at column h * qr_pitch + qr_col, and tmR, the cache's rows, at column kr_col.
+  const int* exp_off;
+  int dr, qr_pitch, qr_col, kr_col;
 };
 
-// cap tanh(s / cap) up to the constant cap, which soft-max does not see, in log2 units: -2 cap / (1 + e^(2 s / cap))
-__device__ __forceinline__ float capped_log2(float s, float cap_in, float cap_out) {
-  return __fdividef(cap_out, 1.0f + ex2_approx(fminf(s * cap_in, 100.0f)));
+// Capped scores. N raw products of a thread become tanh(y), y = s cap_in; the cap is the factor of the exponent. Where all |y| of the
+// warp are at most 1 -- the usual case, caps being there for outliers -- tanh is a polynomial, two values per instruction, which
+// leaves the special-function unit to the soft-max: y times a Chebyshev fit of tanh(y) / y in y^2 on [0, 1], error 5.5e-7.
+// Otherwise 1 - 2 / (1 + e^(2y)).
+__device__ __forceinline__ uint64_t f2_pack(float a, float b) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
+__device__ __forceinline__ void f2_unpack(uint64_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ uint64_t f2_mul(uint64_t a, uint64_t b) { uint64_t r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+__device__ __forceinline__ uint64_t f2_fma(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+template <int N>
+__device__ __forceinline__ void cap_scores(float (&sv)[N], float cap_in) {
+  float am[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < N; ++i) am[i & 3] = fmaxf(am[i & 3], fabsf(sv[i]));
+  const float most = fmaxf(fmaxf(am[0], am[1]), fmaxf(am[2], am[3]));
+  if (__all_sync(0xffffffffu, most * cap_in <= 1.0f)) {
+    const uint64_t c = f2_pack(cap_in, cap_in);
+    auto k = [](float v) { return f2_pack(v, v); };
+    const uint64_t k0 = k(0.999999463558197f), k1 = k(-0.33329179883003235f), k2 = k(0.13282513618469238f), k3 = k(-0.05163545906543732f),
+                   k4 = k(0.01677677594125271f), k5 = k(-0.0030804092530161142f);
+#pragma unroll
+    for (int i = 0; i < N; i += 2) {
+      const uint64_t y = f2_mul(f2_pack(sv[i], sv[i + 1]), c), z = f2_mul(y, y);
+      uint64_t r = f2_fma(k5, z, k4);
+      r = f2_fma(r, z, k3);
+      r = f2_fma(r, z, k2);
+      r = f2_fma(r, z, k1);
+      r = f2_fma(r, z, k0);
+      f2_unpack(f2_mul(y, r), sv[i], sv[i + 1]);
+    }
+  } else {
+    const float e = 2.0f * 1.4426950408889634f * cap_in;
+#pragma unroll
+    for (int i = 0; i < N; ++i) sv[i] = 1.0f - __fdividef(2.0f, 1.0f + ex2_approx(fminf(sv[i] * e, 100.0f)));
+  }
 }
 
 // o * inv, times the sigmoid of the gate where there is one (`gate`: the row of a swizzled gate tile in shared memory, `sw` =
@@ -410,12 +451,13 @@ struct alignas(8) Tc2Bars {
 };
 
 // WIDE: heads are exactly 128 wide; EXTRA: the launch may have a block-local mask, kept first positions or a gate (plain launches keep
-// an instance with none of them); CAP: scores are capped.
-template <int SPLIT, bool WIDE, bool EXTRA, bool CAP>
-__global__ void __launch_bounds__(64 + 128 * SPLIT, 2)
+// an instance with none of them); CAP: scores are capped; LAT: latent attention over expanded keys and values, heads of up to 128 + 64
+// elements (one CTA per SM).
+template <int SPLIT, bool WIDE, bool EXTRA, bool CAP, bool LAT = false>
+__global__ void __launch_bounds__(64 + 128 * SPLIT, LAT ? 1 : 2)
 attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                        const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmG, const int* __restrict__ block_table,
-                        const int* __restrict__ q_start, const int* __restrict__ q_lens,
+                        const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmG, const __grid_constant__ CUtensorMap tmR,
+                        const int* __restrict__ block_table, const int* __restrict__ q_start, const int* __restrict__ q_lens,
                         const int* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out, int hq, int hkv, int ldo,
                         int max_blocks, int num_blocks, float scale_log2, const PrefillForm f, int* status,
                         const float* __restrict__ sinks) {
@@ -426,9 +468,11 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   extern __shared__ uint8_t smem_raw[];
   __shared__ Tc2Bars bars;
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  constexpr int BLOCKS = LAT ? 3 : 2;                              // 64-column blocks of a Q and a K tile
+  constexpr int K_BYTES = BLOCKS * 8192;
   uint8_t* sQ = smem;
-  uint8_t* sK = smem + TC_Q_BYTES;                                 // two K tiles, then two V tiles
-  uint8_t* sV = sK + 2 * T2_KV_BYTES;
+  uint8_t* sK = smem + BLOCKS * 16384;                             // two K tiles, then two V tiles
+  uint8_t* sV = sK + 2 * K_BYTES;
   const int ctx = ctx_lens[b], qs = q_start[b];
   const int kvh = h / (hq / hkv);
   const int past = ctx - qlen;
@@ -467,8 +511,9 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 
   if (warp == 0) {
     if (lane == 0) {
-      mbar_expect_tx(&bars.q_full, k_hi ? TC_Q_BYTES : TC_Q_BYTES / 2);
+      mbar_expect_tx(&bars.q_full, (k_hi ? TC_Q_BYTES : TC_Q_BYTES / 2) + (LAT ? 16384 : 0));
       tma_load_2d(sQ, &tmQ, &bars.q_full, h * dk, qs + r0);
+      if (LAT) tma_load_2d(sQ + 2 * TC_BM * 128, &tmG, &bars.q_full, h * f.qr_pitch + f.qr_col, qs + r0);
       if (k_hi) tma_load_2d(sQ + TC_BM * 128, &tmQ, &bars.q_full, h * dk + 64, qs + r0);
       bool ok = true, bad = false;
       const int nblk = (ctx + TC_PAGE - 1) / TC_PAGE;
@@ -477,28 +522,31 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         if (page >= nblk) page = nblk - 1;                   // past the context: any valid page, its keys are masked
         int blk = block_table[(size_t)b * max_blocks + page];
         if (blk < 0 || blk >= num_blocks) { bad = true; blk = 0; }
-        return (blk * hkv + kvh) * TC_PAGE;
+        return (blk * hkv + (LAT ? 0 : kvh)) * TC_PAGE;
       };
+      const int exp0 = LAT ? f.exp_off[b] : 0;
       // a tile: block d0 = [64 keys x 64 d] (8 KiB), then block d1. K runs one tile ahead of V: K(j + 1) is free once
       // Q K(j - 1) has run, V(j) only once P V(j - 2) has.
       auto load_k = [&](int j) -> bool {
         const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
         const int row = tile_row(j);
         if (!mbar_wait(&bars.k_empty[st], ph ^ 1, abort_flag, status, KID_ATTN_PREFILL, 21)) return false;
-        mbar_expect_tx(&bars.k_full[st], k_hi ? T2_KV_BYTES : T2_KV_BYTES / 2);
-        tma_load_2d(sK + st * T2_KV_BYTES, &tmK, &bars.k_full[st], 0, row);
-        if (k_hi) tma_load_2d(sK + st * T2_KV_BYTES + 8192, &tmK, &bars.k_full[st], 64, row);
+        mbar_expect_tx(&bars.k_full[st], (k_hi ? T2_KV_BYTES : T2_KV_BYTES / 2) + (LAT ? 8192 : 0));
+        const int kx = LAT ? h * dk : 0, ky = LAT ? (exp0 + tile_page(j)) * TC_PAGE : row;
+        tma_load_2d(sK + st * K_BYTES, &tmK, &bars.k_full[st], kx, ky);
+        if (k_hi) tma_load_2d(sK + st * K_BYTES + 8192, &tmK, &bars.k_full[st], kx + 64, ky);
+        if (LAT) tma_load_2d(sK + st * K_BYTES + 16384, &tmR, &bars.k_full[st], f.kr_col, row);
         return true;
       };
       ok = load_k(0);
       for (int j = 0; j < ntiles && ok; ++j) {
         if (j + 1 < ntiles && !load_k(j + 1)) { ok = false; break; }
         const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
-        const int row = tile_row(j);
+        const int row = LAT ? (exp0 + tile_page(j)) * TC_PAGE : tile_row(j), vx = LAT ? h * dv : 0;
         if (!mbar_wait(&bars.v_empty[st], ph ^ 1, abort_flag, status, KID_ATTN_PREFILL, 22)) { ok = false; break; }
         mbar_expect_tx(&bars.v_full[st], v_hi ? T2_KV_BYTES : T2_KV_BYTES / 2);
-        tma_load_2d(sV + st * T2_KV_BYTES, &tmV, &bars.v_full[st], 0, row);
-        if (v_hi) tma_load_2d(sV + st * T2_KV_BYTES + 8192, &tmV, &bars.v_full[st], 64, row);
+        tma_load_2d(sV + st * T2_KV_BYTES, &tmV, &bars.v_full[st], vx, row);
+        if (v_hi) tma_load_2d(sV + st * T2_KV_BYTES + 8192, &tmV, &bars.v_full[st], vx + 64, row);
       }
       if (ok && gated) {
         // the gate tile takes the place of Q once the last Q Kᵀ has read it; it arrives under the last soft-max and P V
@@ -524,13 +572,22 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         // this S buffer still holds the P of tile j - 2: that tile's P V has to be complete
         if (j >= 2 && !mbar_wait(&bars.pv_done[st], ph ^ 1, abort_flag, status, KID_ATTN_PREFILL, 25)) return false;
         tc_fence_after();
-        const uint32_t k_addr = smem_u32(sK + st * T2_KV_BYTES);
+        const uint32_t k_addr = smem_u32(sK + st * K_BYTES);
+        if (LAT) {
+          const int rsteps = f.dr >> 4;
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            if (k >= rsteps) break;
+            umma_f16(tmem_s + st * T2_BN, umma_desc_sw128(q_addr + 2 * 16384 + k * 32, 16, 1024), umma_desc_sw128(k_addr + 2 * 8192 + k * 32, 16, 1024),
+                     idesc_s, k != 0);
+          }
+        }
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
           if (k >= ksteps) break;
           // Q: 64-column block k / 4 of a 128-row tile (16 KiB), 32 bytes per k-step; K: the same with 64 rows (8 KiB)
           umma_f16(tmem_s + st * T2_BN, umma_desc_sw128(q_addr + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024),
-                   umma_desc_sw128(k_addr + (k >> 2) * 8192 + (k & 3) * 32, 16, 1024), idesc_s, k != 0);
+                   umma_desc_sw128(k_addr + (k >> 2) * 8192 + (k & 3) * 32, 16, 1024), idesc_s, LAT || k != 0);
         }
         umma_commit(&bars.s_full[st]);
         umma_commit(&bars.k_empty[st]);
@@ -587,10 +644,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
           for (int i = 0; i < HB; ++i) sv[i] = __uint_as_float(r[i]);
         }
         const int tile0 = tile_page(j) * T2_BN, k0 = tile0 + hf * HB;
-        if (CAP) {
-#pragma unroll
-          for (int i = 0; i < HB; ++i) sv[i] = capped_log2(sv[i], f.cap_in, f.cap_out);
-        }
+        if (CAP) cap_scores<HB>(sv, f.cap_in);
         float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
         if ((tile0 >= tile_lo_max || (EXTRA && tile0 + T2_BN <= keep)) && tile0 + T2_BN - 1 <= tile_hi_min) {
 #pragma unroll
@@ -604,8 +658,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             mx4[i & 3] = fmaxf(mx4[i & 3], t);
           }
         }
-        mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-        if (!CAP) mx *= scale_log2;
+        mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
       }
       if (SPLIT == 2) {
         // after this barrier both warps of the pair hold their S columns in registers: P may overwrite S
@@ -648,8 +701,8 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
           uint32_t pk[16];
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
-            const float p0 = ex2_approx(CAP ? sv[2 * (c + i)] - mr : fmaf(sv[2 * (c + i)], scale_log2, -mr));
-            const float p1 = ex2_approx(CAP ? sv[2 * (c + i) + 1] - mr : fmaf(sv[2 * (c + i) + 1], scale_log2, -mr));
+            const float p0 = ex2_approx(fmaf(sv[2 * (c + i)], scale_log2, -mr));
+            const float p1 = ex2_approx(fmaf(sv[2 * (c + i) + 1], scale_log2, -mr));
             pk[i] = pack_bf16x2(p0, p1);
             ls4[i & 3] += p0 + p1;
           }
@@ -728,10 +781,10 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
   const uint64_t cache_rows = (uint64_t)num_blocks * hkv * TC_PAGE;
   if (int r = make_tmap_2d(&tmK, kcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dk, cache_rows, dk * 2, 64, TC_PAGE)) return r;
   if (int r = make_tmap_2d(&tmV, vcache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, dv, cache_rows, (uint64_t)ldv * 2, 64, TC_PAGE)) return r;
-  const float scale_log2 = scale * 1.4426950408889634f;
+  const float scale_log2 = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f;
   dim3 grid((max_q_len + TC_BM - 1) / TC_BM, hq, batch);
   const PrefillForm f = {window < 0 ? 0 : window, chunk, window < 0 ? 0 : 1, dk, dv, gate != nullptr ? 1 : 0, window > 0 ? keep : 0,
-                         softcap > 0.f ? 2.0f * scale_log2 / softcap : 0.f, -2.0f * 1.4426950408889634f * softcap, (const __nv_bfloat16*)head_gate, ldhg};
+                         softcap > 0.f ? scale / softcap : 0.f, (const __nv_bfloat16*)head_gate, ldhg, nullptr, 0, 0, 0, 0};
   CUtensorMap tmG = tmQ;
   if (gate != nullptr)
     if (int r = make_tmap_2d(&tmG, gate, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)hq * dv, (uint64_t)total_rows, (uint64_t)ldg * 2, 64, TC_BM)) return r;
@@ -746,7 +799,7 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
     if (split < 0) { const char* e = getenv("FF_ATTN_PREFILL_SPLIT"); split = (e != nullptr && (e[0] == '1' || e[0] == '2')) ? e[0] - '0' : TC2_SPLIT_DEFAULT; }
     auto go = [&](auto kern, int threads) -> int {
       if (int r = opt_in_smem(kern, TC2_SMEM)) return r;
-      kern<<<grid, threads, TC2_SMEM, s>>>(tmQ, tmK, tmV, tmG, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out, hq, hkv, ldo,
+      kern<<<grid, threads, TC2_SMEM, s>>>(tmQ, tmK, tmV, tmG, tmQ, block_table, q_start, q_lens, ctx_lens, (__nv_bfloat16*)out, hq, hkv, ldo,
                                            max_blocks, num_blocks, scale_log2, f, status, sinks);
       return launch_result();
     };
@@ -759,5 +812,37 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
   attn_prefill_tc_kernel<<<grid, 320, TC_SMEM, s>>>(tmQ, tmK, tmV, block_table, q_start, q_lens, ctx_lens,
                                                     (__nv_bfloat16*)out, hq, hkv, ldo, max_blocks, num_blocks, scale_log2,
                                                     f.window, f.causal, status, sinks);
+  return launch_result();
+}
+
+// Latent attention over keys and values expanded from the latents (prefill; one product of all heads' matrices with the rows the queries
+// can see): head h's key is [expanded key (dk) | rotated key of the cache row (dr)]. q: rows [rows, ldq] with head h's unrotated part at
+// column h * dk; q_rot: rows of heads * qr_pitch columns with its rotated part at h * qr_pitch + qr_col; expanded: [exp_rows, lde], head
+// h's key at column h * dk and its value at hq * dk + h * dv; page t of sequence b starts at row (exp_off[b] + t) * 64; cache:
+// [num_blocks, 1, 64, cache_width] with the rotated key at column kr_col. out [rows, ldo]. dk, dv multiples of 16 up to 128, dr up to 64.
+FF_EXPORT int ff_attn_prefill_latent(const void* q, const void* q_rot, const void* expanded, const void* cache, const int* block_table,
+                                     const int* q_start, const int* q_lens, const int* ctx_lens, const int* exp_off, void* out, int batch,
+                                     int total_rows, int max_q_len, int hq, int dk, int dr, int dv, int ldq, int qr_pitch, int qr_col, int lde,
+                                     int exp_rows, int cache_width, int kr_col, int ldo, int max_blocks, int num_blocks, float scale, int window,
+                                     const void* head_gate, int ldhg, int* status, cudaStream_t s) {
+  if (batch <= 0 || max_q_len <= 0 || hq <= 0 || total_rows <= 0 || exp_rows <= 0 || window < 0 || !(scale > 0.f)) return FF_HOST_BAD_SHAPE;
+  if (dk < 16 || dk > TC_HD || dk % 16 || dv < 16 || dv > TC_HD || dv % 16 || dr < 16 || dr > 64 || dr % 16) return FF_HOST_BAD_SHAPE;
+  if (ldq < hq * dk || lde < hq * (dk + dv) || qr_pitch < qr_col + dr || cache_width < kr_col + dr || exp_off == nullptr) return FF_HOST_BAD_SHAPE;
+  if (ldq % 8 || lde % 8 || qr_pitch % 8 || qr_col % 8 || cache_width % 8 || kr_col % 8 || ldo % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return FF_HOST_BAD_ALIGN;
+  constexpr auto BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  CUtensorMap tmQ, tmG, tmK, tmV, tmR;
+  if (int r = make_tmap_2d(&tmQ, q, BF, 2, (uint64_t)hq * dk, total_rows, (uint64_t)ldq * 2, 64, TC_BM)) return r;
+  if (int r = make_tmap_2d(&tmG, q_rot, BF, 2, (uint64_t)hq * qr_pitch, total_rows, (uint64_t)hq * qr_pitch * 2, 64, TC_BM)) return r;
+  if (int r = make_tmap_2d(&tmK, expanded, BF, 2, (uint64_t)hq * dk, exp_rows, (uint64_t)lde * 2, 64, TC_PAGE)) return r;
+  const __nv_bfloat16* values = (const __nv_bfloat16*)expanded + (size_t)hq * dk;
+  if (int r = make_tmap_2d(&tmV, values, BF, 2, (uint64_t)hq * dv, exp_rows, (uint64_t)lde * 2, 64, TC_PAGE)) return r;
+  if (int r = make_tmap_2d(&tmR, cache, BF, 2, cache_width, (uint64_t)num_blocks * TC_PAGE, (uint64_t)cache_width * 2, 64, TC_PAGE)) return r;
+  PrefillForm f = {};
+  f.window = window; f.causal = 1; f.dk = dk; f.dv = dv; f.head_gate = (const __nv_bfloat16*)head_gate; f.ldhg = ldhg;
+  f.exp_off = exp_off; f.dr = dr; f.qr_pitch = qr_pitch; f.qr_col = qr_col; f.kr_col = kr_col;
+  auto kern = dk == TC_HD && dv == TC_HD ? attn_prefill_tc2_kernel<2, true, true, false, true> : attn_prefill_tc2_kernel<2, false, true, false, true>;
+  if (int r = opt_in_smem(kern, LAT_SMEM)) return r;
+  kern<<<dim3((max_q_len + TC_BM - 1) / TC_BM, hq, batch), 320, LAT_SMEM, s>>>(tmQ, tmK, tmV, tmG, tmR, block_table, q_start, q_lens, ctx_lens,
+      (__nv_bfloat16*)out, hq, 1, ldo, max_blocks, num_blocks, scale * 1.4426950408889634f, f, status, nullptr);
   return launch_result();
 }

@@ -151,7 +151,8 @@ static int head_norm_launch(void* qkv, const int* slots, void* kcache, void* vca
 // What row_norm_kv adds: norms over whole projections (weights then cover all heads), pairs (i, i + half).
 struct RowForm { int whole, halves; };
 
-template <typename T>
+// VEC: halves turn and half is a multiple of 8
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(HN_THREADS)
 row_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __restrict__ kcache, T* __restrict__ vcache, int hq, int hkv, int dim,
                    int dk, int dv, int block_size, int num_blocks, int ld, float eps, const float* __restrict__ wq, const float* __restrict__ wk,
@@ -198,9 +199,9 @@ row_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __rest
   if (slot >= 0 && !cached && tid == 0) set_status(status, KID_ROPE_KV, FF_ERR_BOUNDS, row, slot);
   const float tf = query_factor(temp, row);
   const float2* tab = cos_sin != nullptr ? cos_sin + (size_t)row * half : nullptr;
-  const int dims = tab != nullptr ? 2 * half : 0;
+  const int dims = tab != nullptr ? 2 * half : 0, vph = dk / 8;
   for (int i = tid; i < nvec; i += HN_THREADS) {
-    const int h = i * 8 / dk, c = i * 8 - h * dk;
+    const int h = i / vph, c = (i - h * vph) * 8;
     const bool is_q = h < hq;
     if (!is_q && !cached) continue;
     const float* x = rk_row + h * dk;
@@ -208,6 +209,36 @@ row_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __rest
     if (w != nullptr && form.whole) w += (is_q ? h : h - hq) * dk;
     const float r = s_r[h];
     float v[8];
+    if (VEC) {                                             // a vector's partners are a vector
+      float f[8];
+      load8(x + c, v);
+      if (w != nullptr) {
+        load8(w + c, f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] *= f[j];
+      }
+      if (c < dims) {
+        const bool first = c < half;
+        const int o = first ? c + half : c - half;
+        float b[8];
+        load8(x + o, b);
+        if (w != nullptr) {
+          load8(w + o, f);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) b[j] *= f[j];
+        }
+        const float4* tp = reinterpret_cast<const float4*>(tab + (first ? c : o));
+#pragma unroll
+        for (int j = 0; j < 8; j += 2) {
+          const float4 t = tp[j >> 1];                     // (cos, sin) of two pairs
+          v[j] = first ? v[j] * t.x - b[j] * t.y : v[j] * t.x + b[j] * t.y;
+          v[j + 1] = first ? v[j + 1] * t.z - b[j + 1] * t.w : v[j + 1] * t.z + b[j + 1] * t.w;
+        }
+      }
+      const float s = is_q ? r * tf : r;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] *= s;
+    } else
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const int e = c + j;
@@ -309,7 +340,8 @@ static int row_norm_launch(void* qkv, const int* slots, void* kcache, void* vcac
                            const QueryTemp& temp, int* status, cudaStream_t s) {
   const int smem = ((hq + hkv) * dk + hq + hkv) * 4;
   if (smem > 200 * 1024) return FF_HOST_TOO_LARGE;
-  auto kern = row_norm_kv_kernel<T>;
+  const bool vec = (cos_sin == nullptr || (form.halves && half % 8 == 0)) && ((reinterpret_cast<uintptr_t>(wq) | reinterpret_cast<uintptr_t>(wk)) & 15) == 0;
+  auto kern = vec ? row_norm_kv_kernel<T, true> : row_norm_kv_kernel<T, false>;
   if (int r = opt_in_smem(kern, smem)) return r;
   if (int r = launch_pdl(kern, dim3(rows), dim3(HN_THREADS), smem, s, 0, (T*)qkv, slots, (T*)kcache, (T*)vcache, hq, hkv, dim, dk, dv, block_size,
                          num_blocks, ld, eps, wq, wk, cos_sin, half, form, temp, status)) return r;

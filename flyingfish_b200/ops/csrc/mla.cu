@@ -254,6 +254,23 @@ mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ par
   *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(acc[0] * inv, acc[1] * inv), pack_bf16x2(acc[2] * inv, acc[3] * inv));
 }
 
+// rows of cache pages one after the other, their first `cols` columns: out [pages * 64, cols]; grid (pages), 256 threads
+__global__ void __launch_bounds__(256)
+mla_gather_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ blocks, __nv_bfloat16* __restrict__ out, int cols, int ld,
+                  int num_blocks, int* status) {
+  pdl_trigger();
+  pdl_wait();
+  const int page = blockIdx.x;
+  int blk = blocks[page];
+  if (blk < 0 || blk >= num_blocks) { if (threadIdx.x == 0) set_status(status, KID_MLA, FF_ERR_BOUNDS, page, blk); blk = 0; }
+  const int vec = cols / 8;
+  for (int i = threadIdx.x; i < PAGE * vec; i += 256) {
+    const int r = i / vec, c = i - r * vec;
+    reinterpret_cast<uint4*>(out + ((size_t)page * PAGE + r) * cols)[c] =
+        reinterpret_cast<const uint4*>(cache + ((size_t)blk * PAGE + r) * ld)[c];
+  }
+}
+
 // latent cache write: row r -> cache[slot] = [c (512) | k_rope (64)]; slot < 0 skips
 __global__ void mla_cache_write_kernel(const __nv_bfloat16* __restrict__ c, const __nv_bfloat16* __restrict__ kr,
                                        const int* __restrict__ slots, __nv_bfloat16* __restrict__ cache, int rows,
@@ -317,6 +334,14 @@ FF_EXPORT int ff_mla_attn(const void* q, const void* cache, const int* block_tab
     return launch_result();
   }
   return 0;
+}
+
+// out [pages * 64, cols] = the first `cols` columns of the cache pages `blocks` (rows of ld elements)
+FF_EXPORT int ff_mla_gather(const void* cache, const int* blocks, void* out, int pages, int cols, int ld, int num_blocks, int* status, cudaStream_t s) {
+  if (pages <= 0 || cols <= 0 || cols % 8 || ld % 8 || cols > ld) return FF_HOST_BAD_SHAPE;
+  if (int r = launch_pdl(mla::mla_gather_kernel, dim3(pages), dim3(256), 0, s, 0, (const __nv_bfloat16*)cache, blocks, (__nv_bfloat16*)out, cols, ld,
+                         num_blocks, status)) return r;
+  return launch_result();
 }
 
 FF_EXPORT int ff_mla_cache_write(const void* c, const void* k_rope, const int* slots, void* cache, int rows, int ldc,

@@ -6,10 +6,11 @@ from __future__ import annotations
 
 import ctypes
 from ctypes import c_float, c_longlong
+from dataclasses import dataclass
 
 import torch
 
-from . import _count, _head_gate_ld, _require, attn_decode, attn_prefill, workspace
+from . import _count, _head_gate_ld, _require, attn_decode, attn_prefill, linear, workspace
 from .lib import check, kernels, ptr, status_tensor, stream_ptr
 
 F32 = torch.float32
@@ -153,3 +154,62 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Te
         reach = min(max_ctx, window + cache.shape[2]) if window else max_ctx
         return attn_decode(flat, cache, vals, block_table, ctx_lens, heads, 1, width, scale, nq=max_q, max_ctx=reach, **kw)
     return attn_prefill(flat, cache, vals, block_table, q_start, q_lens, ctx_lens, max_q, heads, 1, width, scale, **kw)
+
+
+# ------------------------------------------------------------------------------------------
+# prompts: keys and values expanded from the latents
+# ------------------------------------------------------------------------------------------
+EXPAND_MIN_ROWS = 64             # portions of fewer rows stay in the latent space
+EXPAND_MAX_KEYS = 1 << 16        # most key rows expanded at a time
+
+
+def expands(q: torch.Tensor, width: int, dim: int, rot: int, vdim: int, longest: int) -> bool:
+    """Whether :func:`expanded_attention` serves a batch whose longest portion has ``longest`` rows: on the tensor cores a head of
+    dim + rot elements costs a fraction of one as wide as the latent, which pays for the expansion from a few dozen rows on. Narrow
+    latents have the tcgen05 kernel in the latent space."""
+    return q.is_cuda and q.dtype == torch.bfloat16 and width > 128 and dim <= 128 and rot <= 64 and vdim <= 128 and longest >= EXPAND_MIN_ROWS
+
+
+@dataclass
+class KeyPages:
+    """Cache pages a batch of portions can see, one sequence after the other."""
+    count: int
+    offsets: torch.Tensor            # int32 [sequences]: page t of a sequence is expanded page offsets + t
+    blocks: torch.Tensor             # int32 [count]: the pages' blocks
+
+    @classmethod
+    def of(cls, q_lens: list[int], ctx_lens: list[int], block_table, window: int, page: int, device) -> "KeyPages | None":
+        """``block_table``: rows of block ids on the host. None when the pages hold more than ``EXPAND_MAX_KEYS`` keys."""
+        offsets, blocks = [], []
+        for row, n, ctx in zip(block_table, q_lens, ctx_lens):
+            first = max(ctx - n - window + 1, 0) // page if window else 0
+            offsets.append(len(blocks) - first)
+            blocks += row[first: (ctx + page - 1) // page].tolist()
+        if len(blocks) * page > EXPAND_MAX_KEYS:
+            return None
+        both = torch.tensor(offsets + blocks, dtype=torch.int32, device=device)
+        return cls(len(blocks), both[: len(offsets)], both[len(offsets):])
+
+
+def expanded_attention(q: torch.Tensor, q_full: torch.Tensor, cache: torch.Tensor, w_kv: torch.Tensor, pages: KeyPages, block_table: torch.Tensor,
+                       q_start: torch.Tensor, q_lens: torch.Tensor, ctx_lens: torch.Tensor, max_q: int, dim: int, vdim: int, rank: int, scale: float,
+                       window: int, head_gate: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
+    """Prefill attention with every visible latent expanded once: ``w_kv`` ([heads * (dim + vdim), rank], all key matrices, then all value
+    matrices) makes keys and values of the pages, then the tcgen05 prefill kernel reads them beside the cache's rotated key parts.
+    q: rows with the heads' unrotated parts (``dim`` each); ``q_full`` [rows, heads, rank + rot] holds the rotated ones behind
+    ``rank`` columns. out: [rows, heads * vdim]."""
+    rows, heads, width = q_full.shape
+    nb, one, bs, cw = cache.shape
+    _require(one == 1 and bs == 64 and cw == width and cache.is_contiguous() and q_full.is_contiguous() and q.stride(1) == 1 and out.is_contiguous(),
+             "expanded_attention: layout")
+    latents = torch.empty(pages.count * bs, rank, dtype=q.dtype, device=q.device)
+    check(kernels().ff_mla_gather(ptr(cache), ptr(pages.blocks), ptr(latents), pages.count, rank, cw, nb, ptr(status_tensor(q.device)), stream_ptr()),
+          "ff_mla_gather")
+    both = linear(latents, w_kv)
+    rc = kernels().ff_attn_prefill_latent(ptr(q), ptr(q_full), ptr(both), ptr(cache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens),
+                                          ptr(pages.offsets), ptr(out), block_table.shape[0], rows, max_q, heads, dim, width - rank, vdim, q.stride(0),
+                                          width, rank, both.stride(0), both.shape[0], cw, rank, out.stride(0), block_table.shape[1], nb, c_float(scale),
+                                          window, ptr(head_gate), _head_gate_ld(head_gate, rows, heads), ptr(status_tensor(q.device)), stream_ptr())
+    check(rc, "ff_attn_prefill_latent")
+    _count(2)
+    return out

@@ -442,9 +442,22 @@ def _kabavik_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> 
     gate = p[:, at0 + R + T: at0 + R + T + H]
     unbound = dataclasses.replace(lat, window=0)
     lc = lambda l: cost(l, R + T, seen(l), 2 * R + T, 2 * R + T)
-    pair("latent attention, window, gated", lambda: mla_ops.latent_attention(q, lg.k, lg.table, qs, ql, lg.ctx, rows // batch, ctx, lat.scale, R, lat.window, gate,
-         out, decode=decode), lc(lat), "latent attention, full", lambda: mla_ops.attention(q, lg.k, lg.table, qs, ql, lg.ctx, rows // batch, ctx, lat.scale, R),
-         lc(unbound))
+    like = lambda: mla_ops.attention(q, lg.k, lg.table, qs, ql, lg.ctx, rows // batch, ctx, lat.scale, R)
+    if decode:
+        pair("latent attention, window, gated", lambda: mla_ops.latent_attention(q, lg.k, lg.table, qs, ql, lg.ctx, 1, ctx, lat.scale, R, lat.window, gate, out,
+             decode=True), lc(lat), "latent attention, full", like, lc(unbound))
+    else:       # prompts: expansion and attention here, the latent space there; the cost is that of the expanded form for both
+        def like_latent_attention():
+            mla_ops.per_head_linear(xq.reshape(rows, H, d), uk)
+            mla_ops.per_head_linear(like(), uv)
+        pages = mla_ops.KeyPages.of([ctx] * batch, [ctx] * batch, lg.table.cpu(), lat.window, 64, dev)
+        w_kv, res = rn(H * 2 * d, R), rn(rows, H * d)
+        expansion, ec = pair.gemm(H * 2 * d, R), lambda l: cost(l, R + T, seen(l), 2 * d + T, 2 * d + T)
+        add = lambda a, b: (a[0] + b[0], a[1] + b[1])
+        pair("latents expanded, attention, window, gated", lambda: mla_ops.expanded_attention(xq, q, lg.k, w_kv, pages, lg.table, qs, ql, lg.ctx, ctx, d, d, R,
+             lat.scale, lat.window, gate, res), add(expansion, ec(lat)), "queries to latents, attention, results out of latents",
+             like_latent_attention,
+             add(expansion, ec(unbound)))
     if decode:
         wv = rn(spec.vocab, W)
         pair("logits, 32-bit", lambda: ops.linear(x, wv, out_dtype=f32), pair.gemm(spec.vocab, W, out_bytes=4), "logits", lambda: ops.linear(x, wv),

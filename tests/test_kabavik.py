@@ -346,6 +346,80 @@ def test_latent_attention(device, dtype, rank, rot, heads, size):
         ops.check_status()
 
 
+@GPU
+@pytest.mark.parametrize("heads,dim,rot,vdim,rank", [(4, 128, 64, 128, 512), (3, 32, 16, 48, 128), (17, 64, 32, 112, 160), (2, 80, 48, 16, 608)])
+@pytest.mark.parametrize("size", [0, 1, 45, 64, 190])
+def test_attention_over_expanded_latents(heads, dim, rot, vdim, rank, size):
+    """Portions of several sequences at once, short ones beside long ones; the last query of a sequence looks like the first key of its window
+    or the key before it."""
+    bf, width, device = torch.bfloat16, rank + rot, "cuda"
+    scale = (dim + rot) ** -0.5
+    ctx, qlen = [260, 65, 128, 331, 7, 1], [260, 2, 70, 130, 7, 1]
+    kc, _, bt, ks, _ = paged(device, bf, 1, width, 16, ctx, seed=rank + size)
+    g = torch.Generator().manual_seed(4)
+    n = sum(qlen)
+    w_uk, w_uv = ((torch.randn(heads, d, rank, generator=g) / rank ** 0.5).to(bf) for d in (dim, vdim))
+    p, q_full = torch.randn(n, heads * dim + 24, generator=g).to(bf), torch.randn(n, heads, width, generator=g).to(bf)
+    q_full[..., :rank] = float("nan")                      # the absorbed queries are not there
+    gate = (2 * torch.randn(n, heads + 5, generator=g)).to(bf)
+    starts = torch.tensor([0] + qlen[:-1]).cumsum(0).to(torch.int32)
+    keys, vals = [], []
+    for k in ks:
+        c, r = k[0, :, :rank], k[0, :, rank:]
+        up = lambda w: torch.einsum("tr,hdr->htd", c, w.double()).to(bf).double()
+        keys.append(torch.cat([up(w_uk), r.expand(heads, -1, -1)], -1))
+        vals.append(up(w_uv))
+    w_kv = torch.cat([w_uk.reshape(-1, rank), w_uv.reshape(-1, rank)]).to(device)
+    pages = mla_ops.KeyPages.of(qlen, ctx, bt, size, 64, device)
+    for back in (0, 1):
+        q = torch.cat([p[:, : heads * dim].view(n, heads, dim), q_full[..., rank:]], -1).float()
+        q = _pointed(q.view(n, -1), keys, starts, qlen, ctx, lambda c: c - (size or c) - back, 1, heads * (dim + rot), 1.0).to(bf).view(n, heads, -1)
+        pd, qf = p.clone(), q_full.clone()
+        pd[:, : heads * dim], qf[..., rank:] = q[..., :dim].reshape(n, -1), q[..., dim:]
+        want = _attend_rows(q.reshape(n, -1), keys, vals, starts, qlen, heads, dim + rot, scale, {"size": size} if size else None, None, gate[:, 3: 3 + heads])
+        out = torch.empty(n, heads * vdim, dtype=bf, device=device)
+        mla_ops.expanded_attention(pd.to(device), qf.to(device), kc.to(device), w_kv, pages, bt.to(device), starts.to(device), i32(qlen, device),
+                                   i32(ctx, device), max(qlen), dim, vdim, rank, scale, size, gate.to(device)[:, 3: 3 + heads], out)
+        close(out, want, "bf16", f"back {back}", 2e-2)
+    ops.check_status()
+
+
+@GPU
+def test_expanded_and_absorbed_forms_agree(tmp_path, monkeypatch):
+    """The same prompt with its portions expanded and in the latent space; portions beside single tokens."""
+    cfg = O.config([L(heads=4, kv_rank=200, rot_dim=32, dim=64, vdim=64, size=100), W(), L(heads=2, kv_rank=136, size=70), L(heads=3, kv_rank=136, rot_dim=20)])
+    w = O.tensors(cfg, seed=15)
+    e = load(write(tmp_path, cfg, w), "cuda", "bf16", capacity=512).engine
+    a, b = ids(300, seed=90), ids(80, seed=91)
+    wa, wb = O.forward(cfg, w, a)[0], O.forward(cfg, w, b)[0]
+    asked = []
+    real = mla_ops.expanded_attention
+    monkeypatch.setattr(mla_ops, "expanded_attention", lambda *x, **k: (asked.append(1), real(*x, **k))[1])
+    for least, limit in ((64, 1 << 16), (2, 1 << 16), (10 ** 6, 1 << 16), (64, 128)):
+        monkeypatch.setattr(mla_ops, "EXPAND_MIN_ROWS", least)
+        monkeypatch.setattr(mla_ops, "EXPAND_MAX_KEYS", limit)
+        asked.clear()
+        sa, sb, got = e.add_sequence(a[:130]), e.add_sequence(b[:79]), []
+        got.append(e.feed([Span(sa, a[:130], list(range(130)))]))
+        got.append(e.feed([Span(sb, b[:79], list(range(79))), Span(sa, a[130:131], [0])]))
+        got.append(e.feed([Span(sa, a[131:290], list(range(159))), Span(sb, b[79:], [0])]))
+        got.append(e.feed([Span(sa, a[290:], list(range(10)))]))
+        agree(torch.cat([got[0], got[1][79:], got[2][:159], got[3]]), wa, "bf16", f"first request, {least}")
+        agree(torch.cat([got[1][:79], got[2][159:]]), wb, "bf16", f"second request, {least}")
+        assert len(asked) == {(64, 1 << 16): 9, (2, 1 << 16): 12, (10 ** 6, 1 << 16): 0, (64, 128): 3}[(least, limit)]
+        for s in (sa, sb):
+            e.free_sequence(s.seq_id)
+    ops.check_status()
+
+
+def test_key_pages_of_a_batch():
+    table = torch.arange(40).view(4, 10)
+    p = mla_ops.KeyPages.of([130, 1, 64, 10], [130, 300, 640, 70], table, 70, 64, "cpu")
+    # the first query of the second sequence sits at 299 and sees from 230 on, that of the third at 576 from 507 on
+    assert p.blocks.tolist() == [0, 1, 2, 13, 14, 27, 28, 29, 30, 31] and p.offsets.tolist() == [0, 0, -2, 8] and p.count == 10
+    assert mla_ops.KeyPages.of([10], [640], table, 0, 64, "cpu").blocks.tolist() == list(range(10))
+
+
 def test_mask_restatement():
     show = lambda m: [torch.nonzero(r).flatten().tolist() for r in m]
     assert show(O.visible(6, {"size": 2, "keep_first": 1})) == [[0], [0, 1], [0, 1, 2], [0, 2, 3], [0, 3, 4], [0, 4, 5]]
