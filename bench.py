@@ -7,7 +7,7 @@ head_dim 128, SwiGLU 14336, vocab 128256, BF16, random-init N(0, 0.02) weights, 
 parallel over the N GPUs of one node. ``--config 3`` selects the Llama-3-70B shape (batch 32,
 prompt 4096). A step is one decode step of the whole batch.
 
-``--design duponex`` measures another model design beside its closest relative instead (``utils/designbench.py``).
+``--design duponex|rudorax|kabavik`` measures another model design beside its closest relative instead (``utils/designbench.py``).
 
 Three arms (``--impl``):
   * ``ours``      -- this framework's engine and kernels. Reports

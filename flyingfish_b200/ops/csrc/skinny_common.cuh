@@ -42,7 +42,6 @@ struct SkinnyEpi {
   const int* slots;
   __nv_bfloat16* kcache; __nv_bfloat16* vcache;
   int hq, hkv, rot_dim, block_size, num_blocks;
-  int gate;                    // mode 1: 0 SiLU as above, 3 tanh-GELU on the FP32 sums (one rounding)
 };
 
 __device__ __forceinline__ float bf16r_sk(float x) { return __bfloat162float(__float2bfloat16(x)); }
@@ -57,10 +56,6 @@ __device__ __forceinline__ void emit_pair(const SkinnyEpi& ep, __nv_bfloat16* __
     uint32_t o[4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      if (ep.gate == 3) {
-        o[j] = pack_bf16x2(gelu_tanh_f(lo[2 * j]) * hi[2 * j], gelu_tanh_f(lo[2 * j + 1]) * hi[2 * j + 1]);
-        continue;
-      }
       const float a0 = bf16r_sk(silu_sk(bf16r_sk(lo[2 * j]))), a1 = bf16r_sk(silu_sk(bf16r_sk(lo[2 * j + 1])));
       o[j] = pack_bf16x2(a0 * bf16r_sk(hi[2 * j]), a1 * bf16r_sk(hi[2 * j + 1]));
     }
