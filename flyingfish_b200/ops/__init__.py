@@ -280,7 +280,8 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = Non
 def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor | None = None,
                   mode: int = 0) -> torch.Tensor:
     """Gate/up projection with the SwiGLU activation fused into the GEMM epilogue. The weight is
-    the per-64 interleaved ``[2f, h]`` matrix built by :func:`ref.interleave_gate_up`."""
+    the per-64 interleaved ``[2f, h]`` matrix built by :func:`ref.interleave_gate_up`. ``mode``: the gate, see
+    :func:`ref.silu_mul` (0 and 3 run in the epilogue)."""
     if not _is_cuda(x):
         return ref.linear_swiglu(x, w_interleaved, mode)
     if x.dtype == torch.float32:
