@@ -21,7 +21,7 @@ class MoeSpec:
     num_experts: int
     top_k: int
     expert_ffn: int
-    score: str = "softmax"            # softmax | sigmoid | noaux | sqrt_softplus
+    score: str = "softmax"            # softmax | biased_softmax | sigmoid | noaux | sqrt_softplus
     n_shared: int = 0                 # shared experts (each of width shared_ffn)
     shared_ffn: int = 0
     n_groups: int = 1
@@ -33,6 +33,8 @@ class MoeSpec:
     identity: int = 0                 # router outputs behind the experts whose output is the input itself
     shared_gate: bool = False         # sigmoid gate on the shared expert (Qwen-style)
     expert_format: str = "bf16"       # bf16 | fp8_block | nvfp4
+    limit: float = 0.0                # > 0: the experts' gate is clamped there (g sigmoid(1.702 g) (u + 1)) in place of SiLU
+    shared_limit: float = 0.0         # the same of the shared expert
 
 
 @dataclass
@@ -75,11 +77,16 @@ class LayerSpec:
     dim: int                          # width of a query / key head
     vdim: int                         # width of a value head
     scale: float                      # factor of the attention scores (of the queries, for a matrix memory)
-    mixer: str = "attention"          # attention | mlstm (matrix memory: per-sequence state instead of a cache) | latent (latent attention)
+    # attention | latent (latent attention); with a per-sequence state instead of a cache: mlstm (matrix memory), channel_delta (gated
+    # delta rule with a decay per key channel), ssd (state space: ``dim`` states, ``kv_heads`` groups of input and output maps)
+    mixer: str = "attention"
     chunk: int = 0                    # > 0: position i sees only keys of its own block of ``chunk`` positions
     window: int = 0                   # > 0: position i sees itself and the ``window - 1`` positions before it
     keep_first: int = 0               # with a window: the sequence's first ``keep_first`` positions stay visible
     sink: bool = False                # learnable soft-max: one extra logit per head in the denominator
+    sink_one: bool = False            # the denominator has one more, fixed, term: e^0
+    talk: bool = False                # the heads' weights are mixed by a matrix [heads, heads] before they meet the values
+    v_norm: bool = False              # values are divided by their root mean square per head (and cached so)
     rope: RopeSpec | None = None
     qk_norm: str = "head"             # RMS norm of q and k: over every head, or over the whole projection ("row")
     bias: bool = False                # the projections have biases
@@ -89,6 +96,11 @@ class LayerSpec:
     kv_rank: int = 0                  # latent attention: width of the latent a token caches
     rot_dim: int = 0                  # latent attention: width of the rotated key part all heads share (and of the queries')
     gate_cap: float = 0.0             # matrix memory: soft cap of the gates' logits
+    conv: int = 0                     # channel_delta, ssd: taps of the causal convolution in front of the recurrence
+    decay_rank: int = 0               # channel_delta: width between the two matrices of the decays (0: the checkpoint says)
+    gate_rank: int = 0                # channel_delta: the same of the output gate
+    norm_groups: int = 1              # ssd: equal parts of the heads' outputs, normed each by itself
+    beside: "LayerSpec | None" = None # a second mixer on the same input; the layer's result is half the sum of the two, each normed
     out_gate: bool = True             # the heads' outputs are multiplied by the sigmoid of a projection
     v_mix: bool = False               # values are mixed with those of the first layer that has the flag
     ffn: int = 0                      # width of the feed-forward (0: the layer has none, or experts)
@@ -130,25 +142,48 @@ class LayerSpec:
 
     def cache_bytes_read(self, ctx: int, elem_bytes: int) -> int:
         """Bytes of cache or state one decoded token moves at a context of ``ctx``."""
+        if self.beside is not None:
+            return dataclasses.replace(self, beside=None).cache_bytes_read(ctx, elem_bytes) + self.beside.cache_bytes_read(ctx, elem_bytes)
         if self.mixer == "mlstm":
             return 2 * 4 * self.heads * self.dim * (self.vdim + 1)
+        if self.mixer in ("channel_delta", "ssd"):
+            return 2 * 4 * (self.heads * self.dim * self.vdim + (self.conv - 1) * self.conv_channels)
         if self.mixer == "latent":
             return elem_bytes * self.keys_seen(ctx) * (self.kv_rank + self.rot_dim)
         return elem_bytes * self.keys_seen(ctx) * self.kv_heads * (self.dim + self.vdim)
 
     def mixer_flops(self, n: int) -> int:
         """FLOPs of a prompt of ``n`` positions outside the projections."""
-        if self.mixer == "mlstm":         # the recurrence: state update and read of every position
+        if self.beside is not None:
+            return dataclasses.replace(self, beside=None).mixer_flops(n) + self.beside.mixer_flops(n)
+        if self.mixer in ("mlstm", "ssd"):    # the recurrence: state update and read of every position
             return 4 * n * self.heads * self.dim * self.vdim
+        if self.mixer == "channel_delta":     # two reads and the update
+            return 6 * n * self.heads * self.dim * self.vdim
         if self.mixer == "latent":        # scores and values in the latent space
             return 2 * self.heads * (2 * self.kv_rank + self.rot_dim) * self.pairs_seen(n)
-        return 2 * self.heads * (self.dim + self.vdim) * self.pairs_seen(n)
+        return 2 * self.heads * (self.dim + self.vdim + (self.heads if self.talk else 0)) * self.pairs_seen(n)
+
+    @property
+    def conv_channels(self) -> int:
+        """Channels of the convolution: keys, queries and values, or input, input maps and output maps."""
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    @property
+    def conv_pad(self) -> int:
+        return 2 * self.kv_heads * self.dim_pad + self.heads * self.vdim_pad
 
     @property
     def projection_cols(self) -> int:
         """Columns of the fused input projection, heads padded."""
         if self.mixer == "latent":        # [unrotated queries | rotated queries | latent | rotated key | head gates]
             return self.heads * (self.dim_pad + self.rot_pad) + self.rank_pad + self.rot_pad + pad_to(self.heads, 8)
+        if self.mixer == "channel_delta":     # [q | k | v | decays' inner | gate's inner | step sizes]
+            return self.conv_pad + pad_to(self.decay_rank, 8) + pad_to(self.gate_rank, 8) + pad_to(self.heads, 8)
+        if self.mixer == "ssd":               # [output maps | input maps | input | gate | step sizes]
+            return self.conv_pad + self.heads * self.vdim_pad + pad_to(self.heads, 8)
+        if self.beside is not None:
+            return dataclasses.replace(self, beside=None).projection_cols + self.beside.projection_cols
         if self.kv_from >= 0:
             return self.heads * self.dim_pad
         g = self.heads * self.vdim_pad if self.out_gate else 0
@@ -159,9 +194,17 @@ class LayerSpec:
         if self.mixer == "latent":
             n = hidden * (self.heads * (self.dim + self.rot_dim + self.vdim + 1) + self.kv_rank + self.rot_dim) + \
                 self.heads * self.kv_rank * (self.dim + self.vdim)
+        elif self.mixer == "channel_delta":
+            o = self.heads * self.vdim
+            n = hidden * (self.conv_channels + o + self.decay_rank + self.gate_rank + self.heads) + \
+                self.heads * self.dim * self.decay_rank + o * self.gate_rank + self.conv * self.conv_channels
+        elif self.mixer == "ssd":
+            n = hidden * (self.conv_channels + 2 * self.heads * self.vdim + self.heads) + self.conv * self.conv_channels
         else:
             own = self.kv_heads if self.kv_from < 0 else 0
             n = hidden * (self.heads * (self.dim + self.vdim * (2 if self.out_gate else 1)) + own * (self.dim + self.vdim))
+        if self.beside is not None:
+            n += self.beside.params(hidden) + 2 * hidden
         n += (3 if self.ffn_act == "geglu" else 2) * hidden * self.ffn + (2 * hidden * self.heads if self.mixer == "mlstm" else 0)
         if self.moe is not None:
             m = self.moe
@@ -170,7 +213,7 @@ class LayerSpec:
 
 
 # architectures whose every operator has a 32-bit kernel on the GPU
-GPU_FP32_ARCHS = ("duponex", "rudorax", "kabavik")
+GPU_FP32_ARCHS = ("duponex", "rudorax", "kabavik", "bazulorn")
 
 
 def pad_to(n: int, m: int) -> int:
@@ -180,7 +223,7 @@ def pad_to(n: int, m: int) -> int:
 @dataclass
 class ModelSpec:
     name: str
-    arch: str                         # llama | qwen3 | qwen3_moe | deepseek_v3 | deepseek_v41 | glm5_next | flint | loop_vl | tiny_moe | qwen3_vl | embedding | diffusion_lm | qwen35_text | gemma | duponex | rudorax | kabavik
+    arch: str                         # llama | qwen3 | qwen3_moe | deepseek_v3 | deepseek_v41 | glm5_next | flint | loop_vl | tiny_moe | qwen3_vl | embedding | diffusion_lm | qwen35_text | gemma | duponex | rudorax | kabavik | bazulorn
     layers: int
     hidden: int
     heads: int
@@ -601,6 +644,64 @@ def kabavik_tiny() -> ModelSpec:
                             embed_scale=1.0, residual_mult=0.8, logit_scale=0.5, side_dim=24, eps=1e-5)
 
 
+def _bazulorn_spec_of(name: str, hidden: int, vocab: int, layers: list[LayerSpec], buckets: int, mul_prev: int, mul_cur: int,
+                      eps: float) -> ModelSpec:
+    if not layers:
+        raise ConfigError("a Bazulorn model needs at least one layer")
+    if buckets < 1 or min(mul_prev, mul_cur) < 0 or max(mul_prev, mul_cur) * vocab >= 1 << 62:
+        raise ConfigError("unusable bigram table")
+    for i, l in enumerate(layers):
+        for m in [l] + ([l.beside] if l.beside is not None else []):
+            if min(m.heads, m.kv_heads, m.dim, m.vdim) < 1 or m.heads % m.kv_heads or m.ffn < 0 or not m.scale > 0:
+                raise ConfigError(f"layer {i}: unusable mixer sizes {m}")
+            if m.mixer in ("channel_delta", "ssd") and not 1 <= m.conv <= 8:
+                raise ConfigError(f"layer {i}: convolutions have 1 to 8 taps, not {m.conv}")
+            if m.mixer == "ssd" and (m.norm_groups < 1 or m.heads * m.vdim % m.norm_groups):
+                raise ConfigError(f"layer {i}: {m.heads * m.vdim} outputs in {m.norm_groups} equal parts")
+        if l.beside is not None and l.window < 1:
+            raise ConfigError(f"layer {i}: unusable window {l.window}")
+        if l.mixer == "channel_delta":        # until a checkpoint says otherwise
+            l.decay_rank, l.gate_rank = l.decay_rank or l.dim, l.gate_rank or l.vdim
+    wide = max(layers, key=lambda l: l.heads * l.dim)
+    return ModelSpec(
+        name=name, arch="bazulorn", layers=len(layers), hidden=hidden, heads=wide.heads, kv_heads=wide.kv_heads, head_dim=wide.dim,
+        ffn=max(l.ffn for l in layers), vocab=vocab, rms_eps=eps, tie_embeddings=True, layer_specs=layers,
+        extra={"bazulorn": {"buckets": buckets, "mul_prev": mul_prev, "mul_cur": mul_cur}})
+
+
+def bazulorn_tiny() -> ModelSpec:
+    """Small Bazulorn shape: delta-rule layers with a dense and an expert feed-forward, attention with mixed heads beside a state space,
+    a layer without a feed-forward."""
+    moe = MoeSpec(num_experts=6, top_k=3, expert_ffn=72, score="biased_softmax", limit=1.5, n_shared=1, shared_ffn=104, shared_limit=2.5)
+    delta = dict(mixer="channel_delta", heads=4, kv_heads=2, dim=24, vdim=40, scale=24 ** -0.5, conv=4, decay_rank=20, gate_rank=12, out_gate=False)
+    ssd = LayerSpec(mixer="ssd", heads=6, kv_heads=3, dim=32, vdim=24, scale=1.0, conv=3, norm_groups=4, out_gate=False)
+    both = dict(heads=4, kv_heads=2, dim=32, vdim=48, scale=0.2, window=72, bias=True, sink_one=True, talk=True, v_norm=True, out_gate=False, beside=ssd)
+    return _bazulorn_spec_of("bazulorn-tiny", 160, 512, [LayerSpec(**delta, ffn=200, ffn_act="geglu"), LayerSpec(**both, moe=moe),
+                                                         LayerSpec(**delta, moe=moe), LayerSpec(**both)],
+                             buckets=211, mul_prev=13, mul_cur=5, eps=1e-5)
+
+
+def _bazulorn_bench(name: str, hidden: int, heads: int, kv_heads: int, experts: int, ff: int, vocab: int) -> ModelSpec:
+    moe = MoeSpec(num_experts=experts, top_k=8, expert_ffn=ff, score="biased_softmax", limit=7.0, n_shared=1, shared_ffn=ff, shared_limit=7.0)
+    delta = LayerSpec(mixer="channel_delta", heads=heads, kv_heads=heads, dim=128, vdim=128, scale=128 ** -0.5, conv=4, decay_rank=128, gate_rank=128,
+                      out_gate=False, moe=moe)
+    ssd = LayerSpec(mixer="ssd", heads=hidden // 64, kv_heads=8, dim=128, vdim=64, scale=1.0, conv=4, norm_groups=8, out_gate=False)
+    both = LayerSpec(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, window=1024, bias=True, sink_one=True, talk=True,
+                     v_norm=True, out_gate=False, moe=moe, beside=ssd)
+    return _bazulorn_spec_of(name, hidden, vocab, [delta, delta, both] * 2, buckets=65537, mul_prev=131, mul_cur=3, eps=1e-5)
+
+
+def bazulorn_2k() -> ModelSpec:
+    """Bazulorn layers 2048 wide (random weights, for measurements): 16 delta heads of 128, 16 / 4 attention heads of 128 beside 32
+    state-space heads of 128 x 64, 64 experts of 768, top 8."""
+    return _bazulorn_bench("bazulorn-2k-shape", 2048, 16, 4, 64, 768, 65536)
+
+
+def bazulorn_4k() -> ModelSpec:
+    """As :func:`bazulorn_2k` at 4096: 32 delta heads, 32 / 8 attention heads, 64 state-space heads, experts of 1536."""
+    return _bazulorn_bench("bazulorn-4k-shape", 4096, 32, 8, 64, 1536, 128256)
+
+
 def _kabavik_bench(name: str, hidden: int, heads: int, kv_heads: int, ff: int, vocab: int) -> ModelSpec:
     own = dict(out_gate=False, ffn=ff, ffn_act="geglu", scale=128 ** -0.5)
     win = LayerSpec(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, window=2048, keep_first=64, qk_norm="row", bias=True,
@@ -639,6 +740,7 @@ NAMED_SHAPES = {
     "duponex-tiny": duponex_tiny, "duponex-8b-shape": duponex_8b, "duponex-2b-shape": duponex_2b,
     "rudorax-tiny": rudorax_tiny, "rudorax-2k-shape": rudorax_2k, "rudorax-4k-shape": rudorax_4k,
     "kabavik-tiny": kabavik_tiny, "kabavik-2k-shape": kabavik_2k, "kabavik-4k-shape": kabavik_4k,
+    "bazulorn-tiny": bazulorn_tiny, "bazulorn-2k-shape": bazulorn_2k, "bazulorn-4k-shape": bazulorn_4k,
     "loop-tiny": loop_tiny, "loopvl-text-shape": loopvl_text,
     "qwen3-moe-235b-shape": qwen3_moe_235b, "qwen3-moe-tiny": qwen3_moe_tiny,
 }
@@ -832,6 +934,59 @@ def _kabavik_spec(cfg: dict[str, Any], name: str) -> ModelSpec:
                             side_dim=int(side["dim"]) if side else 0, eps=float(cfg["norm"]["eps"]))
 
 
+def _bazulorn_moe(mlp: dict[str, Any], where: str) -> MoeSpec:
+    r, sh = mlp["router"], mlp.get("shared")
+    moe = MoeSpec(num_experts=int(r["experts"]), top_k=int(r["top"]), expert_ffn=int(mlp["expert"]["ff"]), score="biased_softmax",
+                  limit=float(mlp["expert"]["limit"]), n_shared=1 if sh else 0, shared_ffn=int(sh["ff"]) if sh else 0,
+                  shared_limit=float(sh["limit"]) if sh else 0.0)
+    if moe.num_experts < 1 or not 1 <= moe.top_k <= min(moe.num_experts, 32) or moe.expert_ffn < 1 or not moe.limit > 0 or \
+            (sh and (moe.shared_ffn < 1 or not moe.shared_limit > 0)):
+        raise ConfigError(f"{where}: unusable experts {moe}")
+    return moe
+
+
+def _bazulorn_spec(cfg: dict[str, Any], name: str) -> ModelSpec:
+    """``"architecture": "Bazulorn"``: a list of layers whose mixer is a channel-wise gated delta rule or windowed attention with
+    mixed heads beside a state space, with dense or expert feed-forwards; bigrams are embedded beside tokens. The widths inside the
+    decays' and the gate's matrix pairs are those of the checkpoint's tensors (:func:`read_model_spec`)."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+        m, mlp, kind = entry["mixer"], entry.get("mlp"), entry.get("type")
+        ff: dict[str, Any] = {}
+        if mlp is not None:
+            if mlp.get("kind") == "dense":
+                ff = dict(ffn=int(mlp["ff"]), ffn_act="geglu")
+            elif mlp.get("kind") == "moe":
+                ff = dict(moe=_bazulorn_moe(mlp, f"layer {i}"))
+            else:
+                raise ConfigError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r}")
+        if kind == "channel_delta":
+            layers.append(LayerSpec(mixer="channel_delta", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                                    vdim=int(m["vdim"]), scale=int(m["dim"]) ** -0.5, conv=int(m["conv"]), out_gate=False, **ff))
+        elif kind == "parallel":
+            a, s = m["left"], m["right"]
+            right = LayerSpec(mixer="ssd", heads=int(s["heads"]), kv_heads=int(s["groups"]), dim=int(s["state"]), vdim=int(s["vdim"]), scale=1.0,
+                              conv=int(s["conv"]), norm_groups=int(s["norm_groups"]), out_gate=False)
+            layers.append(LayerSpec(heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), dim=int(a["dim"]), vdim=int(a["vdim"]),
+                                    scale=float(a["scale"]), window=int(a["mask"]["size"]), bias=True, sink_one=True, talk=True, v_norm=True,
+                                    out_gate=False, beside=right, **ff))
+        else:
+            raise ConfigError(f"layer {i}: unsupported mixer {kind!r}")
+    b = cfg["embedding"]["bigram"]
+    return _bazulorn_spec_of(name, int(cfg["width"]), int(cfg["vocab"]), layers, buckets=int(b["buckets"]), mul_prev=int(b["mul_prev"]),
+                             mul_cur=int(b["mul_cur"]), eps=float(cfg["norm"]["eps"]))
+
+
+def _ranks_from_tensors(spec: ModelSpec, shape) -> None:
+    """Widths inside the matrix pairs of channel_delta layers from the shapes of a checkpoint's tensors."""
+    for i, l in enumerate(spec.layer_specs):
+        if l.mixer == "channel_delta":
+            try:
+                l.decay_rank, l.gate_rank = int(shape(f"l{i}.mix.a1")[0]), int(shape(f"l{i}.mix.g1")[0])
+            except KeyError as e:
+                raise ConfigError(f"layer {i}: the checkpoint lacks {e}") from None
+
+
 def spec_from_hf_config(cfg: dict[str, Any], name: str = "model") -> ModelSpec:
     """Normalise a Hugging Face ``config.json``. Hard checks mirror the reference's: SiLU
     activation only, 16-bit or 32-bit floats, no unsupported rope scaling for plain Llama."""
@@ -841,6 +996,8 @@ def spec_from_hf_config(cfg: dict[str, Any], name: str = "model") -> ModelSpec:
         return _rudorax_spec(cfg, name)
     if cfg.get("architecture") == "Kabavik":
         return _kabavik_spec(cfg, name)
+    if cfg.get("architecture") == "Bazulorn":
+        return _bazulorn_spec(cfg, name)
     archs = cfg.get("architectures") or []
     arch = next((_ARCH_MAP[a] for a in archs if a in _ARCH_MAP), None)
     if arch is None:
@@ -913,7 +1070,16 @@ def spec_from_hf_config(cfg: dict[str, Any], name: str = "model") -> ModelSpec:
 def read_model_spec(model_dir: str | Path) -> ModelSpec:
     p = Path(model_dir)
     cfg = json.loads((p / "config.json").read_text())
-    return spec_from_hf_config(cfg, name=p.name)
+    spec = spec_from_hf_config(cfg, name=p.name)
+    if spec.layer_specs is not None and any(l.mixer == "channel_delta" for l in spec.layer_specs):
+        from .loaders.safetensors_io import MappedCheckpoint
+        if any(p.glob("*.safetensors")):
+            ck = MappedCheckpoint(p)
+            try:
+                _ranks_from_tensors(spec, lambda n: ck.shape(n))
+            finally:
+                ck.close()
+    return spec
 
 
 # ------------------------------------------------------------------------------------------

@@ -182,6 +182,9 @@ class MappedCheckpoint:
     def tensor(self, name: str) -> torch.Tensor:
         return self.where[name].tensor(name)
 
+    def shape(self, name: str) -> tuple[int, ...]:
+        return tuple(self.where[name].tensors[name].shape)
+
     def has(self, name: str) -> bool:
         return name in self.where
 

@@ -6,7 +6,7 @@ from __future__ import annotations
 
 import importlib
 
-MODULES = {"duponex": "duponex", "rudorax": "rudorax", "kabavik": "kabavik"}
+MODULES = {"duponex": "duponex", "rudorax": "rudorax", "kabavik": "kabavik", "bazulorn": "bazulorn"}
 
 
 def design(arch: str):

@@ -29,7 +29,7 @@ from ..config import LayerSpec, ModelSpec, pad_to
 from ..ops import mla_ops, ref, residual_ops
 from ..ops.residual_ops import Norm
 from .decoder import DecoderModel
-from .weights import DTYPES, LayerWeights, ModelWeights, TensorSource, TPInfo, pad_cols, pad_heads, random_tensor
+from .weights import DTYPES, LayerWeights, ModelWeights, TensorSource, TPInfo, pad_cols, pad_heads, pad_rows, random_tensor
 
 
 # ------------------------------------------------------------------------------------------
@@ -86,10 +86,6 @@ def unused_tensors(spec: ModelSpec) -> tuple[str, ...]:
     return tuple(names)
 
 
-def _pad_rows(t: torch.Tensor, rows: int) -> torch.Tensor:
-    return t if t.shape[0] == rows else torch.cat([t, t.new_zeros(rows - t.shape[0], *t.shape[1:])])
-
-
 def build_weights(spec: ModelSpec, source: TensorSource) -> ModelWeights:
     """Fused and padded weights. ``wqkv`` = [q | k | v] with one bias vector (layers that share keys and values: q) or, for latent
     attention, [unrotated queries | rotated queries | latent | rotated key | gates]; heads padded to 16 elements. Norms are FP32,
@@ -107,15 +103,15 @@ def build_weights(spec: ModelSpec, source: TensorSource) -> ModelWeights:
         p, dk, dv = f"l{i}.mix.", l.dim_pad, l.vdim_pad
         lw = LayerWeights()
         lw.extra["norms"] = {n: norm(f"l{i}.{n}", mult if n.endswith("b") else 1.0) for n in _norm_names(l)}
-        lw.wo = _pad_rows(pad_heads(get(p + "o").t().contiguous(), l.heads, l.vdim, dv).t(), wp).contiguous()
+        lw.wo = pad_rows(pad_heads(get(p + "o").t().contiguous(), l.heads, l.vdim, dv).t(), wp).contiguous()
         if l.mixer == "latent":
             rp, tp, d = l.rank_pad, l.rot_pad, l.dim + l.rot_dim
             q = pad_cols(get(p + "q"), wp).view(l.heads, d, wp)
             down = pad_cols(get(p + "dkv"), wp)
             lw.wqkv = torch.cat([pad_heads(q[:, : l.dim].reshape(-1, wp), l.heads, l.dim, dk),
                                  pad_heads(q[:, l.dim:].reshape(-1, wp), l.heads, l.rot_dim, tp),
-                                 _pad_rows(down[: l.kv_rank], rp), _pad_rows(down[l.kv_rank:], tp),
-                                 _pad_rows(pad_cols(get(p + "g"), wp), pad_to(l.heads, 8))]).contiguous()
+                                 pad_rows(down[: l.kv_rank], rp), pad_rows(down[l.kv_rank:], tp),
+                                 pad_rows(pad_cols(get(p + "g"), wp), pad_to(l.heads, 8))]).contiguous()
             lw.extra["latent_norm"] = pad_cols(get(p + "dkv.norm").float(), rp).contiguous()
             # all key matrices, then all value matrices; a head's unrotated query goes into the latent space through [rank_pad, dim_pad]
             # and its result out of it through [vdim_pad, rank_pad]
@@ -132,16 +128,16 @@ def build_weights(spec: ModelSpec, source: TensorSource) -> ModelWeights:
             lw.k_norm = wide(p + "k.norm", l.kv_heads) if l.kv_from < 0 else None
         if l.ffn:
             p, fp = f"l{i}.mlp.", pad_to(l.ffn, 128)
-            lw.wgu = ref.interleave_gate_up(*(_pad_rows(pad_cols(get(p + n), wp), fp) for n in ("gate", "up")))
-            lw.wdown = _pad_rows(pad_cols(get(p + "down"), fp), wp).contiguous()
+            lw.wgu = ref.interleave_gate_up(*(pad_rows(pad_cols(get(p + n), wp), fp) for n in ("gate", "up")))
+            lw.wdown = pad_rows(pad_cols(get(p + "down"), fp), wp).contiguous()
         if sp:
             p = f"l{i}.side."
-            lw.extra["side_gate"] = _pad_rows(pad_cols(get(p + "gate"), wp), sp).contiguous()
-            lw.extra["side_proj"] = _pad_rows(pad_cols(get(p + "proj"), sp), wp).contiguous()
+            lw.extra["side_gate"] = pad_rows(pad_cols(get(p + "gate"), wp), sp).contiguous()
+            lw.extra["side_proj"] = pad_rows(pad_cols(get(p + "proj"), sp), wp).contiguous()
             lw.extra["norms"]["side"] = Norm("rms", vec(p + "norm", mult))
         layers.append(lw)
     w = ModelWeights(spec=spec, embed=pad_cols(get("embed"), wp).contiguous(), final_norm=norm("final.norm", float(cfg["logit_scale"])),
-                     lm_head=_pad_rows(pad_cols(get("head"), wp), pad_to(spec.vocab, 8)).contiguous(), layers=layers, tp=TPInfo(),
+                     lm_head=pad_rows(pad_cols(get("head"), wp), pad_to(spec.vocab, 8)).contiguous(), layers=layers, tp=TPInfo(),
                      vocab_shard=(0, spec.vocab))
     if sp:
         n = len(spec.layer_specs)

@@ -27,9 +27,9 @@ import torch
 
 from .. import ops
 from ..config import LayerSpec, ModelSpec, pad_to
-from ..ops import mlstm_ops, moe_ops, ref, residual_ops
+from ..ops import mlstm_ops, moe_ops, residual_ops
 from .decoder import DecoderModel
-from .weights import DTYPES, LayerWeights, ModelWeights, TensorSource, TPInfo, pad_cols, pad_heads, random_tensor
+from .weights import DTYPES, LayerWeights, ModelWeights, TensorSource, TPInfo, ffn_pair, pad_cols, pad_heads, pad_rows, random_tensor
 
 
 # ------------------------------------------------------------------------------------------
@@ -60,16 +60,6 @@ def unused_tensors(spec: ModelSpec) -> tuple[str, ...]:
     return tuple(f"l{i}.norm2" for i, l in enumerate(spec.layer_specs) if l.moe is None)
 
 
-def _pad_rows(t: torch.Tensor, rows: int) -> torch.Tensor:
-    return t if t.shape[0] == rows else torch.cat([t, t.new_zeros(rows - t.shape[0], *t.shape[1:])])
-
-
-def _ffn_pair(get, p: str, f: int, h: int, wp: int, fp: int) -> tuple[torch.Tensor, torch.Tensor]:
-    """Gate and up rows interleaved per 64, and the down matrix, of one feed-forward padded to ``fp``."""
-    gu = ref.interleave_gate_up(*(_pad_rows(pad_cols(get(p + n), wp), fp) for n in ("gate", "up")))
-    return gu, _pad_rows(pad_cols(get(p + "down"), fp), wp).contiguous()
-
-
 def build_weights(spec: ModelSpec, source: TensorSource) -> ModelWeights:
     """Fused and padded weights: ``wqkv`` = [q | k | v] (matrix memory: and the output gate) with heads padded to 16 elements; the
     gate projections of a matrix memory as one matrix; experts stacked. Norm weights (with their offset), biases, sinks and
@@ -88,29 +78,29 @@ def build_weights(spec: ModelSpec, source: TensorSource) -> ModelWeights:
         if l.out_gate:
             parts.append(("g", l.heads, l.vdim, dv))
         lw.wqkv = torch.cat([pad_heads(pad_cols(get(p + n), wp), *s) for n, *s in parts]).contiguous()
-        lw.wo = _pad_rows(pad_heads(get(p + "o").t().contiguous(), l.heads, l.vdim, dv).t(), wp).contiguous()
+        lw.wo = pad_rows(pad_heads(get(p + "o").t().contiguous(), l.heads, l.vdim, dv).t(), wp).contiguous()
         if l.mixer == "attention":
             lw.q_norm, lw.k_norm = (pad_cols(get(p + n).float(), dk).contiguous() for n in ("q.norm", "k.norm"))
             lw.extra["sinks"] = get(p + "sink").float().contiguous()
         else:
-            lw.extra["w_gates"] = _pad_rows(torch.cat([pad_cols(get(p + n), wp) for n in ("i", "f")]), pad_to(2 * l.heads, 16)).contiguous()
+            lw.extra["w_gates"] = pad_rows(torch.cat([pad_cols(get(p + n), wp) for n in ("i", "f")]), pad_to(2 * l.heads, 16)).contiguous()
             lw.extra["b_gates"] = torch.cat([get(p + n).float() for n in ("i.b", "f.b")]).contiguous()
             lw.extra["norm"] = pad_heads(get(p + "norm").float(), l.heads, l.vdim, dv).contiguous()
         if l.moe is not None:
             e, p = l.moe, f"l{i}.mlp."
             lw.post_ln = vec(f"l{i}.norm2")
             n = e.num_experts + e.identity
-            lw.router = _pad_rows(pad_cols(get(p + "router"), wp), pad_to(n, 16)).contiguous()
+            lw.router = pad_rows(pad_cols(get(p + "router"), wp), pad_to(n, 16)).contiguous()
             lw.router_bias = get(p + "correction").float().contiguous()
             fp = pad_to(e.expert_ffn, 64)
             lw.experts_gu = lw.router.new_empty(e.num_experts, 2 * fp, wp)
             lw.experts_down = lw.router.new_empty(e.num_experts, wp, fp)
             for j in range(e.num_experts):
-                lw.experts_gu[j], lw.experts_down[j] = _ffn_pair(get, p + f"e{j}.", e.expert_ffn, h, wp, fp)
+                lw.experts_gu[j], lw.experts_down[j] = ffn_pair(get, p + f"e{j}.", wp, fp)
             if e.n_shared:
-                lw.shared_gu, lw.shared_down = _ffn_pair(get, p + "shared.", e.shared_ffn, h, wp, pad_to(e.shared_ffn, 128))
+                lw.shared_gu, lw.shared_down = ffn_pair(get, p + "shared.", wp, pad_to(e.shared_ffn, 128))
         layers.append(lw)
-    head = _pad_rows(pad_cols(get("head"), wp), pad_to(spec.vocab, 8)).contiguous()
+    head = pad_rows(pad_cols(get("head"), wp), pad_to(spec.vocab, 8)).contiguous()
     return ModelWeights(spec=spec, embed=pad_cols(get("embed"), wp).contiguous(), final_norm=vec("final.norm"), lm_head=head, layers=layers,
                         tp=TPInfo(), vocab_shard=(0, spec.vocab))
 

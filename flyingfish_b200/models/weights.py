@@ -148,6 +148,18 @@ def pad_heads(t: torch.Tensor, heads: int, width: int, padded: int) -> torch.Ten
     return out.reshape(heads * padded, *t.shape[1:])
 
 
+def pad_rows(t: torch.Tensor, rows: int) -> torch.Tensor:
+    """The first dimension lengthened to ``rows`` with zeros."""
+    return t if t.shape[0] == rows else torch.cat([t, t.new_zeros(rows - t.shape[0], *t.shape[1:])])
+
+
+def ffn_pair(get, p: str, wp: int, fp: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """Gate and up rows interleaved per 64, and the down matrix, of one gated feed-forward (tensors ``p`` + gate / up / down) padded to
+    width ``wp`` and ``fp`` inner columns."""
+    gu = ref.interleave_gate_up(*(pad_rows(pad_cols(get(p + n), wp), fp) for n in ("gate", "up")))
+    return gu, pad_rows(pad_cols(get(p + "down"), fp), wp).contiguous()
+
+
 def pack_ffn_fp8(lw: "LayerWeights") -> None:
     """Re-encode a layer's feed-forward matrices as FP8-resident weights (E4M3 codes + 128x128 block scales): the
     dense gate/up and down projections, the shared expert, and the routed experts (gate/up interleaved per 64 rows,

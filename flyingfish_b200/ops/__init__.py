@@ -278,25 +278,25 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = Non
 
 
 def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor | None = None,
-                  mode: int = 0) -> torch.Tensor:
+                  mode: int = 0, limit: float = 0.0) -> torch.Tensor:
     """Gate/up projection with the SwiGLU activation fused into the GEMM epilogue. The weight is
     the per-64 interleaved ``[2f, h]`` matrix built by :func:`ref.interleave_gate_up`. ``mode``: the gate, see
-    :func:`ref.silu_mul` (0 and 3 run in the epilogue)."""
+    :func:`ref.silu_mul` (0, 3 and 5 run in the epilogue); ``limit`` goes with the clamped ones."""
     if not _is_cuda(x):
-        return ref.linear_swiglu(x, w_interleaved, mode)
+        return ref.linear_swiglu(x, w_interleaved, mode, limit)
     if x.dtype == torch.float32:
-        return silu_mul_interleaved(linear(x, w_interleaved), out, mode)
+        return silu_mul_interleaved(linear(x, w_interleaved), out, mode, limit)
     m, ldx = _rows2d(x)
     n, ldw = _rows2d(w_interleaved)
     k = x.shape[1]
     _require(n % 256 == 0, "linear_swiglu: N must be a multiple of 256")
     if out is None:
         out = torch.empty(m, n // 2, dtype=BF16, device=x.device)
-    if mode not in (0, 3):
-        # the GEMM epilogues implement modes 0 and 3 (tanh-GELU rounded once); other gates run as the activation kernel
-        return silu_mul_interleaved(linear(x, w_interleaved), out, mode)
+    if mode not in (0, 3, 5):
+        # the GEMM epilogues implement modes 0, 3 (tanh-GELU rounded once) and 5; other gates run as the activation kernel
+        return silu_mul_interleaved(linear(x, w_interleaved), out, mode, limit)
     if m <= SKINNY_MAX_M and not FUSE_SWIGLU:
-        return silu_mul_interleaved(linear(x, w_interleaved), out)
+        return silu_mul_interleaved(linear(x, w_interleaved), out, mode, limit)
     if m <= SKINNY_MAX_M:
         # decode shapes: the weight-streaming kernel applies SwiGLU row-wise in its epilogue
         lib = kernels()
@@ -307,21 +307,21 @@ def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tenso
         scratch = ws.ensure("gemm_scratch", scratch_b.value // 4) if scratch_b.value > 0 else None
         _require(counter_b.value // 4 <= ws.gemm_counters.numel(), "linear_swiglu: too many column tiles for counters")
         rc = lib.ff_gemm_skinny_swiglu(ptr(x), ptr(w_interleaved), ptr(out), m, n, k, ldx, ldw, out.stride(0), grid,
-                                       ptr(scratch), ptr(ws.gemm_counters), mode, ptr(status_tensor(x.device)), stream_ptr())
+                                       ptr(scratch), ptr(ws.gemm_counters), mode, c_float(limit), ptr(status_tensor(x.device)), stream_ptr())
         check(rc, "ff_gemm_skinny_swiglu")
         _count()
         return out
     args = (ptr(x), ptr(w_interleaved), ptr(out), m, n, k, ldx, ldw, out.stride(0))
     st = ptr(status_tensor(x.device))
-    rc = kernels().ff_gemm_bf16_geglu(*args, st, stream_ptr()) if mode == 3 else kernels().ff_gemm_bf16(*args, 1, st, stream_ptr())
+    rc = kernels().ff_gemm_bf16_gated(*args, mode, c_float(limit), st, stream_ptr()) if mode else kernels().ff_gemm_bf16(*args, 1, st, stream_ptr())
     check(rc, "ff_gemm_bf16(swiglu)")
     _count()
     return out
 
 
-def silu_mul_interleaved(gu: torch.Tensor, out: torch.Tensor | None = None, mode: int = 0) -> torch.Tensor:
+def silu_mul_interleaved(gu: torch.Tensor, out: torch.Tensor | None = None, mode: int = 0, limit: float = 0.0) -> torch.Tensor:
     """SwiGLU on the per-64 interleaved gate/up layout produced by the fused weight."""
-    return silu_mul(gu, mode=mode, out=out, interleaved=True)
+    return silu_mul(gu, mode=mode, limit=limit, out=out, interleaved=True)
 
 
 # ------------------------------------------------------------------------------------------
@@ -494,7 +494,7 @@ def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, v
                  dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0,
                  q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None,
                  cos_sin: torch.Tensor | None = None, whole: bool = False, halves: bool = False,
-                 temp: tuple[torch.Tensor, float, int] | None = None) -> None:
+                 temp: tuple[torch.Tensor, float, int] | None = None, norm_qk: bool = True, norm_v: bool = False) -> None:
     """Packed rows ``[q heads | k heads | v heads | ...]``: q and k are divided by their root mean square per head
     (``dim`` elements count, the row's heads may carry padding up to the cache's width), v is blended with
     ``first_v`` (``(1 - mix) v + mix first_v``; a column slice of an earlier layer's packed rows), k and v are written to
@@ -503,9 +503,10 @@ def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, v
 
     ``whole``: q and k are normed over all their heads together (weights then cover every head). ``halves``: elements (i, i + half)
     turn instead of neighbours. ``temp`` = (int32 positions, coef, every): the query at p is multiplied by
-    ``1 + coef ln((p + 1) // every + 1)``. ``hkv`` 0 (no caches): a row of queries alone."""
+    ``1 + coef ln((p + 1) // every + 1)``. ``hkv`` 0 (no caches): a row of queries alone. ``norm_qk`` False: q and k stay as they
+    are; ``norm_v``: values are divided by their root mean square per head."""
     if not _is_cuda(qkv):
-        ref.head_norm_kv(qkv, slots, kcache, vcache, hq, hkv, dim, vdim, eps, first_v, mix, q_weight, k_weight, cos_sin, whole, halves, temp)
+        ref.head_norm_kv(qkv, slots, kcache, vcache, hq, hkv, dim, vdim, eps, first_v, mix, q_weight, k_weight, cos_sin, whole, halves, temp, norm_qk, norm_v)
         return
     rows, ld = _rows2d(qkv)
     if hkv:
@@ -534,7 +535,7 @@ def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, v
     pos, coef, every = temp if temp is not None else (None, 0.0, 1)
     _require(pos is None or (pos.dtype == torch.int32 and pos.numel() == rows), "head_norm_kv: int32 positions")
     if whole or halves:
-        _require(first_v is None, "head_norm_kv: values are blended by the per-head form only")
+        _require(norm_qk and not norm_v and first_v is None, "head_norm_kv: values are blended by the per-head form only")
         rc = kernels().ff_row_norm_kv(ptr(qkv), ptr(slots), ptr(kcache), ptr(vcache), rows, hq, hkv, dim, dk, dv, bs, nb, ld, c_float(eps),
                                       ptr(q_weight), ptr(k_weight), ptr(cos_sin), half, int(whole), int(halves), ptr(pos), c_float(coef), every,
                                       int(qkv.dtype == torch.float32), ptr(status_tensor(qkv.device)), stream_ptr())
@@ -543,7 +544,8 @@ def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, v
         return
     rc = kernels().ff_head_norm_kv(ptr(qkv), ptr(slots), ptr(kcache), ptr(vcache), ptr(first_v), rows, hq, hkv, dim, dk, dv, bs, nb, ld,
                                    ldf, c_float(eps), c_float(mix), ptr(q_weight), ptr(k_weight), ptr(cos_sin), half, ptr(pos),
-                                   c_float(coef), every, int(qkv.dtype == torch.float32), ptr(status_tensor(qkv.device)), stream_ptr())
+                                   c_float(coef), every, int(norm_qk), vdim if norm_v else 0, int(qkv.dtype == torch.float32),
+                                   ptr(status_tensor(qkv.device)), stream_ptr())
     check(rc, "ff_head_norm_kv")
     _count()
 
@@ -580,10 +582,11 @@ def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0, out: torch.Ten
     rows, ld = _rows2d(gu)
     f = gu.shape[1] // 2
     if gu.dtype == torch.float32:          # 32-bit form: nothing in between is rounded
-        _require(mode in (0, 1, 2, 3), "silu_mul: the FP32 form has no clamped gate")
+        _require(mode in (0, 1, 2, 3, 5), "silu_mul: the FP32 form has no mode 4")
         if out is None:
             out = torch.empty(rows, f, dtype=torch.float32, device=gu.device)
-        check(kernels().ff_silu_mul_f32(ptr(gu), ptr(out), rows, f, ld, out.stride(0), mode, int(interleaved), stream_ptr()), "ff_silu_mul_f32")
+        check(kernels().ff_silu_mul_f32(ptr(gu), ptr(out), rows, f, ld, out.stride(0), mode, c_float(limit), int(interleaved), stream_ptr()),
+              "ff_silu_mul_f32")
         _count()
         return out
     if out is None:

@@ -126,11 +126,12 @@ __device__ __forceinline__ int comm_tm(int tm, int tiles_per_rank, int rank, int
 
 // Optional tail of the plain BF16 store (epi 0): bias per output column, then act 1 = square of the positive part or
 // 3 = tanh-GELU, then a factor per element (row mul_rows[row] of a table). All on the FP32 accumulator; the result is rounded once.
-// gate: activation of the gated epilogue (epi 1), 0 SiLU with the reference's roundings, 3 tanh-GELU with one rounding.
+// gate: activation of the gated epilogue (epi 1), 0 SiLU with the reference's roundings, 3 tanh-GELU with one rounding, 5 the clamped
+// gate (limit) with one rounding.
 struct LinTail {
   const __nv_bfloat16* bias; int act;
   const __nv_bfloat16* mul; const int* mul_rows; int ldm, mul_table;
-  int gate;
+  int gate; float limit;
 };
 
 constexpr int RS_STG_PITCH = 144, RS_STG_BYTES = 32 * RS_STG_PITCH;   // COMM 2 epilogue staging, per warp
@@ -263,6 +264,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
               const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
               const float u0 = __uint_as_float(u[2 * j]), u1 = __uint_as_float(u[2 * j + 1]);
               if (COMM == 0 && tail.gate == 3) { o[j] = pack_bf16x2(gelu_tanh_f(g0) * u0, gelu_tanh_f(g1) * u1); continue; }
+              if (COMM == 0 && tail.gate == 5) { o[j] = pack_bf16x2(gate_clamped_f(g0, u0, tail.limit), gate_clamped_f(g1, u1, tail.limit)); continue; }
               // rounding policy "mode 0" of the reference's silu_mul (kernels/act.cu:220-262):
               // gate and up are BF16 values, silu rounded to BF16, product rounded again.
               const float a0 = __bfloat162float(__float2bfloat16(silu_f(__bfloat162float(__float2bfloat16(g0)))));
@@ -599,11 +601,14 @@ FF_EXPORT int ff_gemm_bf16_act(const void* X, const void* W, void* Y, int M, int
                           status, stream);
 }
 
-// Gate/up projection (rows interleaved per 64) with tanh-GELU(gate) * up in the epilogue, rounded once. Y has N / 2 columns.
-FF_EXPORT int ff_gemm_bf16_geglu(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy, int* status,
-                                 cudaStream_t stream) {
+// Gate/up projection (rows interleaved per 64) with the activation in the epilogue, rounded once. gate 3: tanh-GELU(gate) * up, 5: the
+// clamped gate (`limit`). Y has N / 2 columns.
+FF_EXPORT int ff_gemm_bf16_gated(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy, int gate, float limit,
+                                 int* status, cudaStream_t stream) {
+  if (gate != 3 && gate != 5) return FF_HOST_UNSUPPORTED;
   LinTail tail = {};
-  tail.gate = 3;
+  tail.gate = gate;
+  tail.limit = limit;
   return gemm_bf16_launch(X, W, Y, M, N, K, ldx, ldw, ldy, 1, tail, status, stream);
 }
 
@@ -635,9 +640,10 @@ FF_EXPORT int ff_gemm_bf16_heads(const void* X, const void* W, void* Y, int M, i
 
 // Grouped GEMM over expert segments with 128-row token tiles (prefill sizes; the swap-AB kernel of moe.cu serves
 // segments of a few rows): Y[seg rows, Nw] = Xs[seg rows, K] · W[e][Nw, K]ᵀ. Xs [capacity, K] and Y rows are
-// addressed by seg_off / counts (device arrays, no host read-back); W is [E_local * Nw, K]. epi 0 / 1 as above.
+// addressed by seg_off / counts (device arrays, no host read-back); W is [E_local * Nw, K]. epi 0 / 1 as above; limit > 0: epi 1 applies
+// the clamped gate.
 FF_EXPORT int ff_moe_grouped_gemm_tiled(const void* Xs, const void* W, void* Y, const int* seg_off, const int* counts,
-                                        int E_local, int Nw, int K, int capacity, int ldy, int epi, int* status,
+                                        int E_local, int Nw, int K, int capacity, int ldy, int epi, float limit, int* status,
                                         cudaStream_t stream) {
   if (E_local <= 0 || Nw <= 0 || K <= 0 || capacity <= 0 || !seg_off || !counts) return FF_HOST_BAD_SHAPE;
   if ((K % 8) || (epi != 0 && epi != 1) || (epi == 1 && (Nw % 256))) return FF_HOST_BAD_SHAPE;
@@ -654,7 +660,9 @@ FF_EXPORT int ff_moe_grouped_gemm_tiled(const void* Xs, const void* W, void* Y, 
   r = opt_in_smem(kern, smem); if (r) return r;
   CommArgs none = {};
   GroupArgs ga = {seg_off, counts, E_local};
-  kern<<<sm_count(), 192, smem, stream>>>(tmA, tmA, tmA, tmB, Y, capacity, Nw, K, ldy, epi, status, none, ga, LinTail{});
+  LinTail tail = {};
+  if (limit > 0.f) { tail.gate = 5; tail.limit = limit; }
+  kern<<<sm_count(), 192, smem, stream>>>(tmA, tmA, tmA, tmB, Y, capacity, Nw, K, ldy, epi, status, none, ga, tail);
   return launch_result();
 }
 

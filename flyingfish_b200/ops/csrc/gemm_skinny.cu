@@ -50,22 +50,24 @@ struct alignas(8) SkinnyBars {
 
 // What is done to the finished sums of a plain tile: bias per column, act 1 square of the positive part, 2 nothing (Y is FP32), 3
 // tanh-GELU, then a factor per element (row mul_rows[token] of a table). gate: activation of a gated epilogue (SkinnyEpi mode 1), 0 SiLU
-// with the stand-alone kernel's roundings, 3 tanh-GELU on the FP32 sums, rounded once.
+// with the stand-alone kernel's roundings, 3 tanh-GELU on the FP32 sums, rounded once, 5 the clamped gate (limit) rounded once.
 struct SkinnyTail {
   const __nv_bfloat16* bias; int act;
   const __nv_bfloat16* mul; const int* mul_rows; int ldm, mul_table;
-  int gate;
+  int gate; float limit;
 };
 
 // emit_pair with the choice of the gate
-__device__ __forceinline__ void emit_gated(const SkinnyEpi& ep, int gate, __nv_bfloat16* __restrict__ Y, int N, int ldy, int t, int tile, int j8,
+__device__ __forceinline__ void emit_gated(const SkinnyEpi& ep, const SkinnyTail& tail, __nv_bfloat16* __restrict__ Y, int N, int ldy, int t, int tile, int j8,
                                            const float* lo, const float* hi, int* status) {
-  if (gate != 3) { emit_pair(ep, Y, N, ldy, t, tile, j8, lo, hi, status); return; }
+  if (tail.gate == 0) { emit_pair(ep, Y, N, ldy, t, tile, j8, lo, hi, status); return; }
   const int col = tile * 64 + j8 * 8;
   if (col >= N / 2) return;
   uint32_t o[4];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) o[j] = pack_bf16x2(gelu_tanh_f(lo[2 * j]) * hi[2 * j], gelu_tanh_f(lo[2 * j + 1]) * hi[2 * j + 1]);
+  for (int j = 0; j < 4; ++j)
+    o[j] = tail.gate == 5 ? pack_bf16x2(gate_clamped_f(lo[2 * j], hi[2 * j], tail.limit), gate_clamped_f(lo[2 * j + 1], hi[2 * j + 1], tail.limit))
+                          : pack_bf16x2(gelu_tanh_f(lo[2 * j]) * hi[2 * j], gelu_tanh_f(lo[2 * j + 1]) * hi[2 * j + 1]);
   *reinterpret_cast<uint4*>(Y + (size_t)t * ldy + col) = make_uint4(o[0], o[1], o[2], o[3]);
 }
 
@@ -424,7 +426,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
             if (t_own < M) {
 #pragma unroll
               for (int h = 0; h < 2; ++h)
-                emit_gated(ep, tail.gate, Y, N, ldy, t_own, sg.tile, (c >> 3) + h, reinterpret_cast<const float*>(g) + 8 * h,
+                emit_gated(ep, tail, Y, N, ldy, t_own, sg.tile, (c >> 3) + h, reinterpret_cast<const float*>(g) + 8 * h,
                           reinterpret_cast<const float*>(u) + 8 * h, status);
             }
           }
@@ -527,7 +529,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
 #pragma unroll
             for (int g = 0; g < 4; g += 2) {
               const int pr = i0 + 128 * (g >> 1);
-              if (pr < i_end) emit_gated(ep, tail.gate, Y, N, ldy, pr >> 3, sg.tile, pr & 7, a8[g], a8[g + 1], status);
+              if (pr < i_end) emit_gated(ep, tail, Y, N, ldy, pr >> 3, sg.tile, pr & 7, a8[g], a8[g + 1], status);
             }
           } else {
 #pragma unroll
@@ -565,7 +567,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
               lo[0] += l0.x; lo[1] += l0.y; lo[2] += l0.z; lo[3] += l0.w; lo[4] += l1.x; lo[5] += l1.y; lo[6] += l1.z; lo[7] += l1.w;
               hi[0] += h0.x; hi[1] += h0.y; hi[2] += h0.z; hi[3] += h0.w; hi[4] += h1.x; hi[5] += h1.y; hi[6] += h1.z; hi[7] += h1.w;
             }
-            emit_gated(ep, tail.gate, Y, N, ldy, crank + ti * cl_size, sg.tile, j8, lo, hi, status);
+            emit_gated(ep, tail, Y, N, ldy, crank + ti * cl_size, sg.tile, j8, lo, hi, status);
           }
         } else
         for (int i = e; i < rows * vpr; i += 128) {
@@ -918,14 +920,15 @@ FF_EXPORT int ff_gemm_skinny_f32out(const void* X, const void* W, float* Y, int 
 }
 
 // Gate/up projection with the SwiGLU applied in the epilogue: W is [N, K] with gate/up rows interleaved per
-// 64, Y is [M, N/2]. gate 0: SiLU, 3: tanh-GELU rounded once. `grid` from ff_gemm_skinny_plan_epi(M, N, K, 1).
+// 64, Y is [M, N/2]. gate 0: SiLU, 3: tanh-GELU, 5: clamped gate (`limit`), both rounded once. `grid` from ff_gemm_skinny_plan_epi(M, N, K, 1).
 FF_EXPORT int ff_gemm_skinny_swiglu(const void* X, const void* W, void* Y, int M, int N, int K, int ldx, int ldw, int ldy,
-                                    int grid, float* scratch, int* counters, int gate, int* status, cudaStream_t stream) {
-  if (gate != 0 && gate != 3) return FF_HOST_UNSUPPORTED;
+                                    int grid, float* scratch, int* counters, int gate, float limit, int* status, cudaStream_t stream) {
+  if (gate != 0 && gate != 3 && gate != 5) return FF_HOST_UNSUPPORTED;
   SkinnyEpi ep = {};
   ep.mode = 1;
   SkinnyTail tail = {};
   tail.gate = gate;
+  tail.limit = limit;
   return gemm_skinny_launch(X, W, Y, M, N, K, ldx, ldw, ldy, grid, scratch, counters, status, stream, nullptr, &ep, tail);
 }
 

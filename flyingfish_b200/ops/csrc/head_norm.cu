@@ -6,6 +6,7 @@
 //   q <- rot(q / rms(q) * wq)            in the row         (weights and rotation where they are given: neighbours 2i, 2i + 1 of
 //   k <- rot(k / rms(k) * wk)            to its slot         the first elements turn by the row's table of cosines and sines)
 //                                        to its slot of the K cache [block][kv head][block_size][dk]
+//   (q and k may also stay as they are: then q is not touched; v may be divided by its root mean square)
 //   v <- (1 - mix) v + mix first_v       to its slot of the V cache (first_v: the same token's values of an earlier layer)
 // FP32 arithmetic, BF16 or FP32 storage. A group of G lanes owns one head of one row and keeps it in registers.
 // Optional query temperature: the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
@@ -27,20 +28,23 @@ __device__ __forceinline__ float query_factor(const QueryTemp& t, int row) {
   return 1.0f + t.coef * logf((float)((max(t.positions[row], 0) + 1) / t.every) + 1.0f);
 }
 
+// Which heads are normed: qk 0: q and k stay as they are; vdim > 0: values are divided by their root mean square over vdim elements.
+struct HeadForm { int qk = 1, vdim = 0; };
+
 // NV: vectors of 8 elements a lane holds
 template <typename T, int G, int NV>
 __global__ void __launch_bounds__(HN_THREADS)
 head_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __restrict__ kcache, T* __restrict__ vcache,
                     const T* __restrict__ first_v, int rows, int hq, int hkv, int dim, int dk, int dv, int block_size, int num_blocks,
                     int ld, int ldf, float eps, float mix, const float* __restrict__ wq, const float* __restrict__ wk,
-                    const float2* __restrict__ cos_sin, int half, const QueryTemp temp, int* status) {
+                    const float2* __restrict__ cos_sin, int half, const QueryTemp temp, const HeadForm form, int* status) {
   pdl_trigger();
   pdl_wait();
-  const int heads = hq + 2 * hkv;
+  const int first = form.qk ? 0 : hq, heads = hq + 2 * hkv - first;
   const long long item = ((long long)blockIdx.x * HN_THREADS + threadIdx.x) / G;
   const int gl = threadIdx.x & (G - 1);
   const bool live = item < (long long)rows * heads;
-  const int row = live ? (int)(item / heads) : 0, head = live ? (int)(item % heads) : 0;
+  const int row = live ? (int)(item / heads) : 0, head = first + (live ? (int)(item % heads) : 0);
   const bool is_q = head < hq, is_v = head >= hq + hkv;
   const int d = is_v ? dv : dk;
   T* base = qkv + (size_t)row * ld + (is_v ? (size_t)(hq + hkv) * dk + (size_t)(head - hq - hkv) * dv : (size_t)head * dk);
@@ -58,7 +62,14 @@ head_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __res
 #pragma unroll
   for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o, G);
   if (!live) return;
-  if (!is_v) {
+  if (is_v && form.vdim > 0) {
+    const float r = 1.0f / sqrtf(ss / (float)form.vdim + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] *= r;
+  }
+  if (!is_v && form.qk) {
     const float r = 1.0f / sqrtf(ss / (float)dim + eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i)
@@ -99,7 +110,7 @@ head_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __res
 #pragma unroll
         for (int j = 0; j < 8; ++j) v[i][j] *= f;
     }
-  } else if (first_v != nullptr) {
+  } else if (is_v && first_v != nullptr) {
     const T* fv = first_v + (size_t)row * ldf + (size_t)(head - hq - hkv) * dv;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
@@ -132,13 +143,13 @@ head_norm_kv_kernel(T* __restrict__ qkv, const int* __restrict__ slots, T* __res
 template <typename T>
 static int head_norm_launch(void* qkv, const int* slots, void* kcache, void* vcache, const void* first_v, int rows, int hq, int hkv, int dim,
                             int dk, int dv, int block_size, int num_blocks, int ld, int ldf, float eps, float mix, const float* wq, const float* wk,
-                            const float2* cos_sin, int half, const QueryTemp& temp, int* status, cudaStream_t s) {
+                            const float2* cos_sin, int half, const QueryTemp& temp, const HeadForm& form, int* status, cudaStream_t s) {
   const int vecs = (dk > dv ? dk : dv) / 8;
-  const long long items = (long long)rows * (hq + 2 * hkv);
+  const long long items = (long long)rows * ((form.qk ? hq : 0) + 2 * hkv);
   auto go = [&](auto kern, int g) -> int {
     const long long blocks = (items * g + HN_THREADS - 1) / HN_THREADS;
     if (int r = launch_pdl(kern, dim3((unsigned)blocks), dim3(HN_THREADS), 0, s, 0, (T*)qkv, slots, (T*)kcache, (T*)vcache, (const T*)first_v,
-                           rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, wq, wk, cos_sin, half, temp, status)) return r;
+                           rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, wq, wk, cos_sin, half, temp, form, status)) return r;
     return launch_result();
   };
   if (vecs <= 8) return go(head_norm_kv_kernel<T, 8, 1>, 8);
@@ -388,17 +399,20 @@ FF_EXPORT int ff_latent_norm_kv(const void* p, const int* slots, void* cache, vo
 }
 
 // wq, wk: FP32 norm weights of dk elements, or null; cos_sin: float2 [rows, half], or null; positions: query temperature, or null;
-// hkv = 0: queries only
+// hkv = 0: queries only; norm_qk, v_norm_dim: HeadForm
 FF_EXPORT int ff_head_norm_kv(void* qkv, const int* slots, void* kcache, void* vcache, const void* first_v, int rows, int hq, int hkv,
                               int dim, int dk, int dv, int block_size, int num_blocks, int ld, int ldf, float eps, float mix,
                               const float* wq, const float* wk, const float* cos_sin, int half, const int* positions, float coef,
-                              int every, int f32, int* status, cudaStream_t s) {
+                              int every, int norm_qk, int v_norm_dim, int f32, int* status, cudaStream_t s) {
+  if (!norm_qk && (hkv == 0 || wq != nullptr || wk != nullptr || cos_sin != nullptr || positions != nullptr)) return FF_HOST_UNSUPPORTED;
+  if (v_norm_dim < 0 || v_norm_dim > dv) return FF_HOST_BAD_SHAPE;
+  const HeadForm form = {norm_qk, v_norm_dim};
   if (rows <= 0 || hq <= 0 || hkv < 0 || (positions != nullptr && every < 1) || dim <= 0 || dk < dim || dk % 8 || dv <= 0 || dv % 8 || block_size <= 0) return FF_HOST_BAD_SHAPE;
   if (half < 0 || 2 * half > dim || (cos_sin != nullptr && half == 0)) return FF_HOST_BAD_SHAPE;
   if ((reinterpret_cast<uintptr_t>(wq) & 15) || (reinterpret_cast<uintptr_t>(wk) & 15)) return FF_HOST_BAD_ALIGN;
   const float2* cs = reinterpret_cast<const float2*>(cos_sin);
   const QueryTemp temp = {positions, coef, every};
   if (ld % 8 || (first_v != nullptr && ldf % 8)) return FF_HOST_BAD_ALIGN;
-  if (f32) return head_norm_launch<float>(qkv, slots, kcache, vcache, first_v, rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, wq, wk, cs, half, temp, status, s);
-  return head_norm_launch<__nv_bfloat16>(qkv, slots, kcache, vcache, first_v, rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, wq, wk, cs, half, temp, status, s);
+  if (f32) return head_norm_launch<float>(qkv, slots, kcache, vcache, first_v, rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, wq, wk, cs, half, temp, form, status, s);
+  return head_norm_launch<__nv_bfloat16>(qkv, slots, kcache, vcache, first_v, rows, hq, hkv, dim, dk, dv, block_size, num_blocks, ld, ldf, eps, mix, wq, wk, cs, half, temp, form, status, s);
 }

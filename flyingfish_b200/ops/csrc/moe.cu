@@ -9,7 +9,7 @@
 //   moe_grouped_gemm : Y[seg rows, N] = Xsorted[seg rows, K] · W[e][N, K]ᵀ for every expert segment,
 //                   swap-AB on tcgen05 (a 128-row slice of the expert weight is the UMMA A operand,
 //                   up to 256 tokens of the segment are the UMMA N dimension), optional SwiGLU
-//                   epilogue for gate/up weights interleaved per 64 rows
+//                   epilogue (or the clamped gate, limit > 0) for gate/up weights interleaved per 64 rows
 //   moe_combine   : FP32 sum of a row's k contributions in ascending expert id, one BF16 rounding
 // Semantics follow kernels/moe_route.cu:1-30,155-390, kernels/moe_prefill.cu and
 // kernels/moe_combine.cu:1-96 of the reference.
@@ -20,7 +20,7 @@ namespace ff {
 
 // ---------------------------------------------------------------------------------------
 // routing: one warp per row, scores in shared memory
-// score_mode: 0 softmax (bias: for the selection only), 1 sigmoid, 2 noaux (sigmoid + bias for selection, groups), 3 as 2 with sqrt(softplus(x)) scores
+// score_mode: 0 softmax (bias: for the selection only), 4 softmax of the logits with the bias added, 1 sigmoid, 2 noaux (sigmoid + bias for selection, groups), 3 as 2 with sqrt(softplus(x)) scores
 // ---------------------------------------------------------------------------------------
 constexpr int ROUTE_WARPS = 4;
 constexpr int ROUTE_MAX_E = 512;
@@ -40,12 +40,14 @@ template <typename T>
 __device__ __forceinline__ void route_row(const T* __restrict__ lg, const float* __restrict__ bias, float* sc, float* sel, int row, int E,
                                           int top_k, int score_mode, int n_groups, int topk_groups, int lane, float& my_w, int& my_id,
                                           float& wsum, int* status) {
-  if (score_mode == 0) {
+  if (score_mode == 0 || score_mode == 4) {
+    const float* add = score_mode == 4 ? bias : nullptr;
+    if (score_mode == 4) bias = nullptr;
     float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, to_float(lg[e]));
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, to_float(lg[e]) + (add ? add[e] : 0.f));
     mx = warp_max(mx);
     float sum = 0.f;
-    for (int e = lane; e < E; e += 32) { const float v = expf(to_float(lg[e]) - mx); sc[e] = v; sum += v; }
+    for (int e = lane; e < E; e += 32) { const float v = expf(to_float(lg[e]) + (add ? add[e] : 0.f) - mx); sc[e] = v; sum += v; }
     sum = warp_sum(sum);
     const float inv = 1.0f / sum;
     for (int e = lane; e < E; e += 32) { sc[e] *= inv; sel[e] = bias ? sc[e] + bias[e] : sc[e]; }
@@ -58,7 +60,7 @@ __device__ __forceinline__ void route_row(const T* __restrict__ lg, const float*
     }
   }
   __syncwarp();
-  if (score_mode >= 2 && n_groups > 1) {
+  if ((score_mode == 2 || score_mode == 3) && n_groups > 1) {
     const int gsz = E / n_groups;
     // group score = sum of the two best selection scores of the group
     float gscore = -INFINITY;
@@ -276,7 +278,7 @@ __device__ __forceinline__ float bfr(float x) { return __bfloat162float(__float2
 __global__ void __launch_bounds__(192, 1)
 moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
                         __nv_bfloat16* __restrict__ Y, const int* __restrict__ seg_off, const int* __restrict__ counts,
-                        int Nw, int K, int ldy, int epi, int pipe_bytes, int stage_off, int* status, int capacity) {
+                        int Nw, int K, int ldy, int epi, float limit, int pipe_bytes, int stage_off, int* status, int capacity) {
   pdl_trigger();
   pdl_wait();
   int stages;
@@ -384,6 +386,11 @@ moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_co
 #pragma unroll
               for (int j = 0; j < 4; ++j) {
                 const int col = c8 * 8 + 2 * j;
+                if (limit > 0.f) {                          // clamped gate, rounded once
+                  o[j] = pack_bf16x2(gate_clamped_f(sT[t * GBM + col], sT[t * GBM + 64 + col], limit),
+                                     gate_clamped_f(sT[t * GBM + col + 1], sT[t * GBM + 64 + col + 1], limit));
+                  continue;
+                }
                 const float g0 = bfr(sT[t * GBM + col]), g1 = bfr(sT[t * GBM + col + 1]);
                 const float u0 = bfr(sT[t * GBM + 64 + col]), u1 = bfr(sT[t * GBM + 64 + col + 1]);
                 o[j] = pack_bf16x2(bfr(silu_g(g0)) * u0, bfr(silu_g(g1)) * u1);
@@ -527,7 +534,7 @@ FF_EXPORT int ff_moe_dispatch_local(const void* x, const int* ids, int rows, int
 }
 
 FF_EXPORT int ff_moe_grouped_gemm(const void* xs, const void* w, void* y, const int* seg_off, const int* counts,
-                                  int E_local, int Nw, int K, int capacity, int ldy, int epi, int* status,
+                                  int E_local, int Nw, int K, int capacity, int ldy, int epi, float limit, int* status,
                                   cudaStream_t s) {
   // a plain store cuts its last tile at Nw (multiples of 8); the SwiGLU epilogue takes whole 128-row tiles
   if (E_local < 1 || Nw % (epi == 1 ? 128 : 8) || K % 8 || capacity % 16) return FF_HOST_BAD_SHAPE;
@@ -547,7 +554,7 @@ FF_EXPORT int ff_moe_grouped_gemm(const void* xs, const void* w, void* y, const 
   const int smem = staging + pipe_bytes + 1024;
   r = opt_in_smem(moe_grouped_gemm_kernel, 200 * 1024); if (r) return r;
   dim3 grid((Nw + GBM - 1) / GBM, E_local);
-  if (int lr = launch_pdl(moe_grouped_gemm_kernel, grid, dim3(192), smem, s, 0, tmW, tmX, (__nv_bfloat16*)y, seg_off, counts, Nw, K, ldy, epi,
+  if (int lr = launch_pdl(moe_grouped_gemm_kernel, grid, dim3(192), smem, s, 0, tmW, tmX, (__nv_bfloat16*)y, seg_off, counts, Nw, K, ldy, epi, limit,
                           pipe_bytes, staging, status, capacity)) return lr;
   return launch_result();
 }

@@ -357,6 +357,12 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   return __fdividef(z, 1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
+// clamped gate of an expert: g sigmoid(1.702 g) (u + 1) with g at most `limit` and u within it
+__device__ __forceinline__ float gate_clamped_f(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fmaxf(fminf(u, limit), -limit);
+  return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+}
 __device__ __forceinline__ float2 unpack_bf16x2(uint32_t u) {
   __nv_bfloat162 v = *reinterpret_cast<__nv_bfloat162*>(&u);
   return __bfloat1622float2(v);

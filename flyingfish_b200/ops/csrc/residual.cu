@@ -1,6 +1,9 @@
 // FP32 residual stream of layers whose mixer and feed-forward read the same rows through two norms (parallel layers):
 //   embed : x = table[id] * scale
 //   step  : x += a + b + sum_j w_j y_j          a, b: rows of the mixer and of a dense or shared feed-forward
+// With inner norms (a second mixer beside the first, embeddings of bigrams beside those of tokens):
+//   embed : x = t / rms(t) * w,  t = table[id] + table2[id2]         bigram_rows: id2 from the token and the one before it
+//   step  : x += a / rms(a) * wa + a2 / rms(a2) * wa2 + b + ..
 //   n1 = x / rms(x) * w1     n2 = x / rms(x) * w2      the operands of the next layer (n2 optional)
 // The sum over a row's chosen experts is taken here, straight from the rows the grouped GEMM wrote (y_j = y[pos_j]; a choice
 // beyond the last expert is an identity output: y_j is the row h the experts were given), so a layer ends in one kernel: the
@@ -13,6 +16,7 @@
 // statistics of the row); outer may also be a plain copy in the GEMM operand's type.
 #include "dtype_io.cuh"
 #include "host_util.h"
+#include <type_traits>
 
 namespace ff {
 
@@ -26,10 +30,24 @@ struct ExpertRows {
   int top, experts, ldy;
 };
 
-template <typename T, bool EMBED>
+// inner norms; t2, rows2: the second table and its row per row of the batch (embed), a2: rows of the second mixer (step)
+template <typename T>
+struct InnerNorms { const T* t2; const int* rows2; int rows_t2; const T* a2; const float* w; const float* w2; };
+
+// all threads of the block: one over the root mean square from the threads' sums of squares
+__device__ __forceinline__ float block_rms(float ss, float* s_red, int true_width, float eps) {
+  ss = warp_sum(ss);
+  __syncthreads();                                         // the previous reduction has been read
+  if ((threadIdx.x & 31) == 0) s_red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  const float tot = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? s_red[threadIdx.x & 31] : 0.f);
+  return 1.0f / sqrtf(tot / (float)true_width + eps);
+}
+
+template <typename T, bool EMBED, bool INNER>
 __global__ void __launch_bounds__(RN_THREADS)
 residual_norms_kernel(float* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ table, float scale, int vocab,
-                      const T* __restrict__ a, const T* __restrict__ b, const ExpertRows<T> ex, const float* __restrict__ w1,
+                      const T* __restrict__ a, const T* __restrict__ b, const ExpertRows<T> ex, const InnerNorms<T> in, const float* __restrict__ w1,
                       const float* __restrict__ w2, T* __restrict__ n1, T* __restrict__ n2, int width, int true_width, float eps,
                       int* status) {
   pdl_trigger();
@@ -53,6 +71,33 @@ residual_norms_kernel(float* __restrict__ x, const int* __restrict__ ids, const 
     __syncthreads();
   }
   float* xr = x + (size_t)row * width;
+  float ra = 1.f, ra2 = 1.f;
+  const T* src2 = nullptr;
+  if constexpr (INNER) {
+    const T* one = EMBED ? src : a + (size_t)row * width;
+    if (EMBED) {
+      int r2 = in.rows2[row];
+      if (r2 < 0 || r2 >= in.rows_t2) { if (tid == 0) set_status(status, KID_EMBED, FF_ERR_BOUNDS, row, r2); r2 = 0; }
+      src2 = in.t2 + (size_t)r2 * width;
+    } else {
+      src2 = in.a2 + (size_t)row * width;
+    }
+    float s1 = 0.f, s2 = 0.f;
+    for (int c = tid * 4; c < width; c += blockDim.x * 4) {
+      float u[4], t[4];
+      load4(one + c, u);
+      load4(src2 + c, t);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        if (EMBED) u[j] = u[j] * scale + t[j];
+        s1 = fmaf(u[j], u[j], s1);
+        s2 = fmaf(t[j], t[j], s2);
+      }
+    }
+    ra = block_rms(s1, s_red, true_width, eps);
+    if (!EMBED) ra2 = block_rms(s2, s_red, true_width, eps);
+    __syncthreads();
+  }
   float ss = 0.f;
   for (int c = tid * 4; c < width; c += blockDim.x * 4) {
     float v[4];
@@ -60,10 +105,25 @@ residual_norms_kernel(float* __restrict__ x, const int* __restrict__ ids, const 
       load4(src + c, v);
 #pragma unroll
       for (int j = 0; j < 4; ++j) v[j] *= scale;
+      if constexpr (INNER) {
+        float t[4], f[4];
+        load4(src2 + c, t);
+        load4(in.w + c, f);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[j] = (v[j] + t[j]) * ra * f[j];
+      }
     } else {
       float t[4];
       load4(xr + c, v);
       load4(a + (size_t)row * width + c, t);
+      if constexpr (INNER) {
+        float f[4], u[4], f2[4];
+        load4(in.w + c, f);
+        load4(src2 + c, u);
+        load4(in.w2 + c, f2);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) t[j] = t[j] * ra * f[j] + u[j] * ra2 * f2[j];
+      }
 #pragma unroll
       for (int j = 0; j < 4; ++j) v[j] += t[j];
       if (b != nullptr) {
@@ -107,21 +167,39 @@ residual_norms_kernel(float* __restrict__ x, const int* __restrict__ ids, const 
   }
 }
 
-template <typename T, bool EMBED>
+// rows of a second embedding table: (previous token * mul_prev + token * mul_cur) mod buckets, `buckets` for a sequence's first token.
+// The previous token of a sequence's first new row is its state (negative: none), which then takes the last one. A block per sequence.
+__global__ void __launch_bounds__(256)
+bigram_rows_kernel(const int* __restrict__ ids, int* __restrict__ out, int* __restrict__ last, const int* __restrict__ row_start,
+                   const int* __restrict__ slots, int buckets, long long mul_prev, long long mul_cur) {
+  pdl_trigger();
+  pdl_wait();
+  const int r0 = row_start[blockIdx.x], r1 = row_start[blockIdx.x + 1], slot = slots[blockIdx.x];
+  if (r1 <= r0) return;
+  for (int r = r0 + threadIdx.x; r < r1; r += blockDim.x) {
+    const int before = r == r0 ? last[slot] : max(ids[r - 1], 0);     // ids outside the vocabulary are reported by the embedding
+    out[r] = before < 0 ? buckets : (int)((before * mul_prev + max(ids[r], 0) * mul_cur) % buckets);
+  }
+  if (threadIdx.x == 0) last[slot] = ids[r1 - 1];          // the thread that read it
+}
+
+template <typename T, bool EMBED, bool INNER>
 static int residual_launch(float* x, const int* ids, const void* table, float scale, int vocab, const void* a, const void* b,
-                           const ExpertRows<T>& ex, const float* w1, const float* w2, void* n1, void* n2, int rows, int width, int true_width,
+                           const ExpertRows<T>& ex, const InnerNorms<T>& in, const float* w1, const float* w2, void* n1, void* n2, int rows, int width, int true_width,
                            float eps, int* status, cudaStream_t s) {
   if (rows <= 0 || width <= 0 || width % 8 || true_width <= 0 || true_width > width || (w2 == nullptr) != (n2 == nullptr)) return FF_HOST_BAD_SHAPE;
   if (ex.top < 0 || ex.top > RN_TOP_MAX || (ex.top > 0 && (ex.ldy % 8 || ex.pos == nullptr || ex.ids == nullptr || ex.w == nullptr))) return FF_HOST_BAD_SHAPE;
   const int smem = width * 4;
   if (smem > 200 * 1024) return FF_HOST_TOO_LARGE;
-  auto kern = residual_norms_kernel<T, EMBED>;
+  if ((reinterpret_cast<uintptr_t>(in.w) & 15) || (reinterpret_cast<uintptr_t>(in.w2) & 15)) return FF_HOST_BAD_ALIGN;
+  if (INNER && (in.w == nullptr || (EMBED ? in.t2 == nullptr || in.rows2 == nullptr : in.a2 == nullptr || in.w2 == nullptr))) return FF_HOST_BAD_SHAPE;
+  auto kern = residual_norms_kernel<T, EMBED, INNER>;
   if (int r = opt_in_smem(kern, smem)) return r;
   int threads = (width / 4 + 31) / 32 * 32;
   // a few rows (a decode step): wide blocks, for latency; many: more, smaller blocks per SM keep more loads in flight
   const int cap = rows >= 2 * sm_count() ? RN_THREADS / 2 : RN_THREADS;
   if (threads > cap) threads = cap;
-  if (int r = launch_pdl(kern, dim3(rows), dim3(threads), smem, s, 0, x, ids, (const T*)table, scale, vocab, (const T*)a, (const T*)b, ex, w1,
+  if (int r = launch_pdl(kern, dim3(rows), dim3(threads), smem, s, 0, x, ids, (const T*)table, scale, vocab, (const T*)a, (const T*)b, ex, in, w1,
                          w2, (T*)n1, (T*)n2, width, true_width, eps, status)) return r;
   return launch_result();
 }
@@ -152,16 +230,6 @@ __device__ __forceinline__ void apply_norm(const NormArgs& a, int c, float r, fl
   load4(a.b + c, b);
 #pragma unroll
   for (int j = 0; j < 4; ++j) v[j] = fmaf(norm_tanh(a.alpha * v[j], T()), w[j], b[j]);
-}
-
-// all threads of the block: one over the root mean square from the threads' sums of squares
-__device__ __forceinline__ float block_rms(float ss, float* s_red, int true_width, float eps) {
-  ss = warp_sum(ss);
-  __syncthreads();                                         // the previous reduction has been read
-  if ((threadIdx.x & 31) == 0) s_red[threadIdx.x >> 5] = ss;
-  __syncthreads();
-  const float tot = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? s_red[threadIdx.x & 31] : 0.f);
-  return 1.0f / sqrtf(tot / (float)true_width + eps);
 }
 
 template <typename T, bool EMBED>
@@ -273,22 +341,42 @@ FF_EXPORT int ff_residual_add_normed(float* x, const void* y, int ikind, const f
   return sandwich_launch<__nv_bfloat16, false>(x, nullptr, nullptr, 1.f, 0, y, inner, outer, n, rows, width, true_width, eps, nullptr, s);
 }
 
-// x FP32 [rows, width]; table, n1, n2 in BF16 (f32 = 0) or FP32; w1, w2 FP32 [width] (w2, n2: both or neither)
-FF_EXPORT int ff_residual_embed(const int* ids, const void* table, float scale, float* x, const float* w1, const float* w2, void* n1, void* n2,
-                                int rows, int width, int true_width, int vocab, float eps, int f32, int* status, cudaStream_t s) {
-  if (f32) return residual_launch<float, true>(x, ids, table, scale, vocab, nullptr, nullptr, ExpertRows<float>{}, w1, w2, n1, n2, rows, width, true_width, eps, status, s);
-  return residual_launch<__nv_bfloat16, true>(x, ids, table, scale, vocab, nullptr, nullptr, ExpertRows<__nv_bfloat16>{}, w1, w2, n1, n2, rows, width, true_width, eps, status, s);
+// x FP32 [rows, width]; table, n1, n2 in BF16 (f32 = 0) or FP32; w1, w2 FP32 [width] (w2, n2: both or neither). table2 [rows_t2, width],
+// rows2 [rows], w_in FP32 [width]: the second table and the norm of the sum, or null
+FF_EXPORT int ff_residual_embed(const int* ids, const void* table, float scale, const void* table2, const int* rows2, int rows_t2, const float* w_in,
+                                float* x, const float* w1, const float* w2, void* n1, void* n2, int rows, int width, int true_width, int vocab,
+                                float eps, int f32, int* status, cudaStream_t s) {
+  auto go = [&](auto* t) -> int {
+    using T = std::remove_pointer_t<decltype(t)>;
+    const InnerNorms<T> in = {(const T*)table2, rows2, rows_t2, nullptr, w_in, nullptr};
+    if (table2 != nullptr)
+      return residual_launch<T, true, true>(x, ids, table, scale, vocab, nullptr, nullptr, ExpertRows<T>{}, in, w1, w2, n1, n2, rows, width, true_width, eps, status, s);
+    return residual_launch<T, true, false>(x, ids, table, scale, vocab, nullptr, nullptr, ExpertRows<T>{}, in, w1, w2, n1, n2, rows, width, true_width, eps, status, s);
+  };
+  return f32 ? go((float*)nullptr) : go((__nv_bfloat16*)nullptr);
 }
 
-// a: [rows, width]; b: the same or null; y, pos, eids, ew, h: the experts' rows, the row of every choice (negative: none), the
-// choices [rows, top] and weights, and the experts' input (top = 0: no experts)
-FF_EXPORT int ff_residual_step(float* x, const void* a, const void* b, const void* y, const int* pos, const int* eids, const float* ew,
-                               const void* h, int top, int experts, int ldy, const float* w1, const float* w2, void* n1, void* n2, int rows,
-                               int width, int true_width, float eps, int f32, cudaStream_t s) {
-  if (f32) {
-    const ExpertRows<float> ex = {(const float*)y, pos, eids, ew, (const float*)h, top, experts, ldy};
-    return residual_launch<float, false>(x, nullptr, nullptr, 1.f, 0, a, b, ex, w1, w2, n1, n2, rows, width, true_width, eps, nullptr, s);
-  }
-  const ExpertRows<__nv_bfloat16> ex = {(const __nv_bfloat16*)y, pos, eids, ew, (const __nv_bfloat16*)h, top, experts, ldy};
-  return residual_launch<__nv_bfloat16, false>(x, nullptr, nullptr, 1.f, 0, a, b, ex, w1, w2, n1, n2, rows, width, true_width, eps, nullptr, s);
+// a: [rows, width]; a2: the same or null, then wa and wa2 FP32 [width] are the weights of the norms of both; b: the same or null; y, pos,
+// eids, ew, h: the experts' rows, the row of every choice (negative: none), the choices [rows, top] and weights, and the experts' input
+// (top = 0: no experts)
+FF_EXPORT int ff_residual_step(float* x, const void* a, const void* a2, const float* wa, const float* wa2, const void* b, const void* y,
+                               const int* pos, const int* eids, const float* ew, const void* h, int top, int experts, int ldy, const float* w1,
+                               const float* w2, void* n1, void* n2, int rows, int width, int true_width, float eps, int f32, cudaStream_t s) {
+  auto go = [&](auto* t) -> int {
+    using T = std::remove_pointer_t<decltype(t)>;
+    const ExpertRows<T> ex = {(const T*)y, pos, eids, ew, (const T*)h, top, experts, ldy};
+    const InnerNorms<T> in = {nullptr, nullptr, 0, (const T*)a2, wa, wa2};
+    if (a2 != nullptr)
+      return residual_launch<T, false, true>(x, nullptr, nullptr, 1.f, 0, a, b, ex, in, w1, w2, n1, n2, rows, width, true_width, eps, nullptr, s);
+    return residual_launch<T, false, false>(x, nullptr, nullptr, 1.f, 0, a, b, ex, in, w1, w2, n1, n2, rows, width, true_width, eps, nullptr, s);
+  };
+  return f32 ? go((float*)nullptr) : go((__nv_bfloat16*)nullptr);
+}
+
+// ids int[rows], out int[rows], last int[slots]
+FF_EXPORT int ff_bigram_rows(const int* ids, int* out, int* last, const int* row_start, const int* slots, int sequences, int buckets,
+                             long long mul_prev, long long mul_cur, cudaStream_t s) {
+  if (sequences <= 0 || buckets < 1 || mul_prev < 0 || mul_cur < 0) return FF_HOST_BAD_SHAPE;
+  if (int r = launch_pdl(bigram_rows_kernel, dim3(sequences), dim3(256), 0, s, 0, ids, out, last, row_start, slots, buckets, mul_prev, mul_cur)) return r;
+  return launch_result();
 }

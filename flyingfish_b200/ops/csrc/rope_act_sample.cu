@@ -88,6 +88,7 @@ __global__ void rope_kv_paged_kernel(__nv_bfloat16* __restrict__ qkv, const int*
 
 // mode 0: bf16(silu(g)) * u rounded again   mode 1: single rounding
 // mode 2: tanh-GELU(g) twice rounded         mode 4: clamped (DeepSeek) form in FP32, limit given
+// mode 5: gate_clamped_f
 __device__ __forceinline__ float act_combine(float g, float u, int mode, float limit) {
   if (mode == 0) return bf16r(g / (1.f + __expf(-g))) * u;
   if (mode == 1) return (g / (1.f + __expf(-g))) * u;
@@ -97,6 +98,7 @@ __device__ __forceinline__ float act_combine(float g, float u, int mode, float l
     return bf16r(0.5f * g * (1.f + t)) * u;
   }
   if (mode == 3) return gelu_tanh_f(g) * u;
+  if (mode == 5) return gate_clamped_f(g, u, limit);
   // clamped: gate <= limit, up in [-limit, limit]
   g = fminf(g, limit); u = fmaxf(fminf(u, limit), -limit);
   return (g / (1.f + __expf(-g))) * u;
@@ -142,9 +144,9 @@ __global__ void silu_mul_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloa
   reinterpret_cast<uint4*>(out + (size_t)row * ldo)[c] = o;
 }
 
-// the same in FP32 (no intermediate rounding; mode 2 and 3: tanh-GELU, otherwise SiLU), four elements per thread
+// the same in FP32 (no intermediate rounding; mode 2 and 3: tanh-GELU, 5: clamped gate, otherwise SiLU), four elements per thread
 __global__ void silu_mul_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int f, int ldgu, int ldo,
-                                    int mode, int interleaved) {
+                                    int mode, float limit, int interleaved) {
   pdl_trigger();
   pdl_wait();
   const int vec_per_row = f >> 2;
@@ -157,6 +159,11 @@ __global__ void silu_mul_f32_kernel(const float* __restrict__ gu, float* __restr
   load4(gu + (size_t)row * ldgu + uc, u);
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
+    if (mode == 5) {
+      const float c = fminf(g[j], limit);
+      g[j] = c * sigmoid_f(1.702f * c) * (fmaxf(fminf(u[j], limit), -limit) + 1.0f);
+      continue;
+    }
     const float z = g[j];
     g[j] = (mode >= 2 ? 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))) : z * sigmoid_f(z)) * u[j];
   }
@@ -458,12 +465,12 @@ FF_EXPORT int ff_silu_mul(const void* gu, void* out, int rows, int f, int ldgu, 
   return launch_result();
 }
 
-// gate/up rows in FP32: out = act(gate) * up; mode 0 and 1: SiLU, 2 and 3: tanh-GELU
-FF_EXPORT int ff_silu_mul_f32(const float* gu, float* out, int rows, int f, int ldgu, int ldo, int mode, int interleaved, cudaStream_t s) {
-  if (mode < 0 || mode > 3) return FF_HOST_UNSUPPORTED;
+// gate/up rows in FP32: out = act(gate) * up; mode 0 and 1: SiLU, 2 and 3: tanh-GELU, 5: clamped gate
+FF_EXPORT int ff_silu_mul_f32(const float* gu, float* out, int rows, int f, int ldgu, int ldo, int mode, float limit, int interleaved, cudaStream_t s) {
+  if (mode < 0 || mode == 4 || mode > 5) return FF_HOST_UNSUPPORTED;
   if (rows <= 0 || f <= 0 || f % 4 || ldgu % 4 || ldo % 4 || (interleaved && f % 64)) return FF_HOST_BAD_SHAPE;
   const long long total = (long long)rows * (f / 4);
-  if (int r = launch_pdl(silu_mul_f32_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, 0, gu, out, rows, f, ldgu, ldo, mode, interleaved)) return r;
+  if (int r = launch_pdl(silu_mul_f32_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, 0, gu, out, rows, f, ldgu, ldo, mode, limit, interleaved)) return r;
   return launch_result();
 }
 

@@ -13,7 +13,7 @@ import torch
 from . import _count, _require, linear, workspace
 from .lib import check, kernels, ptr, status_tensor, stream_ptr
 
-SCORE_MODES = {"softmax": 0, "sigmoid": 1, "noaux": 2, "sqrt_softplus": 3}
+SCORE_MODES = {"softmax": 0, "sigmoid": 1, "noaux": 2, "sqrt_softplus": 3, "biased_softmax": 4}
 
 
 def route(x, w_router, top_k, score, bias, n_groups, topk_groups, routed_scaling, renormalize, exact=False, experts=None):
@@ -84,16 +84,17 @@ TILED_MIN_ROWS = int(os.environ.get("FF_MOE_TILED_MIN", "96"))
 
 
 def grouped_gemm(xs, w, seg_off, counts, capacity: int, epi: int, rows_per_expert: float = 0.0,
-                 out: torch.Tensor | None = None) -> torch.Tensor:
+                 out: torch.Tensor | None = None, limit: float = 0.0) -> torch.Tensor:
     """``rows_per_expert`` is the caller's estimate of the mean segment length (assignments / local experts; the
     true counts stay on the device): from ``TILED_MIN_ROWS`` on, the 128-row-tile kernel (tokens on the UMMA M
-    side, double-buffered accumulators) runs instead of the swap-AB kernel that streams each weight slice once."""
+    side, double-buffered accumulators) runs instead of the swap-AB kernel that streams each weight slice once. ``epi`` 1: SwiGLU, or the
+    clamped gate with ``limit > 0``."""
     el, nw, k = w.shape
     n_out = nw // 2 if epi == 1 else nw
     y = out if out is not None else torch.empty(capacity, n_out, dtype=torch.bfloat16, device=xs.device)
     tiled = rows_per_expert >= TILED_MIN_ROWS and (epi == 0 or nw % 256 == 0)
     fn = kernels().ff_moe_grouped_gemm_tiled if tiled else kernels().ff_moe_grouped_gemm
-    rc = fn(ptr(xs), ptr(w), ptr(y), ptr(seg_off), ptr(counts), el, nw, k, capacity, n_out, epi,
+    rc = fn(ptr(xs), ptr(w), ptr(y), ptr(seg_off), ptr(counts), el, nw, k, capacity, n_out, epi, c_float(limit),
             ptr(status_tensor(xs.device)), stream_ptr())
     check(rc, "ff_moe_grouped_gemm")
     _count()
@@ -112,16 +113,16 @@ def _grouped_gemm_f32(xs, w, seg_off, counts, capacity: int) -> torch.Tensor:
 PLAN_MAX_ROWS, PLAN_MAX_OUTPUTS = 64, 256
 
 
-def expert_rows(x, weights, ids, gu, down):
+def expert_rows(x, weights, ids, gu, down, limit=0.0):
     """See :func:`moe_ops.expert_rows`."""
-    return _served(x, weights, ids, gu, down, dispatch_local(x, ids, 1 << 30, 0, gu.shape[0]))
+    return _served(x, weights, ids, gu, down, dispatch_local(x, ids, 1 << 30, 0, gu.shape[0]), limit)
 
 
-def routed_rows(x, w_router, top_k, score, bias, outputs: int, gu, down):
+def routed_rows(x, w_router, top_k, score, bias, outputs: int, gu, down, limit=0.0):
     """See :func:`moe_ops.routed_rows`; batches of up to ``PLAN_MAX_ROWS`` rows are routed and dispatched by one block."""
     rows, el = x.shape[0], gu.shape[0]
     if rows > PLAN_MAX_ROWS or outputs > PLAN_MAX_OUTPUTS:
-        return expert_rows(x, *route(x, w_router, top_k, score, bias, 1, 1, 1.0, True, True, outputs), gu, down)
+        return expert_rows(x, *route(x, w_router, top_k, score, bias, 1, 1, 1.0, True, True, outputs), gu, down, limit)
     logits = linear(x, w_router, out_dtype=torch.float32)
     dev, cap = x.device, ((rows * top_k + 16 * el + 15) // 16) * 16
     weights = torch.empty(rows, top_k, dtype=torch.float32, device=dev)
@@ -134,10 +135,10 @@ def routed_rows(x, w_router, top_k, score, bias, outputs: int, gu, down):
                                ptr(status_tensor(dev)), stream_ptr())
     check(rc, "ff_moe_plan")
     _count(2)
-    return _served(x, weights, ids.view(rows, top_k), gu, down, (xs, pos, seg_off, counts, cap))
+    return _served(x, weights, ids.view(rows, top_k), gu, down, (xs, pos, seg_off, counts, cap), limit)
 
 
-def _served(x, weights, ids, gu, down, plan):
+def _served(x, weights, ids, gu, down, plan, limit=0.0):
     """The experts' two products over dispatched rows."""
     from . import silu_mul
     from .moe_ops import ExpertRows
@@ -145,10 +146,11 @@ def _served(x, weights, ids, gu, down, plan):
     _require(gu.shape[1] == 2 * down.shape[2] and gu.shape[1] % 128 == 0 and gu.is_contiguous() and down.is_contiguous(), "expert stacks")
     xs, pos, seg_off, counts, cap = plan
     if x.dtype == torch.float32:
-        y = _grouped_gemm_f32(silu_mul(_grouped_gemm_f32(xs, gu, seg_off, counts, cap), interleaved=True), down, seg_off, counts, cap)
+        h = silu_mul(_grouped_gemm_f32(xs, gu, seg_off, counts, cap), mode=5 if limit else 0, limit=limit, interleaved=True)
+        y = _grouped_gemm_f32(h, down, seg_off, counts, cap)
     else:
         rpe = x.shape[0] * ids.shape[1] / el
-        h = grouped_gemm(xs, gu, seg_off, counts, cap, epi=1, rows_per_expert=rpe)
+        h = grouped_gemm(xs, gu, seg_off, counts, cap, epi=1, rows_per_expert=rpe, limit=limit)
         y = grouped_gemm(h, down, seg_off, counts, cap, epi=0, rows_per_expert=rpe)
     return ExpertRows(y, pos, ids, weights, x, el)
 

@@ -48,19 +48,20 @@ class ExpertRows:
         return out
 
 
-def expert_rows(x: torch.Tensor, weights: torch.Tensor, ids: torch.Tensor, gu: torch.Tensor, down: torch.Tensor) -> ExpertRows:
+def expert_rows(x: torch.Tensor, weights: torch.Tensor, ids: torch.Tensor, gu: torch.Tensor, down: torch.Tensor, limit: float = 0.0) -> ExpertRows:
     """SwiGLU experts on the rows that chose them, without the final sum. ``gu`` [E, 2f, h] with gate / up rows interleaved per
-    64, ``down`` [E, h, f]; ids from ``E`` on are not served here (identity outputs). BF16 or FP32."""
+    64, ``down`` [E, h, f]; ids from ``E`` on are not served here (identity outputs). ``limit > 0``: the clamped gate (``ref.silu_mul`` mode 5) in place of SiLU.
+    BF16 or FP32."""
     if x.is_cuda:
         from . import moe_cuda
-        return moe_cuda.expert_rows(x, weights, ids, gu, down)
+        return moe_cuda.expert_rows(x, weights, ids, gu, down, limit)
     e = gu.shape[0]
     y = torch.zeros(ids.numel(), x.shape[1], dtype=x.dtype)
     pos = torch.where(ids < e, torch.arange(ids.numel()).view(ids.shape), -1).reshape(-1)
     for k in range(e):
         r, c = torch.nonzero(ids == k, as_tuple=True)
         if r.numel():
-            y[r * ids.shape[1] + c] = ref.linear(ref.linear_swiglu(x[r], gu[k]), down[k])
+            y[r * ids.shape[1] + c] = ref.linear(ref.linear_swiglu(x[r], gu[k], 5 if limit else 0, limit), down[k])
     return ExpertRows(y, pos, ids, weights, x, e)
 
 
@@ -82,11 +83,11 @@ def add_shared(routed: torch.Tensor, shared: torch.Tensor) -> torch.Tensor:
 
 
 def routed_rows(x: torch.Tensor, w_router: torch.Tensor, top_k: int, score: str, bias: torch.Tensor | None, outputs: int, gu: torch.Tensor,
-                down: torch.Tensor) -> ExpertRows:
+                down: torch.Tensor, limit: float = 0.0) -> ExpertRows:
     """:func:`route` with FP32 logits over the first ``outputs`` rows of ``w_router`` and renormalised weights, then
     :func:`expert_rows`."""
     if x.is_cuda:
         from . import moe_cuda
-        return moe_cuda.routed_rows(x, w_router, top_k, score, bias, outputs, gu, down)
+        return moe_cuda.routed_rows(x, w_router, top_k, score, bias, outputs, gu, down, limit)
     weights, ids = route(x, w_router, top_k, score, bias, exact=True, experts=outputs)
-    return expert_rows(x, weights, ids, gu, down)
+    return expert_rows(x, weights, ids, gu, down, limit)

@@ -44,7 +44,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = Non
     return y.to(out_dtype or x.dtype)
 
 
-def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, mode: int = 0) -> torch.Tensor:
+def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, mode: int = 0, limit: float = 0.0) -> torch.Tensor:
     """Fused gate/up projection + SwiGLU for a weight whose rows are interleaved per 64:
     rows [128*t, 128*t+64) are gate rows for outputs [64*t, 64*t+64), the next 64 the
     matching up rows (one 128-row weight tile of the decode GEMM holds both)."""
@@ -53,9 +53,9 @@ def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, mode: int = 0) -
     y = y.view(*y.shape[:-1], n // 128, 2, 64)
     gate, up = y[..., 0, :], y[..., 1, :]
     gu = torch.cat([gate.reshape(*y.shape[:-3], -1), up.reshape(*y.shape[:-3], -1)], dim=-1)
-    if mode == 3:                                   # rounded once
-        return silu_mul(gu, mode=mode).to(x.dtype)
-    return silu_mul(gu.to(x.dtype), mode=mode)
+    if mode in (3, 5):                              # rounded once
+        return silu_mul(gu, mode=mode, limit=limit).to(x.dtype)
+    return silu_mul(gu.to(x.dtype), mode=mode, limit=limit)
 
 
 def interleave_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor:
@@ -152,7 +152,8 @@ def rope_kv_paged(qkv: torch.Tensor, positions: torch.Tensor, slots: torch.Tenso
 # ------------------------------------------------------------------------------------------
 def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0) -> torch.Tensor:
     """gu: [..., 2f] = gate | up. Modes: 0 = silu rounded then product rounded, 1 = single rounding,
-    2 = tanh-GELU twice rounded, 3 = tanh-GELU with a single rounding, 4 = clamped SwiGLU in FP32 (gate <= limit, |up| <= limit)."""
+    2 = tanh-GELU twice rounded, 3 = tanh-GELU with a single rounding, 4 = clamped SwiGLU in FP32 (gate <= limit, |up| <= limit),
+    5 = clamped as 4, ``g sigmoid(1.702 g) (u + 1)``."""
     f = gu.shape[-1] // 2
     dt = gu.dtype
     g, u = gu[..., :f].to(F32), gu[..., f:].to(F32)
@@ -169,6 +170,9 @@ def silu_mul(gu: torch.Tensor, mode: int = 0, limit: float = 0.0) -> torch.Tenso
         g = torch.clamp(g, max=limit)
         u = torch.clamp(u, min=-limit, max=limit)
         y = g * torch.sigmoid(g) * u
+    elif mode == 5:
+        g = torch.clamp(g, max=limit)
+        y = g * torch.sigmoid(1.702 * g) * (torch.clamp(u, min=-limit, max=limit) + 1.0)
     else:
         raise ValueError(f"unknown SwiGLU mode {mode}")
     return y.to(dt)
@@ -259,15 +263,17 @@ def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, v
                  dim: int, vdim: int, eps: float, first_v: torch.Tensor | None = None, mix: float = 0.0,
                  q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None,
                  cos_sin: torch.Tensor | None = None, whole: bool = False, halves: bool = False,
-                 temp: tuple[torch.Tensor, float, int] | None = None) -> None:
+                 temp: tuple[torch.Tensor, float, int] | None = None, norm_qk: bool = True, norm_v: bool = False) -> None:
     """In place on the q heads of ``qkv``: q and k divided by their root mean square over ``dim`` (heads may be padded in
     the row: the caches' widths are the row's head widths), or over all heads (``whole``), weighted and rotated where that is
-    given, v blended with ``first_v``; k and v go to ``slots``."""
+    given, v blended with ``first_v`` or normed; k and v go to ``slots``."""
     rows = qkv.shape[0]
     dk = kcache.shape[3] if hkv else qkv.shape[1] // hq
     nq, nk = hq * dk, hkv * dk
     qk = qkv[:, : nq + nk].to(F32).view(rows, hq + hkv, dk)
-    if whole:
+    if not norm_qk:
+        pass
+    elif whole:
         ss = qk.square().sum(-1)
         mean = torch.cat([ss[:, :hq].sum(-1, keepdim=True).expand(rows, hq) / hq, ss[:, hq:].sum(-1, keepdim=True).expand(rows, hkv) / max(hkv, 1)], 1)
         qk = qk * torch.rsqrt(mean[..., None] / dim + eps)
@@ -288,13 +294,17 @@ def head_norm_kv(qkv: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, v
         positions, coef, every = temp
         f = 1.0 + coef * torch.log(torch.div(positions + 1, every, rounding_mode="floor").to(F32) + 1.0)
         qk[:, :hq] *= f[:, None, None]
-    qkv[:, : nq] = qk[:, :hq].reshape(rows, nq).to(qkv.dtype)
+    if norm_qk:
+        qkv[:, : nq] = qk[:, :hq].reshape(rows, nq).to(qkv.dtype)
     if not hkv:
         return
     bs, dv = kcache.shape[2], vcache.shape[3]
     v = qkv[:, nq + nk: nq + nk + hkv * dv].to(F32)
     if first_v is not None:
         v = (1.0 - mix) * v + mix * first_v.to(F32)
+    if norm_v:
+        v = v.view(rows, hkv, dv)
+        v = (v * torch.rsqrt((v * v).sum(-1, keepdim=True) / vdim + eps)).reshape(rows, hkv * dv)
     for r in range(rows):
         s = int(slots[r])
         if s >= 0:
@@ -405,6 +415,7 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top_k: int, score: str = 
 
     * logits = x @ w_router.T accumulated in FP32, rounded to the activation dtype;
     * ``softmax``: softmax over all experts, top-k (on ``score + bias`` where a bias is given), renormalise;
+    * ``biased_softmax``: as ``softmax`` over ``logit + bias`` (the bias is part of the weights too);
     * ``sigmoid``: sigmoid scores, top-k, renormalise;
     * ``noaux``: selection on ``sigmoid(logit) + bias`` restricted to the ``topk_groups`` best of
       ``n_groups`` groups (group score = sum of its two best biased scores), weights are the
@@ -413,6 +424,8 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top_k: int, score: str = 
     Returns (weights FP32 [rows, k], ids int32 [rows, k]) with ids in selection order."""
     dt = logits_dtype or x.dtype
     logits = _r((x.to(torch.float64) @ w_router.to(torch.float64).t()).to(F32), dt)
+    if score == "biased_softmax":
+        score, logits, bias = "softmax", logits + bias.to(F32), None
     if score == "softmax":
         s = torch.softmax(logits, dim=-1)
         _, ids = topk_lower_tie(s if bias is None else s + bias.to(F32), top_k)

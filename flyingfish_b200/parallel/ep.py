@@ -223,7 +223,7 @@ class EPComm:
         fn = lib.ff_moe_grouped_gemm_tiled if self._rows_per_expert >= moe_cuda.TILED_MIN_ROWS else lib.ff_moe_grouped_gemm
         rc = fn(oplib.ptr(h), oplib.ptr(lw.experts_down), oplib.ptr(self.out_y),
                                      oplib.ptr(self._seg_off), oplib.ptr(self._counts), self.El, self.hidden, h.shape[1],
-                                     self.capacity, self.hidden, 0, oplib.ptr(oplib.status_tensor(h.device)),
+                                     self.capacity, self.hidden, 0, ctypes.c_float(0.0), oplib.ptr(oplib.status_tensor(h.device)),
                                      oplib.stream_ptr())
         oplib.check(rc, "ff_moe_grouped_gemm(down)")
         ops._count(1)
