@@ -259,7 +259,7 @@ class BazulornModel(DecoderModel):
         s, rows = self._split(b)
         args = (l.heads, l.kv_heads, l.scale, l.window, lw.extra["talk"], l.sink_one)
         if s:
-            talk_ops.talk_prefill(p[:rows], kv.k[i], kv.v[i], b.block_table[:s], b.q_start[:s], b.q_lens[:s], b.ctx_lens[:s], b.max_q_len, *args,
+            talk_ops.talk_prefill(p[:rows], kv.k[i], kv.v[i], b.block_table[:s], b.q_start[:s], b.q_lens[:s], b.ctx_lens[:s], b.max_q_len, b.max_ctx, *args,
                                   out=out[:rows])
         if s < b.batch:
             talk_ops.talk_decode(p[rows:], kv.k[i], kv.v[i], b.block_table[s:], b.ctx_lens[s:], b.max_ctx, *args, out=out[rows:])

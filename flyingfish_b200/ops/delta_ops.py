@@ -11,10 +11,14 @@ from dataclasses import dataclass
 
 import torch
 
-from . import _count, _require
+from . import _count, _require, workspace
 from .lib import check, kernels, ptr, stream_ptr
 
 CONV_MAX_TAPS = 8
+CHUNK = 64                   # tokens of a chunk
+CHUNK_MIN_ROWS = 12          # shortest longest portion of a launch for which the chunked form is used
+CHUNK_MAX_KEY = 128
+SCRATCH_BYTES = 512 << 20    # the chunked form takes the chunks of a batch in rounds whose scratch stays below this
 
 
 @dataclass
@@ -133,8 +137,17 @@ def delta_rule(x: torch.Tensor, unit: torch.Tensor, decay: torch.Tensor, beta: t
     _require(row_start.dtype == slots.dtype == torch.int32 and row_start.numel() == n + 1 and out.is_contiguous(), "delta_rule: metadata")
     args = (ptr(x), ptr(unit), ptr(decay), ptr(beta), ptr(rate), ptr(dt_bias), ptr(st.S), ptr(out), ptr(row_start), ptr(slots), n, x.stride(0),
             decay.stride(0), beta.stride(0), st.heads, st.kv_heads, st.dk, st.dv)
-    check(kernels().ff_delta_recurrent(*args, int(x.dtype == torch.float32), stream_ptr()), "ff_delta_recurrent")
-    _count()
+    if x.dtype == torch.float32 or max_rows < CHUNK_MIN_ROWS or st.dk > CHUNK_MAX_KEY:
+        check(kernels().ff_delta_recurrent(*args, int(x.dtype == torch.float32), stream_ptr()), "ff_delta_recurrent")
+        _count()
+        return
+    chunks = (max_rows + CHUNK - 1) // CHUNK
+    record = kernels().ff_delta_chunk_record(st.dk, st.dv) * n * st.heads
+    rounds = -(-chunks // max(1, SCRATCH_BYTES // record))
+    per_round = -(-chunks // rounds)
+    scratch = workspace(x.device).ensure("delta_chunks", record * per_round // 4)
+    check(kernels().ff_delta_chunked(*args, chunks, per_round, ptr(scratch), stream_ptr()), "ff_delta_chunked")
+    _count(2 * -(-chunks // per_round))
 
 
 def head_out(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, vdim: int, eps: float) -> torch.Tensor:

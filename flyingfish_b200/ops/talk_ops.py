@@ -1,5 +1,6 @@
 """Windowed attention whose heads' weights are mixed by a matrix before they meet the values (talking heads behind the soft-max). CUDA:
-``csrc/talk_simt.cu`` (any head width, BF16 or FP32); CPU: FP32 arithmetic.
+``csrc/talk_tc.cu`` (tensor cores: BF16, heads of up to 128 elements) and ``csrc/talk_simt.cu`` (any head width, BF16 or FP32); CPU: FP32
+arithmetic.
 
 The heads do not separate: a row's weights of every head, normalised, go into every head's sum. ``one`` adds a fixed 1 to the soft-max's
 denominator."""
@@ -9,8 +10,15 @@ from ctypes import c_float
 
 import torch
 
-from . import _count, _require, _rows2d
+from . import BF16, _count, _require, _rows2d, attn_prefill, workspace
 from .lib import check, kernels, ptr, status_tensor, stream_ptr
+
+PAGE = 64
+SMEM = 227 * 1024
+ROUND_BYTES = 80 << 20        # prompts: scratch of a round, to stay in the L2 cache
+FILL_CTAS = 148
+DECODE_CTAS = 592             # decode: CTAs a launch should have
+DECODE_SPLITS = 32
 
 
 def _cpu(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, vdim, scale, window, talk, one) -> torch.Tensor:
@@ -26,7 +34,8 @@ def _cpu(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim
         see = (key <= pos) & (pos - key < window)
         s = torch.einsum("nhd,hkd->hnk", q[r0: r0 + n, : hq * dim].float().view(n, hq, dim), rows(kcache, dim)) * scale
         s = s.masked_fill(~see, float("-inf"))
-        m = s.amax(-1, keepdim=True).clamp(min=0.0 if one else None)
+        m = s.amax(-1, keepdim=True)
+        m = m.clamp(min=0.0) if one else m
         e = torch.exp(s - m)
         w = e / (e.sum(-1, keepdim=True) + (torch.exp(-m) if one else 0.0))
         w = torch.einsum("hg,gnk->hnk", talk, w)
@@ -34,38 +43,86 @@ def _cpu(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim
     return out.to(q.dtype)
 
 
-def talk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_table: torch.Tensor, q_start: torch.Tensor,
-                   q_lens: torch.Tensor, ctx_lens: torch.Tensor, max_q_len: int, hq: int, hkv: int, scale: float, window: int,
-                   talk: torch.Tensor, one: bool, out: torch.Tensor) -> torch.Tensor:
-    """``q`` [rows, >= hq * dim]: rows ``q_start[s] .. + q_lens[s]`` of sequence s, the last of them seeing ``ctx_lens[s]`` keys. ``talk``
-    FP32 [hq, hq]. Writes ``out`` [rows, hq * vdim]."""
+def _simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq: int, hkv: int, scale: float, window: int, talk, one: bool, out) -> None:
+    rows, ldq = _rows2d(q)
+    rc = kernels().ff_talk_simt(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(talk), ptr(out),
+                                block_table.shape[0], rows, 1, hq, hkv, kcache.shape[3], vcache.shape[3], ldq, out.stride(0), kcache.shape[2],
+                                block_table.stride(0), kcache.shape[0], window, c_float(scale), c_float(float(one)), int(q.dtype == torch.float32),
+                                ptr(status_tensor(q.device)), stream_ptr())
+    check(rc, "ff_talk_simt")
+    _count()
+
+
+def _check(q, kcache, vcache, hq: int, talk, out, *metadata) -> bool:
+    """Whether the tensor-core kernels take these operands."""
+    rows, ldq = _rows2d(q)
+    dim, vdim = kcache.shape[3], vcache.shape[3]
+    _require(q.dtype == kcache.dtype == vcache.dtype == out.dtype and kcache.is_contiguous() and vcache.is_contiguous(), "talk attention: one type throughout")
+    _require(talk.dtype == torch.float32 and talk.shape == (hq, hq) and talk.is_contiguous() and out.stride(1) == 1 and out.shape == (rows, hq * vdim),
+             "talk attention: mixing matrix, output")
+    _require(all(t.dtype == torch.int32 for t in metadata), "talk attention: int32 metadata")
+    return q.dtype == BF16 and max(dim, vdim) <= 128 and dim % 16 == vdim % 16 == 0 and kcache.shape[2] == PAGE and ldq % 8 == out.stride(0) % 8 == 0
+
+
+def _band(max_ctx: int, window: int, rows: int) -> int:
+    """Pages that ``rows`` consecutive positions see at most."""
+    return min(-(-max_ctx // PAGE), (window + rows + 61) // PAGE + 1)
+
+
+def talk_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_table: torch.Tensor, q_start: torch.Tensor,
+                 q_lens: torch.Tensor, ctx_lens: torch.Tensor, max_q_len: int, max_ctx: int, hq: int, hkv: int, scale: float, window: int,
+                 talk: torch.Tensor, one: bool, out: torch.Tensor) -> torch.Tensor:
+    """Portions of prompts. ``q`` [rows, >= hq * dim]: rows ``q_start[s] .. + q_lens[s]`` of sequence s, the last of them seeing
+    ``ctx_lens[s]`` (at most ``max_ctx``) keys through ``window``. ``talk`` FP32 [hq, hq]. Writes ``out`` [rows, hq * vdim]."""
     dim, vdim = kcache.shape[3], vcache.shape[3]
     if not q.is_cuda:
         out.copy_(_cpu(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, vdim, scale, window, talk, one))
         return out
-    rows, ldq = _rows2d(q)
-    _require(q.dtype == kcache.dtype == vcache.dtype == out.dtype and kcache.is_contiguous() and vcache.is_contiguous(), "talk_attention: one type throughout")
-    _require(talk.dtype == torch.float32 and talk.shape == (hq, hq) and talk.is_contiguous() and out.stride(1) == 1 and out.shape == (rows, hq * vdim),
-             "talk_attention: mixing matrix, output")
-    _require(block_table.dtype == q_start.dtype == q_lens.dtype == ctx_lens.dtype == torch.int32, "talk_attention: int32 metadata")
-    rc = kernels().ff_talk_simt(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(talk), ptr(out),
-                                block_table.shape[0], rows, 1, hq, hkv, dim, vdim, ldq, out.stride(0), kcache.shape[2], block_table.stride(0),
-                                kcache.shape[0], window, c_float(scale), c_float(float(one)), int(q.dtype == torch.float32),
-                                ptr(status_tensor(q.device)), stream_ptr())
-    check(rc, "ff_talk_simt")
-    _count()
+    tensor = _check(q, kcache, vcache, hq, talk, out, block_table, q_start, q_lens, ctx_lens)
+    kp = 64 if dim <= 64 else 128
+    need = hq * 32 * kp + hkv * 64 * kp + -(-hq // 16) * 16384 + hq * 64 + 128
+    if not tensor or hq > 32 or need > SMEM:
+        _simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, scale, window, talk, one, out)
+        return out
+    rows, batch = q.shape[0], block_table.shape[0]
+    z = torch.empty(rows, hq, dtype=torch.float32, device=q.device)
+    sinks = torch.zeros(hq, dtype=torch.float32, device=q.device) if one else None
+    attn_prefill(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, max_q_len, hq, hkv, dim, scale, window=window, out=out, sinks=sinks,
+                 vdim=vdim, lse=z)                       # its result is overwritten
+    band = _band(max_ctx, window, 64)
+    tiles, tile_bytes = -(-max_q_len // 64), batch * hq * 64 * band * PAGE * 2
+    rounds = -(-tiles // max(1, ROUND_BYTES // tile_bytes))
+    per_round = -(-tiles // rounds)
+    parts = max(1, min(-(-FILL_CTAS // (4 * per_round * batch)), band))
+    scratch = workspace(q.device).ensure("talk_weights", tile_bytes * per_round // 4)
+    rc = kernels().ff_talk_prefill(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(talk), ptr(z),
+                                   ptr(out), ptr(scratch), batch, max_q_len, hq, hkv, dim, vdim, q.stride(0), out.stride(0), block_table.stride(0),
+                                   kcache.shape[0], window, band, per_round, parts, c_float(scale), ptr(status_tensor(q.device)), stream_ptr())
+    check(rc, "ff_talk_prefill")
+    _count(2 * -(-tiles // per_round))
     return out
 
 
-def talk_prefill(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, max_q_len: int, hq: int, hkv: int, scale: float, window: int, talk,
-                 one: bool, out: torch.Tensor) -> torch.Tensor:
-    """Portions of prompts: see :func:`talk_attention`."""
-    return talk_attention(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, max_q_len, hq, hkv, scale, window, talk, one, out)
-
-
-def talk_decode(q, kcache, vcache, block_table, ctx_lens, max_ctx: int, hq: int, hkv: int, scale: float, window: int, talk, one: bool,
-                out: torch.Tensor) -> torch.Tensor:
-    """One row per sequence: see :func:`talk_attention`."""
-    n = block_table.shape[0]
-    start = torch.arange(n, dtype=torch.int32, device=q.device)
-    return talk_attention(q, kcache, vcache, block_table, start, torch.ones_like(start), ctx_lens, 1, hq, hkv, scale, window, talk, one, out)
+def talk_decode(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_table: torch.Tensor, ctx_lens: torch.Tensor, max_ctx: int, hq: int,
+                hkv: int, scale: float, window: int, talk: torch.Tensor, one: bool, out: torch.Tensor) -> torch.Tensor:
+    """One row per sequence: as :func:`talk_prefill`."""
+    dim, vdim, batch = kcache.shape[3], vcache.shape[3], block_table.shape[0]
+    if not q.is_cuda or not _check(q, kcache, vcache, hq, talk, out, block_table, ctx_lens) or hq > 64 or hq // hkv > 16:
+        start = torch.arange(batch, dtype=torch.int32, device=q.device)
+        args = (q, kcache, vcache, block_table, start, torch.ones_like(start), ctx_lens, hq, hkv)
+        if q.is_cuda:
+            _simt(*args, scale, window, talk, one, out)
+        else:
+            out.copy_(_cpu(*args, dim, vdim, scale, window, talk, one))
+        return out
+    band = _band(max_ctx, window, 1)
+    splits = max(1, min(-(-DECODE_CTAS // (hkv * batch)), band, DECODE_SPLITS))
+    ws = workspace(q.device)
+    scores, ml = ws.ensure("talk_scores", batch * hq * band * PAGE), ws.ensure("talk_ml", batch * splits * hq * 2)
+    part = ws.ensure("attn_o", batch * splits * hq * vdim) if splits > 1 else None
+    rc = kernels().ff_talk_decode(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(ctx_lens), ptr(talk), ptr(out), ptr(scores), ptr(ml), ptr(part),
+                                  batch, hq, hkv, dim, vdim, q.stride(0), out.stride(0), block_table.stride(0), kcache.shape[0], window, band, splits,
+                                  c_float(scale), c_float(float(one)), ptr(status_tensor(q.device)), stream_ptr())
+    check(rc, "ff_talk_decode")
+    _count(2 if splits == 1 else 3)
+    return out
