@@ -812,12 +812,11 @@ def attn_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
                  hkv: int, dim: int, scale: float, window: int = 0, out: torch.Tensor | None = None,
                  sinks: torch.Tensor | None = None, chunk: int = 0, vdim: int | None = None,
                  gate: torch.Tensor | None = None, keep: int = 0, softcap: float = 0.0,
-                 head_gate: torch.Tensor | None = None, lse: torch.Tensor | None = None) -> torch.Tensor:
+                 head_gate: torch.Tensor | None = None) -> torch.Tensor:
     """Causal chunked-prefill attention of packed query rows against the paged cache. ``window < 0`` makes it
     bidirectional: every query row sees all ``ctx_lens`` keys of its sequence (encoders, vision towers). ``sinks``
     (float32 [hq]): learnable soft-max, one sink logit per head in the denominator (tcgen05 kernel only). ``chunk``,
-    ``vdim``, ``gate``, ``keep``, ``softcap`` and ``head_gate`` as in :func:`attn_decode`. ``lse`` (float32 [rows, hq], tcgen05 kernel only) takes
-    the base-2 logarithm of every soft-max's denominator."""
+    ``vdim``, ``gate``, ``keep``, ``softcap`` and ``head_gate`` as in :func:`attn_decode`."""
     vdim = vdim or dim
     keep = keep if window > 0 else 0
     _require(not (softcap and sinks is not None), "attn_prefill: capped scores come without sinks")
@@ -835,7 +834,6 @@ def attn_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
     if out is None:
         out = torch.empty(rows, hq * vdim, dtype=q.dtype, device=q.device)
     nb = kcache.shape[0]
-    _require(lse is None or (q.dtype == BF16 and max(dim, vdim) <= 128), "attn_prefill: denominators come from the tcgen05 kernel")
     if q.dtype == torch.float32 or max(dim, vdim) > 128:
         return _attn_simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, 1, hq, hkv, dim, vdim, scale, window, chunk, gate, out,
                           sinks, keep, softcap, head_gate)
@@ -847,15 +845,13 @@ def attn_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
     if sinks is not None:
         _require(sinks.dtype == torch.float32 and sinks.numel() == hq and sinks.is_contiguous(), "attn_prefill: sinks float32 [hq]")
         _require(out.stride(0) % 8 == 0 and ldq % 8 == 0, "attn_prefill: sinks need the tcgen05 kernel (16-byte aligned rows)")
-    _require(lse is None or (lse.dtype == torch.float32 and lse.shape == (rows, hq) and lse.is_contiguous() and out.stride(0) % 8 == 0 and ldq % 8 == 0),
-             "attn_prefill: denominators float32 [rows, hq]")
-    if (ATTN_PREFILL_TC or sinks is not None or general or lse is not None) and out.stride(0) % 8 == 0 and ldq % 8 == 0:
+    if (ATTN_PREFILL_TC or sinks is not None or general) and out.stride(0) % 8 == 0 and ldq % 8 == 0:
         # tcgen05 kernel: Q Kᵀ and P V on the tensor cores with S and O in tensor memory
         rc = kernels().ff_attn_prefill_tc(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens),
                                           ptr(ctx_lens), ptr(out), batch, rows, max_q_len, hq, hkv, dim, vdim, ldq, out.stride(0),
                                           block_table.shape[1], nb, c_float(scale), window, chunk, ptr(sinks), ptr(gate),
                                           _gate_ld(gate, rows, hq * vdim), vcache.stride(2), keep, c_float(softcap), ptr(head_gate),
-                                          _head_gate_ld(head_gate, rows, hq), ptr(lse), ptr(status_tensor(q.device)), stream_ptr())
+                                          _head_gate_ld(head_gate, rows, hq), ptr(status_tensor(q.device)), stream_ptr())
         check(rc, "ff_attn_prefill_tc")
         _count()
         return out

@@ -56,7 +56,7 @@ ARCH_SOURCES = {
                 "kv_util", "mlstm", "moe", "residual", "rope_act_sample"),
     "kabavik": ("attention_paged", "attention_simt", "attention_tc", "gemm_bf16", "gemm_f32", "gemm_skinny", "head_norm",
                 "kv_util", "mla", "residual", "rope_act_sample"),
-    "bazulorn": ("attention_tc", "delta", "delta_chunk", "gemm_bf16", "gemm_f32", "gemm_skinny", "head_norm", "kv_util", "mlstm", "moe", "residual",
+    "bazulorn": ("delta", "delta_chunk", "gemm_bf16", "gemm_f32", "gemm_skinny", "head_norm", "kv_util", "mlstm", "moe", "residual",
                  "rope_act_sample", "short_conv", "talk_simt", "talk_tc"),
 }
 

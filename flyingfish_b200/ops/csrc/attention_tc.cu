@@ -378,7 +378,6 @@ struct PrefillForm {
   // head h at column h * qr_pitch + qr_col, and tmR, the cache's rows, at column kr_col.
   const int* exp_off;
   int dr, qr_pitch, qr_col, kr_col;
-  float* lse = nullptr;            // [rows, hq]: base-2 logarithm of the soft-max's denominator
 };
 
 // Capped scores. N raw products of a thread become tanh(y), y = s cap_in; the cap is the factor of the exponent. Where all |y| of the
@@ -731,7 +730,6 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     if (ok) {
       tc_fence_after();
       if (sinks != nullptr) l_sum += (m_ref == -INFINITY) ? 1.f : exp2f(sinks[h] * 1.4426950408889634f - m_ref);
-      if (f.lse != nullptr && live && hf == 0) f.lse[(size_t)(qs + r0 + row) * hq + h] = (m_ref == -INFINITY ? 0.f : m_ref) + log2f(l_sum);
       float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
       if (EXTRA && f.head_gate != nullptr && live)
         inv = __fdividef(inv, 1.0f + __expf(-__bfloat162float(f.head_gate[(size_t)(qs + r0 + row) * f.ldhg + h])));
@@ -764,13 +762,12 @@ using namespace ff;
 // of its own block of `chunk` positions that are not after it. dk / dv: widths of the key and value heads (multiples of 16,
 // at most 128); ldv: pitch of the value cache's rows (dv, or the key rows' width where the values are their first columns). gate:
 // optional [rows, hq * dv] with row pitch ldg, 16-byte aligned. keep: with a window, the first `keep` positions stay visible.
-// softcap > 0: scores become softcap tanh(score / softcap). head_gate: optional [rows, hq] with row pitch ldhg. lse: optional FP32 [rows, hq], takes the base-2
-// logarithm of every soft-max's denominator (sinks included).
+// softcap > 0: scores become softcap tanh(score / softcap). head_gate: optional [rows, hq] with row pitch ldhg.
 FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* vcache, const int* block_table,
                                  const int* q_start, const int* q_lens, const int* ctx_lens, void* out, int batch,
                                  int total_rows, int max_q_len, int hq, int hkv, int dk, int dv, int ldq, int ldo,
                                  int max_blocks, int num_blocks, float scale, int window, int chunk, const float* sinks,
-                                 const void* gate, int ldg, int ldv, int keep, float softcap, const void* head_gate, int ldhg, float* lse, int* status,
+                                 const void* gate, int ldg, int ldv, int keep, float softcap, const void* head_gate, int ldhg, int* status,
                                  cudaStream_t s) {
   if (ldv < dv || ldv % 8 || keep < 0 || !(softcap >= 0.f) || (softcap > 0.f && sinks != nullptr)) return FF_HOST_BAD_SHAPE;
   if (batch <= 0 || max_q_len <= 0 || hq <= 0 || hkv <= 0 || hq % hkv || total_rows <= 0) return FF_HOST_BAD_SHAPE;
@@ -787,7 +784,7 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
   const float scale_log2 = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f;
   dim3 grid((max_q_len + TC_BM - 1) / TC_BM, hq, batch);
   const PrefillForm f = {window < 0 ? 0 : window, chunk, window < 0 ? 0 : 1, dk, dv, gate != nullptr ? 1 : 0, window > 0 ? keep : 0,
-                         softcap > 0.f ? scale / softcap : 0.f, (const __nv_bfloat16*)head_gate, ldhg, nullptr, 0, 0, 0, 0, lse};
+                         softcap > 0.f ? scale / softcap : 0.f, (const __nv_bfloat16*)head_gate, ldhg, nullptr, 0, 0, 0, 0};
   CUtensorMap tmG = tmQ;
   if (gate != nullptr)
     if (int r = make_tmap_2d(&tmG, gate, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)hq * dv, (uint64_t)total_rows, (uint64_t)ldg * 2, 64, TC_BM)) return r;
@@ -796,7 +793,7 @@ FF_EXPORT int ff_attn_prefill_tc(const void* q, const void* kcache, const void* 
   static int two = -1;
   if (two < 0) { const char* e = getenv("FF_ATTN_PREFILL_CTAS"); two = (e != nullptr && e[0] == '1') ? 0 : TC_TWO_CTAS_DEFAULT; }
   const bool wide = dk == TC_HD && dv == TC_HD, extra = chunk > 0 || gate != nullptr || f.keep > 0 || head_gate != nullptr, cap = softcap > 0.f;
-  if (two || extra || cap || !wide || lse != nullptr) {
+  if (two || extra || cap || !wide) {
     // FF_ATTN_PREFILL_SPLIT = 2: two softmax warps per lane quadrant (64 columns each) instead of one
     static int split = -1;
     if (split < 0) { const char* e = getenv("FF_ATTN_PREFILL_SPLIT"); split = (e != nullptr && (e[0] == '1' || e[0] == '2')) ? e[0] - '0' : TC2_SPLIT_DEFAULT; }

@@ -510,7 +510,7 @@ static int delta_chunked_launch(const DeltaArgs<__nv_bfloat16>& p, int sequences
 using namespace ff;
 
 // Bytes of scratch per (sequence, chunk of a round, head)
-FF_EXPORT long long ff_delta_chunk_record(int dk, int dv) { return (long long)(dk <= 64 ? delta_record<64>(dv) : delta_record<128>(dv)); }
+FF_EXPORT int ff_delta_chunk_record(int dk, int dv) { return (int)(dk <= 64 ? delta_record<64>(dv) : delta_record<128>(dv)); }
 
 // As ff_delta_recurrent for BF16 rows, dk <= 128 and dk, dv multiples of 8. chunks: those of the longest sequence (64 rows each), taken
 // per_round at a time; scratch: sequences * per_round * heads records, 16-byte aligned.

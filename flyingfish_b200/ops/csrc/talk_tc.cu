@@ -2,12 +2,13 @@
 // elements, paged cache with 64-token pages.
 //   w_g(i, j) = 2^(s_g(i, j) - z_g(i)),  z_g(i) the logarithm of the soft-max's denominator      M_h = sum_g talk[h, g] w_g      o_h = M_h v
 // The mixed weights of a head need the normalised weights of every head, so no head can run its soft-max and its value product in one
-// pass. Prompts take three:
-//   1. attn_prefill_tc (attention_tc.cu) leaves z of every row and head;
-//   2. talk_weights : 16 query rows and all heads per CTA, 32 keys at a time: scores again, weights in FP16 through shared memory, the
-//      product with the mixing matrix (heads as its inner dimension), mixed weights in BF16 to scratch;
-//   3. talk_values  : scratch times values, 64 query rows of up to four heads that share a value head per CTA.
-// 2 and 3 go over the prompt in rounds whose scratch stays in the L2 cache. Decoded tokens take two and a merge:
+// pass. Prompts take three, over tiles of 128 query rows:
+//   1. talk_weights : scores on tcgen05 as in attention_tc.cu, 64 keys at a time; 2^(s - m) in FP16 goes to scratch by TMA, m being the
+//                     row's maximum so far, and with it m of every step and z at the end;
+//   2. talk_mix     : a warp takes a query row, 64 keys of all heads at a time: the weights times 2^(m - z), then their product with the
+//                     mixing matrix (mma.sync, heads as its inner dimension); mixed weights in BF16 replace the others in scratch;
+//   3. talk_values  : scratch times values on tcgen05, two heads that share a value head per CTA.
+// They go over a prompt in rounds whose scratch stays in the L2 cache. Decoded tokens take two and a merge:
 //   talk_scores : scores of a key / value head's query heads over a range of pages, in FP32, and their maximum and sum;
 //   talk_decode : the weights of all heads for a page, mixed for the heads of one value head (the accumulators of that product are the
 //                 operand of the next), times the values.
@@ -30,29 +31,37 @@ __device__ __forceinline__ void mma_f16(float (&d)[4], const uint32_t (&a)[4], u
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+constexpr int TK_ROWS = 128;                 // query rows of a tile
+
 struct TalkArgs {
-  const __nv_bfloat16* q; const __nv_bfloat16* kcache; const __nv_bfloat16* vcache;
   const int* block_table; const int* q_start; const int* q_lens; const int* ctx_lens;
-  const float* talk; const float* z;         // z: [rows, H], base 2 (prompts)
-  __nv_bfloat16* out; __nv_bfloat16* scratch;
-  int H, G, dk, dv, ldq, ldo, max_blocks, num_blocks, window, band;      // band: pages a tile's rows see at most
-  int tile0, tiles;                          // this round's tiles of 64 rows
-  int parts;                                 // CTAs that share the keys of 16 rows (talk_weights)
-  float scale_log2;
+  const float* talk;
+  __nv_bfloat16* out;
+  // a slot is a tile of this round: weights [slot, H, 128, band * 64], m [slot, H, band, 128], z [slot, H, 128]
+  __nv_bfloat16* weights; float* m; float* z;
+  int H, G, dk, dv, ldo, max_blocks, num_blocks, window, band;         // band: pages a tile's rows see at most
+  int tile0, tiles, parts;                   // this round's tiles; warps that share a row's keys (talk_mix)
+  float scale_log2, one;
   int* status;
 };
 
-// pages and positions of a 64-row tile
+// rows, positions and pages of a tile
 struct TalkTile {
-  int real, first, lo_page, hi_page;         // rows, position of row 0
+  int real, first, lo_page, pages;           // first: position of row 0
   __device__ TalkTile(const TalkArgs& p, int b, int tile) {
-    const int qlen = p.q_lens[b], past = p.ctx_lens[b] - qlen, r0 = tile * 64;
-    real = min(64, qlen - r0);
+    const int qlen = p.q_lens[b], past = p.ctx_lens[b] - qlen, r0 = tile * TK_ROWS;
+    real = min(TK_ROWS, qlen - r0);
     first = past + r0;
     lo_page = max(0, first - p.window + 1) / TK_PAGE;
-    hi_page = (first + max(real, 1) - 1) / TK_PAGE;
+    pages = min(p.band, (first + max(real, 1) - 1) / TK_PAGE - lo_page + 1);
   }
 };
+__device__ __forceinline__ int talk_page(const TalkArgs& p, int b, int page, bool& bad) {
+  const int blk = p.block_table[(size_t)b * p.max_blocks + page];
+  if (blk >= 0 && blk < p.num_blocks) return blk;
+  bad = true;
+  return 0;
+}
 
 // a fragment of the mixing matrix: 16 heads from row0 (rows past `rows` of them and columns past H are zero), 16 columns from col0
 __device__ __forceinline__ void talk_frag(const float* talk, int H, int row0, int rows, int col0, int lane, uint32_t (&a)[4]) {
@@ -66,238 +75,347 @@ __device__ __forceinline__ void talk_frag(const float* talk, int H, int row0, in
 }
 
 // ---------------------------------------------------------------------------------------
-// talk_weights: grid (4 * tiles, parts, sequences), 256 threads. KP: key width padded to 64 or 128; HB: blocks of 16 heads; NB: query heads
-// of one key head that a warp takes together
+// talk_weights: grid (tiles, H, sequences), 192 threads: TMA warp, MMA warp, four warps whose threads own a row each. Shared memory: Q
+// (two blocks of 64 columns), two K tiles, two staging tiles of 32 rows per row warp. Tensor memory: two score tiles of 64 columns.
 // ---------------------------------------------------------------------------------------
-constexpr int TW_KEYS = 32;
-__device__ __forceinline__ uint32_t tw_off(int h, int chunk) {        // byte offset of 16-byte chunk 0..63 of head h's 16 x 32 weights
-  return (uint32_t)(h * 1024 + ((chunk & ~7) | ((chunk ^ ((chunk >> 3) & 3) ^ h) & 7)) * 16);
+constexpr int TW_Q = TK_ROWS * 128 * 2, TW_K = TK_PAGE * 128 * 2, TW_P = 32 * TK_PAGE * 2;
+constexpr int TW_SMEM = TW_Q + 2 * TW_K + 8 * TW_P + 1024;
+
+struct alignas(8) TalkWeightBars {
+  uint64_t q_full, k_full[2], k_empty[2], s_full[2], s_empty[2];
+  uint32_t tmem_base;
+  int abort_flag;
+};
+
+__global__ void __launch_bounds__(192, 2)
+talk_weights_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmP,
+                    const TalkArgs p) {
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.z, h = blockIdx.y, tile = p.tile0 + blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const TalkTile tl(p, b, tile);
+  if (tl.real <= 0) return;
+  extern __shared__ uint8_t tk_raw[];
+  __shared__ TalkWeightBars bars;
+  uint8_t* sQ = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tk_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* sK = sQ + TW_Q;
+  uint8_t* sP = sK + 2 * TW_K;
+  const bool hi = p.dk > 64;
+  const size_t slot_head = ((size_t)b * p.tiles + blockIdx.x) * p.H + h;
+  if (threadIdx.x == 0) {
+    tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmP);
+    mbar_init(&bars.q_full, 1);
+    for (int i = 0; i < 2; ++i) { mbar_init(&bars.k_full[i], 1); mbar_init(&bars.k_empty[i], 1); mbar_init(&bars.s_full[i], 1); mbar_init(&bars.s_empty[i], 4); }
+    bars.abort_flag = 0;
+    mbar_fence_init();
+  }
+  if (warp == 1) { tmem_alloc(&bars.tmem_base, 128); tmem_relinquish(); }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_s = bars.tmem_base;
+  volatile int* abort_flag = &bars.abort_flag;
+  if (warp == 0) {
+    if (lane == 0) {
+      const int row = p.q_start[b] + tile * TK_ROWS;
+      mbar_expect_tx(&bars.q_full, hi ? TW_Q : TW_Q / 2);
+      tma_load_2d(sQ, &tmQ, &bars.q_full, h * p.dk, row);
+      if (hi) tma_load_2d(sQ + TW_Q / 2, &tmQ, &bars.q_full, h * p.dk + 64, row);
+      bool bad = false;
+      for (int j = 0; j < tl.pages; ++j) {
+        const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
+        const int krow = (talk_page(p, b, tl.lo_page + j, bad) * p.G + h / (p.H / p.G)) * TK_PAGE;
+        if (!mbar_wait(&bars.k_empty[st], ph ^ 1, abort_flag, p.status, KID_ATTN_PREFILL, 41)) break;
+        mbar_expect_tx(&bars.k_full[st], hi ? TW_K : TW_K / 2);
+        tma_load_2d(sK + st * TW_K, &tmK, &bars.k_full[st], 0, krow);
+        if (hi) tma_load_2d(sK + st * TW_K + TW_K / 2, &tmK, &bars.k_full[st], 64, krow);
+      }
+      if (bad) set_status(p.status, KID_ATTN_PREFILL, FF_ERR_BOUNDS, b, tile);
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      const uint32_t idesc = umma_idesc(1, 1, 0, 0, TK_ROWS, TK_PAGE), q_addr = smem_u32(sQ);
+      const int ksteps = p.dk >> 4;
+      bool ok = mbar_wait(&bars.q_full, 0, abort_flag, p.status, KID_ATTN_PREFILL, 42);
+      for (int j = 0; j < tl.pages && ok; ++j) {
+        const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
+        if (!mbar_wait(&bars.k_full[st], ph, abort_flag, p.status, KID_ATTN_PREFILL, 43)) break;
+        if (!mbar_wait(&bars.s_empty[st], ph ^ 1, abort_flag, p.status, KID_ATTN_PREFILL, 44)) break;
+        tc_fence_after();
+        const uint32_t k_addr = smem_u32(sK + st * TW_K);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          if (k >= ksteps) break;
+          umma_f16(tmem_s + st * TK_PAGE, umma_desc_sw128(q_addr + (k >> 2) * (TW_Q / 2) + (k & 3) * 32, 16, 1024),
+                   umma_desc_sw128(k_addr + (k >> 2) * (TW_K / 2) + (k & 3) * 32, 16, 1024), idesc, k != 0);
+        }
+        umma_commit(&bars.s_full[st]);
+        umma_commit(&bars.k_empty[st]);
+      }
+    }
+  } else {
+    const int q = warp & 3, row = q * 32 + lane, pos = tl.first + row;
+    const bool live = row < tl.real;
+    const int last = live ? pos : -1, from = live ? max(0, pos - p.window + 1) : 0;
+    const int all_lo = max(0, tl.first + tl.real - p.window), all_hi = tl.real == TK_ROWS ? tl.first : -1;     // keys every row sees
+    uint8_t* stg = sP + q * 2 * TW_P;
+    float m = -INFINITY, l = 0.f;
+    bool ok = true;
+    for (int j = 0; j < tl.pages; ++j) {
+      const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
+      if (!mbar_wait(&bars.s_full[st], ph, abort_flag, p.status, KID_ATTN_PREFILL, 45)) ok = false;
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      tc_fence_after();
+      float sv[64];
+      {
+        uint32_t r[64];
+        const uint32_t at = tmem_s + (uint32_t(q * 32) << 16) + st * TK_PAGE;
+        tmem_ld_x32(at, r);
+        tmem_ld_x32(at + 32, r + 32);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 64; ++i) sv[i] = __uint_as_float(r[i]);
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars.s_empty[st]);
+      const int k0 = (tl.lo_page + j) * TK_PAGE;
+      float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+      if (!(k0 >= all_lo && k0 + TK_PAGE - 1 <= all_hi)) {
+#pragma unroll
+        for (int i = 0; i < 64; ++i) sv[i] = k0 + i >= from && k0 + i <= last ? sv[i] : -INFINITY;
+      }
+#pragma unroll
+      for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
+      const float mn = fmaxf(m, fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2), mr = mn == -INFINITY ? 0.f : mn;
+      l *= m == -INFINITY ? 0.f : tk_ex2(m - mr);
+      m = mn;
+      p.m[(slot_head * p.band + j) * TK_ROWS + row] = m;
+      if (lane == 0) tma_store_wait_read<1>();             // the staging tile's previous contents have left
+      __syncwarp();
+      uint8_t* at = stg + st * TW_P + lane * 128;
+      float ls[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int c = 0; c < 8; ++c) {
+        uint32_t w[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float x = tk_ex2(fmaf(sv[8 * c + 2 * i], p.scale_log2, -mr)), y = tk_ex2(fmaf(sv[8 * c + 2 * i + 1], p.scale_log2, -mr));
+          ls[i] += x + y;
+          w[i] = pack_half2(x, y);
+        }
+        *reinterpret_cast<uint4*>(at + ((c ^ (lane & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+      }
+      l += (ls[0] + ls[1]) + (ls[2] + ls[3]);
+      fence_proxy_async_smem();
+      __syncwarp();
+      if (lane == 0) {
+        tma_store_2d(&tmP, stg + st * TW_P, j * TK_PAGE, (int)(slot_head * TK_ROWS) + q * 32);
+        tma_store_commit();
+      }
+    }
+    const float n = p.one > 0.f ? fmaxf(m, 0.f) : m;
+    p.z[slot_head * TK_ROWS + row] = n == -INFINITY ? 0.f : n + log2f(l * tk_ex2(m - n) + (p.one > 0.f ? p.one * tk_ex2(-n) : 0.f));
+    if (lane == 0) tma_store_wait<0>();
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (bars.abort_flag) {
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) { __nanosleep(1000); }
+  }
+  if (warp == 1) { __syncwarp(); tc_fence_after(); tmem_dealloc(tmem_s, 128); }
 }
 
-template <int KP, int HB, int NB>
-__global__ void __launch_bounds__(256, 1)
-talk_weights_kernel(const TalkArgs p) {
+// ---------------------------------------------------------------------------------------
+// talk_mix: grid (16 * tiles, parts, sequences), 256 threads, a row per warp; HB: blocks of 16 heads
+// ---------------------------------------------------------------------------------------
+template <int HB>
+__global__ void __launch_bounds__(256)
+talk_mix_kernel(const TalkArgs p) {
   pdl_trigger();
   extern __shared__ __align__(128) uint8_t tk_raw[];
-  constexpr int KCH = KP / 8, QB = 16 * KP * 2, KB = TW_KEYS * KP * 2;
-  uint8_t* sQ = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tk_raw) + 127) & ~uintptr_t(127));
-  uint8_t* sK = sQ + p.H * QB;                             // [G][32 keys]
-  uint8_t* sP = sK + p.G * KB;                             // [16 HB][16 x 32]
-  float* sZ = reinterpret_cast<float*>(sP + HB * 16 * 1024);           // [H][16]
+  constexpr int TB = HB * 16 * 128;                        // [heads][64 keys]
   pdl_wait();
-  const int b = blockIdx.z, tile = p.tile0 + (blockIdx.x >> 2), sub = blockIdx.x & 3, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int gq = lane >> 2, tq = lane & 3, H = p.H, G = p.G, per = H / G;
-  const TalkTile tl(p, b, tile);
-  const int rows = min(16, tl.real - sub * 16);
-  if (rows <= 0) return;
-  const int row0 = p.q_start[b] + tile * 64 + sub * 16, pos0 = tl.first + sub * 16;
-  const int bandw = p.band * TK_PAGE, keys = (tl.hi_page - tl.lo_page + 1) * TK_PAGE, base = tl.lo_page * TK_PAGE;
-  __nv_bfloat16* dst = p.scratch + ((((size_t)b * p.tiles + (blockIdx.x >> 2)) * H) * 64 + sub * 16) * bandw;
-  // visible steps of 32 keys; the first part writes the zeros of the others
-  const int v0 = max(0, pos0 - p.window + 1 - base) / TW_KEYS, v1 = min(keys, pos0 + rows - base + TW_KEYS - 1) / TW_KEYS;
-  if (blockIdx.y == 0)
-    for (int step = 0; step < keys / TW_KEYS; ++step)
-      if (step < v0 || step >= v1)
-        for (int i = tid; i < H * 64; i += 256)
-          *reinterpret_cast<uint4*>(dst + ((size_t)(i >> 6) * 64 + ((i >> 2) & 15)) * bandw + step * TW_KEYS + (i & 3) * 8) = make_uint4(0, 0, 0, 0);
-  const int ka = v0 + (v1 - v0) * (int)blockIdx.y / p.parts, kb = v0 + (v1 - v0) * ((int)blockIdx.y + 1) / p.parts;
-  if (ka >= kb) return;
-  for (int i = tid; i < H * 16 * KCH; i += 256) {
-    const int h = i / (16 * KCH), r = (i / KCH) & 15, c = i % KCH;
-    uint8_t* at = sQ + h * QB + ms_off(r, c, KCH);
-    if (r < rows && c * 8 < p.dk) tk_cp16(at, p.q + (size_t)(row0 + r) * p.ldq + (size_t)h * p.dk + c * 8);
-    else *reinterpret_cast<uint4*>(at) = make_uint4(0, 0, 0, 0);
-  }
-  for (int i = tid; i < H * 16; i += 256) { const int h = i >> 4, r = i & 15; sZ[i] = r < rows ? p.z[(size_t)(row0 + r) * H + h] : 0.f; }
-  for (int i = tid; i < HB * 16 * 1024 / 16; i += 256) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);       // rows past H stay zero
-  auto fetch = [&](int step) {
-    const int k0 = base + step * TW_KEYS;
-    int blk = p.block_table[(size_t)b * p.max_blocks + k0 / TK_PAGE];
-    const bool ok = blk >= 0 && blk < p.num_blocks;
-    if (!ok) { if (tid == 0) set_status(p.status, KID_ATTN_PREFILL, FF_ERR_BOUNDS, b, k0); blk = 0; }
-    for (int i = tid; i < G * TW_KEYS * KCH; i += 256) {
-      const int g = i / (TW_KEYS * KCH), r = (i / KCH) & (TW_KEYS - 1), c = i % KCH;
-      uint8_t* at = sK + g * KB + ms_off(r, c, KCH);
-      if (c * 8 < p.dk) tk_cp16(at, p.kcache + (((size_t)blk * G + g) * TK_PAGE + k0 % TK_PAGE + r) * p.dk + c * 8);
-      else *reinterpret_cast<uint4*>(at) = make_uint4(0, 0, 0, 0);
-    }
+  const int b = blockIdx.z, slot = b * p.tiles + (blockIdx.x >> 4), warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
+  const int row = (blockIdx.x & 15) * 8 + warp, H = p.H;
+  const TalkTile tl(p, b, p.tile0 + (blockIdx.x >> 4));
+  if (row >= tl.real) return;
+  uint8_t* buf = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tk_raw) + 127) & ~uintptr_t(127)) + warp * 2 * TB;
+  const int pos = tl.first + row, j0 = max(0, pos - p.window + 1) / TK_PAGE - tl.lo_page, j1 = min(tl.pages, pos / TK_PAGE - tl.lo_page + 1);     // the others are zero
+  const int ja = j0 + (j1 - j0) * (int)blockIdx.y / p.parts, jb = j0 + (j1 - j0) * ((int)blockIdx.y + 1) / p.parts;
+  if (ja >= jb) return;
+  const size_t bandw = (size_t)p.band * TK_PAGE;
+  __nv_bfloat16* base = p.weights + ((size_t)slot * H * TK_ROWS + row) * bandw;
+  auto fetch = [&](int j) {
+    uint8_t* d = buf + (j & 1) * TB;
+    for (int i = lane; i < H * 8; i += 32) { const int h = i >> 3, c = i & 7; tk_cp16(d + ms_off(h, c, 8), base + (size_t)h * TK_ROWS * bandw + j * TK_PAGE + c * 8); }
   };
-  fetch(ka);
+  for (int i = H * 8 + lane; i < HB * 16 * 8; i += 32) {   // heads past H
+    *reinterpret_cast<uint4*>(buf + ms_off(i >> 3, i & 7, 8)) = make_uint4(0, 0, 0, 0);
+    *reinterpret_cast<uint4*>(buf + TB + ms_off(i >> 3, i & 7, 8)) = make_uint4(0, 0, 0, 0);
+  }
+  fetch(ja);
   tk_commit();
   uint32_t tf[HB][HB][4];
 #pragma unroll
   for (int i = 0; i < HB; ++i)
 #pragma unroll
     for (int j = 0; j < HB; ++j) talk_frag(p.talk, H, 16 * i, 16, 16 * j, lane, tf[i][j]);
-  const int batches = (per + NB - 1) / NB, ksteps = p.dk / 16;
-  for (int step = ka; step < kb; ++step) {
-    tk_wait<0>();
-    __syncthreads();
-    const int k0 = base + step * TW_KEYS;
-    // ---- scores and weights
-    for (int unit = warp; unit < G * batches; unit += 8) {
-      const int g = unit / batches, h0 = g * per + (unit - g * batches) * NB, last = (g + 1) * per - 1;
-      float s[NB][4][4];
-#pragma unroll
-      for (int n = 0; n < NB; ++n)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) s[n][i][0] = s[n][i][1] = s[n][i][2] = s[n][i][3] = 0.f;
-      const uint32_t ak = smem_u32(sK + g * KB);
-#pragma unroll 2
-      for (int ks = 0; ks < ksteps; ++ks) {
-        uint32_t bf[2][4];
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-          ms_ldsm4(ak + ms_off(16 * j + ((lane >> 4) << 3) + (lane & 7), 2 * ks + ((lane >> 3) & 1), KCH), bf[j][0], bf[j][1], bf[j][2], bf[j][3]);
-#pragma unroll
-        for (int n = 0; n < NB; ++n) {
-          uint32_t a[4];
-          ms_ldsm4(smem_u32(sQ + min(h0 + n, last) * QB) + ms_off((lane & 7) + (((lane >> 3) & 1) << 3), 2 * ks + (lane >> 4), KCH), a[0], a[1], a[2], a[3]);
-#pragma unroll
-          for (int j = 0; j < 2; ++j) { ms_mma(s[n][2 * j], a, bf[j][0], bf[j][1]); ms_mma(s[n][2 * j + 1], a, bf[j][2], bf[j][3]); }
-        }
-      }
-      const bool inside = k0 + TW_KEYS - 1 <= pos0 && k0 > pos0 + 15 - p.window;
-#pragma unroll
-      for (int n = 0; n < NB; ++n) {
-        const int h = h0 + n;
-        if (h > last) continue;
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int r = gq + 8 * e, pos = pos0 + r;
-          const float z = sZ[h * 16 + r];
-          uint32_t w[4];
-#pragma unroll
-          for (int i = 0; i < 4; ++i) {
-            const int key = k0 + 8 * i + 2 * tq;
-            float x = tk_ex2(fmaf(s[n][i][2 * e], p.scale_log2, -z)), y = tk_ex2(fmaf(s[n][i][2 * e + 1], p.scale_log2, -z));
-            if (!inside) {
-              x = key <= pos && key > pos - p.window ? x : 0.f;
-              y = key + 1 <= pos && key + 1 > pos - p.window ? y : 0.f;
-            }
-            w[i] = pack_half2(x, y);
-          }
-          // keys 8 i + 2 t + {0, 1} of row r: chunk 4 r + t
-          *reinterpret_cast<uint4*>(sP + tw_off(h, 4 * r + tq)) = make_uint4(w[0], w[1], w[2], w[3]);
-        }
-      }
-    }
-    __syncthreads();
-    if (step + 1 < kb) fetch(step + 1);
+  const float* mrow = p.m + ((size_t)slot * H + min(lane, H - 1)) * p.band * TK_ROWS + row;          // lane: head
+  const float z = p.z[((size_t)slot * H + min(lane, H - 1)) * TK_ROWS + row];
+  for (int j = ja; j < jb; ++j) {
+    if (j + 1 < jb) fetch(j + 1);
     tk_commit();
-    // ---- mixed: a warp takes two rows; column n of chunk 4 r + c is key 8 (n / 2) + 2 c + n % 2, so a thread gets keys 8 t .. 8 t + 7
-    const uint32_t ap = smem_u32(sP);
+    const float f = lane < H ? tk_ex2(mrow[(size_t)j * TK_ROWS] - z) : 0.f;
+    uint32_t fac[HB][2];
 #pragma unroll
-    for (int rr = 0; rr < 2; ++rr) {
-      const int r = 2 * warp + rr;
-      uint32_t bf[HB][2][4];
+    for (int k = 0; k < HB; ++k)
 #pragma unroll
-      for (int j = 0; j < HB; ++j)
-#pragma unroll
-        for (int c = 0; c < 2; ++c)
-          ms_ldsm4t(ap + tw_off(16 * j + (lane & 7) + (((lane >> 3) & 1) << 3), 4 * r + 2 * c + (lane >> 4)), bf[j][c][0], bf[j][c][1], bf[j][c][2], bf[j][c][3]);
-#pragma unroll
-      for (int i = 0; i < HB; ++i) {
-        float m[4][4];
-#pragma unroll
-        for (int c = 0; c < 4; ++c) m[c][0] = m[c][1] = m[c][2] = m[c][3] = 0.f;
-#pragma unroll
-        for (int j = 0; j < HB; ++j)
-#pragma unroll
-          for (int c = 0; c < 2; ++c) { mma_f16(m[2 * c], tf[i][j], bf[j][c][0], bf[j][c][1]); mma_f16(m[2 * c + 1], tf[i][j], bf[j][c][2], bf[j][c][3]); }
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int h = 16 * i + gq + 8 * e;
-          if (h < H)
-            *reinterpret_cast<uint4*>(dst + ((size_t)h * 64 + r) * bandw + step * TW_KEYS + 8 * tq) =
-                make_uint4(pack_bf16x2(m[0][2 * e], m[0][2 * e + 1]), pack_bf16x2(m[1][2 * e], m[1][2 * e + 1]), pack_bf16x2(m[2][2 * e], m[2][2 * e + 1]),
-                           pack_bf16x2(m[3][2 * e], m[3][2 * e + 1]));
-        }
+      for (int e = 0; e < 2; ++e) {
+        const int h = 16 * k + 8 * e + 2 * tq;
+        fac[k][e] = pack_half2(__shfl_sync(0xffffffffu, f, h), __shfl_sync(0xffffffffu, f, h + 1));
       }
+    tk_wait<1>();
+    __syncwarp();
+    uint8_t* d = buf + (j & 1) * TB;
+    const uint32_t ad = smem_u32(d);
+    uint32_t bf[HB][8][2];
+#pragma unroll
+    for (int k = 0; k < HB; ++k)
+#pragma unroll
+      for (int c = 0; c < 8; c += 2) {
+        ms_ldsm4t(ad + ms_off(16 * k + (lane & 7) + (((lane >> 3) & 1) << 3), c + (lane >> 4), 8), bf[k][c][0], bf[k][c][1], bf[k][c + 1][0], bf[k][c + 1][1]);
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const __half2 x = __hmul2(*reinterpret_cast<const __half2*>(&bf[k][c + i][e]), *reinterpret_cast<const __half2*>(&fac[k][e]));
+            bf[k][c + i][e] = *reinterpret_cast<const uint32_t*>(&x);
+          }
+      }
+    __syncwarp();                                          // all lanes hold their operands: the tile may be overwritten
+#pragma unroll
+    for (int i = 0; i < HB; ++i)
+#pragma unroll
+      for (int c = 0; c < 8; ++c) {
+        float o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int k = 0; k < HB; ++k) mma_f16(o, tf[i][k], bf[k][c][0], bf[k][c][1]);
+        ms_store2(d, 16 * i + gq, 8 * c + 2 * tq, 8, o[0], o[1]);
+        ms_store2(d, 16 * i + gq + 8, 8 * c + 2 * tq, 8, o[2], o[3]);
+      }
+    __syncwarp();
+    for (int i = lane; i < H * 8; i += 32) {
+      const int h = i >> 3, c = i & 7;
+      *reinterpret_cast<uint4*>(base + (size_t)h * TK_ROWS * bandw + j * TK_PAGE + c * 8) = *reinterpret_cast<const uint4*>(d + ms_off(h, c, 8));
     }
+    __syncwarp();                                          // read before the next tile but one arrives there
   }
 }
 
 // ---------------------------------------------------------------------------------------
-// talk_values: grid (tiles, G * batches of NH heads, sequences), 64 NH threads: a warp owns 32 rows of a head. DV: value width padded to
-// 64 or 128
+// talk_values: grid (tiles, G * batches of NH heads, sequences), 192 threads: TMA warp, MMA warp, four warps that store the result. Two
+// stages of NH weight tiles [128 rows, 64 keys] and a page of values.
 // ---------------------------------------------------------------------------------------
-template <int DV, int NH>
-__global__ void __launch_bounds__(64 * NH)
-talk_values_kernel(const TalkArgs p) {
+constexpr int TV_W = TK_ROWS * TK_PAGE * 2, TV_V = TK_PAGE * 128 * 2, TV_STAGES = 2;
+struct alignas(8) TalkValueBars {
+  uint64_t full[TV_STAGES], empty[TV_STAGES], done;
+  uint32_t tmem_base;
+  int abort_flag;
+};
+
+template <int NH>
+__global__ void __launch_bounds__(192, 2)
+talk_values_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmV, const TalkArgs p) {
   pdl_trigger();
-  extern __shared__ __align__(128) uint8_t tk_raw[];
-  constexpr int THREADS = 64 * NH, MB = NH * 64 * 128, VB = TK_PAGE * DV * 2, VCH = DV / 8;
-  uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tk_raw) + 127) & ~uintptr_t(127));     // two of [weights | values]
   pdl_wait();
-  const int b = blockIdx.z, tile = p.tile0 + blockIdx.x, per = p.H / p.G, batches = (per + NH - 1) / NH;
+  const int b = blockIdx.z, tile = p.tile0 + blockIdx.x, per = p.H / p.G, batches = (per + NH - 1) / NH, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = blockIdx.y / batches, h0 = g * per + (blockIdx.y % batches) * NH, heads = min(NH, (g + 1) * per - h0);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
   const TalkTile tl(p, b, tile);
   if (tl.real <= 0) return;
-  const int bandw = p.band * TK_PAGE, pages = tl.hi_page - tl.lo_page + 1;
-  const __nv_bfloat16* src = p.scratch + (((size_t)b * p.tiles + blockIdx.x) * p.H + h0) * 64 * bandw;
-  auto fetch = [&](int page) {
-    uint8_t* m = sm + (page & 1) * (MB + VB);
-    uint8_t* v = m + MB;
-    for (int i = tid; i < heads * 64 * 8; i += THREADS) {
-      const int r = i >> 3, c = i & 7;                     // rows past the prompt: never written, their products are not stored
-      tk_cp16(m + ms_off(r, c, 8), src + (size_t)r * bandw + page * TK_PAGE + c * 8);
+  extern __shared__ uint8_t tk_raw[];
+  __shared__ TalkValueBars bars;
+  constexpr int STAGE = NH * TV_W + TV_V;
+  uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tk_raw) + 1023) & ~uintptr_t(1023));
+  const bool hi = p.dv > 64;
+  if (threadIdx.x == 0) {
+    tma_prefetch_desc(&tmW); tma_prefetch_desc(&tmV);
+    for (int i = 0; i < TV_STAGES; ++i) { mbar_init(&bars.full[i], 1); mbar_init(&bars.empty[i], 1); }
+    mbar_init(&bars.done, 1);
+    bars.abort_flag = 0;
+    mbar_fence_init();
+  }
+  if (warp == 1) { tmem_alloc(&bars.tmem_base, NH * 128); tmem_relinquish(); }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_o = bars.tmem_base;
+  volatile int* abort_flag = &bars.abort_flag;
+  if (warp == 0) {
+    if (lane == 0) {
+      const int wrow = (((int)b * p.tiles + (int)blockIdx.x) * p.H + h0) * TK_ROWS;
+      bool bad = false;
+      for (int j = 0; j < tl.pages; ++j) {
+        const int st = j % TV_STAGES; const uint32_t ph = (j / TV_STAGES) & 1;
+        const int vrow = (talk_page(p, b, tl.lo_page + j, bad) * p.G + g) * TK_PAGE;
+        if (!mbar_wait(&bars.empty[st], ph ^ 1, abort_flag, p.status, KID_ATTN_PREFILL, 51)) break;
+        uint8_t* at = sm + st * STAGE;
+        mbar_expect_tx(&bars.full[st], heads * TV_W + (hi ? TV_V : TV_V / 2));
+        for (int n = 0; n < heads; ++n) tma_load_2d(at + n * TV_W, &tmW, &bars.full[st], j * TK_PAGE, wrow + n * TK_ROWS);
+        tma_load_2d(at + NH * TV_W, &tmV, &bars.full[st], 0, vrow);
+        if (hi) tma_load_2d(at + NH * TV_W + TV_V / 2, &tmV, &bars.full[st], 64, vrow);
+      }
+      if (bad) set_status(p.status, KID_ATTN_PREFILL, FF_ERR_BOUNDS, b, tile);
     }
-    int blk = p.block_table[(size_t)b * p.max_blocks + tl.lo_page + page];
-    if (blk < 0 || blk >= p.num_blocks) { if (tid == 0) set_status(p.status, KID_ATTN_PREFILL, FF_ERR_BOUNDS, b, page); blk = 0; }
-    const __nv_bfloat16* vp = p.vcache + ((size_t)blk * p.G + g) * TK_PAGE * p.dv;
-    for (int i = tid; i < TK_PAGE * VCH; i += THREADS) {
-      const int r = i / VCH, c = i - r * VCH;
-      if (c * 8 < p.dv) tk_cp16(v + ms_off(r, c, VCH), vp + (size_t)r * p.dv + c * 8);
-      else *reinterpret_cast<uint4*>(v + ms_off(r, c, VCH)) = make_uint4(0, 0, 0, 0);
+  } else if (warp == 1) {
+    if (lane == 0) {
+      const uint32_t idesc = umma_idesc(1, 1, 0, 1, TK_ROWS, hi ? 128 : 64);
+      bool ok = true;
+      for (int j = 0; j < tl.pages && ok; ++j) {
+        const int st = j % TV_STAGES; const uint32_t ph = (j / TV_STAGES) & 1;
+        if (!mbar_wait(&bars.full[st], ph, abort_flag, p.status, KID_ATTN_PREFILL, 52)) { ok = false; break; }
+        tc_fence_after();
+        const uint32_t at = smem_u32(sm + st * STAGE), v_addr = at + NH * TV_W;
+        for (int n = 0; n < heads; ++n)
+#pragma unroll
+          for (int k = 0; k < TK_PAGE / 16; ++k)
+            umma_f16(tmem_o + n * 128, umma_desc_sw128(at + n * TV_W + k * 32, 16, 1024), umma_desc_sw128(v_addr + k * 2048, TV_V / 2, 1024), idesc, (j | k) != 0);
+        umma_commit(&bars.empty[st]);
+      }
+      if (ok) umma_commit(&bars.done);
     }
-  };
-  float o[2][DV / 8][4];
+  } else {
+    const int q = warp & 3, row = q * 32 + lane;
+    bool ok = mbar_wait(&bars.done, 0, abort_flag, p.status, KID_ATTN_PREFILL, 53);
+    ok = __all_sync(0xffffffffu, ok);
+    if (ok) {
+      tc_fence_after();
+      for (int n = 0; n < heads; ++n) {
+        __nv_bfloat16* dst = p.out + (size_t)(p.q_start[b] + tile * TK_ROWS + row) * p.ldo + (size_t)(h0 + n) * p.dv;
+        for (int c = 0; c < p.dv; c += 16) {
+          uint32_t r[16];
+          tmem_ld_x16(tmem_o + (uint32_t(q * 32) << 16) + n * 128 + c, r);
+          tmem_ld_wait();
+          if (row < tl.real) {
+            uint32_t o[8];
 #pragma unroll
-  for (int i = 0; i < 2; ++i)
-#pragma unroll
-    for (int n = 0; n < DV / 8; ++n) o[i][n][0] = o[i][n][1] = o[i][n][2] = o[i][n][3] = 0.f;
-  fetch(0);
-  tk_commit();
-  const bool on = warp / 2 < heads;
-  for (int page = 0; page < pages; ++page) {
-    if (page + 1 < pages) fetch(page + 1);
-    tk_commit();
-    tk_wait<1>();
-    __syncthreads();
-    const uint32_t am = smem_u32(sm + (page & 1) * (MB + VB)), av = am + MB;
-    if (on) {
-#pragma unroll
-      for (int ks = 0; ks < 4; ++ks) {
-        uint32_t a[2][4];
-#pragma unroll
-        for (int i = 0; i < 2; ++i)
-          ms_ldsm4(am + ms_off(warp * 32 + 16 * i + (lane & 7) + (((lane >> 3) & 1) << 3), 2 * ks + (lane >> 4), 8), a[i][0], a[i][1], a[i][2], a[i][3]);
-#pragma unroll
-        for (int np = 0; np < DV / 16; ++np) {
-          uint32_t b0, b1, b2, b3;
-          ms_ldsm4t(av + ms_off(ks * 16 + (((lane >> 3) & 1) << 3) + (lane & 7), 2 * np + (lane >> 4), VCH), b0, b1, b2, b3);
-#pragma unroll
-          for (int i = 0; i < 2; ++i) { ms_mma(o[i][2 * np], a[i], b0, b1); ms_mma(o[i][2 * np + 1], a[i], b2, b3); }
+            for (int i = 0; i < 8; ++i) o[i] = pack_bf16x2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1]));
+            reinterpret_cast<uint4*>(dst + c)[0] = make_uint4(o[0], o[1], o[2], o[3]);
+            reinterpret_cast<uint4*>(dst + c)[1] = make_uint4(o[4], o[5], o[6], o[7]);
+          }
         }
       }
     }
-    __syncthreads();
   }
-  if (!on) return;
-  const int h = h0 + warp / 2;
-#pragma unroll
-  for (int i = 0; i < 2; ++i)
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int r = (warp & 1) * 32 + 16 * i + gq + 8 * e;
-      if (r >= tl.real) continue;
-      __nv_bfloat16* orow = p.out + (size_t)(p.q_start[b] + tile * 64 + r) * p.ldo + (size_t)h * p.dv;
-#pragma unroll
-      for (int n = 0; n < DV / 8; ++n)
-        if (8 * n + 2 * tq < p.dv) *reinterpret_cast<uint32_t*>(orow + 8 * n + 2 * tq) = pack_bf16x2(o[i][n][2 * e], o[i][n][2 * e + 1]);
-    }
+  tc_fence_before();
+  __syncthreads();
+  if (bars.abort_flag) {
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) { __nanosleep(1000); }
+  }
+  if (warp == 1) { __syncwarp(); tc_fence_after(); tmem_dealloc(tmem_o, NH * 128); }
 }
 
 // ---------------------------------------------------------------------------------------
@@ -317,7 +435,7 @@ struct TalkSpan {
   __device__ TalkSpan(const TalkDecodeArgs& p, int b, int split) {
     ctx = p.ctx_lens[b];
     lo_page = max(0, ctx - p.window) / TK_PAGE;
-    const int pages = ctx > 0 ? (ctx - 1) / TK_PAGE - lo_page + 1 : 0, each = (pages + p.splits - 1) / p.splits;
+    const int pages = ctx > 0 ? min(p.band, (ctx - 1) / TK_PAGE - lo_page + 1) : 0, each = (pages + p.splits - 1) / p.splits;
     page = min(pages, split * each);
     end = min(pages, page + each);
   }
@@ -523,60 +641,52 @@ talk_merge_kernel(const TalkDecodeArgs p) {
   p.out[(size_t)b * p.ldo + i] = __float2bfloat16(v);
 }
 
-template <int KP, int HB, int NB>
-static int talk_weights_launch(const TalkArgs& p, int batch, cudaStream_t s) {
-  const int smem = p.H * 16 * KP * 2 + p.G * TW_KEYS * KP * 2 + HB * 16 * 1024 + p.H * 16 * 4 + 128;
-  if (smem > 227 * 1024) return FF_HOST_TOO_LARGE;
-  if (int r = opt_in_smem(talk_weights_kernel<KP, HB, NB>, smem)) return r;
-  return launch_pdl(talk_weights_kernel<KP, HB, NB>, dim3(4 * p.tiles, p.parts, batch), dim3(256), smem, s, 0, p);
+template <int HB>
+static int talk_mix_launch(const TalkArgs& p, int batch, cudaStream_t s) {
+  const int smem = 8 * 2 * HB * 16 * 128 + 128;
+  if (int r = opt_in_smem(talk_mix_kernel<HB>, smem)) return r;
+  return launch_pdl(talk_mix_kernel<HB>, dim3(16 * p.tiles, p.parts, batch), dim3(256), smem, s, 0, p);
 }
-template <int KP, int HB>
-static int talk_weights_batch(const TalkArgs& p, int batch, cudaStream_t s) {
-  const int per = p.H / p.G;
-  if (per >= 4 && p.G * ((per + 3) / 4) >= 8) return talk_weights_launch<KP, HB, 4>(p, batch, s);
-  if (per >= 2 && p.G * ((per + 1) / 2) >= 8) return talk_weights_launch<KP, HB, 2>(p, batch, s);
-  return talk_weights_launch<KP, HB, 1>(p, batch, s);
-}
-template <int KP>
-static int talk_weights_heads(const TalkArgs& p, int batch, cudaStream_t s) {
-  if (p.H <= 16) return talk_weights_batch<KP, 1>(p, batch, s);
-  if (p.H <= 32) return talk_weights_batch<KP, 2>(p, batch, s);
-  return FF_HOST_TOO_LARGE;
-}
-template <int DV, int NH>
-static int talk_values_launch(const TalkArgs& p, int batch, cudaStream_t s) {
-  const int per = p.H / p.G, smem = 2 * (NH * 64 * 128 + TK_PAGE * DV * 2) + 128;
-  if (int r = opt_in_smem(talk_values_kernel<DV, NH>, smem)) return r;
-  return launch_pdl(talk_values_kernel<DV, NH>, dim3(p.tiles, p.G * ((per + NH - 1) / NH), batch), dim3(64 * NH), smem, s, 0, p);
-}
-template <int DV>
-static int talk_values_heads(const TalkArgs& p, int batch, cudaStream_t s) {
-  const int per = p.H / p.G;
-  if (per >= 3) return talk_values_launch<DV, 4>(p, batch, s);
-  if (per == 2) return talk_values_launch<DV, 2>(p, batch, s);
-  return talk_values_launch<DV, 1>(p, batch, s);
+template <int NH>
+static int talk_values_launch(const CUtensorMap& tmW, const CUtensorMap& tmV, const TalkArgs& p, int batch, cudaStream_t s) {
+  const int per = p.H / p.G, smem = TV_STAGES * (NH * TV_W + TV_V) + 1024;
+  if (int r = opt_in_smem(talk_values_kernel<NH>, smem)) return r;
+  return launch_pdl(talk_values_kernel<NH>, dim3(p.tiles, p.G * ((per + NH - 1) / NH), batch), dim3(192), smem, s, 0, tmW, tmV, p);
 }
 
 }  // namespace ff
 using namespace ff;
 
-// Mixed weights and value product of prompts. z [rows, H]: base-2 logarithm of every row's and head's soft-max denominator; scratch BF16
-// [batch, tiles_per_round, H, 64, band * 64], band: the pages the 64 rows of a tile see at most; parts: CTAs that share a tile's keys; caches [num_blocks, G, 64, dk / dv].
-// dk, dv multiples of 16 up to 128, H up to 32.
+// Prompts. q: packed rows [total_rows, ldq] with head h at column h * dk; caches [num_blocks, G, 64, dk / dv]; talk FP32 [H, H]; out rows of
+// pitch ldo; scratch: batch * tiles_per_round slots of H * 128 * (33 band + 1) floats; parts: warps that share a row's keys in talk_mix; one: the extra term of the
+// denominator (0 or 1). dk, dv multiples of 16 up to 128, H up to 32.
 FF_EXPORT int ff_talk_prefill(const void* q, const void* kcache, const void* vcache, const int* block_table, const int* q_start, const int* q_lens,
-                              const int* ctx_lens, const float* talk, const float* z, void* out, void* scratch, int batch, int max_q_len, int H, int G,
-                              int dk, int dv, int ldq, int ldo, int max_blocks, int num_blocks, int window, int band, int tiles_per_round, int parts, float scale,
-                              int* status, cudaStream_t s) {
-  if (batch <= 0 || batch > 65535 || max_q_len <= 0 || H <= 0 || G <= 0 || H % G || window < 1 || band < 1 || tiles_per_round < 1 || parts < 1 || parts > 64 || scratch == nullptr) return FF_HOST_BAD_SHAPE;
-  if (dk < 16 || dk > 128 || dk % 16 || dv < 16 || dv > 128 || dv % 16) return FF_HOST_BAD_SHAPE;
-  if (ldq % 8 || ldo % 2 || (reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(scratch) & 15) || (reinterpret_cast<uintptr_t>(out) & 3)) return FF_HOST_BAD_ALIGN;
-  const int tiles = (max_q_len + 63) / 64;
+                              const int* ctx_lens, const float* talk, void* out, float* scratch, int batch, int total_rows, int max_q_len, int H, int G,
+                              int dk, int dv, int ldq, int ldo, int max_blocks, int num_blocks, int window, int band, int tiles_per_round, int parts,
+                              float scale, float one, int* status, cudaStream_t s) {
+  if (batch <= 0 || batch > 65535 || total_rows <= 0 || max_q_len <= 0 || H <= 0 || G <= 0 || H % G || window < 1 || band < 1 || tiles_per_round < 1 ||
+      parts < 1 || parts > 1024 || scratch == nullptr || !(scale > 0.f) || !(one >= 0.f)) return FF_HOST_BAD_SHAPE;
+  if (dk < 16 || dk > 128 || dk % 16 || dv < 16 || dv > 128 || dv % 16 || ldq < H * dk || ldo < H * dv) return FF_HOST_BAD_SHAPE;
+  const long long rows = (long long)batch * tiles_per_round * H * TK_ROWS;
+  if (H > 32 || rows > (1ll << 30)) return FF_HOST_TOO_LARGE;
+  if (ldq % 8 || ldo % 8 || (reinterpret_cast<uintptr_t>(scratch) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return FF_HOST_BAD_ALIGN;
+  constexpr auto BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;    // weights: two bytes either way
+  const uint64_t bandw = (uint64_t)band * TK_PAGE, cache_rows = (uint64_t)num_blocks * G * TK_PAGE;
+  CUtensorMap tmQ, tmK, tmV, tmP, tmW;
+  if (int r = make_tmap_2d(&tmQ, q, BF, 2, (uint64_t)ldq, total_rows, (uint64_t)ldq * 2, 64, TK_ROWS)) return r;
+  if (int r = make_tmap_2d(&tmK, kcache, BF, 2, dk, cache_rows, (uint64_t)dk * 2, 64, TK_PAGE)) return r;
+  if (int r = make_tmap_2d(&tmV, vcache, BF, 2, dv, cache_rows, (uint64_t)dv * 2, 64, TK_PAGE)) return r;
+  if (int r = make_tmap_2d(&tmP, scratch, BF, 2, bandw, rows, bandw * 2, 64, 32)) return r;
+  if (int r = make_tmap_2d(&tmW, scratch, BF, 2, bandw, rows, bandw * 2, 64, TK_ROWS)) return r;
+  if (int r = opt_in_smem(talk_weights_kernel, TW_SMEM)) return r;
+  float* m = scratch + rows * (long long)bandw / 2;
+  const int tiles = (max_q_len + TK_ROWS - 1) / TK_ROWS;
   for (int t0 = 0; t0 < tiles; t0 += tiles_per_round) {
-    const TalkArgs p = {(const __nv_bfloat16*)q, (const __nv_bfloat16*)kcache, (const __nv_bfloat16*)vcache, block_table, q_start, q_lens, ctx_lens, talk, z,
-                        (__nv_bfloat16*)out, (__nv_bfloat16*)scratch, H, G, dk, dv, ldq, ldo, max_blocks, num_blocks, window, band, t0,
-                        tiles - t0 < tiles_per_round ? tiles - t0 : tiles_per_round, parts, scale * TK_LOG2E, status};
-    if (int r = dk <= 64 ? talk_weights_heads<64>(p, batch, s) : talk_weights_heads<128>(p, batch, s)) return r;
-    if (int r = dv <= 64 ? talk_values_heads<64>(p, batch, s) : talk_values_heads<128>(p, batch, s)) return r;
+    const TalkArgs p = {block_table, q_start, q_lens, ctx_lens, talk, (__nv_bfloat16*)out, (__nv_bfloat16*)scratch, m, m + rows * band, H, G, dk, dv, ldo,
+                        max_blocks, num_blocks, window, band, t0, tiles - t0 < tiles_per_round ? tiles - t0 : tiles_per_round, parts, scale * TK_LOG2E, one, status};
+    if (int r = launch_pdl(talk_weights_kernel, dim3(p.tiles, H, batch), dim3(192), TW_SMEM, s, 0, tmQ, tmK, tmP, p)) return r;
+    if (int r = H <= 16 ? talk_mix_launch<1>(p, batch, s) : talk_mix_launch<2>(p, batch, s)) return r;
+    if (int r = H / G >= 2 ? talk_values_launch<2>(tmW, tmV, p, batch, s) : talk_values_launch<1>(tmW, tmV, p, batch, s)) return r;
   }
   return launch_result();
 }

@@ -10,13 +10,13 @@ from ctypes import c_float
 
 import torch
 
-from . import BF16, _count, _require, _rows2d, attn_prefill, workspace
+from . import BF16, _count, _require, _rows2d, workspace
 from .lib import check, kernels, ptr, status_tensor, stream_ptr
 
 PAGE = 64
-SMEM = 227 * 1024
+ROWS = 128                    # query rows of a tile of the prompt kernels
 ROUND_BYTES = 80 << 20        # prompts: scratch of a round, to stay in the L2 cache
-FILL_CTAS = 148
+MIX_WARPS = 148 * 24          # prompts: warps the mixing kernel should have
 DECODE_CTAS = 592             # decode: CTAs a launch should have
 DECODE_SPLITS = 32
 
@@ -79,27 +79,21 @@ def talk_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
         out.copy_(_cpu(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, vdim, scale, window, talk, one))
         return out
     tensor = _check(q, kcache, vcache, hq, talk, out, block_table, q_start, q_lens, ctx_lens)
-    kp = 64 if dim <= 64 else 128
-    need = hq * 32 * kp + hkv * 64 * kp + -(-hq // 16) * 16384 + hq * 64 + 128
-    if not tensor or hq > 32 or need > SMEM:
+    if not tensor or hq > 32:
         _simt(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, scale, window, talk, one, out)
         return out
     rows, batch = q.shape[0], block_table.shape[0]
-    z = torch.empty(rows, hq, dtype=torch.float32, device=q.device)
-    sinks = torch.zeros(hq, dtype=torch.float32, device=q.device) if one else None
-    attn_prefill(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, max_q_len, hq, hkv, dim, scale, window=window, out=out, sinks=sinks,
-                 vdim=vdim, lse=z)                       # its result is overwritten
-    band = _band(max_ctx, window, 64)
-    tiles, tile_bytes = -(-max_q_len // 64), batch * hq * 64 * band * PAGE * 2
-    rounds = -(-tiles // max(1, ROUND_BYTES // tile_bytes))
+    band, tiles = _band(max_ctx, window, ROWS), -(-max_q_len // ROWS)
+    rounds = -(-tiles // max(1, ROUND_BYTES // (batch * hq * ROWS * band * PAGE * 2)))
     per_round = -(-tiles // rounds)
-    parts = max(1, min(-(-FILL_CTAS // (4 * per_round * batch)), band))
-    scratch = workspace(q.device).ensure("talk_weights", tile_bytes * per_round // 4)
-    rc = kernels().ff_talk_prefill(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(talk), ptr(z),
-                                   ptr(out), ptr(scratch), batch, max_q_len, hq, hkv, dim, vdim, q.stride(0), out.stride(0), block_table.stride(0),
-                                   kcache.shape[0], window, band, per_round, parts, c_float(scale), ptr(status_tensor(q.device)), stream_ptr())
+    parts = max(1, min(-(-MIX_WARPS // (ROWS * per_round * batch)), band))
+    scratch = workspace(q.device).ensure("talk_weights", batch * per_round * hq * ROWS * (band * (PAGE // 2 + 1) + 1))
+    rc = kernels().ff_talk_prefill(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(talk), ptr(out),
+                                   ptr(scratch), batch, rows, max_q_len, hq, hkv, dim, vdim, q.stride(0), out.stride(0), block_table.stride(0),
+                                   kcache.shape[0], window, band, per_round, parts, c_float(scale), c_float(float(one)), ptr(status_tensor(q.device)),
+                                   stream_ptr())
     check(rc, "ff_talk_prefill")
-    _count(2 * -(-tiles // per_round))
+    _count(3 * -(-tiles // per_round))
     return out
 
 
