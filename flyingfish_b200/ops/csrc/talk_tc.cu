@@ -4,11 +4,12 @@
 // The mixed weights of a head need the normalised weights of every head, so no head can run its soft-max and its value product in one
 // pass. Prompts take three, over tiles of 128 query rows:
 //   1. talk_weights : scores on tcgen05 as in attention_tc.cu, 64 keys at a time; 2^(s - m) in FP16 goes to scratch by TMA, m being the
-//                     row's maximum so far, and with it m of every step and z at the end;
+//                     maximum a thread has seen so far (two threads share a row, 32 keys each), and with it m of every step and z at
+//                     the end;
 //   2. talk_mix     : a warp takes a query row, 64 keys of all heads at a time: the weights times 2^(m - z), then their product with the
 //                     mixing matrix (mma.sync, heads as its inner dimension); mixed weights in BF16 replace the others in scratch;
 //   3. talk_values  : scratch times values on tcgen05, two heads that share a value head per CTA.
-// They go over a prompt in rounds whose scratch stays in the L2 cache. Decoded tokens take two and a merge:
+// They go over a prompt in rounds that bound the scratch. Decoded tokens take two and a merge:
 //   talk_scores : scores of a key / value head's query heads over a range of pages, in FP32, and their maximum and sum;
 //   talk_decode : the weights of all heads for a page, mixed for the heads of one value head (the accumulators of that product are the
 //                 operand of the next), times the values.
@@ -37,10 +38,10 @@ struct TalkArgs {
   const int* block_table; const int* q_start; const int* q_lens; const int* ctx_lens;
   const float* talk;
   __nv_bfloat16* out;
-  // a slot is a tile of this round: weights [slot, H, 128, band * 64], m [slot, H, band, 128], z [slot, H, 128]
+  // a slot is a tile of this round: weights [slot, H, 128, band * 64], m [slot, H, band, 2 halves, 128], z [slot, H, 128]
   __nv_bfloat16* weights; float* m; float* z;
   int H, G, dk, dv, ldo, max_blocks, num_blocks, window, band;         // band: pages a tile's rows see at most
-  int tile0, tiles, parts;                   // this round's tiles; warps that share a row's keys (talk_mix)
+  int tile0, tiles;                          // this round's tiles
   float scale_log2, one;
   int* status;
 };
@@ -75,22 +76,22 @@ __device__ __forceinline__ void talk_frag(const float* talk, int H, int row0, in
 }
 
 // ---------------------------------------------------------------------------------------
-// talk_weights: grid (tiles, H, sequences), 192 threads: TMA warp, MMA warp, four warps whose threads own a row each. Shared memory: Q
-// (two blocks of 64 columns), two K tiles, two staging tiles of 32 rows per row warp. Tensor memory: two score tiles of 64 columns.
+// talk_weights: grid (tiles, H, sequences), 320 threads: TMA warp, MMA warp, eight warps whose threads own 32 keys of a row each. Shared
+// memory: Q (two blocks of 64 columns), two K tiles, two staging tiles of 32 rows and 32 keys per such warp. Tensor memory: two score tiles of 64 columns.
 // ---------------------------------------------------------------------------------------
-constexpr int TW_Q = TK_ROWS * 128 * 2, TW_K = TK_PAGE * 128 * 2, TW_P = 32 * TK_PAGE * 2;
-constexpr int TW_SMEM = TW_Q + 2 * TW_K + 8 * TW_P + 1024;
+constexpr int TW_Q = TK_ROWS * 128 * 2, TW_K = TK_PAGE * 128 * 2, TW_P = 32 * 32 * 2;
+constexpr int TW_SMEM = TW_Q + 2 * TW_K + 16 * TW_P + 1024;
 
 struct alignas(8) TalkWeightBars {
   uint64_t q_full, k_full[2], k_empty[2], s_full[2], s_empty[2];
   uint32_t tmem_base;
   int abort_flag;
+  float m[TK_ROWS], l[TK_ROWS];
 };
 
-__global__ void __launch_bounds__(192, 2)
+__global__ void __launch_bounds__(320, 2)
 talk_weights_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmP,
                     const TalkArgs p) {
-  pdl_trigger();
   pdl_wait();
   const int b = blockIdx.z, h = blockIdx.y, tile = p.tile0 + blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const TalkTile tl(p, b, tile);
@@ -105,7 +106,7 @@ talk_weights_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   if (threadIdx.x == 0) {
     tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmP);
     mbar_init(&bars.q_full, 1);
-    for (int i = 0; i < 2; ++i) { mbar_init(&bars.k_full[i], 1); mbar_init(&bars.k_empty[i], 1); mbar_init(&bars.s_full[i], 1); mbar_init(&bars.s_empty[i], 4); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&bars.k_full[i], 1); mbar_init(&bars.k_empty[i], 1); mbar_init(&bars.s_full[i], 1); mbar_init(&bars.s_empty[i], 8); }
     bars.abort_flag = 0;
     mbar_fence_init();
   }
@@ -154,11 +155,11 @@ talk_weights_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
     }
   } else {
-    const int q = warp & 3, row = q * 32 + lane, pos = tl.first + row;
+    const int q = warp & 3, half = (warp - 2) >> 2, row = q * 32 + lane, pos = tl.first + row;
     const bool live = row < tl.real;
     const int last = live ? pos : -1, from = live ? max(0, pos - p.window + 1) : 0;
     const int all_lo = max(0, tl.first + tl.real - p.window), all_hi = tl.real == TK_ROWS ? tl.first : -1;     // keys every row sees
-    uint8_t* stg = sP + q * 2 * TW_P;
+    uint8_t* stg = sP + (q * 2 + half) * 2 * TW_P;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < tl.pages; ++j) {
@@ -167,37 +168,35 @@ talk_weights_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      float sv[64];
+      float sv[32];
       {
-        uint32_t r[64];
-        const uint32_t at = tmem_s + (uint32_t(q * 32) << 16) + st * TK_PAGE;
-        tmem_ld_x32(at, r);
-        tmem_ld_x32(at + 32, r + 32);
+        uint32_t r[32];
+        tmem_ld_x32(tmem_s + (uint32_t(q * 32) << 16) + st * TK_PAGE + 32 * half, r);
         tmem_ld_wait();
 #pragma unroll
-        for (int i = 0; i < 64; ++i) sv[i] = __uint_as_float(r[i]);
+        for (int i = 0; i < 32; ++i) sv[i] = __uint_as_float(r[i]);
       }
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars.s_empty[st]);
-      const int k0 = (tl.lo_page + j) * TK_PAGE;
+      const int k0 = (tl.lo_page + j) * TK_PAGE + 32 * half;
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      if (!(k0 >= all_lo && k0 + TK_PAGE - 1 <= all_hi)) {
+      if (!(k0 >= all_lo && k0 + 31 <= all_hi)) {
 #pragma unroll
-        for (int i = 0; i < 64; ++i) sv[i] = k0 + i >= from && k0 + i <= last ? sv[i] : -INFINITY;
+        for (int i = 0; i < 32; ++i) sv[i] = k0 + i >= from && k0 + i <= last ? sv[i] : -INFINITY;
       }
 #pragma unroll
-      for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
+      for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
       const float mn = fmaxf(m, fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2), mr = mn == -INFINITY ? 0.f : mn;
       l *= m == -INFINITY ? 0.f : tk_ex2(m - mr);
       m = mn;
-      p.m[(slot_head * p.band + j) * TK_ROWS + row] = m;
+      p.m[((slot_head * p.band + j) * 2 + half) * TK_ROWS + row] = m;
       if (lane == 0) tma_store_wait_read<1>();             // the staging tile's previous contents have left
       __syncwarp();
-      uint8_t* at = stg + st * TW_P + lane * 128;
+      uint8_t* at = stg + st * TW_P + lane * 64;
       float ls[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int c = 0; c < 8; ++c) {
+      for (int c = 0; c < 4; ++c) {
         uint32_t w[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
@@ -205,18 +204,22 @@ talk_weights_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           ls[i] += x + y;
           w[i] = pack_half2(x, y);
         }
-        *reinterpret_cast<uint4*>(at + ((c ^ (lane & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+        *reinterpret_cast<uint4*>(at + ((c ^ ((lane >> 1) & 3)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);      // 64-byte swizzle
       }
       l += (ls[0] + ls[1]) + (ls[2] + ls[3]);
       fence_proxy_async_smem();
       __syncwarp();
       if (lane == 0) {
-        tma_store_2d(&tmP, stg + st * TW_P, j * TK_PAGE, (int)(slot_head * TK_ROWS) + q * 32);
+        tma_store_2d(&tmP, stg + st * TW_P, j * TK_PAGE + 32 * half, (int)(slot_head * TK_ROWS) + q * 32);
         tma_store_commit();
       }
     }
-    const float n = p.one > 0.f ? fmaxf(m, 0.f) : m;
-    p.z[slot_head * TK_ROWS + row] = n == -INFINITY ? 0.f : n + log2f(l * tk_ex2(m - n) + (p.one > 0.f ? p.one * tk_ex2(-n) : 0.f));
+    if (half == 1) { bars.m[row] = m; bars.l[row] = l; }
+    asm volatile("bar.sync 1, 256;" ::: "memory");
+    if (half == 0) {
+      const float om = bars.m[row], n = fmaxf(fmaxf(m, om), p.one > 0.f ? 0.f : -INFINITY);
+      p.z[slot_head * TK_ROWS + row] = n == -INFINITY ? 0.f : n + log2f(l * tk_ex2(m - n) + bars.l[row] * tk_ex2(om - n) + (p.one > 0.f ? p.one * tk_ex2(-n) : 0.f));
+    }
     if (lane == 0) tma_store_wait<0>();
   }
   tc_fence_before();
@@ -229,90 +232,125 @@ talk_weights_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 }
 
 // ---------------------------------------------------------------------------------------
-// talk_mix: grid (16 * tiles, parts, sequences), 256 threads, a row per warp; HB: blocks of 16 heads
+// talk_mix: grid (16 * tiles, parts, sequences), 256 threads: eight neighbouring rows, a warp each, 64 keys of all heads at a time by TMA
+// (one box of H rows of 128 bytes), three tiles per warp: one on its way in, one being worked on, one on its way out. HB: blocks of 16
+// heads.
 // ---------------------------------------------------------------------------------------
+constexpr int TM_STAGES = 3;
+
+__device__ __forceinline__ void stmatrix4(uint32_t a, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
+  asm volatile("stmatrix.sync.aligned.m8n8.x4.shared.b16 [%0], {%1,%2,%3,%4};" ::"r"(a), "r"(r0), "r"(r1), "r"(r2), "r"(r3) : "memory");
+}
+__device__ __forceinline__ void talk_load_row(uint32_t dst, const CUtensorMap* m, uint64_t* bar, int key, int row, int slot) {
+  asm volatile("cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];"
+               ::"r"(dst), "l"(reinterpret_cast<uint64_t>(m)), "r"(smem_u32(bar)), "r"(key), "r"(row), "r"(0), "r"(slot) : "memory");
+}
+__device__ __forceinline__ void talk_store_row(const CUtensorMap* m, uint32_t src, int key, int row, int slot) {
+  asm volatile("cp.async.bulk.tensor.4d.global.shared::cta.bulk_group [%0, {%2, %3, %4, %5}], [%1];"
+               ::"l"(reinterpret_cast<uint64_t>(m)), "r"(src), "r"(key), "r"(row), "r"(0), "r"(slot) : "memory");
+}
+
 template <int HB>
-__global__ void __launch_bounds__(256)
-talk_mix_kernel(const TalkArgs p) {
-  pdl_trigger();
+__global__ void __launch_bounds__(256, 2)
+talk_mix_kernel(const __grid_constant__ CUtensorMap tmM, const TalkArgs p) {
   extern __shared__ __align__(128) uint8_t tk_raw[];
-  constexpr int TB = HB * 16 * 128;                        // [heads][64 keys]
+  constexpr int TB = HB * 16 * 128;                        // [heads][64 keys], 128-byte swizzle
+  __shared__ uint64_t s_full[8][TM_STAGES];
   pdl_wait();
-  const int b = blockIdx.z, slot = b * p.tiles + (blockIdx.x >> 4), warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
-  const int row = (blockIdx.x & 15) * 8 + warp, H = p.H;
+  const int b = blockIdx.z, slot = b * p.tiles + (blockIdx.x >> 4), row0 = (blockIdx.x & 15) * 8, H = p.H;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, tq = lane & 3;
   const TalkTile tl(p, b, p.tile0 + (blockIdx.x >> 4));
-  if (row >= tl.real) return;
-  uint8_t* buf = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tk_raw) + 127) & ~uintptr_t(127)) + warp * 2 * TB;
-  const int pos = tl.first + row, j0 = max(0, pos - p.window + 1) / TK_PAGE - tl.lo_page, j1 = min(tl.pages, pos / TK_PAGE - tl.lo_page + 1);     // the others are zero
-  const int ja = j0 + (j1 - j0) * (int)blockIdx.y / p.parts, jb = j0 + (j1 - j0) * ((int)blockIdx.y + 1) / p.parts;
-  if (ja >= jb) return;
-  const size_t bandw = (size_t)p.band * TK_PAGE;
-  __nv_bfloat16* base = p.weights + ((size_t)slot * H * TK_ROWS + row) * bandw;
-  auto fetch = [&](int j) {
-    uint8_t* d = buf + (j & 1) * TB;
-    for (int i = lane; i < H * 8; i += 32) { const int h = i >> 3, c = i & 7; tk_cp16(d + ms_off(h, c, 8), base + (size_t)h * TK_ROWS * bandw + j * TK_PAGE + c * 8); }
-  };
-  for (int i = H * 8 + lane; i < HB * 16 * 8; i += 32) {   // heads past H
-    *reinterpret_cast<uint4*>(buf + ms_off(i >> 3, i & 7, 8)) = make_uint4(0, 0, 0, 0);
-    *reinterpret_cast<uint4*>(buf + TB + ms_off(i >> 3, i & 7, 8)) = make_uint4(0, 0, 0, 0);
+  const int rows = min(8, tl.real - row0);
+  if (rows <= 0) return;
+  // steps that some row sees, and this CTA's share of them
+  const int pos = tl.first + row0, v0 = max(0, pos - p.window + 1) / TK_PAGE - tl.lo_page, v1 = min(tl.pages, (pos + rows - 1) / TK_PAGE - tl.lo_page + 1);
+  const int j0 = v0 + (v1 - v0) * (int)blockIdx.y / (int)gridDim.y, j1 = v0 + (v1 - v0) * ((int)blockIdx.y + 1) / (int)gridDim.y, n = j1 - j0;
+  if (n <= 0) return;
+  uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tk_raw) + 1023) & ~uintptr_t(1023));
+  __half* s_f = reinterpret_cast<__half*>(base + 8 * TM_STAGES * TB);  // [step][row][half][heads]
+  const uint32_t buf = smem_u32(base) + warp * TM_STAGES * TB;
+  uint64_t* full = s_full[warp];
+  if (lane == 0) {
+    for (int i = 0; i < TM_STAGES; ++i) mbar_init(&full[i], 1);
+    mbar_fence_init();
   }
-  fetch(ja);
-  tk_commit();
+  for (int i = H * 8 + lane; i < HB * 16 * 8; i += 32)     // heads past H
+    for (int st = 0; st < TM_STAGES; ++st)
+      asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(buf + st * TB + ms_off(i >> 3, i & 7, 8)), "r"(0) : "memory");
+  __syncwarp();
+  const bool live = warp < rows;
+  if (live && lane == 0) {
+    mbar_expect_tx(&full[0], H * 128);
+    talk_load_row(buf, &tmM, &full[0], j0 * TK_PAGE, row0 + warp, slot);
+  }
+  // the factors 2^(m - z) of all steps: a thread takes a row and heads tid / 8, + 32
+  for (int h = tid >> 3; h < HB * 16; h += 32) {
+    const int r = tid & 7;
+    const size_t sh = (size_t)slot * H + min(h, H - 1);
+    const float z = p.z[sh * TK_ROWS + row0 + r];
+    const float* mp = p.m + (sh * p.band + j0) * 2 * TK_ROWS + row0 + r;
+    for (int k = 0; k < 2 * n; ++k) s_f[((k >> 1) * 16 + 2 * r + (k & 1)) * HB * 16 + h] = __float2half(h < H ? tk_ex2(mp[(size_t)k * TK_ROWS] - z) : 0.f);
+  }
   uint32_t tf[HB][HB][4];
 #pragma unroll
   for (int i = 0; i < HB; ++i)
 #pragma unroll
-    for (int j = 0; j < HB; ++j) talk_frag(p.talk, H, 16 * i, 16, 16 * j, lane, tf[i][j]);
-  const float* mrow = p.m + ((size_t)slot * H + min(lane, H - 1)) * p.band * TK_ROWS + row;          // lane: head
-  const float z = p.z[((size_t)slot * H + min(lane, H - 1)) * TK_ROWS + row];
-  for (int j = ja; j < jb; ++j) {
-    if (j + 1 < jb) fetch(j + 1);
-    tk_commit();
-    const float f = lane < H ? tk_ex2(mrow[(size_t)j * TK_ROWS] - z) : 0.f;
-    uint32_t fac[HB][2];
-#pragma unroll
-    for (int k = 0; k < HB; ++k)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int h = 16 * k + 8 * e + 2 * tq;
-        fac[k][e] = pack_half2(__shfl_sync(0xffffffffu, f, h), __shfl_sync(0xffffffffu, f, h + 1));
-      }
-    tk_wait<1>();
-    __syncwarp();
-    uint8_t* d = buf + (j & 1) * TB;
-    const uint32_t ad = smem_u32(d);
-    uint32_t bf[HB][8][2];
-#pragma unroll
-    for (int k = 0; k < HB; ++k)
-#pragma unroll
-      for (int c = 0; c < 8; c += 2) {
-        ms_ldsm4t(ad + ms_off(16 * k + (lane & 7) + (((lane >> 3) & 1) << 3), c + (lane >> 4), 8), bf[k][c][0], bf[k][c][1], bf[k][c + 1][0], bf[k][c + 1][1]);
-#pragma unroll
-        for (int i = 0; i < 2; ++i)
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const __half2 x = __hmul2(*reinterpret_cast<const __half2*>(&bf[k][c + i][e]), *reinterpret_cast<const __half2*>(&fac[k][e]));
-            bf[k][c + i][e] = *reinterpret_cast<const uint32_t*>(&x);
-          }
-      }
-    __syncwarp();                                          // all lanes hold their operands: the tile may be overwritten
-#pragma unroll
-    for (int i = 0; i < HB; ++i)
-#pragma unroll
-      for (int c = 0; c < 8; ++c) {
-        float o[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-        for (int k = 0; k < HB; ++k) mma_f16(o, tf[i][k], bf[k][c][0], bf[k][c][1]);
-        ms_store2(d, 16 * i + gq, 8 * c + 2 * tq, 8, o[0], o[1]);
-        ms_store2(d, 16 * i + gq + 8, 8 * c + 2 * tq, 8, o[2], o[3]);
-      }
-    __syncwarp();
-    for (int i = lane; i < H * 8; i += 32) {
-      const int h = i >> 3, c = i & 7;
-      *reinterpret_cast<uint4*>(base + (size_t)h * TK_ROWS * bandw + j * TK_PAGE + c * 8) = *reinterpret_cast<const uint4*>(d + ms_off(h, c, 8));
+    for (int k = 0; k < HB; ++k) talk_frag(p.talk, H, 16 * i, 16, 16 * k, lane, tf[i][k]);
+  __syncthreads();
+  if (!live) return;
+  const int r16 = (lane & 7) + (((lane >> 3) & 1) << 3);
+  int st = 0; uint32_t ph = 0;
+  for (int k = 0; k < n; ++k) {
+    const int nx = st + 1 == TM_STAGES ? 0 : st + 1;
+    if (lane == 0 && k + 1 < n) {
+      tma_store_wait_read<1>();                            // the tile that left from there
+      mbar_expect_tx(&full[nx], H * 128);
+      talk_load_row(buf + nx * TB, &tmM, &full[nx], (j0 + k + 1) * TK_PAGE, row0 + warp, slot);
     }
-    __syncwarp();                                          // read before the next tile but one arrives there
+    if (!mbar_wait(&full[st], ph, nullptr, p.status, KID_ATTN_PREFILL, 61)) break;
+    __syncwarp();
+    const uint32_t d = buf + st * TB;
+    const uint32_t* fr = reinterpret_cast<const uint32_t*>(s_f + (k * 16 + 2 * warp) * HB * 16);
+#pragma unroll
+    for (int c = 0; c < 8; c += 2) {                       // 16 keys of all heads
+      const uint32_t at = d + r16 * 128 + (((c + (lane >> 4)) ^ (lane & 7)) << 4);
+      uint32_t bf[HB][4];
+#pragma unroll
+      for (int i = 0; i < HB; ++i) {
+        ms_ldsm4t(at + i * 2048, bf[i][0], bf[i][1], bf[i][2], bf[i][3]);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const uint32_t f = fr[((c >> 2) * HB * 16 + 16 * i + 8 * e) / 2 + tq];
+          const __half2 x = __hmul2(*reinterpret_cast<const __half2*>(&bf[i][e]), *reinterpret_cast<const __half2*>(&f));
+          const __half2 y = __hmul2(*reinterpret_cast<const __half2*>(&bf[i][2 + e]), *reinterpret_cast<const __half2*>(&f));
+          bf[i][e] = *reinterpret_cast<const uint32_t*>(&x);
+          bf[i][2 + e] = *reinterpret_cast<const uint32_t*>(&y);
+        }
+      }
+      float a[HB][2][4];
+#pragma unroll
+      for (int i = 0; i < HB; ++i) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[i][0][e] = a[i][1][e] = 0.f;
+#pragma unroll
+        for (int q = 0; q < HB; ++q) { mma_f16(a[i][0], tf[i][q], bf[q][0], bf[q][1]); mma_f16(a[i][1], tf[i][q], bf[q][2], bf[q][3]); }
+      }
+      __syncwarp();                                        // these keys are in registers: their place takes the result
+#pragma unroll
+      for (int i = 0; i < HB; ++i)
+        stmatrix4(at + i * 2048, pack_bf16x2(a[i][0][0], a[i][0][1]), pack_bf16x2(a[i][0][2], a[i][0][3]), pack_bf16x2(a[i][1][0], a[i][1][1]),
+                  pack_bf16x2(a[i][1][2], a[i][1][3]));
+    }
+    fence_proxy_async_smem();
+    __syncwarp();
+    if (lane == 0) {
+      talk_store_row(&tmM, d, (j0 + k) * TK_PAGE, row0 + warp, slot);
+      tma_store_commit();
+    }
+    st = nx;
+    if (st == 0) ph ^= 1;
   }
+  if (lane == 0) tma_store_wait<0>();
 }
 
 // ---------------------------------------------------------------------------------------
@@ -329,7 +367,6 @@ struct alignas(8) TalkValueBars {
 template <int NH>
 __global__ void __launch_bounds__(192, 2)
 talk_values_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmV, const TalkArgs p) {
-  pdl_trigger();
   pdl_wait();
   const int b = blockIdx.z, tile = p.tile0 + blockIdx.x, per = p.H / p.G, batches = (per + NH - 1) / NH, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = blockIdx.y / batches, h0 = g * per + (blockIdx.y % batches) * NH, heads = min(NH, (g + 1) * per - h0);
@@ -641,11 +678,38 @@ talk_merge_kernel(const TalkDecodeArgs p) {
   p.out[(size_t)b * p.ldo + i] = __float2bfloat16(v);
 }
 
+// boxes of 32 keys and 32 rows, 64-byte swizzle
+static int talk_store_map(CUtensorMap* out, void* base, uint64_t inner, uint64_t outer) {
+  EncodeTiledFn fn = encode_tiled_fn();
+  if (!fn) return FF_HOST_NO_DRIVER;
+  const cuuint64_t dims[2] = {inner, outer}, strides[1] = {inner * 2};
+  const cuuint32_t box[2] = {32, 32}, step[2] = {1, 1};
+  const CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, base, dims, strides, box, step, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_64B,
+                        CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? FF_HOST_OK : FF_HOST_TMAP_FAIL;
+}
+
+// weights as (key, row, head, slot), boxes of 64 keys of all heads
+static int talk_row_map(CUtensorMap* out, void* base, uint64_t bandw, uint64_t heads, uint64_t slots) {
+  EncodeTiledFn fn = encode_tiled_fn();
+  if (!fn) return FF_HOST_NO_DRIVER;
+  const cuuint64_t dims[4] = {bandw, TK_ROWS, heads, slots}, strides[3] = {bandw * 2, bandw * 2 * TK_ROWS, bandw * 2 * TK_ROWS * heads};
+  const cuuint32_t box[4] = {TK_PAGE, 1, (cuuint32_t)heads, 1}, step[4] = {1, 1, 1, 1};
+  const CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, base, dims, strides, box, step, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+                        CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? FF_HOST_OK : FF_HOST_TMAP_FAIL;
+}
+
 template <int HB>
-static int talk_mix_launch(const TalkArgs& p, int batch, cudaStream_t s) {
-  const int smem = 8 * 2 * HB * 16 * 128 + 128;
+static int talk_mix_launch(const CUtensorMap& tmM, const TalkArgs& p, int batch, cudaStream_t s) {
+  // CTAs that share a row's keys: enough for the device, and few enough steps each for the factors
+  const int groups = batch * p.tiles * (TK_ROWS / 8), fit = 2 * sm_count(), most = HB == 1 ? 32 : 16;
+  int parts = groups < fit ? (fit + groups - 1) / groups : 1;
+  if (parts < (p.band + most - 1) / most) parts = (p.band + most - 1) / most;
+  const int steps = (p.band + parts - 1) / parts, smem = 8 * TM_STAGES * HB * 16 * 128 + steps * 16 * HB * 16 * 2 + 1024;
+  if (parts > 65535) return FF_HOST_TOO_LARGE;
   if (int r = opt_in_smem(talk_mix_kernel<HB>, smem)) return r;
-  return launch_pdl(talk_mix_kernel<HB>, dim3(16 * p.tiles, p.parts, batch), dim3(256), smem, s, 0, p);
+  return launch_pdl(talk_mix_kernel<HB>, dim3(16 * p.tiles, parts, batch), dim3(256), smem, s, 0, tmM, p);
 }
 template <int NH>
 static int talk_values_launch(const CUtensorMap& tmW, const CUtensorMap& tmV, const TalkArgs& p, int batch, cudaStream_t s) {
@@ -658,34 +722,36 @@ static int talk_values_launch(const CUtensorMap& tmW, const CUtensorMap& tmV, co
 using namespace ff;
 
 // Prompts. q: packed rows [total_rows, ldq] with head h at column h * dk; caches [num_blocks, G, 64, dk / dv]; talk FP32 [H, H]; out rows of
-// pitch ldo; scratch: batch * tiles_per_round slots of H * 128 * (33 band + 1) floats; parts: warps that share a row's keys in talk_mix; one: the extra term of the
+// pitch ldo; scratch: batch * tiles_per_round slots of H * 128 * (34 band + 1) floats; the call takes the rounds
+// first_round, first_round + round_step, ..; one: the extra term of the
 // denominator (0 or 1). dk, dv multiples of 16 up to 128, H up to 32.
 FF_EXPORT int ff_talk_prefill(const void* q, const void* kcache, const void* vcache, const int* block_table, const int* q_start, const int* q_lens,
                               const int* ctx_lens, const float* talk, void* out, float* scratch, int batch, int total_rows, int max_q_len, int H, int G,
-                              int dk, int dv, int ldq, int ldo, int max_blocks, int num_blocks, int window, int band, int tiles_per_round, int parts,
+                              int dk, int dv, int ldq, int ldo, int max_blocks, int num_blocks, int window, int band, int tiles_per_round, int first_round, int round_step,
                               float scale, float one, int* status, cudaStream_t s) {
   if (batch <= 0 || batch > 65535 || total_rows <= 0 || max_q_len <= 0 || H <= 0 || G <= 0 || H % G || window < 1 || band < 1 || tiles_per_round < 1 ||
-      parts < 1 || parts > 1024 || scratch == nullptr || !(scale > 0.f) || !(one >= 0.f)) return FF_HOST_BAD_SHAPE;
+      first_round < 0 || round_step < 1 || scratch == nullptr || !(scale > 0.f) || !(one >= 0.f)) return FF_HOST_BAD_SHAPE;
   if (dk < 16 || dk > 128 || dk % 16 || dv < 16 || dv > 128 || dv % 16 || ldq < H * dk || ldo < H * dv) return FF_HOST_BAD_SHAPE;
   const long long rows = (long long)batch * tiles_per_round * H * TK_ROWS;
   if (H > 32 || rows > (1ll << 30)) return FF_HOST_TOO_LARGE;
   if (ldq % 8 || ldo % 8 || (reinterpret_cast<uintptr_t>(scratch) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return FF_HOST_BAD_ALIGN;
   constexpr auto BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;    // weights: two bytes either way
   const uint64_t bandw = (uint64_t)band * TK_PAGE, cache_rows = (uint64_t)num_blocks * G * TK_PAGE;
-  CUtensorMap tmQ, tmK, tmV, tmP, tmW;
+  CUtensorMap tmQ, tmK, tmV, tmP, tmW, tmM;
   if (int r = make_tmap_2d(&tmQ, q, BF, 2, (uint64_t)ldq, total_rows, (uint64_t)ldq * 2, 64, TK_ROWS)) return r;
   if (int r = make_tmap_2d(&tmK, kcache, BF, 2, dk, cache_rows, (uint64_t)dk * 2, 64, TK_PAGE)) return r;
   if (int r = make_tmap_2d(&tmV, vcache, BF, 2, dv, cache_rows, (uint64_t)dv * 2, 64, TK_PAGE)) return r;
-  if (int r = make_tmap_2d(&tmP, scratch, BF, 2, bandw, rows, bandw * 2, 64, 32)) return r;
+  if (int r = talk_store_map(&tmP, scratch, bandw, rows)) return r;
   if (int r = make_tmap_2d(&tmW, scratch, BF, 2, bandw, rows, bandw * 2, 64, TK_ROWS)) return r;
+  if (int r = talk_row_map(&tmM, scratch, bandw, H, (uint64_t)batch * tiles_per_round)) return r;
   if (int r = opt_in_smem(talk_weights_kernel, TW_SMEM)) return r;
   float* m = scratch + rows * (long long)bandw / 2;
   const int tiles = (max_q_len + TK_ROWS - 1) / TK_ROWS;
-  for (int t0 = 0; t0 < tiles; t0 += tiles_per_round) {
-    const TalkArgs p = {block_table, q_start, q_lens, ctx_lens, talk, (__nv_bfloat16*)out, (__nv_bfloat16*)scratch, m, m + rows * band, H, G, dk, dv, ldo,
-                        max_blocks, num_blocks, window, band, t0, tiles - t0 < tiles_per_round ? tiles - t0 : tiles_per_round, parts, scale * TK_LOG2E, one, status};
-    if (int r = launch_pdl(talk_weights_kernel, dim3(p.tiles, H, batch), dim3(192), TW_SMEM, s, 0, tmQ, tmK, tmP, p)) return r;
-    if (int r = H <= 16 ? talk_mix_launch<1>(p, batch, s) : talk_mix_launch<2>(p, batch, s)) return r;
+  for (int t0 = first_round * tiles_per_round; t0 < tiles; t0 += round_step * tiles_per_round) {
+    const TalkArgs p = {block_table, q_start, q_lens, ctx_lens, talk, (__nv_bfloat16*)out, (__nv_bfloat16*)scratch, m, m + 2 * rows * band, H, G, dk, dv, ldo,
+                        max_blocks, num_blocks, window, band, t0, tiles - t0 < tiles_per_round ? tiles - t0 : tiles_per_round, scale * TK_LOG2E, one, status};
+    if (int r = launch_pdl(talk_weights_kernel, dim3(p.tiles, H, batch), dim3(320), TW_SMEM, s, 0, tmQ, tmK, tmP, p)) return r;
+    if (int r = H <= 16 ? talk_mix_launch<1>(tmM, p, batch, s) : talk_mix_launch<2>(tmM, p, batch, s)) return r;
     if (int r = H / G >= 2 ? talk_values_launch<2>(tmW, tmV, p, batch, s) : talk_values_launch<1>(tmW, tmV, p, batch, s)) return r;
   }
   return launch_result();

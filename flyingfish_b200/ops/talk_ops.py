@@ -10,15 +10,15 @@ from ctypes import c_float
 
 import torch
 
-from . import BF16, _count, _require, _rows2d, workspace
+from . import BF16, _count, _require, SideLane, _rows2d, workspace
 from .lib import check, kernels, ptr, status_tensor, stream_ptr
 
 PAGE = 64
 ROWS = 128                    # query rows of a tile of the prompt kernels
-ROUND_BYTES = 80 << 20        # prompts: scratch of a round, to stay in the L2 cache
-MIX_WARPS = 148 * 24          # prompts: warps the mixing kernel should have
+ROUND_BYTES = 100 << 20       # prompts: scratch of a round
 DECODE_CTAS = 592             # decode: CTAs a launch should have
 DECODE_SPLITS = 32
+_lanes: dict[int, SideLane] = {}
 
 
 def _cpu(q, kcache, vcache, block_table, q_start, q_lens, ctx_lens, hq, hkv, dim, vdim, scale, window, talk, one) -> torch.Tensor:
@@ -86,13 +86,26 @@ def talk_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
     band, tiles = _band(max_ctx, window, ROWS), -(-max_q_len // ROWS)
     rounds = -(-tiles // max(1, ROUND_BYTES // (batch * hq * ROWS * band * PAGE * 2)))
     per_round = -(-tiles // rounds)
-    parts = max(1, min(-(-MIX_WARPS // (ROWS * per_round * batch)), band))
-    scratch = workspace(q.device).ensure("talk_weights", batch * per_round * hq * ROWS * (band * (PAGE // 2 + 1) + 1))
-    rc = kernels().ff_talk_prefill(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(talk), ptr(out),
-                                   ptr(scratch), batch, rows, max_q_len, hq, hkv, dim, vdim, q.stride(0), out.stride(0), block_table.stride(0),
-                                   kcache.shape[0], window, band, per_round, parts, c_float(scale), c_float(float(one)), ptr(status_tensor(q.device)),
-                                   stream_ptr())
-    check(rc, "ff_talk_prefill")
+    floats = batch * per_round * hq * ROWS * (band * (PAGE // 2 + 2) + 1)
+
+    def run(first: int, step: int) -> None:
+        scratch = workspace(q.device).ensure("talk_weights", floats)
+        rc = kernels().ff_talk_prefill(ptr(q), ptr(kcache), ptr(vcache), ptr(block_table), ptr(q_start), ptr(q_lens), ptr(ctx_lens), ptr(talk), ptr(out),
+                                       ptr(scratch), batch, rows, max_q_len, hq, hkv, dim, vdim, q.stride(0), out.stride(0), block_table.stride(0),
+                                       kcache.shape[0], window, band, per_round, first, step, c_float(scale), c_float(float(one)),
+                                       ptr(status_tensor(q.device)), stream_ptr())
+        check(rc, "ff_talk_prefill")
+    if rounds == 1:
+        run(0, 1)
+    else:                              # every other round on a second stream: a round's tail runs under the next one
+        lane = _lanes.get(q.device.index)
+        if lane is None:
+            lane = _lanes[q.device.index] = SideLane(q.device)
+        lane.fork()
+        with lane:
+            run(1, 2)
+        run(0, 2)
+        lane.join()
     _count(3 * -(-tiles // per_round))
     return out
 
