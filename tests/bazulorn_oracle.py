@@ -172,7 +172,7 @@ def experts(h, t, p, cfg):
 MIXERS = {"channel_delta": channel_delta, "parallel": side_by_side}
 
 
-def run(cfg, tensors, ids, dt=torch.float64):
+def forward(cfg, tensors, ids, dt=torch.float64):
     """(logits [n, vocab], residual after every layer [layers, n, width])."""
     t = lambda name: tensors[name].to(dt)
     eps = cfg["norm"]["eps"]
@@ -188,3 +188,83 @@ def run(cfg, tensors, ids, dt=torch.float64):
         x = x + y
         after.append(x)
     return (rms(x, eps) * t("final.norm")) @ t("embed").T, torch.stack(after)
+
+
+# ------------------------------------------------------------------------------------------
+# configurations and weights for the tests
+# ------------------------------------------------------------------------------------------
+def moe(experts=6, top=3, ff=40, limit=1.5, shared=56, shared_limit=0.8):
+    return {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff, "limit": limit},
+            "shared": {"ff": shared, "limit": shared_limit} if shared else None}
+
+
+def dense(ff=88):
+    return {"kind": "dense", "ff": ff}
+
+
+def delta_layer(heads=4, kv_heads=2, dim=24, vdim=40, conv=4, mlp="moe", ranks=(20, 12)):
+    """``ranks``: widths inside the matrix pairs of the decays and of the gate; a checkpoint's tensors have them, its configuration not."""
+    return {"type": "channel_delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv},
+            "mlp": moe() if mlp == "moe" else mlp, "_ranks": ranks}
+
+
+def pair_layer(heads=4, kv_heads=2, dim=32, vdim=24, size=50, scale=0.2, ssd=None, mlp="moe"):
+    right = dict(heads=6, groups=3, state=20, vdim=28, conv=3, norm_groups=4)
+    right.update(ssd or {})
+    return {"type": "parallel", "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": size}},
+                                          "right": right}, "mlp": moe() if mlp == "moe" else mlp}
+
+
+def config(layers, width=104, vocab=198, eps=1e-5, buckets=61, mul_prev=13, mul_cur=5):
+    return {"architecture": "Bazulorn", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers,
+            "embedding": {"bigram": {"buckets": buckets, "mul_prev": mul_prev, "mul_cur": mul_cur}}}
+
+
+def public(cfg):
+    """The configuration as a checkpoint holds it."""
+    return dict(cfg, layers=[{k: v for k, v in l.items() if k != "_ranks"} for l in cfg["layers"]])
+
+
+def tensors(cfg, seed=0):
+    """Seeded BF16 weights in which every mechanism counts."""
+    g = torch.Generator().manual_seed(seed)
+    W = cfg["width"]
+    t = {}
+    rn = lambda *s: torch.randn(*s, generator=g)
+    lin = lambda o, i, f=1.0: f * rn(o, i) / i ** 0.5
+    vec = lambda n, c=1.0, s=0.3: c + s * rn(n)
+
+    def ff(p, f):
+        t.update({p + "gate": lin(f, W, 1.5), p + "up": lin(f, W), p + "down": lin(W, f)})
+    t.update({"embed": rn(cfg["vocab"], W), "bigram": rn(cfg["embedding"]["bigram"]["buckets"] + 1, W), "embed.norm": vec(W), "final.norm": vec(W)})
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.mix.", layer["mixer"]
+        t[f"l{i}.norm1"] = vec(W)
+        if layer["type"] == "channel_delta":
+            ra, rg = layer["_ranks"]
+            qk, v, k = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"], m["heads"] * m["dim"]
+            for n, rows in (("q", qk), ("k", qk), ("v", v)):
+                t.update({p + n: lin(rows, W), p + n + ".conv": 0.5 * rn(rows, m["conv"])})
+            t.update({p + "b": lin(m["heads"], W), p + "A_log": vec(m["heads"], -1.5, 1.5), p + "norm": vec(m["vdim"]), p + "a1": lin(ra, W),
+                      p + "a2": lin(k, ra), p + "dt_bias": vec(k, -2.0, 1.0), p + "g1": lin(rg, W), p + "g2": lin(v, rg), p + "o": lin(W, v)})
+        else:
+            a, r = m["left"], m["right"]
+            for n, rows in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])):
+                t.update({p + f"left.{n}": lin(rows, W), p + f"left.{n}.b": 0.3 * rn(rows)})
+            o, inner, maps = a["heads"] * a["vdim"], r["heads"] * r["vdim"], r["groups"] * r["state"]
+            t.update({p + "left.talk": torch.eye(a["heads"]) + 0.4 * rn(a["heads"], a["heads"]), p + "left.o": lin(W, o), p + "left.out": vec(W)})
+            t.update({p + "right.in": lin(2 * inner + 2 * maps + r["heads"], W), p + "right.conv": 0.5 * rn(inner + 2 * maps, r["conv"]),
+                      p + "right.conv.b": 0.3 * rn(inner + 2 * maps), p + "right.dt_bias": vec(r["heads"], -2.0, 1.0),
+                      p + "right.A_log": vec(r["heads"], -1.5, 1.5), p + "right.D": vec(r["heads"]), p + "right.norm": vec(inner),
+                      p + "right.o": lin(W, inner), p + "right.out": vec(W)})
+        mlp, p = layer.get("mlp"), f"l{i}.mlp."
+        if mlp is not None and mlp["kind"] == "dense":
+            ff(p, mlp["ff"])
+        elif mlp is not None:
+            e = mlp["router"]["experts"]
+            t.update({p + "router": lin(e, W, 3.0), p + "router.b": rn(e)})
+            for j in range(e):
+                ff(p + f"e{j}.", mlp["expert"]["ff"])
+            if mlp.get("shared"):
+                ff(p + "shared.", mlp["shared"]["ff"])
+    return {n: x.to(torch.bfloat16) for n, x in t.items()}
