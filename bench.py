@@ -7,7 +7,7 @@ head_dim 128, SwiGLU 14336, vocab 128256, BF16, random-init N(0, 0.02) weights, 
 parallel over the N GPUs of one node. ``--config 3`` selects the Llama-3-70B shape (batch 32,
 prompt 4096). A step is one decode step of the whole batch.
 
-``--design duponex|rudorax|kabavik`` measures another model design beside its closest relative instead (``utils/designbench.py``).
+``--design duponex|rudorax|kabavik|bazulorn`` measures another model design beside its closest relative instead (``utils/designbench.py``).
 
 Three arms (``--impl``):
   * ``ours``      -- this framework's engine and kernels. Reports
@@ -76,7 +76,7 @@ def parse() -> argparse.Namespace:
     p.add_argument("--skip-e2e", action="store_true")
     p.add_argument("--skip-baseline", action="store_true")
     p.add_argument("--skip-extras", action="store_true", help="no TTFT run and no other batch sizes")
-    p.add_argument("--design", default=None, choices=["duponex", "rudorax", "kabavik"],
+    p.add_argument("--design", default=None, choices=["duponex", "rudorax", "kabavik", "bazulorn"],
                    help="instead of the headline benchmark: throughput and kernels of this design beside the closest model at equal size")
     p.add_argument("--device", default="cuda", choices=["cuda", "cpu"], help="cpu is for debugging the harness only")
     a = p.parse_args()

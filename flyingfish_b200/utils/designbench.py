@@ -1,11 +1,13 @@
-"""A design's throughput and kernels beside the closest other model at equal size (``bench.py --design duponex|rudorax|kabavik``).
+"""A design's throughput and kernels beside the closest other model at equal size (``bench.py --design duponex|rudorax|kabavik|bazulorn``).
 
 The closest model of a Rudorax shape is the Flint layout (QK-norm, windowed attention with sinks, routed and shared experts): same
 width, heads, window, experts and number of layers (Rudorax: layer runs); a memory layer's kernels are timed beside those of the
 gated delta net. The closest model of a Duponex shape is the Gemma layout (QK-norm, local attention in every layer, extra norms per
 sub-layer, operator-by-operator decode step): same width, heads and layers, a sliding window as long as the block, and a
 gated feed-forward of the width that makes the layers' weights equal. A Kabavik shape is measured beside the Gemma layout too, with a
-feed-forward that makes the mean weights of a layer equal; the kernels of its latent layers beside those of the DeepSeek layout.
+feed-forward that makes the mean weights of a layer equal; the kernels of its latent layers beside those of the DeepSeek layout. A
+Bazulorn shape is measured beside the Flint layout as well (same attention in every layer, same experts); its delta rule and its
+state space beside the gated delta net with as many state elements, its short convolution beside that net's.
 Prompts end inside a block, so both attentions see
 the same keys. Weights are random. Every kernel of the design is timed beside its like kernel on the same rows; a
 fraction of the roofline is algorithmic bytes (or FLOPs) over time over the measured peak, and ``distance`` is the ratio
@@ -19,20 +21,21 @@ import torch
 
 from .. import ops
 from ..config import ModelSpec, MoeSpec, Settings, named_shape
-from ..ops import gdn_ops, mla_ops, mlstm_ops, moe_cuda, moe_ops, residual_ops, stream_ops
+from ..ops import delta_ops, gdn_ops, mla_ops, mlstm_ops, moe_cuda, moe_ops, residual_ops, ssd_ops, stream_ops, talk_ops
 from .kbench import Flusher, peaks, time_op
 
 SIZES = {"duponex": ("duponex-2b-shape", "duponex-8b-shape"), "rudorax": ("rudorax-2k-shape", "rudorax-4k-shape"),
-         "kabavik": ("kabavik-2k-shape", "kabavik-4k-shape")}
+         "kabavik": ("kabavik-2k-shape", "kabavik-4k-shape"), "bazulorn": ("bazulorn-2k-shape", "bazulorn-4k-shape")}
 
 
 def closest_spec(spec: ModelSpec) -> ModelSpec:
     """Gemma-layout shape with the layer weights of a Duponex shape of equal layers or the mean layer weights of a Kabavik shape;
-    Flint-layout shape with the attention and experts of a Rudorax shape."""
+    Flint-layout shape with the attention and experts of a Rudorax or Bazulorn shape."""
     l = spec.layer_specs[0]
-    if spec.arch == "rudorax":
+    if spec.arch in ("rudorax", "bazulorn"):
+        l = next(x for x in spec.layer_specs if x.mixer == "attention")
         m = l.moe
-        return ModelSpec(name=spec.name.replace("rudorax", "flint-layout"), arch="flint", layers=spec.layers, hidden=spec.hidden, heads=l.heads,
+        return ModelSpec(name=spec.name.replace(spec.arch, "flint-layout"), arch="flint", layers=spec.layers, hidden=spec.hidden, heads=l.heads,
                          kv_heads=l.kv_heads, head_dim=l.dim, ffn=m.expert_ffn, vocab=spec.vocab, qk_norm=True, rms_eps=spec.rms_eps,
                          moe=MoeSpec(num_experts=m.num_experts, top_k=m.top_k, expert_ffn=m.expert_ffn, score="sigmoid", n_shared=1,
                                      shared_ffn=m.shared_ffn),
@@ -137,7 +140,8 @@ class _Pairs:
 def kernel_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> list[dict]:
     """One line per pair: the design's kernel and its like on ``rows`` rows (``rows`` <= 128: a decode step of that batch at
     context ``ctx``; more: prefill of rows / ctx prompts)."""
-    return {"duponex": _duponex_table, "rudorax": _rudorax_table, "kabavik": _kabavik_table}[spec.arch](spec, rows, ctx, iters, device)
+    return {"duponex": _duponex_table, "rudorax": _rudorax_table, "kabavik": _kabavik_table,
+            "bazulorn": _bazulorn_table}[spec.arch](spec, rows, ctx, iters, device)
 
 
 def _duponex_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> list[dict]:
@@ -458,6 +462,140 @@ def _kabavik_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> 
              lat.scale, lat.window, gate, res), add(expansion, ec(lat)), "queries to latents, attention, results out of latents",
              like_latent_attention,
              add(expansion, ec(unbound)))
+    if decode:
+        wv = rn(spec.vocab, W)
+        pair("logits, 32-bit", lambda: ops.linear(x, wv, out_dtype=f32), pair.gemm(spec.vocab, W, out_bytes=4), "logits", lambda: ops.linear(x, wv),
+             pair.gemm(spec.vocab, W))
+    ops.check_status()
+    return pair.lines
+
+
+def _bazulorn_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) -> list[dict]:
+    delta, both = (next(x for x in spec.layer_specs if x.mixer == k) for k in ("channel_delta", "attention"))
+    ssd, e = both.beside, both.moe
+    dev, bf, f32 = torch.device(device), torch.bfloat16, torch.float32
+    W, H, G, d, f = spec.hidden, both.heads, both.kv_heads, both.dim, e.expert_ffn
+    rn = lambda *s: torch.randn(*s, device=dev).to(bf)
+    fl = lambda *s: torch.randn(*s, device=dev)
+    i32 = lambda t: t.to(torch.int32)
+    decode = rows <= 128
+    batch = rows if decode else rows // ctx
+    pair = _Pairs(rows, iters, dev)
+    x = rn(rows, W)
+    starts, sl = i32(torch.arange(batch + 1, device=dev) * (rows // batch)), i32(torch.randperm(batch, device=dev))
+    # projections
+    nd, nb = delta.projection_cols, both.projection_cols
+    for name, n, k in (("delta projection", nd, W), ("projection of the pair, bias", nb, W), ("output projection", W, H * d)):
+        w, r, b = rn(n, k), x if k == W else rn(rows, k), rn(n) if "bias" in name else None
+        pair(name, lambda: ops.linear(r, w, bias=b), pair.gemm(n, k), "projection of that size", lambda: ops.linear(r, w), pair.gemm(n, k))
+    wr, low = rn(delta.heads * delta.dim, delta.decay_rank), rn(rows, delta.decay_rank)
+    n = wr.shape[0]
+    pair("decay logits, 32-bit", lambda: ops.linear(low, wr, out_dtype=f32), pair.gemm(n, delta.decay_rank, out_bytes=4), "projection of that size",
+         lambda: ops.linear(low, wr), pair.gemm(n, delta.decay_rank))
+    # convolutions
+    V = delta.heads
+    for name, l, unit in (("short convolution, unit factors", delta, 0.1), ("short convolution, bias", ssd, None)):
+        conv = delta_ops.ConvWeights(fl(l.conv, l.conv_pad), None if unit else fl(l.conv_pad), 2 * l.kv_heads, l.dim_pad, l.heads, l.vdim_pad)
+        ch, cs = l.conv_pad, delta_ops.ConvState(batch, conv, dev)
+        px, gw, hist = rn(rows, ch), rn(ch, 4), torch.zeros(batch, ch, 3, device=dev)
+        cost = (rows * ch * 4 + batch * ch * 24, 0)
+        pair(name, lambda: delta_ops.short_conv(px, conv, cs, starts, sl, rows // batch, unit_scale=unit), cost, "convolution of the gated delta net",
+             lambda: gdn_ops.conv_batched(px, gw, hist, starts, sl), cost)
+    del px, hist, cs
+    # recurrences against the gated delta net
+    def like_net(V):
+        q, k, v = (fl(rows, V, 128) for _ in range(3))
+        k = k / k.norm(dim=-1, keepdim=True)
+        beta, dec, gst = torch.rand(rows, V, device=dev), -torch.rand(rows, V, device=dev), torch.zeros(batch, V, 128, 128, device=dev)
+        run = gdn_ops.recurrent_slots if decode else gdn_ops.chunked_slots
+        flops = 4 * rows * V * 128 * 128 + (0 if decode else 2 * rows * 64 * V * 128 * 4)
+        return lambda: run(q, k, v, beta, dec, gst, starts, sl), (8 * batch * V * 128 * 128 + rows * V * 128 * 14, flops)
+    form = "recurrence" if decode else "chunked"
+    cx, unit, dz, db, o = rn(rows, delta.conv_pad), fl(rows, 2 * V).abs() * 0.01, fl(rows, V * 128), rn(rows, V), torch.empty(rows, V, 128, device=dev)
+    unit = torch.rsqrt((cx[:, : 2 * V * 128].float().view(rows, 2 * V, 128) ** 2).sum(-1) + 1e-6)
+    st, rate, dtb = delta_ops.DeltaState(batch, V, delta.kv_heads, 128, 128, dev), -torch.rand(V, device=dev), fl(V * 128) - 4.0
+    like, like_cost = like_net(V)
+    pair(f"delta rule by channel, {form}", lambda: delta_ops.delta_rule(cx, unit, dz, db, rate, dtb, st, starts, sl, o, rows // batch),
+         (8 * batch * V * 128 * 128 + rows * V * 128 * (3 * 2 + 4 + 4), like_cost[1]), f"gated delta net, {form}", like, like_cost)
+    gate, wn, z, qn, on = rn(rows, V * 128), fl(128), rn(rows, V * 128), rn(128), rn(rows * V, 128)
+    like_out = lambda: (ops.rmsnorm(on, qn, 1e-5).view(rows, -1).float() * torch.nn.functional.silu(z.float())).to(bf)
+    pair("head norm + output gate", lambda: delta_ops.head_out(o, gate, wn, 128, 1e-5), (rows * V * 128 * 8, 0), "head norm, output gate", like_out,
+         (rows * V * 128 * 8, 0))
+    del cx, dz, st, like
+    M, dk, dv = ssd.heads, ssd.dim_pad, ssd.vdim_pad
+    cx, steps, sb, sa, skip, o = rn(rows, ssd.conv_pad), rn(rows, M), fl(M) - 4.0, -torch.rand(M, device=dev), fl(M), torch.empty(rows, M, dv, device=dev)
+    st = ssd_ops.SsdState(batch, M, ssd.kv_heads, dk, dv, dev)
+    like, like_cost = like_net(M * dk * dv // (128 * 128))
+    flops = 4 * rows * M * dk * dv + (0 if decode else 2 * rows * 64 * M * (dk + dv))
+    pair(f"state space, {form}", lambda: ssd_ops.state_space(cx, steps, sb, sa, skip, st, starts, sl, o, rows // batch),
+         (8 * batch * M * dk * dv + rows * (2 * ssd.conv_pad + M * dv * 4), flops), f"gated delta net, {form}", like, like_cost)
+    sz, sw = rn(rows, M * dv), fl(M * dv)
+    pair("output gate + norm of groups", lambda: ssd_ops.gated_out(o, sz, sw, dv, ssd.norm_groups, 1e-5), (rows * M * dv * 8, 0), "head norm, output gate", like_out,
+         (rows * V * 128 * 8, 0))
+    del cx, st, like, o, sz, gate, z, on
+    # value norm + cache write, attention
+    pg = _Paged(batch, ctx, G, d, dev)
+    slots, pos = i32(torch.randperm(pg.k.shape[0] * 64, device=dev)[:rows]), i32(torch.arange(rows, device=dev)) % ctx
+    qkv = rn(rows, (H + 2 * G) * d)
+    pair("value norm + cache write", lambda: ops.head_norm_kv(qkv, slots, pg.k, pg.v, H, G, d, d, 1e-5, norm_qk=False, norm_v=True), (2 * rows * d * 4 * G, 0),
+         "rotation + cache write", lambda: ops.rope_kv_paged(qkv, pos, slots, pg.k, pg.v, H, G, d, 1e4), (2 * rows * d * (2 * H + 4 * G), 0))
+    talk, sinks, out = fl(H, H), fl(H), torch.empty(rows, H * d, dtype=bf, device=dev)
+    mine, plain = H * (4 * d + 2 * H), H * 4 * d
+    args = (H, G, both.scale, both.window, talk, True)
+    if decode:
+        byts, seen = 2 * rows * (2 * both.keys_seen(ctx) * G * d + 2 * H * d), rows * both.keys_seen(ctx)
+        pair("attention, window, mixed heads", lambda: talk_ops.talk_decode(qkv, pg.k, pg.v, pg.table, pg.ctx, ctx, *args, out=out), (byts, seen * mine),
+             "attention, window + sinks", lambda: ops.attn_decode(qkv, pg.k, pg.v, pg.table, pg.ctx, H, G, d, both.scale, max_ctx=ctx, window=both.window,
+             sinks=sinks), (byts, seen * plain))
+    else:
+        qs, ql = i32(torch.arange(batch, device=dev) * ctx), torch.full((batch,), ctx, dtype=torch.int32, device=dev)
+        byts, seen = 2 * rows * (2 * H * d + 2 * G * d), batch * both.pairs_seen(ctx)
+        pair("attention, window, mixed heads", lambda: talk_ops.talk_prefill(qkv, pg.k, pg.v, pg.table, qs, ql, pg.ctx, ctx, ctx, *args, out=out),
+             (byts, seen * mine), "attention, window + sinks", lambda: ops.attn_prefill(qkv, pg.k, pg.v, pg.table, qs, ql, pg.ctx, ctx, H, G, d, both.scale,
+             window=both.window, sinks=sinks), (byts, seen * plain))
+    del pg, qkv, out
+    # router, experts
+    wr, bias = rn((e.num_experts + 15) // 16 * 16, W) * 0.02, fl(e.num_experts) * 0.01
+    gu, down = rn(e.num_experts, 2 * f, W), rn(e.num_experts, W, f)
+    weights, ids = moe_ops.route(x, wr, e.top_k, e.score, bias, exact=True, experts=e.num_experts)
+    lw, lids = moe_ops.route(x, wr[: e.num_experts], e.top_k, "sigmoid")
+    holder = {}
+
+    def expert_cost(ids):
+        touched = int(torch.unique(ids).numel())
+        return (2 * (touched * 3 * f * W + ids.numel() * (2 * W + 3 * f)), 2 * ids.numel() * 3 * f * W)
+
+    def like_routed():
+        moe_ops.route(x, wr[: e.num_experts], e.top_k, "sigmoid")
+        xs, p, so, ct, cap = moe_cuda.dispatch_local(x, lids, e.num_experts, 0, e.num_experts)
+        rpe = rows * e.top_k / e.num_experts
+        h = moe_cuda.grouped_gemm(xs, gu, so, ct, cap, epi=1, rows_per_expert=rpe)
+        holder["y"], holder["pos"] = moe_cuda.grouped_gemm(h, down, so, ct, cap, epi=0, rows_per_expert=rpe), p
+    add = lambda p, q: (p[0] + q[0], p[1] + q[1])
+    pair("router, dispatch, two grouped GEMMs, clamped gate", lambda: moe_ops.routed_rows(x, wr, e.top_k, e.score, bias, e.num_experts, gu, down, e.limit),
+         add(expert_cost(ids), pair.gemm(e.num_experts, W, out_bytes=8)), "router, dispatch, two grouped GEMMs", like_routed,
+         add(expert_cost(lids), pair.gemm(e.num_experts, W, out_bytes=4)))
+    er = moe_ops.expert_rows(x, weights, ids, gu, down, e.limit)
+    like_routed()
+    sg, sd = rn(2 * e.shared_ffn, W), rn(W, e.shared_ffn)
+    cost = (2 * (3 * e.shared_ffn * W + rows * (2 * W + 2 * e.shared_ffn)), 6 * rows * e.shared_ffn * W)
+    pair("shared expert, clamped gate", lambda: ops.linear(ops.linear_swiglu(x, sg, mode=5, limit=e.shared_limit), sd), cost, "shared expert",
+         lambda: ops.linear(ops.silu_mul(ops.linear(x, sg)), sd), cost)
+    # the layer's end and its begin
+    xs, a, b, r, w1, w2, w3, w16, r16 = fl(rows, W), rn(rows, W), rn(rows, W), rn(rows, W), fl(W), fl(W), fl(W), rn(W), rn(rows, W)
+
+    def like_end():
+        y = moe_cuda.combine(holder["y"], holder["pos"], lids, lw, rows, W)
+        ops.add_rmsnorm(a, r16, w16, 1e-5)
+        ops.add_rmsnorm(moe_ops.add_shared(y, b), r16, w16, 1e-5)
+    pair("residual step (all sums, three norms)", lambda: residual_ops.step(xs, a, b, er, w1, None, 1e-5, W, beside=residual_ops.Beside(r, w2, w3)),
+         (rows * W * (8 + 2 + 6 + 2 * e.top_k), 0), "expert sum, shared sum, two add + norm", like_end, (rows * W * (2 * e.top_k + 2 * 6), 0))
+    tok, tab = i32(torch.randint(0, 1024, (rows,), device=dev)), rn(1024, W)
+    last = torch.full((batch,), -1, dtype=torch.int32, device=dev)
+    big = lambda: residual_ops.bigram_rows(tok, last, starts, sl, buckets=1023, mul_prev=31, mul_cur=3)
+    pair("bigram rows, embed of two tables + norms", lambda: residual_ops.embed(tok, tab, 1.0, w1, None, 1e-5, W, second=residual_ops.Second(tab, big(), w2)),
+         (rows * W * 10, 0), "embed + norm", lambda: ops.embed_rmsnorm(tok, tab, w16, 1e-5), (rows * W * 6, 0))
+    del gu, down, er, holder, xs
     if decode:
         wv = rn(spec.vocab, W)
         pair("logits, 32-bit", lambda: ops.linear(x, wv, out_dtype=f32), pair.gemm(spec.vocab, W, out_bytes=4), "logits", lambda: ops.linear(x, wv),

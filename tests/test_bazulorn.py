@@ -389,7 +389,9 @@ def test_whole_prompt_and_layers(base, device, dtype):
     path, w = base
     m = load(path, device, dtype)
     toks = ids(150)
+    O.MARGINS.clear()
     want, after = O.forward(CFG, w, toks)
+    assert min(O.MARGINS) > 0.1
     got, seq = feed_in_cuts(m.engine, toks, [150])
     agree(got, want, dtype, "logits")
     m.engine.free_sequence(seq.seq_id)
@@ -476,7 +478,8 @@ def plain_start(cfg, seed):
     w = O.tensors(cfg, seed=seed)
     w["bigram"].zero_()
     w["embed.norm"].fill_(1.0)
-    w["embed"][:, 0], w["embed"][:, 1] = 3.0, 0.0
+    w["embed"][:, :4] = 0.0
+    w["embed"][:, 0] = 3.0
     w["embed"][7, 1] = 9.0
     return w
 
@@ -612,9 +615,9 @@ def test_the_extra_term_and_the_mixing_matter(tmp_path, device, dtype, monkeypat
         m.setattr(O, "softmax_with_one", lambda s: torch.softmax(s, -1))
         assert relative_change(O.forward(cfg, w, toks)[0], want).median() > 0.02
     plain = {n: (torch.eye(4).to(torch.bfloat16) if n.endswith("talk") else t) for n, t in w.items()}
-    assert relative_change(O.forward(cfg, plain, toks)[0], want).min() > 0.1
+    assert relative_change(O.forward(cfg, plain, toks)[0], want).median() > 0.1
     turned = {n: (t.t().contiguous() if n.endswith("talk") else t) for n, t in w.items()}
-    assert relative_change(O.forward(cfg, turned, toks)[0], want).min() > 0.1
+    assert relative_change(O.forward(cfg, turned, toks)[0], want).median() > 0.1
     e = load(write(tmp_path, cfg, w), device, dtype).engine
     for cuts in ([60], [3, 40, 1]):
         got, seq = feed_in_cuts(e, toks, cuts)
@@ -650,19 +653,11 @@ def test_other_sizes(tmp_path, device, dtype, name):
     toks = ids(135, vocab=cfg["vocab"], seed=8)
     O.MARGINS.clear()
     want, _ = O.forward(cfg, w, toks)
-    sure = not O.MARGINS or min(O.MARGINS) > 0.05                 # no choice that rounding could turn
-    assert sure or dtype == "fp32" or name in UNSURE
+    assert not O.MARGINS or min(O.MARGINS) > 0.1                  # no choice that rounding could turn
     for cuts in ([135], [70, 1, 1, 2, 50, 1]):
         got, seq = feed_in_cuts(e, toks, cuts)
         e.free_sequence(seq.seq_id)
-        if sure or dtype == "fp32":
-            agree(got, want, dtype, f"{name} {cuts}")
-        else:
-            err = relative_change(got.double(), want)
-            assert err.median() < MODEL_LIMIT[dtype] and torch.isfinite(got).all(), name
-
-
-UNSURE: set[str] = set()
+        agree(got, want, dtype, f"{name} {cuts}")
 
 
 @each_form
