@@ -384,14 +384,6 @@ struct PrefillForm {
 // warp are at most 1 -- the usual case, caps being there for outliers -- tanh is a polynomial, two values per instruction, which
 // leaves the special-function unit to the soft-max: y times a Chebyshev fit of tanh(y) / y in y^2 on [0, 1], error 5.5e-7.
 // Otherwise 1 - 2 / (1 + e^(2y)).
-__device__ __forceinline__ uint64_t f2_pack(float a, float b) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
-__device__ __forceinline__ void f2_unpack(uint64_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
-__device__ __forceinline__ uint64_t f2_mul(uint64_t a, uint64_t b) { uint64_t r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
-__device__ __forceinline__ uint64_t f2_fma(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
 template <int N>
 __device__ __forceinline__ void cap_scores(float (&sv)[N], float cap_in) {
   float am[4] = {0.f, 0.f, 0.f, 0.f};

@@ -4,8 +4,8 @@
 // The mixed weights of a head need the normalised weights of every head, so no head can run its soft-max and its value product in one
 // pass. Prompts take three, over tiles of 128 query rows:
 //   1. talk_weights : scores on tcgen05 as in attention_tc.cu, 64 keys at a time; 2^(s - m) in FP16 goes to scratch by TMA, m being the
-//                     maximum a thread has seen so far (two threads share a row, 32 keys each), and with it m of every step and z at
-//                     the end;
+//                     maximum a thread has seen so far (two threads share a row, every other page each), and with it m of every 32
+//                     keys and z at the end;
 //   2. talk_mix     : a warp takes a query row, 64 keys of all heads at a time: the weights times 2^(m - z), then their product with the
 //                     mixing matrix (mma.sync, heads as its inner dimension); mixed weights in BF16 replace the others in scratch;
 //   3. talk_values  : scratch times values on tcgen05, two heads that share a value head per CTA.
@@ -76,149 +76,195 @@ __device__ __forceinline__ void talk_frag(const float* talk, int H, int row0, in
 }
 
 // ---------------------------------------------------------------------------------------
-// talk_weights: grid (tiles, H, sequences), 320 threads: TMA warp, MMA warp, eight warps whose threads own 32 keys of a row each. Shared
-// memory: Q (two blocks of 64 columns), two K tiles, two staging tiles of 32 rows and 32 keys per such warp. Tensor memory: two score tiles of 64 columns.
+// talk_weights: as many CTAs as fit, each takes every so many-th (sequence, tile, head). 320 threads: TMA warp, MMA warp, and two times
+// four warps whose threads own a row of the even or of the odd pages. Shared memory: Q (two blocks of 64 columns), two K tiles, a staging
+// tile of 32 rows and 64 keys per such warp. Tensor memory: four score tiles of 64 columns.
 // ---------------------------------------------------------------------------------------
-constexpr int TW_Q = TK_ROWS * 128 * 2, TW_K = TK_PAGE * 128 * 2, TW_P = 32 * 32 * 2;
-constexpr int TW_SMEM = TW_Q + 2 * TW_K + 16 * TW_P + 1024;
+constexpr int TW_Q = TK_ROWS * 128 * 2, TW_K = TK_PAGE * 128 * 2, TW_P = 32 * TK_PAGE * 2;
+constexpr int TW_SMEM = TW_Q + 2 * TW_K + 8 * TW_P + 1024;
 
 struct alignas(8) TalkWeightBars {
-  uint64_t q_full, k_full[2], k_empty[2], s_full[2], s_empty[2];
+  uint64_t q_full, q_empty, k_full[2], k_empty[2], s_full[4], s_empty[4];
   uint32_t tmem_base;
   int abort_flag;
-  float m[TK_ROWS], l[TK_ROWS];
+  float m[2][TK_ROWS], l[2][TK_ROWS];        // of the odd pages; two, so that a head's do not meet the next one's
+};
+
+// (sequence, tile of the round, head) number i
+struct TalkItem {
+  int b, tile, h;
+  __device__ TalkItem(const TalkArgs& p, int i) { h = i % p.H; i /= p.H; tile = i % p.tiles; b = i / p.tiles; }
 };
 
 __global__ void __launch_bounds__(320, 2)
 talk_weights_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmP,
-                    const TalkArgs p) {
+                    const TalkArgs p, int items) {
   pdl_wait();
-  const int b = blockIdx.z, h = blockIdx.y, tile = p.tile0 + blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const TalkTile tl(p, b, tile);
-  if (tl.real <= 0) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   extern __shared__ uint8_t tk_raw[];
   __shared__ TalkWeightBars bars;
   uint8_t* sQ = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tk_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sK = sQ + TW_Q;
   uint8_t* sP = sK + 2 * TW_K;
   const bool hi = p.dk > 64;
-  const size_t slot_head = ((size_t)b * p.tiles + blockIdx.x) * p.H + h;
   if (threadIdx.x == 0) {
     tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmP);
-    mbar_init(&bars.q_full, 1);
-    for (int i = 0; i < 2; ++i) { mbar_init(&bars.k_full[i], 1); mbar_init(&bars.k_empty[i], 1); mbar_init(&bars.s_full[i], 1); mbar_init(&bars.s_empty[i], 8); }
+    mbar_init(&bars.q_full, 1); mbar_init(&bars.q_empty, 1);
+    for (int i = 0; i < 2; ++i) { mbar_init(&bars.k_full[i], 1); mbar_init(&bars.k_empty[i], 1); }
+    for (int i = 0; i < 4; ++i) { mbar_init(&bars.s_full[i], 1); mbar_init(&bars.s_empty[i], 4); }
     bars.abort_flag = 0;
     mbar_fence_init();
   }
-  if (warp == 1) { tmem_alloc(&bars.tmem_base, 128); tmem_relinquish(); }
+  if (warp == 1) { tmem_alloc(&bars.tmem_base, 256); tmem_relinquish(); }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_s = bars.tmem_base;
   volatile int* abort_flag = &bars.abort_flag;
+  int c = 0, n = 0;                                          // pages and items so far
   if (warp == 0) {
     if (lane == 0) {
-      const int row = p.q_start[b] + tile * TK_ROWS;
-      mbar_expect_tx(&bars.q_full, hi ? TW_Q : TW_Q / 2);
-      tma_load_2d(sQ, &tmQ, &bars.q_full, h * p.dk, row);
-      if (hi) tma_load_2d(sQ + TW_Q / 2, &tmQ, &bars.q_full, h * p.dk + 64, row);
-      bool bad = false;
-      for (int j = 0; j < tl.pages; ++j) {
-        const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
-        const int krow = (talk_page(p, b, tl.lo_page + j, bad) * p.G + h / (p.H / p.G)) * TK_PAGE;
-        if (!mbar_wait(&bars.k_empty[st], ph ^ 1, abort_flag, p.status, KID_ATTN_PREFILL, 41)) break;
-        mbar_expect_tx(&bars.k_full[st], hi ? TW_K : TW_K / 2);
-        tma_load_2d(sK + st * TW_K, &tmK, &bars.k_full[st], 0, krow);
-        if (hi) tma_load_2d(sK + st * TW_K + TW_K / 2, &tmK, &bars.k_full[st], 64, krow);
+      bool ok = true;
+      for (int i = blockIdx.x; i < items && ok; i += gridDim.x) {
+        const TalkItem it(p, i);
+        const TalkTile tl(p, it.b, p.tile0 + it.tile);
+        if (tl.real <= 0) continue;
+        const int row = p.q_start[it.b] + (p.tile0 + it.tile) * TK_ROWS;
+        if (!mbar_wait(&bars.q_empty, (n & 1) ^ 1, abort_flag, p.status, KID_ATTN_PREFILL, 40)) break;
+        mbar_expect_tx(&bars.q_full, hi ? TW_Q : TW_Q / 2);
+        tma_load_2d(sQ, &tmQ, &bars.q_full, it.h * p.dk, row);
+        if (hi) tma_load_2d(sQ + TW_Q / 2, &tmQ, &bars.q_full, it.h * p.dk + 64, row);
+        bool bad = false;
+        for (int j = 0; j < tl.pages; ++j, ++c) {
+          const int st = c & 1;
+          const int krow = (talk_page(p, it.b, tl.lo_page + j, bad) * p.G + it.h / (p.H / p.G)) * TK_PAGE;
+          ok = mbar_wait(&bars.k_empty[st], ((c >> 1) & 1) ^ 1, abort_flag, p.status, KID_ATTN_PREFILL, 41);
+          if (!ok) break;
+          mbar_expect_tx(&bars.k_full[st], hi ? TW_K : TW_K / 2);
+          tma_load_2d(sK + st * TW_K, &tmK, &bars.k_full[st], 0, krow);
+          if (hi) tma_load_2d(sK + st * TW_K + TW_K / 2, &tmK, &bars.k_full[st], 64, krow);
+        }
+        if (bad) set_status(p.status, KID_ATTN_PREFILL, FF_ERR_BOUNDS, it.b, p.tile0 + it.tile);
+        ++n;
       }
-      if (bad) set_status(p.status, KID_ATTN_PREFILL, FF_ERR_BOUNDS, b, tile);
     }
   } else if (warp == 1) {
     if (lane == 0) {
       const uint32_t idesc = umma_idesc(1, 1, 0, 0, TK_ROWS, TK_PAGE), q_addr = smem_u32(sQ);
       const int ksteps = p.dk >> 4;
-      bool ok = mbar_wait(&bars.q_full, 0, abort_flag, p.status, KID_ATTN_PREFILL, 42);
-      for (int j = 0; j < tl.pages && ok; ++j) {
-        const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
-        if (!mbar_wait(&bars.k_full[st], ph, abort_flag, p.status, KID_ATTN_PREFILL, 43)) break;
-        if (!mbar_wait(&bars.s_empty[st], ph ^ 1, abort_flag, p.status, KID_ATTN_PREFILL, 44)) break;
-        tc_fence_after();
-        const uint32_t k_addr = smem_u32(sK + st * TW_K);
+      bool ok = true;
+      for (int i = blockIdx.x; i < items && ok; i += gridDim.x) {
+        const TalkItem it(p, i);
+        const TalkTile tl(p, it.b, p.tile0 + it.tile);
+        if (tl.real <= 0) continue;
+        ok = mbar_wait(&bars.q_full, n & 1, abort_flag, p.status, KID_ATTN_PREFILL, 42);
+        for (int j = 0; j < tl.pages && ok; ++j, ++c) {
+          const int st = c & 1, sb = c & 3;
+          ok = mbar_wait(&bars.k_full[st], (c >> 1) & 1, abort_flag, p.status, KID_ATTN_PREFILL, 43) &&
+               mbar_wait(&bars.s_empty[sb], ((c >> 2) & 1) ^ 1, abort_flag, p.status, KID_ATTN_PREFILL, 44);
+          if (!ok) break;
+          tc_fence_after();
+          const uint32_t k_addr = smem_u32(sK + st * TW_K);
 #pragma unroll
-        for (int k = 0; k < 8; ++k) {
-          if (k >= ksteps) break;
-          umma_f16(tmem_s + st * TK_PAGE, umma_desc_sw128(q_addr + (k >> 2) * (TW_Q / 2) + (k & 3) * 32, 16, 1024),
-                   umma_desc_sw128(k_addr + (k >> 2) * (TW_K / 2) + (k & 3) * 32, 16, 1024), idesc, k != 0);
+          for (int k = 0; k < 8; ++k) {
+            if (k >= ksteps) break;
+            umma_f16(tmem_s + sb * TK_PAGE, umma_desc_sw128(q_addr + (k >> 2) * (TW_Q / 2) + (k & 3) * 32, 16, 1024),
+                     umma_desc_sw128(k_addr + (k >> 2) * (TW_K / 2) + (k & 3) * 32, 16, 1024), idesc, k != 0);
+          }
+          umma_commit(&bars.s_full[sb]);
+          umma_commit(&bars.k_empty[st]);
         }
-        umma_commit(&bars.s_full[st]);
-        umma_commit(&bars.k_empty[st]);
+        if (ok) umma_commit(&bars.q_empty);
+        ++n;
       }
     }
   } else {
-    const int q = warp & 3, half = (warp - 2) >> 2, row = q * 32 + lane, pos = tl.first + row;
-    const bool live = row < tl.real;
-    const int last = live ? pos : -1, from = live ? max(0, pos - p.window + 1) : 0;
-    const int all_lo = max(0, tl.first + tl.real - p.window), all_hi = tl.real == TK_ROWS ? tl.first : -1;     // keys every row sees
-    uint8_t* stg = sP + (q * 2 + half) * 2 * TW_P;
-    float m = -INFINITY, l = 0.f;
+    const int q = warp & 3, odd = (warp - 2) >> 2, row = q * 32 + lane;
+    uint8_t* stg = sP + (q * 2 + odd) * TW_P;
+    const uint64_t scale2 = f2_pack(p.scale_log2, p.scale_log2);
     bool ok = true;
-    for (int j = 0; j < tl.pages; ++j) {
-      const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
-      if (!mbar_wait(&bars.s_full[st], ph, abort_flag, p.status, KID_ATTN_PREFILL, 45)) ok = false;
-      ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
-      tc_fence_after();
-      float sv[32];
-      {
-        uint32_t r[32];
-        tmem_ld_x32(tmem_s + (uint32_t(q * 32) << 16) + st * TK_PAGE + 32 * half, r);
-        tmem_ld_wait();
+    for (int i = blockIdx.x; i < items; i += gridDim.x) {
+      const TalkItem it(p, i);
+      const TalkTile tl(p, it.b, p.tile0 + it.tile);
+      if (tl.real <= 0) continue;
+      const size_t slot_head = ((size_t)it.b * p.tiles + it.tile) * p.H + it.h;
+      const int pos = tl.first + row;
+      const bool live = row < tl.real;
+      const int last = live ? pos : -1, from = live ? max(0, pos - p.window + 1) : 0;
+      const int all_lo = max(0, tl.first + tl.real - p.window), all_hi = tl.real == TK_ROWS ? tl.first : -1;     // keys every row sees
+      float m = -INFINITY, l = 0.f;
+      for (int j = odd; j < tl.pages && ok; j += 2) {
+        const int sb = (c + j) & 3;
+        if (!mbar_wait(&bars.s_full[sb], ((c + j) >> 2) & 1, abort_flag, p.status, KID_ATTN_PREFILL, 45)) ok = false;
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        tc_fence_after();
+#pragma unroll 1
+        for (int half = 0; half < 2; ++half) {
+          float sv[32];
+          {
+            uint32_t r[32];
+            tmem_ld_x32(tmem_s + (uint32_t(q * 32) << 16) + sb * TK_PAGE + 32 * half, r);
+            tmem_ld_wait();
 #pragma unroll
-        for (int i = 0; i < 32; ++i) sv[i] = __uint_as_float(r[i]);
-      }
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&bars.s_empty[st]);
-      const int k0 = (tl.lo_page + j) * TK_PAGE + 32 * half;
-      float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      if (!(k0 >= all_lo && k0 + 31 <= all_hi)) {
+            for (int e = 0; e < 32; ++e) sv[e] = __uint_as_float(r[e]);
+          }
+          if (half == 1) {
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&bars.s_empty[sb]);
+          }
+          const int k0 = (tl.lo_page + j) * TK_PAGE + 32 * half;
+          float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+          if (!(k0 >= all_lo && k0 + 31 <= all_hi)) {
 #pragma unroll
-        for (int i = 0; i < 32; ++i) sv[i] = k0 + i >= from && k0 + i <= last ? sv[i] : -INFINITY;
-      }
+            for (int e = 0; e < 32; ++e) sv[e] = k0 + e >= from && k0 + e <= last ? sv[e] : -INFINITY;
+          }
 #pragma unroll
-      for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], sv[i]);
-      const float mn = fmaxf(m, fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2), mr = mn == -INFINITY ? 0.f : mn;
-      l *= m == -INFINITY ? 0.f : tk_ex2(m - mr);
-      m = mn;
-      p.m[((slot_head * p.band + j) * 2 + half) * TK_ROWS + row] = m;
-      if (lane == 0) tma_store_wait_read<1>();             // the staging tile's previous contents have left
-      __syncwarp();
-      uint8_t* at = stg + st * TW_P + lane * 64;
-      float ls[4] = {0.f, 0.f, 0.f, 0.f};
+          for (int e = 0; e < 32; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], sv[e]);
+          const float mn = fmaxf(m, fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2), mr = mn == -INFINITY ? 0.f : mn;
+          l *= m == -INFINITY ? 0.f : tk_ex2(m - mr);
+          m = mn;
+          p.m[((slot_head * p.band + j) * 2 + half) * TK_ROWS + row] = m;
+          if (half == 0) {
+            if (lane == 0) tma_store_wait_read<0>();         // the staging tile's previous contents have left
+            __syncwarp();
+          }
+          const uint64_t neg = f2_pack(-mr, -mr);
+          uint64_t ls[2] = {0ull, 0ull};
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        uint32_t w[4];
+          for (int e = 0; e < 4; ++e) {
+            uint32_t w[4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float x = tk_ex2(fmaf(sv[8 * c + 2 * i], p.scale_log2, -mr)), y = tk_ex2(fmaf(sv[8 * c + 2 * i + 1], p.scale_log2, -mr));
-          ls[i] += x + y;
-          w[i] = pack_half2(x, y);
+            for (int k = 0; k < 4; ++k) {
+              float x, y;
+              f2_unpack(f2_fma(f2_pack(sv[8 * e + 2 * k], sv[8 * e + 2 * k + 1]), scale2, neg), x, y);
+              x = tk_ex2(x);
+              y = tk_ex2(y);
+              ls[k & 1] = f2_add(ls[k & 1], f2_pack(x, y));
+              w[k] = pack_half2(x, y);
+            }
+            *reinterpret_cast<uint4*>(stg + lane * 128 + (((4 * half + e) ^ (lane & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+          }
+          float la, lb;
+          f2_unpack(f2_add(ls[0], ls[1]), la, lb);
+          l += la + lb;
         }
-        *reinterpret_cast<uint4*>(at + ((c ^ ((lane >> 1) & 3)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);      // 64-byte swizzle
+        fence_proxy_async_smem();
+        __syncwarp();
+        if (lane == 0) {
+          tma_store_2d(&tmP, stg, j * TK_PAGE, (int)(slot_head * TK_ROWS) + q * 32);
+          tma_store_commit();
+        }
       }
-      l += (ls[0] + ls[1]) + (ls[2] + ls[3]);
-      fence_proxy_async_smem();
-      __syncwarp();
-      if (lane == 0) {
-        tma_store_2d(&tmP, stg + st * TW_P, j * TK_PAGE + 32 * half, (int)(slot_head * TK_ROWS) + q * 32);
-        tma_store_commit();
+      if (odd) { bars.m[n & 1][row] = m; bars.l[n & 1][row] = l; }
+      asm volatile("bar.sync 1, 256;" ::: "memory");
+      if (!odd) {
+        const float om = bars.m[n & 1][row], mx = fmaxf(fmaxf(m, om), p.one > 0.f ? 0.f : -INFINITY);
+        p.z[slot_head * TK_ROWS + row] = mx == -INFINITY ? 0.f : mx + log2f(l * tk_ex2(m - mx) + bars.l[n & 1][row] * tk_ex2(om - mx) + (p.one > 0.f ? p.one * tk_ex2(-mx) : 0.f));
       }
-    }
-    if (half == 1) { bars.m[row] = m; bars.l[row] = l; }
-    asm volatile("bar.sync 1, 256;" ::: "memory");
-    if (half == 0) {
-      const float om = bars.m[row], n = fmaxf(fmaxf(m, om), p.one > 0.f ? 0.f : -INFINITY);
-      p.z[slot_head * TK_ROWS + row] = n == -INFINITY ? 0.f : n + log2f(l * tk_ex2(m - n) + bars.l[row] * tk_ex2(om - n) + (p.one > 0.f ? p.one * tk_ex2(-n) : 0.f));
+      c += tl.pages;
+      ++n;
     }
     if (lane == 0) tma_store_wait<0>();
   }
@@ -228,12 +274,12 @@ talk_weights_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     const uint64_t t0 = globaltimer_ns();
     while (globaltimer_ns() - t0 < 200000ull) { __nanosleep(1000); }
   }
-  if (warp == 1) { __syncwarp(); tc_fence_after(); tmem_dealloc(tmem_s, 128); }
+  if (warp == 1) { __syncwarp(); tc_fence_after(); tmem_dealloc(tmem_s, 256); }
 }
 
 // ---------------------------------------------------------------------------------------
 // talk_mix: grid (16 * tiles, parts, sequences), 256 threads: eight neighbouring rows, a warp each, 64 keys of all heads at a time by TMA
-// (one box of H rows of 128 bytes), three tiles per warp: one on its way in, one being worked on, one on its way out. HB: blocks of 16
+// (one box of H rows of 128 bytes), three tiles per warp: two on their way in and one being worked on, which then is on its way out. HB: blocks of 16
 // heads.
 // ---------------------------------------------------------------------------------------
 constexpr int TM_STAGES = 3;
@@ -279,17 +325,27 @@ talk_mix_kernel(const __grid_constant__ CUtensorMap tmM, const TalkArgs p) {
       asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(buf + st * TB + ms_off(i >> 3, i & 7, 8)), "r"(0) : "memory");
   __syncwarp();
   const bool live = warp < rows;
-  if (live && lane == 0) {
-    mbar_expect_tx(&full[0], H * 128);
-    talk_load_row(buf, &tmM, &full[0], j0 * TK_PAGE, row0 + warp, slot);
-  }
+  if (live && lane == 0)
+    for (int k = 0; k < min(n, 2); ++k) {
+      mbar_expect_tx(&full[k], H * 128);
+      talk_load_row(buf + k * TB, &tmM, &full[k], (j0 + k) * TK_PAGE, row0 + warp, slot);
+    }
   // the factors 2^(m - z) of all steps: a thread takes a row and heads tid / 8, + 32
   for (int h = tid >> 3; h < HB * 16; h += 32) {
     const int r = tid & 7;
     const size_t sh = (size_t)slot * H + min(h, H - 1);
     const float z = p.z[sh * TK_ROWS + row0 + r];
     const float* mp = p.m + (sh * p.band + j0) * 2 * TK_ROWS + row0 + r;
-    for (int k = 0; k < 2 * n; ++k) s_f[((k >> 1) * 16 + 2 * r + (k & 1)) * HB * 16 + h] = __float2half(h < H ? tk_ex2(mp[(size_t)k * TK_ROWS] - z) : 0.f);
+    for (int k0 = 0; k0 < 2 * n; k0 += 8) {                // eight loads on their way together
+      float m[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) m[e] = mp[(size_t)min(k0 + e, 2 * n - 1) * TK_ROWS];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const int k = k0 + e;
+        if (k < 2 * n) s_f[((k >> 1) * 16 + 2 * r + (k & 1)) * HB * 16 + h] = __float2half(h < H ? tk_ex2(m[e] - z) : 0.f);
+      }
+    }
   }
   uint32_t tf[HB][HB][4];
 #pragma unroll
@@ -301,12 +357,6 @@ talk_mix_kernel(const __grid_constant__ CUtensorMap tmM, const TalkArgs p) {
   const int r16 = (lane & 7) + (((lane >> 3) & 1) << 3);
   int st = 0; uint32_t ph = 0;
   for (int k = 0; k < n; ++k) {
-    const int nx = st + 1 == TM_STAGES ? 0 : st + 1;
-    if (lane == 0 && k + 1 < n) {
-      tma_store_wait_read<1>();                            // the tile that left from there
-      mbar_expect_tx(&full[nx], H * 128);
-      talk_load_row(buf + nx * TB, &tmM, &full[nx], (j0 + k + 1) * TK_PAGE, row0 + warp, slot);
-    }
     if (!mbar_wait(&full[st], ph, nullptr, p.status, KID_ATTN_PREFILL, 61)) break;
     __syncwarp();
     const uint32_t d = buf + st * TB;
@@ -344,11 +394,16 @@ talk_mix_kernel(const __grid_constant__ CUtensorMap tmM, const TalkArgs p) {
     fence_proxy_async_smem();
     __syncwarp();
     if (lane == 0) {
+      if (k + 2 < n) {
+        const int free = st == 0 ? TM_STAGES - 1 : st - 1;
+        tma_store_wait_read<0>();                          // the tile that left from there
+        mbar_expect_tx(&full[free], H * 128);
+        talk_load_row(buf + free * TB, &tmM, &full[free], (j0 + k + 2) * TK_PAGE, row0 + warp, slot);
+      }
       talk_store_row(&tmM, d, (j0 + k) * TK_PAGE, row0 + warp, slot);
       tma_store_commit();
     }
-    st = nx;
-    if (st == 0) ph ^= 1;
+    if (++st == TM_STAGES) { st = 0; ph ^= 1; }
   }
   if (lane == 0) tma_store_wait<0>();
 }
@@ -678,17 +733,6 @@ talk_merge_kernel(const TalkDecodeArgs p) {
   p.out[(size_t)b * p.ldo + i] = __float2bfloat16(v);
 }
 
-// boxes of 32 keys and 32 rows, 64-byte swizzle
-static int talk_store_map(CUtensorMap* out, void* base, uint64_t inner, uint64_t outer) {
-  EncodeTiledFn fn = encode_tiled_fn();
-  if (!fn) return FF_HOST_NO_DRIVER;
-  const cuuint64_t dims[2] = {inner, outer}, strides[1] = {inner * 2};
-  const cuuint32_t box[2] = {32, 32}, step[2] = {1, 1};
-  const CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, base, dims, strides, box, step, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_64B,
-                        CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? FF_HOST_OK : FF_HOST_TMAP_FAIL;
-}
-
 // weights as (key, row, head, slot), boxes of 64 keys of all heads
 static int talk_row_map(CUtensorMap* out, void* base, uint64_t bandw, uint64_t heads, uint64_t slots) {
   EncodeTiledFn fn = encode_tiled_fn();
@@ -704,7 +748,7 @@ template <int HB>
 static int talk_mix_launch(const CUtensorMap& tmM, const TalkArgs& p, int batch, cudaStream_t s) {
   // CTAs that share a row's keys: enough for the device, and few enough steps each for the factors
   const int groups = batch * p.tiles * (TK_ROWS / 8), fit = 2 * sm_count(), most = HB == 1 ? 32 : 16;
-  int parts = groups < fit ? (fit + groups - 1) / groups : 1;
+  int parts = groups < fit ? fit / groups : 1;
   if (parts < (p.band + most - 1) / most) parts = (p.band + most - 1) / most;
   const int steps = (p.band + parts - 1) / parts, smem = 8 * TM_STAGES * HB * 16 * 128 + steps * 16 * HB * 16 * 2 + 1024;
   if (parts > 65535) return FF_HOST_TOO_LARGE;
@@ -741,7 +785,7 @@ FF_EXPORT int ff_talk_prefill(const void* q, const void* kcache, const void* vca
   if (int r = make_tmap_2d(&tmQ, q, BF, 2, (uint64_t)ldq, total_rows, (uint64_t)ldq * 2, 64, TK_ROWS)) return r;
   if (int r = make_tmap_2d(&tmK, kcache, BF, 2, dk, cache_rows, (uint64_t)dk * 2, 64, TK_PAGE)) return r;
   if (int r = make_tmap_2d(&tmV, vcache, BF, 2, dv, cache_rows, (uint64_t)dv * 2, 64, TK_PAGE)) return r;
-  if (int r = talk_store_map(&tmP, scratch, bandw, rows)) return r;
+  if (int r = make_tmap_2d(&tmP, scratch, BF, 2, bandw, rows, bandw * 2, 64, 32)) return r;
   if (int r = make_tmap_2d(&tmW, scratch, BF, 2, bandw, rows, bandw * 2, 64, TK_ROWS)) return r;
   if (int r = talk_row_map(&tmM, scratch, bandw, H, (uint64_t)batch * tiles_per_round)) return r;
   if (int r = opt_in_smem(talk_weights_kernel, TW_SMEM)) return r;
@@ -750,7 +794,8 @@ FF_EXPORT int ff_talk_prefill(const void* q, const void* kcache, const void* vca
   for (int t0 = first_round * tiles_per_round; t0 < tiles; t0 += round_step * tiles_per_round) {
     const TalkArgs p = {block_table, q_start, q_lens, ctx_lens, talk, (__nv_bfloat16*)out, (__nv_bfloat16*)scratch, m, m + 2 * rows * band, H, G, dk, dv, ldo,
                         max_blocks, num_blocks, window, band, t0, tiles - t0 < tiles_per_round ? tiles - t0 : tiles_per_round, scale * TK_LOG2E, one, status};
-    if (int r = launch_pdl(talk_weights_kernel, dim3(p.tiles, H, batch), dim3(320), TW_SMEM, s, 0, tmQ, tmK, tmP, p)) return r;
+    const int items = batch * p.tiles * H, fit = 2 * sm_count();
+    if (int r = launch_pdl(talk_weights_kernel, dim3(items < fit ? items : fit), dim3(320), TW_SMEM, s, 0, tmQ, tmK, tmP, p, items)) return r;
     if (int r = H <= 16 ? talk_mix_launch<1>(tmM, p, batch, s) : talk_mix_launch<2>(tmM, p, batch, s)) return r;
     if (int r = H / G >= 2 ? talk_values_launch<2>(tmW, tmV, p, batch, s) : talk_values_launch<1>(tmW, tmV, p, batch, s)) return r;
   }

@@ -15,7 +15,7 @@ from .lib import check, kernels, ptr, status_tensor, stream_ptr
 
 PAGE = 64
 ROWS = 128                    # query rows of a tile of the prompt kernels
-ROUND_BYTES = 100 << 20       # prompts: scratch of a round
+ROUND_BYTES = 160 << 20       # prompts: scratch of a round
 DECODE_CTAS = 592             # decode: CTAs a launch should have
 DECODE_SPLITS = 32
 _lanes: dict[int, SideLane] = {}
@@ -85,6 +85,7 @@ def talk_prefill(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, bl
     rows, batch = q.shape[0], block_table.shape[0]
     band, tiles = _band(max_ctx, window, ROWS), -(-max_q_len // ROWS)
     rounds = -(-tiles // max(1, ROUND_BYTES // (batch * hq * ROWS * band * PAGE * 2)))
+    rounds += rounds > 1 and rounds % 2    # two streams share them
     per_round = -(-tiles // rounds)
     floats = batch * per_round * hq * ROWS * (band * (PAGE // 2 + 2) + 1)
 
