@@ -592,7 +592,7 @@ def _bazulorn_table(spec: ModelSpec, rows: int, ctx: int, iters: int, device) ->
          (rows * W * (8 + 2 + 6 + 2 * e.top_k), 0), "expert sum, shared sum, two add + norm", like_end, (rows * W * (2 * e.top_k + 2 * 6), 0))
     tok, tab = i32(torch.randint(0, 1024, (rows,), device=dev)), rn(1024, W)
     last = torch.full((batch,), -1, dtype=torch.int32, device=dev)
-    big = lambda: residual_ops.bigram_rows(tok, last, starts, sl, buckets=1023, mul_prev=31, mul_cur=3)
+    big = lambda: residual_ops.bigram_rows(tok, last, starts, sl, buckets=1021, mul_prev=37, mul_cur=3)
     pair("bigram rows, embed of two tables + norms", lambda: residual_ops.embed(tok, tab, 1.0, w1, None, 1e-5, W, second=residual_ops.Second(tab, big(), w2)),
          (rows * W * 10, 0), "embed + norm", lambda: ops.embed_rmsnorm(tok, tab, w16, 1e-5), (rows * W * 6, 0))
     del gu, down, er, holder, xs
