@@ -38,10 +38,10 @@ struct TalkArgs {
   const int* block_table; const int* q_start; const int* q_lens; const int* ctx_lens;
   const float* talk;
   __nv_bfloat16* out;
-  // a slot is a tile of this round: weights [slot, H, 128, band * 64], m [slot, H, band, 2 halves, 128], z [slot, H, 128]
+  // a slot is one of the tiles worked on together: weights [slot, H, 128, band * 64], m [slot, H, band, 2 halves, 128], z [slot, H, 128]
   __nv_bfloat16* weights; float* m; float* z;
   int H, G, dk, dv, ldo, max_blocks, num_blocks, window, band;         // band: pages a tile's rows see at most
-  int tile0, tiles;                          // this round's tiles
+  int tile0, tiles;                          // the tiles worked on together
   float scale_log2, one;
   int* status;
 };
@@ -90,7 +90,7 @@ struct alignas(8) TalkWeightBars {
   float m[2][TK_ROWS], l[2][TK_ROWS];        // of the odd pages; two, so that a head's do not meet the next one's
 };
 
-// (sequence, tile of the round, head) number i
+// (sequence, tile, head) number i
 struct TalkItem {
   int b, tile, h;
   __device__ TalkItem(const TalkArgs& p, int i) { h = i % p.H; i /= p.H; tile = i % p.tiles; b = i / p.tiles; }
